@@ -617,17 +617,19 @@ __global__ void sum_rows_kernel(const float* __restrict__ v, long long n, float*
   if (threadIdx.x == 0) *out = accumulate ? *out + s : s;
 }
 
-// argmax over the first `vocab` columns of each row of bf16 logits; ties -> lowest index.
-__global__ void argmax_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int vocab,
-                              long long* __restrict__ out) {
+// argmax over the first `vocab` columns of each row of bf16 or fp32 logits; ties -> lowest index.
+__device__ __forceinline__ float logit_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float logit_f(float v) { return v; }
+template <typename T>
+__global__ void argmax_kernel(const T* __restrict__ logits, long long ld, int vocab, long long* __restrict__ out) {
   pdl_sync();
   __shared__ float sv[32];
   __shared__ int si[32];
-  const __nv_bfloat16* lr = logits + (long long)blockIdx.x * ld;
+  const T* lr = logits + (long long)blockIdx.x * ld;
   float best = -INFINITY;
   int bi = 0x7fffffff;
   for (int c = threadIdx.x; c < vocab; c += blockDim.x) {
-    const float f = __bfloat162float(lr[c]);
+    const float f = logit_f(lr[c]);
     if (f > best || (f == best && c < bi)) { best = f; bi = c; }
   }
 #pragma unroll
@@ -1004,9 +1006,11 @@ extern "C" int b200_xent(void* logits, const long long* targets, float* loss, fl
   CHECK_LAUNCH();
 }
 
-extern "C" int b200_argmax(const void* logits, long long rows, long long ld, int vocab, long long* out, cudaStream_t st) {
+extern "C" int b200_argmax(const void* logits, long long rows, long long ld, int vocab, int f32, long long* out,
+                           cudaStream_t st) {
   if (rows == 0) return 0;
-  launch_dep(argmax_kernel, (unsigned)rows, 256, 0, st, (const __nv_bfloat16*)logits, ld, vocab, out);
+  if (f32) launch_dep(argmax_kernel<float>, (unsigned)rows, 256, 0, st, (const float*)logits, ld, vocab, out);
+  else launch_dep(argmax_kernel<__nv_bfloat16>, (unsigned)rows, 256, 0, st, (const __nv_bfloat16*)logits, ld, vocab, out);
   CHECK_LAUNCH();
 }
 

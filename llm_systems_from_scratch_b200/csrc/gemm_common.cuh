@@ -17,6 +17,8 @@ enum GemmEpilogue : int {
   // Backward of h = silu(gate) * up fused into the GEMM that produces dh = acc (M x N): R holds gate | up
   // (M x 2N, bf16) and C (M x 2N, bf16) receives d(gate) | d(up).
   EPI_SWIGLU_BWD = 4,
+  // C = bf16(acc * sigmoid(R)): the output gate of an attention layer, R bf16 of C's shape.
+  EPI_BF16_GATE = 5,
   // Flag or-ed into the epilogue code by the caller (CTA-pair kernel): output columns from N up to the next 16-byte
   // boundary lie inside the row pitch and may be overwritten with zeros.
   EPI_PAD_WRITABLE = 0x100,
@@ -71,6 +73,14 @@ struct GemmParams {
   // B (the weights) does not depend on the kernel before this one: as a programmatic dependent the kernel requests
   // its first B tiles before it waits for that kernel, so the weights' DRAM latency overlaps the predecessor's tail.
   int b_early;
+  // Several problems in one launch (single-CTA kernel, K-major operands):
+  //   by rows    (`tile_group`): 128-row tile m multiplies with rows [group * group_rows, ...) of B, group = tile_group[m]
+  //              (a mixture of experts whose tokens are sorted by expert); a negative group skips the tile
+  //   by columns (`batch` > 1): problem g reads A columns from g * a_step, B rows from g * group_rows and writes C (and
+  //              reads R) columns from g * c_step (one small matrix per attention head)
+  const int* tile_group;
+  int group_rows;
+  int batch, a_step, c_step;
   int splits;
   float* ws;                  // splits * tiles partial tiles of BM x BN floats
   uint32_t* tile_counters;    // four per tile (one per 32-row quarter), zero between launches (the last warp resets its own)
@@ -111,8 +121,9 @@ __device__ __forceinline__ void epilogue_rope(const GemmParams& p, int row, int 
   }
 }
 
-// One 32-column chunk of one output row.
-__device__ __forceinline__ void epilogue_store(const GemmParams& p, int row, int col0, uint32_t (&acc)[32]) {
+// One 32-column chunk of one output row.  `coff` shifts the columns of C and R (one of several problems side by side).
+__device__ __forceinline__ void epilogue_store(const GemmParams& p, int row, int col0, uint32_t (&acc)[32],
+                                               int coff = 0) {
   if (row >= p.M) return;
   const int ncols = min(32, p.N - col0);
   if (ncols <= 0) return;
@@ -144,11 +155,17 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, int row, int
     }
     return;
   }
-  if (p.epi == EPI_BF16 || p.epi == EPI_BF16_RES) {
-    __nv_bfloat16* c = reinterpret_cast<__nv_bfloat16*>(p.C) + (long long)row * p.ldc + col0;
-    const bool vec_ok = (ncols == 32) && ((p.ldc & 7) == 0) && ((reinterpret_cast<uintptr_t>(p.C) & 15) == 0);
-    if (p.epi == EPI_BF16_RES) {
-      const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.R) + (long long)row * p.ldr + col0;
+  if (p.epi == EPI_BF16 || p.epi == EPI_BF16_RES || p.epi == EPI_BF16_GATE) {
+    __nv_bfloat16* c = reinterpret_cast<__nv_bfloat16*>(p.C) + (long long)row * p.ldc + coff + col0;
+    const bool vec_ok = (ncols == 32) && ((p.ldc & 7) == 0) && ((coff & 7) == 0) &&
+                        ((reinterpret_cast<uintptr_t>(p.C) & 15) == 0);
+    if (p.epi == EPI_BF16_GATE) {
+      const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.R) + (long long)row * p.ldr + coff + col0;
+#pragma unroll
+      for (int j = 0; j < 32; ++j)
+        if (j < ncols) c[j] = __float2bfloat16(__uint_as_float(acc[j]) / (1.f + __expf(-__bfloat162float(r[j]))));
+    } else if (p.epi == EPI_BF16_RES) {
+      const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.R) + (long long)row * p.ldr + coff + col0;
       const bool rvec = vec_ok && ((p.ldr & 7) == 0) && ((reinterpret_cast<uintptr_t>(p.R) & 15) == 0);
       if (rvec) {
 #pragma unroll
@@ -184,8 +201,9 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, int row, int
         if (j < ncols) c[j] = __float2bfloat16(__uint_as_float(acc[j]));
     }
   } else {
-    float* c = reinterpret_cast<float*>(p.C) + (long long)row * p.ldc + col0;
-    const bool vec_ok = (ncols == 32) && ((p.ldc & 3) == 0) && ((reinterpret_cast<uintptr_t>(p.C) & 15) == 0);
+    float* c = reinterpret_cast<float*>(p.C) + (long long)row * p.ldc + coff + col0;
+    const bool vec_ok = (ncols == 32) && ((p.ldc & 3) == 0) && ((coff & 3) == 0) &&
+                        ((reinterpret_cast<uintptr_t>(p.C) & 15) == 0);
     if (p.epi == EPI_F32) {
       if (vec_ok) {
 #pragma unroll

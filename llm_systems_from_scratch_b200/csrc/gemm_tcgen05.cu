@@ -27,7 +27,12 @@ struct GemmSmem {
   static constexpr int TOTAL = DATA_BYTES + BAR_BYTES + 1024;  // + alignment slack
 };
 
-template <int BN, bool A_MN, bool B_MN, int STAGES>
+// How a tile index maps onto the operands: one problem, one group of B rows per row tile, or one problem per head.
+enum GemmGroup : int { GROUP_NONE = 0, GROUP_ROWS = 1, GROUP_COLS = 2 };
+
+// SWIGLU (grouped kernels): B holds group_rows = 2 N rows per group, gate rows first; a BN-wide tile is BN / 2 gate rows
+// and the matching BN / 2 up rows, and the epilogue stores silu(gate) * up.
+template <int BN, bool A_MN, bool B_MN, int STAGES, int GROUP = GROUP_NONE, bool SWIGLU = false>
 __global__ void __launch_bounds__(192, 1)
 gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                          const GemmParams p) {
@@ -66,14 +71,16 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
       const int sp = p.splits > 1 ? p.splits : 1;
       const int nkb = (p.K + BK - 1) / BK;
       const int unit = blockIdx.x;
-      if (unit < p.num_m_tiles * p.num_n_tiles * sp) {
+      const int per_problem = p.num_m_tiles * p.num_n_tiles;
+      if (unit < per_problem * (GROUP == GROUP_COLS ? p.batch : 1) * sp) {
         const int tile = unit / sp, split = unit - tile * sp;
         const int kb_lo = split * nkb / sp, kb_hi = (split + 1) * nkb / sp;
         int m_blk, n_blk;
-        tile_coords(tile, p, m_blk, n_blk);
+        tile_coords(GROUP == GROUP_COLS ? tile % per_problem : tile, p, m_blk, n_blk);
+        const int brow = (GROUP == GROUP_COLS ? (tile / per_problem) * p.group_rows : 0) + n_blk * BN;
         for (int i = 0; i < STAGES && kb_lo + i < kb_hi; ++i) {
           mbar_expect_tx(&full_bar[i], S::A_BYTES + S::B_BYTES);
-          tma_load_2d(smem_b + i * S::B_BYTES, &tmB, &full_bar[i], (kb_lo + i) * BK, n_blk * BN);
+          tma_load_2d(smem_b + i * S::B_BYTES, &tmB, &full_bar[i], (kb_lo + i) * BK, brow);
         }
       }
     }
@@ -90,7 +97,9 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
   tc_fence_after();
   const uint32_t tmem_base = *tmem_holder;
 
-  const int num_tiles = p.num_m_tiles * p.num_n_tiles;
+  const int tiles_one = p.num_m_tiles * p.num_n_tiles;
+  const int num_tiles = GROUP == GROUP_COLS ? tiles_one * p.batch : tiles_one;
+  constexpr int BN_OUT = SWIGLU ? BN / 2 : BN;      // output columns of a tile
   const int num_kb = (p.K + BK - 1) / BK;
   // work unit = (tile, K slice); consecutive units are the slices of one tile, so they run at the same time on
   // neighbouring CTAs
@@ -108,8 +117,12 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
         const int tile = unit / splits, split = unit - tile * splits;
         const int kb_lo = split * num_kb / splits, kb_hi = (split + 1) * num_kb / splits;
         int m_blk, n_blk;
-        tile_coords(tile, p, m_blk, n_blk);
-        const int m0 = m_blk * BM, n0 = n_blk * BN;
+        tile_coords(GROUP == GROUP_COLS ? tile % tiles_one : tile, p, m_blk, n_blk);
+        int group = 0;
+        if (GROUP == GROUP_ROWS) group = p.tile_group[m_blk];
+        if (GROUP == GROUP_COLS) group = tile / tiles_one;
+        if (GROUP == GROUP_ROWS && group < 0) continue;
+        const int m0 = m_blk * BM, n0 = (GROUP != GROUP_NONE ? group * p.group_rows : 0) + n_blk * BN_OUT;
         if (unit != (int)blockIdx.x) early = 0;
         for (int kb = kb_lo; kb < kb_hi; ++kb) {
           const bool posted = kb - kb_lo < early;
@@ -126,11 +139,14 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
 #pragma unroll
             for (int j = 0; j < BM / 64; ++j) tma_load_2d(a_dst + j * 8192, &tmA, &full_bar[stage], m0 + j * 64, k0);
           } else {
-            tma_load_2d(a_dst, &tmA, &full_bar[stage], k0, m0);
+            tma_load_2d(a_dst, &tmA, &full_bar[stage], (GROUP == GROUP_COLS ? group * p.a_step : 0) + k0, m0);
           }
           if (B_MN) {
 #pragma unroll
             for (int j = 0; j < BN / 64; ++j) tma_load_2d(b_dst + j * 8192, &tmB, &full_bar[stage], n0 + j * 64, k0);
+          } else if (SWIGLU) {
+            tma_load_2d(b_dst, &tmB, &full_bar[stage], k0, n0);
+            tma_load_2d(b_dst + S::B_BYTES / 2, &tmB, &full_bar[stage], k0, n0 + p.N);
           } else if (!posted) {
             tma_load_2d(b_dst, &tmB, &full_bar[stage], k0, n0);
           }
@@ -150,8 +166,13 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
       uint32_t acc_phase[2] = {0, 0};
       int local = 0;
       bool ok = true;
-      for (int unit = blockIdx.x; unit < num_units && ok; unit += gridDim.x, ++local) {
+      for (int unit = blockIdx.x; unit < num_units && ok; unit += gridDim.x) {
         const int split = unit % splits;
+        if (GROUP == GROUP_ROWS) {
+          int m_blk, n_blk;
+          tile_coords(unit / splits, p, m_blk, n_blk);
+          if (p.tile_group[m_blk] < 0) continue;
+        }
         const int kb_lo = split * num_kb / splits, kb_hi = (split + 1) * num_kb / splits;
         const int acc = local & 1;
         if (!mbar_wait(&tmem_empty[acc], acc_phase[acc] ^ 1, abort_word)) {
@@ -186,6 +207,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
           }
         }
         if (ok) umma_commit(&tmem_full[acc]);  // accumulator complete
+        ++local;
       }
     }
   } else {
@@ -194,11 +216,14 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
     uint32_t acc_phase[2] = {0, 0};
     int local = 0;
     bool ok = true;
-    for (int unit = blockIdx.x; unit < num_units && ok; unit += gridDim.x, ++local) {
+    for (int unit = blockIdx.x; unit < num_units && ok; unit += gridDim.x) {
       const int tile = unit / splits;
       int m_blk, n_blk;
-      tile_coords(tile, p, m_blk, n_blk);
+      tile_coords(GROUP == GROUP_COLS ? tile % tiles_one : tile, p, m_blk, n_blk);
+      if (GROUP == GROUP_ROWS && p.tile_group[m_blk] < 0) continue;
+      const int coff = GROUP == GROUP_COLS ? (tile / tiles_one) * p.c_step : 0;
       const int acc = local & 1;
+      ++local;
       if (!mbar_wait(&tmem_full[acc], acc_phase[acc], abort_word)) {
         if (lane == 0) report(p, abort_word, ERR_WAIT_TMEM_FULL);
         ok = false;
@@ -208,8 +233,27 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
       tc_fence_after();
       const int row_in_tile = quarter * 32 + lane;
       const int row = m_blk * BM + row_in_tile;
-      const int n0 = n_blk * BN;
+      const int n0 = n_blk * BN_OUT;
       const uint32_t taddr = tmem_base + (uint32_t(quarter * 32) << 16) + acc * BN;
+      if (SWIGLU) {
+#pragma unroll 1
+        for (int c = 0; c < BN_OUT / 32; ++c) {
+          if (n0 + c * 32 >= p.N) break;
+          uint32_t r[32], u[32];
+          tmem_ld_32x32(taddr + c * 32, r);
+          tmem_ld_32x32(taddr + BN_OUT + c * 32, u);
+          tmem_ld_wait();
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float g = __uint_as_float(r[j]);
+            r[j] = __float_as_uint(g / (1.f + __expf(-g)) * __uint_as_float(u[j]));
+          }
+          epilogue_store(p, row, n0 + c * 32, r);
+        }
+        tc_fence_before();
+        mbar_arrive(&tmem_empty[acc]);
+        continue;
+      }
       if (splits == 1) {
 #pragma unroll 1
         for (int c = 0; c < BN / 32; ++c) {
@@ -217,7 +261,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
           uint32_t r[32];
           tmem_ld_32x32(taddr + c * 32, r);
           tmem_ld_wait();
-          epilogue_store(p, row, n0 + c * 32, r);
+          epilogue_store(p, row, n0 + c * 32, r, coff);
         }
         tc_fence_before();
         mbar_arrive(&tmem_empty[acc]);
@@ -371,20 +415,21 @@ static int num_sms() {
   return g_num_sms;
 }
 
-template <int BN, bool A_MN, bool B_MN>
+template <int BN, bool A_MN, bool B_MN, int GROUP = GROUP_NONE, bool SWIGLU = false>
 static int launch_gemm(const CUtensorMap& tmA, const CUtensorMap& tmB, GemmParams p, int max_ctas, cudaStream_t stream) {
   constexpr int STAGES = (BN == 256) ? 4 : (BN == 128 ? 6 : 8);
   using S = GemmSmem<BN, STAGES>;
-  auto kern = gemm_bf16_tcgen05_kernel<BN, A_MN, B_MN, STAGES>;
+  auto kern = gemm_bf16_tcgen05_kernel<BN, A_MN, B_MN, STAGES, GROUP, SWIGLU>;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S::TOTAL) != cudaSuccess) return -3;
     configured = true;
   }
   p.num_m_tiles = (p.M + BM - 1) / BM;
-  p.num_n_tiles = (p.N + BN - 1) / BN;
+  constexpr int BN_OUT = SWIGLU ? BN / 2 : BN;
+  p.num_n_tiles = (p.N + BN_OUT - 1) / BN_OUT;
   p.group_m = 16;
-  const int units = p.num_m_tiles * p.num_n_tiles * (p.splits > 1 ? p.splits : 1);
+  const int units = p.num_m_tiles * p.num_n_tiles * (p.splits > 1 ? p.splits : 1) * (GROUP == GROUP_COLS ? p.batch : 1);
   int grid = num_sms();
   if (max_ctas > 0 && max_ctas < grid) grid = max_ctas;
   if (units < grid) grid = units;
@@ -468,6 +513,7 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, const void* R, 
   p.swiglu_f = 0; p.H = nullptr; p.ldh = 0;
   p.splits = splits > 1 ? splits : 1; p.ws = ws; p.tile_counters = tile_counters;
   p.b_early = b_early;
+  p.tile_group = nullptr; p.group_rows = 0; p.batch = 1; p.a_step = p.c_step = 0;
 
 #define DISPATCH(BN_)                                                                    \
   if (a_mn && b_mn) return launch_gemm<BN_, true, true>(tmA, tmB, p, max_ctas, stream);   \
@@ -543,4 +589,71 @@ extern "C" int b200_gemm_bf16_splitk(const void* A, const void* B, void* C, cons
     return gemm_bf16_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, 0, 0, epi, 0, 0, 1, nullptr, nullptr, status, stream);
   return gemm_bf16_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, 0, 0, epi, bn, 0, splits, ws, tile_counters, status,
                         stream);
+}
+
+// Several GEMMs in one launch, K-major bf16 operands (see GemmParams):
+//   tile_group != null: A is (M, K) with M a multiple of 128, its 128-row tiles belong to the groups in `tile_group`
+//     (device int per tile, -1 = skip); B is (n_groups * group_rows, K).  With `swiglu` group_rows == 2 N and the output is
+//     silu(gate) * up, otherwise group_rows == N.
+//   tile_group == null: `batch` problems side by side: problem g multiplies A[:, g * a_step : g * a_step + K] with
+//     B[g * group_rows : g * group_rows + N, :] into C[:, g * c_step : g * c_step + N].  a_step must be a multiple of 8.
+// Columns of A past a problem's K (up to the next multiple of 64) are multiplied with zeros, so they must be finite.
+extern "C" int b200_gemm_bf16_grouped(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
+                                      long long lda, long long ldb, long long ldc, long long ldr, const int* tile_group,
+                                      int n_groups, int group_rows, int batch, int a_step, int c_step, int swiglu,
+                                      int epi, uint32_t* status, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15) || (lda & 7) || (ldb & 7))
+    return -10;
+  const bool rows = tile_group != nullptr;
+  const int b_early = (!rows && (epi & EPI_B_STABLE)) ? 1 : 0;
+  epi &= ~EPI_B_STABLE;
+  if (epi != EPI_BF16 && epi != EPI_F32 && epi != EPI_BF16_GATE) return -11;
+  if (epi == EPI_BF16_GATE && (R == nullptr || rows)) return -11;
+  if (rows && ((M % BM) || n_groups <= 0 || group_rows != (swiglu ? 2 * N : N))) return -12;
+  if (!rows && (swiglu || batch <= 0 || (a_step & 7) || group_rows < N)) return -12;
+  const int sms = num_sms();
+  const long long mt = (M + BM - 1) / BM, problems = rows ? 1 : batch;
+  int bn = 64;
+  long long best = -1;
+  const int cand[3] = {64, 128, 256};
+  for (int ci = 0; ci < 3; ++ci) {
+    const int out = swiglu ? cand[ci] / 2 : cand[ci];
+    const long long tiles = mt * problems * ((N + out - 1) / out);
+    const long long cost = ((tiles + sms - 1) / sms) * (BM + cand[ci]);
+    if (best < 0 || cost < best) { best = cost; bn = cand[ci]; }
+  }
+  CUtensorMap tmA, tmB;
+  const uint64_t a_cols = rows ? (uint64_t)K : (uint64_t)(batch - 1) * a_step + K;
+  const uint64_t b_rows = rows ? (uint64_t)n_groups * group_rows : (uint64_t)batch * group_rows;
+  int rc = make_tmap_bf16_2d(&tmA, A, (uint64_t)M, a_cols, (uint64_t)lda, 64, BM);
+  if (rc) return -20 + rc;
+  rc = make_tmap_bf16_2d(&tmB, B, b_rows, (uint64_t)K, (uint64_t)ldb, 64, swiglu ? bn / 2 : bn);
+  if (rc) return -30 + rc;
+  GemmParams p;
+  p.M = M; p.N = N; p.K = K;
+  p.C = C; p.ldc = ldc; p.R = R; p.ldr = ldr; p.epi = epi; p.status = status;
+  p.num_m_tiles = p.num_n_tiles = p.group_m = 0;
+  p.gather.dst = nullptr; p.gather.done = nullptr; p.gather.shard_vec = 0; p.gather.world = 0; p.gather.rank = 0;
+  p.reduce.n = 0;
+  p.tma_store = 0;
+  p.wait_counter = nullptr; p.wait_value = 0; p.wait_limit_ns = 0;
+  p.rope_cs = nullptr; p.rope_seq = p.rope_d = p.rope_dh = p.rope_ctx = 0;
+  p.swiglu_f = 0; p.H = nullptr; p.ldh = 0;
+  p.splits = 1; p.ws = nullptr; p.tile_counters = nullptr;
+  p.b_early = b_early;
+  p.tile_group = tile_group; p.group_rows = group_rows; p.batch = rows ? 1 : batch; p.a_step = a_step; p.c_step = c_step;
+  if (rows && swiglu) {
+    if (bn == 256) return launch_gemm<256, false, false, GROUP_ROWS, true>(tmA, tmB, p, 0, stream);
+    if (bn == 128) return launch_gemm<128, false, false, GROUP_ROWS, true>(tmA, tmB, p, 0, stream);
+    return launch_gemm<64, false, false, GROUP_ROWS, true>(tmA, tmB, p, 0, stream);
+  }
+  if (rows) {
+    if (bn == 256) return launch_gemm<256, false, false, GROUP_ROWS>(tmA, tmB, p, 0, stream);
+    if (bn == 128) return launch_gemm<128, false, false, GROUP_ROWS>(tmA, tmB, p, 0, stream);
+    return launch_gemm<64, false, false, GROUP_ROWS>(tmA, tmB, p, 0, stream);
+  }
+  if (bn == 256) return launch_gemm<256, false, false, GROUP_COLS>(tmA, tmB, p, 0, stream);
+  if (bn == 128) return launch_gemm<128, false, false, GROUP_COLS>(tmA, tmB, p, 0, stream);
+  return launch_gemm<64, false, false, GROUP_COLS>(tmA, tmB, p, 0, stream);
 }

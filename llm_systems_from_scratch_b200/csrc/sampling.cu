@@ -4,9 +4,9 @@
 // torch.multinomial) without materialising probabilities or sorting the vocabulary.
 //
 // One block per row:
-//   1. top-k threshold by radix select on the order-preserving 16-bit key of the bf16 logit: a 256-bin
-//      histogram of the high byte, then of the low byte inside the selected bin.  Every logit >= the k-th
-//      largest is kept (ties included, like `logits < kth -> -inf`).
+//   1. top-k threshold by radix select on the order-preserving key of the logit (16 bits for bf16, 32 for fp32): a
+//      256-bin histogram of the highest byte, then of each lower byte inside the bin selected so far.  Every logit >=
+//      the k-th largest is kept (ties included, like `logits < kth -> -inf`).
 //   2. row maximum and sum of exp((x - max) / T) over the kept logits (fp32).
 //   3. inverse-CDF draw with the caller's uniform u in [0, 1): each thread owns a contiguous slice of the
 //      vocabulary, a block scan of the slice sums finds the slice, a serial walk finds the token.
@@ -16,9 +16,19 @@ namespace b200 {
 
 constexpr int SAMPLE_THREADS = 1024;
 
-__device__ __forceinline__ uint32_t bf16_key(uint16_t bits) {   // larger float <=> larger key
-  return (bits & 0x8000u) ? (~bits & 0xffffu) : (bits | 0x8000u);
-}
+// Order-preserving key of a logit (larger value <=> larger key) and the value itself, from the raw bits.
+struct Bf16Logit {
+  using Bits = uint16_t;
+  static constexpr int BYTES = 2;
+  static __device__ __forceinline__ uint32_t key(uint16_t b) { return (b & 0x8000u) ? (~b & 0xffffu) : (b | 0x8000u); }
+  static __device__ __forceinline__ float value(uint16_t b) { return __uint_as_float((uint32_t)b << 16); }
+};
+struct F32Logit {
+  using Bits = uint32_t;
+  static constexpr int BYTES = 4;
+  static __device__ __forceinline__ uint32_t key(uint32_t b) { return (b & 0x80000000u) ? ~b : (b | 0x80000000u); }
+  static __device__ __forceinline__ float value(uint32_t b) { return __uint_as_float(b); }
+};
 
 __device__ __forceinline__ float block_reduce(float v, float* red, bool is_max) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -54,36 +64,38 @@ __device__ __forceinline__ void select_bin(const uint32_t* hist, uint32_t need, 
   __syncthreads();
 }
 
+template <typename L>
 __global__ void __launch_bounds__(SAMPLE_THREADS)
-sample_topk_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int vocab, const float* __restrict__ uniforms,
+sample_topk_kernel(const typename L::Bits* __restrict__ logits, long long ld, int vocab, const float* __restrict__ uniforms,
                    float inv_temperature, int top_k, long long* __restrict__ out) {
   __shared__ uint32_t hist[256];
   __shared__ uint32_t sel[2];
   __shared__ float red[32];
   __shared__ float warp_sums[32];
   __shared__ int result;
-  const uint16_t* row = reinterpret_cast<const uint16_t*>(logits) + (long long)blockIdx.x * ld;
+  using Bits = typename L::Bits;
+  const Bits* row = logits + (long long)blockIdx.x * ld;
   const int tid = threadIdx.x;
 
   // ---- 1. threshold key: all logits with key >= thr are kept
   uint32_t thr = 0;
   if (top_k > 0 && top_k < vocab) {
-    if (tid < 256) hist[tid] = 0;
-    __syncthreads();
-    for (int i = tid; i < vocab; i += SAMPLE_THREADS) atomicAdd(&hist[bf16_key(row[i]) >> 8], 1u);
-    __syncthreads();
-    select_bin(hist, (uint32_t)top_k, sel);
-    const uint32_t hi = sel[0], need_lo = (uint32_t)top_k - sel[1];
-    __syncthreads();
-    if (tid < 256) hist[tid] = 0;
-    __syncthreads();
-    for (int i = tid; i < vocab; i += SAMPLE_THREADS) {
-      const uint32_t key = bf16_key(row[i]);
-      if ((key >> 8) == hi) atomicAdd(&hist[key & 0xff], 1u);
+    uint32_t need = (uint32_t)top_k;                     // rank of the threshold inside the bins selected so far
+#pragma unroll
+    for (int byte = L::BYTES - 1; byte >= 0; --byte) {
+      if (tid < 256) hist[tid] = 0;
+      __syncthreads();
+      for (int i = tid; i < vocab; i += SAMPLE_THREADS) {
+        const uint32_t key = L::key(row[i]);
+        // the higher bytes must equal the threshold's (there are none above the first)
+        if (byte == L::BYTES - 1 || (key >> (8 * byte + 8)) == thr) atomicAdd(&hist[(key >> (8 * byte)) & 0xff], 1u);
+      }
+      __syncthreads();
+      select_bin(hist, need, sel);
+      need -= sel[1];
+      thr = (thr << 8) | sel[0];
+      __syncthreads();
     }
-    __syncthreads();
-    select_bin(hist, need_lo, sel);
-    thr = (hi << 8) | sel[0];
   }
 
   // ---- 2. maximum and normaliser over the kept logits; thread t owns tokens [t*per, (t+1)*per)
@@ -91,15 +103,15 @@ sample_topk_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int v
   const int i0 = min(tid * per, vocab), i1 = min(i0 + per, vocab);
   float mx = -INFINITY;
   for (int i = i0; i < i1; ++i) {
-    const uint16_t b = row[i];
-    if (bf16_key(b) >= thr) mx = fmaxf(mx, __uint_as_float((uint32_t)b << 16));
+    const Bits b = row[i];
+    if (L::key(b) >= thr) mx = fmaxf(mx, L::value(b));
   }
   mx = block_reduce(mx, red, true);
   const float c = inv_temperature * 1.4426950408889634f;
   float part = 0.f;
   for (int i = i0; i < i1; ++i) {
-    const uint16_t b = row[i];
-    if (bf16_key(b) >= thr) part += exp2f((__uint_as_float((uint32_t)b << 16) - mx) * c);
+    const Bits b = row[i];
+    if (L::key(b) >= thr) part += exp2f((L::value(b) - mx) * c);
   }
   const float total = block_reduce(part, red, false);
 
@@ -124,9 +136,9 @@ sample_topk_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int v
     float run = before;
     int pick = -1;
     for (int i = i0; i < i1; ++i) {
-      const uint16_t b = row[i];
-      if (bf16_key(b) < thr) continue;
-      run += exp2f((__uint_as_float((uint32_t)b << 16) - mx) * c);
+      const Bits b = row[i];
+      if (L::key(b) < thr) continue;
+      run += exp2f((L::value(b) - mx) * c);
       pick = i;
       if (target < run) break;
     }
@@ -137,7 +149,7 @@ sample_topk_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int v
     // the target fell on or past the total through rounding: take the last kept token
     int last = -1;
     for (int i = i1 - 1; i >= i0; --i)
-      if (bf16_key(row[i]) >= thr) { last = i; break; }
+      if (L::key(row[i]) >= thr) { last = i; break; }
     if (last >= 0) atomicMax(&result, last);
     __syncthreads();
   }
@@ -148,13 +160,17 @@ sample_topk_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int v
 
 using namespace b200;
 
-// logits: (rows, ld) bf16 with `vocab` valid columns; uniforms: (rows) fp32 in [0, 1); out: (rows) int64.
+// logits: (rows, ld) bf16 (or fp32 with f32 != 0) with `vocab` valid columns; uniforms: (rows) fp32 in [0, 1); out: (rows) int64.
 // temperature > 0; top_k <= 0 or >= vocab keeps the whole vocabulary.
-extern "C" int b200_sample_topk(const void* logits, long long rows, long long ld, int vocab, const float* uniforms,
-                                float temperature, int top_k, long long* out, cudaStream_t st) {
+extern "C" int b200_sample_topk(const void* logits, long long rows, long long ld, int vocab, int f32,
+                                const float* uniforms, float temperature, int top_k, long long* out, cudaStream_t st) {
   if (!(temperature > 0.f) || vocab <= 0 || ld < vocab) return -10;
   if (rows == 0) return 0;
-  sample_topk_kernel<<<(unsigned)rows, SAMPLE_THREADS, 0, st>>>((const __nv_bfloat16*)logits, ld, vocab, uniforms,
-                                                              1.f / temperature, top_k, out);
+  if (f32)
+    sample_topk_kernel<F32Logit><<<(unsigned)rows, SAMPLE_THREADS, 0, st>>>((const uint32_t*)logits, ld, vocab, uniforms,
+                                                                            1.f / temperature, top_k, out);
+  else
+    sample_topk_kernel<Bf16Logit><<<(unsigned)rows, SAMPLE_THREADS, 0, st>>>((const uint16_t*)logits, ld, vocab, uniforms,
+                                                                             1.f / temperature, top_k, out);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -1,0 +1,169 @@
+"""Sublayers of layered decoders: token mixers and feed-forwards that a model puts together by configuration.
+
+Each class takes its sizes and constants as arguments, packs its weights for the kernels (matrices that read the same
+input become one product; heads are padded to what the kernels tile by) and runs one step of the engine:
+
+* a mixer is called with the normed rows ``h``, the fp32 residual stream ``x`` (it adds its output there in the epilogue
+  of its output projection), the ``StepBatch`` and its own part of the cache; ``cache_spec()`` says what that is
+* a feed-forward returns outputs that the next pass over the residual stream adds (``ops.mixer_ops.residual_norm``)
+
+``get(name)`` gives a weight in its stored layout ([out, in])."""
+from __future__ import annotations
+
+import torch
+
+from ..ops import mixer_ops as mo
+from ..serving.kv_cache import PagedSpec, StateSpec
+
+
+def _head_pad(w, heads: int, rows: int, to: int):
+    """[heads * rows, in] -> [heads * to, in] with zero rows after each head's."""
+    if rows == to:
+        return w
+    out = torch.zeros((heads, to, w.shape[1]), dtype=w.dtype)
+    out[:, :rows] = w.view(heads, rows, -1)
+    return out.view(heads * to, -1)
+
+
+def _expect(name: str, t, *shape):
+    if tuple(t.shape) != shape:
+        raise ValueError(f"{name} has shape {tuple(t.shape)}, expected {shape}")
+    return t
+
+
+class LatentAttention:
+    """Attention whose keys and values are linear images of one cached latent per token; no positions.
+
+    q = W_uq rms_norm(W_dq h), c = rms_norm(W_dkv h), k_h = W_uk,h c, v_h = W_uv,h c, softmax(scale q.k) over the last
+    ``window`` positions (0 = all), heads multiplied by sigmoid(W_g h), then W_o.  Only c is cached."""
+
+    def __init__(self, get, width: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, window: int,
+                 eps: float, dtype, device):
+        self.heads, self.dim, self.vdim, self.q_rank, self.kv_rank = heads, dim, vdim, q_rank, kv_rank
+        self.scale, self.window, self.eps = float(scale), int(window), float(eps)
+        self.latent = mo.pitch(kv_rank)                  # cached vector, zero padded
+        w = lambda name, *shape: _expect(name, get(name), *shape)
+        dq, dkv = w("dq", q_rank, width), w("dkv", kv_rank, width)
+        uq, uk = w("uq", heads * dim, q_rank), w("uk", heads * dim, kv_rank)
+        uv, g = w("uv", heads * vdim, kv_rank), w("g", heads * vdim, width)
+        o = w("o", width, heads * vdim)
+        pack = lambda t: mo.padded_weight(t, dtype, device)
+        # the tensor-core prefill takes heads of 64 or 128; elsewhere a head only has to start on a 16-byte boundary
+        self.flash_dim = 0 if max(dim, vdim) > 128 else (64 if max(dim, vdim) <= 64 else 128)
+        if dtype != torch.bfloat16 or torch.device(device).type != "cuda":
+            self.flash_dim = 0
+        self.qdim = self.flash_dim or mo.pitch(dim)
+        self.w_in = pack(torch.cat((dq, dkv, g)))
+        self.w_uq = pack(_head_pad(uq, heads, dim, self.qdim))
+        ukt = torch.zeros((heads, self.latent, self.qdim), dtype=uk.dtype)        # q_h -> latent space: W_uk,h^T
+        ukt[:, :kv_rank, :dim] = uk.view(heads, dim, kv_rank).transpose(1, 2)
+        self.w_ukt = pack(ukt.reshape(heads * self.latent, self.qdim))
+        uvp = torch.zeros((heads * vdim, self.latent), dtype=uv.dtype)
+        uvp[:, :kv_rank] = uv
+        self.w_uv = pack(uvp)
+        if self.flash_dim:
+            kv = torch.zeros((2 * heads * self.flash_dim, self.latent), dtype=uk.dtype)
+            kv[:heads * self.flash_dim, :kv_rank] = _head_pad(uk, heads, dim, self.flash_dim)
+            kv[heads * self.flash_dim:, :kv_rank] = _head_pad(uv, heads, vdim, self.flash_dim)
+            self.w_ukv = pack(kv)
+        self.w_o = pack(o)
+        self.n_q = w("dq.norm", q_rank).to(device=device, dtype=dtype).contiguous()
+        self.n_kv = w("dkv.norm", kv_rank).to(device=device, dtype=dtype).contiguous()
+
+    def cache_spec(self):
+        return PagedSpec(self.latent)
+
+    def __call__(self, h, x, batch, cache):
+        heads, n = self.heads, batch.n_single
+        proj = mo.linear(h, self.w_in)
+        cq = mo.latent_norm_append(proj, self.n_q, self.n_kv, self.eps, cache, batch.slots)
+        q = mo.linear(cq, self.w_uq)
+        gate = proj[:, self.q_rank + self.kv_rank:]
+        o = mo.rows_buffer(h.shape[0], heads * self.vdim, h.dtype, h.device)
+        if n:
+            self._rows(q[:n], gate[:n], o[:n], batch, cache, slice(0, n))
+        if batch.n_rows > n:
+            self._rows(q[n:], gate[n:], o[n:], batch, cache, slice(n, batch.n_rows))
+        mo.linear(o, self.w_o, out=x, accumulate=True)
+
+    def _rows(self, q, gate, o, batch, cache, rows: slice):
+        ql = mo.gemm_heads(q, self.w_ukt, self.heads, self.qdim, self.latent)
+        ol = mo.latent_attention_rows(ql, cache, batch.row_seq[rows], batch.positions[rows], batch.slots[rows], batch.tables,
+                                      self.heads, self.window, self.scale)
+        mo.gemm_heads(ol, self.w_uv, self.heads, self.latent, self.vdim, out=o, gate=gate)
+
+
+class Retention:
+    """Linear attention with a fixed decay per head, rotary q and k (rotate-half over the first ``rot_dims`` dimensions), no
+    softmax; heads are divided by their root mean square, multiplied by silu(W_g h), then W_o.  The state is fp32."""
+
+    def __init__(self, get, width: int, heads: int, dim: int, vdim: int, decay, rot_dims: int, eps: float, rope, dtype, device):
+        self.heads, self.dim, self.vdim, self.rot, self.eps = heads, dim, vdim, int(rot_dims), float(eps)
+        if len(decay) != heads:
+            raise ValueError(f"{len(decay)} decays for {heads} heads")
+        if self.rot % 2 or self.rot > dim:
+            raise ValueError("the rotated dimensions must be even in number and fit the head")
+        w = lambda name, *shape: _expect(name, get(name), *shape)
+        self.w_in = mo.padded_weight(torch.cat((w("q", heads * dim, width), w("k", heads * dim, width),
+                                                w("v", heads * vdim, width), w("g", heads * vdim, width))), dtype, device)
+        self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
+        self.decay = torch.tensor([float(d) for d in decay], dtype=torch.float32, device=device)
+        self.rope = rope                       # RotaryTable of the model's base and dims, None without rotation
+
+    def cache_spec(self):
+        return StateSpec((self.heads, self.dim, self.vdim))
+
+    def __call__(self, h, x, batch, state):
+        n = batch.n_single
+        proj = mo.linear(h, self.w_in)
+        y = mo.rows_buffer(h.shape[0], self.heads * self.vdim, h.dtype, h.device)
+        table = self.rope.table if self.rope is not None else None
+        run = lambda rows, slots, cu, spans: mo.retention(
+            proj[rows], state, slots, cu, spans, batch.positions[rows], table, self.decay, self.heads, self.dim, self.vdim,
+            self.rot, self.eps, y[rows])
+        if n:
+            run(slice(0, n), batch.state_slots[:n], None, [(i, i + 1) for i in range(n)] if not h.is_cuda else None)
+        if batch.n_rows > n:
+            run(slice(n, batch.n_rows), batch.state_slots[n:], batch.cu, batch.spans)
+        mo.linear(y, self.w_o, out=x, accumulate=True)
+
+
+class RotaryTable:
+    """cos and sin of position * base^(-2 i / dims), rounded once from double precision: (2, positions, dims / 2) fp32.
+    One per (base, dims), shared by the layers that use it; the engine sizes it to its longest context."""
+
+    def __init__(self, base: float, dims: int, device):
+        self.base, self.dims, self.device = float(base), int(dims), device
+        self.table = None
+
+    def resize(self, positions: int):
+        if self.table is None or self.table.shape[1] != positions:
+            freq = self.base ** (-2.0 * torch.arange(self.dims // 2, dtype=torch.float64) / self.dims)
+            angle = torch.outer(torch.arange(positions, dtype=torch.float64), freq)
+            self.table = torch.stack((angle.cos(), angle.sin())).float().contiguous().to(self.device)
+
+
+class TableExperts:
+    """SwiGLU experts chosen by a table row per token id, each with weight 1 / top; no router network.
+
+    A step's rows are sorted by expert into 128-row tiles (``ops.mixer_ops.moe_plan``, once per step for all layers); the
+    pass that norms a row also writes it where its experts read it, and the pass over the residual stream that follows
+    adds the outputs up."""
+
+    def __init__(self, get, width: int, ff: int, experts: int, top: int, vocab: int, dtype, device):
+        self.ff, self.experts, self.top, self.width = ff, experts, top, width
+        self.table = _expect("table", get("table"), vocab, top).to(device=device, dtype=torch.int32).contiguous()
+        if int(self.table.min()) < 0 or int(self.table.max()) >= experts:
+            raise ValueError("the expert table names an expert that does not exist")
+        gu = torch.cat([_expect(f"e{e}.{k}", get(f"e{e}.{k}"), ff, width) for e in range(experts) for k in ("gate", "up")])
+        self.w_gu = mo.padded_weight(gu, dtype, device)                            # (experts * 2 ff, width), gate first
+        self.w_down = mo.padded_weight(torch.cat([_expect(f"e{e}.down", get(f"e{e}.down"), width, ff)
+                                                  for e in range(experts)]), dtype, device)
+
+    def rows(self, tokens: int) -> int:
+        """Rows of the expert-sorted buffers for a step of ``tokens`` rows."""
+        return mo.plan_tiles(tokens, self.experts, self.top) * mo.TILE
+
+    def __call__(self, xg, tile_group):
+        hidden = mo.gemm_rows(xg, self.w_gu, tile_group, self.ff, swiglu=True)
+        return mo.gemm_rows(hidden, self.w_down, tile_group, self.width, swiglu=False)

@@ -24,6 +24,7 @@ from __future__ import annotations
 import json
 import logging
 import math
+import os
 
 import torch
 from torch import Tensor, nn
@@ -212,6 +213,8 @@ class TransformerBlock(nn.Module):
 
 
 class TransformerLM(nn.Module):
+    GPU_DTYPES = (torch.bfloat16,)          # what the kernels that serve it compute in
+
     def __init__(self, vocab_size: int, context_length: int, d_model: int, num_layers: int, num_heads: int,
                  d_ff: int, rope_theta: float, use_flash_attn: bool = False, use_custom_triton: bool = False):
         self.config = dict(vocab_size=vocab_size, context_length=context_length, d_model=d_model,
@@ -400,10 +403,27 @@ class TransformerLM(nn.Module):
             new.append(nxt)
         return torch.cat(new, dim=-1) if new else ids[:, :0]
 
+    def serving_backend(self):
+        from ..serving.backends import TransformerBackend
+        return TransformerBackend(self)
+
+    @classmethod
+    def from_folder(cls, folder: str, dtype=torch.bfloat16, device="cuda") -> "TransformerLM":
+        """Load ``ckpt_final.pt`` (or ``model.pt``) beside the folder's config.json (or model_config.json)."""
+        if dtype != torch.bfloat16 and torch.device(device).type == "cuda":
+            raise ValueError("TransformerLM is served in bfloat16")
+        find = lambda names: next((os.path.join(folder, n) for n in names if os.path.exists(os.path.join(folder, n))), None)
+        config, weights = find(("config.json", "model_config.json")), find(("ckpt_final.pt", "model.pt"))
+        if config is None or weights is None:
+            raise FileNotFoundError(f"{folder} needs a configuration and ckpt_final.pt or model.pt")
+        model = cls.from_pretrained(config, weights).to(device).eval()
+        model.use_custom_triton = True
+        return model
+
     @classmethod
     def from_pretrained(cls, config_path: str, checkpoint_path: str) -> "TransformerLM":
         with open(config_path) as f:
-            model = cls(**json.load(f))
+            model = cls(**{k: v for k, v in json.load(f).items() if k != "architecture"})
         state = torch.load(checkpoint_path, map_location="cpu")
         state = state.get("model", state) if isinstance(state, dict) else state
         state = {(k[len("_orig_mod."):] if k.startswith("_orig_mod.") else k): v for k, v in state.items()}

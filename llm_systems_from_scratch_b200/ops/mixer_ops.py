@@ -1,0 +1,270 @@
+"""Ops of the layered decoders (mixers, token-table experts, 32-bit residual stream): CUDA tensors go to the sm_100a
+kernels, CPU tensors to the PyTorch statements in ``mixer_torch``.  Activations are bf16 (serving) or fp32 (a model run
+in 32-bit); the residual stream, scores, norms and recurrent states are fp32 either way.
+
+Matrices whose rows are read by TMA have a row pitch that is a multiple of 8 elements (``rows_buffer``,
+``padded_weight``), so no width has to be."""
+from __future__ import annotations
+
+import ctypes
+
+import torch
+
+from . import mixer_torch, native
+from .native import _check, _ptr, _req, _stream
+
+TILE = 128                 # rows of an expert tile (csrc/mixer_elementwise.cu: PLAN_TILE)
+_declared = False
+
+
+def _lib():
+    global _declared
+    lib = native.load()
+    if not _declared:
+        P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
+        for name, args in {
+            "b200_residual_norm": [P, P, I, P, P, P, P, I, I, F, L, P, P, L, F, P, P, I, I, L, I, I, I, I, P, P],
+            "b200_moe_plan": [P, P, I, I, I, P, P, P, P, L, P, I, P, P],
+            "b200_moe_plan_layers": [],
+            "b200_silu_mul_any": [P, P, L, I, L, L, I, P],
+            "b200_gate_sigmoid": [P, P, L, I, L, L, I, P],
+            "b200_gemm_f32": [P, P, P, I, I, I, L, L, L, I, P, I, I, I, I, P],
+            "b200_gemm_bf16_grouped": [P, P, P, P, I, I, I, L, L, L, L, P, I, I, I, I, I, I, I, P, P],
+            "b200_latent_norm_append": [P, L, P, P, P, L, P, P, I, I, I, I, L, F, I, P, P],
+            "b200_latent_gather": [P, P, P, P, P, I, I, I, I, I, I, P, P],
+            "b200_latent_attn_rows": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
+            "b200_retention_recurrent": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
+        }.items():
+            fn = getattr(lib, name)
+            fn.argtypes, fn.restype = args, ctypes.c_int
+        _declared = True
+    return lib
+
+
+def _f32(t) -> int:
+    _req(t.dtype in (torch.float32, torch.bfloat16), "activations must be bf16 or fp32")
+    return int(t.dtype == torch.float32)
+
+
+def pitch(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+def rows_buffer(rows: int, n: int, dtype, device):
+    """Uninitialised (rows, n) matrix with an 8-element row pitch."""
+    return torch.empty((rows, pitch(n)), dtype=dtype, device=device)[:, :n]
+
+
+def padded_weight(w, dtype, device):
+    """(out, in) weight copied to ``device`` with zeros up to an 8-element row pitch."""
+    buf = torch.zeros((w.shape[0], pitch(w.shape[1])), dtype=dtype, device=device)
+    buf[:, :w.shape[1]] = w.to(device=device, dtype=dtype)
+    return buf[:, :w.shape[1]]
+
+
+# --------------------------------------------------------------------------------- matrix products
+def linear(a, w, out=None, accumulate=False, out_dtype=None):
+    """a (R, K) @ w (N, K)^T.  ``accumulate`` adds to an fp32 ``out``."""
+    if out is None:
+        out = rows_buffer(a.shape[0], w.shape[0], out_dtype or a.dtype, a.device)
+    if not a.is_cuda:
+        r = a.float() @ w.float().t()
+        out.copy_(out + r if accumulate else r)
+        return out
+    if a.dtype == torch.bfloat16:
+        return native.gemm(a, w, "nt", out=out, accumulate=accumulate, b_stable=True)
+    _req(out.dtype == torch.float32 and w.dtype == torch.float32 and a.shape[1] == w.shape[1], "fp32 product of fp32 operands")
+    _check(_lib().b200_gemm_f32(_ptr(a), _ptr(w), _ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0), w.stride(0),
+                                out.stride(0), int(accumulate), None, 0, 1, 0, 0, _stream()), "gemm_f32")
+    return out
+
+
+def gemm_rows(a, w, tile_group, n: int, swiglu: bool):
+    """Every 128-row tile t of a (P, K) times the rows of w that belong to group tile_group[t] (negative: skipped, the
+    rows of the result stay undefined).  ``swiglu``: a group has 2 n rows, gate rows first, and the result is
+    silu(gate) * up; otherwise n rows."""
+    rows = 2 * n if swiglu else n
+    if not a.is_cuda:
+        return mixer_torch.gemm_rows(a, w, tile_group, rows, n, swiglu)
+    lib = _lib()
+    p, k = a.shape
+    _req(tile_group.dtype == torch.int32 and tile_group.is_contiguous() and tile_group.numel() * TILE >= p and p % TILE == 0
+         and w.shape[0] % rows == 0 and w.shape[1] == k, "bad grouped product")
+    if a.dtype == torch.bfloat16:
+        out = rows_buffer(p, n, a.dtype, a.device)
+        _check(lib.b200_gemm_bf16_grouped(_ptr(a), _ptr(w), _ptr(out), None, p, n, k, a.stride(0), w.stride(0), out.stride(0),
+                                          0, _ptr(tile_group), w.shape[0] // rows, rows, 1, 0, 0, int(swiglu), 0,
+                                          _ptr(native.status_word(a.device)), _stream()), "gemm_grouped")
+        return out
+    out = rows_buffer(p, rows, a.dtype, a.device)
+    _check(lib.b200_gemm_f32(_ptr(a), _ptr(w), _ptr(out), p, rows, k, a.stride(0), w.stride(0), out.stride(0), 0,
+                             _ptr(tile_group), rows, 1, 0, 0, _stream()), "gemm_f32")
+    if not swiglu:
+        return out
+    h = rows_buffer(p, n, a.dtype, a.device)
+    _check(lib.b200_silu_mul_any(_ptr(out), _ptr(h), p, n, out.stride(0), h.stride(0), 1, _stream()), "silu_mul_any")
+    return h
+
+
+def gemm_heads(a, w, heads: int, k: int, n: int, out=None, gate=None):
+    """One product per head, side by side: out[:, h n : (h+1) n] = a[:, h k : (h+1) k] @ w_h^T, w_h = rows
+    [h w.shape[0] / heads, ...) of w; ``gate`` multiplies with sigmoid(gate), element by element."""
+    if out is None:
+        out = rows_buffer(a.shape[0], heads * n, a.dtype, a.device)
+    if not a.is_cuda:
+        return mixer_torch.gemm_heads(a, w, heads, k, n, out, gate)
+    lib = _lib()
+    _req(w.shape[0] % heads == 0 and w.shape[1] == k and a.shape[1] >= heads * k and out.shape[1] >= heads * n, "bad head product")
+    if a.dtype == torch.bfloat16:
+        _req(k % 8 == 0, "a head's columns must start on a 16-byte boundary")
+        epi = (5 if gate is not None else 0) | native.EPI_B_STABLE
+        _check(lib.b200_gemm_bf16_grouped(_ptr(a), _ptr(w), _ptr(out), _ptr(gate), a.shape[0], n, k, a.stride(0), w.stride(0),
+                                          out.stride(0), 0 if gate is None else gate.stride(0), None, 0, w.shape[0] // heads,
+                                          heads, k, n, 0, epi, _ptr(native.status_word(a.device)), _stream()), "gemm_heads")
+        return out
+    _check(lib.b200_gemm_f32(_ptr(a), _ptr(w), _ptr(out), a.shape[0], n, k, a.stride(0), w.stride(0), out.stride(0), 0, None,
+                             w.shape[0] // heads, heads, k, n, _stream()), "gemm_f32")
+    if gate is not None:
+        gate_sigmoid_(out, gate)
+    return out
+
+
+def gate_sigmoid_(o, gate):
+    if not o.is_cuda:
+        return o.mul_(torch.sigmoid(gate.float()).to(o.dtype))
+    _req(o.shape == gate.shape and o.dtype == gate.dtype, "gate and output must match")
+    _check(_lib().b200_gate_sigmoid(_ptr(o), _ptr(gate), o.shape[0], o.shape[1], o.stride(0), gate.stride(0), _f32(o),
+                                    _stream()), "gate_sigmoid")
+    return o
+
+
+# ------------------------------------------------------------------------------- residual and norm
+def residual_norm(x, w=None, eps: float = 0.0, tokens=None, embed=None, row_index=None, pending=None, scatter=None):
+    """One pass over the fp32 residual stream x (R, d):
+
+    * ``tokens`` / ``embed``: x = embed[tokens] first
+    * ``pending`` = (y, pos (R, top), scale): x += scale * sum_k y[pos[row, k]] (expert outputs; -1 = none)
+    * ``w``: h = x / rms(x) * w, returned in w's dtype (no ``w``: only x is updated)
+    * ``row_index``: h for these rows of x only, x itself stays as it is
+    * ``scatter`` = (pos (R, top), rows): also returns the normed rows at the places the experts read them from
+
+    Returns (h, scattered)."""
+    if not x.is_cuda:
+        return mixer_torch.residual_norm(x, tokens, embed, row_index, pending, w, eps, scatter)
+    lib = _lib()
+    _req(x.dtype == torch.float32 and x.is_contiguous(), "the residual stream is contiguous fp32")
+    d = x.shape[1]
+    rows = x.shape[0] if row_index is None else row_index.numel()
+    act = w if w is not None else (embed if embed is not None else pending[0])
+    h = xg = None
+    if w is not None:
+        _req(w.numel() == d and w.is_contiguous(), "bad norm weight")
+        h = rows_buffer(rows, d, w.dtype, x.device)
+    if tokens is not None:
+        _req(tokens.dtype == torch.int64 and tokens.numel() == rows and embed.is_contiguous() and embed.shape[1] == d
+             and embed.dtype == act.dtype, "bad embedding")
+    if row_index is not None:
+        _req(row_index.dtype == torch.int64 and row_index.is_contiguous(), "row_index must be int64")
+    y = ypos = None
+    scale = 1.0
+    if pending is not None:
+        y, ypos, scale = pending
+        _req(y.dtype == act.dtype and y.shape[1] == d and ypos.dtype == torch.int32 and ypos.is_contiguous()
+             and ypos.shape[0] == x.shape[0], "bad expert outputs")
+    gpos, g_rows = scatter if scatter is not None else (None, 0)
+    if scatter is not None:
+        _req(gpos.dtype == torch.int32 and gpos.is_contiguous() and gpos.shape[0] == rows, "bad expert positions")
+        xg = rows_buffer(g_rows, d, w.dtype, x.device)
+    _check(lib.b200_residual_norm(
+        _ptr(tokens), _ptr(embed), 0 if embed is None else embed.shape[0], _ptr(x), _ptr(row_index), _ptr(y), _ptr(ypos),
+        0 if ypos is None else ypos.shape[1], 0 if y is None else y.shape[0], float(scale), 0 if y is None else y.stride(0),
+        _ptr(w), _ptr(h), 0 if h is None else h.stride(0), float(eps), _ptr(xg), _ptr(gpos),
+        0 if gpos is None else gpos.shape[1], g_rows, 0 if xg is None else xg.stride(0), rows, x.shape[0], d, _f32(act),
+        _ptr(native.status_word(x.device)), _stream()), "residual_norm")
+    return h, xg
+
+
+# ------------------------------------------------------------------------------ mixture of experts
+def plan_tiles(rows: int, experts: int, top: int) -> int:
+    """Row tiles that ``rows`` tokens can need at most: every expert in use leaves one tile partly empty."""
+    return min(experts, rows * top) + rows * top // TILE
+
+
+def moe_plan(tokens, slots, tables, experts):
+    """Sort the (row, choice) pairs of a step by expert, for several layers at once (each with its own table).
+    Returns per layer pos (R, top) int32 and tile_group (tiles,) int32.  Rows with a negative slot are left out."""
+    rows = tokens.numel()
+    tiles = max(plan_tiles(rows, n, t.shape[1]) for t, n in zip(tables, experts))
+    if not tokens.is_cuda:
+        return mixer_torch.moe_plan(tokens, slots, tables, experts, tiles)
+    lib = _lib()
+    _req(tokens.dtype == torch.int64 and slots.dtype == torch.int64 and slots.numel() == rows, "bad plan inputs")
+    top = max(t.shape[1] for t in tables)
+    pos = torch.empty((len(tables), rows * top), dtype=torch.int32, device=tokens.device)
+    group = torch.empty((len(tables), tiles), dtype=torch.int32, device=tokens.device)
+    step = lib.b200_moe_plan_layers()
+    for a in range(0, len(tables), step):
+        part = tables[a:a + step]
+        n = len(part)
+        for t in part:
+            _req(t.dtype == torch.int32 and t.is_contiguous() and t.shape[0] == tables[0].shape[0], "bad expert table")
+        ptrs = (ctypes.c_void_p * n)(*[t.data_ptr() for t in part])
+        ne = (ctypes.c_int * n)(*experts[a:a + step])
+        nt = (ctypes.c_int * n)(*[t.shape[1] for t in part])
+        _check(lib.b200_moe_plan(_ptr(tokens), _ptr(slots), rows, tables[0].shape[0], n, ptrs, ne, nt, _ptr(pos[a]),
+                                 pos.stride(0), _ptr(group[a]), tiles, _ptr(native.status_word(tokens.device)), _stream()),
+               "moe_plan")
+    return ([pos[i, :rows * t.shape[1]].view(rows, t.shape[1]) for i, t in enumerate(tables)], [group[i] for i in range(len(tables))])
+
+
+# -------------------------------------------------------------------------------- latent attention
+def latent_norm_append(proj, wq, wkv, eps: float, cache, slots):
+    """Norm of both latents in proj (columns [0, q_rank) and [q_rank, q_rank + kv_rank)): returns the query latent and
+    writes the key/value latent to its cache slot (negative slot: not written)."""
+    qr, kvr = wq.numel(), wkv.numel()
+    cq = rows_buffer(proj.shape[0], qr, proj.dtype, proj.device)
+    if not proj.is_cuda:
+        return mixer_torch.latent_norm_append(proj, wq, wkv, eps, cache, slots, cq)
+    _req(cache.is_contiguous() and cache.dtype == proj.dtype and cache.shape[-1] >= kvr and slots.dtype == torch.int64
+         and slots.numel() == proj.shape[0], "bad latent cache")
+    _check(_lib().b200_latent_norm_append(_ptr(proj), proj.stride(0), _ptr(wq), _ptr(wkv), _ptr(cq), cq.stride(0), _ptr(cache),
+                                          _ptr(slots), proj.shape[0], qr, kvr, cache.shape[-1],
+                                          cache.shape[0] * cache.shape[1], float(eps), _f32(proj),
+                                          _ptr(native.status_word(proj.device)), _stream()), "latent_norm_append")
+    return cq
+
+
+def latent_attention_rows(q, cache, row_seq, positions, slots, tables, heads: int, window: int, scale: float):
+    """q (R, heads * width) in latent space against the paged latents; every row has its own position and line of
+    ``tables`` (``row_seq`` None: line i for row i).  window 0 = none.  Returns (R, heads * width)."""
+    if not q.is_cuda:
+        return mixer_torch.latent_attention(q, cache, row_seq, positions, slots, tables, heads, window, scale)
+    _req(q.is_contiguous() and cache.is_contiguous() and q.dtype == cache.dtype and q.shape[1] == heads * cache.shape[-1],
+         "bad latent queries")
+    _req(tables.dtype == torch.int32 and tables.is_contiguous() and positions.dtype == torch.int32, "bad tables")
+    out = torch.empty_like(q)
+    _check(_lib().b200_latent_attn_rows(_ptr(q), _ptr(cache), _ptr(out), _ptr(row_seq), _ptr(positions), _ptr(slots),
+                                        _ptr(tables), tables.shape[0], q.shape[0], heads, cache.shape[-1], tables.shape[1],
+                                        cache.shape[1], cache.shape[0], window, float(scale), _f32(q),
+                                        _ptr(native.status_word(q.device)), _stream()), "latent_attn_rows")
+    return out
+
+
+# --------------------------------------------------------------------------------------- retention
+def retention(proj, state, state_slots, cu, spans, positions, cos_sin, decay, heads: int, dim: int, vdim: int, rot: int,
+              eps: float, y):
+    """Retention over the rows of ``proj`` (q | k | v | gate).  ``cu`` (sequences + 1, int32) delimits the sequences, None
+    = one row each; ``spans`` says the same on the host.  The states are read and left in their slots; y (R, heads * vdim)
+    receives the normalised, gated heads."""
+    if not proj.is_cuda:
+        return mixer_torch.retention(proj, state, state_slots, spans, positions, cos_sin, decay, heads, dim, vdim, rot, eps, y)
+    seqs = state_slots.numel()
+    _req(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, dim, vdim), "bad state")
+    _req(state_slots.dtype == torch.int32 and positions.dtype == torch.int32 and decay.dtype == torch.float32, "bad inputs")
+    _req(rot == 0 or (cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[2] == rot // 2), "bad rotary table")
+    _req(proj.shape[1] == 2 * heads * (dim + vdim) and y.shape == (proj.shape[0], heads * vdim) and y.dtype == proj.dtype, "bad shapes")
+    _check(_lib().b200_retention_recurrent(
+        _ptr(proj), proj.stride(0), _ptr(y), y.stride(0), _ptr(state), _ptr(state_slots), _ptr(cu), _ptr(positions),
+        _ptr(cos_sin), _ptr(decay), seqs, proj.shape[0], heads, dim, vdim, rot, 0 if rot == 0 else cos_sin.shape[1],
+        state.shape[0], float(eps), _f32(proj), _ptr(native.status_word(proj.device)), _stream()), "retention")
+    return y

@@ -1,0 +1,176 @@
+"""What the serving engine needs from a model: its cache, one step of its layers, its logits.
+
+``ServingEngine`` owns requests, pages, slots, batches, graphs and sampling; a backend runs the layers of one
+``StepBatch``.  ``forward`` returns whatever ``logits`` takes; both run inside CUDA-graph capture when the batch has no
+portions.  ``splits_prompts`` says whether a long prompt is fed in several portions (its backend reads the earlier ones
+from the cache efficiently)."""
+from __future__ import annotations
+
+import numpy as np
+import torch
+
+from .. import ops
+from ..ops import mixer_ops as mo
+from ..ops import serving_ops
+from .kv_cache import LayerCache, PagedKVCache
+
+
+class TransformerBackend:
+    """``TransformerLM``: packed QKV attention with rotary pairs, K and V pages, bf16 residual stream."""
+
+    splits_prompts = False
+
+    def __init__(self, model):
+        model.use_custom_triton = True
+        eng = model.engine()
+        prov = eng.provider
+        prov.begin_step()                       # builds the bf16 weight mirror and its views
+        self.cfg = eng.cfg
+        self.layers = [prov.block_weights(i) for i in range(self.cfg.n_layers)]
+        self.head = prov.head_weights()
+        self.rope = eng.rope_cache
+        self.device = self.head.emb.device
+        self.dtype = self.head.emb.dtype
+        self.vocab = self.cfg.vocab
+        self.context_limit = min(model.context_length, self.rope.shape[1])
+        self.default_context = self.context_limit
+
+    def set_context(self, positions: int):
+        pass
+
+    def page_bytes(self, page_size: int) -> int:
+        return PagedKVCache.bytes_per_page(self.cfg.n_layers, self.cfg.d_model, page_size,
+                                           2 if self.dtype == torch.bfloat16 else 4)
+
+    def make_cache(self, num_pages: int, page_size: int, max_batch: int):
+        self.cache = PagedKVCache(self.cfg.n_layers, self.cfg.d_model, num_pages, page_size, self.device, self.dtype)
+        return self.cache
+
+    def choose_splits(self, rows: int, max_context: int) -> int:
+        return serving_ops.choose_splits(rows, self.cfg.n_heads, max_context, head_dim=self.cfg.d_model // self.cfg.n_heads)
+
+    def _block(self, x, w, li: int, batch, attend):
+        cfg = self.cfg
+        h, _ = ops.rmsnorm_fwd(x, w.n1, cfg.eps)
+        qkv = ops.gemm(h, w.wqkv, "nt", b_stable=True)
+        # rotary embedding of Q and K in place and the append of K, V to the paged cache: one kernel on the GPU
+        serving_ops.rope_kv_append(qkv, self.rope, batch.positions, self.cache.k[li], self.cache.v[li], batch.slots, cfg.n_heads)
+        o = attend(qkv, li)
+        x = ops.gemm(o, w.wo, "nt", residual=x, b_stable=True)
+        h, _ = ops.rmsnorm_fwd(x, w.n2, cfg.eps)
+        gu = ops.gemm(h, w.wgu, "nt", b_stable=True)
+        return ops.gemm(ops.silu_mul_fwd(gu), w.wdown, "nt", residual=x, b_stable=True)
+
+    def forward(self, batch):
+        heads = self.cfg.n_heads
+        if batch.n_single == batch.n_rows:
+            tables, ctx = batch.tables, batch.ctx
+        elif batch.n_single == 0 and all(start == 0 for start, _ in batch.portions):
+            tables = None
+        else:
+            # portions that continue a prompt, or portions beside single tokens: every row attends to its own request's
+            # pages up to its position, as a decode step does (its K and V are in the cache by then)
+            tables, ctx = batch.tables[batch.row_seq.long()], batch.positions + 1
+
+        def attend(qkv, li):
+            if tables is not None:
+                return serving_ops.paged_decode_attention(qkv, self.cache.k[li], self.cache.v[li], tables, ctx, heads,
+                                                          batch.splits)
+            if qkv.is_cuda:
+                from ..ops import attention
+                return attention.varlen_attention_fwd(qkv, batch.cu, batch.max_portion, heads)
+            return ops.torch_impl.varlen_attention_fwd(qkv, batch.cu, heads)
+
+        x = ops.embedding_fwd(batch.tokens, self.head.emb)
+        for li, w in enumerate(self.layers):
+            x = self._block(x, w, li, batch, attend)
+        return x
+
+    def logits(self, x, rows=None):
+        """(rows, padded vocabulary): only the first ``vocab`` columns are defined."""
+        if rows is not None:
+            x = x[rows].contiguous()
+        h, _ = ops.rmsnorm_fwd(x, self.head.norm, self.cfg.eps)
+        buf = torch.empty((x.shape[0], self.cfg.vocab_padded), dtype=x.dtype, device=x.device)
+        ops.gemm(h, self.head.lm, "nt", out=buf[:, :self.cfg.vocab], b_stable=True)
+        return buf
+
+
+class LayeredBackend:
+    """Models made of listed layers (``models/tedirax.py``): parallel sublayers on one norm, mixers of several kinds, token-
+    table experts, fp32 residual stream.
+
+    A layer run is: one pass over the residual stream (add the previous run's expert outputs, norm, copy rows to where
+    the experts read them), the mixer (adds to the residual stream in its last product), the experts."""
+
+    splits_prompts = True
+
+    def __init__(self, model):
+        self.model = model
+        self.device, self.dtype, self.vocab = model.device, model.dtype, model.vocab_size
+        self.context_limit = None
+        self.default_context = model.DEFAULT_CONTEXT
+        self.specs = [layer.mixer.cache_spec() for layer in model.runs]
+        self.expert_layers = [layer for layer in model.layers if layer.experts is not None]
+
+    def set_context(self, positions: int):
+        for table in self.model.rotary.values():
+            table.resize(positions)
+
+    def page_bytes(self, page_size: int) -> int:
+        return LayerCache.bytes_per_page(self.specs, page_size, self.dtype.itemsize)
+
+    def make_cache(self, num_pages: int, page_size: int, max_batch: int):
+        self.cache = LayerCache(self.specs, num_pages, page_size, max_batch, self.device, self.dtype)
+        return self.cache
+
+    def choose_splits(self, rows: int, max_context: int) -> int:
+        return 0
+
+    def forward(self, batch, trace=None):
+        """``trace``: a list that receives the residual stream after every layer run (a copy; for tests)."""
+        m = self.model
+        x = torch.empty((batch.n_rows, m.config.width), dtype=torch.float32, device=self.device)
+        plan = {}
+        if self.expert_layers:
+            pos, groups = mo.moe_plan(batch.tokens, batch.slots, [la.experts.table for la in self.expert_layers],
+                                      [la.experts.experts for la in self.expert_layers])
+            plan = {la.index: (p, g) for la, p, g in zip(self.expert_layers, pos, groups)}
+        embed, pending = (batch.tokens, m.embed), None
+        for run, layer in enumerate(m.runs):
+            ex = layer.experts
+            scatter = None
+            if ex is not None:
+                pos, groups = plan[layer.index]
+                scatter = (pos, ex.rows(batch.n_rows))
+            h, xg = mo.residual_norm(x, layer.norm, m.config.eps, tokens=embed[0], embed=embed[1], pending=pending,
+                                     scatter=scatter)
+            embed, pending = (None, None), None
+            layer.mixer(h, x, batch, self.cache.entries[run])
+            if ex is not None:
+                pending = (ex(xg, groups), pos, 1.0 / ex.top)
+            if trace is not None:
+                if pending is not None:
+                    mo.residual_norm(x, pending=pending)
+                    pending = None
+                trace.append(x.clone())
+        if not m.runs:
+            mo.residual_norm(x, tokens=batch.tokens, embed=m.embed)
+        return x, pending
+
+    def logits(self, hidden, rows=None):
+        """(rows, vocabulary) fp32."""
+        x, pending = hidden
+        m = self.model
+        if rows is None:
+            h, _ = mo.residual_norm(x, m.final_norm, m.config.eps, pending=pending)
+        else:
+            h, _ = mo.residual_norm(x, m.final_norm, m.config.eps, row_index=rows, pending=pending)
+        out = torch.empty((h.shape[0], mo.pitch(self.vocab)), dtype=torch.float32, device=self.device)
+        mo.linear(h, m.head, out=out[:, :self.vocab])
+        return out
+
+
+def wanted_index(rows: np.ndarray, device) -> torch.Tensor:
+    t = torch.from_numpy(np.ascontiguousarray(rows, dtype=np.int64))
+    return t.pin_memory().to(device, non_blocking=True) if torch.device(device).type == "cuda" else t

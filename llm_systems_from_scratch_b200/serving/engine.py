@@ -1,14 +1,17 @@
-"""Continuous-batching inference engine with a paged KV cache.
+"""Continuous-batching inference engine over a paged cache (and recurrent state slots, for models that have them).
 
 New capability relative to the reference, whose only inference path is ``TransformerLM.generate``
 (batch 1, no KV cache, llm-core/llm_core/model.py:187-236).  One engine instance drives one GPU;
 data-parallel serving runs one replica process per GPU.
 
-Per iteration: newly admitted prompts are packed into one variable-length prefill (FlashAttention
-over the packed rows, K/V written straight into the cache pages), then every running request
-advances by one token in a single decode step (paged-KV attention).  Decode steps are captured in
+Per iteration: newly admitted prompts are packed into one variable-length step whose keys and states go straight
+into the cache (models that can continue a prompt get long ones in portions of at most ``max_prefill_tokens``), then
+every running request advances by one token in a single decode step.  Decode steps are captured in
 CUDA graphs, one per padded batch-size bucket, because at a few milliseconds per step the ~250 kernel
 launches of a step would otherwise be launch bound.  Greedy sampling runs on the device.
+
+The layers belong to the model's backend (``serving.backends``): the engine hands it one ``StepBatch`` at a time,
+whether that is a prompt, a decode step or - ``extend``, for callers that bring the tokens themselves - any mixture.
 """
 from __future__ import annotations
 
@@ -18,9 +21,9 @@ import numpy as np
 import torch
 
 from .. import ops
-from ..ops import serving_ops
 from ..utils.metrics import Percentiles
-from .kv_cache import PagedKVCache
+from .backends import wanted_index
+from .batch import StepBatch
 from .scheduler import Request, Scheduler
 
 
@@ -30,31 +33,27 @@ class ServingEngine:
     def __init__(self, model, num_pages: int | None = None, page_size: int = 16, max_batch: int = 64,
                  max_context: int | None = None, max_prefill_tokens: int = 8192, use_cuda_graphs: bool = True,
                  kv_memory_fraction: float = 0.5):
-        model.use_custom_triton = True
-        eng = model.engine()
-        prov = eng.provider
-        prov.begin_step()                       # builds the bf16 weight mirror and its views
-        self.cfg = eng.cfg
-        self.layers = [prov.block_weights(i) for i in range(self.cfg.n_layers)]
-        self.head = prov.head_weights()
-        self.rope = eng.rope_cache
-        self.device = self.head.emb.device
+        self.backend = be = model.serving_backend()
+        self.device, self.dtype = be.device, be.dtype
         self.cuda = self.device.type == "cuda"
-        self.dtype = self.head.emb.dtype
-        self.max_context = min(max_context or model.context_length, self.rope.shape[1])
+        self.max_context = max_context or be.default_context
+        if be.context_limit is not None:
+            self.max_context = min(self.max_context, be.context_limit)
+        be.set_context(self.max_context)
         self.page_size = page_size
         self.max_pages_per_req = -(-self.max_context // page_size)
         if num_pages is None:
-            per_page = PagedKVCache.bytes_per_page(self.cfg.n_layers, self.cfg.d_model, page_size,
-                                                   2 if self.dtype == torch.bfloat16 else 4)
-            if self.cuda:
+            per_page = be.page_bytes(page_size)
+            if self.cuda and per_page:
                 free, _ = torch.cuda.mem_get_info(self.device)
                 num_pages = max(self.max_pages_per_req * 2, int(free * kv_memory_fraction) // per_page)
                 num_pages = min(num_pages, self.max_pages_per_req * max_batch + 8)
             else:
                 num_pages = self.max_pages_per_req * max_batch
-        self.cache = PagedKVCache(self.cfg.n_layers, self.cfg.d_model, num_pages, page_size, self.device, self.dtype)
-        self.sched = Scheduler(self.cache.allocator, page_size, max_batch, max_prefill_tokens, self.max_context)
+        self.cache = be.make_cache(num_pages, page_size, max_batch)
+        self.sched = Scheduler(self.cache.allocator, page_size, max_batch, max_prefill_tokens, self.max_context,
+                               self.cache.slot_allocator)
+        self._prefilling: list[Request] = []        # admitted, prompt not yet fed completely
         self.max_batch = max_batch
         self.use_graphs = use_cuda_graphs and self.cuda
         self._graphs: dict[int, dict] = {}
@@ -66,35 +65,17 @@ class ServingEngine:
         self._temperature, self._top_k = 0.0, None
         self.stats = {"prefill_tokens": 0, "decode_tokens": 0, "decode_steps": 0, "prefill_steps": 0}
 
-    # ------------------------------------------------------------------ model pieces
-    def _block(self, x, w, li: int, positions, slots, attend):
-        cfg = self.cfg
-        h, _ = ops.rmsnorm_fwd(x, w.n1, cfg.eps)
-        qkv = ops.gemm(h, w.wqkv, "nt", b_stable=True)
-        # rotary embedding of Q and K in place and the append of K, V to the paged cache: one kernel on the GPU
-        serving_ops.rope_kv_append(qkv, self.rope, positions, self.cache.k[li], self.cache.v[li], slots, cfg.n_heads)
-        o = attend(qkv, li)
-        x = ops.gemm(o, w.wo, "nt", residual=x, b_stable=True)
-        h, _ = ops.rmsnorm_fwd(x, w.n2, cfg.eps)
-        gu = ops.gemm(h, w.wgu, "nt", b_stable=True)
-        return ops.gemm(ops.silu_mul_fwd(gu), w.wdown, "nt", residual=x, b_stable=True)
-
-    def _logits(self, x):
-        h, _ = ops.rmsnorm_fwd(x, self.head.norm, self.cfg.eps)
-        buf = torch.empty((x.shape[0], self.cfg.vocab_padded), dtype=x.dtype, device=x.device)
-        ops.gemm(h, self.head.lm, "nt", out=buf[:, :self.cfg.vocab], b_stable=True)
-        return buf
-
+    # ----------------------------------------------------------------------- sampling
     def _greedy(self, logits_buf):
         """Next token per row: argmax, or a draw from softmax(logits / temperature) over the top-k logits when
         ``set_sampling`` asked for one (one kernel on the GPU: filter, softmax and inverse-CDF draw, no sort)."""
         if self._temperature == 0:
-            return ops.argmax_rows(logits_buf, self.cfg.vocab)
+            return ops.argmax_rows(logits_buf, self.backend.vocab)
         rows = logits_buf.shape[0]
-        if logits_buf.is_cuda and logits_buf.dtype == torch.bfloat16:
+        if logits_buf.is_cuda:
             u = torch.rand(rows, device=logits_buf.device)
-            return ops.sample_topk(logits_buf, u, self._temperature, self._top_k, self.cfg.vocab)
-        last = logits_buf[:, :self.cfg.vocab].float() / self._temperature
+            return ops.sample_topk(logits_buf, u, self._temperature, self._top_k, self.backend.vocab)
+        last = logits_buf[:, :self.backend.vocab].float() / self._temperature
         if self._top_k:
             kth = torch.topk(last, min(self._top_k, last.shape[-1])).values[:, -1:]
             last = last.masked_fill(last < kth, float("-inf"))
@@ -107,50 +88,90 @@ class ServingEngine:
             self._graphs.clear()
 
     # ------------------------------------------------------------------------ prefill
-    @torch.no_grad()
-    def prefill(self, reqs: list[Request]) -> torch.Tensor:
-        """Run the prompts of ``reqs`` (pages already reserved); returns their first generated tokens."""
-        ps = self.page_size
-        lens = [len(r.prompt) for r in reqs]
-        # packed inputs built with numpy (one C loop per request instead of one Python iteration per token)
-        tok_np = np.concatenate([np.asarray(r.prompt, dtype=np.int64) for r in reqs])
-        pos_np = np.concatenate([np.arange(n, dtype=np.int32) for n in lens])
-        slot_np = np.concatenate([np.asarray(r.pages, dtype=np.int64)[np.arange(n) // ps] * ps + np.arange(n) % ps
-                                  for r, n in zip(reqs, lens)])
-        cu_np = np.zeros(len(reqs) + 1, dtype=np.int32)
-        cu_np[1:] = np.cumsum(lens)
-        tokens, positions, slots, cu = (torch.from_numpy(a) for a in (tok_np, pos_np, slot_np, cu_np))
-        last = (cu[1:] - 1).long()
-        if self.cuda:
-            tokens, positions, slots, cu_d, last = (t.pin_memory().to(self.device, non_blocking=True)
-                                                    for t in (tokens, positions, slots, cu, last))
-        else:
-            cu_d = cu
-        max_len = max(lens)
-
-        def attend(qkv, li):
-            if qkv.is_cuda:
-                from ..ops import attention
-                return attention.varlen_attention_fwd(qkv, cu_d, max_len, self.cfg.n_heads)
-            return ops.torch_impl.varlen_attention_fwd(qkv, cu, self.cfg.n_heads)
-
-        x = ops.embedding_fwd(tokens, self.head.emb)
-        for li, w in enumerate(self.layers):
-            x = self._block(x, w, li, positions, slots, attend)
-        first = self._greedy(self._logits(x[last].contiguous()))
-        self.stats["prefill_tokens"] += sum(lens)
+    def _run_portions(self, work: list[tuple[Request, int]]) -> torch.Tensor:
+        """Feed the next ``n`` prompt tokens of every (request, n); returns the token sampled behind each portion."""
+        batch = StepBatch.build([(r, r.fed, r.prompt[r.fed:r.fed + n]) for r, n in work], self.page_size,
+                                self.max_pages_per_req, self.device)
+        hidden = self.backend.forward(batch)
+        first = self._greedy(self.backend.logits(hidden, wanted_index(batch.last_rows(), self.device)))
+        for r, n in work:
+            r.fed += n
+        self.stats["prefill_tokens"] += sum(n for _, n in work)
         self.stats["prefill_steps"] += 1
         return first
 
+    @torch.no_grad()
+    def prefill(self, reqs: list[Request]) -> torch.Tensor:
+        """Run the prompts of ``reqs`` (pages already reserved) in one step; returns their first generated tokens."""
+        return self._run_portions([(r, len(r.prompt) - r.fed) for r in reqs])
+
+    # ------------------------------------------------------------- tokens brought by the caller
+    def open(self, rid) -> Request:
+        """A request whose tokens the caller brings step by step (``extend``) until ``close``."""
+        req = Request(rid, [], 0)
+        self.sched.open(req)
+        return req
+
+    def close(self, req: Request):
+        self.sched.finish(req)
+
+    @torch.no_grad()
+    def extend(self, entries: list[tuple[Request, list[int], list[int]]]) -> torch.Tensor | None:
+        """Run one step that brings (request, its next tokens, places among them whose logits are wanted) for every
+        entry, all as one batch: single tokens beside portions of any length.  Returns the logits of the wanted places,
+        entry by entry, (wanted, vocabulary) fp32, or None when nothing is wanted."""
+        for r, ids, _ in entries:
+            if not ids:
+                raise ValueError(f"request {r.rid} brings no token")
+            self.sched.grow(r, r.fed + len(ids))
+        if not entries:
+            return None
+        batch = StepBatch.build([(r, r.fed, ids) for r, ids, _ in entries], self.page_size, self.max_pages_per_req,
+                                self.device)
+        hidden = self.backend.forward(batch)
+        for r, ids, _ in entries:
+            r.fed += len(ids)
+        rows = batch.wanted_rows([want for _, _, want in entries])
+        if not len(rows):
+            return None
+        return self.backend.logits(hidden, wanted_index(rows, self.device))[:, :self.backend.vocab].float()
+
     # ------------------------------------------------------------------------- decode
-    def _decode_body(self, tokens, positions, slots, tables, ctx_lens, splits):
-        def attend(qkv, li):
-            return serving_ops.paged_decode_attention(qkv, self.cache.k[li], self.cache.v[li], tables, ctx_lens,
-                                                      self.cfg.n_heads, splits)
-        x = ops.embedding_fwd(tokens, self.head.emb)
-        for li, w in enumerate(self.layers):
-            x = self._block(x, w, li, positions, slots, attend)
-        return self._greedy(self._logits(x))
+    def _decode_body(self, d: dict, n: int, splits: int):
+        """One decode step of the first ``n`` rows of the device arrays ``d``; returns their next tokens."""
+        batch = StepBatch(d["tokens"][:n], d["positions"][:n], d["slots"][:n], d["tables"][:n], d["ctx"][:n],
+                          d["state"][:n], d["rows"][:n], n, splits=splits)
+        return self._greedy(self.backend.logits(self.backend.forward(batch)))
+
+    def _arrays(self, n: int) -> dict:
+        """Device arrays of a decode step of ``n`` rows, all rows idle."""
+        dev = self.device
+        return {"tokens": torch.zeros(n, dtype=torch.int64, device=dev),
+                "positions": torch.zeros(n, dtype=torch.int32, device=dev),
+                "slots": torch.full((n,), -1, dtype=torch.int64, device=dev),
+                "ctx": torch.ones(n, dtype=torch.int32, device=dev),
+                "state": torch.full((n,), -1, dtype=torch.int32, device=dev),
+                "rows": torch.arange(n, dtype=torch.int32, device=dev),
+                "tables": torch.zeros((n, self.max_pages_per_req), dtype=torch.int32, device=dev)}
+
+    def _capture(self, d: dict, n: int, run) -> torch.cuda.CUDAGraph:
+        """Capture ``run`` (a decode step of the first n rows of ``d``).  The warm-up run before it, where first-launch
+        set-up happens, sees idle rows only: a recurrent state must not advance twice."""
+        keep = {k: d[k][:n].clone() for k in ("tokens", "slots", "state")}
+        d["slots"][:n] = -1
+        d["state"][:n] = -1
+        side = torch.cuda.Stream(device=self.device)
+        side.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(side):
+            run()
+        torch.cuda.current_stream().wait_stream(side)
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            run()
+        for k, v in keep.items():
+            d[k][:n].copy_(v)
+        return graph
 
     def _bucket(self, n: int) -> int:
         for b in self.BUCKETS:
@@ -162,27 +183,16 @@ class ServingEngine:
         g = self._graphs.get(bucket)
         if g is not None:
             return g
-        dev = self.device
-        st = {"tokens": torch.zeros(bucket, dtype=torch.int64, device=dev),
-              "positions": torch.zeros(bucket, dtype=torch.int32, device=dev),
-              "slots": torch.full((bucket,), -1, dtype=torch.int64, device=dev),
-              "tables": torch.zeros((bucket, self.max_pages_per_req), dtype=torch.int32, device=dev),
-              "ctx": torch.ones(bucket, dtype=torch.int32, device=dev)}
-        st["splits"] = serving_ops.choose_splits(bucket, self.cfg.n_heads, self.max_context,
-                                                  head_dim=self.cfg.d_model // self.cfg.n_heads)
-        run = lambda: self._decode_body(st["tokens"], st["positions"], st["slots"], st["tables"], st["ctx"], st["splits"])
+        st = self._arrays(bucket)
+        splits = self.backend.choose_splits(bucket, self.max_context)
+        st["out"] = torch.zeros(bucket, dtype=torch.int64, device=self.device)
+
+        def run():
+            st["out"].copy_(self._decode_body(st, bucket, splits))
         if self.use_graphs:
-            side = torch.cuda.Stream(device=dev)
-            side.wait_stream(torch.cuda.current_stream())
-            with torch.cuda.stream(side):            # warm-up outside capture: first-launch set-up happens here
-                run()
-            torch.cuda.current_stream().wait_stream(side)
-            torch.cuda.synchronize()
-            graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph):
-                st["out"] = run()
-            st["graph"] = graph
+            st["graph"] = self._capture(st, bucket, run)
         st["run"] = run
+        st["splits"] = splits
         self._graphs[bucket] = st
         return st
 
@@ -200,6 +210,7 @@ class ServingEngine:
             mk = lambda shape, dt: torch.zeros(shape, dtype=dt, pin_memory=self.cuda)
             host = st["host"] = {"tokens": mk(bucket, torch.int64), "positions": mk(bucket, torch.int32),
                                  "slots": mk(bucket, torch.int64), "ctx": mk(bucket, torch.int32),
+                                 "state": mk(bucket, torch.int32),
                                  "tables": mk((bucket, self.max_pages_per_req), torch.int32)}
             st["host_np"] = {k: v.numpy() for k, v in host.items()}
         hn = st["host_np"]
@@ -212,6 +223,8 @@ class ServingEngine:
         hn["slots"][n:] = -1
         hn["ctx"][:n] = p + 1
         hn["ctx"][n:] = 1
+        hn["state"][:n] = [r.slot for r in reqs]
+        hn["state"][n:] = -1
         if self._host_rt is not None:
             self._host_rt.block_table_into([r.pages for r in reqs], host["tables"], 0)
         else:
@@ -219,14 +232,13 @@ class ServingEngine:
             tb[:] = 0
             for i, r in enumerate(reqs):
                 tb[i, :len(r.pages)] = r.pages
-        for name in ("tokens", "positions", "slots", "ctx", "tables"):
+        for name in ("tokens", "positions", "slots", "ctx", "state", "tables"):
             st[name].copy_(host[name], non_blocking=True)
         if self.use_graphs:
             st["graph"].replay()
-            out = st["out"]
         else:
-            out = st["run"]()
-        new = out[:n].tolist()
+            st["run"]()
+        new = st["out"][:n].tolist()
         self.stats["decode_tokens"] += n
         self.stats["decode_steps"] += 1
         return new
@@ -238,22 +250,19 @@ class ServingEngine:
     # step k's tokens, retires finished requests and prepares step k + 2.
     def _rows_init(self):
         n = self._bucket(self.max_batch)
-        dev = self.device
         self._row_req: list[Request | None] = [None] * n
         self._row_pos = np.full(n, -1, dtype=np.int64)        # position of the token the row feeds next; -1 = idle
         self._row_tab = np.zeros((n, self.max_pages_per_req), dtype=np.int64)
         self._free_rows = list(range(n - 1, -1, -1))
-        self._d = {"tokens": torch.zeros(n, dtype=torch.int64, device=dev),
-                   "positions": torch.zeros(n, dtype=torch.int32, device=dev),
-                   "slots": torch.full((n,), -1, dtype=torch.int64, device=dev),
-                   "ctx": torch.ones(n, dtype=torch.int32, device=dev),
-                   "tables": torch.zeros((n, self.max_pages_per_req), dtype=torch.int32, device=dev)}
+        self._d = self._arrays(n)
         mk = lambda shape, dt: torch.zeros(shape, dtype=dt, pin_memory=self.cuda)
         # two sets of pinned staging used in turn: a set is refilled only after the step before last has completed
         self._stage = [{"positions": mk(n, torch.int32), "slots": mk(n, torch.int64), "ctx": mk(n, torch.int32),
-                        "out": mk(n, torch.int64)} for _ in range(2)]
+                        "state": mk(n, torch.int32), "out": mk(n, torch.int64)} for _ in range(2)]
         self._stage_np = [{k: v.numpy() for k, v in st.items()} for st in self._stage]
         self._tab_host = mk((n, self.max_pages_per_req), torch.int32)
+        self._state_host = mk(n, torch.int32)
+        self._state_host.fill_(-1)
         self._tab_dirty = False
         self._parity = 0
         self._pending: list[tuple] = []
@@ -264,28 +273,14 @@ class ServingEngine:
         if g is not None:
             return g
         d = self._d
-        splits = serving_ops.choose_splits(bucket, self.cfg.n_heads, self.max_context,
-                                           head_dim=self.cfg.d_model // self.cfg.n_heads)
+        splits = self.backend.choose_splits(bucket, self.max_context)
 
         def run():
-            out = self._decode_body(d["tokens"][:bucket], d["positions"][:bucket], d["slots"][:bucket],
-                                    d["tables"][:bucket], d["ctx"][:bucket], splits)
+            out = self._decode_body(d, bucket, splits)
             d["tokens"][:bucket].copy_(out)          # the next step of every row starts from this token
         g = {"run": run}
         if self.use_graphs:
-            side = torch.cuda.Stream(device=self.device)
-            side.wait_stream(torch.cuda.current_stream())
-            keep = d["tokens"][:bucket].clone()
-            with torch.cuda.stream(side):            # warm-up outside capture: first-launch set-up happens here
-                run()
-            torch.cuda.current_stream().wait_stream(side)
-            d["tokens"][:bucket].copy_(keep)
-            torch.cuda.synchronize()
-            graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph):
-                run()
-            d["tokens"][:bucket].copy_(keep)         # capture does not execute, but keep the contract obvious
-            g["graph"] = graph
+            g["graph"] = self._capture(d, bucket, run)
         self._row_graphs[bucket] = g
         return g
 
@@ -313,6 +308,7 @@ class ServingEngine:
             if r.issued >= r.max_new_tokens:
                 self._row_pos[row] = -1                      # nothing left to decode
         self._tab_host.numpy()[rows] = self._row_tab[rows]
+        self._state_host.numpy()[rows] = [r.slot for r in reqs]
         self._tab_dirty = True
         idx = torch.tensor(rows, dtype=torch.int64)
         if self.cuda:
@@ -351,6 +347,9 @@ class ServingEngine:
         if self._tab_dirty:
             d["tables"].copy_(self._tab_host, non_blocking=True)
             self._tab_dirty = False
+        # an idle row must not touch a state: its slot may belong to another request by now
+        st["state"][:bucket] = np.where(live, self._state_host.numpy()[:bucket], -1)
+        d["state"][:bucket].copy_(host["state"][:bucket], non_blocking=True)
         g = self._row_graph(bucket)
         if self.use_graphs:
             g["graph"].replay()
@@ -405,6 +404,11 @@ class ServingEngine:
             self.sched.waiting.remove(req)
             req.t_done = self._clock()
             return True
+        if req in self._prefilling:
+            self._prefilling.remove(req)
+            req.t_done = self._clock()
+            self.sched.finish(req)
+            return True
         if req.row < 0 or self._row_req[req.row] is not req:
             return False
         row = req.row
@@ -422,13 +426,37 @@ class ServingEngine:
             self._rows_init()
         admitted = self.sched.admit(now)
         if admitted:
-            first = self.prefill(admitted)
             self.sched.start(admitted)
-            self._admit_rows(admitted, first)
+            self._prefilling.extend(admitted)
+        if self._prefilling:
+            self._prefill_step()
         launched = self._launch_decode()
         # on the GPU the newest read-back stays in flight while the host goes on; when nothing was launched (every
         # row's last token is already in flight) or without streams, everything is collected now
         return self._finish(keep_last=1 if (self.cuda and launched) else 0)
+
+    @torch.no_grad()
+    def _prefill_step(self):
+        """Feed prompts, oldest request first, up to the token budget of a step; requests whose prompt is complete join
+        the decode rows.  Without portions every prompt goes whole (admission kept their sum to the budget)."""
+        budget, work = self.sched.max_prefill_tokens, []
+        for r in self._prefilling:
+            n = len(r.prompt) - r.fed
+            if self.backend.splits_prompts:
+                n = min(n, budget)
+                if n <= 0:
+                    break
+                budget -= n
+            work.append((r, n))
+        first = self._run_portions(work)
+        done = [i for i, (r, _) in enumerate(work) if r.fed == len(r.prompt)]
+        if not done:
+            return
+        ready = [work[i][0] for i in done]
+        self._prefilling = [r for r in self._prefilling if r.fed < len(r.prompt)]
+        if len(done) < len(work):
+            first = first[wanted_index(np.asarray(done), self.device)]
+        self._admit_rows(ready, first)
 
     def _clock(self) -> float:
         return time.perf_counter() - self._t0 if self._realtime else self._virtual

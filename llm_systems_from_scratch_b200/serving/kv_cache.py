@@ -1,14 +1,32 @@
-"""Paged KV cache: fixed-size pages (16 tokens by default), a free-list allocator and per-request
+"""Cache manager of the serving engine: fixed-size pages (16 tokens by default), a free-list allocator and per-request
 block tables.  The reference keeps no KV cache (its ``generate`` recomputes the whole context for
 every token, llm-core/llm_core/model.py:210-233); everything here is new capability.
 
 Memory: one K and one V tensor of shape (layers, num_pages, page_size, d_model) in bf16.  For the
 1.3B model a page costs 2 * 24 * 16 * 2048 * 2 B = 3 MiB over all layers, so a 180 GB GPU holds tens
 of thousands of pages next to the 2.8 GB of weights.
+
+``LayerCache`` is the same for models whose layers differ: every layer run says what it keeps per token
+(``PagedSpec``: one vector in a paged pool) or per request (``StateSpec``: a recurrent state in a slot).  All paged
+layers share the page ids of a request, all recurrent layers its slot.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
+
 import torch
+
+
+@dataclass(frozen=True)
+class PagedSpec:
+    """A layer run that caches ``width`` activations per token."""
+    width: int
+
+
+@dataclass(frozen=True)
+class StateSpec:
+    """A layer run that carries one fp32 state of this shape per request."""
+    shape: tuple
 
 
 class PageAllocator:
@@ -55,6 +73,7 @@ class PagedKVCache:
         self.k = torch.zeros((n_layers, num_pages, page_size, d_model), dtype=dtype, device=device)
         self.v = torch.zeros((n_layers, num_pages, page_size, d_model), dtype=dtype, device=device)
         self.allocator = PageAllocator(num_pages)
+        self.slot_allocator = None                 # nothing is carried per request besides its pages
 
     @staticmethod
     def pages_for(tokens: int, page_size: int = 16) -> int:
@@ -74,3 +93,41 @@ class PagedKVCache:
             from ..utils import host_runtime
             return host_runtime.slots(pages, ps, start, count)
         return [pages[t // ps] * ps + t % ps for t in range(start, start + count)]
+
+
+class LayerCache:
+    """Paged pools and state slots, one entry per layer run in ``entries``.
+
+    Freed pages and slots are handed out again as they are: a position's cached vector is written before anything reads
+    it, and a recurrent layer starts from the zero state at position 0 whatever the slot held."""
+
+    def __init__(self, specs: list, num_pages: int, page_size: int, num_slots: int, device, dtype):
+        self.specs, self.page_size, self.num_pages, self.num_slots = specs, page_size, num_pages, num_slots
+        self.entries = []
+        for s in specs:
+            if isinstance(s, PagedSpec):
+                self.entries.append(torch.zeros((num_pages, page_size, s.width), dtype=dtype, device=device))
+            elif isinstance(s, StateSpec):
+                self.entries.append(torch.zeros((num_slots, *s.shape), dtype=torch.float32, device=device))
+            else:
+                self.entries.append(None)
+        self.allocator = PageAllocator(num_pages)
+        self.slot_allocator = PageAllocator(num_slots)
+
+    @staticmethod
+    def bytes_per_page(specs: list, page_size: int, itemsize: int) -> int:
+        return sum(s.width for s in specs if isinstance(s, PagedSpec)) * page_size * itemsize
+
+    @staticmethod
+    def bytes_per_slot(specs: list) -> int:
+        total = 0
+        for s in specs:
+            if isinstance(s, StateSpec):
+                n = 4
+                for k in s.shape:
+                    n *= k
+                total += n
+        return total
+
+    def occupancy(self) -> float:
+        return 1.0 - self.allocator.free / max(1, self.num_pages)

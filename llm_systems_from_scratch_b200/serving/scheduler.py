@@ -5,7 +5,11 @@ order, as long as the running batch has room, the prefill token budget is not ex
 cache can hold the request's whole lifetime (prompt + maximum output, reserved up front so a
 running request is never pre-empted), and (2) hands all running requests to one decode step.
 Finished requests return their pages immediately, so a request that arrives mid-flight joins the
-batch at the next iteration instead of waiting for the batch to drain.
+batch at the next iteration instead of waiting for the batch to drain.  Models with recurrent layers
+also give every running request a state slot (``slots``), which comes and goes with the pages.
+
+A request whose tokens come from outside step by step (``open`` / ``grow``) reserves pages as it grows
+instead of up front.
 
 The reference has no serving loop: its ``generate`` (llm-core/llm_core/model.py:187-236) handles one prompt at a
 time and ``generate.py`` is a REPL around it.
@@ -30,6 +34,8 @@ class Request:
     output: list[int] = field(default_factory=list)
     t_first: float | None = None
     t_done: float | None = None
+    slot: int = -1           # state slot while running, for models with recurrent layers
+    fed: int = 0             # tokens that have gone through the model so far, while the prompt is fed in portions
     row: int = -1            # row of the engine's batch arrays while running
     issued: int = 0          # tokens produced on the device so far (the host may not have read the last one yet)
 
@@ -60,8 +66,9 @@ def poisson_trace(num_requests: int, rate: float, prompt_len: tuple[int, int], o
 
 class Scheduler:
     def __init__(self, allocator, page_size: int, max_batch: int, max_prefill_tokens: int = 8192,
-                 max_context: int = 2560):
+                 max_context: int = 2560, slots=None):
         self.alloc = allocator
+        self.slots = slots
         self.page_size = page_size
         self.max_batch = max_batch
         self.max_prefill_tokens = max_prefill_tokens
@@ -92,10 +99,13 @@ class Scheduler:
             need = self._pages_needed(req)
             if need > self.alloc.free:
                 break                                   # FCFS: do not let later requests overtake
+            if self.slots is not None and self.slots.free < 1:
+                break
             if batch and tokens + len(req.prompt) > self.max_prefill_tokens:
                 break
             self.waiting.popleft()
             req.pages = self.alloc.take(need)
+            self._take_slot(req)
             tokens += len(req.prompt)
             batch.append(req)
         return batch
@@ -109,15 +119,39 @@ class Scheduler:
             self.running = [r for r in self.running if not r.finished]
             for r in done:
                 r.t_done = now
-                self.alloc.give(r.pages)
-                r.pages = []
+                self._give_back(r)
         return done
 
     def finish(self, req: Request):
         """``req`` has produced its last token: return its pages and drop it from the running set."""
         self.running.remove(req)
+        self._give_back(req)
+
+    def _take_slot(self, req: Request):
+        if self.slots is not None:
+            req.slot = self.slots.take(1)[0]
+
+    def _give_back(self, req: Request):
         self.alloc.give(req.pages)
         req.pages = []
+        if req.slot >= 0:
+            self.slots.give([req.slot])
+            req.slot = -1
+
+    def open(self, req: Request):
+        """Run a request whose tokens arrive step by step: it gets a state slot now and pages as it grows."""
+        if len(self.running) >= self.max_batch:
+            raise MemoryError(f"{self.max_batch} requests are running already")
+        self._take_slot(req)
+        self.running.append(req)
+
+    def grow(self, req: Request, tokens: int):
+        """Reserve pages until ``req`` can hold ``tokens`` positions."""
+        if tokens > self.max_context:
+            raise ValueError(f"request {req.rid} needs {tokens} positions, limit is {self.max_context}")
+        need = -(-tokens // self.page_size) - len(req.pages)
+        if need > 0:
+            req.pages = req.pages + self.alloc.take(need)
 
     @property
     def idle(self) -> bool:
