@@ -13,6 +13,10 @@
 //               straight from tensor memory.  O is rescaled in TMEM only when the running max moved by more
 //               than 2^8 (vote per warp).
 // Tensor-pipe order per key tile j: P_A V_j, S_A(j+1), P_B V_j, S_B(j+1).
+//
+// WINDOW instances (b200_flash_window_fwd) serve portions of prompts under a sliding window: queries and keys come from
+// separate matrices, a sequence has more keys than queries (the earlier tokens its first queries can still see), tile X
+// walks only the key tiles its window touches, and the epilogue can multiply with sigmoid(gate).
 #include "ptx.cuh"
 
 namespace b200 {
@@ -84,6 +88,14 @@ struct FlashFwdParams {
   int n_qblk;            // 128-query tiles per sequence; a CTA takes two of them
   float scale_log2;      // softmax scale * log2(e)
   uint32_t* status;
+  // WINDOW instances only
+  const int* cu_k;       // (batch+1) row offsets of the keys; queries are the last positions of their sequence's keys
+  int window;            // a query sees the `window` keys up to and including its own position
+  int vdim;              // columns of a head that are written (<= DH)
+  long long ld_o;
+  const __nv_bfloat16* gate;   // optional (rows, heads * vdim), row pitch ld_gate
+  long long ld_gate;
+  int out_vec, gate_vec; // 16-byte stores / loads are possible
   long long* trace;      // optional timeline of CTA `trace_cta` (tuning aid); null = off
   int trace_cta;
 };
@@ -107,9 +119,10 @@ struct FlashFwdSmem {
   static constexpr int TOTAL = OFF_BAR + NUM_BARS * 8 + 16 + 1024;
 };
 
-template <int DH>
+template <int DH, bool WINDOW>
 __global__ void __launch_bounds__(FA_THREADS, 1)
-flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParams p) {
+flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_constant__ CUtensorMap tm_kv,
+                 const FlashFwdParams p) {
   using L = FlashFwdSmem<DH>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -141,13 +154,22 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
     row_base = b * p.seq;
     seq_len = p.seq;
   }
-  // CTA-uniform tile geometry: tile X covers queries [q0[X], q0[X] + 128) and key tiles 0 .. n_kv_t[X] - 1
+  int key_base = row_base, shift = 0;      // first key row; position of query 0 among the keys
+  if (WINDOW) {
+    key_base = p.cu_k[b];
+    shift = p.cu_k[b + 1] - key_base - seq_len;
+  }
+  // CTA-uniform tile geometry: tile X covers queries [q0[X], q0[X] + 128) and key tiles lo_t[X] .. n_kv_t[X] - 1.  Tile A's
+  // range starts and ends no later than tile B's and the two ranges leave no gap, so the CTA walks lo_t[0] .. n_kv - 1.
   const int q0_t[2] = {pair * 2 * FA_BQ, pair * 2 * FA_BQ + FA_BQ};
-  int n_kv_t[2];
+  int n_kv_t[2], lo_t[2];
 #pragma unroll
-  for (int x = 0; x < 2; ++x)
-    n_kv_t[x] = q0_t[x] < seq_len ? (min(q0_t[x] + FA_BQ, seq_len) + FA_BK - 1) / FA_BK : 0;
+  for (int x = 0; x < 2; ++x) {
+    n_kv_t[x] = q0_t[x] < seq_len ? (min(q0_t[x] + FA_BQ, seq_len) + shift + FA_BK - 1) / FA_BK : 0;
+    lo_t[x] = (WINDOW && n_kv_t[x] > 0) ? max(0, q0_t[x] + shift - p.window + 1) / FA_BK : 0;
+  }
   const int n_kv = max(n_kv_t[0], n_kv_t[1]);
+  const int j0 = lo_t[0];
   const bool active = n_kv > 0;
 
   if (threadIdx.x == 0) {
@@ -165,6 +187,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
     *abort_word = 0;
     fence_barrier_init();
     prefetch_tensormap(&tm_qkv);
+    if (WINDOW) prefetch_tensormap(&tm_kv);
   }
   if (warp == 1) {
     tmem_alloc(tmem_holder, 512);
@@ -176,7 +199,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
   const uint32_t tmem_base = *tmem_holder;
   // columns: S_A [0,128)  S_B [128,256)  O_A [256,256+DH)  O_B [384,384+DH); P_X overlays the first 64 columns of S_X
 
-  const int col_q = h * DH, col_k = p.d + h * DH, col_v = 2 * p.d + h * DH;
+  const int col_q = h * DH, col_k = (WINDOW ? 0 : p.d) + h * DH, col_v = (WINDOW ? p.d : 2 * p.d) + h * DH;
+  const CUtensorMap* const map_kv = WINDOW ? &tm_kv : &tm_qkv;
 
   if (warp == 0) {
     if (active && elect_one()) {   // elect.sync keeps the issuing code warp-uniform (descriptors in uniform registers)
@@ -188,20 +212,20 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
         for (int pn = 0; pn < L::PANELS; ++pn)
           tma_load_2d(smem + L::OFF_Q + x * L::TILE_BYTES + pn * 16384, &tm_qkv, q_full, col_q + pn * 64,
                       row_base + q0_t[x]);
-      for (int j = 0; j < n_kv; ++j) {
-        const int st = j & 1;
-        const uint32_t ph = (j >> 1) & 1;
-        const int krow = row_base + j * FA_BK;
+      for (int j = j0; j < n_kv; ++j) {
+        const int st = (j - j0) & 1;
+        const uint32_t ph = ((j - j0) >> 1) & 1;
+        const int krow = key_base + j * FA_BK;
         if (!mbar_wait(&k_empty[st], ph ^ 1, abort_word)) { *abort_word = ERR_WAIT_EMPTY; break; }
         mbar_expect_tx(&k_full[st], L::TILE_BYTES);
 #pragma unroll
         for (int pn = 0; pn < L::PANELS; ++pn)
-          tma_load_2d(smem + L::OFF_K + st * L::TILE_BYTES + pn * 16384, &tm_qkv, &k_full[st], col_k + pn * 64, krow);
+          tma_load_2d(smem + L::OFF_K + st * L::TILE_BYTES + pn * 16384, map_kv, &k_full[st], col_k + pn * 64, krow);
         if (!mbar_wait(&v_empty[st], ph ^ 1, abort_word)) { *abort_word = ERR_WAIT_EMPTY; break; }
         mbar_expect_tx(&v_full[st], L::TILE_BYTES);
 #pragma unroll
         for (int pn = 0; pn < L::PANELS; ++pn)
-          tma_load_2d(smem + L::OFF_V + st * L::TILE_BYTES + pn * 16384, &tm_qkv, &v_full[st], col_v + pn * 64, krow);
+          tma_load_2d(smem + L::OFF_V + st * L::TILE_BYTES + pn * 16384, map_kv, &v_full[st], col_v + pn * 64, krow);
       }
     }
   } else if (warp == 1) {
@@ -212,7 +236,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
       constexpr uint32_t idesc_pv = make_idesc_bf16(128, DH, false, true);
       auto issue_s = [&](int x, int j) {   // S_X(j) = Q_X K_j^T
         const uint64_t q_desc = make_smem_desc(smem_u32(smem + L::OFF_Q + x * L::TILE_BYTES), 16, 1024);
-        const uint64_t k_desc = make_smem_desc(smem_u32(smem + L::OFF_K + (j & 1) * L::TILE_BYTES), 16, 1024);
+        const uint64_t k_desc = make_smem_desc(smem_u32(smem + L::OFF_K + ((j - j0) & 1) * L::TILE_BYTES), 16, 1024);
 #pragma unroll
         for (int k = 0; k < DH / 16; ++k) {
           const uint32_t off = ((k / 4) * 16384 + (k % 4) * 32) >> 4;
@@ -224,44 +248,44 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
       // A = P from tensor memory (16 keys = 8 packed columns), B = V MN-major (dh contiguous, keys are rows of
       // 128 B): 16 keys = 2048 B; dh panels 16384 B apart.
       auto issue_pv = [&](int x, int j, int half) {
-        const uint64_t v_desc = make_smem_desc(smem_u32(smem + L::OFF_V + (j & 1) * L::TILE_BYTES), 16384, 1024);
+        const uint64_t v_desc = make_smem_desc(smem_u32(smem + L::OFF_V + ((j - j0) & 1) * L::TILE_BYTES), 16384, 1024);
 #pragma unroll
         for (int kk = 0; kk < FA_BK / 32; ++kk) {
           const int k = half * (FA_BK / 32) + kk;
           umma_f16_ts(tmem_base + 256 + x * 128, tmem_base + x * 128 + k * 8, v_desc + ((k * 2048) >> 4), idesc_pv,
-                      (j > 0 || k > 0) ? 1u : 0u);
+                      (j > lo_t[x] || k > 0) ? 1u : 0u);
         }
         if (half == 1 && j == n_kv_t[x] - 1) umma_commit(&o_full[x]);
       };
       bool ok = mbar_wait(q_full, 0, abort_word) && mbar_wait(&k_full[0], 0, abort_word);
       if (ok) {
         tc_fence_after();
-        if (n_kv_t[0] > 0) issue_s(0, 0);
-        if (n_kv_t[1] > 0) issue_s(1, 0);
+        if (n_kv_t[0] > 0) issue_s(0, j0);
+        if (n_kv_t[1] > 0 && lo_t[1] == j0) issue_s(1, j0);
         umma_commit(&k_empty[0]);
       }
-      for (int j = 0; j < n_kv && ok; ++j) {
-        const int st = j & 1;
-        const uint32_t ph = (j >> 1) & 1;
+      for (int j = j0; j < n_kv && ok; ++j) {
+        const int st = (j - j0) & 1;
+        const uint32_t ph = ((j - j0) >> 1) & 1;
         bool v_ready = false, k_ready = false;
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
-          if (j < n_kv_t[x]) {
-            ok = mbar_wait(&p_full[2 * x], j & 1, abort_word) && (v_ready || mbar_wait(&v_full[st], ph, abort_word));
+          if (j >= lo_t[x] && j < n_kv_t[x]) {
+            ok = mbar_wait(&p_full[2 * x], (j - lo_t[x]) & 1, abort_word) && (v_ready || mbar_wait(&v_full[st], ph, abort_word));
             if (!ok) break;
             v_ready = true;
             tc_fence_after();
             FWD_TRACE(1, j, x * 4 + 0);
             issue_pv(x, j, 0);
-            ok = mbar_wait(&p_full[2 * x + 1], j & 1, abort_word);
+            ok = mbar_wait(&p_full[2 * x + 1], (j - lo_t[x]) & 1, abort_word);
             if (!ok) break;
             tc_fence_after();
             issue_pv(x, j, 1);
             FWD_TRACE(1, j, x * 4 + 1);
           }
           if (x == 1) umma_commit(&v_empty[st]);   // both tiles are done with V_j
-          if (j + 1 < n_kv_t[x]) {
-            ok = k_ready || mbar_wait(&k_full[st ^ 1], ((j + 1) >> 1) & 1, abort_word);
+          if (j + 1 >= lo_t[x] && j + 1 < n_kv_t[x]) {
+            ok = k_ready || mbar_wait(&k_full[st ^ 1], ((j + 1 - j0) >> 1) & 1, abort_word);
             if (!ok) break;
             k_ready = true;
             tc_fence_after();
@@ -279,22 +303,26 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
     const int quarter = warp & 3;               // TMEM lanes [32*quarter, 32*quarter+32) are visible to this warp
     const int r = quarter * 32 + lane;          // row inside the query tile
     const int q0 = (pair * 2 + x) * FA_BQ;
-    const int n_kv_x = q0 < seq_len ? (min(q0 + FA_BQ, seq_len) + FA_BK - 1) / FA_BK : 0;
-    const int q_idx = q0 + r;                   // position inside the sequence
+    const int n_kv_x = x == 0 ? n_kv_t[0] : n_kv_t[1];
+    const int lo_x = x == 0 ? lo_t[0] : lo_t[1];
+    const int q_idx = q0 + r;                   // query of this thread
+    const int q_key = q_idx + shift;            // its position among the keys
+    const int q_low = WINDOW ? q_key - p.window : -1;   // the last key it no longer sees
     const uint32_t lane_addr = uint32_t(quarter * 32) << 16;
     const uint32_t tm_s = tmem_base + x * 128 + lane_addr;
     const uint32_t tm_o = tmem_base + 256 + x * 128 + lane_addr;
     float m_run = -INFINITY;                    // running reference max in scaled log2 units
     float l_run = 0.f;                          // running row sum relative to m_run
     bool ok = true;
-    for (int j = 0; j < n_kv_x; ++j) {
+    for (int j = lo_x; j < n_kv_x; ++j) {
       const int trole = warp;
       FWD_TRACE(trole, j, 0);
-      if (!mbar_wait(&s_full[x], j & 1, abort_word)) { ok = false; break; }
+      if (!mbar_wait(&s_full[x], (j - lo_x) & 1, abort_word)) { ok = false; break; }
       tc_fence_after();
       FWD_TRACE(trole, j, 1);
       const int k0 = j * FA_BK;
-      const bool diag = (k0 + FA_BK - 1 > q0);   // tile touches the diagonal (warp-uniform)
+      // tile touches the diagonal or the lower edge of the window (warp-uniform)
+      const bool diag = (k0 + FA_BK - 1 > q0 + shift) || (WINDOW && k0 <= q0 + FA_BQ - 1 + shift - p.window);
       // pass 1: row maximum over the raw scores (the softmax scale is positive, so it is applied afterwards).
       // The load of chunk c+1 is in flight while chunk c is reduced.
       float mx = -INFINITY;
@@ -310,7 +338,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
           if (diag) {
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              if (k0 + c * 32 + i > q_idx) cur[i] = 0xff800000u;   // -inf
+              if (k0 + c * 32 + i > q_key || (WINDOW && k0 + c * 32 + i <= q_low)) cur[i] = 0xff800000u;   // -inf
           }
 #pragma unroll
           for (int i = 0; i < 32; i += 2) mx = fmax3(mx, __uint_as_float(cur[i]), __uint_as_float(cur[i + 1]));
@@ -325,7 +353,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
       const bool need = m_new != m_run;
       const float alpha = (m_run == -INFINITY) ? 0.f : fa_exp2(m_run - m_new);
       // S_X(j) was issued after P_X V_{j-1}, so that MMA has completed and O_X may be rescaled here.
-      if (j > 0 && __any_sync(0xffffffffu, need)) {
+      if (j > lo_x && __any_sync(0xffffffffu, need)) {
         const float f = need ? alpha : 1.f;
 #pragma unroll 1
         for (int c = 0; c < DH / 32; ++c) {
@@ -340,6 +368,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
       FWD_TRACE(trole, j, 3);
       // pass 2: P = exp2(S * scale - m), row sum, bf16 pack; P chunk c (16 packed columns) lands on S columns
       // [16c, 16c+16), all of which this thread has already read.
+      // (a row whose window starts in a later tile has seen no key yet: every P is masked to zero below)
+      const float m_ref = (WINDOW && m_new == -INFINITY) ? 0.f : m_new;
       float sum = 0.f, sum1 = 0.f;
       {
         uint32_t sa[32], sb[32];
@@ -354,12 +384,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
             float x0, x1;
-            fma2(x0, x1, __uint_as_float(s[i]), __uint_as_float(s[i + 1]), p.scale_log2, -m_new);
+            fma2(x0, x1, __uint_as_float(s[i]), __uint_as_float(s[i + 1]), p.scale_log2, -m_ref);
             float e0 = ((i & 7) < FA_POLY_PER_8) ? fa_exp2_poly(x0) : fa_exp2(x0);
             float e1 = (((i + 1) & 7) < FA_POLY_PER_8) ? fa_exp2_poly(x1) : fa_exp2(x1);
             if (diag) {
-              e0 = (k0 + c * 32 + i > q_idx) ? 0.f : e0;
-              e1 = (k0 + c * 32 + i + 1 > q_idx) ? 0.f : e1;
+              const int key = k0 + c * 32 + i;
+              e0 = (key > q_key || (WINDOW && key <= q_low)) ? 0.f : e0;
+              e1 = (key + 1 > q_key || (WINDOW && key + 1 <= q_low)) ? 0.f : e1;
             }
             add2(sum, sum1, e0, e1);
             pk[i / 2] = pack_bf16x2(e0, e1);
@@ -383,13 +414,49 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
       tc_fence_after();
       const float inv_l = 1.f / l_run;
       const bool valid = q_idx < seq_len;
-      __nv_bfloat16* orow = p.o + (size_t)(row_base + q_idx) * p.d + h * DH;
+      __nv_bfloat16* orow = WINDOW ? p.o + (long long)(row_base + q_idx) * p.ld_o + h * p.vdim
+                                   : p.o + (size_t)(row_base + q_idx) * p.d + h * DH;
 #pragma unroll 1
       for (int c = 0; c < DH / 32; ++c) {
         uint32_t o[32];
         tmem_ld_32x32(tm_o + c * 32, o);
         tmem_ld_wait();
-        if (valid) {
+        if (WINDOW) {
+          if (valid && c * 32 < p.vdim) {      // no early continue: the next tensor-memory load needs the whole warp
+            const __nv_bfloat16* grow =
+                p.gate != nullptr ? p.gate + (long long)(row_base + q_idx) * p.ld_gate + h * p.vdim + c * 32 : nullptr;
+            const int n = min(32, p.vdim - c * 32);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+              if (q * 8 >= n) break;
+              float f[8];
+#pragma unroll
+              for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(o[q * 8 + i]) * inv_l;
+              if (grow != nullptr && p.gate_vec && q * 8 + 8 <= n) {
+                const uint4 gv = *reinterpret_cast<const uint4*>(grow + q * 8);
+                const uint32_t gg[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                  const float2 g2 = unpack_bf16x2(gg[i]);
+                  f[2 * i] = __fdividef(f[2 * i], 1.f + __expf(-g2.x));
+                  f[2 * i + 1] = __fdividef(f[2 * i + 1], 1.f + __expf(-g2.y));
+                }
+              } else if (grow != nullptr) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                  if (q * 8 + i < n) f[i] = __fdividef(f[i], 1.f + __expf(-__bfloat162float(grow[q * 8 + i])));
+              }
+              if (p.out_vec && q * 8 + 8 <= n) {
+                *reinterpret_cast<uint4*>(orow + c * 32 + q * 8) =
+                    make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+              } else {
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                  if (q * 8 + i < n) orow[c * 32 + q * 8 + i] = __float2bfloat16(f[i]);
+              }
+            }
+          }
+        } else if (valid) {
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
             uint4 v = make_uint4(pack_bf16x2(__uint_as_float(o[q * 8 + 0]) * inv_l, __uint_as_float(o[q * 8 + 1]) * inv_l),
@@ -422,17 +489,17 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const FlashFwdParam
   }
 }
 
-template <int DH>
-static int launch_flash_fwd(const CUtensorMap& tm, const FlashFwdParams& p, cudaStream_t stream) {
+template <int DH, bool WINDOW>
+static int launch_flash_fwd(const CUtensorMap& tm, const CUtensorMap& tm_kv, const FlashFwdParams& p, cudaStream_t stream) {
   using L = FlashFwdSmem<DH>;
-  auto kern = flash_fwd_kernel<DH>;
+  auto kern = flash_fwd_kernel<DH, WINDOW>;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL) != cudaSuccess) return -3;
     configured = true;
   }
   const int grid = p.batch * p.heads * ((p.n_qblk + 1) / 2);   // one CTA per pair of query tiles
-  kern<<<grid, FA_THREADS, L::TOTAL, stream>>>(tm, p);
+  kern<<<grid, FA_THREADS, L::TOTAL, stream>>>(tm, tm_kv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -460,14 +527,14 @@ extern "C" int b200_flash_fwd(const void* qkv, void* o, float* lse, int batch, i
   const int d = heads * dh;
   CUtensorMap tm;
   if (make_tmap_bf16_2d(&tm, qkv, (uint64_t)batch * seq, (uint64_t)3 * d, (uint64_t)3 * d, 64, 128)) return -20;
-  FlashFwdParams p;
+  FlashFwdParams p = {};
   p.o = (__nv_bfloat16*)o; p.lse = lse; p.cu_seqlens = nullptr;
   p.batch = batch; p.seq = seq; p.heads = heads; p.d = d;
   p.n_qblk = (seq + FA_BQ - 1) / FA_BQ;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
   p.trace = g_fwd_trace; p.trace_cta = g_fwd_trace_cta;
-  return dh == 64 ? launch_flash_fwd<64>(tm, p, stream) : launch_flash_fwd<128>(tm, p, stream);
+  return dh == 64 ? launch_flash_fwd<64, false>(tm, tm, p, stream) : launch_flash_fwd<128, false>(tm, tm, p, stream);
 }
 
 // Packed variable-length sequences (serving prefill): cu_seqlens (batch+1) int32 on the device,
@@ -481,12 +548,41 @@ extern "C" int b200_flash_varlen_fwd(const void* qkv, void* o, const int* cu_seq
   const int d = heads * dh;
   CUtensorMap tm;
   if (make_tmap_bf16_2d(&tm, qkv, (uint64_t)total_rows, (uint64_t)3 * d, (uint64_t)3 * d, 64, 128)) return -20;
-  FlashFwdParams p;
+  FlashFwdParams p = {};
   p.o = (__nv_bfloat16*)o; p.lse = nullptr; p.cu_seqlens = cu_seqlens;
   p.batch = batch; p.seq = max_seq; p.heads = heads; p.d = d;
   p.n_qblk = (max_seq + FA_BQ - 1) / FA_BQ;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
   p.trace = g_fwd_trace; p.trace_cta = g_fwd_trace_cta;
-  return dh == 64 ? launch_flash_fwd<64>(tm, p, stream) : launch_flash_fwd<128>(tm, p, stream);
+  return dh == 64 ? launch_flash_fwd<64, false>(tm, tm, p, stream) : launch_flash_fwd<128, false>(tm, tm, p, stream);
+}
+
+// Portions of prompts under a sliding window.  q: (total_q, heads * dh), kv: (total_k, 2 * heads * dh) = K | V, heads padded
+// with zero columns to dh = 64 or 128; cu_q / cu_k: (batch + 1) row offsets on the device; query i of a sequence with Lq
+// queries and Lk keys sits at key position i + Lk - Lq and sees the `window` keys up to it (window <= 0: all of them).
+// o: (total_q, heads * vdim), row pitch ld_o, multiplied by sigmoid(gate) when gate is given.  scale must be positive.
+extern "C" int b200_flash_window_fwd(const void* q, const void* kv, void* o, const void* gate, const int* cu_q,
+                                     const int* cu_k, int batch, int max_q, int total_q, int total_k, int heads, int dh,
+                                     int vdim, int window, float scale, long long ld_q, long long ld_kv, long long ld_o,
+                                     long long ld_gate, uint32_t* status, cudaStream_t stream) {
+  if ((dh != 64 && dh != 128) || vdim <= 0 || vdim > dh || !(scale > 0.f)) return -10;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv)) & 15 || ld_q % 8 || ld_kv % 8) return -10;
+  if (batch <= 0 || total_q <= 0) return 0;
+  const int d = heads * dh;
+  CUtensorMap tm, tm_kv;
+  if (make_tmap_bf16_2d(&tm, q, (uint64_t)total_q, (uint64_t)d, (uint64_t)ld_q, 64, 128)) return -20;
+  if (make_tmap_bf16_2d(&tm_kv, kv, (uint64_t)total_k, (uint64_t)2 * d, (uint64_t)ld_kv, 64, 128)) return -21;
+  FlashFwdParams p = {};
+  p.o = (__nv_bfloat16*)o; p.cu_seqlens = cu_q; p.cu_k = cu_k;
+  p.batch = batch; p.seq = max_q; p.heads = heads; p.d = d;
+  p.n_qblk = (max_q + FA_BQ - 1) / FA_BQ;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.window = window > 0 ? window : (1 << 30);
+  p.vdim = vdim; p.ld_o = ld_o;
+  p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate;
+  p.out_vec = vdim % 8 == 0 && ld_o % 8 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0;
+  p.gate_vec = vdim % 8 == 0 && ld_gate % 8 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0;
+  p.status = status;
+  return dh == 64 ? launch_flash_fwd<64, true>(tm, tm_kv, p, stream) : launch_flash_fwd<128, true>(tm, tm_kv, p, stream);
 }

@@ -115,6 +115,293 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(
   for (int c = lane; c < width; c += 32) from_f(orow[c], acc[c] * inv);
 }
 
+// ------------------------------------------------------------------------------- decode, bf16, on the tensor cores
+// One CTA = one row (request), up to 16 * MT of its heads and one split of the window.  All heads share the cached latents,
+// so the score and value products are (heads x width) by (width x tokens) and back: with 16 heads that is ~32 FLOP per
+// cached byte, too much for the FMA pipes but little for mma.sync at M = 16, and the kernel stays bound by reading the
+// cache.  Tiles of 32 tokens are copied by cp.async into a two-stage ring straight from the pages; four warps compute
+// 8 tokens' scores each, then own a quarter of the latent columns of the output.  The softmax is online, in fp32.
+constexpr int LD_BT = 32;       // tokens per tile
+constexpr int LD_THREADS = 128;
+
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr)
+               : "memory");
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr)
+               : "memory");
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+      "{%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+
+struct LatentDecodeParams {
+  const __nv_bfloat16* q;       // (rows, heads * width)
+  const __nv_bfloat16* cache;
+  __nv_bfloat16* o;             // (rows, heads * width)
+  float* part_o;                // (rows, heads, splits, width) when splits > 1
+  float* part_ml;               // (rows, heads, splits, 2)
+  const int* positions;
+  const long long* slots;
+  const int* tables;            // line i for row i
+  int rows, heads, width, max_pages, page_size, num_pages, window, splits;
+  float scale_log2;
+  uint32_t* status;
+};
+
+template <int NT>
+struct LatentDecodeSmem {
+  static constexpr int KP = NT * 64;            // latent columns, padded
+  static constexpr int PITCH = KP + 8;          // an odd number of 16-byte pieces: ldmatrix without bank conflicts
+  static constexpr int bytes(int mt) {
+    return (mt * 16 * PITCH + 2 * LD_BT * PITCH) * 2 + mt * 16 * (LD_BT + 4) * 4 + mt * 16 * (LD_BT + 8) * 2 + mt * 16 * 8;
+  }
+};
+
+template <int NT, int MT>
+__global__ void __launch_bounds__(LD_THREADS, (NT <= 4 || MT == 1) ? 2 : 1) latent_decode_kernel(const LatentDecodeParams p) {
+  using L = LatentDecodeSmem<NT>;
+  constexpr int KP = L::KP, PITCH = L::PITCH, M = MT * 16, SP = LD_BT + 4, PP = LD_BT + 8;
+  extern __shared__ __align__(16) uint8_t ld_smem[];
+  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(ld_smem);            // [M][PITCH]
+  __nv_bfloat16* sc = sq + M * PITCH;                                       // [2][LD_BT][PITCH]
+  float* ss = reinterpret_cast<float*>(sc + 2 * LD_BT * PITCH);             // [M][SP]
+  __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(ss + M * SP);        // [M][PP]
+  float* salpha = reinterpret_cast<float*>(sp + M * PP);                    // [M]
+  float* sl = salpha + M;                                                   // [M]
+  pdl_sync();
+  const int row = blockIdx.x, h0 = blockIdx.y * M, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = p.positions[row];
+  const bool live = p.slots[row] >= 0 && pos >= 0;
+  const int lo = (p.window > 0 && pos - p.window + 1 > 0) ? pos - p.window + 1 : 0;
+  const int n = live ? pos - lo + 1 : 0;
+  const int per = ((n + p.splits - 1) / p.splits + LD_BT - 1) / LD_BT * LD_BT;
+  const int t0 = lo + split * per;
+  const int t1 = min(lo + n, t0 + per);
+  const int tiles = t1 > t0 ? (t1 - t0 + LD_BT - 1) / LD_BT : 0;
+  const int vecs = p.width / 8;                                             // 16-byte pieces of a latent
+  const int* table = p.tables + (long long)row * p.max_pages;
+
+  for (int i = threadIdx.x; i < M * (KP / 8); i += LD_THREADS) {            // queries, zero beyond heads and width
+    const int r = i / (KP / 8), v = i - r * (KP / 8);
+    uint4 val = make_uint4(0, 0, 0, 0);
+    if (h0 + r < p.heads && v < vecs)
+      val = *reinterpret_cast<const uint4*>(p.q + ((long long)row * p.heads + h0 + r) * p.width + v * 8);
+    *reinterpret_cast<uint4*>(sq + r * PITCH + v * 8) = val;
+  }
+  if (p.width < KP) {                                                       // pad columns of the ring stay zero
+    for (int i = threadIdx.x; i < 2 * LD_BT * (KP / 8 - vecs); i += LD_THREADS) {
+      const int r = i / (KP / 8 - vecs), v = vecs + i - r * (KP / 8 - vecs);
+      *reinterpret_cast<uint4*>(sc + r * PITCH + v * 8) = make_uint4(0, 0, 0, 0);
+    }
+  }
+  auto request = [&](int tile) {
+    __nv_bfloat16* dst = sc + (tile & 1) * LD_BT * PITCH;
+    const int first = t0 + tile * LD_BT + warp * 8;
+    // lanes 0-7 look up the cache row of one token each
+    long long src = -1;
+    const int t = first + (lane & 7);
+    if (t < t1) {
+      const int pg = t / p.page_size;
+      const int page = pg < p.max_pages ? table[pg] : -1;
+      if ((unsigned)page < (unsigned)p.num_pages) src = (long long)page * p.page_size + t % p.page_size;
+      else report_bad_arg(p.status, 9);
+    }
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const long long s = __shfl_sync(0xffffffffu, src, r);
+      __nv_bfloat16* d = dst + (warp * 8 + r) * PITCH;
+      for (int v = lane; v < vecs; v += 32) {
+        if (s >= 0) cp_async16(smem_u32(d + v * 8), p.cache + s * p.width + v * 8);
+        else *reinterpret_cast<uint4*>(d + v * 8) = make_uint4(0, 0, 0, 0);  // past the end: finite, masked below
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+
+  float acc[MT][NT * 2][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int j = 0; j < NT * 2; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[m][j][i] = 0.f;
+  float m_run[MT], l_run[MT];              // of head row (threadIdx.x / 8) + 16 m, the same in its 8 threads
+#pragma unroll
+  for (int m = 0; m < MT; ++m) { m_run[m] = -INFINITY; l_run[m] = 0.f; }
+
+  if (tiles > 0) request(0);
+  for (int it = 0; it < tiles; ++it) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                       // tile `it` is in shared memory, everybody is done with tile it - 1
+    if (it + 1 < tiles) request(it + 1);
+    const __nv_bfloat16* c = sc + (it & 1) * LD_BT * PITCH;
+    // ---- scores of this warp's 8 tokens, all heads
+    float s[MT][2][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[m][u][i] = 0.f;
+    const uint32_t b_addr = smem_u32(c + (warp * 8 + (lane & 7)) * PITCH + (lane >> 3) * 8);
+    const uint32_t a_addr = smem_u32(sq + ((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + (lane >> 4) * 8);
+#pragma unroll 4
+    for (int k = 0; k < KP / 32; ++k) {
+      uint32_t b[4];
+      ldsm_x4(b, b_addr + k * 64);
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        uint32_t a[4];
+        ldsm_x4(a, a_addr + m * 16 * PITCH * 2 + k * 64);
+        mma_bf16(s[m][0], a, b[0], b[1]);
+        ldsm_x4(a, a_addr + m * 16 * PITCH * 2 + k * 64 + 32);
+        mma_bf16(s[m][1], a, b[2], b[3]);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const int r = m * 16 + (lane >> 2), col = warp * 8 + (lane & 3) * 2;
+      const int tok = t0 + it * LD_BT + col;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float v = (s[m][0][i] + s[m][1][i]) * p.scale_log2;
+        ss[(r + (i >> 1) * 8) * SP + col + (i & 1)] = (tok + (i & 1) < t1) ? v : -INFINITY;
+      }
+    }
+    __syncthreads();
+    // ---- online softmax: eight threads per head row
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const int r = m * 16 + (threadIdx.x >> 3), e = (threadIdx.x & 7) * 4;
+      const float4 v = *reinterpret_cast<const float4*>(ss + r * SP + e);
+      float mx = fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w));
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float mn = fmaxf(m_run[m], mx);            // finite: every tile holds at least one token
+      const float p0 = exp2f(v.x - mn), p1 = exp2f(v.y - mn), p2 = exp2f(v.z - mn), p3 = exp2f(v.w - mn);
+      float sum = (p0 + p1) + (p2 + p3);
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      const float alpha = exp2f(m_run[m] - mn);
+      l_run[m] = l_run[m] * alpha + sum;
+      m_run[m] = mn;
+      *reinterpret_cast<uint2*>(sp + r * PP + e) = make_uint2(pack_bf16x2(p0, p1), pack_bf16x2(p2, p3));
+      if ((threadIdx.x & 7) == 0) salpha[r] = alpha;
+    }
+    __syncthreads();
+    // ---- O = alpha O + P C for this warp's quarter of the columns
+    const uint32_t v_addr = smem_u32(c + ((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + warp * (NT * 16) + (lane >> 4) * 8);
+    const uint32_t p_addr = smem_u32(sp + ((lane & 7) + ((lane >> 3) & 1) * 8) * PP + (lane >> 4) * 8);
+    uint32_t a[MT][LD_BT / 16][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float a0 = salpha[m * 16 + (lane >> 2)], a1 = salpha[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+      for (int j = 0; j < NT * 2; ++j) {
+        acc[m][j][0] *= a0; acc[m][j][1] *= a0; acc[m][j][2] *= a1; acc[m][j][3] *= a1;
+      }
+#pragma unroll
+      for (int k = 0; k < LD_BT / 16; ++k) ldsm_x4(a[m][k], p_addr + m * 16 * PP * 2 + k * 32);
+    }
+#pragma unroll
+    for (int k = 0; k < LD_BT / 16; ++k)
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        uint32_t b[4];
+        ldsm_x4_t(b, v_addr + k * 16 * PITCH * 2 + j * 32);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_bf16(acc[m][2 * j], a[m][k], b[0], b[1]);
+          mma_bf16(acc[m][2 * j + 1], a[m][k], b[2], b[3]);
+        }
+      }
+  }
+  // ---- results: normalised here, or left as (max, sum, unnormalised output) for the merge
+#pragma unroll
+  for (int m = 0; m < MT; ++m) {
+    const int r = m * 16 + (threadIdx.x >> 3);
+    if ((threadIdx.x & 7) == 0) {
+      sl[r] = l_run[m];
+      if (p.splits > 1 && h0 + r < p.heads) {
+        float* ml = p.part_ml + (((long long)row * p.heads + h0 + r) * p.splits + split) * 2;
+        ml[0] = m_run[m];
+        ml[1] = l_run[m];
+      }
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = m * 16 + (lane >> 2) + half * 8;
+      if (h0 + r >= p.heads) continue;
+      const float inv = sl[r] > 0.f ? 1.f / sl[r] : 0.f;
+#pragma unroll
+      for (int j = 0; j < NT * 2; ++j) {
+        const int col = warp * (NT * 16) + j * 8 + (lane & 3) * 2;
+        if (col >= p.width) continue;
+        const float x = acc[m][j][half * 2], y = acc[m][j][half * 2 + 1];
+        if (p.splits > 1)
+          *reinterpret_cast<float2*>(p.part_o + (((long long)row * p.heads + h0 + r) * p.splits + split) * p.width + col) =
+              make_float2(x, y);
+        else
+          *reinterpret_cast<uint32_t*>(p.o + ((long long)row * p.heads + h0 + r) * p.width + col) = pack_bf16x2(x * inv, y * inv);
+      }
+    }
+}
+
+__global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                           __nv_bfloat16* __restrict__ o, int splits, int width) {
+  pdl_sync();
+  const long long base = (long long)blockIdx.x * splits;          // (row, head)
+  float gm = -INFINITY;
+  for (int s = 0; s < splits; ++s) gm = fmaxf(gm, part_ml[(base + s) * 2]);
+  float gl = 0.f;
+  for (int s = 0; s < splits; ++s) {
+    const float ms = part_ml[(base + s) * 2];
+    gl += ms == -INFINITY ? 0.f : part_ml[(base + s) * 2 + 1] * exp2f(ms - gm);
+  }
+  const float inv = gl > 0.f ? 1.f / gl : 0.f;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    float v = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float ms = part_ml[(base + s) * 2];
+      if (ms != -INFINITY) v += part_o[(base + s) * width + c] * exp2f(ms - gm);
+    }
+    o[(long long)blockIdx.x * width + c] = __float2bfloat16(v * inv);
+  }
+}
+
+template <int NT, int MT>
+static int launch_latent_decode(const LatentDecodeParams& p, cudaStream_t st) {
+  constexpr int smem = LatentDecodeSmem<NT>::bytes(MT);
+  auto kern = latent_decode_kernel<NT, MT>;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
+    configured = true;
+  }
+  launch_dep(kern, dim3(p.rows, (p.heads + MT * 16 - 1) / (MT * 16), p.splits), LD_THREADS, smem, st, p);
+  if (p.splits > 1)
+    launch_dep(latent_merge_kernel, p.rows * p.heads, 128, 0, st, p.part_o, p.part_ml, p.o, p.splits, p.width);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -176,4 +463,26 @@ extern "C" int b200_latent_attn_rows(const void* q, const void* cache, void* o, 
                max_pages, page_size, num_pages, window, scale, status);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// Decode on the tensor cores: bf16, one query row per line of the tables, width a multiple of 8 up to 512.  splits > 1 needs
+// part_o (rows * heads * splits * width floats) and part_ml (rows * heads * splits * 2 floats).
+extern "C" int b200_latent_decode(const void* q, const void* cache, void* o, float* part_o, float* part_ml,
+                                  const int* positions, const long long* slots, const int* tables, int rows, int heads,
+                                  int width, int max_pages, int page_size, int num_pages, int window, int splits,
+                                  float scale, uint32_t* status, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (width % 8 || width <= 0 || width > 512 || heads <= 0 || page_size <= 0 || splits < 1 || splits > 65535) return -10;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(o)) & 15) return -10;
+  if (splits > 1 && (part_o == nullptr || part_ml == nullptr)) return -11;
+  LatentDecodeParams p;
+  p.q = (const __nv_bfloat16*)q; p.cache = (const __nv_bfloat16*)cache; p.o = (__nv_bfloat16*)o;
+  p.part_o = part_o; p.part_ml = part_ml; p.positions = positions; p.slots = slots; p.tables = tables;
+  p.rows = rows; p.heads = heads; p.width = width; p.max_pages = max_pages; p.page_size = page_size;
+  p.num_pages = num_pages; p.window = window; p.splits = splits; p.scale_log2 = scale * 1.4426950408889634f;
+  p.status = status;
+  const bool wide = heads > 16;
+  if (width <= 128) return wide ? launch_latent_decode<2, 2>(p, st) : launch_latent_decode<2, 1>(p, st);
+  if (width <= 256) return wide ? launch_latent_decode<4, 2>(p, st) : launch_latent_decode<4, 1>(p, st);
+  return wide ? launch_latent_decode<8, 2>(p, st) : launch_latent_decode<8, 1>(p, st);
 }

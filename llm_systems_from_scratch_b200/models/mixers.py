@@ -50,7 +50,7 @@ class LatentAttention:
         pack = lambda t: mo.padded_weight(t, dtype, device)
         # the tensor-core prefill takes heads of 64 or 128; elsewhere a head only has to start on a 16-byte boundary
         self.flash_dim = 0 if max(dim, vdim) > 128 else (64 if max(dim, vdim) <= 64 else 128)
-        if dtype != torch.bfloat16 or torch.device(device).type != "cuda":
+        if dtype != torch.bfloat16 or torch.device(device).type != "cuda" or scale <= 0:
             self.flash_dim = 0
         self.qdim = self.flash_dim or mo.pitch(dim)
         self.w_in = pack(torch.cat((dq, dkv, g)))
@@ -81,16 +81,27 @@ class LatentAttention:
         gate = proj[:, self.q_rank + self.kv_rank:]
         o = mo.rows_buffer(h.shape[0], heads * self.vdim, h.dtype, h.device)
         if n:
-            self._rows(q[:n], gate[:n], o[:n], batch, cache, slice(0, n))
+            ql = mo.gemm_heads(q[:n], self.w_ukt, heads, self.qdim, self.latent)
+            ol = mo.latent_decode(ql, cache, batch.positions[:n], batch.slots[:n], batch.tables[:n], heads, self.window, self.scale)
+            mo.gemm_heads(ol, self.w_uv, heads, self.latent, self.vdim, out=o[:n], gate=gate[:n])
         if batch.n_rows > n:
-            self._rows(q[n:], gate[n:], o[n:], batch, cache, slice(n, batch.n_rows))
+            self._portions(q[n:], gate[n:], o[n:], batch, cache, slice(n, batch.n_rows))
         mo.linear(o, self.w_o, out=x, accumulate=True)
 
-    def _rows(self, q, gate, o, batch, cache, rows: slice):
-        ql = mo.gemm_heads(q, self.w_ukt, self.heads, self.qdim, self.latent)
+    def _portions(self, q, gate, o, batch, cache, rows: slice):
+        heads = self.heads
+        if self.flash_dim:
+            # keys and values of everything the portions can see, expanded from the cached latents
+            cu_k, first, total, _ = batch.key_ranges(self.window)
+            c = mo.latent_gather(cache, cu_k, first, batch.tables[batch.n_single:], total)
+            kv = mo.linear(c, self.w_ukv)
+            mo.window_attention(q, kv, batch.cu, cu_k, batch.max_portion, heads, self.flash_dim, self.vdim, self.window,
+                                self.scale, o, gate)
+            return
+        ql = mo.gemm_heads(q, self.w_ukt, heads, self.qdim, self.latent)
         ol = mo.latent_attention_rows(ql, cache, batch.row_seq[rows], batch.positions[rows], batch.slots[rows], batch.tables,
-                                      self.heads, self.window, self.scale)
-        mo.gemm_heads(ol, self.w_uv, self.heads, self.latent, self.vdim, out=o, gate=gate)
+                                      heads, self.window, self.scale)
+        mo.gemm_heads(ol, self.w_uv, heads, self.latent, self.vdim, out=o, gate=gate)
 
 
 class Retention:

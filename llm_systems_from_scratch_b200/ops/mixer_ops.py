@@ -33,6 +33,8 @@ def _lib():
             "b200_latent_norm_append": [P, L, P, P, P, L, P, P, I, I, I, I, L, F, I, P, P],
             "b200_latent_gather": [P, P, P, P, P, I, I, I, I, I, I, P, P],
             "b200_latent_attn_rows": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
+            "b200_latent_decode": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
+            "b200_flash_window_fwd": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, L, L, L, L, P, P],
             "b200_retention_recurrent": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
         }.items():
             fn = getattr(lib, name)
@@ -247,6 +249,64 @@ def latent_attention_rows(q, cache, row_seq, positions, slots, tables, heads: in
                                         _ptr(tables), tables.shape[0], q.shape[0], heads, cache.shape[-1], tables.shape[1],
                                         cache.shape[1], cache.shape[0], window, float(scale), _f32(q),
                                         _ptr(native.status_word(q.device)), _stream()), "latent_attn_rows")
+    return out
+
+
+DECODE_MAX_WIDTH = 512           # latents the tensor-core decode kernel holds in shared memory
+DECODE_TILE = 32
+
+
+def latent_splits(rows: int, heads: int, keys: int, sms: int = 148) -> int:
+    """Splits of the window per row of a decode step: two CTAs fit on an SM, and a CTA should have a few tiles to walk."""
+    groups = rows * -(-heads // (16 if heads <= 16 else 32))
+    most = max(1, keys // (4 * DECODE_TILE))
+    return max(1, min(most, -(-2 * sms // groups)))
+
+
+def latent_decode(q, cache, positions, slots, tables, heads: int, window: int, scale: float, splits: int = 0):
+    """``latent_attention_rows`` for one query row per request: line i of ``tables`` belongs to row i."""
+    width = cache.shape[-1]
+    if not q.is_cuda or q.dtype != torch.bfloat16 or width > DECODE_MAX_WIDTH:
+        return latent_attention_rows(q, cache, None, positions, slots, tables, heads, window, scale)
+    rows = q.shape[0]
+    _req(q.is_contiguous() and cache.is_contiguous() and q.shape[1] == heads * width and tables.shape[0] >= rows, "bad latent queries")
+    _req(tables.dtype == torch.int32 and tables.is_contiguous() and positions.dtype == torch.int32, "bad tables")
+    page = cache.shape[1]
+    keys = tables.shape[1] * page
+    splits = splits or latent_splits(rows, heads, min(window, keys) if window > 0 else keys)
+    out = torch.empty_like(q)
+    part = torch.empty(rows * heads * splits * (width + 2) if splits > 1 else 0, dtype=torch.float32, device=q.device)
+    ml = part[rows * heads * splits * width:]
+    _check(_lib().b200_latent_decode(_ptr(q), _ptr(cache), _ptr(out), _ptr(part), _ptr(ml), _ptr(positions), _ptr(slots),
+                                     _ptr(tables), rows, heads, width, tables.shape[1], page, cache.shape[0], window, splits,
+                                     float(scale), _ptr(native.status_word(q.device)), _stream()),
+           "latent_decode" if splits > 1 else "latent_decode_one")
+    return out
+
+
+def latent_gather(cache, cu_k, first_k, tables, total: int):
+    """Cached latents of the keys a step's portions can see, packed (total, width): rows cu_k[b] .. of portion b start at
+    position first_k[b]."""
+    width = cache.shape[-1]
+    out = torch.empty((total, width), dtype=cache.dtype, device=cache.device)
+    _req(cache.dtype == torch.bfloat16 and cache.is_contiguous() and tables.dtype == torch.int32 and tables.is_contiguous(), "bad cache")
+    _check(_lib().b200_latent_gather(_ptr(cache), _ptr(out), _ptr(cu_k), _ptr(first_k), _ptr(tables), cu_k.numel() - 1, total,
+                                     tables.shape[1], cache.shape[1], cache.shape[0], width,
+                                     _ptr(native.status_word(cache.device)), _stream()), "latent_gather")
+    return out
+
+
+def window_attention(q, kv, cu_q, cu_k, max_q: int, heads: int, head_dim: int, vdim: int, window: int, scale: float, out, gate=None):
+    """Softmax attention of packed portions under a sliding window on the tensor cores: q (Rq, heads * head_dim), kv (Rk, 2 *
+    heads * head_dim) = K | V with zero columns up to head_dim (64 or 128); the queries of a portion are the last
+    positions of its keys.  out (Rq, heads * vdim), times sigmoid(gate)."""
+    _req(q.dtype == torch.bfloat16 and kv.dtype == torch.bfloat16 and q.stride(1) == 1 and kv.stride(1) == 1, "bf16 queries and keys")
+    _req(q.shape[1] == heads * head_dim and kv.shape[1] == 2 * heads * head_dim and out.shape == (q.shape[0], heads * vdim), "bad shapes")
+    _req(cu_q.dtype == torch.int32 and cu_k.dtype == torch.int32 and cu_q.numel() == cu_k.numel(), "bad row offsets")
+    _check(_lib().b200_flash_window_fwd(
+        _ptr(q), _ptr(kv), _ptr(out), _ptr(gate), _ptr(cu_q), _ptr(cu_k), cu_q.numel() - 1, max_q, q.shape[0], kv.shape[0], heads,
+        head_dim, vdim, window, float(scale), q.stride(0), kv.stride(0), out.stride(0), 0 if gate is None else gate.stride(0),
+        _ptr(native.status_word(q.device)), _stream()), "flash_window_fwd")
     return out
 
 
