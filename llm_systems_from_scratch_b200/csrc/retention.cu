@@ -127,6 +127,377 @@ __global__ void __launch_bounds__(256) retention_recurrent_kernel(const Retentio
   }
 }
 
+// ------------------------------------------------------------------------------------ prompts, bf16, on the tensor cores
+// One CTA = one (portion, head), chunks of n <= 128 tokens in order.  With r the last row of a chunk, scale the rotated
+// rows in fp32:  q~_i = decay^(i-r) q_i,  k~_j = decay^(r-j) k_j  and let S' = decay^n S.  Then
+//     O = causal(Q~ K~^T) V + Q~ S',        S <- S' + K~^T V,
+// so the decays need no further work in the products.  What enters the recurrence keeps (close to) 32-bit precision:
+// q~, k~, the scores and S' are each split into two bf16 parts (hi + lo, 16 significant bits) and the products of the
+// parts are accumulated in fp32 (v is bf16 as projected); S itself stays fp32, in tensor memory between chunks.
+//   tensor memory: scores [0, 128)  O [128, 128 + EP)  S [256, 256 + EP)  P hi [384, 448)  P lo [448, 512)
+//   shared memory: Q~ hi, lo | K~ hi, lo | V | S' hi, lo, all 128-byte swizzled panels of 64 columns
+// K~ and V serve two products each in the same storage (K-major and MN-major descriptors).
+// Eight warps do the element-wise phases (two warps per 32 lanes of tensor memory, half of the columns each); one thread
+// issues the MMAs.  M3 (state) and Q~ S' run on the tensor pipe while the scores are masked and split.
+constexpr int RC_CHUNK = 128;
+constexpr int RC_THREADS = 256;
+
+template <int EP>
+struct RetChunkSmem {
+  static constexpr int TILE = 32768;                 // 128 rows x 128 columns of bf16: two panels
+  static constexpr int VT = EP / 64 * 16384;
+  static constexpr int OFF_QH = 0, OFF_QL = TILE, OFF_KH = 2 * TILE, OFF_KL = 3 * TILE;
+  static constexpr int OFF_V = 4 * TILE, OFF_SH = OFF_V + VT, OFF_SL = OFF_SH + VT;
+  static constexpr int OFF_RMS = OFF_SL + VT;        // [2][128] floats
+  static constexpr int OFF_POW = OFF_RMS + 1024;     // [129] floats
+  static constexpr int OFF_BAR = OFF_POW + 520;
+  static constexpr int TOTAL = OFF_BAR + 3 * 8 + 16 + 1024;
+};
+
+// 16-byte piece `c8` (8 columns) of row `r` in a tile of 64-column panels, 128-byte swizzle
+__device__ __forceinline__ uint32_t swz(int r, int c8) {
+  return (uint32_t)(c8 >> 3) * 16384u + (uint32_t)r * 128u + (uint32_t)(((c8 & 7) ^ (r & 7)) << 4);
+}
+
+// x = hi + lo with both parts bf16, eight values at a time
+__device__ __forceinline__ void split8(const float (&x)[8], uint4& hi, uint4& lo) {
+  uint32_t h[4], l[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    h[i] = pack_bf16x2(x[2 * i], x[2 * i + 1]);
+    const float2 b = unpack_bf16x2(h[i]);
+    l[i] = pack_bf16x2(x[2 * i] - b.x, x[2 * i + 1] - b.y);
+  }
+  hi = make_uint4(h[0], h[1], h[2], h[3]);
+  lo = make_uint4(l[0], l[1], l[2], l[3]);
+}
+__device__ __forceinline__ void unpack8f(const uint4& v, float (&f)[8]) {
+  const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y), c = unpack_bf16x2(v.z), d = unpack_bf16x2(v.w);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
+}
+
+template <int EP>
+__global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const RetentionParams p, const float* __restrict__ powers) {
+  using L = RetChunkSmem<EP>;
+  constexpr int HE = EP / 2;                          // columns of O and S that a thread handles
+  extern __shared__ uint8_t rc_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(rc_raw) + 1023) & ~uintptr_t(1023));
+  float* srms = reinterpret_cast<float*>(smem + L::OFF_RMS);
+  float* spow = reinterpret_cast<float*>(smem + L::OFF_POW);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR);
+  uint64_t *bar_a = bars, *bar_s = bars + 1, *bar_o = bars + 2;
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 3);
+  volatile uint32_t* abort_word = tmem_holder + 1;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+
+  if (tid == 0) {
+    for (int i = 0; i < 3; ++i) mbar_init(&bars[i], 1);
+    *abort_word = 0;
+    fence_barrier_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_holder, 512);
+    tmem_relinquish();
+  }
+  // columns beyond dim and vdim are never written again
+  for (int i = tid; i < (L::OFF_RMS >> 4); i += RC_THREADS) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
+  pdl_sync();
+  const int seq = blockIdx.x / p.heads, h = blockIdx.x - seq * p.heads;
+  const int D = p.dim, E = p.vdim;
+  for (int i = tid; i <= RC_CHUNK; i += RC_THREADS) spow[i] = powers[h * (RC_CHUNK + 1) + i];
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_holder;
+
+  const int row0 = p.cu[seq], rows = p.cu[seq + 1] - row0;
+  const int slot = p.state_slots[seq];
+  const bool live = slot >= 0 && slot < p.num_slots;
+  if (!live && slot >= p.num_slots && tid == 0) report_bad_arg(p.status, 10);
+  const int pos0 = rows > 0 ? p.positions[row0] : 0;
+  float* state = p.state + ((long long)(live ? slot : 0) * p.heads + h) * D * E;
+  const __nv_bfloat16* proj = reinterpret_cast<const __nv_bfloat16*>(p.proj) + (long long)row0 * p.ld_proj;
+  const __nv_bfloat16* gq = proj + h * D;
+  const __nv_bfloat16* gk = proj + p.heads * D + h * D;
+  const __nv_bfloat16* gv = proj + 2 * p.heads * D + h * E;
+  const __nv_bfloat16* gg = proj + 2 * p.heads * D + p.heads * E + h * E;
+  __nv_bfloat16* gy = reinterpret_cast<__nv_bfloat16*>(p.y) + (long long)row0 * p.ld_y + h * E;
+
+  const int quarter = warp & 3, half = warp >> 2;
+  const int r = quarter * 32 + lane;                  // this thread's row of tensor memory: a token, or a dim of S
+  const uint32_t lane_addr = uint32_t(quarter * 32) << 16;
+  const uint32_t tm_a = tmem + lane_addr, tm_o = tmem + 128 + lane_addr, tm_s = tmem + 256 + lane_addr,
+                 tm_p = tmem + 384 + lane_addr;
+  const int rot2 = p.rot / 2, n_rot = p.rot / 16, n_items = n_rot + (D - p.rot) / 8;
+  const float kscale = rsqrtf((float)D);
+  const int chunks = live ? (rows + RC_CHUNK - 1) / RC_CHUNK : 0;
+  bool ok = true;
+
+  // S' of the first chunk from the request's slot (the zero state at position 0)
+  auto publish_state = [&](const float (&s)[32], int c) {       // columns [half * HE + 32 c, + 32) of row r
+    uint32_t raw[32];
+#pragma unroll
+    for (int i = 0; i < 32; ++i) raw[i] = __float_as_uint(s[i]);
+    tmem_st_32x32(tm_s + half * HE + c * 32, raw);
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      float f[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] = s[q * 8 + i];
+      uint4 hi, lo;
+      split8(f, hi, lo);
+      const uint32_t at = swz(r, (half * HE + c * 32) / 8 + q);
+      *reinterpret_cast<uint4*>(smem + L::OFF_SH + at) = hi;
+      *reinterpret_cast<uint4*>(smem + L::OFF_SL + at) = lo;
+    }
+  };
+  if (chunks > 0) {
+    const float f = spow[min(rows, RC_CHUNK)];
+#pragma unroll 1
+    for (int c = 0; c < HE / 32; ++c) {
+      float s[32];
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        const int e = half * HE + c * 32 + i;
+        s[i] = (pos0 > 0 && r < D && e < E) ? state[(long long)r * E + e] * f : 0.f;
+      }
+      publish_state(s, c);
+    }
+    tmem_st_wait();
+  }
+
+  for (int ch = 0; ch < chunks; ++ch) {
+    const int t0 = ch * RC_CHUNK, n = min(RC_CHUNK, rows - t0);
+    // ---- q~, k~ (rotated, scaled, split) and v to shared memory; rows past the end are zero
+#pragma unroll 2
+    for (int idx = tid; idx < RC_CHUNK * n_items; idx += RC_THREADS) {
+      const int t = idx / n_items, it = idx - t * n_items;
+      const bool in = t < n;
+      const bool turn = it < n_rot;
+      const int d0 = turn ? it * 8 : p.rot + (it - n_rot) * 8;
+      const long long at = (long long)(t0 + t) * p.ld_proj + d0;
+      uint4 hi, lo;
+      float qa[8], qb[8], ka[8], kb[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) qa[i] = qb[i] = ka[i] = kb[i] = 0.f;
+      if (in) {
+        unpack8f(*reinterpret_cast<const uint4*>(gq + at), qa);
+        unpack8f(*reinterpret_cast<const uint4*>(gk + at), ka);
+        const float fq = 1.f / spow[n - 1 - t], fk = spow[n - 1 - t] * kscale;
+        if (turn) {
+          unpack8f(*reinterpret_cast<const uint4*>(gq + at + rot2), qb);
+          unpack8f(*reinterpret_cast<const uint4*>(gk + at + rot2), kb);
+          int pos = pos0 + t0 + t;
+          if (pos >= p.ctx) { report_bad_arg(p.status, 11); pos = 0; }
+          const float* cs = p.cos_sin + (long long)pos * rot2 + d0;
+          const float* sn = cs + (long long)p.ctx * rot2;
+          float c[8], s[8];
+#pragma unroll
+          for (int i = 0; i < 8; i += 4) {
+            const float4 c4 = *reinterpret_cast<const float4*>(cs + i), s4 = *reinterpret_cast<const float4*>(sn + i);
+            c[i] = c4.x; c[i + 1] = c4.y; c[i + 2] = c4.z; c[i + 3] = c4.w;
+            s[i] = s4.x; s[i + 1] = s4.y; s[i + 2] = s4.z; s[i + 3] = s4.w;
+          }
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const float q0 = qa[i], q1 = qb[i], k0 = ka[i], k1 = kb[i];
+            qa[i] = (q0 * c[i] - q1 * s[i]) * fq;
+            qb[i] = (q1 * c[i] + q0 * s[i]) * fq;
+            ka[i] = (k0 * c[i] - k1 * s[i]) * fk;
+            kb[i] = (k1 * c[i] + k0 * s[i]) * fk;
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) { qa[i] *= fq; ka[i] *= fk; }
+        }
+      }
+      const uint32_t o0 = swz(t, d0 / 8), o1 = swz(t, (d0 + rot2) / 8);
+      split8(qa, hi, lo);
+      *reinterpret_cast<uint4*>(smem + L::OFF_QH + o0) = hi;
+      *reinterpret_cast<uint4*>(smem + L::OFF_QL + o0) = lo;
+      split8(ka, hi, lo);
+      *reinterpret_cast<uint4*>(smem + L::OFF_KH + o0) = hi;
+      *reinterpret_cast<uint4*>(smem + L::OFF_KL + o0) = lo;
+      if (turn) {
+        split8(qb, hi, lo);
+        *reinterpret_cast<uint4*>(smem + L::OFF_QH + o1) = hi;
+        *reinterpret_cast<uint4*>(smem + L::OFF_QL + o1) = lo;
+        split8(kb, hi, lo);
+        *reinterpret_cast<uint4*>(smem + L::OFF_KH + o1) = hi;
+        *reinterpret_cast<uint4*>(smem + L::OFF_KL + o1) = lo;
+      }
+    }
+    const int vg = E / 8;
+#pragma unroll 4
+    for (int idx = tid; idx < RC_CHUNK * vg; idx += RC_THREADS) {
+      const int t = idx / vg, c8 = idx - t * vg;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (t < n) v = *reinterpret_cast<const uint4*>(gv + (long long)(t0 + t) * p.ld_proj + c8 * 8);
+      *reinterpret_cast<uint4*>(smem + L::OFF_V + swz(t, c8)) = v;
+    }
+    fence_proxy_async_smem();
+    tc_fence_before();
+    __syncthreads();
+
+    if (warp == 0 && elect_one()) {
+      tc_fence_after();
+      constexpr uint32_t id_qk = make_idesc_bf16(128, 128, false, false);
+      constexpr uint32_t id_xv = make_idesc_bf16(128, EP, false, true);
+      constexpr uint32_t id_kv = make_idesc_bf16(128, EP, true, true);
+      auto kmaj = [&](int off) { return make_smem_desc(smem_u32(smem + off), 16, 1024); };
+      auto mnmaj = [&](int off) { return make_smem_desc(smem_u32(smem + off), 16384, 1024); };
+      auto kstep = [](int k) { return (uint32_t)(((k / 4) * 16384 + (k % 4) * 32) >> 4); };
+      const uint64_t qh = kmaj(L::OFF_QH), ql = kmaj(L::OFF_QL), kh = kmaj(L::OFF_KH), kl = kmaj(L::OFF_KL);
+      const uint64_t v = mnmaj(L::OFF_V), sh = mnmaj(L::OFF_SH), sl = mnmaj(L::OFF_SL);
+      const uint64_t kht = mnmaj(L::OFF_KH), klt = mnmaj(L::OFF_KL);
+#pragma unroll
+      for (int part = 0; part < 3; ++part)             // scores = Qh Kh^T + Qh Kl^T + Ql Kh^T
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          umma_f16_ss(tmem, (part == 2 ? ql : qh) + kstep(k), (part == 1 ? kl : kh) + kstep(k), id_qk, (part | k) ? 1u : 0u);
+      umma_commit(bar_a);
+#pragma unroll
+      for (int part = 0; part < 3; ++part)             // O = Qh S'h + Qh S'l + Ql S'h
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          umma_f16_ss(tmem + 128, (part == 2 ? ql : qh) + kstep(k), (part == 1 ? sl : sh) + (uint32_t)(k * 128), id_xv,
+                      (part | k) ? 1u : 0u);
+#pragma unroll
+      for (int part = 0; part < 2; ++part)             // S = S' + Kh^T V + Kl^T V
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          umma_f16_ss(tmem + 256, (part ? klt : kht) + (uint32_t)(k * 128), v + (uint32_t)(k * 128), id_kv, 1u);
+      umma_commit(bar_s);
+    }
+    __syncwarp();
+    const uint32_t ph = ch & 1;
+    // ---- scores -> causal, split, back to tensor memory as the A operand of P V
+    if (!mbar_wait(bar_a, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
+    tc_fence_after();
+#pragma unroll 1
+    for (int c = 0; c < 2; ++c) {
+      uint32_t a[32];
+      const int k0 = half * 64 + c * 32;
+      tmem_ld_32x32(tm_a + k0, a);
+      tmem_ld_wait();
+      uint32_t hi[16], lo[16];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const float x = k0 + 2 * i <= r ? __uint_as_float(a[2 * i]) : 0.f;
+        const float y = k0 + 2 * i + 1 <= r ? __uint_as_float(a[2 * i + 1]) : 0.f;
+        hi[i] = pack_bf16x2(x, y);
+        const float2 b = unpack_bf16x2(hi[i]);
+        lo[i] = pack_bf16x2(x - b.x, y - b.y);
+      }
+      tmem_st_32x16(tm_p + half * 32 + c * 16, hi);
+      tmem_st_32x16(tm_p + 64 + half * 32 + c * 16, lo);
+    }
+    tmem_st_wait();
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 0 && elect_one()) {
+      tc_fence_after();
+      constexpr uint32_t id_xv = make_idesc_bf16(128, EP, false, true);
+      const uint64_t v = make_smem_desc(smem_u32(smem + L::OFF_V), 16384, 1024);
+#pragma unroll
+      for (int part = 0; part < 2; ++part)             // O += P V
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          umma_f16_ts(tmem + 128, tmem + 384 + part * 64 + k * 8, v + (uint32_t)(k * 128), id_xv, 1u);
+      umma_commit(bar_o);
+    }
+    __syncwarp();
+    // ---- state: keep it for the next chunk, or leave it in the slot after the last one
+    if (!mbar_wait(bar_s, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
+    tc_fence_after();
+    const bool last = ch + 1 == chunks;
+    const float f = last ? 1.f : spow[min(RC_CHUNK, rows - t0 - RC_CHUNK)];
+#pragma unroll 1
+    for (int c = 0; c < HE / 32; ++c) {
+      uint32_t raw[32];
+      tmem_ld_32x32(tm_s + half * HE + c * 32, raw);
+      tmem_ld_wait();
+      if (last) {
+        if (r < D && ok) {
+#pragma unroll
+          for (int q = 0; q < 8; ++q)
+            if (half * HE + c * 32 + q * 4 < E)          // vdim is a multiple of 8
+              *reinterpret_cast<float4*>(state + (long long)r * E + half * HE + c * 32 + q * 4) =
+                  make_float4(__uint_as_float(raw[q * 4]), __uint_as_float(raw[q * 4 + 1]), __uint_as_float(raw[q * 4 + 2]),
+                              __uint_as_float(raw[q * 4 + 3]));
+        }
+      } else {
+        float s[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) s[i] = __uint_as_float(raw[i]) * f;
+        publish_state(s, c);
+      }
+    }
+    tmem_st_wait();
+    // ---- output: root mean square of the head, gate, bf16
+    if (!mbar_wait(bar_o, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
+    tc_fence_after();
+    uint32_t o[HE / 32][32];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < HE / 32; ++c) tmem_ld_32x32(tm_o + half * HE + c * 32, o[c]);
+    tmem_ld_wait();
+#pragma unroll
+    for (int c = 0; c < HE / 32; ++c)
+#pragma unroll
+      for (int i = 0; i < 32; ++i) ss = fmaf(__uint_as_float(o[c][i]), __uint_as_float(o[c][i]), ss);
+    srms[half * 128 + r] = ss;                          // columns beyond vdim are zero
+    __syncthreads();
+    const float inv = rsqrtf((srms[r] + srms[128 + r]) / (float)E + p.eps);
+    if (r < n) {
+      const __nv_bfloat16* grow = gg + (long long)(t0 + r) * p.ld_proj + half * HE;
+      __nv_bfloat16* yrow = gy + (long long)(t0 + r) * p.ld_y + half * HE;
+#pragma unroll
+      for (int c = 0; c < HE / 32; ++c)
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          if (half * HE + c * 32 + q * 8 >= E) continue;
+          float g[8];
+          unpack8f(*reinterpret_cast<const uint4*>(grow + c * 32 + q * 8), g);
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            g[i] = __uint_as_float(o[c][q * 8 + i]) * inv * __fdividef(g[i], 1.f + __expf(-g[i]));
+          *reinterpret_cast<uint4*>(yrow + c * 32 + q * 8) =
+              make_uint4(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]), pack_bf16x2(g[4], g[5]), pack_bf16x2(g[6], g[7]));
+        }
+    }
+    tc_fence_before();
+  }
+  if (!live) {
+    for (int t = tid / 32; t < rows; t += RC_THREADS / 32)
+      for (int c = lane * 8; c < E; c += 256) *reinterpret_cast<uint4*>(gy + (long long)t * p.ld_y + c) = make_uint4(0, 0, 0, 0);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (*abort_word != 0) {
+    if (tid == 0 && p.status != nullptr) atomicCAS(p.status, 0u, (*abort_word) | (blockIdx.x << 8));
+    const uint64_t w0 = globaltimer_ns();
+    while (globaltimer_ns() - w0 < 200000ull) __nanosleep(1000);
+    __syncthreads();
+  }
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 512);
+  }
+}
+
+template <int EP>
+static int launch_retention_chunk(const RetentionParams& p, const float* powers, cudaStream_t st) {
+  auto kern = retention_chunk_kernel<EP>;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, RetChunkSmem<EP>::TOTAL) != cudaSuccess) return -3;
+    configured = true;
+  }
+  launch_dep(kern, p.seqs * p.heads, RC_THREADS, RetChunkSmem<EP>::TOTAL, st, p, powers);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -159,4 +530,25 @@ extern "C" int b200_retention_recurrent(const void* proj, long long ld_proj, voi
     else launch_dep(retention_recurrent_kernel<__nv_bfloat16, 1>, grid, 256, smem, st, p);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// Prompts on the tensor cores (bf16): cu (seqs + 1) delimits the portions; `powers` (heads, 129) holds decay^m.  dim and vdim
+// multiples of 8 up to 128, rot a multiple of 16, and decay^127 must stay well inside the range of bf16 exponents.
+extern "C" int b200_retention_chunk(const void* proj, long long ld_proj, void* y, long long ld_y, float* state,
+                                    const int* state_slots, const int* cu, const int* positions, const float* cos_sin,
+                                    const float* powers, int seqs, int rows, int heads, int dim, int vdim, int rot, int ctx,
+                                    int num_slots, float eps, uint32_t* status, cudaStream_t st) {
+  if (seqs <= 0 || rows <= 0) return 0;
+  if (heads <= 0 || dim <= 0 || vdim <= 0 || dim > 128 || vdim > 128 || dim % 8 || vdim % 8 || rot % 16 || rot < 0 ||
+      rot > dim || cu == nullptr || powers == nullptr || (rot > 0 && cos_sin == nullptr))
+    return -10;
+  if (ld_proj % 8 || ld_y % 8 ||
+      (reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(state) |
+       reinterpret_cast<uintptr_t>(cos_sin)) & 15)
+    return -11;
+  RetentionParams p;
+  p.proj = proj; p.ld_proj = ld_proj; p.y = y; p.ld_y = ld_y; p.state = state; p.state_slots = state_slots; p.cu = cu;
+  p.positions = positions; p.cos_sin = cos_sin; p.decay = nullptr; p.seqs = seqs; p.rows = rows; p.heads = heads;
+  p.dim = dim; p.vdim = vdim; p.rot = rot; p.ctx = ctx; p.num_slots = num_slots; p.eps = eps; p.status = status;
+  return vdim <= 64 ? launch_retention_chunk<64>(p, powers, st) : launch_retention_chunk<128>(p, powers, st);
 }

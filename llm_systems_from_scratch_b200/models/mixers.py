@@ -108,6 +108,8 @@ class Retention:
     """Linear attention with a fixed decay per head, rotary q and k (rotate-half over the first ``rot_dims`` dimensions), no
     softmax; heads are divided by their root mean square, multiplied by silu(W_g h), then W_o.  The state is fp32."""
 
+    MIN_CHUNKED = 8            # the longest portion of a step from which the chunked kernel is used
+
     def __init__(self, get, width: int, heads: int, dim: int, vdim: int, decay, rot_dims: int, eps: float, rope, dtype, device):
         self.heads, self.dim, self.vdim, self.rot, self.eps = heads, dim, vdim, int(rot_dims), float(eps)
         if len(decay) != heads:
@@ -119,6 +121,9 @@ class Retention:
                                                 w("v", heads * vdim, width), w("g", heads * vdim, width))), dtype, device)
         self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
         self.decay = torch.tensor([float(d) for d in decay], dtype=torch.float32, device=device)
+        self.powers = None                     # for prompts on the tensor cores, where sizes and decays allow it
+        if torch.device(device).type == "cuda" and mo.chunkable(dtype, dim, vdim, self.rot):
+            self.powers = mo.retention_powers(decay, device)
         self.rope = rope                       # RotaryTable of the model's base and dims, None without rotation
 
     def cache_spec(self):
@@ -134,7 +139,10 @@ class Retention:
             self.rot, self.eps, y[rows])
         if n:
             run(slice(0, n), batch.state_slots[:n], None, [(i, i + 1) for i in range(n)] if not h.is_cuda else None)
-        if batch.n_rows > n:
+        if batch.n_rows > n and self.powers is not None and batch.max_portion >= self.MIN_CHUNKED:
+            mo.retention_chunked(proj[n:], state, batch.state_slots[n:], batch.cu, batch.positions[n:], table, self.powers,
+                                 self.heads, self.dim, self.vdim, self.rot, self.eps, y[n:])
+        elif batch.n_rows > n:
             run(slice(n, batch.n_rows), batch.state_slots[n:], batch.cu, batch.spans)
         mo.linear(y, self.w_o, out=x, accumulate=True)
 

@@ -35,6 +35,7 @@ def _lib():
             "b200_latent_attn_rows": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
             "b200_latent_decode": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
             "b200_flash_window_fwd": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, L, L, L, L, P, P],
+            "b200_retention_chunk": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
             "b200_retention_recurrent": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
         }.items():
             fn = getattr(lib, name)
@@ -311,6 +312,38 @@ def window_attention(q, kv, cu_q, cu_k, max_q: int, heads: int, head_dim: int, v
 
 
 # --------------------------------------------------------------------------------------- retention
+CHUNK = 128                      # tokens per chunk of the tensor-core prompt kernel
+
+
+def retention_powers(decay, device):
+    """decay^m for m = 0 .. CHUNK per head, (heads, CHUNK + 1) fp32 rounded from double, for ``retention_chunked``; None when
+    a head forgets so fast that a chunk's powers would leave the range the kernel's scaled rows can have."""
+    d = torch.tensor([float(x) for x in decay], dtype=torch.float64)
+    if len(d) == 0 or float(d.min()) < 2.0 ** (-40.0 / (CHUNK - 1)) or float(d.max()) > 2.0 ** (40.0 / (CHUNK - 1)):
+        return None
+    return (d[:, None] ** torch.arange(CHUNK + 1, dtype=torch.float64)).float().contiguous().to(device)
+
+
+def chunkable(dtype, dim: int, vdim: int, rot: int) -> bool:
+    return dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and vdim <= 128 and rot % 16 == 0
+
+
+def retention_chunked(proj, state, state_slots, cu, positions, cos_sin, powers, heads: int, dim: int, vdim: int, rot: int,
+                      eps: float, y):
+    """``retention`` for portions of prompts on the tensor cores (bf16 projections, fp32 state and accumulation)."""
+    _req(chunkable(proj.dtype, dim, vdim, rot) and proj.is_cuda, "sizes the chunked kernel does not take")
+    _req(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, dim, vdim), "bad state")
+    _req(state_slots.dtype == torch.int32 and positions.dtype == torch.int32 and cu.dtype == torch.int32
+         and cu.numel() == state_slots.numel() + 1 and powers.shape == (heads, CHUNK + 1), "bad inputs")
+    _req(proj.shape[1] == 2 * heads * (dim + vdim) and y.shape == (proj.shape[0], heads * vdim) and y.dtype == proj.dtype, "bad shapes")
+    _check(_lib().b200_retention_chunk(
+        _ptr(proj), proj.stride(0), _ptr(y), y.stride(0), _ptr(state), _ptr(state_slots), _ptr(cu), _ptr(positions),
+        _ptr(cos_sin), _ptr(powers), state_slots.numel(), proj.shape[0], heads, dim, vdim, rot,
+        0 if rot == 0 else cos_sin.shape[1], state.shape[0], float(eps), _ptr(native.status_word(proj.device)), _stream()),
+        "retention_chunk")
+    return y
+
+
 def retention(proj, state, state_slots, cu, spans, positions, cos_sin, decay, heads: int, dim: int, vdim: int, rot: int,
               eps: float, y):
     """Retention over the rows of ``proj`` (q | k | v | gate).  ``cu`` (sequences + 1, int32) delimits the sequences, None
