@@ -136,7 +136,11 @@ def parse_args():
                          "(the switch adds the copies) instead of peer loads")
     ap.add_argument("--activation-checkpointing", choices=["config", "on", "off"], default="config",
                     help="per-block activation checkpointing: as the config names it (on for fsdp_7b), or forced")
-    ap.add_argument("--workload", choices=["train", "serve"], default="train")
+    ap.add_argument("--workload", choices=["train", "serve", "layers"], default="train",
+                    help="train (default) and serve: the headline metric; layers: the layered decoder (Tedirax) beside the "
+                         "TransformerLM at equal size, prompt and decode steps and every kernel, 1 GPU")
+    ap.add_argument("--layers-sizes", default="0.35b,1.3b,7b-8layers", help="layers: sizes to run, with commas between them")
+    ap.add_argument("--no-kernels", action="store_true", help="layers: whole steps only")
     ap.add_argument("--serving-requests", type=int, default=None,
                     help="requests of the Poisson trace per GPU (serve: default 1024; train: a short serving run of "
                          "this many requests is appended to the line, default 160, 0 = none)")
@@ -484,6 +488,26 @@ def run_reference(args, cfg, rank, local_rank, world):
                           "reference FusedAdamW (Triton), global-norm clip 1.0"), None
 
 
+def run_layers(args, local_rank, world):
+    """The layered decoder beside the closest model at equal size: one JSON line per size."""
+    if args.impl == "reference":
+        print(json.dumps({"impl": "reference", "workload": "layers", "unavailable": "the reference has no layered decoder"}))
+        return 0
+    if world > 1:
+        raise SystemExit("--workload layers runs on one GPU")
+    sys.path.insert(0, ROOT)
+    from llm_systems_from_scratch_b200.ops import bench_layers
+    for size in args.layers_sizes.split(","):
+        clocks = ClockSampler(local_rank)
+        clocks.start()
+        rec = next(bench_layers.run([size], args.steps, max(3, args.warmup), not args.no_kernels))
+        print(json.dumps({"metric": "layered_decoder_steps", "data": "synthetic", "dtype": "bf16", "steps": args.steps,
+                          "warmup": max(3, args.warmup), **rec, "clocks": clocks.stop(),
+                          "l2_policy": "steps: weights and caches larger than L2 are streamed every step; kernels: L2 replaced "
+                                       "between runs"}), flush=True)
+    return 0
+
+
 def main():
     args = parse_args()
     cfg = CONFIGS[args.config]
@@ -497,6 +521,8 @@ def main():
             return 0
         raise
     rank, local_rank, world = init_dist(args)
+    if args.workload == "layers":
+        return run_layers(args, local_rank, world)
     if args.workload == "serve":
         n_req = args.serving_requests if args.serving_requests is not None else 1024
         clocks = ClockSampler(local_rank) if rank == 0 else None

@@ -5,6 +5,9 @@
 
 namespace b200 {
 
+int make_tmap_bf16_2d(CUtensorMap* tm, const void* ptr, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_cols,
+                      uint32_t box_rows);
+
 struct RetentionParams {
   const void* proj;          // (rows, ld_proj): q | k | v | gate, heads contiguous inside each
   long long ld_proj;
@@ -137,10 +140,15 @@ __global__ void __launch_bounds__(256) retention_recurrent_kernel(const Retentio
 //   tensor memory: scores [0, 128)  O [128, 128 + EP)  S [256, 256 + EP)  P hi [384, 448)  P lo [448, 512)
 //   shared memory: Q~ hi, lo | K~ hi, lo | V | S' hi, lo, all 128-byte swizzled panels of 64 columns
 // K~ and V serve two products each in the same storage (K-major and MN-major descriptors).
-// Eight warps do the element-wise phases (two warps per 32 lanes of tensor memory, half of the columns each); one thread
-// issues the MMAs.  M3 (state) and Q~ S' run on the tensor pipe while the scores are masked and split.
+// Eight warps do the element-wise phases (two warps per 32 lanes of tensor memory, half of the columns each); a ninth
+// issues TMA and MMAs, so that Q~ S' and the state's product run while the scores are masked and split.  TMA brings q, k
+// and v of the next chunk while the outputs of this one are written: q and k land where their lo parts will be and are
+// rotated, scaled and split in place (with shared memory full there is no L1 left that would hold loads in flight).
 constexpr int RC_CHUNK = 128;
-constexpr int RC_THREADS = 256;
+constexpr int RC_WORKERS = 256;
+constexpr int RC_THREADS = RC_WORKERS + 32;
+
+__device__ __forceinline__ void worker_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }   // RC_WORKERS threads
 
 template <int EP>
 struct RetChunkSmem {
@@ -151,12 +159,18 @@ struct RetChunkSmem {
   static constexpr int OFF_RMS = OFF_SL + VT;        // [2][128] floats
   static constexpr int OFF_POW = OFF_RMS + 1024;     // [129] floats
   static constexpr int OFF_BAR = OFF_POW + 520;
-  static constexpr int TOTAL = OFF_BAR + 3 * 8 + 16 + 1024;
+  static constexpr int TOTAL = OFF_BAR + 4 * 8 + 16 + 1024;
 };
 
 // 16-byte piece `c8` (8 columns) of row `r` in a tile of 64-column panels, 128-byte swizzle
 __device__ __forceinline__ uint32_t swz(int r, int c8) {
   return (uint32_t)(c8 >> 3) * 16384u + (uint32_t)r * 128u + (uint32_t)(((c8 & 7) ^ (r & 7)) << 4);
+}
+
+__device__ __forceinline__ float silu_fast(float g) {      // g sigmoid(g) = g (1 + tanh(g / 2)) / 2
+  float t;
+  asm("tanh.approx.f32 %0, %1;" : "=f"(t) : "f"(0.5f * g));
+  return 0.5f * g * (1.f + t);
 }
 
 // x = hi + lo with both parts bf16, eight values at a time
@@ -177,7 +191,8 @@ __device__ __forceinline__ void unpack8f(const uint4& v, float (&f)[8]) {
 }
 
 template <int EP>
-__global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const RetentionParams p, const float* __restrict__ powers) {
+__global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const __grid_constant__ CUtensorMap tm_proj, const RetentionParams p,
+                                                                         const float* __restrict__ powers) {
   using L = RetChunkSmem<EP>;
   constexpr int HE = EP / 2;                          // columns of O and S that a thread handles
   extern __shared__ uint8_t rc_raw[];
@@ -185,26 +200,27 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
   float* srms = reinterpret_cast<float*>(smem + L::OFF_RMS);
   float* spow = reinterpret_cast<float*>(smem + L::OFF_POW);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR);
-  uint64_t *bar_a = bars, *bar_s = bars + 1, *bar_o = bars + 2;
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 3);
+  uint64_t *bar_a = bars, *bar_s = bars + 1, *bar_o = bars + 2, *bar_l = bars + 3;
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 4);
   volatile uint32_t* abort_word = tmem_holder + 1;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
   if (tid == 0) {
-    for (int i = 0; i < 3; ++i) mbar_init(&bars[i], 1);
+    for (int i = 0; i < 4; ++i) mbar_init(&bars[i], 1);
     *abort_word = 0;
     fence_barrier_init();
+    prefetch_tensormap(&tm_proj);
   }
   if (warp == 1) {
     tmem_alloc(tmem_holder, 512);
     tmem_relinquish();
   }
-  // columns beyond dim and vdim are never written again
   for (int i = tid; i < (L::OFF_RMS >> 4); i += RC_THREADS) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
   pdl_sync();
   const int seq = blockIdx.x / p.heads, h = blockIdx.x - seq * p.heads;
   const int D = p.dim, E = p.vdim;
   for (int i = tid; i <= RC_CHUNK; i += RC_THREADS) spow[i] = powers[h * (RC_CHUNK + 1) + i];
+  fence_proxy_async_smem();           // the zeros above come before what TMA writes
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -217,10 +233,8 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
   const int pos0 = rows > 0 ? p.positions[row0] : 0;
   float* state = p.state + ((long long)(live ? slot : 0) * p.heads + h) * D * E;
   const __nv_bfloat16* proj = reinterpret_cast<const __nv_bfloat16*>(p.proj) + (long long)row0 * p.ld_proj;
-  const __nv_bfloat16* gq = proj + h * D;
-  const __nv_bfloat16* gk = proj + p.heads * D + h * D;
-  const __nv_bfloat16* gv = proj + 2 * p.heads * D + h * E;
   const __nv_bfloat16* gg = proj + 2 * p.heads * D + p.heads * E + h * E;
+  if (tid == 0 && live && p.rot > 0 && rows > 0 && pos0 + rows > p.ctx) report_bad_arg(p.status, 11);
   __nv_bfloat16* gy = reinterpret_cast<__nv_bfloat16*>(p.y) + (long long)row0 * p.ld_y + h * E;
 
   const int quarter = warp & 3, half = warp >> 2;
@@ -251,7 +265,27 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
       *reinterpret_cast<uint4*>(smem + L::OFF_SL + at) = lo;
     }
   };
-  if (chunks > 0) {
+  const bool worker = warp < RC_WORKERS / 32;
+  // q, k, v of the chunk at row t: 64-column panels, swizzled like the operands; columns past the head are zeroed later
+  auto load_chunk = [&](int t) {
+    const int pd = (D + 63) / 64, pe = (E + 63) / 64;
+    mbar_expect_tx(bar_l, (uint32_t)(2 * pd + pe) * 16384u);
+    for (int i = 0; i < pd; ++i) {
+      tma_load_2d(smem + L::OFF_QL + i * 16384, &tm_proj, bar_l, h * D + i * 64, row0 + t);
+      tma_load_2d(smem + L::OFF_KL + i * 16384, &tm_proj, bar_l, p.heads * D + h * D + i * 64, row0 + t);
+    }
+    for (int i = 0; i < pe; ++i)
+      tma_load_2d(smem + L::OFF_V + i * 16384, &tm_proj, bar_l, 2 * p.heads * D + h * E + i * 64, row0 + t);
+  };
+  if (!worker && chunks > 0 && elect_one()) load_chunk(0);
+  __syncwarp();
+  // Row-wise work: a thread owns one 16-byte piece (or one pair of rotated pieces) of rows t, t + step, ...
+  const int vg = E / 8, v_step = RC_WORKERS / vg, v_t = tid / vg, v_c8 = tid - v_t * vg;
+  const bool v_on = v_t < v_step;
+  const int i_step = RC_WORKERS / n_items, i_t = tid / n_items, i_it = tid - i_t * n_items;
+  const bool i_turn = i_it < n_rot;
+  const int i_d0 = i_turn ? i_it * 8 : p.rot + (i_it - n_rot) * 8, i_d1 = i_turn ? i_d0 + rot2 : i_d0;
+  if (worker && chunks > 0) {
     const float f = spow[min(rows, RC_CHUNK)];
 #pragma unroll 1
     for (int c = 0; c < HE / 32; ++c) {
@@ -268,78 +302,67 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
 
   for (int ch = 0; ch < chunks; ++ch) {
     const int t0 = ch * RC_CHUNK, n = min(RC_CHUNK, rows - t0);
-    // ---- q~, k~ (rotated, scaled, split) and v to shared memory; rows past the end are zero
+    if (worker) {
+      // ---- q~, k~: rotated, scaled, split; rows past the end become zero
+      if (!mbar_wait(bar_l, ch & 1, abort_word)) { ok = false; *abort_word = ERR_WAIT_FULL; }
+      if (i_t < i_step) {
 #pragma unroll 2
-    for (int idx = tid; idx < RC_CHUNK * n_items; idx += RC_THREADS) {
-      const int t = idx / n_items, it = idx - t * n_items;
-      const bool in = t < n;
-      const bool turn = it < n_rot;
-      const int d0 = turn ? it * 8 : p.rot + (it - n_rot) * 8;
-      const long long at = (long long)(t0 + t) * p.ld_proj + d0;
-      uint4 hi, lo;
-      float qa[8], qb[8], ka[8], kb[8];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) qa[i] = qb[i] = ka[i] = kb[i] = 0.f;
-      if (in) {
-        unpack8f(*reinterpret_cast<const uint4*>(gq + at), qa);
-        unpack8f(*reinterpret_cast<const uint4*>(gk + at), ka);
-        const float fq = 1.f / spow[n - 1 - t], fk = spow[n - 1 - t] * kscale;
-        if (turn) {
-          unpack8f(*reinterpret_cast<const uint4*>(gq + at + rot2), qb);
-          unpack8f(*reinterpret_cast<const uint4*>(gk + at + rot2), kb);
-          int pos = pos0 + t0 + t;
-          if (pos >= p.ctx) { report_bad_arg(p.status, 11); pos = 0; }
-          const float* cs = p.cos_sin + (long long)pos * rot2 + d0;
-          const float* sn = cs + (long long)p.ctx * rot2;
+        for (int t = i_t; t < RC_CHUNK; t += i_step) {
           float c[8], s[8];
 #pragma unroll
-          for (int i = 0; i < 8; i += 4) {
-            const float4 c4 = *reinterpret_cast<const float4*>(cs + i), s4 = *reinterpret_cast<const float4*>(sn + i);
-            c[i] = c4.x; c[i + 1] = c4.y; c[i + 2] = c4.z; c[i + 3] = c4.w;
-            s[i] = s4.x; s[i + 1] = s4.y; s[i + 2] = s4.z; s[i + 3] = s4.w;
-          }
+          for (int i = 0; i < 8; ++i) { c[i] = 1.f; s[i] = 0.f; }
+          if (i_turn) {
+            const float* cs = p.cos_sin + (long long)min(pos0 + t0 + min(t, n - 1), p.ctx - 1) * rot2 + i_d0;
+            const float* sn = cs + (long long)p.ctx * rot2;
 #pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            const float q0 = qa[i], q1 = qb[i], k0 = ka[i], k1 = kb[i];
-            qa[i] = (q0 * c[i] - q1 * s[i]) * fq;
-            qb[i] = (q1 * c[i] + q0 * s[i]) * fq;
-            ka[i] = (k0 * c[i] - k1 * s[i]) * fk;
-            kb[i] = (k1 * c[i] + k0 * s[i]) * fk;
+            for (int i = 0; i < 8; i += 4) {
+              const float4 c4 = *reinterpret_cast<const float4*>(cs + i), s4 = *reinterpret_cast<const float4*>(sn + i);
+              c[i] = c4.x; c[i + 1] = c4.y; c[i + 2] = c4.z; c[i + 3] = c4.w;
+              s[i] = s4.x; s[i + 1] = s4.y; s[i + 2] = s4.z; s[i + 3] = s4.w;
+            }
           }
-        } else {
+          const float pw = t < n ? spow[n - 1 - t] : 1.f;
+          const float fq = t < n ? __fdividef(1.f, pw) : 0.f, fk = t < n ? pw * kscale : 0.f;
+          const uint32_t o0 = swz(t, i_d0 / 8), o1 = swz(t, i_d1 / 8);
+          auto put = [&](float f, int off_hi, int off_lo) {
+            float a[8], b2[8];
+            unpack8f(*reinterpret_cast<const uint4*>(smem + off_lo + o0), a);
+            unpack8f(*reinterpret_cast<const uint4*>(smem + off_lo + o1), b2);
 #pragma unroll
-          for (int i = 0; i < 8; ++i) { qa[i] *= fq; ka[i] *= fk; }
+            for (int i = 0; i < 8; ++i) {
+              const float x = a[i], z = b2[i];
+              a[i] = (x * c[i] - z * s[i]) * f;
+              b2[i] = (z * c[i] + x * s[i]) * f;
+            }
+            uint4 hi, lo;
+            split8(a, hi, lo);
+            *reinterpret_cast<uint4*>(smem + off_hi + o0) = hi;
+            *reinterpret_cast<uint4*>(smem + off_lo + o0) = lo;
+            if (i_turn) {
+              split8(b2, hi, lo);
+              *reinterpret_cast<uint4*>(smem + off_hi + o1) = hi;
+              *reinterpret_cast<uint4*>(smem + off_lo + o1) = lo;
+            }
+          };
+          put(fq, L::OFF_QH, L::OFF_QL);
+          put(fk, L::OFF_KH, L::OFF_KL);
         }
       }
-      const uint32_t o0 = swz(t, d0 / 8), o1 = swz(t, (d0 + rot2) / 8);
-      split8(qa, hi, lo);
-      *reinterpret_cast<uint4*>(smem + L::OFF_QH + o0) = hi;
-      *reinterpret_cast<uint4*>(smem + L::OFF_QL + o0) = lo;
-      split8(ka, hi, lo);
-      *reinterpret_cast<uint4*>(smem + L::OFF_KH + o0) = hi;
-      *reinterpret_cast<uint4*>(smem + L::OFF_KL + o0) = lo;
-      if (turn) {
-        split8(qb, hi, lo);
-        *reinterpret_cast<uint4*>(smem + L::OFF_QH + o1) = hi;
-        *reinterpret_cast<uint4*>(smem + L::OFF_QL + o1) = lo;
-        split8(kb, hi, lo);
-        *reinterpret_cast<uint4*>(smem + L::OFF_KH + o1) = hi;
-        *reinterpret_cast<uint4*>(smem + L::OFF_KL + o1) = lo;
+      for (int c8 = D / 8 + (tid >> 7); c8 < 16; c8 += 2) {          // columns past dim and vdim: neighbours' data
+        const uint32_t at = swz(tid & 127, c8);
+        *reinterpret_cast<uint4*>(smem + L::OFF_QH + at) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(smem + L::OFF_QL + at) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(smem + L::OFF_KH + at) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(smem + L::OFF_KL + at) = make_uint4(0, 0, 0, 0);
       }
-    }
-    const int vg = E / 8;
-#pragma unroll 4
-    for (int idx = tid; idx < RC_CHUNK * vg; idx += RC_THREADS) {
-      const int t = idx / vg, c8 = idx - t * vg;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (t < n) v = *reinterpret_cast<const uint4*>(gv + (long long)(t0 + t) * p.ld_proj + c8 * 8);
-      *reinterpret_cast<uint4*>(smem + L::OFF_V + swz(t, c8)) = v;
+      for (int c8 = E / 8 + (tid >> 7); c8 < EP / 8; c8 += 2)
+        *reinterpret_cast<uint4*>(smem + L::OFF_V + swz(tid & 127, c8)) = make_uint4(0, 0, 0, 0);
     }
     fence_proxy_async_smem();
     tc_fence_before();
     __syncthreads();
 
-    if (warp == 0 && elect_one()) {
+    if (!worker && elect_one()) {
       tc_fence_after();
       constexpr uint32_t id_qk = make_idesc_bf16(128, 128, false, false);
       constexpr uint32_t id_xv = make_idesc_bf16(128, EP, false, true);
@@ -371,6 +394,14 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
     }
     __syncwarp();
     const uint32_t ph = ch & 1;
+    uint4 gate[EP / 16];
+    if (worker) {
+#pragma unroll
+      for (int j = 0; j < EP / 16; ++j) {
+        const int t = v_t + j * v_step;
+        gate[j] = make_uint4(0, 0, 0, 0);
+        if (v_on && t < n) gate[j] = *reinterpret_cast<const uint4*>(gg + (long long)(t0 + t) * p.ld_proj + v_c8 * 8);
+      }
     // ---- scores -> causal, split, back to tensor memory as the A operand of P V
     if (!mbar_wait(bar_a, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
     tc_fence_after();
@@ -394,8 +425,9 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
     }
     tmem_st_wait();
     tc_fence_before();
+    }
     __syncthreads();
-    if (warp == 0 && elect_one()) {
+    if (!worker && elect_one()) {
       tc_fence_after();
       constexpr uint32_t id_xv = make_idesc_bf16(128, EP, false, true);
       const uint64_t v = make_smem_desc(smem_u32(smem + L::OFF_V), 16384, 1024);
@@ -406,7 +438,14 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
           umma_f16_ts(tmem + 128, tmem + 384 + part * 64 + k * 8, v + (uint32_t)(k * 128), id_xv, 1u);
       umma_commit(bar_o);
     }
-    __syncwarp();
+    if (!worker) {
+      if (ch + 1 < chunks) {                            // every MMA of this chunk is done: its operands can be replaced
+        if (!mbar_wait(bar_o, ph, abort_word)) *abort_word = ERR_WAIT_MISC;
+        if (elect_one()) load_chunk(t0 + RC_CHUNK);
+      }
+      __syncwarp();
+      continue;
+    }
     // ---- state: keep it for the next chunk, or leave it in the slot after the last one
     if (!mbar_wait(bar_s, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
     tc_fence_after();
@@ -447,25 +486,37 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
 #pragma unroll
       for (int i = 0; i < 32; ++i) ss = fmaf(__uint_as_float(o[c][i]), __uint_as_float(o[c][i]), ss);
     srms[half * 128 + r] = ss;                          // columns beyond vdim are zero
-    __syncthreads();
+    worker_barrier();
     const float inv = rsqrtf((srms[r] + srms[128 + r]) / (float)E + p.eps);
-    if (r < n) {
-      const __nv_bfloat16* grow = gg + (long long)(t0 + r) * p.ld_proj + half * HE;
-      __nv_bfloat16* yrow = gy + (long long)(t0 + r) * p.ld_y + half * HE;
+    // rows -> columns through shared memory (the tiles of the hi parts are free now, each half of the columns in one), so
+    // that the gate and y move in whole rows
+    constexpr int PIECES = EP / 8;                      // 16-byte pieces of half an fp32 row
+    float4* stage = reinterpret_cast<float4*>(smem + (half ? L::OFF_KH : L::OFF_QH)) + r * PIECES;
 #pragma unroll
-      for (int c = 0; c < HE / 32; ++c)
+    for (int c = 0; c < HE / 32; ++c)
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          if (half * HE + c * 32 + q * 8 >= E) continue;
-          float g[8];
-          unpack8f(*reinterpret_cast<const uint4*>(grow + c * 32 + q * 8), g);
+      for (int q = 0; q < 8; ++q)
+        stage[(c * 8 + q) ^ (r & (PIECES - 1))] =
+            make_float4(__uint_as_float(o[c][q * 4]) * inv, __uint_as_float(o[c][q * 4 + 1]) * inv,
+                        __uint_as_float(o[c][q * 4 + 2]) * inv, __uint_as_float(o[c][q * 4 + 3]) * inv);
+    worker_barrier();
 #pragma unroll
-          for (int i = 0; i < 8; ++i)
-            g[i] = __uint_as_float(o[c][q * 8 + i]) * inv * __fdividef(g[i], 1.f + __expf(-g[i]));
-          *reinterpret_cast<uint4*>(yrow + c * 32 + q * 8) =
-              make_uint4(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]), pack_bf16x2(g[4], g[5]), pack_bf16x2(g[6], g[7]));
-        }
+    for (int j = 0; j < EP / 16; ++j) {
+      const int t = v_t + j * v_step;
+      if (!v_on || t >= n) continue;
+      const float4* from =
+          reinterpret_cast<const float4*>(smem + (2 * v_c8 < PIECES ? L::OFF_QH : L::OFF_KH)) + t * PIECES;
+      const int x = t & (PIECES - 1), pc = (2 * v_c8) & (PIECES - 1);
+      const float4 y0 = from[pc ^ x], y1 = from[(pc + 1) ^ x];
+      float g[8];
+      unpack8f(gate[j], g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) g[i] = silu_fast(g[i]);
+      *reinterpret_cast<uint4*>(gy + (long long)(t0 + t) * p.ld_y + v_c8 * 8) =
+          make_uint4(pack_bf16x2(y0.x * g[0], y0.y * g[1]), pack_bf16x2(y0.z * g[2], y0.w * g[3]),
+                     pack_bf16x2(y1.x * g[4], y1.y * g[5]), pack_bf16x2(y1.z * g[6], y1.w * g[7]));
     }
+    worker_barrier();
     tc_fence_before();
   }
   if (!live) {
@@ -487,14 +538,14 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const Re
 }
 
 template <int EP>
-static int launch_retention_chunk(const RetentionParams& p, const float* powers, cudaStream_t st) {
+static int launch_retention_chunk(const CUtensorMap& tm, const RetentionParams& p, const float* powers, cudaStream_t st) {
   auto kern = retention_chunk_kernel<EP>;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, RetChunkSmem<EP>::TOTAL) != cudaSuccess) return -3;
     configured = true;
   }
-  launch_dep(kern, p.seqs * p.heads, RC_THREADS, RetChunkSmem<EP>::TOTAL, st, p, powers);
+  launch_dep(kern, p.seqs * p.heads, RC_THREADS, RetChunkSmem<EP>::TOTAL, st, tm, p, powers);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -550,5 +601,7 @@ extern "C" int b200_retention_chunk(const void* proj, long long ld_proj, void* y
   p.proj = proj; p.ld_proj = ld_proj; p.y = y; p.ld_y = ld_y; p.state = state; p.state_slots = state_slots; p.cu = cu;
   p.positions = positions; p.cos_sin = cos_sin; p.decay = nullptr; p.seqs = seqs; p.rows = rows; p.heads = heads;
   p.dim = dim; p.vdim = vdim; p.rot = rot; p.ctx = ctx; p.num_slots = num_slots; p.eps = eps; p.status = status;
-  return vdim <= 64 ? launch_retention_chunk<64>(p, powers, st) : launch_retention_chunk<128>(p, powers, st);
+  CUtensorMap tm;
+  if (make_tmap_bf16_2d(&tm, proj, (uint64_t)rows, (uint64_t)2 * heads * (dim + vdim), (uint64_t)ld_proj, 64, RC_CHUNK)) return -20;
+  return vdim <= 64 ? launch_retention_chunk<64>(tm, p, powers, st) : launch_retention_chunk<128>(tm, p, powers, st);
 }

@@ -20,7 +20,7 @@ def _head_pad(w, heads: int, rows: int, to: int):
     """[heads * rows, in] -> [heads * to, in] with zero rows after each head's."""
     if rows == to:
         return w
-    out = torch.zeros((heads, to, w.shape[1]), dtype=w.dtype)
+    out = torch.zeros((heads, to, w.shape[1]), dtype=w.dtype, device=w.device)
     out[:, :rows] = w.view(heads, rows, -1)
     return out.view(heads * to, -1)
 
@@ -55,14 +55,14 @@ class LatentAttention:
         self.qdim = self.flash_dim or mo.pitch(dim)
         self.w_in = pack(torch.cat((dq, dkv, g)))
         self.w_uq = pack(_head_pad(uq, heads, dim, self.qdim))
-        ukt = torch.zeros((heads, self.latent, self.qdim), dtype=uk.dtype)        # q_h -> latent space: W_uk,h^T
+        ukt = torch.zeros((heads, self.latent, self.qdim), dtype=uk.dtype, device=uk.device)        # q_h -> latent space: W_uk,h^T
         ukt[:, :kv_rank, :dim] = uk.view(heads, dim, kv_rank).transpose(1, 2)
         self.w_ukt = pack(ukt.reshape(heads * self.latent, self.qdim))
-        uvp = torch.zeros((heads * vdim, self.latent), dtype=uv.dtype)
+        uvp = torch.zeros((heads * vdim, self.latent), dtype=uv.dtype, device=uv.device)
         uvp[:, :kv_rank] = uv
         self.w_uv = pack(uvp)
         if self.flash_dim:
-            kv = torch.zeros((2 * heads * self.flash_dim, self.latent), dtype=uk.dtype)
+            kv = torch.zeros((2 * heads * self.flash_dim, self.latent), dtype=uk.dtype, device=uk.device)
             kv[:heads * self.flash_dim, :kv_rank] = _head_pad(uk, heads, dim, self.flash_dim)
             kv[heads * self.flash_dim:, :kv_rank] = _head_pad(uv, heads, vdim, self.flash_dim)
             self.w_ukv = pack(kv)

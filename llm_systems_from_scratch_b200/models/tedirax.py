@@ -168,7 +168,7 @@ class Tedirax:
     @classmethod
     def random(cls, config: dict, seed: int = 0, dtype=torch.bfloat16, device="cuda") -> "Tedirax":
         """Random weights of the configuration's shapes (tests, benchmarks)."""
-        return cls(config, RandomTensors(config, seed), dtype, device)
+        return cls(config, RandomTensors(config, seed, device), dtype, device)
 
     def eval(self):
         return self
@@ -199,9 +199,9 @@ class Tedirax:
 class RandomTensors:
     """Weights made on demand: normal with variance 1 / fan-in, norms around one, experts drawn without repetition."""
 
-    def __init__(self, config: dict, seed: int = 0):
-        self.shapes = tensor_shapes(TediraxConfig.from_dict(config))
-        self.cfg, self.seed = TediraxConfig.from_dict(config), seed
+    def __init__(self, config: dict, seed: int = 0, device="cpu"):
+        self.cfg, self.seed, self.device = TediraxConfig.from_dict(config), seed, torch.device(device)
+        self.shapes = tensor_shapes(self.cfg)
         self._order = {name: i for i, name in enumerate(self.shapes)}
 
     def keys(self):
@@ -209,14 +209,15 @@ class RandomTensors:
 
     def __getitem__(self, name: str):
         shape = self.shapes[name]
-        g = torch.Generator().manual_seed(self.seed * 1000003 + self._order[name])
+        g = torch.Generator(self.device).manual_seed(self.seed * 1000003 + self._order[name])
+        kw = {"generator": g, "device": self.device}
         if name.endswith(".table"):
             experts = self.cfg.layers[int(name[1:].split(".")[0])].mlp["router"]["experts"]
-            return torch.rand((shape[0], experts), generator=g).argsort(1)[:, :shape[1]].to(torch.int32)
+            return torch.rand((shape[0], experts), **kw).argsort(1)[:, :shape[1]].to(torch.int32)
         if len(shape) == 1:
-            return (1.0 + 0.1 * torch.randn(shape, generator=g)).to(torch.bfloat16)
+            return (1.0 + 0.1 * torch.randn(shape, **kw)).to(torch.bfloat16)
         std = 1.0 if name == "embed" else shape[1] ** -0.5
-        return (std * torch.randn(shape, generator=g)).to(torch.bfloat16)
+        return (std * torch.randn(shape, **kw)).to(torch.bfloat16)
 
 
 def tensor_shapes(cfg: TediraxConfig) -> dict[str, tuple[int, ...]]:
