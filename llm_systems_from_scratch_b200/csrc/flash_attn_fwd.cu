@@ -30,6 +30,12 @@ __device__ __forceinline__ float fa_exp2(float x) {
   return y;
 }
 
+__device__ __forceinline__ float fa_sigmoid(float g) {     // (1 + tanh(g / 2)) / 2, one special-function instruction
+  float t;
+  asm("tanh.approx.f32 %0, %1;" : "=f"(t) : "f"(0.5f * g));
+  return fmaf(0.5f, t, 0.5f);
+}
+
 __device__ __forceinline__ float fmax3(float a, float b, float c) {
   float r;
   asm("max.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
@@ -314,6 +320,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
     float m_run = -INFINITY;                    // running reference max in scaled log2 units
     float l_run = 0.f;                          // running row sum relative to m_run
     bool ok = true;
+    if (WINDOW && p.gate != nullptr && q_idx < seq_len) {      // the epilogue's gate row into L2
+      const __nv_bfloat16* grow = p.gate + (long long)(row_base + q_idx) * p.ld_gate + h * p.vdim;
+      for (int i = 0; i < p.vdim; i += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(grow + i));
+    }
     for (int j = lo_x; j < n_kv_x; ++j) {
       const int trole = warp;
       FWD_TRACE(trole, j, 0);
@@ -326,7 +336,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
       // pass 1: row maximum over the raw scores (the softmax scale is positive, so it is applied afterwards).
       // The load of chunk c+1 is in flight while chunk c is reduced.
       float mx = -INFINITY;
-      {
+      // Key k0 + e is visible iff e - first <= span as unsigned numbers (one comparison for both edges of the window).
+      const int first = q_low + 1 - k0;
+      const uint32_t span = WINDOW ? (uint32_t)(p.window - 1) : 0u;
+      auto hidden = [&](int e) { return WINDOW ? (uint32_t)(e - first) > span : k0 + e > q_key; };
+      auto row_max = [&](const bool masked) __attribute__((always_inline)) {
         uint32_t sa[32], sb[32];
         tmem_ld_32x32(tm_s, sa);
         tmem_ld_wait();
@@ -335,15 +349,21 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
           uint32_t (&cur)[32] = (c & 1) ? sb : sa;
           uint32_t (&nxt)[32] = (c & 1) ? sa : sb;
           if (c + 1 < FA_BK / 32) tmem_ld_32x32(tm_s + (c + 1) * 32, nxt);
-          if (diag) {
+          if (masked) {
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              if (k0 + c * 32 + i > q_key || (WINDOW && k0 + c * 32 + i <= q_low)) cur[i] = 0xff800000u;   // -inf
+              if (hidden(c * 32 + i)) cur[i] = 0xff800000u;   // -inf
           }
 #pragma unroll
           for (int i = 0; i < 32; i += 2) mx = fmax3(mx, __uint_as_float(cur[i]), __uint_as_float(cur[i + 1]));
           if (c + 1 < FA_BK / 32) tmem_ld_wait();
         }
+      };
+      if (WINDOW) {                    // two copies: tiles inside the window pay nothing for its edges
+        if (diag) row_max(true);
+        else row_max(false);
+      } else {
+        row_max(diag);
       }
       mx *= p.scale_log2;
       FWD_TRACE(trole, j, 2);
@@ -371,7 +391,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
       // (a row whose window starts in a later tile has seen no key yet: every P is masked to zero below)
       const float m_ref = (WINDOW && m_new == -INFINITY) ? 0.f : m_new;
       float sum = 0.f, sum1 = 0.f;
-      {
+      auto weights = [&](const bool masked) __attribute__((always_inline)) {
         uint32_t sa[32], sb[32];
         tmem_ld_32x32(tm_s, sa);
         tmem_ld_wait();
@@ -387,10 +407,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
             fma2(x0, x1, __uint_as_float(s[i]), __uint_as_float(s[i + 1]), p.scale_log2, -m_ref);
             float e0 = ((i & 7) < FA_POLY_PER_8) ? fa_exp2_poly(x0) : fa_exp2(x0);
             float e1 = (((i + 1) & 7) < FA_POLY_PER_8) ? fa_exp2_poly(x1) : fa_exp2(x1);
-            if (diag) {
-              const int key = k0 + c * 32 + i;
-              e0 = (key > q_key || (WINDOW && key <= q_low)) ? 0.f : e0;
-              e1 = (key + 1 > q_key || (WINDOW && key + 1 <= q_low)) ? 0.f : e1;
+            if (masked) {
+              e0 = hidden(c * 32 + i) ? 0.f : e0;
+              e1 = hidden(c * 32 + i + 1) ? 0.f : e1;
             }
             add2(sum, sum1, e0, e1);
             pk[i / 2] = pack_bf16x2(e0, e1);
@@ -403,6 +422,12 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
             mbar_arrive(&p_full[2 * x + (c >> 1)]);
           }
         }
+      };
+      if (WINDOW) {
+        if (diag) weights(true);
+        else weights(false);
+      } else {
+        weights(diag);
       }
       l_run = l_run * (need ? alpha : 1.f) + (sum + sum1);
       m_run = m_new;
@@ -438,13 +463,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                   const float2 g2 = unpack_bf16x2(gg[i]);
-                  f[2 * i] = __fdividef(f[2 * i], 1.f + __expf(-g2.x));
-                  f[2 * i + 1] = __fdividef(f[2 * i + 1], 1.f + __expf(-g2.y));
+                  f[2 * i] *= fa_sigmoid(g2.x);
+                  f[2 * i + 1] *= fa_sigmoid(g2.y);
                 }
               } else if (grow != nullptr) {
 #pragma unroll
                 for (int i = 0; i < 8; ++i)
-                  if (q * 8 + i < n) f[i] = __fdividef(f[i], 1.f + __expf(-__bfloat162float(grow[q * 8 + i])));
+                  if (q * 8 + i < n) f[i] *= fa_sigmoid(__bfloat162float(grow[q * 8 + i]));
               }
               if (p.out_vec && q * 8 + 8 <= n) {
                 *reinterpret_cast<uint4*>(orow + c * 32 + q * 8) =

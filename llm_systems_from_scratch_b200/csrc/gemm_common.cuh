@@ -161,9 +161,25 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, int row, int
                         ((reinterpret_cast<uintptr_t>(p.C) & 15) == 0);
     if (p.epi == EPI_BF16_GATE) {
       const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.R) + (long long)row * p.ldr + coff + col0;
+      if (vec_ok && (p.ldr & 7) == 0 && (reinterpret_cast<uintptr_t>(p.R) & 15) == 0) {
 #pragma unroll
-      for (int j = 0; j < 32; ++j)
-        if (j < ncols) c[j] = __float2bfloat16(__uint_as_float(acc[j]) / (1.f + __expf(-__bfloat162float(r[j]))));
+        for (int j = 0; j < 4; ++j) {
+          const uint4 rv = *reinterpret_cast<const uint4*>(r + j * 8);
+          const uint32_t rr[4] = {rv.x, rv.y, rv.z, rv.w};
+          uint32_t o[4];
+#pragma unroll
+          for (int t = 0; t < 4; ++t) {
+            const float2 g = unpack_bf16x2(rr[t]);
+            o[t] = pack_bf16x2(__fdividef(__uint_as_float(acc[j * 8 + 2 * t]), 1.f + __expf(-g.x)),
+                               __fdividef(__uint_as_float(acc[j * 8 + 2 * t + 1]), 1.f + __expf(-g.y)));
+          }
+          *reinterpret_cast<uint4*>(c + j * 8) = make_uint4(o[0], o[1], o[2], o[3]);
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+          if (j < ncols) c[j] = __float2bfloat16(__fdividef(__uint_as_float(acc[j]), 1.f + __expf(-__bfloat162float(r[j]))));
+      }
     } else if (p.epi == EPI_BF16_RES) {
       const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.R) + (long long)row * p.ldr + coff + col0;
       const bool rvec = vec_ok && ((p.ldr & 7) == 0) && ((reinterpret_cast<uintptr_t>(p.R) & 15) == 0);

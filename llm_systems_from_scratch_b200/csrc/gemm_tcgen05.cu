@@ -246,7 +246,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const float g = __uint_as_float(r[j]);
-            r[j] = __float_as_uint(g / (1.f + __expf(-g)) * __uint_as_float(u[j]));
+            r[j] = __float_as_uint(__fdividef(g, 1.f + __expf(-g)) * __uint_as_float(u[j]));
           }
           epilogue_store(p, row, n0 + c * 32, r);
         }

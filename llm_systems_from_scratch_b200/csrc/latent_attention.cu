@@ -10,30 +10,65 @@ namespace b200 {
 
 // Row-wise norms of the two latents of a layer and the append to the cache:
 //   cq[row] = rms_norm(proj[row, 0 : q_rank]) * wq,   cache[slot[row]] = rms_norm(proj[row, q_rank : q_rank + kv_rank]) * wkv
-template <typename T>
+// One warp per row; the row is read twice (the second read hits L1).
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) latent_norm_append_kernel(
     const T* __restrict__ proj, long long ld_proj, const T* __restrict__ wq, const T* __restrict__ wkv, T* __restrict__ cq,
-    long long ld_cq, T* __restrict__ cache, const long long* __restrict__ slots, int q_rank, int kv_rank, int width,
+    long long ld_cq, T* __restrict__ cache, const long long* __restrict__ slots, int rows, int q_rank, int kv_rank, int width,
     long long num_slots, float eps, uint32_t* __restrict__ status) {
   pdl_sync();
-  __shared__ float red[32];
-  const int row = blockIdx.x;
+  const int lane = threadIdx.x & 31;
+  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (row >= rows) return;
   const T* pr = proj + (long long)row * ld_proj;
-  const long long slot = slots[row];
+  const T* pk = pr + q_rank;
   float sq = 0.f, skv = 0.f;
-  for (int c = threadIdx.x; c < q_rank; c += blockDim.x) { const float v = to_f(pr[c]); sq += v * v; }
-  for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) { const float v = to_f(pr[q_rank + c]); skv += v * v; }
-  const float rq = rsqrtf(block_total(sq, red) / (float)q_rank + eps);
-  const float rkv = rsqrtf(block_total(skv, red) / (float)kv_rank + eps);
+#pragma unroll 4
+  for (int c = lane * VEC; c < q_rank; c += 32 * VEC) {
+    float f[VEC];
+    load_vec<VEC>(pr + c, f);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) sq += f[i] * f[i];
+  }
+#pragma unroll 4
+  for (int c = lane * VEC; c < kv_rank; c += 32 * VEC) {
+    float f[VEC];
+    load_vec<VEC>(pk + c, f);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) skv += f[i] * f[i];
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    skv += __shfl_xor_sync(0xffffffffu, skv, o);
+  }
+  const float rq = rsqrtf(sq / (float)q_rank + eps), rkv = rsqrtf(skv / (float)kv_rank + eps);
   T* q = cq + (long long)row * ld_cq;
-  for (int c = threadIdx.x; c < q_rank; c += blockDim.x) from_f(q[c], to_f(pr[c]) * rq * to_f(wq[c]));
+#pragma unroll 4
+  for (int c = lane * VEC; c < q_rank; c += 32 * VEC) {
+    float f[VEC], g[VEC];
+    load_vec<VEC>(pr + c, f);
+    load_vec<VEC>(wq + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) f[i] = f[i] * rq * g[i];
+    store_vec<VEC>(q + c, f);
+  }
+  const long long slot = slots[row];
   if (slot < 0) return;                       // padding row of the batch
   if (slot >= num_slots) {
-    if (threadIdx.x == 0) report_bad_arg(status, 4);
+    if (lane == 0) report_bad_arg(status, 4);
     return;
   }
   T* dst = cache + slot * width;
-  for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) from_f(dst[c], to_f(pr[q_rank + c]) * rkv * to_f(wkv[c]));
+#pragma unroll 4
+  for (int c = lane * VEC; c < kv_rank; c += 32 * VEC) {
+    float f[VEC], g[VEC];
+    load_vec<VEC>(pk + c, f);
+    load_vec<VEC>(wkv + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) f[i] = f[i] * rkv * g[i];
+    store_vec<VEC>(dst + c, f);
+  }
 }
 
 // Latents of the keys that the portions of a step can see, packed for the prefill kernel:
@@ -116,13 +151,16 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(
 }
 
 // ------------------------------------------------------------------------------- decode, bf16, on the tensor cores
-// One CTA = one row (request), up to 16 * MT of its heads and one split of the window.  All heads share the cached latents,
+// One CTA = one row (request), up to 16 * HG of its heads and one split of the window.  All heads share the cached latents,
 // so the score and value products are (heads x width) by (width x tokens) and back: with 16 heads that is ~32 FLOP per
 // cached byte, too much for the FMA pipes but little for mma.sync at M = 16, and the kernel stays bound by reading the
-// cache.  Tiles of 32 tokens are copied by cp.async into a two-stage ring straight from the pages; four warps compute
-// 8 tokens' scores each, then own a quarter of the latent columns of the output.  The softmax is online, in fp32.
+// cache.  Tiles of 32 tokens are copied by cp.async into a three-stage ring straight from the pages; the eight warps of a
+// group of 16 heads compute 8 tokens' scores over half of the latent columns each (the softmax adds the halves), then own
+// an eighth of the latent columns of the output: many short chains of MMAs instead of few long ones.  The queries
+// stay in registers as MMA fragments, the page of a tile's tokens is looked up a tile earlier than its copy is issued, and
+// the softmax is online, in fp32.
 constexpr int LD_BT = 32;       // tokens per tile
-constexpr int LD_THREADS = 128;
+constexpr int LD_STAGES = 3;
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -165,25 +203,28 @@ template <int NT>
 struct LatentDecodeSmem {
   static constexpr int KP = NT * 64;            // latent columns, padded
   static constexpr int PITCH = KP + 8;          // an odd number of 16-byte pieces: ldmatrix without bank conflicts
-  static constexpr int bytes(int mt) {
-    return (mt * 16 * PITCH + 2 * LD_BT * PITCH) * 2 + mt * 16 * (LD_BT + 4) * 4 + mt * 16 * (LD_BT + 8) * 2 + mt * 16 * 8;
+  static constexpr int bytes(int hg) {
+    return LD_STAGES * LD_BT * PITCH * 2 + hg * 16 * (2 * (LD_BT + 4) * 4 + (LD_BT + 8) * 2 + 8);
   }
 };
 
-template <int NT, int MT>
-__global__ void __launch_bounds__(LD_THREADS, (NT <= 4 || MT == 1) ? 2 : 1) latent_decode_kernel(const LatentDecodeParams p) {
+template <int NT, int HG>
+__global__ void __launch_bounds__(256 * HG, HG == 1 ? 2 : 1) latent_decode_kernel(const LatentDecodeParams p) {
   using L = LatentDecodeSmem<NT>;
-  constexpr int KP = L::KP, PITCH = L::PITCH, M = MT * 16, SP = LD_BT + 4, PP = LD_BT + 8;
+  constexpr int KP = L::KP, PITCH = L::PITCH, M = HG * 16, SP = LD_BT + 4, PP = LD_BT + 8, THREADS = 256 * HG;
+  constexpr int ROWS = LD_BT / (8 * HG);                                    // token rows a warp copies per tile
   extern __shared__ __align__(16) uint8_t ld_smem[];
-  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(ld_smem);            // [M][PITCH]
-  __nv_bfloat16* sc = sq + M * PITCH;                                       // [2][LD_BT][PITCH]
-  float* ss = reinterpret_cast<float*>(sc + 2 * LD_BT * PITCH);             // [M][SP]
-  __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(ss + M * SP);        // [M][PP]
+  __nv_bfloat16* sc = reinterpret_cast<__nv_bfloat16*>(ld_smem);            // [LD_STAGES][LD_BT][PITCH]
+  float* ss = reinterpret_cast<float*>(sc + LD_STAGES * LD_BT * PITCH);     // [2][M][SP]
+  __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(ss + 2 * M * SP);        // [M][PP]
   float* salpha = reinterpret_cast<float*>(sp + M * PP);                    // [M]
   float* sl = salpha + M;                                                   // [M]
   pdl_sync();
-  const int row = blockIdx.x, h0 = blockIdx.y * M, split = blockIdx.z;
+  const int row = blockIdx.x, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int grp = warp >> 3, wq = warp & 7;                                 // group of 16 heads, warp inside it
+  const int tq = wq & 3, kh = wq >> 2;                                      // its 8 tokens, its half of the columns
+  const int h0 = blockIdx.y * M;
   const int pos = p.positions[row];
   const bool live = p.slots[row] >= 0 && pos >= 0;
   const int lo = (p.window > 0 && pos - p.window + 1 > 0) ? pos - p.window + 1 : 0;
@@ -195,174 +236,167 @@ __global__ void __launch_bounds__(LD_THREADS, (NT <= 4 || MT == 1) ? 2 : 1) late
   const int vecs = p.width / 8;                                             // 16-byte pieces of a latent
   const int* table = p.tables + (long long)row * p.max_pages;
 
-  for (int i = threadIdx.x; i < M * (KP / 8); i += LD_THREADS) {            // queries, zero beyond heads and width
-    const int r = i / (KP / 8), v = i - r * (KP / 8);
-    uint4 val = make_uint4(0, 0, 0, 0);
-    if (h0 + r < p.heads && v < vecs)
-      val = *reinterpret_cast<const uint4*>(p.q + ((long long)row * p.heads + h0 + r) * p.width + v * 8);
-    *reinterpret_cast<uint4*>(sq + r * PITCH + v * 8) = val;
-  }
+  // cache row of token (warp * ROWS + lane) of a tile, looked up by the first ROWS lanes; -1 = past the end
+  auto look_up = [&](int tile) -> long long {
+    const int t = t0 + tile * LD_BT + warp * ROWS + (lane & (ROWS - 1));
+    if (t >= t1) return -1;
+    const int pg = t / p.page_size;
+    const int page = pg < p.max_pages ? table[pg] : -1;
+    if ((unsigned)page < (unsigned)p.num_pages) return (long long)page * p.page_size + t % p.page_size;
+    report_bad_arg(p.status, 9);
+    return -1;
+  };
+  auto request = [&](int tile, long long src) {
+    __nv_bfloat16* dst = sc + (tile % LD_STAGES) * LD_BT * PITCH;
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+      const long long s = __shfl_sync(0xffffffffu, src, r);
+      __nv_bfloat16* d = dst + (warp * ROWS + r) * PITCH;
+      for (int v = lane; v < vecs; v += 32) {
+        if (s >= 0) cp_async16(smem_u32(d + v * 8), p.cache + s * p.width + v * 8);
+        else *reinterpret_cast<uint4*>(d + v * 8) = make_uint4(0, 0, 0, 0);  // finite; masked below
+      }
+    }
+  };
+  auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+
   if (p.width < KP) {                                                       // pad columns of the ring stay zero
-    for (int i = threadIdx.x; i < 2 * LD_BT * (KP / 8 - vecs); i += LD_THREADS) {
+    for (int i = threadIdx.x; i < LD_STAGES * LD_BT * (KP / 8 - vecs); i += THREADS) {
       const int r = i / (KP / 8 - vecs), v = vecs + i - r * (KP / 8 - vecs);
       *reinterpret_cast<uint4*>(sc + r * PITCH + v * 8) = make_uint4(0, 0, 0, 0);
     }
   }
-  auto request = [&](int tile) {
-    __nv_bfloat16* dst = sc + (tile & 1) * LD_BT * PITCH;
-    const int first = t0 + tile * LD_BT + warp * 8;
-    // lanes 0-7 look up the cache row of one token each
-    long long src = -1;
-    const int t = first + (lane & 7);
-    if (t < t1) {
-      const int pg = t / p.page_size;
-      const int page = pg < p.max_pages ? table[pg] : -1;
-      if ((unsigned)page < (unsigned)p.num_pages) src = (long long)page * p.page_size + t % p.page_size;
-      else report_bad_arg(p.status, 9);
+  // The queries pass through the ring's last stage, which no tile uses before the first iteration.
+  {
+    __nv_bfloat16* sq = sc + (LD_STAGES - 1) * LD_BT * PITCH;               // [M][PITCH], M <= LD_BT
+    const int q_rows = min(M, p.heads - h0);
+    for (int i = threadIdx.x; i < q_rows * vecs; i += THREADS) {
+      const int r = i / vecs, v = i - r * vecs;
+      cp_async16(smem_u32(sq + r * PITCH + v * 8), p.q + ((long long)row * p.heads + h0 + r) * p.width + v * 8);
     }
+    commit();
+  }
 #pragma unroll
-    for (int r = 0; r < 8; ++r) {
-      const long long s = __shfl_sync(0xffffffffu, src, r);
-      __nv_bfloat16* d = dst + (warp * 8 + r) * PITCH;
-      for (int v = lane; v < vecs; v += 32) {
-        if (s >= 0) cp_async16(smem_u32(d + v * 8), p.cache + s * p.width + v * 8);
-        else *reinterpret_cast<uint4*>(d + v * 8) = make_uint4(0, 0, 0, 0);  // past the end: finite, masked below
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
+  for (int i = 0; i < LD_STAGES - 1; ++i) {                                 // one group per tile, empty ones included
+    if (i < tiles) request(i, look_up(i));
+    commit();
+  }
+  long long next_src = LD_STAGES - 1 < tiles ? look_up(LD_STAGES - 1) : -1;
+  asm volatile("cp.async.wait_group %0;" ::"n"(LD_STAGES - 1) : "memory");  // the queries have landed
+  __syncthreads();
+  uint32_t qf[NT * 2][4];                  // A fragments of this group's 16 heads, this warp's half of the columns
+  {
+    const uint32_t a_addr = smem_u32(sc + ((LD_STAGES - 1) * LD_BT + grp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PITCH +
+                                     kh * NT * 32 + (lane >> 4) * 8);
+#pragma unroll
+    for (int k = 0; k < NT * 2; ++k) ldsm_x4(qf[k], a_addr + k * 32);
+  }
+  float acc[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
+  const int sr = grp * 16 + ((threadIdx.x & 255) >> 4), se = (threadIdx.x & 15) * 2;  // softmax: row, first of two columns
+  float m_run = -INFINITY, l_run = 0.f;                                     // of row sr, the same in its 16 threads
 
-  float acc[MT][NT * 2][4];
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int j = 0; j < NT * 2; ++j)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) acc[m][j][i] = 0.f;
-  float m_run[MT], l_run[MT];              // of head row (threadIdx.x / 8) + 16 m, the same in its 8 threads
-#pragma unroll
-  for (int m = 0; m < MT; ++m) { m_run[m] = -INFINITY; l_run[m] = 0.f; }
-
-  if (tiles > 0) request(0);
   for (int it = 0; it < tiles; ++it) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    asm volatile("cp.async.wait_group %0;" ::"n"(LD_STAGES - 2) : "memory");
     __syncthreads();                       // tile `it` is in shared memory, everybody is done with tile it - 1
-    if (it + 1 < tiles) request(it + 1);
-    const __nv_bfloat16* c = sc + (it & 1) * LD_BT * PITCH;
-    // ---- scores of this warp's 8 tokens, all heads
-    float s[MT][2][4];
+    if (it + LD_STAGES - 1 < tiles) {
+      request(it + LD_STAGES - 1, next_src);
+      next_src = it + LD_STAGES < tiles ? look_up(it + LD_STAGES) : -1;
+    }
+    commit();
+    const __nv_bfloat16* c = sc + (it % LD_STAGES) * LD_BT * PITCH;
+    // ---- scores of 8 tokens for the group's heads
+    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+    const uint32_t b_addr = smem_u32(c + (tq * 8 + (lane & 7)) * PITCH + kh * NT * 32 + (lane >> 3) * 8);
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int u = 0; u < 2; ++u)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) s[m][u][i] = 0.f;
-    const uint32_t b_addr = smem_u32(c + (warp * 8 + (lane & 7)) * PITCH + (lane >> 3) * 8);
-    const uint32_t a_addr = smem_u32(sq + ((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + (lane >> 4) * 8);
-#pragma unroll 4
-    for (int k = 0; k < KP / 32; ++k) {
+    for (int k = 0; k < NT; ++k) {
       uint32_t b[4];
       ldsm_x4(b, b_addr + k * 64);
-#pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        uint32_t a[4];
-        ldsm_x4(a, a_addr + m * 16 * PITCH * 2 + k * 64);
-        mma_bf16(s[m][0], a, b[0], b[1]);
-        ldsm_x4(a, a_addr + m * 16 * PITCH * 2 + k * 64 + 32);
-        mma_bf16(s[m][1], a, b[2], b[3]);
-      }
+      mma_bf16(s0, qf[2 * k], b[0], b[1]);
+      mma_bf16(s1, qf[2 * k + 1], b[2], b[3]);
     }
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const int r = m * 16 + (lane >> 2), col = warp * 8 + (lane & 3) * 2;
+    {
+      const int r = kh * M + grp * 16 + (lane >> 2), col = tq * 8 + (lane & 3) * 2;
       const int tok = t0 + it * LD_BT + col;
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float v = (s[m][0][i] + s[m][1][i]) * p.scale_log2;
+        const float v = (s0[i] + s1[i]) * p.scale_log2;
         ss[(r + (i >> 1) * 8) * SP + col + (i & 1)] = (tok + (i & 1) < t1) ? v : -INFINITY;
       }
     }
     __syncthreads();
-    // ---- online softmax: eight threads per head row
+    // ---- online softmax: sixteen threads per head row
+    {
+      const float2 va = *reinterpret_cast<const float2*>(ss + sr * SP + se);
+      const float2 vb = *reinterpret_cast<const float2*>(ss + (M + sr) * SP + se);
+      const float x = va.x + vb.x, y = va.y + vb.y;
+      float mx = fmaxf(x, y);
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const int r = m * 16 + (threadIdx.x >> 3), e = (threadIdx.x & 7) * 4;
-      const float4 v = *reinterpret_cast<const float4*>(ss + r * SP + e);
-      float mx = fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w));
+      for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float mn = fmaxf(m_run, mx);               // finite: every tile holds at least one token
+      const float p0 = exp2f(x - mn), p1 = exp2f(y - mn);
+      float sum = p0 + p1;
 #pragma unroll
-      for (int o = 4; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float mn = fmaxf(m_run[m], mx);            // finite: every tile holds at least one token
-      const float p0 = exp2f(v.x - mn), p1 = exp2f(v.y - mn), p2 = exp2f(v.z - mn), p3 = exp2f(v.w - mn);
-      float sum = (p0 + p1) + (p2 + p3);
-#pragma unroll
-      for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-      const float alpha = exp2f(m_run[m] - mn);
-      l_run[m] = l_run[m] * alpha + sum;
-      m_run[m] = mn;
-      *reinterpret_cast<uint2*>(sp + r * PP + e) = make_uint2(pack_bf16x2(p0, p1), pack_bf16x2(p2, p3));
-      if ((threadIdx.x & 7) == 0) salpha[r] = alpha;
+      for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      const float alpha = exp2f(m_run - mn);
+      l_run = l_run * alpha + sum;
+      m_run = mn;
+      *reinterpret_cast<uint32_t*>(sp + sr * PP + se) = pack_bf16x2(p0, p1);
+      if ((threadIdx.x & 15) == 0) salpha[sr] = alpha;
     }
     __syncthreads();
-    // ---- O = alpha O + P C for this warp's quarter of the columns
-    const uint32_t v_addr = smem_u32(c + ((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + warp * (NT * 16) + (lane >> 4) * 8);
-    const uint32_t p_addr = smem_u32(sp + ((lane & 7) + ((lane >> 3) & 1) * 8) * PP + (lane >> 4) * 8);
-    uint32_t a[MT][LD_BT / 16][4];
+    // ---- O = alpha O + P C for this warp's eighth of the columns
+    const uint32_t v_addr = smem_u32(c + ((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + wq * (NT * 8) + (lane >> 4) * 8);
+    const uint32_t p_addr = smem_u32(sp + (grp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PP + (lane >> 4) * 8);
+    const float a0 = salpha[grp * 16 + (lane >> 2)], a1 = salpha[grp * 16 + (lane >> 2) + 8];
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const float a0 = salpha[m * 16 + (lane >> 2)], a1 = salpha[m * 16 + (lane >> 2) + 8];
-#pragma unroll
-      for (int j = 0; j < NT * 2; ++j) {
-        acc[m][j][0] *= a0; acc[m][j][1] *= a0; acc[m][j][2] *= a1; acc[m][j][3] *= a1;
-      }
-#pragma unroll
-      for (int k = 0; k < LD_BT / 16; ++k) ldsm_x4(a[m][k], p_addr + m * 16 * PP * 2 + k * 32);
+    for (int j = 0; j < NT; ++j) {
+      acc[j][0] *= a0; acc[j][1] *= a0; acc[j][2] *= a1; acc[j][3] *= a1;
     }
 #pragma unroll
-    for (int k = 0; k < LD_BT / 16; ++k)
+    for (int k = 0; k < LD_BT / 16; ++k) {
+      uint32_t a[4];
+      ldsm_x4(a, p_addr + k * 32);
 #pragma unroll
-      for (int j = 0; j < NT; ++j) {
+      for (int j = 0; j < NT / 2; ++j) {
         uint32_t b[4];
         ldsm_x4_t(b, v_addr + k * 16 * PITCH * 2 + j * 32);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          mma_bf16(acc[m][2 * j], a[m][k], b[0], b[1]);
-          mma_bf16(acc[m][2 * j + 1], a[m][k], b[2], b[3]);
-        }
+        mma_bf16(acc[2 * j], a, b[0], b[1]);
+        mma_bf16(acc[2 * j + 1], a, b[2], b[3]);
       }
+    }
   }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   // ---- results: normalised here, or left as (max, sum, unnormalised output) for the merge
-#pragma unroll
-  for (int m = 0; m < MT; ++m) {
-    const int r = m * 16 + (threadIdx.x >> 3);
-    if ((threadIdx.x & 7) == 0) {
-      sl[r] = l_run[m];
-      if (p.splits > 1 && h0 + r < p.heads) {
-        float* ml = p.part_ml + (((long long)row * p.heads + h0 + r) * p.splits + split) * 2;
-        ml[0] = m_run[m];
-        ml[1] = l_run[m];
-      }
+  if ((threadIdx.x & 15) == 0) {
+    sl[sr] = l_run;
+    if (p.splits > 1 && h0 + sr < p.heads) {
+      float* ml = p.part_ml + (((long long)row * p.heads + h0 + sr) * p.splits + split) * 2;
+      ml[0] = m_run;
+      ml[1] = l_run;
     }
   }
   __syncthreads();
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int half = 0; half < 2; ++half) {
+    const int r = grp * 16 + (lane >> 2) + half * 8;
+    if (h0 + r >= p.heads) continue;
+    const float inv = sl[r] > 0.f ? 1.f / sl[r] : 0.f;
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int r = m * 16 + (lane >> 2) + half * 8;
-      if (h0 + r >= p.heads) continue;
-      const float inv = sl[r] > 0.f ? 1.f / sl[r] : 0.f;
-#pragma unroll
-      for (int j = 0; j < NT * 2; ++j) {
-        const int col = warp * (NT * 16) + j * 8 + (lane & 3) * 2;
-        if (col >= p.width) continue;
-        const float x = acc[m][j][half * 2], y = acc[m][j][half * 2 + 1];
-        if (p.splits > 1)
-          *reinterpret_cast<float2*>(p.part_o + (((long long)row * p.heads + h0 + r) * p.splits + split) * p.width + col) =
-              make_float2(x, y);
-        else
-          *reinterpret_cast<uint32_t*>(p.o + ((long long)row * p.heads + h0 + r) * p.width + col) = pack_bf16x2(x * inv, y * inv);
-      }
+    for (int j = 0; j < NT; ++j) {
+      const int col = wq * (NT * 8) + j * 8 + (lane & 3) * 2;
+      if (col >= p.width) continue;
+      const float x = acc[j][half * 2], y = acc[j][half * 2 + 1];
+      if (p.splits > 1)
+        *reinterpret_cast<float2*>(p.part_o + (((long long)row * p.heads + h0 + r) * p.splits + split) * p.width + col) =
+            make_float2(x, y);
+      else
+        *reinterpret_cast<uint32_t*>(p.o + ((long long)row * p.heads + h0 + r) * p.width + col) = pack_bf16x2(x * inv, y * inv);
     }
+  }
 }
 
 __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
@@ -387,16 +421,16 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
   }
 }
 
-template <int NT, int MT>
+template <int NT, int HG>
 static int launch_latent_decode(const LatentDecodeParams& p, cudaStream_t st) {
-  constexpr int smem = LatentDecodeSmem<NT>::bytes(MT);
-  auto kern = latent_decode_kernel<NT, MT>;
+  constexpr int smem = LatentDecodeSmem<NT>::bytes(HG);
+  auto kern = latent_decode_kernel<NT, HG>;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
     configured = true;
   }
-  launch_dep(kern, dim3(p.rows, (p.heads + MT * 16 - 1) / (MT * 16), p.splits), LD_THREADS, smem, st, p);
+  launch_dep(kern, dim3(p.rows, (p.heads + HG * 16 - 1) / (HG * 16), p.splits), 256 * HG, smem, st, p);
   if (p.splits > 1)
     launch_dep(latent_merge_kernel, p.rows * p.heads, 128, 0, st, p.part_o, p.part_ml, p.o, p.splits, p.width);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
@@ -412,16 +446,23 @@ extern "C" int b200_latent_norm_append(const void* proj, long long ld_proj, cons
                                        cudaStream_t st) {
   if (rows <= 0) return 0;
   if (q_rank <= 0 || kv_rank <= 0 || width < kv_rank) return -10;
-  const int big = q_rank > kv_rank ? q_rank : kv_rank;
-  int threads = (big / 4 + 31) / 32 * 32;
-  threads = threads < 32 ? 32 : (threads > 256 ? 256 : threads);
-  if (f32)
-    launch_dep(latent_norm_append_kernel<float>, rows, threads, 0, st, (const float*)proj, ld_proj, (const float*)wq,
-               (const float*)wkv, (float*)cq, ld_cq, (float*)cache, slots, q_rank, kv_rank, width, num_slots, eps, status);
-  else
-    launch_dep(latent_norm_append_kernel<__nv_bfloat16>, rows, threads, 0, st, (const __nv_bfloat16*)proj, ld_proj,
-               (const __nv_bfloat16*)wq, (const __nv_bfloat16*)wkv, (__nv_bfloat16*)cq, ld_cq, (__nv_bfloat16*)cache,
-               slots, q_rank, kv_rank, width, num_slots, eps, status);
+  const bool vec = q_rank % 4 == 0 && kv_rank % 4 == 0 && ld_proj % 4 == 0 && ld_cq % 4 == 0 && width % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(cq) | reinterpret_cast<uintptr_t>(cache) |
+                     reinterpret_cast<uintptr_t>(wq) | reinterpret_cast<uintptr_t>(wkv)) & 15) == 0;
+  // few rows: a warp per block, so that they spread over the SMs
+  const int warps = rows >= 148 * 8 ? 8 : 1;
+  const unsigned grid = (unsigned)((rows + warps - 1) / warps);
+#define LATENT_NORM(T, V)                                                                                               \
+  launch_dep(latent_norm_append_kernel<T, V>, grid, warps * 32, 0, st, (const T*)proj, ld_proj, (const T*)wq,           \
+             (const T*)wkv, (T*)cq, ld_cq, (T*)cache, slots, rows, q_rank, kv_rank, width, num_slots, eps, status)
+  if (f32) {
+    if (vec) LATENT_NORM(float, 4);
+    else LATENT_NORM(float, 1);
+  } else {
+    if (vec) LATENT_NORM(__nv_bfloat16, 4);
+    else LATENT_NORM(__nv_bfloat16, 1);
+  }
+#undef LATENT_NORM
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -130,6 +130,89 @@ __global__ void __launch_bounds__(256) retention_recurrent_kernel(const Retentio
   }
 }
 
+// Decode step of a state that fits the block's registers (NR rows of four columns per thread): one block per (request,
+// head), the whole state is requested before anything else, so the rotation, which needs little, runs under its latency.
+template <typename T, int NR>
+__global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) retention_step_kernel(const RetentionParams p) {
+  pdl_sync();
+  extern __shared__ float rsm[];
+  __shared__ float red[32];
+  const int seq = blockIdx.x / p.heads, h = blockIdx.x - seq * p.heads;
+  const int D = p.dim, E = p.vdim, groups = E / 4, rg = 256 / groups;
+  float *qs = rsm, *ks = rsm + D, *part = rsm + 2 * D;         // [D], [D], [rg][E]
+  const int ty = threadIdx.x / groups, tx = threadIdx.x - ty * groups;
+  const int slot = p.state_slots[seq];
+  const T* pr = reinterpret_cast<const T*>(p.proj) + (long long)seq * p.ld_proj;
+  T* y = reinterpret_cast<T*>(p.y) + (long long)seq * p.ld_y + h * E;
+  if (slot < 0 || slot >= p.num_slots) {
+    if (slot >= p.num_slots && threadIdx.x == 0) report_bad_arg(p.status, 7);
+    for (int c = threadIdx.x; c < E; c += 256) from_f(y[c], 0.f);
+    return;
+  }
+  int pos = p.positions[seq];
+  const bool on = ty < rg;
+  float4* S = reinterpret_cast<float4*>(p.state + ((long long)slot * p.heads + h) * D * E) + tx;
+  float4 s[NR];
+#pragma unroll
+  for (int j = 0; j < NR; ++j) {
+    const int d = ty + j * rg;
+    s[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (on && d < D && pos != 0) s[j] = __ldcs(S + (long long)d * groups);
+  }
+  const T* qr = pr + h * D;
+  const T* kr = pr + p.heads * D + h * D;
+  if (pos < 0 || (p.rot > 0 && pos >= p.ctx)) {
+    if (threadIdx.x == 0) report_bad_arg(p.status, 8);
+    pos = 0;
+  }
+  const int half = p.rot / 2;
+  const float kscale = rsqrtf((float)D);
+  for (int d = threadIdx.x; d < D; d += 256) {
+    float qv = to_f(qr[d]), kv = to_f(kr[d]);
+    if (d < p.rot) {
+      const int i = d < half ? d : d - half, o = d < half ? d + half : d - half;
+      const float c = p.cos_sin[(long long)pos * half + i];
+      const float sn = d < half ? -p.cos_sin[((long long)p.ctx + pos) * half + i] : p.cos_sin[((long long)p.ctx + pos) * half + i];
+      qv = qv * c + to_f(qr[o]) * sn;
+      kv = kv * c + to_f(kr[o]) * sn;
+    }
+    qs[d] = qv;
+    ks[d] = kv * kscale;
+  }
+  float v[4] = {0.f, 0.f, 0.f, 0.f};
+  if (on) load_vec<4>(pr + 2 * p.heads * D + h * E + tx * 4, v);
+  const float decay = p.decay[h];
+  __syncthreads();
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < NR; ++j) {
+    const int d = ty + j * rg;
+    if (!on || d >= D) continue;
+    const float kd = ks[d], qd = qs[d];
+    s[j].x = fmaf(decay, s[j].x, kd * v[0]); s[j].y = fmaf(decay, s[j].y, kd * v[1]);
+    s[j].z = fmaf(decay, s[j].z, kd * v[2]); s[j].w = fmaf(decay, s[j].w, kd * v[3]);
+    o.x = fmaf(s[j].x, qd, o.x); o.y = fmaf(s[j].y, qd, o.y); o.z = fmaf(s[j].z, qd, o.z); o.w = fmaf(s[j].w, qd, o.w);
+    __stcs(S + (long long)d * groups, s[j]);
+  }
+  if (on) *reinterpret_cast<float4*>(part + ty * E + tx * 4) = o;
+  __syncthreads();
+  float ss = 0.f, mine[4];
+  int n = 0;
+  for (int c = threadIdx.x; c < E && n < 4; c += 256, ++n) {           // E <= 1024
+    float t = 0.f;
+    for (int r = 0; r < rg; ++r) t += part[r * E + c];
+    mine[n] = t;
+    ss += t * t;
+  }
+  const float inv = rsqrtf(block_total(ss, red) / (float)E + p.eps);
+  const T* gr = pr + 2 * p.heads * D + p.heads * E + h * E;
+  n = 0;
+  for (int c = threadIdx.x; c < E && n < 4; c += 256, ++n) {
+    const float g = to_f(gr[c]);
+    from_f(y[c], mine[n] * inv * (g / (1.f + __expf(-g))));
+  }
+}
+
 // ------------------------------------------------------------------------------------ prompts, bf16, on the tensor cores
 // One CTA = one (portion, head), chunks of n <= 128 tokens in order.  With r the last row of a chunk, scale the rotated
 // rows in fp32:  q~_i = decay^(i-r) q_i,  k~_j = decay^(r-j) k_j  and let S' = decay^n S.  Then
@@ -573,6 +656,18 @@ extern "C" int b200_retention_recurrent(const void* proj, long long ld_proj, voi
   const size_t smem = (2ull * dim + (size_t)rg * vdim) * sizeof(float);
   if (smem > 48 * 1024) return -12;
   const dim3 grid(seqs, heads);
+  if (vec && cu == nullptr && groups <= 256 && (dim + rg - 1) / rg <= 16 && (dim & 3) == 0) {
+    const long long blocks = (long long)seqs * heads;
+    const bool small = (dim + rg - 1) / rg <= 4;
+    if (f32) {
+      if (small) launch_dep(retention_step_kernel<float, 4>, (unsigned)blocks, 256, smem, st, p);
+      else launch_dep(retention_step_kernel<float, 16>, (unsigned)blocks, 256, smem, st, p);
+    } else {
+      if (small) launch_dep(retention_step_kernel<__nv_bfloat16, 4>, (unsigned)blocks, 256, smem, st, p);
+      else launch_dep(retention_step_kernel<__nv_bfloat16, 16>, (unsigned)blocks, 256, smem, st, p);
+    }
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  }
   if (f32) {
     if (vec) launch_dep(retention_recurrent_kernel<float, 4>, grid, 256, smem, st, p);
     else launch_dep(retention_recurrent_kernel<float, 1>, grid, 256, smem, st, p);

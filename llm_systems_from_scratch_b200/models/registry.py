@@ -22,6 +22,10 @@ def model_class(config: dict):
     return MODELS[name]
 
 
+def vocabulary(config: dict) -> int:
+    return config["vocab_size"] if "vocab_size" in config else config["vocab"]
+
+
 def read_config(path: str) -> dict:
     """``path``: a configuration file, or a model folder with config.json (or model_config.json)."""
     if os.path.isdir(path):

@@ -258,10 +258,17 @@ DECODE_TILE = 32
 
 
 def latent_splits(rows: int, heads: int, keys: int, sms: int = 148) -> int:
-    """Splits of the window per row of a decode step: two CTAs fit on an SM, and a CTA should have a few tiles to walk."""
-    groups = rows * -(-heads // (16 if heads <= 16 else 32))
-    most = max(1, keys // (4 * DECODE_TILE))
-    return max(1, min(most, -(-2 * sms // groups)))
+    """Splits of the window per row of a decode step, by a cost in tiles: a CTA starts up for about two tiles, two CTAs that
+    share an SM (up to 16 heads; with more there is one) take 1.7 times as long as one, a merge costs about two tiles."""
+    groups = rows * (1 if heads <= 16 else -(-heads // 32))
+    best, best_cost = 1, None
+    for n in range(1, max(1, min(32, keys // (2 * DECODE_TILE))) + 1):
+        per_sm = -(-groups * n // sms)
+        load = per_sm if heads > 16 else per_sm // 2 * 1.7 + per_sm % 2
+        cost = load * (-(-keys // (n * DECODE_TILE)) + 2) + (2 if n > 1 else 0)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = n, cost
+    return best
 
 
 def latent_decode(q, cache, positions, slots, tables, heads: int, window: int, scale: float, splits: int = 0):

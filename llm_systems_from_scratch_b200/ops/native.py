@@ -640,7 +640,8 @@ def sample_topk(logits, uniforms, temperature: float, top_k: int | None = None, 
     _req(temperature > 0, "temperature must be positive (use argmax_rows for greedy decoding)")
     out = torch.empty(rows, dtype=torch.int64, device=logits.device)
     _check(lib.b200_sample_topk(_ptr(logits), rows, logits.stride(0), valid_cols or cols,
-                                int(logits.dtype == torch.float32), _ptr(uniforms), float(temperature), int(top_k or 0), _ptr(out), _stream()), "sample_topk")
+                                int(logits.dtype == torch.float32), _ptr(uniforms), float(temperature), int(top_k or 0),
+                                _ptr(out), _stream()), "sample_topk")
     return out
 
 

@@ -5,6 +5,9 @@ Required sections and keys are those the reference indexes without defaults: ``m
 defaults: ``training.seed``, ``training.dtype``, ``training.activation_checkpointing``,
 ``training.resume``, ``training.step_timeout_s``, ``optimizer.betas``, ``optimizer.eps``, ``fsdp.comm``,
 ``fsdp.fused_optimizer``, ``ddp.bucket_size_mb``, and a whole optional ``serving`` section.
+
+A ``model`` section with ``architecture`` is that registered model's own configuration (``models.registry``), which checks
+it itself; such a configuration is for serving and needs no training sections.
 """
 from __future__ import annotations
 
@@ -40,7 +43,12 @@ def load_config(path: str) -> dict:
 def validate(cfg: dict, world_size: int = 1, require_dataset: bool = True) -> dict:
     """Check required keys, fill optional ones, coerce numeric strings such as ``6.0e-4``."""
     out = {k: dict(v) if isinstance(v, dict) else v for k, v in cfg.items()}
+    other = out.get("model", {}).get("architecture", "TransformerLM") != "TransformerLM"
+    if other:
+        out.setdefault("serving", {})
     for section, keys in REQUIRED.items():
+        if other:
+            continue
         if section == "dataset" and not require_dataset:
             continue
         if section not in out:
@@ -52,6 +60,8 @@ def validate(cfg: dict, world_size: int = 1, require_dataset: bool = True) -> di
         sec = out.setdefault(section, {})
         for k, v in defaults.items():
             sec.setdefault(k, v)
+    if other:
+        return out
     o = out["optimizer"]
     for k in ("learning_rate_max", "learning_rate_min", "weight_decay", "max_grad_norm", "eps"):
         o[k] = float(o[k])

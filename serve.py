@@ -5,7 +5,9 @@
     python -m torch.distributed.run --nproc-per-node N --master-addr 127.0.0.1 serve.py ...   (one replica per GPU)
     python serve.py --config configures/serve_1p3b.yaml --checkpoint ckpt_final.pt --http 8000   (online: POST /generate)
 
-Weights are random-init unless ``--checkpoint`` points at a checkpoint written by train.py.  Each replica
+Weights are random-init unless ``--checkpoint`` points at a checkpoint written by train.py, or ``--model`` at a model
+folder (config.json and weights of any registered model; the serving section still comes from ``--config``).  The
+``model`` section of the configuration may be that of any registered model (``architecture``).  Each replica
 serves its own trace (seed + rank); rank 0 prints one JSON line with the aggregate decode tokens/s and
 the time-to-first-token percentiles.  ``--impl reference`` replays the head of the same trace through
 the reference-style loop (one request at a time, greedy argmax over a full re-forward, no KV cache).
@@ -69,12 +71,14 @@ def serve_http(engine, args):
 
 
 def main(argv=None):
-    from llm_systems_from_scratch_b200.models.transformer import TransformerLM
+    from llm_systems_from_scratch_b200.models.registry import build_model, load_model, vocabulary
     from llm_systems_from_scratch_b200.serving import ServingEngine, poisson_trace
     from llm_systems_from_scratch_b200.utils.config import load_config, validate
     ap = argparse.ArgumentParser()
     ap.add_argument("--config", default=os.path.join(ROOT, "configures", "serve_1p3b.yaml"))
     ap.add_argument("--checkpoint", default=None)
+    ap.add_argument("--model", default=None, metavar="FOLDER", help="model folder of any registered model")
+    ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16", help="what a --model folder is served in")
     ap.add_argument("--num-requests", type=int, default=None)
     ap.add_argument("--rate", type=float, default=None, help="arrivals per second per GPU")
     ap.add_argument("--offline", action="store_true", help="ignore arrival times (throughput mode)")
@@ -104,16 +108,20 @@ def main(argv=None):
         dist.init_process_group("nccl" if cuda else "gloo")
     torch.manual_seed(0)
     keys = ("vocab_size", "context_length", "d_model", "num_layers", "num_heads", "d_ff", "rope_theta")
+    model = None
+    if args.model is not None:
+        model = load_model(args.model, getattr(torch, args.dtype), device)
+    vocab = model.vocab_size if model is not None else vocabulary(m)
     trace = poisson_trace(args.num_requests or s["num_requests"], args.rate or s["arrival_rate"], tuple(s["prompt_len"]),
-                          tuple(s["output_len"]), m["vocab_size"], seed=s["seed"] + rank)
+                          tuple(s["output_len"]), vocab, seed=s["seed"] + rank)
     if args.impl == "reference":
         sys.path.insert(0, os.path.join(ROOT, "baseline", "_ref"))
         from llm_core.model import TransformerLM as RefLM
         model = RefLM(**{k: m[k] for k in keys}, use_flash_attn=True).to(device).eval()
         res = naive_loop(model, trace, device, args.time_limit)
     else:
-        with torch.device(device):
-            model = TransformerLM(**{k: m[k] for k in keys}, use_flash_attn=True, use_custom_triton=True)
+        if model is None:
+            model = build_model(m if "architecture" in m else {k: m[k] for k in keys}, device=device)
         if args.checkpoint:
             state = torch.load(args.checkpoint, map_location="cpu")
             model.load_state_dict(state.get("model", state))
@@ -136,7 +144,7 @@ def main(argv=None):
         dist.destroy_process_group()
     if rank == 0:
         res.update(metric="serving_decode_tok_per_s", impl=args.impl, n_gpus=world, model="TransformerLM-1.3B"
-                   if m["d_model"] == 2048 else "custom", rate_per_gpu=args.rate or s["arrival_rate"])
+                   if m.get("d_model") == 2048 else type(model).__name__, rate_per_gpu=args.rate or s["arrival_rate"])
         print(json.dumps(res))
 
 
