@@ -96,8 +96,9 @@ def feed(engine, seqs, schedule, poison=False):
     """Run ``schedule`` (a list of steps, each a list of (sequence, tokens)) through ``engine.extend``, all logits wanted;
     a sequence is closed when its tokens are used up.  Returns the logits per sequence."""
     if poison:
-        for e in engine.cache.entries:
-            e.fill_(float("nan"))            # nothing may be read that was not written by its own request
+        # nothing may be read that was not written by its own request (the zero padding of a latent is not data)
+        for run, e in zip(engine.backend.model.runs, engine.cache.entries):
+            e[..., :getattr(run.mixer, "kv_rank", e.shape[-1])] = float("nan")
     at, live, got = [0] * len(seqs), {}, [[] for _ in seqs]
     for step in schedule:
         entries = []
