@@ -142,7 +142,9 @@ def _ptr(t) -> int:
 
 def status_word(device=None) -> torch.Tensor:
     """Per-device uint32 status word written by kernels whose bounded waits gave up."""
-    dev = torch.cuda.current_device() if device is None else torch.device(device).index
+    dev = None if device is None else torch.device(device).index
+    if dev is None:                      # no device, or "cuda" without an index
+        dev = torch.cuda.current_device()
     if dev not in _STATUS:
         _STATUS[dev] = torch.zeros(4, dtype=torch.int32, device=f"cuda:{dev}")
     return _STATUS[dev]
