@@ -5,6 +5,9 @@ ctypes, so no PyTorch headers are needed and a full rebuild takes seconds.  The 
 object is written next to this file (``_b200_kernels.so``): it is git-ignored but
 travels with the source tree to the GPU machine.
 
+``build_serving`` compiles only what serving needs (without the backward kernels) into ``_b200_serving.so``, for a
+fresh checkout whose first command serves a model; objects are shared, so a full build later compiles the rest.
+
 Usage:  python -m llm_systems_from_scratch_b200.build_ext [--force] [--verbose]
 """
 from __future__ import annotations
@@ -21,6 +24,8 @@ PKG_DIR = Path(__file__).resolve().parent
 CSRC = PKG_DIR / "csrc"
 BUILD_DIR = PKG_DIR / "csrc" / "build"
 LIB_PATH = PKG_DIR / "_b200_kernels.so"
+SERVING_LIB_PATH = PKG_DIR / "_b200_serving.so"
+NOT_FOR_SERVING = {"flash_attn_bwd.cu"}     # training only (comm_kernels.cu holds host code of the GEMMs)
 HOST_SRC = CSRC / "host" / "host_runtime.cpp"
 HOST_LIB_PATH = PKG_DIR / "_b200_host.so"
 
@@ -82,19 +87,21 @@ def build_host(force: bool = False) -> Path | None:
     return HOST_LIB_PATH
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every ``csrc/*.cu`` for sm_100a and link ``_b200_kernels.so``; also builds the host runtime."""
-    build_host(force)
-    if not force and not needs_build():
-        return LIB_PATH
+def headers() -> list[Path]:
+    return sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+
+
+def _compile_and_link(srcs: list[Path], target: Path, force: bool = False, verbose: bool = False):
+    """Compile ``srcs`` (skipping objects that are up to date) and link them into ``target``."""
     nvcc = _nvcc()
     BUILD_DIR.mkdir(parents=True, exist_ok=True)
-    srcs = sources()
     if not srcs:
         raise RuntimeError(f"no CUDA sources under {CSRC}")
 
     def compile_one(src: Path):
-        obj = BUILD_DIR / (src.stem + ".o")
+        obj, stamp, digest = BUILD_DIR / (src.stem + ".o"), BUILD_DIR / (src.stem + ".stamp"), _digest([src, *headers()])
+        if not force and obj.exists() and stamp.exists() and stamp.read_text() == digest:
+            return obj
         cmd = [nvcc, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
         proc = subprocess.run(cmd, capture_output=True, text=True)
         log = BUILD_DIR / (src.stem + ".ptxas.log")
@@ -103,19 +110,40 @@ def build(force: bool = False, verbose: bool = False) -> Path:
             raise RuntimeError(f"nvcc failed for {src.name}:\n{proc.stdout}\n{proc.stderr}")
         if verbose:
             sys.stderr.write(proc.stderr)
+        stamp.write_text(digest)
         return obj
 
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         objs = list(ex.map(compile_one, srcs))
-    tmp = LIB_PATH.with_suffix(".so.tmp")
+    tmp = target.with_suffix(".so.tmp")
     link = [nvcc, "-shared", "-o", str(tmp), *map(str, objs)]
     proc = subprocess.run(link, capture_output=True, text=True)
     if proc.returncode != 0:
         raise RuntimeError(f"link failed:\n{proc.stdout}\n{proc.stderr}")
-    os.replace(tmp, LIB_PATH)
-    deps = srcs + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    (BUILD_DIR / "stamp.txt").write_text(_digest(deps))
+    os.replace(tmp, target)
+
+
+def build(force: bool = False, verbose: bool = False) -> Path:
+    """Compile every ``csrc/*.cu`` for sm_100a and link ``_b200_kernels.so``; also builds the host runtime."""
+    build_host(force)
+    if not force and not needs_build():
+        return LIB_PATH
+    _compile_and_link(sources(), LIB_PATH, force, verbose)
+    (BUILD_DIR / "stamp.txt").write_text(_digest(sources() + headers()))
     return LIB_PATH
+
+
+def build_serving() -> Path:
+    """The library a serving command loads: the full one if it has been built, else the serving kernels alone."""
+    build_host()
+    if LIB_PATH.exists():
+        return LIB_PATH
+    srcs = [s for s in sources() if s.name not in NOT_FOR_SERVING]
+    stamp, digest = BUILD_DIR / "serving_stamp.txt", _digest(srcs + headers())
+    if not (SERVING_LIB_PATH.exists() and stamp.exists() and stamp.read_text() == digest):
+        _compile_and_link(srcs, SERVING_LIB_PATH)
+        stamp.write_text(digest)
+    return SERVING_LIB_PATH
 
 
 if __name__ == "__main__":

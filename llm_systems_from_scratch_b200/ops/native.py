@@ -34,6 +34,16 @@ def lib_path() -> Path:
     return _LIB_PATH
 
 
+def load_serving():
+    """Load the library for serving: the full one if it is there, else one of the serving kernels alone, built if need be
+    (``build_ext.build_serving``).  Training then needs a process of its own."""
+    global _LIB_PATH
+    if _LIB is None:
+        from ..build_ext import build_serving
+        _LIB_PATH = build_serving()
+    return load()
+
+
 def load(required: bool = True):
     """Load the kernel library once.  ``required`` raises if it is missing."""
     global _LIB
@@ -113,7 +123,7 @@ def _declare(lib):
     for name, args in {**sigs, **optional}.items():
         fn = getattr(lib, name, None)
         if fn is None:
-            if name in sigs:
+            if name in sigs and _LIB_PATH.stem != "_b200_serving":
                 raise KernelError(f"symbol {name} missing from {_LIB_PATH}")
             continue
         fn.argtypes = args

@@ -72,6 +72,8 @@ def main(argv=None) -> int:
     if args.dtype == "float32" and torch.float32 not in getattr(model_class(read_config(args.model)), "GPU_DTYPES", ()):
         print("this model is served in bfloat16 only", file=sys.stderr)
         return 3
+    from ..ops import native
+    native.load_serving()
     engine = open_engine(args.model, getattr(torch, args.dtype), args.max_tokens)
     replay(engine, sys.stdin, args.out)
     return 0
