@@ -2,8 +2,10 @@
 
 ``models(size)`` times whole steps through the serving engine (a prompt step of several prompts; a decode step at a batch
 and a context), on the device with CUDA events; every step streams weights and caches that are larger than L2.
-``kernels(size)`` times each kernel alone on one layer's shapes, L2 replaced between runs: achieved bytes or FLOPs per
-second over the measured copy bandwidth or GEMM throughput.  Weights are random."""
+``kernels(size)`` times each kernel alone on one layer's shapes: achieved bytes or FLOPs per second over the measured copy
+bandwidth or GEMM throughput.  Prompt kernels: one launch between two events, L2 replaced between runs.  Decode kernels,
+which are as short as a launch: a CUDA graph of launches on different inputs that exceed L2 together, divided by their
+number.  Weights are random."""
 from __future__ import annotations
 
 import gc
@@ -142,6 +144,21 @@ class _Table:
                           "tflops": round(flops / ms / 1e9, 1), "fraction_of_roofline": round(roof / ms, 3)})
 
 
+def graph_ms(make, nbytes: float) -> float:
+    """Milliseconds per launch of the closures that ``make()`` returns, each on inputs of its own (``nbytes`` apiece), in one
+    captured graph; together they read at least 400 MB, so nothing is found in L2 from the launch before."""
+    fns = [make() for _ in range(int(max(4, min(48, 400e6 // max(1.0, nbytes) + 1))))]
+    for f in fns[:2]:
+        f()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    keep = []
+    with torch.cuda.graph(graph):
+        for f in fns:
+            keep.append(f())
+    return timeit(graph.replay, iters=7, warm=2, flush=True) / len(fns)
+
+
 def _bf(*shape):
     return torch.randn(*shape, device="cuda").bfloat16()
 
@@ -204,7 +221,7 @@ def _prompt_kernels(s, t):
     # residual stream
     nw = torch.ones(w, device="cuda").bfloat16()
     t.add("rmsnorm_fwd (TransformerLM)", "-", timeit(lambda: native.rmsnorm_fwd(res, nw, 1e-6)), rows * w * 4)
-    _residual_kernel(s, t, rows, "")
+    _residual_kernel(s, t, rows)
     # latents
     pr = _bf(rows, s["q_rank"] + s["kv_rank"] + hd)
     nq, nkv = _bf(s["q_rank"]), _bf(s["kv_rank"])
@@ -237,7 +254,7 @@ def _expert_kernels(s, t, rows, tokens):
           (n * ff + active * ff * w + n * w) * 2, 2.0 * n * w * ff)
 
 
-def _residual_kernel(s, t, rows, label):
+def _residual_kernel(s, t, rows):
     w = s["width"]
     x = torch.randn(rows, w, device="cuda")
     p = mo.plan_tiles(rows, EXPERTS, TOP) * mo.TILE
@@ -254,49 +271,96 @@ def _decode_kernels(s, t, b):
     w, heads = s["width"], s["heads"]
     hd = heads * 128
     pages = -(-(CONTEXT + 16) // 16)
-    tables = torch.randperm(b * pages, device="cuda").int().view(b, pages).contiguous()
-    full = torch.zeros(b, 128, dtype=torch.int32, device="cuda")
-    full[:, :pages] = tables
-    qkv = _bf(b, 3 * hd)
-    kc, vc = _bf(b * pages, 16, hd), _bf(b * pages, 16, hd)
     ctx = torch.full((b,), CONTEXT, dtype=torch.int32, device="cuda")
-    t.add(f"paged_decode, batch {b} (TransformerLM)", "-",
-          timeit(lambda: serving_ops.paged_decode_attention(qkv, kc, vc, full, ctx, heads)), b * CONTEXT * hd * 4)
-    del kc, vc
-    kvr, win = s["kv_rank"], min(s["window"], CONTEXT)
-    cache = _bf(b * pages, 16, kvr)
-    ql = _bf(b, heads * kvr)
     pos, slots = ctx - 1, torch.zeros(b, dtype=torch.int64, device="cuda")
-    t.add(f"latent_decode, batch {b}, window {win}", "paged_decode",
-          timeit(lambda: mo.latent_decode(ql, cache, pos, slots, full, heads, s["window"], 0.1)), b * (win * kvr * 2 + heads * kvr * 4),
-          4.0 * b * heads * win * kvr)
-    state = torch.randn(b, heads, 128, 128, device="cuda")
-    sl = torch.randperm(b, device="cuda").int()
-    proj, y = _bf(b, 4 * hd), _bf(b, hd)
-    table = torch.randn(2, 2048, 64, device="cuda")
-    decay = torch.full((heads,), 0.99, device="cuda")
-    t.add(f"retention step, batch {b}", "paged_decode",
-          timeit(lambda: mo.retention(proj, state, sl, None, None, pos, table, decay, heads, 128, 128, 128, 1e-6, y)),
-          b * heads * 128 * 128 * 8)
-    for name, n, k in (("qkv", 3 * hd, w), ("gate|up", 2 * s["ff"], w), ("down", w, s["ff"])):
-        a, wt = _bf(b, k), _bf(n, k)
-        t.add(f"{name} GEMM, batch {b} (TransformerLM)", "-", timeit(lambda: native.gemm(a, wt, "nt", b_stable=True)), (n * k + b * (n + k)) * 2)
-    for name, n, k in (("retention q|k|v|g", 4 * hd, w), ("latent dq|dkv|g", s["q_rank"] + kvr + hd, w), ("uq", hd, s["q_rank"])):
-        a, wt = _bf(b, k), _bf(n, k)
-        t.add(f"{name} GEMM, batch {b}", "qkv GEMM", timeit(lambda: mo.linear(a, wt)), (n * k + b * (n + k)) * 2)
-    a, wt, x = _bf(b, hd), _bf(w, hd), torch.zeros(b, w, device="cuda")
-    t.add(f"output GEMM into the residual, batch {b}", "down GEMM", timeit(lambda: mo.linear(a, wt, out=x, accumulate=True)),
-          (w * hd + b * hd) * 2 + b * w * 8)
-    q, wk = _bf(b, hd), _bf(heads * kvr, 128)
-    t.add(f"query into latent space, batch {b}", "qkv GEMM", timeit(lambda: mo.gemm_heads(q, wk, heads, 128, kvr)),
-          (heads * kvr * 128 + b * hd + b * heads * kvr) * 2)
-    wv, gate = _bf(hd, kvr), _bf(b, hd)
-    t.add(f"latent output to heads + gate, batch {b}", "qkv GEMM", timeit(lambda: mo.gemm_heads(ql, wv, heads, kvr, 128, gate=gate)),
-          (heads * kvr * 128 + 2 * b * hd + b * heads * kvr) * 2)
-    _expert_kernels(s, t, b, torch.randint(0, s["vocab"], (b,), device="cuda"))
-    _residual_kernel(s, t, b, "")
-    xr, nw = _bf(b, w), torch.ones(w, device="cuda").bfloat16()
-    t.add(f"rmsnorm_fwd, {b} rows (TransformerLM)", "-", timeit(lambda: native.rmsnorm_fwd(xr, nw, 1e-6)), b * w * 4)
+    kvr, win = s["kv_rank"], min(s["window"], CONTEXT)
+
+    def tables():
+        full = torch.zeros(b, 128, dtype=torch.int32, device="cuda")
+        full[:, :pages] = torch.randperm(b * pages, device="cuda").int().view(b, pages)
+        return full
+
+    def add(name, like, nbytes, flops, make):
+        t.add(f"{name}, batch {b}", like, graph_ms(make, nbytes), nbytes, flops)
+        torch.cuda.empty_cache()
+
+    def paged():
+        qkv, kc, vc, tb = _bf(b, 3 * hd), _bf(b * pages, 16, hd), _bf(b * pages, 16, hd), tables()
+        return lambda: serving_ops.paged_decode_attention(qkv, kc, vc, tb, ctx, heads)
+    add("paged_decode (TransformerLM)", "-", b * CONTEXT * hd * 4, 0, paged)
+
+    def latent():
+        ql, cache, tb = _bf(b, heads * kvr), _bf(b * pages, 16, kvr), tables()
+        return lambda: mo.latent_decode(ql, cache, pos, slots, tb, heads, s["window"], 0.1)
+    add(f"latent_decode, window {win}", "paged_decode", b * (win * kvr * 2 + heads * kvr * 4), 4.0 * b * heads * win * kvr, latent)
+    table, decay = torch.randn(2, 2048, 64, device="cuda"), torch.full((heads,), 0.99, device="cuda")
+
+    def step():
+        state, sl = torch.randn(b, heads, 128, 128, device="cuda"), torch.randperm(b, device="cuda").int()
+        proj, y = _bf(b, 4 * hd), _bf(b, hd)
+        return lambda: mo.retention(proj, state, sl, None, None, pos, table, decay, heads, 128, 128, 128, 1e-6, y)
+    add("retention step", "paged_decode", b * heads * 128 * 128 * 8, 0, step)
+
+    def plain(n, k):
+        def make():
+            a, wt = _bf(b, k), _bf(n, k)
+            return lambda: mo.linear(a, wt)
+        return make
+    size = lambda n, k: (n * k + b * (n + k)) * 2
+    for name, like, n, k in (("qkv GEMM (TransformerLM)", "-", 3 * hd, w), ("output GEMM (TransformerLM)", "-", w, hd),
+                             ("gate|up GEMM (TransformerLM)", "-", 2 * s["ff"], w), ("down GEMM (TransformerLM)", "-", w, s["ff"]),
+                             ("retention q|k|v|g GEMM", "qkv GEMM", 4 * hd, w),
+                             ("latent dq|dkv|g GEMM", "qkv GEMM", s["q_rank"] + kvr + hd, w), ("latent uq GEMM", "output GEMM", hd, s["q_rank"])):
+        add(name, like, size(n, k), 0, plain(n, k))
+
+    def out_gemm():
+        a, wt, x = _bf(b, hd), _bf(w, hd), torch.zeros(b, w, device="cuda")
+        return lambda: mo.linear(a, wt, out=x, accumulate=True)
+    add("output GEMM into the fp32 residual", "output GEMM", (w * hd + b * hd) * 2 + b * w * 8, 0, out_gemm)
+
+    def to_latent():
+        q, wk = _bf(b, hd), _bf(heads * kvr, 128)
+        return lambda: mo.gemm_heads(q, wk, heads, 128, kvr)
+    add("queries into latent space", "output GEMM", (heads * kvr * 128 + b * hd + b * heads * kvr) * 2, 0, to_latent)
+
+    def from_latent():
+        ol, wv, gate = _bf(b, heads * kvr), _bf(hd, kvr), _bf(b, hd)
+        return lambda: mo.gemm_heads(ol, wv, heads, kvr, 128, gate=gate)
+    add("latent outputs to heads, gate", "output GEMM", (heads * kvr * 128 + 2 * b * hd + b * heads * kvr) * 2, 0, from_latent)
+    ff, n = s["ff"] // TOP, b * TOP
+    tab = torch.rand(s["vocab"], EXPERTS, device="cuda").argsort(1)[:, :TOP].int().contiguous()
+    tokens = torch.randint(0, s["vocab"], (b,), device="cuda")
+    add("moe_plan, 12 layers", "-", 12 * n * 8, 0, lambda: (lambda: mo.moe_plan(tokens, slots, [tab] * 12, [EXPERTS] * 12)))
+    (mpos,), (group,) = mo.moe_plan(tokens, slots, [tab], [EXPERTS])
+    p, active = mo.plan_tiles(b, EXPERTS, TOP) * mo.TILE, min(EXPERTS, n)
+
+    def gate_up():
+        xg, wt = _bf(p, w), _bf(EXPERTS * 2 * ff, w)
+        return lambda: mo.gemm_rows(xg, wt, group, ff, True)
+    add("experts gate|up + SwiGLU", "gate|up GEMM", (n * w + active * 2 * ff * w + n * ff) * 2, 4.0 * n * w * ff, gate_up)
+
+    def down():
+        hid, wt = _bf(p, ff), _bf(EXPERTS * w, ff)
+        return lambda: mo.gemm_rows(hid, wt, group, w, False)
+    add("experts down", "down GEMM", (n * ff + active * ff * w + n * w) * 2, 2.0 * n * w * ff, down)
+    nw = torch.ones(w, device="cuda").bfloat16()
+
+    def resid():
+        x, y = torch.randn(b, w, device="cuda"), _bf(p, w)
+        return lambda: mo.residual_norm(x, nw, 1e-6, pending=(y, mpos, 0.0), scatter=(mpos, p))
+    add("residual_norm with experts", "rmsnorm_fwd", b * w * (8 + 2 * TOP + 2 + 2 * TOP), 0, resid)
+
+    def norm():
+        x = _bf(b, w)
+        return lambda: native.rmsnorm_fwd(x, nw, 1e-6)
+    add("rmsnorm_fwd (TransformerLM)", "-", b * w * 4, 0, norm)
+    nq, nkv = _bf(s["q_rank"]), _bf(kvr)
+
+    def append():
+        pr, cache = _bf(b, s["q_rank"] + kvr + hd), _bf(b, 16, kvr)
+        sl = torch.arange(b, device="cuda") * 16
+        return lambda: mo.latent_norm_append(pr, nq, nkv, 1e-6, cache, sl)
+    add("latent_norm_append", "rmsnorm_fwd", b * (s["q_rank"] + kvr) * 4, 0, append)
 
 
 def run(sizes, steps: int = 10, warmup: int = 3, per_kernel: bool = True):
