@@ -386,24 +386,29 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const __
   for (int ch = 0; ch < chunks; ++ch) {
     const int t0 = ch * RC_CHUNK, n = min(RC_CHUNK, rows - t0);
     if (worker) {
-      // ---- q~, k~: rotated, scaled, split; rows past the end become zero
+      // ---- q~, k~: rotated, scaled, split; rows past the end become zero.  The angles of the first PRE rows are requested
+      // before the wait: there is no L1 to speak of beside this much shared memory.
+      constexpr int PRE = 4;
+      float4 ang[PRE][4];                               // cos, cos, sin, sin
+      auto load_angles = [&](int t, float4 (&a)[4]) {
+        const float* cs = p.cos_sin + (long long)min(pos0 + t0 + min(t, n - 1), p.ctx - 1) * rot2 + i_d0;
+        const float* sn = cs + (long long)p.ctx * rot2;
+        a[0] = __ldg(reinterpret_cast<const float4*>(cs));
+        a[1] = __ldg(reinterpret_cast<const float4*>(cs + 4));
+        a[2] = __ldg(reinterpret_cast<const float4*>(sn));
+        a[3] = __ldg(reinterpret_cast<const float4*>(sn + 4));
+      };
+#pragma unroll
+      for (int j = 0; j < PRE; ++j) {
+        ang[j][0] = ang[j][1] = make_float4(1.f, 1.f, 1.f, 1.f);
+        ang[j][2] = ang[j][3] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i_turn && i_t < i_step && i_t + j * i_step < RC_CHUNK) load_angles(i_t + j * i_step, ang[j]);
+      }
       if (!mbar_wait(bar_l, ch & 1, abort_word)) { ok = false; *abort_word = ERR_WAIT_FULL; }
       if (i_t < i_step) {
-#pragma unroll 2
-        for (int t = i_t; t < RC_CHUNK; t += i_step) {
-          float c[8], s[8];
-#pragma unroll
-          for (int i = 0; i < 8; ++i) { c[i] = 1.f; s[i] = 0.f; }
-          if (i_turn) {
-            const float* cs = p.cos_sin + (long long)min(pos0 + t0 + min(t, n - 1), p.ctx - 1) * rot2 + i_d0;
-            const float* sn = cs + (long long)p.ctx * rot2;
-#pragma unroll
-            for (int i = 0; i < 8; i += 4) {
-              const float4 c4 = *reinterpret_cast<const float4*>(cs + i), s4 = *reinterpret_cast<const float4*>(sn + i);
-              c[i] = c4.x; c[i + 1] = c4.y; c[i + 2] = c4.z; c[i + 3] = c4.w;
-              s[i] = s4.x; s[i + 1] = s4.y; s[i + 2] = s4.z; s[i + 3] = s4.w;
-            }
-          }
+        auto item = [&](int t, const float4 (&an)[4]) __attribute__((always_inline)) {
+          const float c[8] = {an[0].x, an[0].y, an[0].z, an[0].w, an[1].x, an[1].y, an[1].z, an[1].w};
+          const float s[8] = {an[2].x, an[2].y, an[2].z, an[2].w, an[3].x, an[3].y, an[3].z, an[3].w};
           const float pw = t < n ? spow[n - 1 - t] : 1.f;
           const float fq = t < n ? __fdividef(1.f, pw) : 0.f, fk = t < n ? pw * kscale : 0.f;
           const uint32_t o0 = swz(t, i_d0 / 8), o1 = swz(t, i_d1 / 8);
@@ -429,6 +434,17 @@ __global__ void __launch_bounds__(RC_THREADS, 1) retention_chunk_kernel(const __
           };
           put(fq, L::OFF_QH, L::OFF_QL);
           put(fk, L::OFF_KH, L::OFF_KL);
+        };
+#pragma unroll
+        for (int j = 0; j < PRE; ++j)
+          if (i_t + j * i_step < RC_CHUNK) item(i_t + j * i_step, ang[j]);
+#pragma unroll 1
+        for (int t = i_t + PRE * i_step; t < RC_CHUNK; t += i_step) {
+          float4 an[4];
+          an[0] = an[1] = make_float4(1.f, 1.f, 1.f, 1.f);
+          an[2] = an[3] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (i_turn) load_angles(t, an);
+          item(t, an);
         }
       }
       for (int c8 = D / 8 + (tid >> 7); c8 < 16; c8 += 2) {          // columns past dim and vdim: neighbours' data
