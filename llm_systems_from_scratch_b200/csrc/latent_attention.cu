@@ -421,6 +421,11 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
   }
 }
 
+void launch_latent_merge(const float* part_o, const float* part_ml, __nv_bfloat16* o, int items, int splits, int width,
+                         cudaStream_t st) {
+  launch_dep(latent_merge_kernel, items, 128, 0, st, part_o, part_ml, o, splits, width);
+}
+
 template <int NT, int HG>
 static int launch_latent_decode(const LatentDecodeParams& p, cudaStream_t st) {
   constexpr int smem = LatentDecodeSmem<NT>::bytes(HG);
@@ -432,7 +437,7 @@ static int launch_latent_decode(const LatentDecodeParams& p, cudaStream_t st) {
   }
   launch_dep(kern, dim3(p.rows, (p.heads + HG * 16 - 1) / (HG * 16), p.splits), 256 * HG, smem, st, p);
   if (p.splits > 1)
-    launch_dep(latent_merge_kernel, p.rows * p.heads, 128, 0, st, p.part_o, p.part_ml, p.o, p.splits, p.width);
+    launch_latent_merge(p.part_o, p.part_ml, p.o, p.rows * p.heads, p.splits, p.width, st);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

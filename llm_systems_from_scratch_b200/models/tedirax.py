@@ -188,7 +188,7 @@ class Tedirax:
         total = len(ids) + max_new_tokens
         if self._engine is None or self._engine.max_context < total:
             ctx = -(-total // 256) * 256
-            self._engine = ServingEngine(self, num_pages=-(-ctx // 16), page_size=16, max_batch=1, max_context=ctx,
+            self._engine = ServingEngine(self, num_pages=-(-ctx // 64), page_size=64, max_batch=1, max_context=ctx,
                                          use_cuda_graphs=False)
         out = self._engine.generate([ids], max_new_tokens, eos_token_id, temperature, top_k)[0]
         if eos_token_id is not None and out and out[-1] == eos_token_id:

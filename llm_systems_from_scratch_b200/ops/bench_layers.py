@@ -70,13 +70,13 @@ def step_times(kind: str, s: dict, steps: int, warmup: int) -> dict:
     rec = {}
     g = torch.Generator().manual_seed(1)
     ids = lambda n: torch.randint(0, s["vocab"], (n,), generator=g).tolist()
-    eng = ServingEngine(model, num_pages=PROMPTS * PROMPT_LEN // 16, page_size=16, max_batch=PROMPTS, max_context=PROMPT_LEN,
+    eng = ServingEngine(model, num_pages=PROMPTS * PROMPT_LEN // 16, max_batch=PROMPTS, max_context=PROMPT_LEN,
                         max_prefill_tokens=PROMPTS * PROMPT_LEN)
     reqs = [Request(i, ids(PROMPT_LEN), 0) for i in range(PROMPTS)]
     for r in reqs:
         eng.sched.open(r)
         eng.sched.grow(r, PROMPT_LEN)
-    batch = StepBatch.build([(r, 0, r.prompt) for r in reqs], 16, eng.max_pages_per_req, eng.device)
+    batch = StepBatch.build([(r, 0, r.prompt) for r in reqs], eng.page_size, eng.max_pages_per_req, eng.device)
     last = torch.from_numpy(batch.last_rows()).to(eng.device)
     with torch.no_grad():
         run = lambda: eng.backend.logits(eng.backend.forward(batch), last)
@@ -88,7 +88,7 @@ def step_times(kind: str, s: dict, steps: int, warmup: int) -> dict:
     native.check_status()
     del eng, batch
     for b in DECODE_BATCHES:
-        eng = ServingEngine(model, num_pages=b * (-(-(CONTEXT + 64) // 16)) + 8, page_size=16, max_batch=b, max_context=2048)
+        eng = ServingEngine(model, num_pages=b * (-(-(CONTEXT + 64) // 16)) + 8, max_batch=b, max_context=2048)
         for i in range(b):
             eng.sched.add(Request(i, ids(CONTEXT), 64))
         eng._realtime, eng._virtual = False, float("inf")
@@ -225,13 +225,18 @@ def _prompt_kernels(s, t):
     # latents
     pr = _bf(rows, s["q_rank"] + s["kv_rank"] + hd)
     nq, nkv = _bf(s["q_rank"]), _bf(s["kv_rank"])
-    cache = torch.zeros(rows // 16, 16, s["kv_rank"], dtype=torch.bfloat16, device="cuda")
+    cache = torch.zeros(rows // 64, 64, s["kv_rank"], dtype=torch.bfloat16, device="cuda")
     sl = torch.randperm(rows, device="cuda")
     t.add("latent_norm_append", "rmsnorm_fwd", timeit(lambda: mo.latent_norm_append(pr, nq, nkv, 1e-6, cache, sl)),
           rows * (s["q_rank"] + s["kv_rank"]) * 4)
-    tables = torch.randperm(rows // 16, device="cuda").int().view(PROMPTS, PROMPT_LEN // 16)
+    tables = torch.randperm(rows // 64, device="cuda").int().view(PROMPTS, PROMPT_LEN // 64)
     first = torch.zeros(PROMPTS, dtype=torch.int32, device="cuda")
-    t.add("latent_gather", "rmsnorm_fwd", timeit(lambda: mo.latent_gather(cache, cu, first, tables, rows)), rows * s["kv_rank"] * 4)
+    del cache
+
+    def gather():
+        c = torch.zeros(rows // 64, 64, s["kv_rank"], dtype=torch.bfloat16, device="cuda")
+        return lambda: mo.latent_gather(c, cu, first, tables, rows)
+    t.add("latent_gather", "rmsnorm_fwd", graph_ms(gather, rows * s["kv_rank"] * 4), rows * s["kv_rank"] * 4)
 
 
 def _expert_kernels(s, t, rows, tokens):
@@ -290,7 +295,10 @@ def _decode_kernels(s, t, b):
     add("paged_decode (TransformerLM)", "-", b * CONTEXT * hd * 4, 0, paged)
 
     def latent():
-        ql, cache, tb = _bf(b, heads * kvr), _bf(b * pages, 16, kvr), tables()
+        n = -(-pages // 4)                            # pages of 64 tokens
+        tb = torch.zeros(b, 32, dtype=torch.int32, device="cuda")
+        tb[:, :n] = torch.randperm(b * n, device="cuda").int().view(b, n)
+        ql, cache = _bf(b, heads * kvr), _bf(b * n, 64, kvr)
         return lambda: mo.latent_decode(ql, cache, pos, slots, tb, heads, s["window"], 0.1)
     add(f"latent_decode, window {win}", "paged_decode", b * (win * kvr * 2 + heads * kvr * 4), 4.0 * b * heads * win * kvr, latent)
     table, decay = torch.randn(2, 2048, 64, device="cuda"), torch.full((heads,), 0.99, device="cuda")

@@ -34,6 +34,7 @@ def _lib():
             "b200_latent_gather": [P, P, P, P, P, I, I, I, I, I, I, P, P],
             "b200_latent_attn_rows": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
             "b200_latent_decode": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
+            "b200_latent_decode_tc": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
             "b200_flash_window_fwd": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, L, L, L, L, P, P],
             "b200_retention_chunk": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
             "b200_retention_recurrent": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
@@ -271,23 +272,43 @@ def latent_splits(rows: int, heads: int, keys: int, sms: int = 148) -> int:
     return best
 
 
-def latent_decode(q, cache, positions, slots, tables, heads: int, window: int, scale: float, splits: int = 0):
-    """``latent_attention_rows`` for one query row per request: line i of ``tables`` belongs to row i."""
-    width = cache.shape[-1]
-    if not q.is_cuda or q.dtype != torch.bfloat16 or width > DECODE_MAX_WIDTH:
+def latent_splits_tc(rows: int, keys: int, sms: int = 148) -> int:
+    """The same for the tcgen05 kernel: one CTA per SM, tiles of 128 tokens (one more for the page border the window starts
+    behind), a start-up worth about one and a half tiles and a merge worth about one."""
+    best, best_cost = 1, None
+    for n in range(1, max(1, min(16, keys // 256)) + 1):
+        cost = -(-rows * n // sms) * (-(-(keys // 128 + 1) // n) + 1.5) + (1 if n > 1 else 0)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = n, cost
+    return best
+
+
+def latent_decode(q, cache, positions, slots, tables, heads: int, window: int, scale: float, splits: int = 0, kernel: str = "auto"):
+    """``latent_attention_rows`` for one query row per request: line i of ``tables`` belongs to row i.  ``kernel``: "tcgen05"
+    (widths that are multiples of 128, up to 64 heads, pages that divide 128), "mma" (any width up to 512), "rows"; "auto"
+    takes the first that fits, and "mma" for small batches, whose CTAs it spreads over the SMs with shorter chains."""
+    width, page = cache.shape[-1], cache.shape[1]
+    if kernel == "auto":
+        fits = q.is_cuda and q.dtype == torch.bfloat16 and width <= DECODE_MAX_WIDTH
+        tc = fits and width % 128 == 0 and heads <= 64 and page >= 8 and 128 % page == 0 and q.shape[0] * max(heads, 16) >= 1024
+        kernel = "tcgen05" if tc else ("mma" if fits else "rows")
+    if kernel == "rows":
         return latent_attention_rows(q, cache, None, positions, slots, tables, heads, window, scale)
     rows = q.shape[0]
     _req(q.is_contiguous() and cache.is_contiguous() and q.shape[1] == heads * width and tables.shape[0] >= rows, "bad latent queries")
+    _req(q.dtype == torch.bfloat16 and cache.dtype == q.dtype, "bf16 queries and latents")
     _req(tables.dtype == torch.int32 and tables.is_contiguous() and positions.dtype == torch.int32, "bad tables")
-    page = cache.shape[1]
     keys = tables.shape[1] * page
-    splits = splits or latent_splits(rows, heads, min(window, keys) if window > 0 else keys)
+    keys = min(window, keys) if window > 0 else keys
+    if kernel == "tcgen05":
+        fn, splits = _lib().b200_latent_decode_tc, splits or latent_splits_tc(rows, keys)
+    else:
+        fn, splits = _lib().b200_latent_decode, splits or latent_splits(rows, heads, keys)
     out = torch.empty_like(q)
     part = torch.empty(rows * heads * splits * (width + 2) if splits > 1 else 0, dtype=torch.float32, device=q.device)
     ml = part[rows * heads * splits * width:]
-    _check(_lib().b200_latent_decode(_ptr(q), _ptr(cache), _ptr(out), _ptr(part), _ptr(ml), _ptr(positions), _ptr(slots),
-                                     _ptr(tables), rows, heads, width, tables.shape[1], page, cache.shape[0], window, splits,
-                                     float(scale), _ptr(native.status_word(q.device)), _stream()),
+    _check(fn(_ptr(q), _ptr(cache), _ptr(out), _ptr(part), _ptr(ml), _ptr(positions), _ptr(slots), _ptr(tables), rows, heads, width,
+              tables.shape[1], page, cache.shape[0], window, splits, float(scale), _ptr(native.status_word(q.device)), _stream()),
            "latent_decode" if splits > 1 else "latent_decode_one")
     return out
 

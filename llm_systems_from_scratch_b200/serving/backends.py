@@ -19,6 +19,7 @@ class TransformerBackend:
     """``TransformerLM``: packed QKV attention with rotary pairs, K and V pages, bf16 residual stream."""
 
     splits_prompts = False
+    page_size = 16
 
     def __init__(self, model):
         model.use_custom_triton = True
@@ -104,6 +105,7 @@ class LayeredBackend:
     the experts read them), the mixer (adds to the residual stream in its last product), the experts."""
 
     splits_prompts = True
+    page_size = 64                    # tokens: the decode kernel copies whole pages as TMA boxes
 
     def __init__(self, model):
         self.model = model

@@ -30,7 +30,7 @@ from .scheduler import Request, Scheduler
 class ServingEngine:
     BUCKETS = (1, 2, 4, 8, 16, 32, 64, 128, 256)
 
-    def __init__(self, model, num_pages: int | None = None, page_size: int = 16, max_batch: int = 64,
+    def __init__(self, model, num_pages: int | None = None, page_size: int | None = None, max_batch: int = 64,
                  max_context: int | None = None, max_prefill_tokens: int = 8192, use_cuda_graphs: bool = True,
                  kv_memory_fraction: float = 0.5):
         self.backend = be = model.serving_backend()
@@ -40,7 +40,7 @@ class ServingEngine:
         if be.context_limit is not None:
             self.max_context = min(self.max_context, be.context_limit)
         be.set_context(self.max_context)
-        self.page_size = page_size
+        self.page_size = page_size = page_size or be.page_size
         self.max_pages_per_req = -(-self.max_context // page_size)
         if num_pages is None:
             per_page = be.page_bytes(page_size)

@@ -21,9 +21,8 @@ import sys
 
 import torch
 
-PAGE_SIZE = 16
 MAX_REQUESTS = 4            # live at a time
-ROUND_TO = 64               # --max-tokens counts every request rounded up to this
+ROUND_TO = 64               # --max-tokens counts every request rounded up to this: a multiple of every page size in use
 
 
 def open_engine(folder: str, dtype: torch.dtype, max_tokens: int, device="cuda"):
@@ -31,7 +30,8 @@ def open_engine(folder: str, dtype: torch.dtype, max_tokens: int, device="cuda")
     from ..models.registry import load_model
     from .engine import ServingEngine
     model = load_model(folder, dtype, device)
-    return ServingEngine(model, num_pages=-(-max_tokens // PAGE_SIZE), page_size=PAGE_SIZE, max_batch=MAX_REQUESTS,
+    page = model.serving_backend().page_size
+    return ServingEngine(model, num_pages=-(-max_tokens // page), page_size=page, max_batch=MAX_REQUESTS,
                          max_context=-(-max_tokens // ROUND_TO) * ROUND_TO, use_cuda_graphs=False)
 
 

@@ -193,7 +193,8 @@ def stand_out(latents, q, pos, window, heads, width):
 
 
 @pytest.mark.parametrize("width,heads,window,page", [(24, 3, 7, 4), (128, 16, 40, 16), (72, 6, 33, 16), (136, 20, 64, 16),
-                                                     (256, 8, 1, 16), (512, 17, 300, 16), (512, 16, 0, 64), (8, 40, 65, 5)])
+                                                     (256, 8, 1, 16), (512, 17, 300, 16), (512, 16, 0, 64), (8, 40, 65, 5),
+                                                     (384, 33, 130, 8), (512, 5, 129, 32), (256, 64, 128, 128)])
 @pytest.mark.parametrize("splits", [0, 1, 3])
 def test_latent_decode_at_every_edge(width, heads, window, page, splits):
     mo = mops()
@@ -208,17 +209,19 @@ def test_latent_decode_at_every_edge(width, heads, window, page, splits):
     pos = torch.tensor([n - 1 for n in lens], dtype=torch.int32, device="cuda")
     slots = torch.zeros(len(lens), dtype=torch.int64, device="cuda")
     slots[4] = -1
-    got = mo.latent_decode(q, cache, pos, slots, tables, heads, window, scale, splits)
+    got = [mo.latent_decode(q, cache, pos, slots, tables, heads, window, scale, splits, k)
+           for k in ("mma", *(("tcgen05",) if width % 128 == 0 else ()))]
     rows = mo.latent_attention_rows(q, cache, None, pos, slots, tables, heads, window, scale)
     for i, n in enumerate(lens):
         if i == 4:
-            assert float(got[i].abs().sum()) == 0.0 and float(rows[i].abs().sum()) == 0.0
+            assert all(float(g[i].abs().sum()) == 0.0 for g in (*got, rows))
             continue
         c = lat[i].double().cpu()[:, None, :].expand(n, heads, width)
         qs = torch.zeros(n, heads, width, dtype=torch.float64)
         qs[-1] = q[i].double().cpu().view(heads, width)
         want = O.window_attention(qs, c, c, scale, window or 10 ** 6)[-1].reshape(-1)
-        close(got[i], want, 1.5e-2)
+        for g in got:
+            close(g[i], want, 1.5e-2)
         close(rows[i], want, 1e-2)
 
 
@@ -430,6 +433,20 @@ def test_models_in_every_cut_and_company(name, dtype):
         for i in range(6):
             assert H.error(got[i], want[i]) < TOL[dtype], (i, schedule[:3])
         assert eng.cache.allocator.free == 64 and eng.cache.slot_allocator.free == 4
+
+
+@pytest.mark.parametrize("heads", [8, 20])
+def test_a_large_batch_decodes_on_the_token_tiles(heads):
+    """Enough requests for the tcgen05 decode kernel, which small batches do not use; a page holds more than one window."""
+    cfg = H.config(90, 48, [H.latent(heads, 24, 16, 40, 128, 30, mlp=H.moe(16, 3, 2)), H.retention(2, 16, 16, [0.98, 0.9])])
+    ts = H.tensors(cfg)
+    lens = [5 + (7 * i) % 90 for i in range(70)]
+    seqs = H.prompts(cfg, lens)
+    want = H.expected(cfg, ts, seqs)
+    eng = engine(cfg, ts, BF, num_pages=160, page_size=64, max_batch=70)
+    steps = [[(i, n - 4) for i, n in enumerate(lens)]] + [[(i, 1) for i in range(70)]] * 4
+    for g, w in zip(H.feed(eng, seqs, steps, poison=True), want):
+        assert H.error(g, w) < TOL[BF]
 
 
 def test_long_decoding_stays_exact():
