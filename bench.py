@@ -29,6 +29,11 @@ version of the same measurement (``--serving-requests`` requests, 0 switches it 
 ``serving`` of its JSON line, so that one command reports both halves.  The reference has no serving
 engine; its arm replays the head of the same trace through its ``TransformerLM`` with a per-request greedy
 loop that re-runs the whole context for every token (what its ``generate`` does) for a bounded time.
+
+    python bench.py --workload layers [--layers-sizes 0.35b,1.3b,7b-8layers]
+
+times the layered decoder (Tedirax) beside the TransformerLM at equal size on one GPU: whole prompt and decode steps and
+every kernel against its roofline, one line per size (``ops/bench_layers.py``).
 """
 from __future__ import annotations
 

@@ -1,4 +1,4 @@
-// Retention: linear attention with a fixed decay per head.  Per head S_t = decay S_(t-1) + k_t v_t^T and o_t = S_t^T q_t with
+// Retention: attention without softmax whose memory is a decaying matrix.  Per head S_t = decay S_(t-1) + k_t v_t^T and o_t = S_t^T q_t with
 // rotated q, k (rotate-half pairs, 32-bit angles) and k scaled by dim^(-1/2); the output of a head is divided by its root
 // mean square and multiplied by silu(gate).  The state (heads, dim, vdim) is fp32 and lives in a slot per request.
 #include "typed.cuh"

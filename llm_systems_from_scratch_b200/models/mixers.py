@@ -35,7 +35,7 @@ class LatentAttention:
     """Attention whose keys and values are linear images of one cached latent per token; no positions.
 
     q = W_uq rms_norm(W_dq h), c = rms_norm(W_dkv h), k_h = W_uk,h c, v_h = W_uv,h c, softmax(scale q.k) over the last
-    ``window`` positions (0 = all), heads multiplied by sigmoid(W_g h), then W_o.  Only c is cached."""
+    ``window`` positions (0 = all), heads multiplied by sigmoid(W_g h), then W_o.  The cache holds c alone."""
 
     def __init__(self, get, width: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, window: int,
                  eps: float, dtype, device):
@@ -105,8 +105,8 @@ class LatentAttention:
 
 
 class Retention:
-    """Linear attention with a fixed decay per head, rotary q and k (rotate-half over the first ``rot_dims`` dimensions), no
-    softmax; heads are divided by their root mean square, multiplied by silu(W_g h), then W_o.  The state is fp32."""
+    """Attention without softmax whose memory is a decaying matrix per head: S <- d S + k v^T, read by q; rotary q and k (rotate-half over the
+    first ``rot_dims`` dimensions); heads are divided by their root mean square, multiplied by silu(W_g h), then W_o.  The state is fp32."""
 
     MIN_CHUNKED = 8            # the longest portion of a step from which the chunked kernel is used
 

@@ -182,7 +182,7 @@ class Tedirax:
     def generate(self, prompt_ids, max_new_tokens: int, temperature: float = 1.0, top_k: int | None = None,
                  eos_token_id: int | None = None):
         """Up to ``max_new_tokens`` ids after the prompt, shape (1, n), through the serving engine; the stop token is not
-        returned (the contract of ``TransformerLM.generate``)."""
+        returned (as in ``TransformerLM.generate``)."""
         from ..serving import ServingEngine
         ids = prompt_ids.reshape(-1).tolist()
         total = len(ids) + max_new_tokens

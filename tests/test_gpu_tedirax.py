@@ -192,7 +192,7 @@ def stand_out(latents, q, pos, window, heads, width):
     return c
 
 
-@pytest.mark.parametrize("width,heads,window,page", [(24, 3, 7, 4), (128, 16, 40, 16), (72, 6, 33, 16), (136, 20, 64, 16),
+@pytest.mark.parametrize("width,heads,window,page", [(24, 3, 7, 4), (128, 16, 44, 16), (72, 6, 33, 16), (136, 20, 64, 16),
                                                      (256, 8, 1, 16), (512, 17, 300, 16), (512, 16, 0, 64), (8, 40, 65, 5),
                                                      (384, 33, 130, 8), (512, 5, 129, 32), (256, 64, 128, 128)])
 @pytest.mark.parametrize("splits", [0, 1, 3])
@@ -245,7 +245,7 @@ def test_latent_rows_of_portions(dtype):
 
 
 @pytest.mark.parametrize("dh,vdim,heads", [(64, 64, 2), (64, 20, 3), (128, 128, 2), (128, 72, 1)])
-@pytest.mark.parametrize("window", [0, 1, 40, 127, 128, 129, 300])
+@pytest.mark.parametrize("window", [0, 1, 45, 127, 128, 129, 300])
 def test_window_attention_of_portions(dh, vdim, heads, window):
     """Portions of unequal length, some with earlier tokens in front; one key just inside and one just outside the last
     query's window stand out."""
@@ -304,8 +304,8 @@ def retention_case(lens, heads, dim, vdim, dims, decay, dtype, start_states=None
     return proj, outs, states
 
 
-CASES = [(3, 10, 7, 6, [0.9, 0.5, 0.99]), (2, 64, 64, 64, [0.99, 0.96875]), (3, 48, 24, 16, [0.9, 0.97, 0.995]),
-         (1, 128, 128, 128, [0.9990234375]), (2, 128, 72, 0, [0.85, 1.0]), (1, 16, 136, 16, [0.75]),
+CASES = [(3, 10, 7, 6, [0.9, 0.5, 0.99]), (3, 64, 64, 48, [0.99, 0.96875, 0.95]), (3, 48, 24, 16, [0.9, 0.97, 0.995]),
+         (1, 128, 128, 128, [0.9985]), (2, 128, 72, 0, [0.85, 1.0]), (1, 16, 136, 16, [0.75]),
          (1, 40, 96, 32, [0.97]), (14, 128, 128, 96, [0.9 + 0.007 * i for i in range(14)])]
 
 
@@ -362,7 +362,7 @@ def test_retention_token_by_token_and_in_portions(heads, dim, vdim, dims, decay,
 def test_retention_remembers_a_far_token():
     """One token 250 positions back carries nearly all of the state; a lost or wrongly decayed state shows at once."""
     mo = mops()
-    decay, n = [0.9990234375], 260
+    decay, n = [0.9985], 260
     proj = randn(n, 4 * 64, seed=1, dtype=BF, scale=0.05)
     proj[3, 64:128], proj[3, 128:192] = 8.0, 5.0
     proj[:, 192:] *= 30.0
