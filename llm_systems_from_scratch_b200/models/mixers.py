@@ -105,8 +105,9 @@ class LatentAttention:
 
 
 class Retention:
-    """Attention without softmax whose memory is a decaying matrix per head: S <- d S + k v^T, read by q; rotary q and k (rotate-half over the
-    first ``rot_dims`` dimensions); heads are divided by their root mean square, multiplied by silu(W_g h), then W_o.  The state is fp32."""
+    """Attention without softmax whose memory is a decaying matrix per head: S <- d S + k v^T, read by q.  q and k are
+    rotated (rotate-half over the first ``rot_dims`` dimensions); heads are divided by their root mean square, multiplied
+    by silu(W_g h), then W_o.  The state is fp32."""
 
     MIN_CHUNKED = 8            # the longest portion of a step from which the chunked kernel is used
 
