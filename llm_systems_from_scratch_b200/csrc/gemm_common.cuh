@@ -81,6 +81,7 @@ struct GemmParams {
   const int* tile_group;
   int group_rows;
   int batch, a_step, c_step;
+  int relu;                   // gated instances of the single-CTA kernel: relu(gate) * up instead of silu(gate) * up
   int splits;
   float* ws;                  // splits * tiles partial tiles of BM x BN floats
   uint32_t* tile_counters;    // four per tile (one per 32-row quarter), zero between launches (the last warp resets its own)

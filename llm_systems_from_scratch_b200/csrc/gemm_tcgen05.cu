@@ -31,7 +31,7 @@ struct GemmSmem {
 enum GemmGroup : int { GROUP_NONE = 0, GROUP_ROWS = 1, GROUP_COLS = 2 };
 
 // SWIGLU (grouped kernels): B holds group_rows = 2 N rows per group, gate rows first; a BN-wide tile is BN / 2 gate rows
-// and the matching BN / 2 up rows, and the epilogue stores silu(gate) * up.
+// and the matching BN / 2 up rows, and the epilogue stores silu(gate) * up (or relu(gate) * up).
 template <int BN, bool A_MN, bool B_MN, int STAGES, int GROUP = GROUP_NONE, bool SWIGLU = false>
 __global__ void __launch_bounds__(192, 1)
 gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
@@ -77,10 +77,11 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
         const int kb_lo = split * nkb / sp, kb_hi = (split + 1) * nkb / sp;
         int m_blk, n_blk;
         tile_coords(GROUP == GROUP_COLS ? tile % per_problem : tile, p, m_blk, n_blk);
-        const int brow = (GROUP == GROUP_COLS ? (tile / per_problem) * p.group_rows : 0) + n_blk * BN;
+        const int brow = (GROUP == GROUP_COLS ? (tile / per_problem) * p.group_rows : 0) + n_blk * (SWIGLU ? BN / 2 : BN);
         for (int i = 0; i < STAGES && kb_lo + i < kb_hi; ++i) {
           mbar_expect_tx(&full_bar[i], S::A_BYTES + S::B_BYTES);
           tma_load_2d(smem_b + i * S::B_BYTES, &tmB, &full_bar[i], (kb_lo + i) * BK, brow);
+          if (SWIGLU) tma_load_2d(smem_b + i * S::B_BYTES + S::B_BYTES / 2, &tmB, &full_bar[i], (kb_lo + i) * BK, brow + p.N);
         }
       }
     }
@@ -144,10 +145,10 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
           if (B_MN) {
 #pragma unroll
             for (int j = 0; j < BN / 64; ++j) tma_load_2d(b_dst + j * 8192, &tmB, &full_bar[stage], n0 + j * 64, k0);
-          } else if (SWIGLU) {
+          } else if (SWIGLU && !posted) {
             tma_load_2d(b_dst, &tmB, &full_bar[stage], k0, n0);
             tma_load_2d(b_dst + S::B_BYTES / 2, &tmB, &full_bar[stage], k0, n0 + p.N);
-          } else if (!posted) {
+          } else if (!SWIGLU && !posted) {
             tma_load_2d(b_dst, &tmB, &full_bar[stage], k0, n0);
           }
           if (++stage == STAGES) {
@@ -246,9 +247,10 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const float g = __uint_as_float(r[j]);
-            r[j] = __float_as_uint(__fdividef(g, 1.f + __expf(-g)) * __uint_as_float(u[j]));
+            const float a = p.relu ? fmaxf(g, 0.f) : __fdividef(g, 1.f + __expf(-g));
+            r[j] = __float_as_uint(a * __uint_as_float(u[j]));
           }
-          epilogue_store(p, row, n0 + c * 32, r);
+          epilogue_store(p, row, n0 + c * 32, r, coff);
         }
         tc_fence_before();
         mbar_arrive(&tmem_empty[acc]);
@@ -513,7 +515,7 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, const void* R, 
   p.swiglu_f = 0; p.H = nullptr; p.ldh = 0;
   p.splits = splits > 1 ? splits : 1; p.ws = ws; p.tile_counters = tile_counters;
   p.b_early = b_early;
-  p.tile_group = nullptr; p.group_rows = 0; p.batch = 1; p.a_step = p.c_step = 0;
+  p.tile_group = nullptr; p.group_rows = 0; p.batch = 1; p.a_step = p.c_step = 0; p.relu = 0;
 
 #define DISPATCH(BN_)                                                                    \
   if (a_mn && b_mn) return launch_gemm<BN_, true, true>(tmA, tmB, p, max_ctas, stream);   \
@@ -597,6 +599,8 @@ extern "C" int b200_gemm_bf16_splitk(const void* A, const void* B, void* C, cons
 //     silu(gate) * up, otherwise group_rows == N.
 //   tile_group == null: `batch` problems side by side: problem g multiplies A[:, g * a_step : g * a_step + K] with
 //     B[g * group_rows : g * group_rows + N, :] into C[:, g * c_step : g * c_step + N].  a_step must be a multiple of 8.
+//     With `swiglu` B has the 2 N rows of one gated feed-forward per problem, as above (any M).
+// swiglu: 0 off, 1 silu(gate) * up, 2 relu(gate) * up.
 // Columns of A past a problem's K (up to the next multiple of 64) are multiplied with zeros, so they must be finite.
 extern "C" int b200_gemm_bf16_grouped(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
                                       long long lda, long long ldb, long long ldc, long long ldr, const int* tile_group,
@@ -611,7 +615,8 @@ extern "C" int b200_gemm_bf16_grouped(const void* A, const void* B, void* C, con
   if (epi != EPI_BF16 && epi != EPI_F32 && epi != EPI_BF16_GATE) return -11;
   if (epi == EPI_BF16_GATE && (R == nullptr || rows)) return -11;
   if (rows && ((M % BM) || n_groups <= 0 || group_rows != (swiglu ? 2 * N : N))) return -12;
-  if (!rows && (swiglu || batch <= 0 || (a_step & 7) || group_rows < N)) return -12;
+  if (!rows && (batch <= 0 || (a_step & 7) || group_rows < (swiglu ? 2 * N : N))) return -12;
+  if (swiglu < 0 || swiglu > 2 || (swiglu && epi != EPI_BF16)) return -12;
   const int sms = num_sms();
   const long long mt = (M + BM - 1) / BM, problems = rows ? 1 : batch;
   int bn = 64;
@@ -642,7 +647,12 @@ extern "C" int b200_gemm_bf16_grouped(const void* A, const void* B, void* C, con
   p.swiglu_f = 0; p.H = nullptr; p.ldh = 0;
   p.splits = 1; p.ws = nullptr; p.tile_counters = nullptr;
   p.b_early = b_early;
-  p.tile_group = tile_group; p.group_rows = group_rows; p.batch = rows ? 1 : batch; p.a_step = a_step; p.c_step = c_step;
+  p.tile_group = tile_group; p.group_rows = group_rows; p.batch = rows ? 1 : batch; p.a_step = a_step; p.c_step = c_step; p.relu = swiglu == 2;
+  if (!rows && swiglu) {
+    if (bn == 256) return launch_gemm<256, false, false, GROUP_COLS, true>(tmA, tmB, p, 0, stream);
+    if (bn == 128) return launch_gemm<128, false, false, GROUP_COLS, true>(tmA, tmB, p, 0, stream);
+    return launch_gemm<64, false, false, GROUP_COLS, true>(tmA, tmB, p, 0, stream);
+  }
   if (rows && swiglu) {
     if (bn == 256) return launch_gemm<256, false, false, GROUP_ROWS, true>(tmA, tmB, p, 0, stream);
     if (bn == 128) return launch_gemm<128, false, false, GROUP_ROWS, true>(tmA, tmB, p, 0, stream);

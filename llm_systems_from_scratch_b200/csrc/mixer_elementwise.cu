@@ -133,6 +133,89 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormPa
   }
 }
 
+// Norms behind the sublayers: x += y / rms(y) * w for a sublayer's output y, and h = x in the activation type, which the next
+// sublayer reads.  With `tokens` the row starts: x = embed[token].  One block per row; a thread keeps its columns of y and x in
+// registers between the passes (KEEP groups; wider rows are read again).
+struct AddNormedParams {
+  const long long* tokens;
+  const void *embed, *y, *w;
+  float* x;
+  void* h;
+  int vocab, d;
+  long long ld_y, ld_h;
+  float eps;
+  uint32_t* status;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) add_normed_kernel(const AddNormedParams p) {
+  pdl_sync();
+  __shared__ float red[32];
+  const long long row = blockIdx.x;
+  float* xr = p.x + row * p.d;
+  T* hr = reinterpret_cast<T*>(p.h) + row * p.ld_h;
+  if (p.tokens != nullptr) {
+    long long tok = p.tokens[row];
+    if (tok < 0 || tok >= p.vocab) {
+      if (threadIdx.x == 0) report_bad_arg(p.status, 20);
+      tok = 0;
+    }
+    const T* er = reinterpret_cast<const T*>(p.embed) + tok * p.d;
+    for (int c = threadIdx.x * VEC; c < p.d; c += blockDim.x * VEC) {
+      float f[VEC];
+      load_vec<VEC>(er + c, f);
+      store_vec<VEC>(xr + c, f);
+      store_vec<VEC>(hr + c, f);
+    }
+    return;
+  }
+  const T* yr = reinterpret_cast<const T*>(p.y) + row * p.ld_y;
+  const T* w = reinterpret_cast<const T*>(p.w);
+  constexpr int KEEP = 4;
+  float y[KEEP][VEC], x[KEEP][VEC];
+  const int step = blockDim.x * VEC;
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * VEC + j * step;
+    if (c < p.d) {
+      load_vec<VEC>(yr + c, y[j]);
+      load_vec<VEC>(xr + c, x[j]);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss += y[j][i] * y[j][i];
+    }
+  }
+  for (int c = threadIdx.x * VEC + KEEP * step; c < p.d; c += step) {
+    float f[VEC];
+    load_vec<VEC>(yr + c, f);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss += f[i] * f[i];
+  }
+  const float r = rsqrtf(block_total(ss, red) / (float)p.d + p.eps);
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * VEC + j * step;
+    if (c < p.d) {
+      float g[VEC];
+      load_vec<VEC>(w + c, g);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) x[j][i] += y[j][i] * r * g[i];
+      store_vec<VEC>(xr + c, x[j]);
+      store_vec<VEC>(hr + c, x[j]);
+    }
+  }
+  for (int c = threadIdx.x * VEC + KEEP * step; c < p.d; c += step) {
+    float f[VEC], g[VEC], v[VEC];
+    load_vec<VEC>(yr + c, f);
+    load_vec<VEC>(xr + c, v);
+    load_vec<VEC>(w + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] += f[i] * r * g[i];
+    store_vec<VEC>(xr + c, v);
+    store_vec<VEC>(hr + c, v);
+  }
+}
+
 // -------------------------------------------------------------------------------------------------- mixture of experts
 // Plan of a mixture of experts whose experts are looked up by token id: sort the (row, choice) pairs by expert into
 // 128-row tiles that each belong to one expert.  One block per layer (every layer has its own table).
@@ -215,17 +298,17 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const MoePlanParams p) {
   }
 }
 
-// h = silu(gate) * up for gu (rows, 2F), gate columns first; any F, any row pitch.
+// h = act(gate) * up for gu (rows, 2F), gate columns first; any F, any row pitch.  act: silu, or relu.
 template <typename T>
-__global__ void silu_mul_any_kernel(const T* __restrict__ gu, T* __restrict__ h, long long rows, int F, long long ld_gu,
-                                    long long ld_h) {
+__global__ void glu_any_kernel(const T* __restrict__ gu, T* __restrict__ h, long long rows, int F, long long ld_gu,
+                               long long ld_h, int relu) {
   pdl_sync();
   const long long n = rows * F;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / F;
     const int c = (int)(i - r * F);
     const float g = to_f(gu[r * ld_gu + c]), u = to_f(gu[r * ld_gu + F + c]);
-    from_f(h[r * ld_h + c], g / (1.f + expf(-g)) * u);
+    from_f(h[r * ld_h + c], (relu ? fmaxf(g, 0.f) : g / (1.f + expf(-g))) * u);
   }
 }
 
@@ -311,14 +394,39 @@ extern "C" int b200_moe_plan(const long long* tokens, const long long* slots, in
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-extern "C" int b200_silu_mul_any(const void* gu, void* h, long long rows, int F, long long ld_gu, long long ld_h, int f32,
-                                 cudaStream_t st) {
+// y: (rows, ld_y) sublayer output to norm and add, or tokens / embed to start the rows.  See AddNormedParams.
+extern "C" int b200_add_normed(const long long* tokens, const void* embed, int vocab, float* x, const void* y, long long ld_y,
+                               const void* w, void* h, long long ld_h, float eps, int rows, int d, int f32, uint32_t* status,
+                               cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (d <= 0 || x == nullptr || h == nullptr || (tokens != nullptr ? embed == nullptr : (y == nullptr || w == nullptr))) return -10;
+  AddNormedParams p;
+  p.tokens = tokens; p.embed = embed; p.vocab = vocab; p.x = x; p.y = y; p.ld_y = ld_y; p.w = w; p.h = h; p.ld_h = ld_h;
+  p.eps = eps; p.d = d; p.status = status;
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(embed) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) |
+                         reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(h);
+  const bool vec = d % 4 == 0 && ld_y % 4 == 0 && ld_h % 4 == 0 && (ptrs & 15) == 0;
+  const int per = vec ? 8 : 2;                       // two groups per thread
+  int threads = ((d + per - 1) / per + 31) / 32 * 32;
+  if (threads > 256) threads = 256;
+  if (f32) {
+    if (vec) launch_dep(add_normed_kernel<float, 4>, rows, threads, 0, st, p);
+    else launch_dep(add_normed_kernel<float, 1>, rows, threads, 0, st, p);
+  } else {
+    if (vec) launch_dep(add_normed_kernel<__nv_bfloat16, 4>, rows, threads, 0, st, p);
+    else launch_dep(add_normed_kernel<__nv_bfloat16, 1>, rows, threads, 0, st, p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+extern "C" int b200_glu_any(const void* gu, void* h, long long rows, int F, long long ld_gu, long long ld_h, int relu, int f32,
+                            cudaStream_t st) {
   if (rows <= 0) return 0;
   const int g = blocks_for(rows * F, 256);
-  if (f32) launch_dep(silu_mul_any_kernel<float>, g, 256, 0, st, (const float*)gu, (float*)h, rows, F, ld_gu, ld_h);
+  if (f32) launch_dep(glu_any_kernel<float>, g, 256, 0, st, (const float*)gu, (float*)h, rows, F, ld_gu, ld_h, relu);
   else
-    launch_dep(silu_mul_any_kernel<__nv_bfloat16>, g, 256, 0, st, (const __nv_bfloat16*)gu, (__nv_bfloat16*)h, rows, F,
-               ld_gu, ld_h);
+    launch_dep(glu_any_kernel<__nv_bfloat16>, g, 256, 0, st, (const __nv_bfloat16*)gu, (__nv_bfloat16*)h, rows, F, ld_gu, ld_h,
+               relu);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

@@ -3,17 +3,21 @@
 Each class takes its sizes and constants as arguments, packs its weights for the kernels (matrices that read the same
 input become one product; heads are padded to what the kernels tile by) and runs one step of the engine:
 
-* a mixer is called with the normed rows ``h``, the fp32 residual stream ``x`` (it adds its output there in the epilogue
-  of its output projection), the ``StepBatch`` and its own part of the cache; ``cache_spec()`` says what that is
-* a feed-forward returns outputs that the next pass over the residual stream adds (``ops.mixer_ops.residual_norm``)
+* a mixer is called with its input rows ``h``, the fp32 residual stream ``x``, the ``StepBatch`` and its own part of the
+  cache (``cache_spec()`` says what that is).  It adds its output to ``x`` in the epilogue of its output projection, or
+  returns it when ``x`` is None (designs that norm a sublayer's output before they add it)
+* a feed-forward returns outputs that the next pass over the residual stream adds (``ops.mixer_ops.residual_norm``,
+  ``add_normed``)
 
 ``get(name)`` gives a weight in its stored layout ([out, in])."""
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..ops import mixer_ops as mo
-from ..serving.kv_cache import PagedSpec, StateSpec
+from ..serving.kv_cache import PagedSpec, SharedSpec, StateSpec
 
 
 def _head_pad(w, heads: int, rows: int, to: int):
@@ -29,6 +33,11 @@ def _expect(name: str, t, *shape):
     if tuple(t.shape) != shape:
         raise ValueError(f"{name} has shape {tuple(t.shape)}, expected {shape}")
     return t
+
+
+def _project(y, w_o, x):
+    """The output projection, into the residual stream or returned."""
+    return mo.linear(y, w_o) if x is None else mo.linear(y, w_o, out=x, accumulate=True)
 
 
 class LatentAttention:
@@ -86,7 +95,7 @@ class LatentAttention:
             mo.gemm_heads(ol, self.w_uv, heads, self.latent, self.vdim, out=o[:n], gate=gate[:n])
         if batch.n_rows > n:
             self._portions(q[n:], gate[n:], o[n:], batch, cache, slice(n, batch.n_rows))
-        mo.linear(o, self.w_o, out=x, accumulate=True)
+        return _project(o, self.w_o, x)
 
     def _portions(self, q, gate, o, batch, cache, rows: slice):
         heads = self.heads
@@ -145,22 +154,177 @@ class Retention:
                                  self.heads, self.dim, self.vdim, self.rot, self.eps, y[n:])
         elif batch.n_rows > n:
             run(slice(n, batch.n_rows), batch.state_slots[n:], batch.cu, batch.spans)
-        mo.linear(y, self.w_o, out=x, accumulate=True)
+        return _project(y, self.w_o, x)
+
+
+class MatrixMemory:
+    """Matrix memory with exponential gates (mLSTM of xLSTM): per head S <- f S + i k v^T and a normaliser n <- f n + i k, kept
+    in range by a running maximum m of the log gates that starts at zero; o = S^T q / (max(|n . q|, exp(-m)) + 1e-6).
+
+    The log gates are capped softly (cap tanh(z / cap)); heads are divided by their root mean square, multiplied by the
+    weight ``norm`` and by sigmoid(W_g h), then W_o.  S, n and m are fp32 and share one state slot per request."""
+
+    MIN_CHUNKED = 8            # the longest portion of a step from which the chunked kernel is used
+
+    def __init__(self, get, width: int, heads: int, dim: int, vdim: int, gate_cap: float, eps: float, dtype, device):
+        self.heads, self.dim, self.vdim, self.cap, self.eps = heads, dim, vdim, float(gate_cap), float(eps)
+        w = lambda name, *shape: _expect(name, get(name), *shape)
+        pack = lambda *ts: mo.padded_weight(torch.cat(ts), dtype, device)
+        self.w_in = pack(w("q", heads * dim, width), w("k", heads * dim, width), w("v", heads * vdim, width),
+                         w("g", heads * vdim, width))
+        self.w_gates = pack(w("i", heads, width), w("f", heads, width))
+        self.b_gates = torch.cat((w("i.b", heads), w("f.b", heads))).to(device=device, dtype=torch.float32).contiguous()
+        self.norm = w("norm", heads * vdim).to(device=device, dtype=dtype).contiguous()
+        self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
+        self.chunked = torch.device(device).type == "cuda" and mo.mlstm_chunkable(dtype, dim, vdim)
+
+    def cache_spec(self):
+        return StateSpec((self.heads, mo.mlstm_state(self.dim, self.vdim)))
+
+    def __call__(self, h, x, batch, state):
+        n = batch.n_single
+        proj = mo.linear(h, self.w_in)
+        gates = mo.linear(h, self.w_gates, out_dtype=torch.float32)          # the recurrence takes them in 32-bit
+        y = mo.rows_buffer(h.shape[0], self.heads * self.vdim, h.dtype, h.device)
+
+        def run(rows, seqs, cu, spans, chunked):
+            mo.mlstm(proj[rows], gates[rows], self.b_gates, self.norm, state, batch.state_slots[seqs], cu, spans,
+                     batch.positions[rows], self.heads, self.dim, self.vdim, self.cap, self.eps, y[rows], chunked)
+        if n:
+            run(slice(0, n), slice(0, n), None, [(i, i + 1) for i in range(n)] if not h.is_cuda else None, False)
+        if batch.n_rows > n:
+            run(slice(n, batch.n_rows), slice(n, None), batch.cu, batch.spans, self.chunked and batch.max_portion >= self.MIN_CHUNKED)
+        return _project(y, self.w_o, x)
+
+
+class GroupedAttention:
+    """Softmax attention of grouped heads under a sliding window: query head h reads key/value head h // (heads / kv_heads).
+
+    Queries and keys are RMS-normed per head (weights ``q.norm`` / ``k.norm``), rotated in their first ``rot_dims`` dimensions
+    (``rope``), scored with ``scale``.  Optional parts:
+
+    * ``bias_max``: a table ``rel`` (buckets, heads) adds a bias per distance to the scaled scores, exact for near keys and
+      logarithmic up to ``bias_max``
+    * ``difference`` (with ``out_scale``): two maps per head over the same values (queries and keys have twice the rows, laid
+      out head by head); the output is first map - difference * second map, RMS-normed per head, times ``out_scale``
+    * ``gated``: heads are multiplied by sigmoid(W_g h)
+    * ``kv_from``: keys and values of that earlier layer run instead of its own
+
+    The cache holds the normed, rotated keys and the values of a token as one vector, every head padded to 8 elements."""
+
+    def __init__(self, get, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, eps: float,
+                 dtype, device, bias_max: float | None = None, rope=None, rot_dims: int = 0, difference: float | None = None,
+                 out_scale: float = 1.0, gated: bool = False, kv_from: int | None = None):
+        self.gated, self.kv_from, self.rope = gated, kv_from, rope
+        if heads % kv_heads:
+            raise ValueError("the query heads must share the key heads evenly")
+        if rot_dims % 2 or rot_dims > dim:
+            raise ValueError("the rotated dimensions must be even in number and fit the head")
+        maps = 1 if difference is None else 2
+        w = lambda name, *shape: _expect(name, get(name), *shape)
+        parts = [w("q", heads * maps * dim, width)]
+        if kv_from is None:
+            parts += [w("k", kv_heads * maps * dim, width), w("v", kv_heads * vdim, width)]
+        if gated:
+            parts.append(w("g", heads * vdim, width))
+        self.w_in = mo.padded_weight(torch.cat(parts), dtype, device)
+        self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
+        vec = lambda name: w(name, dim).to(device=device, dtype=dtype).contiguous()
+        self.n_q, self.n_k = vec("q.norm"), vec("k.norm") if kv_from is None else None
+        bias = None
+        if bias_max is not None:
+            rel = get("rel")
+            if rel.shape[1] != heads:
+                raise ValueError(f"rel has shape {tuple(rel.shape)}, expected {heads} columns")
+            bias = distance_table(rel, bias_max, window).to(device)
+        self.shape = mo.AttentionShape(heads, kv_heads, maps, dim, vdim, rot_dims, float(scale), int(window), float(eps),
+                                       float(difference or 0.0), float(out_scale), bias)
+        self.tensor_cores = torch.device(device).type == "cuda" and mo.attention_tiles(self.shape, dtype)
+
+    def cache_spec(self):
+        return PagedSpec(self.shape.cache_width) if self.kv_from is None else SharedSpec(self.kv_from)
+
+    def __call__(self, h, x, batch, cache):
+        s, n = self.shape, batch.n_single
+        proj = mo.linear(h, self.w_in)
+        q = mo.attention_prepare(proj, s, self.n_q, self.n_k, self.rope.table if self.rope is not None else None,
+                                 batch.positions, batch.slots, cache)
+        o = mo.rows_buffer(h.shape[0], s.heads * s.vdim, h.dtype, h.device)
+        gate = proj[:, proj.shape[1] - s.heads * s.vdim:] if self.gated else None
+        part = lambda rows: None if gate is None else gate[rows]
+        if n:
+            one = slice(0, n)
+            mo.attention_decode(q[one], s, cache, batch.positions[one], batch.slots[one], batch.tables[one], o[one], part(one))
+        if batch.n_rows > n:
+            rest = slice(n, batch.n_rows)
+            if self.tensor_cores and mo.attention_pages(cache.shape[1]):
+                mo.attention_portions(q[rest], s, cache, batch.positions[rest], batch.cu, batch.max_portion, batch.tables[n:],
+                                      o[rest], part(rest))
+            else:
+                mo.attention_rows(q[rest], s, cache, batch.row_seq[rest], batch.positions[rest], batch.slots[rest],
+                                  batch.tables, o[rest], part(rest))
+        return _project(o, self.w_o, x)
+
+
+def distance_bucket(n: int, rows: int, far: float) -> int:
+    """Row of a distance table of ``rows`` rows for a key ``n`` tokens back: exact in the first half, logarithmic up to ``far`` in
+    the second."""
+    half = rows // 2
+    if n < half:
+        return n
+    if half == 0 or far <= half:
+        return rows - 1
+    return min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half)))
+
+
+def distance_table(rel, far: float, window: int):
+    """(heads, n) fp32: the bias of a key d tokens back in column min(d, n - 1).  Columns end with the window or where the last
+    bucket has been reached."""
+    rows, idx = rel.shape[0], []
+    for d in range(max(1, window)):
+        idx.append(distance_bucket(d, rows, far))
+        if idx[-1] == rows - 1:
+            break
+    return rel.float()[torch.tensor(idx, device=rel.device)].t().contiguous()
 
 
 class RotaryTable:
-    """cos and sin of position * base^(-2 i / dims), rounded once from double precision: (2, positions, dims / 2) fp32.
-    One per (base, dims), shared by the layers that use it; the engine sizes it to its longest context."""
+    """cos and sin of position * frequency, rounded once from double precision: (2, positions, dims / 2) fp32.  One per rotation,
+    shared by the layers that use it; the engine sizes it to its longest context.
 
-    def __init__(self, base: float, dims: int, device):
+    The frequencies are base^(-2 i / dims).  ``scaling`` (factor, original, fast, slow) interpolates them as YaRN does: pairs
+    that turn more than ``fast`` times within ``original`` positions stay, those that turn less than ``slow`` times are slowed
+    down by ``factor``, a linear ramp between; cos and sin are multiplied by 0.1 ln(factor) + 1."""
+
+    def __init__(self, base: float, dims: int, device, scaling: dict | None = None):
         self.base, self.dims, self.device = float(base), int(dims), device
         self.table = None
+        self.freq = self.base ** (-2.0 * torch.arange(self.dims // 2, dtype=torch.float64) / self.dims)
+        self.gain = 1.0
+        if scaling is not None:
+            pair = lambda turns: self.dims * math.log(scaling["original"] / (2 * math.pi * turns)) / (2 * math.log(self.base))
+            lo, hi = max(math.floor(pair(scaling["fast"])), 0), min(math.ceil(pair(scaling["slow"])), self.dims - 1)
+            ramp = ((torch.arange(self.dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+            self.freq = self.freq / scaling["factor"] * ramp + self.freq * (1.0 - ramp)
+            self.gain = 0.1 * math.log(scaling["factor"]) + 1.0
 
     def resize(self, positions: int):
         if self.table is None or self.table.shape[1] != positions:
-            freq = self.base ** (-2.0 * torch.arange(self.dims // 2, dtype=torch.float64) / self.dims)
-            angle = torch.outer(torch.arange(positions, dtype=torch.float64), freq)
-            self.table = torch.stack((angle.cos(), angle.sin())).float().contiguous().to(self.device)
+            angle = torch.outer(torch.arange(positions, dtype=torch.float64), self.freq)
+            self.table = (self.gain * torch.stack((angle.cos(), angle.sin()))).float().contiguous().to(self.device)
+
+
+class GatedFeedForward:
+    """W_down (act(W_gate h) * (W_up h)), ``act`` "silu" or "relu"."""
+
+    def __init__(self, get, width: int, ff: int, act: str, dtype, device):
+        self.ff, self.act = ff, act
+        gu = torch.cat((_expect("gate", get("gate"), ff, width), _expect("up", get("up"), ff, width)))
+        self.w_gu = mo.padded_weight(gu, dtype, device)                           # gate rows first
+        self.w_down = mo.padded_weight(_expect("down", get("down"), width, ff), dtype, device)
+
+    def __call__(self, h):
+        return mo.linear(mo.glu(h, self.w_gu, self.ff, self.act), self.w_down)
 
 
 class TableExperts:

@@ -9,10 +9,11 @@ import os
 
 import torch
 
+from .beledra import Beledra
 from .tedirax import Tedirax
 from .transformer import TransformerLM
 
-MODELS = {"TransformerLM": TransformerLM, "Tedirax": Tedirax}
+MODELS = {"TransformerLM": TransformerLM, "Tedirax": Tedirax, "Beledra": Beledra}
 
 
 def model_class(config: dict):

@@ -18,25 +18,14 @@ This class holds the configuration and the packed weights; caches, batches, sche
 """
 from __future__ import annotations
 
-import json
-import os
-import warnings
 from dataclasses import dataclass, field
 
 import torch
 
 from ..ops import mixer_ops as mo
-from ..utils.safetensors import SafetensorsFile
-from .mixers import LatentAttention, Retention, RotaryTable, TableExperts
-
-
-def _need(d: dict, keys, where: str):
-    missing = [k for k in keys if k not in d]
-    if missing:
-        raise ValueError(f"{where} lacks {', '.join(missing)}")
-    extra = [k for k in d if k not in keys]
-    if extra:
-        warnings.warn(f"{where} has settings this design does not know: {', '.join(extra)}", stacklevel=3)
+from . import layered
+from .layered import LayeredModel, need as _need
+from .mixers import LatentAttention, Retention, TableExperts
 
 
 @dataclass
@@ -109,23 +98,15 @@ class Layer:
         self.index, self.norm, self.mixer, self.experts = index, norm, mixer, experts
 
 
-class Tedirax:
-    GPU_DTYPES = (torch.bfloat16, torch.float32)
-    DEFAULT_CONTEXT = 4096            # positions an engine serves unless it is told otherwise; the design has no limit
-
+class Tedirax(LayeredModel):
     def __init__(self, config: dict, tensors, dtype=torch.bfloat16, device="cuda"):
         """``tensors[name]`` gives a tensor in its stored layout (a dict or a ``SafetensorsFile``)."""
-        if dtype not in self.GPU_DTYPES:
-            raise ValueError("Tedirax runs in bfloat16 or float32")
+        super().__init__(dtype, device)
         self.config = cfg = TediraxConfig.from_dict(config)
-        self.dtype, self.device = dtype, torch.device(device)
-        take = lambda name, *shape: self._shaped(tensors, name, shape)
-        self.embed = take("embed", cfg.vocab, cfg.width).to(device=device, dtype=dtype).contiguous()
-        self.rotary: dict[tuple, RotaryTable] = {}
-        self.layers = []
+        self.embed = self.vector(tensors, "embed", cfg.vocab, cfg.width)
         for i, spec in enumerate(cfg.layers):
             pre = f"l{i}."
-            norm = take(pre + "norm1", cfg.width).to(device=device, dtype=dtype).contiguous()
+            norm = self.vector(tensors, pre + "norm1", cfg.width)
             mixer = self._mixer(spec, lambda name: tensors[pre + "mix." + name])
             experts = None
             if spec.mlp is not None:
@@ -134,90 +115,40 @@ class Tedirax:
                                        r["experts"], r["top"], cfg.vocab, dtype, device)
             self.layers.append(Layer(i, norm, mixer, experts))
         self.runs = [self.layers[i] for i in cfg.runs()]
-        self.final_norm = take("final.norm", cfg.width).to(device=device, dtype=dtype).contiguous()
-        self.head = mo.padded_weight(take("head", cfg.vocab, cfg.width), dtype, device)
+        self.final_norm = self.vector(tensors, "final.norm", cfg.width)
+        self.head = mo.padded_weight(self.shaped(tensors, "head", cfg.vocab, cfg.width), dtype, device)
         self.vocab_size = cfg.vocab
-        self._engine = None
-
-    @staticmethod
-    def _shaped(tensors, name, shape):
-        t = tensors[name]
-        if tuple(t.shape) != shape:
-            raise ValueError(f"{name} has shape {tuple(t.shape)}, expected {shape}")
-        return t
 
     def _mixer(self, spec: LayerSpec, get):
         m, cfg = spec.mixer, self.config
         if spec.type == "latent_attention":
             return LatentAttention(get, cfg.width, m["heads"], m["dim"], m["vdim"], m["q_rank"], m["kv_rank"], m["scale"],
                                    m["mask"]["size"], cfg.eps, self.dtype, self.device)
-        dims = m["rot"]["dims"]
-        rope = None
-        if dims:
-            rope = self.rotary.setdefault((m["rot"]["base"], dims), RotaryTable(m["rot"]["base"], dims, self.device))
-        return Retention(get, cfg.width, m["heads"], m["dim"], m["vdim"], m["decay"], dims, cfg.eps, rope, self.dtype, self.device)
-
-    # ---------------------------------------------------------------------------------- loading
-    @classmethod
-    def from_folder(cls, folder: str, dtype=torch.bfloat16, device="cuda") -> "Tedirax":
-        """``folder``: config.json and model.safetensors."""
-        with open(os.path.join(folder, "config.json")) as f:
-            config = json.load(f)
-        return cls(config, SafetensorsFile(os.path.join(folder, "model.safetensors")), dtype, device)
+        rot = m["rot"]
+        return Retention(get, cfg.width, m["heads"], m["dim"], m["vdim"], m["decay"], rot["dims"], cfg.eps,
+                         self.rotary_table(rot["base"], rot["dims"]), self.dtype, self.device)
 
     @classmethod
     def random(cls, config: dict, seed: int = 0, dtype=torch.bfloat16, device="cuda") -> "Tedirax":
         """Random weights of the configuration's shapes (tests, benchmarks)."""
         return cls(config, RandomTensors(config, seed, device), dtype, device)
 
-    def eval(self):
-        return self
-
     # ------------------------------------------------------------------------------ serving hook
     def serving_backend(self):
-        from ..serving.backends import LayeredBackend
-        return LayeredBackend(self)
-
-    @torch.no_grad()
-    def generate(self, prompt_ids, max_new_tokens: int, temperature: float = 1.0, top_k: int | None = None,
-                 eos_token_id: int | None = None):
-        """Up to ``max_new_tokens`` ids after the prompt, shape (1, n), through the serving engine; the stop token is not
-        returned (as in ``TransformerLM.generate``)."""
-        from ..serving import ServingEngine
-        ids = prompt_ids.reshape(-1).tolist()
-        total = len(ids) + max_new_tokens
-        if self._engine is None or self._engine.max_context < total:
-            ctx = -(-total // 256) * 256
-            self._engine = ServingEngine(self, num_pages=-(-ctx // 64), page_size=64, max_batch=1, max_context=ctx,
-                                         use_cuda_graphs=False)
-        out = self._engine.generate([ids], max_new_tokens, eos_token_id, temperature, top_k)[0]
-        if eos_token_id is not None and out and out[-1] == eos_token_id:
-            out = out[:-1]
-        return torch.tensor([out], dtype=torch.long, device=self.device).reshape(1, -1)
+        from ..serving.backends import ParallelLayers
+        return ParallelLayers(self)
 
 
-class RandomTensors:
-    """Weights made on demand: normal with variance 1 / fan-in, norms around one, experts drawn without repetition."""
+def RandomTensors(config: dict, seed: int = 0, device="cpu"):
+    """Random weights on demand (``layered.RandomTensors``); the experts of a token are drawn without repetition."""
+    cfg = TediraxConfig.from_dict(config)
 
-    def __init__(self, config: dict, seed: int = 0, device="cpu"):
-        self.cfg, self.seed, self.device = TediraxConfig.from_dict(config), seed, torch.device(device)
-        self.shapes = tensor_shapes(self.cfg)
-        self._order = {name: i for i, name in enumerate(self.shapes)}
-
-    def keys(self):
-        return self.shapes.keys()
-
-    def __getitem__(self, name: str):
-        shape = self.shapes[name]
-        g = torch.Generator(self.device).manual_seed(self.seed * 1000003 + self._order[name])
-        kw = {"generator": g, "device": self.device}
+    def table(name, shape, kw):
         if name.endswith(".table"):
-            experts = self.cfg.layers[int(name[1:].split(".")[0])].mlp["router"]["experts"]
+            experts = cfg.layers[int(name[1:].split(".")[0])].mlp["router"]["experts"]
             return torch.rand((shape[0], experts), **kw).argsort(1)[:, :shape[1]].to(torch.int32)
-        if len(shape) == 1:
-            return (1.0 + 0.1 * torch.randn(shape, **kw)).to(torch.bfloat16)
-        std = 1.0 if name == "embed" else shape[1] ** -0.5
-        return (std * torch.randn(shape, **kw)).to(torch.bfloat16)
+        return None
+    return layered.RandomTensors(tensor_shapes(cfg), seed, device, table)
 
 
 def tensor_shapes(cfg: TediraxConfig) -> dict[str, tuple[int, ...]]:

@@ -7,6 +7,7 @@ Matrices whose rows are read by TMA have a row pitch that is a multiple of 8 ele
 from __future__ import annotations
 
 import ctypes
+from dataclasses import dataclass
 
 import torch
 
@@ -26,7 +27,8 @@ def _lib():
             "b200_residual_norm": [P, P, I, P, P, P, P, I, I, F, L, P, P, L, F, P, P, I, I, L, I, I, I, I, P, P],
             "b200_moe_plan": [P, P, I, I, I, P, P, P, P, L, P, I, P, P],
             "b200_moe_plan_layers": [],
-            "b200_silu_mul_any": [P, P, L, I, L, L, I, P],
+            "b200_add_normed": [P, P, I, P, P, L, P, P, L, F, I, I, I, P, P],
+            "b200_glu_any": [P, P, L, I, L, L, I, I, P],
             "b200_gate_sigmoid": [P, P, L, I, L, L, I, P],
             "b200_gemm_f32": [P, P, P, I, I, I, L, L, L, I, P, I, I, I, I, P],
             "b200_gemm_bf16_grouped": [P, P, P, P, I, I, I, L, L, L, L, P, I, I, I, I, I, I, I, P, P],
@@ -37,6 +39,11 @@ def _lib():
             "b200_latent_decode_tc": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
             "b200_flash_window_fwd": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, L, L, L, L, P, P],
             "b200_retention_chunk": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
+            "b200_grouped_prep": [P, L, P, P, P, P, P, P, P, I, I, I, L, P, I, P, P],
+            "b200_grouped_rows": [P, P, P, L, P, L, P, I, P, P, P, P, I, I, I, I, I, P, I, P, P],
+            "b200_grouped_decode": [P, P, P, L, P, L, P, I, P, P, P, P, P, I, I, I, I, I, P, P, P],
+            "b200_grouped_prefill": [P, P, P, L, P, L, P, I, P, P, P, I, I, I, I, I, I, P, P, P],
+            "b200_mlstm": [P, L, P, L, P, P, P, L, P, P, P, P, I, I, I, I, I, I, I, F, F, I, I, P, P],
             "b200_retention_recurrent": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
         }.items():
             fn = getattr(lib, name)
@@ -106,8 +113,26 @@ def gemm_rows(a, w, tile_group, n: int, swiglu: bool):
     if not swiglu:
         return out
     h = rows_buffer(p, n, a.dtype, a.device)
-    _check(lib.b200_silu_mul_any(_ptr(out), _ptr(h), p, n, out.stride(0), h.stride(0), 1, _stream()), "silu_mul_any")
+    _check(lib.b200_glu_any(_ptr(out), _ptr(h), p, n, out.stride(0), h.stride(0), 0, 1, _stream()), "glu_any")
     return h
+
+
+def glu(a, w, n: int, act: str):
+    """act(a @ gate^T) * (a @ up^T) for w (2 n, K), gate rows first; act "silu" or "relu"."""
+    _req(act in ("silu", "relu") and w.shape[0] == 2 * n and w.shape[1] == a.shape[1], "bad gated product")
+    out = rows_buffer(a.shape[0], n, a.dtype, a.device)
+    if not a.is_cuda:
+        return mixer_torch.glu(a, w, n, act, out)
+    lib = _lib()
+    m, k = a.shape
+    if a.dtype == torch.bfloat16:
+        _check(lib.b200_gemm_bf16_grouped(_ptr(a), _ptr(w), _ptr(out), None, m, n, k, a.stride(0), w.stride(0), out.stride(0), 0, None,
+                                          0, 2 * n, 1, 0, 0, 2 if act == "relu" else 1, native.EPI_B_STABLE,
+                                          _ptr(native.status_word(a.device)), _stream()), "gemm_glu")
+        return out
+    gu = linear(a, w)
+    _check(lib.b200_glu_any(_ptr(gu), _ptr(out), m, n, gu.stride(0), out.stride(0), int(act == "relu"), 1, _stream()), "glu_any")
+    return out
 
 
 def gemm_heads(a, w, heads: int, k: int, n: int, out=None, gate=None):
@@ -186,6 +211,25 @@ def residual_norm(x, w=None, eps: float = 0.0, tokens=None, embed=None, row_inde
         0 if gpos is None else gpos.shape[1], g_rows, 0 if xg is None else xg.stride(0), rows, x.shape[0], d, _f32(act),
         _ptr(native.status_word(x.device)), _stream()), "residual_norm")
     return h, xg
+
+
+def add_normed(x, y=None, w=None, eps: float = 0.0, tokens=None, embed=None):
+    """Norm behind a sublayer: x (R, d) fp32 += y / rms(y) * w in place; with ``tokens`` / ``embed`` instead x = embed[tokens].
+    Returns x in the activation type, for the next sublayer to read."""
+    act = embed if tokens is not None else y
+    h = rows_buffer(x.shape[0], x.shape[1], act.dtype, x.device)
+    if not x.is_cuda:
+        return mixer_torch.add_normed(x, y, w, eps, tokens, embed, h)
+    d = x.shape[1]
+    _req(x.dtype == torch.float32 and x.is_contiguous(), "the residual stream is contiguous fp32")
+    if tokens is not None:
+        _req(tokens.dtype == torch.int64 and tokens.numel() == x.shape[0] and embed.is_contiguous() and embed.shape[1] == d, "bad embedding")
+    else:
+        _req(y.shape == x.shape and y.stride(1) == 1 and w.dtype == y.dtype and w.numel() == d and w.is_contiguous(), "bad sublayer output")
+    _check(_lib().b200_add_normed(_ptr(tokens), _ptr(embed), 0 if embed is None else embed.shape[0], _ptr(x), _ptr(y),
+                                  0 if y is None else y.stride(0), _ptr(w), _ptr(h), h.stride(0), float(eps), x.shape[0], d, _f32(act),
+                                  _ptr(native.status_word(x.device)), _stream()), "add_normed")
+    return h
 
 
 # ------------------------------------------------------------------------------ mixture of experts
@@ -389,3 +433,180 @@ def retention(proj, state, state_slots, cu, spans, positions, cos_sin, decay, he
         _ptr(cos_sin), _ptr(decay), seqs, proj.shape[0], heads, dim, vdim, rot, 0 if rot == 0 else cos_sin.shape[1],
         state.shape[0], float(eps), _f32(proj), _ptr(native.status_word(proj.device)), _stream()), "retention")
     return y
+
+
+# --------------------------------------------------------------------------------- matrix memory (mLSTM)
+def mlstm_state(dim: int, vdim: int) -> int:
+    """Floats of one head's state: S (dim, vdim) | n (dim) | m, rounded up to 16 bytes."""
+    return -(-(dim * vdim + dim + 1) // 4) * 4
+
+
+def mlstm_chunkable(dtype, dim: int, vdim: int) -> bool:
+    return dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and vdim <= 128
+
+
+def mlstm(proj, gates, gate_bias, weight, state, state_slots, cu, spans, positions, heads: int, dim: int, vdim: int, cap: float,
+          eps: float, y, chunked: bool = False):
+    """Matrix memory over the rows of ``proj`` (q | k | v | output gate) with the gates' pre-activations ``gates`` (input | forget,
+    fp32, without bias).  ``cu`` (sequences + 1, int32) delimits the sequences, None = one row each; ``spans`` says the same on
+    the host.  The states are read and left in their slots; y (R, heads * vdim) receives the normed, weighted, gated heads.
+    ``chunked``: the tensor-core kernel for portions of prompts (``mlstm_chunkable`` sizes)."""
+    if not proj.is_cuda:
+        return mixer_torch.mlstm(proj, gates, gate_bias, weight, state, state_slots, spans, positions, heads, dim, vdim, cap, eps, y)
+    seqs = state_slots.numel()
+    _req(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, mlstm_state(dim, vdim)), "bad state")
+    _req(state_slots.dtype == torch.int32 and positions.dtype == torch.int32 and gate_bias.dtype == torch.float32
+         and gate_bias.numel() == 2 * heads and gates.dtype == torch.float32 and gates.shape == (proj.shape[0], 2 * heads), "bad inputs")
+    _req(proj.shape[1] == 2 * heads * (dim + vdim) and y.shape == (proj.shape[0], heads * vdim) and y.dtype == proj.dtype
+         and weight.dtype == proj.dtype and weight.numel() == heads * vdim, "bad shapes")
+    _req(cu is None or (cu.dtype == torch.int32 and cu.numel() == seqs + 1), "bad row offsets")
+    _req(not chunked or (mlstm_chunkable(proj.dtype, dim, vdim) and cu is not None), "sizes the chunked kernel does not take")
+    _check(_lib().b200_mlstm(
+        _ptr(proj), proj.stride(0), _ptr(gates), gates.stride(0), _ptr(gate_bias), _ptr(weight), _ptr(y), y.stride(0), _ptr(state),
+        _ptr(state_slots), _ptr(cu), _ptr(positions), seqs, proj.shape[0], heads, dim, vdim, state.shape[2], state.shape[0],
+        float(cap), float(eps), _f32(proj), int(chunked), _ptr(native.status_word(proj.device)), _stream()),
+        "mlstm_chunk" if chunked else "mlstm")
+    return y
+
+
+# ------------------------------------------------------------------------------- grouped attention
+@dataclass
+class AttentionShape:
+    """Sizes and constants of one grouped attention (``models.mixers.GroupedAttention``); ``bias`` (heads, n) fp32 holds the bias
+    per distance, distances from n - 1 on read its last column."""
+    heads: int
+    kv_heads: int
+    maps: int
+    dim: int
+    vdim: int
+    rot: int
+    scale: float
+    window: int
+    eps: float
+    difference: float = 0.0
+    out_scale: float = 1.0
+    bias: torch.Tensor | None = None
+
+    @property
+    def q_pitch(self) -> int:
+        return pitch(self.dim) if self.dim > 128 else (64 if self.dim <= 64 else 128)
+
+    @property
+    def k_pitch(self) -> int:
+        return pitch(self.dim)
+
+    @property
+    def v_pitch(self) -> int:
+        return pitch(self.vdim)
+
+    @property
+    def cache_width(self) -> int:
+        """Elements a token takes in the cache: the keys of all heads and maps, then the values."""
+        return self.kv_heads * (self.maps * self.k_pitch + self.v_pitch)
+
+
+class _NativeShape(ctypes.Structure):
+    """csrc/grouped_attention.cuh: GroupedShape"""
+    _fields_ = [(n, ctypes.c_int) for n in ("heads", "kv_heads", "maps", "dim", "vdim", "qp", "kp", "vp", "window")] + \
+               [(n, ctypes.c_float) for n in ("scale", "eps", "difference", "out_scale")]
+
+
+def _native_shape(s: AttentionShape):
+    got = s.__dict__.get("_native")
+    if got is None:
+        got = s.__dict__["_native"] = _NativeShape(s.heads, s.kv_heads, s.maps, s.dim, s.vdim, s.q_pitch, s.k_pitch, s.v_pitch,
+                                                   s.window, s.scale, s.eps, s.difference, s.out_scale)
+    return ctypes.byref(got)
+
+
+BIAS_MAX = 6000                  # entries of a distance table that fit the portions kernel's shared memory
+
+
+def attention_tiles(s: AttentionShape, dtype) -> bool:
+    """Whether portions of prompts run on the tensor-core kernel."""
+    if dtype != torch.bfloat16 or s.dim > 128 or s.vdim > 128:
+        return False
+    return s.scale > 0 if s.bias is None else s.bias.shape[1] <= BIAS_MAX
+
+
+def attention_pages(page_size: int) -> bool:
+    return page_size >= 8 and 128 % page_size == 0
+
+
+def attention_prepare(proj, s: AttentionShape, wq, wk, cos_sin, positions, slots, cache):
+    """Queries of ``proj`` (q | k | v | ..., or q | ... without ``wk``) normed and rotated, (R, heads * maps * q_pitch) with zeros
+    behind every head; keys, likewise, and values go to their cache slots (negative slot: not written)."""
+    q = torch.empty((proj.shape[0], s.heads * s.maps * s.q_pitch), dtype=proj.dtype, device=proj.device)
+    if not proj.is_cuda:
+        return mixer_torch.attention_prepare(proj, s, wq, wk, cos_sin, positions, slots, cache, q)
+    _req(cache.is_contiguous() and cache.dtype == proj.dtype and cache.shape[-1] == s.cache_width and slots.dtype == torch.int64
+         and slots.numel() == proj.shape[0] and positions.dtype == torch.int32 and wq.dtype == proj.dtype, "bad cache or rows")
+    _req(s.rot == 0 or (cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[2] == s.rot // 2), "bad rotary table")
+    _check(_lib().b200_grouped_prep(_ptr(proj), proj.stride(0), _ptr(q), _ptr(cache), _ptr(wq), _ptr(wk), _ptr(cos_sin),
+                                    _ptr(positions), _ptr(slots), proj.shape[0], s.rot, cos_sin.shape[1] if s.rot else 0,
+                                    cache.shape[0] * cache.shape[1], _native_shape(s), _f32(proj),
+                                    _ptr(native.status_word(proj.device)), _stream()), "grouped_prep")
+    return q
+
+
+def _attention_args(q, s, cache, positions, tables, out, gate):
+    _req(q.is_contiguous() and q.shape[1] == s.heads * s.maps * s.q_pitch and cache.is_contiguous() and cache.dtype == q.dtype
+         and cache.shape[-1] == s.cache_width, "bad queries or cache")
+    _req(tables.dtype == torch.int32 and tables.is_contiguous() and positions.dtype == torch.int32, "bad tables")
+    _req(out.shape == (q.shape[0], s.heads * s.vdim) and out.dtype == q.dtype and out.stride(1) == 1, "bad output")
+    _req(gate is None or (gate.shape == out.shape and gate.dtype == q.dtype and gate.stride(1) == 1), "bad gate")
+    return (_ptr(q), _ptr(cache), _ptr(out), out.stride(0), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(s.bias),
+            0 if s.bias is None else s.bias.shape[1])
+
+
+def attention_rows(q, s: AttentionShape, cache, row_seq, positions, slots, tables, out, gate=None):
+    """The general form: every row of q has its own position and line of ``tables`` (``row_seq`` None: line i for row i)."""
+    if not q.is_cuda:
+        return mixer_torch.attention_rows(q, s, cache, row_seq, positions, slots, tables, out, gate)
+    args = _attention_args(q, s, cache, positions, tables, out, gate)
+    _check(_lib().b200_grouped_rows(*args, _ptr(row_seq), _ptr(positions), _ptr(slots), _ptr(tables), tables.shape[0], q.shape[0],
+                                    tables.shape[1], cache.shape[1], cache.shape[0], _native_shape(s), _f32(q),
+                                    _ptr(native.status_word(q.device)), _stream()), "grouped_rows")
+    return out
+
+
+def attention_splits(s: AttentionShape, rows: int, keys: int, sms: int = 148) -> int:
+    """Splits of the window per row of a decode step: CTAs of four warps that walk 16 tokens at a time, two CTAs to an SM; a start-up
+    is worth about three steps, a merge about two."""
+    groups = rows * s.kv_heads * -(-(s.heads // s.kv_heads) // (16 // s.maps))
+    best, best_cost = 1, None
+    for n in range(1, max(1, min(32, keys // 128)) + 1):
+        cost = -(-groups * n // (2 * sms)) * (-(-keys // (n * 64)) + 3) + (2 if n > 1 else 0)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = n, cost
+    return best
+
+
+def attention_decode(q, s: AttentionShape, cache, positions, slots, tables, out, gate=None, splits: int = 0):
+    """``attention_rows`` for one query row per request: line i of ``tables`` belongs to row i."""
+    fits = q.is_cuda and q.dtype == torch.bfloat16 and s.maps * s.k_pitch <= 256 and s.v_pitch <= 128
+    if not fits:
+        return attention_rows(q, s, cache, None, positions, slots, tables, out, gate)
+    rows, keys = q.shape[0], min(s.window, tables.shape[1] * cache.shape[1])
+    _req(tables.shape[0] >= rows, "bad tables")
+    args = _attention_args(q, s, cache, positions, tables, out, gate)
+    splits = splits or attention_splits(s, rows, keys)
+    n = rows * s.heads * s.maps * splits
+    part = torch.empty(n * (s.vdim + 2) if splits > 1 else 0, dtype=torch.float32, device=q.device)
+    _check(_lib().b200_grouped_decode(*args, _ptr(part), _ptr(part[n * s.vdim:]), _ptr(positions), _ptr(slots), _ptr(tables), rows,
+                                      tables.shape[1], cache.shape[1], cache.shape[0], splits, _native_shape(s),
+                                      _ptr(native.status_word(q.device)), _stream()),
+           "grouped_decode" if splits > 1 else "grouped_decode_one")
+    return out
+
+
+def attention_portions(q, s: AttentionShape, cache, positions, cu, max_q: int, tables, out, gate=None):
+    """Portions of prompts on the tensor cores: rows cu[b] .. cu[b + 1] - 1 of q belong to portion b, line b of ``tables`` to it; its
+    keys and values are in the cache already."""
+    _req(attention_tiles(s, q.dtype) and attention_pages(cache.shape[1]) and q.is_cuda, "sizes the portions kernel does not take")
+    _req(cu.dtype == torch.int32 and tables.shape[0] >= cu.numel() - 1, "bad row offsets")
+    args = _attention_args(q, s, cache, positions, tables, out, gate)
+    _check(_lib().b200_grouped_prefill(*args, _ptr(cu), _ptr(positions), _ptr(tables), cu.numel() - 1, max_q, q.shape[0],
+                                       tables.shape[1], cache.shape[1], cache.shape[0], _native_shape(s),
+                                       _ptr(native.status_word(q.device)), _stream()), "grouped_prefill")
+    return out

@@ -31,6 +31,20 @@ def residual_norm(x, tokens, embed, row_index, pending, w, eps, scatter):
     return h, xg
 
 
+def add_normed(x, y, w, eps, tokens, embed, h):
+    if tokens is not None:
+        x.copy_(embed[tokens.long()].float())
+    else:
+        f = y.float()
+        x.add_(f * torch.rsqrt(f.pow(2).mean(-1, keepdim=True) + eps) * w.float())
+    return h.copy_(x)
+
+
+def glu(a, w, n, act, out):
+    g, u = (a.float() @ w.float().t()).split(n, 1)
+    return out.copy_((torch.relu(g) if act == "relu" else torch.nn.functional.silu(g)) * u)
+
+
 def moe_plan(tokens, slots, tables, experts, tiles):
     pos, groups = [], []
     for table, n in zip(tables, experts):
@@ -131,3 +145,82 @@ def retention(proj, state, state_slots, spans, positions, cos_sin, decay, heads,
             g = qkv[r, 2 * hd + he:2 * hd + 2 * he].view(heads, vdim)
             y[r] = (o * torch.nn.functional.silu(g)).reshape(-1).to(y.dtype)
     return y
+
+
+def mlstm(proj, gates, gate_bias, weight, state, state_slots, spans, positions, heads, dim, vdim, cap, eps, y):
+    """``spans``: (first row, one past the last row) of every sequence."""
+    rows, hd, he = proj.float(), heads * dim, heads * vdim
+    logs = cap * torch.tanh((gates + gate_bias) / cap)
+    for s, (a, b) in enumerate(spans):
+        slot = int(state_slots[s])
+        if slot < 0:
+            y[a:b] = 0
+            continue
+        flat = state[slot]
+        S, N, M = flat[:, :dim * vdim].view(heads, dim, vdim), flat[:, dim * vdim:dim * vdim + dim], flat[:, dim * vdim + dim]
+        for r in range(a, b):
+            if int(positions[r]) == 0:
+                flat.zero_()
+            q, k = rows[r, :hd].view(heads, dim) * dim ** -0.5, rows[r, hd:2 * hd].view(heads, dim)
+            v, g = rows[r, 2 * hd:2 * hd + he].view(heads, vdim), rows[r, 2 * hd + he:2 * hd + 2 * he]
+            i, f = logs[r, :heads], torch.nn.functional.logsigmoid(logs[r, heads:])
+            m = torch.maximum(f + M, i)
+            keep, take = torch.exp(f + M - m), torch.exp(i - m)
+            M.copy_(m)
+            kt = take[:, None] * k
+            S.mul_(keep[:, None, None]).add_(kt[:, :, None] * v[:, None, :])
+            N.mul_(keep[:, None]).add_(kt)
+            o = torch.einsum("hde,hd->he", S, q) / (torch.maximum((N * q).sum(-1).abs(), torch.exp(-m)) + 1e-6)[:, None]
+            o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+            y[r] = (o.reshape(-1) * weight.float() * torch.sigmoid(g)).to(y.dtype)
+    return y
+
+
+def attention_prepare(proj, s, wq, wk, cos_sin, positions, slots, cache, q):
+    half = s.rot // 2
+
+    def vectors(cols, n, w):
+        t = cols.float().reshape(-1, n, s.dim)
+        t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + s.eps) * w.float()
+        if half:
+            c, sn = cos_sin[0, positions.long()][:, None], cos_sin[1, positions.long()][:, None]
+            u, v = t[..., :half], t[..., half:s.rot]
+            t = torch.cat((u * c - v * sn, v * c + u * sn, t[..., s.rot:]), -1)
+        return t
+    nq, nk = s.heads * s.maps, s.kv_heads * s.maps
+    q.zero_().view(-1, nq, s.q_pitch)[..., :s.dim] = vectors(proj[:, :nq * s.dim], nq, wq).to(q.dtype)
+    if wk is not None:
+        live, at = slots >= 0, (nq + nk) * s.dim
+        row = torch.zeros((proj.shape[0], s.cache_width), dtype=cache.dtype)
+        row[:, :nk * s.k_pitch].view(-1, nk, s.k_pitch)[..., :s.dim] = vectors(proj[:, nq * s.dim:at], nk, wk).to(cache.dtype)
+        row[:, nk * s.k_pitch:].view(-1, s.kv_heads, s.v_pitch)[..., :s.vdim] = proj[:, at:at + s.kv_heads * s.vdim].view(-1, s.kv_heads, s.vdim)
+        cache.view(-1, s.cache_width)[slots[live]] = row[live]
+    return q
+
+
+def attention_rows(q, s, cache, row_seq, positions, slots, tables, out, gate):
+    page, flat = cache.shape[1], cache.view(-1, s.cache_width)
+    keys = s.kv_heads * s.maps * s.k_pitch
+    rep = s.heads // s.kv_heads
+    for r in range(q.shape[0]):
+        if slots[r] < 0:
+            out[r] = 0
+            continue
+        p = int(positions[r])
+        j = torch.arange(max(0, p - s.window + 1), p + 1)
+        line = tables[int(row_seq[r]) if row_seq is not None else r].long()
+        c = flat[line[j // page] * page + j % page].float()
+        k = c[:, :keys].view(-1, s.kv_heads, s.maps, s.k_pitch)[..., :s.dim].repeat_interleave(rep, 1)
+        v = c[:, keys:].view(-1, s.kv_heads, s.v_pitch)[..., :s.vdim].repeat_interleave(rep, 1)
+        score = torch.einsum("hmd,jhmd->hmj", q[r].float().view(s.heads, s.maps, s.q_pitch)[..., :s.dim], k) * s.scale
+        if s.bias is not None:
+            score = score + s.bias[:, (p - j).clamp(max=s.bias.shape[1] - 1)][:, None]
+        o = torch.einsum("hmj,jhe->hme", torch.softmax(score, -1), v)
+        if s.maps == 2:
+            o = o[:, 0] - s.difference * o[:, 1]
+            o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + s.eps) * s.out_scale
+        o = o.reshape(-1)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[r].float())
+        out[r] = o.to(out.dtype)
+    return out

@@ -173,7 +173,7 @@ def check_status(device=None):
 
 # Kernels launched per launcher call (a launcher may issue several).  Used to count this package's
 # own launches inside a timed region.
-_KERNELS_PER_CALL = {"rmsnorm_bwd": 2, "xent": 3, "flash_bwd": 3, "latent_decode": 2}
+_KERNELS_PER_CALL = {"rmsnorm_bwd": 2, "xent": 3, "flash_bwd": 3, "latent_decode": 2, "grouped_decode": 2}
 _LAUNCHES = 0
 
 

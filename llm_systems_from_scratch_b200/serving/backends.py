@@ -98,14 +98,11 @@ class TransformerBackend:
 
 
 class LayeredBackend:
-    """Models made of listed layers (``models/tedirax.py``): parallel sublayers on one norm, mixers of several kinds, token-
-    table experts, fp32 residual stream.
-
-    A layer run is: one pass over the residual stream (add the previous run's expert outputs, norm, copy rows to where
-    the experts read them), the mixer (adds to the residual stream in its last product), the experts."""
+    """What models made of listed layers (``models/layered.py``) have in common: one cache entry per layer run, an fp32
+    residual stream, fp32 logits.  A subclass knows the order of a layer's sublayers and norms."""
 
     splits_prompts = True
-    page_size = 64                    # tokens: the decode kernel copies whole pages as TMA boxes
+    page_size = 64                    # tokens: the attention kernels copy whole pages as TMA boxes
 
     def __init__(self, model):
         self.model = model
@@ -113,7 +110,6 @@ class LayeredBackend:
         self.context_limit = None
         self.default_context = model.DEFAULT_CONTEXT
         self.specs = [layer.mixer.cache_spec() for layer in model.runs]
-        self.expert_layers = [layer for layer in model.layers if layer.experts is not None]
 
     def set_context(self, positions: int):
         for table in self.model.rotary.values():
@@ -129,10 +125,31 @@ class LayeredBackend:
     def choose_splits(self, rows: int, max_context: int) -> int:
         return 0
 
+    def stream(self, batch):
+        """The residual stream of a step, not yet written."""
+        return torch.empty((batch.n_rows, self.model.config.width), dtype=torch.float32, device=self.device)
+
+    def head(self, h):
+        """(rows, vocabulary) fp32 of normed rows."""
+        out = torch.empty((h.shape[0], mo.pitch(self.vocab)), dtype=torch.float32, device=self.device)
+        mo.linear(h, self.model.head, out=out[:, :self.vocab])
+        return out
+
+
+class ParallelLayers(LayeredBackend):
+    """Parallel sublayers on one norm, token-table experts (``models/tedirax.py``).
+
+    A layer run is: one pass over the residual stream (add the previous run's expert outputs, norm, copy rows to where
+    the experts read them), the mixer (adds to the residual stream in its last product), the experts."""
+
+    def __init__(self, model):
+        super().__init__(model)
+        self.expert_layers = [layer for layer in model.layers if layer.experts is not None]
+
     def forward(self, batch, trace=None):
         """``trace``: a list that receives the residual stream after every layer run (a copy; for tests)."""
         m = self.model
-        x = torch.empty((batch.n_rows, m.config.width), dtype=torch.float32, device=self.device)
+        x = self.stream(batch)
         plan = {}
         if self.expert_layers:
             pos, groups = mo.moe_plan(batch.tokens, batch.slots, [la.experts.table for la in self.expert_layers],
@@ -168,9 +185,30 @@ class LayeredBackend:
             h, _ = mo.residual_norm(x, m.final_norm, m.config.eps, pending=pending)
         else:
             h, _ = mo.residual_norm(x, m.final_norm, m.config.eps, row_index=rows, pending=pending)
-        out = torch.empty((h.shape[0], mo.pitch(self.vocab)), dtype=torch.float32, device=self.device)
-        mo.linear(h, m.head, out=out[:, :self.vocab])
-        return out
+        return self.head(h)
+
+
+class PostNormLayers(LayeredBackend):
+    """Sublayers one after the other, each reading the residual stream itself, its output normed before it is added
+    (``models/beledra.py``).  The pass that adds a sublayer's output also writes the next one's input."""
+
+    def forward(self, batch, trace=None):
+        """``trace``: a list that receives the residual stream after every layer run (a copy; for tests)."""
+        m, eps = self.model, self.model.config.eps
+        x = self.stream(batch)
+        h = mo.add_normed(x, tokens=batch.tokens, embed=m.embed)
+        for run, layer in enumerate(m.runs):
+            h = mo.add_normed(x, layer.mixer(h, None, batch, self.cache.entries[run]), layer.norm1, eps)
+            if layer.mlp is not None:
+                h = mo.add_normed(x, layer.mlp(h), layer.norm2, eps)
+            if trace is not None:
+                trace.append(x.clone())
+        return x
+
+    def logits(self, x, rows=None):
+        """(rows, vocabulary) fp32."""
+        h, _ = mo.residual_norm(x, self.model.final_norm, self.model.config.eps, row_index=rows)
+        return self.head(h)
 
 
 def wanted_index(rows: np.ndarray, device) -> torch.Tensor:

@@ -7,8 +7,9 @@ Memory: one K and one V tensor of shape (layers, num_pages, page_size, d_model) 
 of thousands of pages next to the 2.8 GB of weights.
 
 ``LayerCache`` is the same for models whose layers differ: every layer run says what it keeps per token
-(``PagedSpec``: one vector in a paged pool) or per request (``StateSpec``: a recurrent state in a slot).  All paged
-layers share the page ids of a request, all recurrent layers its slot.
+(``PagedSpec``: one vector in a paged pool) or per request (``StateSpec``: a recurrent state in a slot), or that it
+reads what an earlier run keeps (``SharedSpec``).  All paged layers share the page ids of a request, all recurrent
+layers its slot.
 """
 from __future__ import annotations
 
@@ -27,6 +28,12 @@ class PagedSpec:
 class StateSpec:
     """A layer run that carries one fp32 state of this shape per request."""
     shape: tuple
+
+
+@dataclass(frozen=True)
+class SharedSpec:
+    """A layer run that keeps nothing of its own and reads the entry of an earlier run."""
+    run: int
 
 
 class PageAllocator:
@@ -109,6 +116,8 @@ class LayerCache:
                 self.entries.append(torch.zeros((num_pages, page_size, s.width), dtype=dtype, device=device))
             elif isinstance(s, StateSpec):
                 self.entries.append(torch.zeros((num_slots, *s.shape), dtype=torch.float32, device=device))
+            elif isinstance(s, SharedSpec):
+                self.entries.append(self.entries[s.run])
             else:
                 self.entries.append(None)
         self.allocator = PageAllocator(num_pages)
