@@ -30,10 +30,10 @@ version of the same measurement (``--serving-requests`` requests, 0 switches it 
 engine; its arm replays the head of the same trace through its ``TransformerLM`` with a per-request greedy
 loop that re-runs the whole context for every token (what its ``generate`` does) for a bounded time.
 
-    python bench.py --workload layers [--layers-sizes 0.35b,1.3b,7b-8layers]
+    python bench.py --workload layers [--layers-model Tedirax|Beledra] [--layers-sizes 0.35b,1.3b,7b-8layers]
 
-times the layered decoder (Tedirax) beside the TransformerLM at equal size on one GPU: whole prompt and decode steps and
-every kernel against its roofline, one line per size (``ops/bench_layers.py``).
+times a layered decoder beside the TransformerLM (Beledra also beside Tedirax) at equal size on one GPU: whole prompt and
+decode steps and every kernel against its roofline, one line per size (``ops/bench_layers.py``, ``ops/bench_beledra.py``).
 """
 from __future__ import annotations
 
@@ -142,9 +142,11 @@ def parse_args():
     ap.add_argument("--activation-checkpointing", choices=["config", "on", "off"], default="config",
                     help="per-block activation checkpointing: as the config names it (on for fsdp_7b), or forced")
     ap.add_argument("--workload", choices=["train", "serve", "layers"], default="train",
-                    help="train (default) and serve: the headline metric; layers: the layered decoder (Tedirax) beside the "
+                    help="train (default) and serve: the headline metric; layers: a layered decoder beside the "
                          "TransformerLM at equal size, prompt and decode steps and every kernel, 1 GPU")
     ap.add_argument("--layers-sizes", default="0.35b,1.3b,7b-8layers", help="layers: sizes to run, with commas between them")
+    ap.add_argument("--layers-model", choices=["Tedirax", "Beledra"], default="Tedirax",
+                    help="layers: which layered decoder (Beledra: beside Tedirax and the TransformerLM)")
     ap.add_argument("--no-kernels", action="store_true", help="layers: whole steps only")
     ap.add_argument("--serving-requests", type=int, default=None,
                     help="requests of the Poisson trace per GPU (serve: default 1024; train: a short serving run of "
@@ -505,7 +507,7 @@ def run_layers(args, local_rank, world):
     for size in args.layers_sizes.split(","):
         clocks = ClockSampler(local_rank)
         clocks.start()
-        rec = next(bench_layers.run([size], args.steps, max(3, args.warmup), not args.no_kernels))
+        rec = next(bench_layers.run([size], args.steps, max(3, args.warmup), not args.no_kernels, args.layers_model))
         print(json.dumps({"metric": "layered_decoder_steps", "data": "synthetic", "dtype": "bf16", "steps": args.steps,
                           "warmup": max(3, args.warmup), **rec, "clocks": clocks.stop(),
                           "l2_policy": "steps: weights and caches larger than L2 are streamed every step; kernels: L2 replaced "

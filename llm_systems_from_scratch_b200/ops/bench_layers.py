@@ -1,4 +1,4 @@
-"""Throughput of the layered decoder beside the TransformerLM at equal size, and the kernels of both against their roofline.
+"""Throughput of the layered decoders beside the TransformerLM at equal size, and the kernels of both against their roofline.
 
 ``models(size)`` times whole steps through the serving engine (a prompt step of several prompts; a decode step at a batch
 and a context), on the device with CUDA events; every step streams weights and caches that are larger than L2.
@@ -56,8 +56,11 @@ def peaks() -> dict:
 
 def build(kind: str, s: dict):
     from ..models.registry import build_model
-    if kind == "layered":
+    if kind == "Tedirax":
         return build_model(layered_config(s))
+    if kind == "Beledra":
+        from .bench_beledra import beledra_config
+        return build_model(beledra_config(s))
     return build_model(dict(vocab_size=s["vocab"], context_length=4096, d_model=s["width"], num_layers=s["runs"],
                             num_heads=s["heads"], d_ff=s["ff"], rope_theta=10000.0))
 
@@ -118,13 +121,12 @@ def step_times(kind: str, s: dict, steps: int, warmup: int) -> dict:
     return rec
 
 
-def models(size: str, steps: int = 10, warmup: int = 3) -> dict:
+def models(size: str, steps: int = 10, warmup: int = 3, kinds=("Tedirax", "TransformerLM")) -> dict:
     s = SIZES[size]
     out = {"size": size, "prompts": PROMPTS, "prompt_len": PROMPT_LEN, "context": CONTEXT}
-    for kind in ("layered", "transformer"):
+    for kind in kinds:
         rec = step_times(kind, s, steps, warmup)
-        name = "Tedirax" if kind == "layered" else "TransformerLM"
-        out[name] = {"prefill_ms": round(rec["prefill_ms"], 3),
+        out[kind] = {"prefill_ms": round(rec["prefill_ms"], 3),
                      "prefill_tok_per_s": round(PROMPTS * PROMPT_LEN / rec["prefill_ms"] * 1e3),
                      "prefill_launches": rec["prefill_launches"],
                      **{f"decode_ms_b{b}": round(rec[f"decode_ms_b{b}"], 3) for b in DECODE_BATCHES},
@@ -371,10 +373,15 @@ def _decode_kernels(s, t, b):
     add("latent_norm_append", "rmsnorm_fwd", b * (s["q_rank"] + kvr) * 4, 0, append)
 
 
-def run(sizes, steps: int = 10, warmup: int = 3, per_kernel: bool = True):
-    """One record per size."""
+def run(sizes, steps: int = 10, warmup: int = 3, per_kernel: bool = True, model: str = "Tedirax"):
+    """One record per size: Tedirax beside the TransformerLM, or Beledra beside both."""
     for size in sizes:
-        rec = models(size, steps, warmup)
+        if model == "Beledra":
+            from . import bench_beledra
+            rec = models(size, steps, warmup, ("Beledra", "Tedirax", "TransformerLM"))
+            more = bench_beledra.kernels
+        else:
+            rec, more = models(size, steps, warmup), kernels
         if per_kernel:
-            rec.update(kernels(size))
+            rec.update(more(size))
         yield rec
