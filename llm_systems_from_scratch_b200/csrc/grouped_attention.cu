@@ -119,6 +119,139 @@ __global__ void __launch_bounds__(256) grouped_prep_kernel(const GroupedPrepPara
   }
 }
 
+// The same for sizes in whole pieces of 8 elements: LPV lanes own a vector, one piece each, in ROWS rows one after the other.
+template <typename T>
+struct Piece {                    // 8 elements as they are stored
+  uint4 v[sizeof(T) / 2];
+};
+__device__ __forceinline__ void unpack(const Piece<__nv_bfloat16>& r, float (&f)[8]) {
+  const float2 a = unpack_bf16x2(r.v[0].x), b = unpack_bf16x2(r.v[0].y), c = unpack_bf16x2(r.v[0].z), d = unpack_bf16x2(r.v[0].w);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
+}
+__device__ __forceinline__ void unpack(const Piece<float>& r, float (&f)[8]) {
+  f[0] = __uint_as_float(r.v[0].x); f[1] = __uint_as_float(r.v[0].y); f[2] = __uint_as_float(r.v[0].z); f[3] = __uint_as_float(r.v[0].w);
+  f[4] = __uint_as_float(r.v[1].x); f[5] = __uint_as_float(r.v[1].y); f[6] = __uint_as_float(r.v[1].z); f[7] = __uint_as_float(r.v[1].w);
+}
+template <typename T>
+__device__ __forceinline__ Piece<T> load_piece(const T* p) {
+  Piece<T> r;
+#pragma unroll
+  for (int j = 0; j < (int)sizeof(T) / 2; ++j) r.v[j] = reinterpret_cast<const uint4*>(p)[j];
+  return r;
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+}
+__device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+}
+
+template <typename T, int LPV, int ROWS>
+__global__ void __launch_bounds__(512, 2) grouped_prep_pieces_kernel(const GroupedPrepParams p) {
+  pdl_sync();
+  const int piece = threadIdx.x % LPV, c = piece * 8;
+  const int nq = p.heads * p.maps, nk = p.wk != nullptr ? p.kv_heads * p.maps : 0, nv = p.wk != nullptr ? p.kv_heads : 0;
+  const int v = blockIdx.y * (blockDim.x / LPV) + threadIdx.x / LPV;             // this thread's vector in every row
+  const bool query = v < nq, value = v >= nq + nk, mine = v < nq + nk + nv;
+  const int row0 = blockIdx.x * ROWS, n = min(ROWS, p.rows - row0);
+  const int src_off = value ? (nq + nk) * p.dim + (v - nq - nk) * p.vdim : v * p.dim;      // the keys follow the queries
+  const int len = value ? p.vdim : p.dim;
+  const T* src = reinterpret_cast<const T*>(p.proj) + row0 * p.ld + src_off;
+  const int half = p.rot / 2, shift = half / 8;
+  const bool low = c < half, turned = c < p.rot && !value;
+  const int partner = turned ? (low ? piece + shift : piece - shift) : piece;    // lane that holds the other half of the pairs
+  const uint32_t lanes = LPV == 32 ? 0xffffffffu : (((1u << (LPV & 31)) - 1u) << ((threadIdx.x & 31) / LPV * LPV));
+  Piece<T> raw[ROWS];
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {                               // all rows are requested before the first is worked on
+#pragma unroll
+    for (int j = 0; j < (int)sizeof(T) / 2; ++j) raw[i].v[j] = make_uint4(0, 0, 0, 0);
+    if (i < n && mine && c < len) raw[i] = load_piece(src + i * p.ld + c);
+  }
+  float w[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) w[j] = 0.f;
+  if (mine && !value && c < p.dim) unpack(load_piece(reinterpret_cast<const T*>(query ? p.wq : p.wk) + c), w);
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    if (i >= n) break;
+    float f[8];
+    unpack(raw[i], f);
+    if (!value) {
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
+#pragma unroll
+      for (int o = LPV / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(lanes, ss, o);
+      const float r = rsqrtf(ss / (float)p.dim + p.eps);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] *= r * w[j];
+      if (p.rot > 0) {
+        float o[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) o[j] = __shfl_sync(lanes, f[j], partner, LPV);
+        if (turned) {
+          int at = p.positions[row0 + i];
+          if (at < 0 || at >= p.ctx) {
+            if (piece == 0) report_bad_arg(p.status, 14);
+            at = 0;
+          }
+          float cs[8], sn[8];
+          const float* tab = p.cos_sin + (long long)at * half + (low ? c : c - half);
+          unpack(load_piece(tab), cs);
+          unpack(load_piece(tab + (long long)p.ctx * half), sn);
+          const float sign = low ? -1.f : 1.f;
+#pragma unroll
+          for (int j = 0; j < 8; ++j) f[j] = fmaf(f[j], cs[j], sign * o[j] * sn[j]);
+        }
+      }
+    }
+    if (!mine) continue;
+    if (query) {
+      T* dst = reinterpret_cast<T*>(p.q) + ((long long)(row0 + i) * nq + v) * p.qp;
+      if (c < p.qp) store8(dst + c, f);                          // lanes past dim: zeros, the pad behind the vector
+      continue;
+    }
+    const long long slot = p.slots[row0 + i];
+    if (slot < 0) continue;                                      // padding row of the batch
+    if (slot >= p.num_slots) {
+      if (piece == 0) report_bad_arg(p.status, 13);
+      continue;
+    }
+    T* dst = reinterpret_cast<T*>(p.cache) + slot * ((long long)p.kv_heads * (p.maps * p.kp + p.vp)) +
+             (value ? nk * p.kp + (v - nq - nk) * p.vp : (v - nq) * p.kp);
+    if (c < len) store8(dst + c, f);
+    if (value)
+      for (int e = c + LPV * 8; e < p.vdim; e += LPV * 8) {      // values longer than a key: copied
+        float g[8];
+        unpack(load_piece(src + i * p.ld + e), g);
+        store8(dst + e, g);
+      }
+  }
+}
+
+template <typename T, int LPV>
+static void launch_prep_lanes(const GroupedPrepParams& p, int vectors, cudaStream_t st) {
+  int threads = (vectors * LPV + 31) / 32 * 32;
+  if (threads > 512) {                                           // several blocks of equal size per row
+    const int blocks = (threads + 511) / 512;
+    threads = (threads / blocks + 31) / 32 * 32;
+  }
+  const int per = threads / LPV;
+  const unsigned ny = (unsigned)((vectors + per - 1) / per);
+  if (p.rows >= 148 * 16) launch_dep(grouped_prep_pieces_kernel<T, LPV, 4>, dim3((p.rows + 3) / 4, ny), threads, 0, st, p);
+  else launch_dep(grouped_prep_pieces_kernel<T, LPV, 1>, dim3(p.rows, ny), threads, 0, st, p);
+}
+
+template <typename T>
+static void launch_prep_pieces(const GroupedPrepParams& p, cudaStream_t st) {
+  const int vectors = p.heads * p.maps + (p.wk != nullptr ? p.kv_heads * (p.maps + 1) : 0);
+  if (p.dim <= 64) launch_prep_lanes<T, 8>(p, vectors, st);
+  else if (p.dim <= 128) launch_prep_lanes<T, 16>(p, vectors, st);
+  else launch_prep_lanes<T, 32>(p, vectors, st);
+}
+
 // ------------------------------------------------------------------------------------------------------ general form
 // One warp per (row, head), keys one after the other; any size, T = bf16 or fp32.  row_seq[row] names the row's line of
 // `tables` (null: line `row`).
@@ -211,8 +344,9 @@ __global__ void __launch_bounds__(128) grouped_rows_kernel(const GroupedRowsPara
 // One CTA = one request, up to 16 query vectors (heads x maps) of one key/value head, one split of the window.  The vectors
 // are the M = 16 rows of mma.sync, so a cached byte is read once for all of them; with two maps a query vector is zero
 // outside its own map's columns and both maps' keys are one key of twice the length.
-// The four warps work on their own tiles of 16 tokens (round robin): own cp.async ring, own softmax state (online, in
-// fragments), own output; nothing is shared before the end, so the loop has no block barrier.
+// The four warps work on their own tiles of 16 tokens (round robin): own ring (bulk copies, one per token and key or value, a lane
+// each), own softmax state (online, in fragments), own output; nothing is shared before the end, so the loop has no block
+// barrier.
 constexpr int GD_WARPS = 4, GD_STAGES = 3, GD_TOK = 16;
 
 __device__ __forceinline__ void gd_ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
@@ -234,10 +368,6 @@ __device__ __forceinline__ void gd_mma(float (&c)[4], const uint32_t (&a)[4], ui
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void gd_copy16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-
 struct GroupedDecodeParams {
   const __nv_bfloat16 *q, *cache, *gate;
   __nv_bfloat16* o;
@@ -258,7 +388,8 @@ struct GroupedDecodeSmem {
   static constexpr int RING = GD_WARPS * GD_STAGES * STAGE * 2;
   static constexpr int OPITCH = VT * 8 + 4;
   static constexpr int MERGE = GD_WARPS * (16 * OPITCH + 32) * 4;
-  static constexpr int TOTAL = RING > MERGE ? RING : MERGE;
+  static constexpr int OFF_BAR = RING > MERGE ? RING : MERGE;              // a barrier per warp and stage, the abort word
+  static constexpr int TOTAL = OFF_BAR + GD_WARPS * GD_STAGES * 8 + 16;
 };
 
 // Heads of one row from their merged maps: value(m, c) gives map m's normalised output.  One warp per head.
@@ -297,19 +428,24 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
   extern __shared__ __align__(16) uint8_t gd_smem[];
   const GroupedShape& s = p.s;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int g = blockIdx.y / p.groups, grp = blockIdx.y - g * p.groups, split = blockIdx.z, row = blockIdx.x;
+  // the key/value heads of a row are neighbours: they read neighbouring parts of the same cache rows at about the same time
+  const int g = blockIdx.x / p.groups, grp = blockIdx.x - g * p.groups, row = blockIdx.y, split = blockIdx.z;
   const int per_kv = s.heads / s.kv_heads, hpg = 16 / s.maps;              // query heads per key/value head and per CTA
   const int h0 = g * per_kv + grp * hpg, nh = min(hpg, per_kv - grp * hpg);
-  const int kd = s.maps * s.kp, kvec = kd / 8, vvec = s.vp / 8;
+  const int kd = s.maps * s.kp;
   const int width = s.kv_heads * (kd + s.vp);
   __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(gd_smem) + warp * GD_STAGES * L::STAGE;
-  // pad columns of the warp's ring: finite
-  for (int i = lane; i < GD_STAGES * GD_TOK; i += 32) {
-    __nv_bfloat16* k = ring + (i / GD_TOK) * L::STAGE + (i % GD_TOK) * L::KPITCH;
-    __nv_bfloat16* v = ring + (i / GD_TOK) * L::STAGE + GD_TOK * L::KPITCH + (i % GD_TOK) * L::VPITCH;
-    for (int c = kvec; c < KT * 2; ++c) *reinterpret_cast<uint4*>(k + c * 8) = make_uint4(0, 0, 0, 0);
-    for (int c = vvec; c < VT; ++c) *reinterpret_cast<uint4*>(v + c * 8) = make_uint4(0, 0, 0, 0);
+  uint64_t* full = reinterpret_cast<uint64_t*>(gd_smem + L::OFF_BAR) + warp * GD_STAGES;
+  volatile uint32_t* abort_word = reinterpret_cast<uint32_t*>(gd_smem + L::OFF_BAR + GD_WARPS * GD_STAGES * 8);
+  // pad columns, and the places of tokens that are not seen, stay finite
+  for (int i = lane; i < GD_STAGES * L::STAGE / 8; i += 32) reinterpret_cast<uint4*>(ring)[i] = make_uint4(0, 0, 0, 0);
+  if (lane == 0) {
+    for (int i = 0; i < GD_STAGES; ++i) mbar_init(&full[i], 1);
+    fence_barrier_init();
   }
+  if (threadIdx.x == 0) *abort_word = 0;
+  fence_proxy_async_smem();
+  __syncthreads();
   pdl_sync();
   const int pos = p.positions[row];
   const bool live = p.slots[row] >= 0 && pos >= 0;
@@ -319,38 +455,32 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
   const int i0 = min(total, split * per), tiles = min(total, i0 + per) - i0;
   const int* table = p.tables + (long long)row * p.max_pages;
 
-  auto request = [&](int i) {              // tile i0 + i of this split; one lane per token looks up the page
-    const int t0 = (first + i0 + i) * GD_TOK, t = t0 + (lane & 15);
-    long long src = -1;
-    if (t >= lo && t <= pos) {
-      const int pg = t / p.page_size;
-      const int page = pg < p.max_pages ? table[pg] : -1;
-      if ((unsigned)page < (unsigned)p.num_pages) src = (long long)page * p.page_size + t % p.page_size;
-      else report_bad_arg(p.status, 16);
-    }
-    __nv_bfloat16* k = ring + ((i / GD_WARPS) % GD_STAGES) * L::STAGE;
-    __nv_bfloat16* v = k + GD_TOK * L::KPITCH;
-    for (int base = 0; base < kvec + vvec; base += 32) {
-      const int c = base + lane;
-      const bool is_k = c < kvec, on = c < kvec + vvec;
-      __nv_bfloat16* d = is_k ? k + c * 8 : v + (c - kvec) * 8;
-      const int dp = is_k ? L::KPITCH : L::VPITCH;
-      const __nv_bfloat16* from = p.cache + (is_k ? g * kd + c * 8 : s.kv_heads * kd + g * s.vp + (c - kvec) * 8);
-#pragma unroll
-      for (int tok = 0; tok < GD_TOK; ++tok) {
-        const long long r = __shfl_sync(0xffffffffu, src, tok);
-        if (!on) continue;
-        if (r >= 0) gd_copy16(smem_u32(d + tok * dp), from + r * width);
-        else *reinterpret_cast<uint4*>(d + tok * dp) = make_uint4(0, 0, 0, 0);          // finite; masked below
-      }
-    }
+  auto look_up = [&](int i) -> long long {     // cache row of this lane's token of tile i0 + i of this split; -1: none
+    if (i >= tiles) return -1;
+    const int t = (first + i0 + i) * GD_TOK + (lane & 15);
+    if (t < lo || t > pos) return -1;
+    const int pg = t / p.page_size;
+    const int page = pg < p.max_pages ? table[pg] : -1;
+    if ((unsigned)page < (unsigned)p.num_pages) return (long long)page * p.page_size + t % p.page_size;
+    report_bad_arg(p.status, 16);
+    return -1;
   };
-  auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+  const uint32_t k_bytes = (uint32_t)kd * 2, v_bytes = (uint32_t)s.vp * 2;
+  const int from = lane < 16 ? g * kd : s.kv_heads * kd + g * s.vp;            // lanes 0 - 15: keys, 16 - 31: values
+  auto request = [&](int i, long long src) {
+    const int st = (i / GD_WARPS) % GD_STAGES;
+    __nv_bfloat16* k = ring + st * L::STAGE;
+    const uint32_t seen = __ballot_sync(0xffffffffu, src >= 0) & 0xffffu;
+    if (lane == 0) mbar_expect_tx(&full[st], __popc(seen) * (k_bytes + v_bytes));
+    __syncwarp();
+    if (src >= 0)
+      bulk_load(lane < 16 ? k + lane * L::KPITCH : k + GD_TOK * L::KPITCH + (lane - 16) * L::VPITCH, p.cache + src * width + from,
+                lane < 16 ? k_bytes : v_bytes, &full[st]);
+  };
 #pragma unroll
-  for (int n = 0; n < GD_STAGES - 1; ++n) {
-    if (warp + n * GD_WARPS < tiles) request(warp + n * GD_WARPS);
-    commit();
-  }
+  for (int n = 0; n < GD_STAGES; ++n)
+    if (warp + n * GD_WARPS < tiles) request(warp + n * GD_WARPS, look_up(warp + n * GD_WARPS));
+  long long next = look_up(warp + GD_STAGES * GD_WARPS);            // looked up a tile earlier than it is requested
   // query fragments: vector r = head * maps + map, columns of its own map only
   uint32_t qf[KT][4];
 #pragma unroll
@@ -375,12 +505,24 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
     for (int i = 0; i < 2; ++i) bias[i] = p.bias + (long long)(h0 + min(((lane >> 2) + i * 8) / s.maps, nh - 1)) * p.bias_len;
   }
 
+  float bn[2][4];                                      // bias of the tile after the one at work
+  auto load_bias = [&](int i) {
+    const int t = (first + i0 + i) * GD_TOK + (lane & 3) * 2;
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) bn[n][e] = __ldg(bias[e >> 1] + max(0, min(pos - (t + n * 8 + (e & 1)), p.bias_len - 1)));
+  };
+  if (p.bias != nullptr) load_bias(warp);
+
   for (int i = warp; i < tiles; i += GD_WARPS) {
-    asm volatile("cp.async.wait_group %0;" ::"n"(GD_STAGES - 2) : "memory");
-    __syncwarp();
-    if (i + (GD_STAGES - 1) * GD_WARPS < tiles) request(i + (GD_STAGES - 1) * GD_WARPS);
-    commit();
-    const __nv_bfloat16* k = ring + ((i / GD_WARPS) % GD_STAGES) * L::STAGE;
+    const int round = i / GD_WARPS, st = round % GD_STAGES;
+    const bool landed = mbar_wait(&full[st], (round / GD_STAGES) & 1, abort_word);
+    if (!__all_sync(0xffffffffu, landed)) {
+      *abort_word = ERR_WAIT_FULL;
+      break;
+    }
+    const __nv_bfloat16* k = ring + st * L::STAGE;
     const __nv_bfloat16* v = k + GD_TOK * L::KPITCH;
     float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
     const uint32_t k_addr = smem_u32(k + ((lane & 7) + (lane >> 4) * 8) * L::KPITCH + ((lane >> 3) & 1) * 8);
@@ -400,11 +542,12 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
         const int t = t0 + n * 8 + (e & 1);
         float x = sc[n][e] * scale_log2;
         const bool seen = t >= lo && t <= pos;
-        if (p.bias != nullptr) x += __ldg(bias[e >> 1] + max(0, min(pos - t, p.bias_len - 1))) * 1.4426950408889634f;
+        if (p.bias != nullptr) x = fmaf(bn[n][e], 1.4426950408889634f, x);
         x = seen ? x : -INFINITY;
         sc[n][e] = x;
         mx[e >> 1] = fmaxf(mx[e >> 1], x);
       }
+    if (p.bias != nullptr && i + GD_WARPS < tiles) load_bias(i + GD_WARPS);
     float alpha[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
@@ -438,10 +581,19 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
       gd_mma(acc[2 * j], pf, b[0], b[1]);
       gd_mma(acc[2 * j + 1], pf, b[2], b[3]);
     }
-    __syncwarp();                                      // the tile's stage is refilled two tiles from now
+    __syncwarp();                                      // everybody has read the stage
+    if (i + GD_STAGES * GD_WARPS < tiles) {
+      request(i + GD_STAGES * GD_WARPS, next);
+      next = look_up(i + (GD_STAGES + 1) * GD_WARPS);
+    }
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();                                     // the rings become the merge buffer
+  if (*abort_word != 0) {                              // give copies that may still be in flight time to land
+    if (threadIdx.x == 0 && p.status != nullptr) atomicCAS(p.status, 0u, *abort_word | (blockIdx.x << 8));
+    const uint64_t w0 = globaltimer_ns();
+    while (globaltimer_ns() - w0 < 200000ull) __nanosleep(1000);
+  }
+  __syncthreads();
   float* mo = reinterpret_cast<float*>(gd_smem) + warp * (16 * L::OPITCH + 32);
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
@@ -547,7 +699,7 @@ static int launch_grouped_decode(const GroupedDecodeParams& p, cudaStream_t st) 
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
     configured = true;
   }
-  launch_dep(kern, dim3(p.rows, p.s.kv_heads * p.groups, p.splits), GD_WARPS * 32, smem, st, p);
+  launch_dep(kern, dim3(p.s.kv_heads * p.groups, p.rows, p.splits), GD_WARPS * 32, smem, st, p);
   if (p.splits > 1)
     launch_dep(grouped_merge_kernel, (unsigned)(((long long)p.rows * p.s.heads + 3) / 4), 128, 0, st, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
@@ -569,6 +721,11 @@ extern "C" int b200_grouped_prep(const void* proj, long long ld, void* q, void* 
   p.eps = s->eps; p.status = status;
   const uintptr_t ptrs = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) |
                          reinterpret_cast<uintptr_t>(wq) | reinterpret_cast<uintptr_t>(wk) | reinterpret_cast<uintptr_t>(cos_sin);
+  if (s->dim % 8 == 0 && s->dim <= 256 && s->vdim % 8 == 0 && (rot / 2) % 8 == 0 && ld % 8 == 0 && (ptrs & 15) == 0) {
+    if (f32) launch_prep_pieces<float>(p, st);
+    else launch_prep_pieces<__nv_bfloat16>(p, st);
+    return cudaGetLastError() == cudaSuccess ? 0 : -4;
+  }
   const bool vec = s->dim % 4 == 0 && s->vdim % 4 == 0 && (rot / 2) % 4 == 0 && ld % 4 == 0 && (ptrs & 15) == 0;
   const long long items = (long long)rows * (s->heads * s->maps + (wk != nullptr ? s->kv_heads * (s->maps + 1) : 0));
   const int warps = items >= 148 * 8 * 4 ? 8 : 2;
@@ -621,7 +778,7 @@ extern "C" int b200_grouped_decode(const void* q, const void* cache, void* o, lo
   p.page_size = page_size; p.num_pages = num_pages; p.splits = splits; p.s = *s; p.status = status;
   const int hpg = 16 / s->maps;
   p.groups = (s->heads / s->kv_heads + hpg - 1) / hpg;
-  if ((long long)s->kv_heads * p.groups > 65535) return -12;
+  if (rows > 65535) return -12;
   const bool v64 = s->vp <= 64;
   if (kd <= 64) return v64 ? launch_grouped_decode<4, 8>(p, st) : launch_grouped_decode<4, 16>(p, st);
   if (kd <= 128) return v64 ? launch_grouped_decode<8, 8>(p, st) : launch_grouped_decode<8, 16>(p, st);

@@ -14,8 +14,11 @@ int make_tmap_bf16_2d(CUtensorMap* tm, const void* ptr, uint64_t rows, uint64_t 
 struct MlstmParams {
   const void* proj;          // (rows, ld_proj): q | k | v | gate, heads contiguous inside each
   long long ld_proj;
-  const float* gates;        // (rows, ld_gates): input gate pre-activations of all heads | forget gates
-  long long ld_gates;
+  const float* gates;        // (rows, ld_gates): input gate pre-activations of all heads | forget gates; null: the decode step
+  long long ld_gates;        // takes the products of its input row with the gates' weights itself
+  const void *h, *w_gates;   // gates null: (rows, ld_h) and (2 * heads, ld_wg), `width` columns
+  long long ld_h, ld_wg;
+  int width;
   const float* gate_bias;    // (2 * heads), the same order
   const void* weight;        // (heads * vdim)
   void* y;                   // (rows, ld_y)
@@ -153,6 +156,16 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) mlstm_step_kernel(const M
   float* base = p.state + ((long long)slot * p.heads + h) * p.stride;
   float* N = base + (long long)D * E;
   float4* S = reinterpret_cast<float4*>(base) + tx;
+  // the gates' operands are few and in L2: the first of them are requested before the state, not behind it
+  float hx[4] = {0.f, 0.f, 0.f, 0.f}, hi[4] = {0.f, 0.f, 0.f, 0.f}, hf[4] = {0.f, 0.f, 0.f, 0.f};
+  const T* hr = reinterpret_cast<const T*>(p.h) + (long long)seq * p.ld_h;
+  const T* wi = reinterpret_cast<const T*>(p.w_gates) + (long long)h * p.ld_wg;
+  const T* wf = wi + (long long)p.heads * p.ld_wg;
+  if (p.gates == nullptr && threadIdx.x * 4 < p.width) {
+    load_vec<4>(hr + threadIdx.x * 4, hx);
+    load_vec<4>(wi + threadIdx.x * 4, hi);
+    load_vec<4>(wf + threadIdx.x * 4, hf);
+  }
   float4 s[NR];
 #pragma unroll
   for (int j = 0; j < NR; ++j) {
@@ -161,9 +174,30 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) mlstm_step_kernel(const M
     if (on && d < D && !fresh) s[j] = __ldcs(S + (long long)d * groups);
   }
   const float m = fresh ? 0.f : N[D];
-  const float* gt = p.gates + (long long)seq * p.ld_gates;
-  const float li = log_input_gate(gt[h] + p.gate_bias[h], p.cap);
-  const float lf = log_forget_gate(gt[p.heads + h] + p.gate_bias[p.heads + h], p.cap);
+  float zi = 0.f, zf = 0.f;
+  if (p.gates != nullptr) {
+    const float* gt = p.gates + (long long)seq * p.ld_gates;
+    zi = gt[h];
+    zf = gt[p.heads + h];
+  } else {
+    for (int c = threadIdx.x * 4; c < p.width; c += 1024) {            // pitches are multiples of 4, what lies in the pads is left out
+      if (c >= 1024) {
+        load_vec<4>(hr + c, hx);
+        load_vec<4>(wi + c, hi);
+        load_vec<4>(wf + c, hf);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float xv = c + i < p.width ? hx[i] : 0.f;
+        zi = fmaf(xv, hi[i], zi);
+        zf = fmaf(xv, hf[i], zf);
+      }
+    }
+    zi = block_total(zi, red);
+    zf = block_total(zf, red);
+  }
+  const float li = log_input_gate(zi + p.gate_bias[h], p.cap);
+  const float lf = log_forget_gate(zf + p.gate_bias[p.heads + h], p.cap);
   const float mn = fmaxf(lf + m, li), keep = expf(lf + m - mn), take = expf(li - mn);
   const float qscale = rsqrtf((float)D);
   const T *qr = pr + h * D, *kr = pr + p.heads * D + h * D;
@@ -220,14 +254,13 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) mlstm_step_kernel(const M
 // bf16 parts (hi + lo, 16 significant bits) whose products accumulate in fp32.  n . q is kept beside it on the FMA pipes.
 //   tensor memory: scores, then P [0, 128)  O_inter [128, 128 + EP)  O_intra [256, 256 + EP)  S [384, 384 + EP)
 //   shared memory: Q | K, then K~ hi | K~ lo, later the outputs on their way | V | S_prev hi, lo, all 128-byte swizzled panels
-// Eight warps do the element-wise phases (two warps per 32 lanes of tensor memory, half of the columns each); a ninth issues TMA
-// and MMAs.
+// Sixteen warps do the element-wise phases (four warps per 32 lanes of tensor memory, a quarter of the columns each); one of them,
+// which has no score that is not masked, also issues TMA and MMAs and scans the next chunk's gates.  The output gates come in and
+// the outputs go out through K~ lo's place, in whole rows.
 constexpr int ML_CHUNK = 128;
-constexpr int ML_WORKERS = 256;
-constexpr int ML_THREADS = ML_WORKERS + 32;
+constexpr int ML_THREADS = 512;
+constexpr int ML_ISSUER = 12;             // rows 0 - 31, keys 96 - 127
 constexpr float ML_NEVER = -1e30f;        // log input gate of a token that is not there
-
-__device__ __forceinline__ void ml_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }   // ML_WORKERS threads
 
 template <int EP>
 struct MlstmSmem {
@@ -235,10 +268,11 @@ struct MlstmSmem {
   static constexpr int VT = EP / 64 * 16384;
   static constexpr int OFF_Q = 0, OFF_K = TILE, OFF_KL = 2 * TILE, OFF_V = 3 * TILE;
   static constexpr int OFF_SH = OFF_V + VT, OFF_SL = OFF_SH + VT, OFF_F = OFF_SL + VT;
-  // floats: a, M, m_t [2][128] each; n [128]; den, sum of squares [2][128] each; column sums of K~ [2048]; m_prev, m_next [2]
-  static constexpr int FLOATS = 3 * 256 + 128 + 2 * 256 + 2048 + 4;
+  // floats: a, M [2][128] in log2 units, m_t [2][128]; n [128]; den, sum of squares [4][128] each; column sums of K~ [4096];
+  // the heads' weight [128]; m_prev [2]
+  static constexpr int FLOATS = 3 * 256 + 128 + 2 * 512 + 4096 + 128 + 4;
   static constexpr int OFF_BAR = OFF_F + FLOATS * 4;
-  static constexpr int TOTAL = OFF_BAR + 4 * 8 + 16 + 1024;
+  static constexpr int TOTAL = OFF_BAR + 5 * 8 + 16 + 1024;
 };
 
 // 16-byte piece `c8` (8 columns) of row `r` in a tile of 64-column panels, 128-byte swizzle
@@ -249,41 +283,59 @@ __device__ __forceinline__ void ml_unpack8(const uint4& v, float (&f)[8]) {
   const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y), c = unpack_bf16x2(v.z), d = unpack_bf16x2(v.w);
   f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
 }
-// x = hi + lo with both parts bf16, eight values at a time
-__device__ __forceinline__ void ml_split8(const float (&x)[8], uint4& hi, uint4& lo) {
-  uint32_t h[4], l[4];
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    h[i] = pack_bf16x2(x[2 * i], x[2 * i + 1]);
-    const float2 b = unpack_bf16x2(h[i]);
-    l[i] = pack_bf16x2(x[2 * i] - b.x, x[2 * i + 1] - b.y);
-  }
-  hi = make_uint4(h[0], h[1], h[2], h[3]);
-  lo = make_uint4(l[0], l[1], l[2], l[3]);
+// Two values as hi + lo, both bf16: hi is cut off (the remainder is exact), lo rounded.  Integer and FMA pipes only: the conversion
+// unit shares its port with ex2.
+__device__ __forceinline__ void ml_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  const uint32_t a = __float_as_uint(x), b = __float_as_uint(y);
+  hi = __byte_perm(a, b, 0x7632);
+  lo = pack_bf16x2_alu(x - __uint_as_float(a & 0xffff0000u), y - __uint_as_float(b & 0xffff0000u));
 }
-__device__ __forceinline__ float ml_exp(float x) {        // x <= 0; far below zero gives zero
+__device__ __forceinline__ void ml_split8(const float (&x)[8], uint4& hi, uint4& lo) {
+  ml_split2(x[0], x[1], hi.x, lo.x);
+  ml_split2(x[2], x[3], hi.y, lo.y);
+  ml_split2(x[4], x[5], hi.z, lo.z);
+  ml_split2(x[6], x[7], hi.w, lo.w);
+}
+__device__ __forceinline__ float ml_exp2(float x) {       // x <= 0; far below zero gives zero
   float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x * 1.4426950408889634f));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+__device__ __forceinline__ float ml_sigmoid(float g) {    // (1 + tanh(g / 2)) / 2
+  float t;
+  asm("tanh.approx.f32 %0, %1;" : "=f"(t) : "f"(0.5f * g));
+  return fmaf(0.5f, t, 0.5f);
+}
+template <int N>                                          // 16 or 32 columns of tensor memory
+__device__ __forceinline__ void ml_tmem_ld(uint32_t addr, uint32_t (&r)[N]) {
+  if constexpr (N == 32) tmem_ld_32x32(addr, r);
+  else tmem_ld_32x16(addr, r);
+}
+template <int N>
+__device__ __forceinline__ void ml_tmem_st(uint32_t addr, const uint32_t (&r)[N]) {
+  if constexpr (N == 32) tmem_st_32x32(addr, r);
+  else tmem_st_32x16(addr, r);
 }
 
 template <int EP>
 __global__ void __launch_bounds__(ML_THREADS, 1) mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tm_proj, const MlstmParams p) {
   using L = MlstmSmem<EP>;
-  constexpr int HE = EP / 2;                          // columns of O and S that a thread handles
+  constexpr int HE = EP / 4;                          // columns of O and S that a thread handles
+  constexpr float LOG2E = 1.4426950408889634f;
   extern __shared__ uint8_t ml_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ml_raw) + 1023) & ~uintptr_t(1023));
-  float* sa = reinterpret_cast<float*>(smem + L::OFF_F);      // [2][128] a_s
-  float *sM = sa + 256, *sm = sM + 256, *sn = sm + 256;       // [2][128] M_t, [2][128] m_t, [128] n
-  float *sden = sn + 128, *srms = sden + 256, *scol = srms + 256, *sprev = scol + 2048;   // m_prev of chunk ch in sprev[ch & 1]
+  float* sa = reinterpret_cast<float*>(smem + L::OFF_F);      // [2][128] a_s, log2 units
+  float *sM = sa + 256, *sm = sM + 256, *sn = sm + 256;       // [2][128] M_t, log2 units; [2][128] m_t; [128] n
+  float *sden = sn + 128, *srms = sden + 512, *scol = srms + 512, *sw = scol + 4096, *sprev = sw + 128;   // m_prev of chunk ch in sprev[ch & 1]
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR);
-  uint64_t *bar_a = bars, *bar_s = bars + 1, *bar_o = bars + 2, *bar_l = bars + 3;
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 4);
+  uint64_t *bar_a = bars, *bar_s = bars + 1, *bar_o = bars + 2, *bar_l = bars + 3, *bar_g = bars + 4;
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 5);
   volatile uint32_t* abort_word = tmem_holder + 1;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const bool issuer = warp == ML_ISSUER;
 
   if (tid == 0) {
-    for (int i = 0; i < 4; ++i) mbar_init(&bars[i], 1);
+    for (int i = 0; i < 5; ++i) mbar_init(&bars[i], 1);
     *abort_word = 0;
     fence_barrier_init();
     prefetch_tensormap(&tm_proj);
@@ -296,6 +348,7 @@ __global__ void __launch_bounds__(ML_THREADS, 1) mlstm_chunk_kernel(const __grid
   pdl_sync();
   const int seq = blockIdx.x / p.heads, h = blockIdx.x - seq * p.heads;
   const int D = p.dim, E = p.vdim;
+  if (tid < 128) sw[tid] = tid < E ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.weight)[h * E + tid]) : 0.f;
   fence_proxy_async_smem();           // the zeros above come before what TMA writes
   tc_fence_before();
   __syncthreads();
@@ -309,88 +362,84 @@ __global__ void __launch_bounds__(ML_THREADS, 1) mlstm_chunk_kernel(const __grid
   const int pos0 = rows > 0 ? p.positions[row0] : 0;
   float* state = p.state + ((long long)(live ? slot : 0) * p.heads + h) * p.stride;
   float* state_n = state + (long long)D * E;
-  const __nv_bfloat16* gg = reinterpret_cast<const __nv_bfloat16*>(p.proj) + (long long)row0 * p.ld_proj + 2 * p.heads * D +
-                            p.heads * E + h * E;
+  const int quarter = warp & 3, cg = warp >> 2;       // lanes of tensor memory, group of columns
+  const int r = quarter * 32 + lane;                  // this thread's row of tensor memory: a token, or a dim of S
+  const int e0 = cg * HE;                             // its first column of O and S
   __nv_bfloat16* gy = reinterpret_cast<__nv_bfloat16*>(p.y) + (long long)row0 * p.ld_y + h * E;
   const float* gates = p.gates + (long long)row0 * p.ld_gates + h;
-
-  const int quarter = warp & 3, half = warp >> 2;
-  const int r = quarter * 32 + lane;                  // this thread's row of tensor memory: a token, or a dim of S
   const uint32_t lane_addr = uint32_t(quarter * 32) << 16;
-  const uint32_t tm_a = tmem + lane_addr, tm_i = tmem + 128 + lane_addr, tm_o = tmem + 256 + lane_addr, tm_s = tmem + 384 + lane_addr;
+  const uint32_t tm_a = tmem + lane_addr + cg * 32, tm_i = tmem + 128 + lane_addr + e0, tm_o = tmem + 256 + lane_addr + e0,
+                 tm_s = tmem + 384 + lane_addr + e0;
   const float qscale = rsqrtf((float)D);
   const int chunks = live ? (rows + ML_CHUNK - 1) / ML_CHUNK : 0;
-  const bool worker = warp < ML_WORKERS / 32;
   bool ok = true;
 
-  // ---- log gates of a chunk, by warp 0: four tokens per lane are requested here ...
-  float gi[4], gf[4];
+  // ---- log gates of a chunk: the threads of the last column group request one token each ...
+  float gi = 0.f, gf = 0.f;
   auto request_gates = [&](int t0) {
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int t = t0 + lane * 4 + j;
-      gi[j] = gf[j] = 0.f;
-      if (t < rows) {
-        gi[j] = gates[(long long)t * p.ld_gates];
-        gf[j] = gates[(long long)t * p.ld_gates + p.heads];
-      }
+    const int t = t0 + tid - 384;
+    gi = gf = 0.f;
+    if (tid >= 384 && t < rows) {
+      gi = gates[(long long)t * p.ld_gates];
+      gf = gates[(long long)t * p.ld_gates + p.heads];
     }
   };
-  // ... and turned into a, M and m here
-  auto scan_gates = [&](int t0, int b, float m_prev) {
-    const float bi = p.gate_bias[h], bf = p.gate_bias[p.heads + h];
-    float F[4], a[4], sum = 0.f, top = ML_NEVER;
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const bool there = t0 + lane * 4 + j < rows;
-      sum += there ? log_forget_gate(gf[j] + bf, p.cap) : 0.f;
-      F[j] = sum;
-      a[j] = there ? log_input_gate(gi[j] + bi, p.cap) : ML_NEVER;
-    }
-    float run = sum;
+  const float bi = p.gate_bias[h], bf = p.gate_bias[p.heads + h];
+  auto log_gates = [&](int t0, int b) {               // ... leave their logarithms where a and M will be
+    if (tid < 384) return;
+    const bool there = t0 + tid - 384 < rows;
+    sa[b * 128 + tid - 384] = there ? log_input_gate(gi + bi, p.cap) : ML_NEVER;
+    sM[b * 128 + tid - 384] = there ? log_forget_gate(gf + bf, p.cap) : 0.f;
+  };
+  // ... and one warp turns them into a, M and m
+  auto scan_gates = [&](int b, float m_prev) {
+    const float4 li = *reinterpret_cast<const float4*>(sa + b * 128 + lane * 4), lf = *reinterpret_cast<const float4*>(sM + b * 128 + lane * 4);
+    float a[4] = {li.x, li.y, li.z, li.w}, F[4] = {lf.x, lf.x + lf.y, lf.x + lf.y + lf.z, lf.x + lf.y + lf.z + lf.w};
+    float run = F[3];
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const float x = __shfl_up_sync(0xffffffffu, run, o);
       if (lane >= o) run += x;
     }
-    run -= sum;                                       // forget gates of the lanes before
+    run -= F[3];                                      // forget gates of the lanes before
+    float top = ML_NEVER;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       F[j] += run;
       a[j] = a[j] == ML_NEVER ? ML_NEVER : a[j] - F[j];
       top = fmaxf(top, a[j]);
     }
-    float before = top;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float x = __shfl_up_sync(0xffffffffu, before, o);
-      if (lane >= o) before = fmaxf(before, x);
+      const float x = __shfl_up_sync(0xffffffffu, top, o);
+      if (lane >= o) top = fmaxf(top, x);
     }
-    before = __shfl_up_sync(0xffffffffu, before, 1);
-    float M = lane == 0 ? m_prev : fmaxf(m_prev, before);
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      M = fmaxf(M, a[j]);
-      sa[b * 128 + lane * 4 + j] = a[j];
-      sM[b * 128 + lane * 4 + j] = M;
-      sm[b * 128 + lane * 4 + j] = F[j] + M;
-    }
-    if (lane == 0) sprev[b] = m_prev;
+    top = __shfl_up_sync(0xffffffffu, top, 1);
+    float M = lane == 0 ? m_prev : fmaxf(m_prev, top);
+    float4 am, Mm, mm;
+    M = fmaxf(M, a[0]); am.x = a[0] * LOG2E; Mm.x = M * LOG2E; mm.x = F[0] + M;
+    M = fmaxf(M, a[1]); am.y = a[1] * LOG2E; Mm.y = M * LOG2E; mm.y = F[1] + M;
+    M = fmaxf(M, a[2]); am.z = a[2] * LOG2E; Mm.z = M * LOG2E; mm.z = F[2] + M;
+    M = fmaxf(M, a[3]); am.w = a[3] * LOG2E; Mm.w = M * LOG2E; mm.w = F[3] + M;
+    *reinterpret_cast<float4*>(sa + b * 128 + lane * 4) = am;
+    *reinterpret_cast<float4*>(sM + b * 128 + lane * 4) = Mm;
+    *reinterpret_cast<float4*>(sm + b * 128 + lane * 4) = mm;
+    if (lane == 0) sprev[b] = m_prev * LOG2E;
   };
-  // S: columns [half * HE + 32 c, + 32) of row r; split into shared memory, times g in tensor memory
-  auto publish_state = [&](const float (&s)[32], int c, float g) {
-    uint32_t raw[32];
+  // S: columns [e0, e0 + HE) of row r; split into shared memory, times g in tensor memory
+  auto publish_state = [&](const float (&s)[HE], float g) __attribute__((always_inline)) {
+    uint32_t raw[HE];
 #pragma unroll
-    for (int i = 0; i < 32; ++i) raw[i] = __float_as_uint(s[i] * g);
-    tmem_st_32x32(tm_s + half * HE + c * 32, raw);
+    for (int i = 0; i < HE; ++i) raw[i] = __float_as_uint(s[i] * g);
+    ml_tmem_st<HE>(tm_s, raw);
 #pragma unroll
-    for (int q = 0; q < 4; ++q) {
+    for (int q = 0; q < HE / 8; ++q) {
       float f[8];
 #pragma unroll
       for (int i = 0; i < 8; ++i) f[i] = r < D ? s[q * 8 + i] : 0.f;
       uint4 hi, lo;
       ml_split8(f, hi, lo);
-      const uint32_t at = ml_swz(r, (half * HE + c * 32) / 8 + q);
+      const uint32_t at = ml_swz(r, e0 / 8 + q);
       *reinterpret_cast<uint4*>(smem + L::OFF_SH + at) = hi;
       *reinterpret_cast<uint4*>(smem + L::OFF_SL + at) = lo;
     }
@@ -406,31 +455,25 @@ __global__ void __launch_bounds__(ML_THREADS, 1) mlstm_chunk_kernel(const __grid
     for (int i = 0; i < pe; ++i)
       tma_load_2d(smem + L::OFF_V + i * 16384, &tm_proj, bar_l, 2 * p.heads * D + h * E + i * 64, row0 + t);
   };
-  if (!worker && chunks > 0 && elect_one()) load_chunk(0);
+  if (issuer && chunks > 0 && elect_one()) load_chunk(0);
   __syncwarp();
-  if (worker && chunks > 0) {
-    if (warp == 0) {
-      request_gates(0);
-      scan_gates(0, 0, pos0 > 0 ? state_n[D] : 0.f);
-    }
-    if (tid >= 128) sn[tid - 128] = pos0 > 0 && tid - 128 < D ? state_n[tid - 128] : 0.f;
-    ml_barrier();
-    const float g = ml_exp(sprev[0] - sM[127]);
-#pragma unroll 1
-    for (int c = 0; c < HE / 32; ++c) {
-      float s[32];
+  if (chunks > 0) {
+    request_gates(0);
+    log_gates(0, 0);
+    request_gates(ML_CHUNK);
+  }
+  __syncthreads();
+  if (issuer && chunks > 0) scan_gates(0, pos0 > 0 ? state_n[D] : 0.f);
+  __syncthreads();
+  if (chunks > 0) {
+    if (tid < 128) sn[tid] = pos0 > 0 && tid < D ? state_n[tid] : 0.f;
+    float s[HE];
 #pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        const int e = half * HE + c * 32 + i;
-        s[i] = (pos0 > 0 && r < D && e < E) ? state[(long long)r * E + e] : 0.f;
-      }
-      publish_state(s, c, g);
-    }
+    for (int i = 0; i < HE; ++i) s[i] = (pos0 > 0 && r < D && e0 + i < E) ? state[(long long)r * E + e0 + i] : 0.f;
+    publish_state(s, ml_exp2(sprev[0] - sM[127]));
     tmem_st_wait();
   }
-  const int kp = D / 8, k_step = ML_WORKERS / kp, k_t = tid / kp, k_c8 = tid - k_t * kp;     // a thread's pieces of K
-  constexpr int PH = HE / 8, O_STEP = ML_WORKERS / PH, O_N = 128 / O_STEP;                   // ... and of half an output row
-  const int o_c8 = tid % PH, o_t = tid / PH;
+  const int kp = D / 8, k_step = ML_THREADS / kp, k_t = tid / kp, k_c8 = tid - k_t * kp;     // a thread's pieces of K
   const int ksteps = (D + 15) / 16;
 
   for (int ch = 0; ch < chunks; ++ch) {
@@ -438,244 +481,228 @@ __global__ void __launch_bounds__(ML_THREADS, 1) mlstm_chunk_kernel(const __grid
     const uint32_t ph = ch & 1;
     const bool last = ch + 1 == chunks;
     const float *a_b = sa + b * 128, *M_b = sM + b * 128;
-    if (worker) {
-      if (warp == 0 && !last) request_gates(t0 + ML_CHUNK);
-      if (!mbar_wait(bar_l, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_FULL; }
-      if (D & 15) {                                   // columns past dim that the last step of the products touches
-        if (half == 0) *reinterpret_cast<uint4*>(smem + L::OFF_Q + ml_swz(r, D / 8)) = make_uint4(0, 0, 0, 0);
-      }
-    }
+    if (!mbar_wait(bar_l, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_FULL; }
+    if ((D & 15) && cg == 0)                          // columns past dim that the last step of the products touches
+      *reinterpret_cast<uint4*>(smem + L::OFF_Q + ml_swz(r, D / 8)) = make_uint4(0, 0, 0, 0);
     fence_proxy_async_smem();
     tc_fence_before();
     __syncthreads();
 
-    if (!worker && elect_one()) {
-      tc_fence_after();
-      constexpr uint32_t id_qk = make_idesc_bf16(128, 128, false, false);
-      constexpr uint32_t id_xv = make_idesc_bf16(128, EP, false, true);
-      auto kstep = [](int k) { return (uint32_t)(((k / 4) * 16384 + (k % 4) * 32) >> 4); };
-      const uint64_t q = make_smem_desc(smem_u32(smem + L::OFF_Q), 16, 1024), k = make_smem_desc(smem_u32(smem + L::OFF_K), 16, 1024);
-      const uint64_t sh = make_smem_desc(smem_u32(smem + L::OFF_SH), 16384, 1024);
-      const uint64_t sl = make_smem_desc(smem_u32(smem + L::OFF_SL), 16384, 1024);
-      for (int i = 0; i < ksteps; ++i) umma_f16_ss(tmem, q + kstep(i), k + kstep(i), id_qk, i ? 1u : 0u);
-      umma_commit(bar_a);
-      for (int i = 0; i < ksteps; ++i) umma_f16_ss(tmem + 128, q + kstep(i), sh + (uint32_t)(i * 128), id_xv, i ? 1u : 0u);
-      for (int i = 0; i < ksteps; ++i) umma_f16_ss(tmem + 128, q + kstep(i), sl + (uint32_t)(i * 128), id_xv, 1u);
-    }
-    __syncwarp();
-    const float M_end = M_b[127], M_r = M_b[r];
-    const float c_r = ml_exp(sprev[b] - M_r);         // how much of the earlier state row r still sees
-    uint4 gate[2][O_N];
-    if (worker) {
-#pragma unroll
-      for (int x = 0; x < 2; ++x)
-#pragma unroll
-        for (int j = 0; j < O_N; ++j) {
-          const int t = o_t + j * O_STEP, c = x * HE + o_c8 * 8;
-          gate[x][j] = make_uint4(0, 0, 0, 0);
-          if (t < n && c < E) gate[x][j] = *reinterpret_cast<const uint4*>(gg + (long long)(t0 + t) * p.ld_proj + c);
-        }
-      // ---- q_t . n_prev, half of the dims per thread
-      float den = 0.f;
-#pragma unroll 1
-      for (int i = 0; i < 8; ++i) {
-        const int c8 = half * 8 + i;
-        if (c8 * 8 >= D) break;
-        float f[8];
-        ml_unpack8(*reinterpret_cast<const uint4*>(smem + L::OFF_Q + ml_swz(r, c8)), f);
-        const float4 n0 = *reinterpret_cast<const float4*>(sn + c8 * 8), n1 = *reinterpret_cast<const float4*>(sn + c8 * 8 + 4);
-        den += f[0] * n0.x + f[1] * n0.y + f[2] * n0.z + f[3] * n0.w + f[4] * n1.x + f[5] * n1.y + f[6] * n1.z + f[7] * n1.w;
+    if (issuer) {
+      if (elect_one()) {
+        tc_fence_after();
+        constexpr uint32_t id_qk = make_idesc_bf16(128, 128, false, false);
+        constexpr uint32_t id_xv = make_idesc_bf16(128, EP, false, true);
+        auto kstep = [](int k) { return (uint32_t)(((k / 4) * 16384 + (k % 4) * 32) >> 4); };
+        const uint64_t q = make_smem_desc(smem_u32(smem + L::OFF_Q), 16, 1024), k = make_smem_desc(smem_u32(smem + L::OFF_K), 16, 1024);
+        const uint64_t sh = make_smem_desc(smem_u32(smem + L::OFF_SH), 16384, 1024);
+        const uint64_t sl = make_smem_desc(smem_u32(smem + L::OFF_SL), 16384, 1024);
+        for (int i = 0; i < ksteps; ++i) umma_f16_ss(tmem, q + kstep(i), k + kstep(i), id_qk, i ? 1u : 0u);
+        umma_commit(bar_a);
+        mbar_expect_tx(bar_g, (uint32_t)((E + 63) / 64) * 16384u);
+        for (int i = 0; i < (E + 63) / 64; ++i)
+          tma_load_2d(smem + L::OFF_KL + i * 16384, &tm_proj, bar_g, 2 * p.heads * D + p.heads * E + h * E + i * 64, row0 + t0);
+        for (int i = 0; i < ksteps; ++i) umma_f16_ss(tmem + 128, q + kstep(i), sh + (uint32_t)(i * 128), id_xv, i ? 1u : 0u);
+        for (int i = 0; i < ksteps; ++i) umma_f16_ss(tmem + 128, q + kstep(i), sl + (uint32_t)(i * 128), id_xv, 1u);
       }
-      den *= c_r;
-      // ---- scores -> weighted, causal, split; back to tensor memory as the A operand of P V, each half over its own columns
-      if (!mbar_wait(bar_a, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
-      tc_fence_after();
-      uint32_t s0[32], s1[32];
-      tmem_ld_32x32(tm_a + half * 64, s0);
-      tmem_ld_32x32(tm_a + half * 64 + 32, s1);
-      tmem_ld_wait();
-      auto weigh = [&](const uint32_t (&s)[32], int c) __attribute__((always_inline)) {
-        uint32_t hi[16], lo[16];
-        const int k0 = half * 64 + c * 32;
+      __syncwarp();
+    }
+    if (!last) {                                      // the gates of the next chunk
+      log_gates(t0 + ML_CHUNK, b ^ 1);
+      request_gates(t0 + 2 * ML_CHUNK);
+    }
+    const float M_end = M_b[127], M_r = M_b[r];
+    const float c_r = ml_exp2(sprev[b] - M_r);        // how much of the earlier state row r still sees
+    // ---- q_t . n_prev, a quarter of the dims per thread
+    float den = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c8 = cg * 4 + i;
+      if (c8 * 8 >= D) break;
+      float f[8];
+      ml_unpack8(*reinterpret_cast<const uint4*>(smem + L::OFF_Q + ml_swz(r, c8)), f);
+      const float4 n0 = *reinterpret_cast<const float4*>(sn + c8 * 8), n1 = *reinterpret_cast<const float4*>(sn + c8 * 8 + 4);
+      den += (f[0] * n0.x + f[1] * n0.y) + (f[2] * n0.z + f[3] * n0.w) + (f[4] * n1.x + f[5] * n1.y) + (f[6] * n1.z + f[7] * n1.w);
+    }
+    den *= c_r;
+    // ---- scores -> weighted, causal, split; back to tensor memory as the A operand of P V, each group over its own columns
+    if (!mbar_wait(bar_a, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
+    tc_fence_after();
+    {
+      uint32_t hi[16], lo[16];
+      if (cg > quarter) {                             // every key lies behind every row
+#pragma unroll
+        for (int i = 0; i < 16; ++i) hi[i] = lo[i] = 0u;
+      } else {
+        uint32_t s[32];
+        tmem_ld_32x32(tm_a, s);
+        tmem_ld_wait();
+        const bool edge = cg == quarter;
+        float den1 = 0.f;
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float2 av = *reinterpret_cast<const float2*>(a_b + k0 + 2 * i);
-          const float x = k0 + 2 * i <= r ? __uint_as_float(s[2 * i]) * ml_exp(av.x - M_r) : 0.f;
-          const float y = k0 + 2 * i + 1 <= r ? __uint_as_float(s[2 * i + 1]) * ml_exp(av.y - M_r) : 0.f;
-          den += x + y;
-          hi[i] = pack_bf16x2(x, y);
-          const float2 back = unpack_bf16x2(hi[i]);
-          lo[i] = pack_bf16x2(x - back.x, y - back.y);
-        }
-        tmem_st_32x16(tm_a + half * 64 + c * 16, hi);
-        tmem_st_32x16(tm_a + half * 64 + 32 + c * 16, lo);
-      };
-      weigh(s0, 0);
-      weigh(s1, 1);
-      sden[half * 128 + r] = den;
-      tmem_st_wait();
-      tc_fence_before();
-    }
-    __syncthreads();
-    if (!worker && elect_one()) {
-      tc_fence_after();
-      constexpr uint32_t id_xv = make_idesc_bf16(128, EP, false, true);
-      const uint64_t v = make_smem_desc(smem_u32(smem + L::OFF_V), 16384, 1024);
-#pragma unroll
-      for (int part = 0; part < 2; ++part)             // O_intra = P V
-#pragma unroll
-        for (int k = 0; k < 8; ++k)
-          umma_f16_ts(tmem + 256, tmem + (k / 4) * 64 + part * 32 + (k % 4) * 8, v + (uint32_t)(k * 128), id_xv, (part | k) ? 1u : 0u);
-      umma_commit(bar_o);
-    }
-    __syncwarp();
-    // ---- K~: weighted rows, split in place (hi) and beside (lo); their column sums for n
-    if (worker) {
-      float col[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      if (k_t < k_step) {
-#pragma unroll 4
-        for (int t = k_t; t < ML_CHUNK; t += k_step) {
-          const float w = ml_exp(a_b[t] - M_end);
-          const uint32_t at = ml_swz(t, k_c8);
-          float f[8];
-          ml_unpack8(*reinterpret_cast<const uint4*>(smem + L::OFF_K + at), f);
-#pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            f[i] = t < n ? f[i] * w : 0.f;
-            col[i] += f[i];
+          const float2 av = *reinterpret_cast<const float2*>(a_b + cg * 32 + 2 * i);
+          float x = __uint_as_float(s[2 * i]) * ml_exp2(av.x - M_r), y = __uint_as_float(s[2 * i + 1]) * ml_exp2(av.y - M_r);
+          if (edge) {
+            x = 2 * i <= lane ? x : 0.f;
+            y = 2 * i + 1 <= lane ? y : 0.f;
           }
-          uint4 hi, lo;
-          ml_split8(f, hi, lo);
-          *reinterpret_cast<uint4*>(smem + L::OFF_K + at) = hi;
-          *reinterpret_cast<uint4*>(smem + L::OFF_KL + at) = lo;
+          den += x;
+          den1 += y;
+          ml_split2(x, y, hi[i], lo[i]);
         }
-        *reinterpret_cast<float4*>(scol + k_t * D + k_c8 * 8) = make_float4(col[0], col[1], col[2], col[3]);
-        *reinterpret_cast<float4*>(scol + k_t * D + k_c8 * 8 + 4) = make_float4(col[4], col[5], col[6], col[7]);
+        den += den1;
       }
+      tmem_st_32x16(tm_a, hi);
+      tmem_st_32x16(tm_a + 16, lo);
+    }
+    sden[cg * 128 + r] = den;
+    if (!mbar_wait(bar_g, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
+    uint4 gate[HE / 8];
+#pragma unroll
+    for (int q = 0; q < HE / 8; ++q) gate[q] = *reinterpret_cast<const uint4*>(smem + L::OFF_KL + ml_swz(r, e0 / 8 + q));
+    tmem_st_wait();
+    tc_fence_before();
+    __syncthreads();
+    if (issuer) {
+      if (elect_one()) {
+        tc_fence_after();
+        constexpr uint32_t id_xv = make_idesc_bf16(128, EP, false, true);
+        const uint64_t v = make_smem_desc(smem_u32(smem + L::OFF_V), 16384, 1024);
+#pragma unroll
+        for (int part = 0; part < 2; ++part)             // O_intra = P V
+#pragma unroll
+          for (int k = 0; k < 8; ++k)
+            umma_f16_ts(tmem + 256, tmem + (k / 2) * 32 + part * 16 + (k % 2) * 8, v + (uint32_t)(k * 128), id_xv, (part | k) ? 1u : 0u);
+        umma_commit(bar_o);
+      }
+      __syncwarp();
+    }
+    // ---- K~: weighted rows, split in place (hi) and beside (lo); their column sums for n
+    if (k_t < k_step) {
+      float col[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+      for (int t = k_t; t < ML_CHUNK; t += k_step) {
+        const float w = ml_exp2(a_b[t] - M_end);
+        const uint32_t at = ml_swz(t, k_c8);
+        float f[8];
+        ml_unpack8(*reinterpret_cast<const uint4*>(smem + L::OFF_K + at), f);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          f[i] = t < n ? f[i] * w : 0.f;
+          col[i] += f[i];
+        }
+        uint4 hi, lo;
+        ml_split8(f, hi, lo);
+        *reinterpret_cast<uint4*>(smem + L::OFF_K + at) = hi;
+        *reinterpret_cast<uint4*>(smem + L::OFF_KL + at) = lo;
+      }
+      *reinterpret_cast<float4*>(scol + k_t * D + k_c8 * 8) = make_float4(col[0], col[1], col[2], col[3]);
+      *reinterpret_cast<float4*>(scol + k_t * D + k_c8 * 8 + 4) = make_float4(col[4], col[5], col[6], col[7]);
     }
     fence_proxy_async_smem();
     __syncthreads();
-    if (!worker && elect_one()) {
-      tc_fence_after();
-      constexpr uint32_t id_kv = make_idesc_bf16(128, EP, true, true);
-      const uint64_t v = make_smem_desc(smem_u32(smem + L::OFF_V), 16384, 1024);
-      const uint64_t kh = make_smem_desc(smem_u32(smem + L::OFF_K), 16384, 1024), kl = make_smem_desc(smem_u32(smem + L::OFF_KL), 16384, 1024);
+    if (issuer) {
+      if (elect_one()) {
+        tc_fence_after();
+        constexpr uint32_t id_kv = make_idesc_bf16(128, EP, true, true);
+        const uint64_t v = make_smem_desc(smem_u32(smem + L::OFF_V), 16384, 1024);
+        const uint64_t kh = make_smem_desc(smem_u32(smem + L::OFF_K), 16384, 1024), kl = make_smem_desc(smem_u32(smem + L::OFF_KL), 16384, 1024);
 #pragma unroll
-      for (int part = 0; part < 2; ++part)             // S = g S_prev + K~^T V
+        for (int part = 0; part < 2; ++part)             // S = g S_prev + K~^T V
 #pragma unroll
-        for (int k = 0; k < 8; ++k)
-          umma_f16_ss(tmem + 384, (part ? kl : kh) + (uint32_t)(k * 128), v + (uint32_t)(k * 128), id_kv, 1u);
-      umma_commit(bar_s);
-    }
-    __syncwarp();
-    if (!worker) {
-      if (!last) {                                      // every MMA of this chunk is done: its operands can be replaced
-        if (!mbar_wait(bar_s, ph, abort_word)) *abort_word = ERR_WAIT_MISC;
-        if (elect_one()) load_chunk(t0 + ML_CHUNK);
+          for (int k = 0; k < 8; ++k)
+            umma_f16_ss(tmem + 384, (part ? kl : kh) + (uint32_t)(k * 128), v + (uint32_t)(k * 128), id_kv, 1u);
+        umma_commit(bar_s);
       }
       __syncwarp();
-      continue;
+      if (!last) scan_gates(b ^ 1, sm[b * 128 + 127]);
     }
-    // ---- n, and the gates of the next chunk
-    if (warp == 0 && !last) scan_gates(t0 + ML_CHUNK, b ^ 1, sm[b * 128 + 127]);
-    if (tid >= 128 && tid - 128 < D) {
-      const int d = tid - 128;
-      float s = ml_exp(sprev[b] - M_end) * sn[d];
-      for (int i = 0; i < k_step; ++i) s += scol[i * D + d];
-      sn[d] = s;
-      if (last && ok) state_n[d] = s;
+    // ---- n
+    if (tid < D) {
+      float s = ml_exp2(sprev[b] - M_end) * sn[tid], s1 = 0.f;
+      int i = 0;
+      for (; i + 1 < k_step; i += 2) {
+        s += scol[i * D + tid];
+        s1 += scol[(i + 1) * D + tid];
+      }
+      if (i < k_step) s += scol[i * D + tid];
+      s += s1;
+      sn[tid] = s;
+      if (last && ok) state_n[tid] = s;
     }
     if (last && tid == 0 && ok) state_n[D] = sm[b * 128 + 127];
-    // ---- outputs of this thread's row and half: both parts, the normaliser, the sum of squares
+    // ---- outputs of this thread's row and columns: both parts, the normaliser, the sum of squares
     if (!mbar_wait(bar_o, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
     tc_fence_after();
     float o[HE];
-    float ss = 0.f;
     {
-      const float den = fabsf((sden[r] + sden[128 + r]) * qscale);
-      const float low = qscale / (fmaxf(den, expf(-sm[b * 128 + r])) + 1e-6f), ci = c_r * low;
-#pragma unroll
-      for (int c = 0; c < HE / 32; ++c) {
-        uint32_t x[32], y[32];
-        tmem_ld_32x32(tm_i + half * HE + c * 32, x);
-        tmem_ld_32x32(tm_o + half * HE + c * 32, y);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          const float v = __uint_as_float(x[i]) * ci + __uint_as_float(y[i]) * low;
-          o[c * 32 + i] = v;
-          if (half * HE + c * 32 + i < E) ss = fmaf(v, v, ss);
-        }
-      }
-    }
-    srms[half * 128 + r] = ss;
-    ml_barrier();                                       // also: the next chunk's gates are there
-    const float inv = rsqrtf((srms[r] + srms[128 + r]) / (float)E + p.eps);
-    // ---- state: keep it for the next chunk, or leave it in the slot after the last one
-    if (!mbar_wait(bar_s, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
-    tc_fence_after();
-    const float g_next = last ? 1.f : ml_exp(sprev[b ^ 1] - sM[(b ^ 1) * 128 + 127]);
-#pragma unroll 1
-    for (int c = 0; c < HE / 32; ++c) {
-      uint32_t raw[32];
-      tmem_ld_32x32(tm_s + half * HE + c * 32, raw);
+      const float d4 = fabsf(((sden[r] + sden[128 + r]) + (sden[256 + r] + sden[384 + r])) * qscale);
+      const float low = qscale / (fmaxf(d4, expf(-sm[b * 128 + r])) + 1e-6f), ci = c_r * low;
+      uint32_t x[HE], y[HE];
+      ml_tmem_ld<HE>(tm_i, x);
+      ml_tmem_ld<HE>(tm_o, y);
       tmem_ld_wait();
-      if (last) {
-        if (r < D && ok) {
+      float ss = 0.f;
 #pragma unroll
-          for (int q = 0; q < 8; ++q)
-            if (half * HE + c * 32 + q * 4 < E)          // vdim is a multiple of 8
-              *reinterpret_cast<float4*>(state + (long long)r * E + half * HE + c * 32 + q * 4) =
-                  make_float4(__uint_as_float(raw[q * 4]), __uint_as_float(raw[q * 4 + 1]), __uint_as_float(raw[q * 4 + 2]),
-                              __uint_as_float(raw[q * 4 + 3]));
-        }
-      } else {
-        float s[32];
-#pragma unroll
-        for (int i = 0; i < 32; ++i) s[i] = __uint_as_float(raw[i]);
-        publish_state(s, c, g_next);
+      for (int i = 0; i < HE; ++i) {
+        o[i] = fmaf(__uint_as_float(x[i]), ci, __uint_as_float(y[i]) * low);
+        if (e0 + i < E) ss = fmaf(o[i], o[i], ss);
       }
-    }
-    tmem_st_wait();
-    // ---- rows -> columns through shared memory (K~ lo is free now), one half of the columns after the other, so that the gate
-    // and y move in whole pieces of rows
-    constexpr int PIECES = HE / 4;                      // 16-byte pieces of half an fp32 row
-    const __nv_bfloat16* wr = reinterpret_cast<const __nv_bfloat16*>(p.weight) + h * E;
-#pragma unroll
-    for (int x = 0; x < 2; ++x) {
-      if (half == x) {
-        float4* stage = reinterpret_cast<float4*>(smem + L::OFF_KL) + r * PIECES;
-#pragma unroll
-        for (int q = 0; q < PIECES; ++q)
-          stage[q ^ (r & (PIECES - 1))] = make_float4(o[q * 4] * inv, o[q * 4 + 1] * inv, o[q * 4 + 2] * inv, o[q * 4 + 3] * inv);
-      }
-      ml_barrier();
-      const int c = x * HE + o_c8 * 8;
-      if (c < E) {
-        float w[8];
-        ml_unpack8(*reinterpret_cast<const uint4*>(wr + c), w);
-#pragma unroll
-        for (int j = 0; j < O_N; ++j) {
-          const int t = o_t + j * O_STEP;
-          if (t >= n) continue;
-          const float4* from = reinterpret_cast<const float4*>(smem + L::OFF_KL) + t * PIECES;
-          const int sx = t & (PIECES - 1);
-          const float4 y0 = from[(2 * o_c8) ^ sx], y1 = from[(2 * o_c8 + 1) ^ sx];
-          float g[8];
-          ml_unpack8(gate[x][j], g);
-#pragma unroll
-          for (int i = 0; i < 8; ++i) g[i] = w[i] * __fdividef(1.f, 1.f + __expf(-g[i]));
-          *reinterpret_cast<uint4*>(gy + (long long)(t0 + t) * p.ld_y + c) =
-              make_uint4(pack_bf16x2(y0.x * g[0], y0.y * g[1]), pack_bf16x2(y0.z * g[2], y0.w * g[3]),
-                         pack_bf16x2(y1.x * g[4], y1.y * g[5]), pack_bf16x2(y1.z * g[6], y1.w * g[7]));
-        }
-      }
-      ml_barrier();
+      srms[cg * 128 + r] = ss;
     }
     tc_fence_before();
+    __syncthreads();
+    // ---- state and outputs once the last product is done
+    if (!mbar_wait(bar_s, ph, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
+    tc_fence_after();
+    if (issuer && !last) {                              // every MMA of this chunk is done: its operands can be replaced
+      if (elect_one()) load_chunk(t0 + ML_CHUNK);
+      __syncwarp();
+    }
+    {
+      const float inv = rsqrtf(((srms[r] + srms[128 + r]) + (srms[256 + r] + srms[384 + r])) / (float)E + p.eps);
+#pragma unroll
+      for (int q = 0; q < HE / 8; ++q) {
+        float g[8];
+        ml_unpack8(gate[q], g);
+        const float4 w0 = *reinterpret_cast<const float4*>(sw + e0 + q * 8), w1 = *reinterpret_cast<const float4*>(sw + e0 + q * 8 + 4);
+        const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+        for (int i = 0; i < 8; ++i) g[i] = o[q * 8 + i] * (inv * w[i]) * ml_sigmoid(g[i]);
+        *reinterpret_cast<uint4*>(smem + L::OFF_KL + ml_swz(r, e0 / 8 + q)) =
+            make_uint4(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]), pack_bf16x2(g[4], g[5]), pack_bf16x2(g[6], g[7]));
+      }
+    }
+    // ---- state: keep it for the next chunk, or leave it in the slot after the last one
+    uint32_t raw[HE];
+    ml_tmem_ld<HE>(tm_s, raw);
+    tmem_ld_wait();
+    if (last) {
+      if (r < D && ok) {
+#pragma unroll
+        for (int q = 0; q < HE / 4; ++q)
+          if (e0 + q * 4 < E)                            // vdim is a multiple of 8
+            *reinterpret_cast<float4*>(state + (long long)r * E + e0 + q * 4) =
+                make_float4(__uint_as_float(raw[q * 4]), __uint_as_float(raw[q * 4 + 1]), __uint_as_float(raw[q * 4 + 2]),
+                            __uint_as_float(raw[q * 4 + 3]));
+      }
+    } else {
+      float s[HE];
+#pragma unroll
+      for (int i = 0; i < HE; ++i) s[i] = __uint_as_float(raw[i]);
+      publish_state(s, ml_exp2(sprev[b ^ 1] - sM[(b ^ 1) * 128 + 127]));
+      tmem_st_wait();
+    }
+    __syncthreads();
+    for (int i = tid; i < n * (EP / 8); i += ML_THREADS) {
+      const int t = i / (EP / 8), c8 = i % (EP / 8);
+      if (c8 * 8 < E)
+        *reinterpret_cast<uint4*>(gy + (long long)(t0 + t) * p.ld_y + c8 * 8) = *reinterpret_cast<const uint4*>(smem + L::OFF_KL + ml_swz(t, c8));
+    }
   }
   if (!live) {
-    for (int t = tid / 32; t < rows; t += ML_THREADS / 32)
+    for (int t = warp; t < rows; t += ML_THREADS / 32)
       for (int c = lane * 8; c < E; c += 256) *reinterpret_cast<uint4*>(gy + (long long)t * p.ld_y + c) = make_uint4(0, 0, 0, 0);
   }
   tc_fence_before();
@@ -710,20 +737,21 @@ using namespace b200;
 
 // See MlstmParams.  f32 != 0: activations are fp32, else bf16.  chunked != 0: the tensor-core kernel (bf16, cu given, dim and vdim
 // multiples of 8 up to 128).
-extern "C" int b200_mlstm(const void* proj, long long ld_proj, const float* gates, long long ld_gates, const float* gate_bias,
-                          const void* weight, void* y, long long ld_y, float* state, const int* state_slots, const int* cu,
+extern "C" int b200_mlstm(const void* proj, long long ld_proj, const float* gates, long long ld_gates, const void* h, long long ld_h,
+                          const void* w_gates, long long ld_wg, int width, const float* gate_bias, const void* weight, void* y, long long ld_y, float* state, const int* state_slots, const int* cu,
                           const int* positions, int seqs, int rows, int heads, int dim, int vdim, int stride, int num_slots,
                           float cap, float eps, int f32, int chunked, uint32_t* status, cudaStream_t st) {
   if (seqs <= 0 || rows <= 0) return 0;
   if (heads <= 0 || dim <= 0 || vdim <= 0 || heads > 65535 || stride < dim * vdim + dim + 1 || stride % 4 || !(cap > 0.f)) return -10;
   MlstmParams p;
-  p.proj = proj; p.ld_proj = ld_proj; p.gates = gates; p.ld_gates = ld_gates; p.gate_bias = gate_bias; p.weight = weight;
+  p.proj = proj; p.ld_proj = ld_proj; p.gates = gates; p.ld_gates = ld_gates; p.h = h; p.ld_h = ld_h; p.w_gates = w_gates;
+  p.ld_wg = ld_wg; p.width = width; p.gate_bias = gate_bias; p.weight = weight;
   p.y = y; p.ld_y = ld_y; p.state = state; p.state_slots = state_slots; p.cu = cu; p.positions = positions; p.seqs = seqs;
   p.rows = rows; p.heads = heads; p.dim = dim; p.vdim = vdim; p.stride = stride; p.num_slots = num_slots; p.cap = cap;
   p.eps = eps; p.status = status;
   const uintptr_t ptrs = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(state);
   if (chunked) {
-    if (f32 || cu == nullptr || dim > 128 || vdim > 128 || dim % 8 || vdim % 8) return -11;
+    if (f32 || cu == nullptr || gates == nullptr || dim > 128 || vdim > 128 || dim % 8 || vdim % 8) return -11;
     if (ld_proj % 8 || ld_y % 8 || (ptrs | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(weight)) & 15) return -11;
     CUtensorMap tm;
     if (make_tmap_bf16_2d(&tm, proj, (uint64_t)rows, (uint64_t)2 * heads * (dim + vdim), (uint64_t)ld_proj, 64, ML_CHUNK)) return -20;
@@ -734,7 +762,11 @@ extern "C" int b200_mlstm(const void* proj, long long ld_proj, const float* gate
   const int rg = groups < 256 ? 256 / groups : 1;
   const size_t smem = (2ull * dim + (size_t)rg * vdim) * sizeof(float);
   if (smem > 48 * 1024) return -12;
-  if (vec && cu == nullptr && groups <= 256 && (dim + rg - 1) / rg <= 16 && (dim & 1) == 0) {
+  const bool step = vec && cu == nullptr && groups <= 256 && (dim + rg - 1) / rg <= 16 && (dim & 1) == 0;
+  if (gates == nullptr && (!step || h == nullptr || w_gates == nullptr || width <= 0 || ld_h % 4 || ld_wg % 4 ||
+                           (reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(w_gates)) & 15))
+    return -13;
+  if (step) {
     const unsigned blocks = (unsigned)((long long)seqs * heads);
     const bool small = (dim + rg - 1) / rg <= 4;
     if (f32) {

@@ -177,6 +177,7 @@ class MatrixMemory:
         self.norm = w("norm", heads * vdim).to(device=device, dtype=dtype).contiguous()
         self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
         self.chunked = torch.device(device).type == "cuda" and mo.mlstm_chunkable(dtype, dim, vdim)
+        self.one_pass = mo.mlstm_steps(dim, vdim)          # a decode step takes the gates' products itself
 
     def cache_spec(self):
         return StateSpec((self.heads, mo.mlstm_state(self.dim, self.vdim)))
@@ -184,11 +185,12 @@ class MatrixMemory:
     def __call__(self, h, x, batch, state):
         n = batch.n_single
         proj = mo.linear(h, self.w_in)
-        gates = mo.linear(h, self.w_gates, out_dtype=torch.float32)          # the recurrence takes them in 32-bit
         y = mo.rows_buffer(h.shape[0], self.heads * self.vdim, h.dtype, h.device)
 
         def run(rows, seqs, cu, spans, chunked):
-            mo.mlstm(proj[rows], gates[rows], self.b_gates, self.norm, state, batch.state_slots[seqs], cu, spans,
+            # the recurrence takes the gates in 32-bit
+            gates = (h[rows], self.w_gates) if cu is None and self.one_pass else mo.linear(h[rows], self.w_gates, out_dtype=torch.float32)
+            mo.mlstm(proj[rows], gates, self.b_gates, self.norm, state, batch.state_slots[seqs], cu, spans,
                      batch.positions[rows], self.heads, self.dim, self.vdim, self.cap, self.eps, y[rows], chunked)
         if n:
             run(slice(0, n), slice(0, n), None, [(i, i + 1) for i in range(n)] if not h.is_cuda else None, False)

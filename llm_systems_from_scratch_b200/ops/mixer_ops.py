@@ -43,7 +43,7 @@ def _lib():
             "b200_grouped_rows": [P, P, P, L, P, L, P, I, P, P, P, P, I, I, I, I, I, P, I, P, P],
             "b200_grouped_decode": [P, P, P, L, P, L, P, I, P, P, P, P, P, I, I, I, I, I, P, P, P],
             "b200_grouped_prefill": [P, P, P, L, P, L, P, I, P, P, P, I, I, I, I, I, I, P, P, P],
-            "b200_mlstm": [P, L, P, L, P, P, P, L, P, P, P, P, I, I, I, I, I, I, I, F, F, I, I, P, P],
+            "b200_mlstm": [P, L, P, L, P, L, P, L, I, P, P, P, L, P, P, P, P, I, I, I, I, I, I, I, F, F, I, I, P, P],
             "b200_retention_recurrent": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
         }.items():
             fn = getattr(lib, name)
@@ -445,24 +445,40 @@ def mlstm_chunkable(dtype, dim: int, vdim: int) -> bool:
     return dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and vdim <= 128
 
 
+def mlstm_steps(dim: int, vdim: int) -> bool:
+    """Whether a decode step of these sizes runs on the one-pass kernel, which also takes the gates' products itself."""
+    groups = vdim // 4
+    return vdim % 4 == 0 and dim % 2 == 0 and 0 < groups <= 256 and -(-dim // max(1, 256 // groups)) <= 16
+
+
 def mlstm(proj, gates, gate_bias, weight, state, state_slots, cu, spans, positions, heads: int, dim: int, vdim: int, cap: float,
           eps: float, y, chunked: bool = False):
     """Matrix memory over the rows of ``proj`` (q | k | v | output gate) with the gates' pre-activations ``gates`` (input | forget,
-    fp32, without bias).  ``cu`` (sequences + 1, int32) delimits the sequences, None = one row each; ``spans`` says the same on
+    fp32, without bias; or, for a decode step of ``mlstm_steps`` sizes, the pair (input rows h, the gates' weights)).  ``cu`` (sequences + 1, int32) delimits the sequences, None = one row each; ``spans`` says the same on
     the host.  The states are read and left in their slots; y (R, heads * vdim) receives the normed, weighted, gated heads.
     ``chunked``: the tensor-core kernel for portions of prompts (``mlstm_chunkable`` sizes)."""
+    h = w_gates = None
+    if isinstance(gates, tuple):
+        h, w_gates = gates
+        gates = None if proj.is_cuda else h.float() @ w_gates.float().t()
     if not proj.is_cuda:
         return mixer_torch.mlstm(proj, gates, gate_bias, weight, state, state_slots, spans, positions, heads, dim, vdim, cap, eps, y)
     seqs = state_slots.numel()
     _req(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, mlstm_state(dim, vdim)), "bad state")
     _req(state_slots.dtype == torch.int32 and positions.dtype == torch.int32 and gate_bias.dtype == torch.float32
-         and gate_bias.numel() == 2 * heads and gates.dtype == torch.float32 and gates.shape == (proj.shape[0], 2 * heads), "bad inputs")
+         and gate_bias.numel() == 2 * heads, "bad inputs")
+    if gates is None:
+        _req(h.dtype == proj.dtype and w_gates.dtype == proj.dtype and h.shape[0] == proj.shape[0] and h.stride(1) == 1
+             and w_gates.shape == (2 * heads, h.shape[1]) and cu is None and mlstm_steps(dim, vdim), "bad inputs of the gates")
+    else:
+        _req(gates.dtype == torch.float32 and gates.shape == (proj.shape[0], 2 * heads), "bad gates")
     _req(proj.shape[1] == 2 * heads * (dim + vdim) and y.shape == (proj.shape[0], heads * vdim) and y.dtype == proj.dtype
          and weight.dtype == proj.dtype and weight.numel() == heads * vdim, "bad shapes")
     _req(cu is None or (cu.dtype == torch.int32 and cu.numel() == seqs + 1), "bad row offsets")
     _req(not chunked or (mlstm_chunkable(proj.dtype, dim, vdim) and cu is not None), "sizes the chunked kernel does not take")
     _check(_lib().b200_mlstm(
-        _ptr(proj), proj.stride(0), _ptr(gates), gates.stride(0), _ptr(gate_bias), _ptr(weight), _ptr(y), y.stride(0), _ptr(state),
+        _ptr(proj), proj.stride(0), _ptr(gates), 0 if gates is None else gates.stride(0), _ptr(h), 0 if h is None else h.stride(0),
+        _ptr(w_gates), 0 if h is None else w_gates.stride(0), 0 if h is None else h.shape[1], _ptr(gate_bias), _ptr(weight), _ptr(y), y.stride(0), _ptr(state),
         _ptr(state_slots), _ptr(cu), _ptr(positions), seqs, proj.shape[0], heads, dim, vdim, state.shape[2], state.shape[0],
         float(cap), float(eps), _f32(proj), int(chunked), _ptr(native.status_word(proj.device)), _stream()),
         "mlstm_chunk" if chunked else "mlstm")

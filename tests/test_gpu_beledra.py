@@ -87,7 +87,8 @@ def rotary(n, base, dims, scaling=None):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("heads,kv,maps,dim,vdim,rot", [(4, 2, 1, 11, 9, 0), (6, 3, 2, 40, 24, 16), (2, 2, 2, 128, 72, 128), (5, 1, 1, 200, 130, 6)])
+@pytest.mark.parametrize("heads,kv,maps,dim,vdim,rot", [(4, 2, 1, 11, 9, 0), (6, 3, 2, 40, 24, 16), (2, 2, 2, 128, 72, 128), (5, 1, 1, 200, 130, 6),
+                                                            (3, 3, 1, 200, 136, 112), (40, 8, 2, 24, 40, 16), (9, 3, 1, 64, 8, 0)])
 def test_prepare_norms_rotates_and_appends(dtype, heads, kv, maps, dim, vdim, rot):
     """Every row at its own position; padding rows and other slots stay untouched."""
     mo = mops()
@@ -318,6 +319,15 @@ def test_memory_token_by_token_and_in_portions(heads, dim, vdim, cap, dtype):
         for i in (2, 5):
             close(state[len(lens) - i, :, :dim * vdim + dim + 1], finals[0][len(lens) - i - 1], 2e-4)
     close(finals[-1], finals[0], 2e-4)
+    if mo.mlstm_steps(dim, vdim):                        # a step that takes the gates' products itself
+        w = mo.padded_weight(randn(2 * heads, 77, seed=93, dtype=dtype, scale=0.2), dtype, "cuda")
+        hin, ys = padded(randn(2, 77, seed=94, dtype=dtype)), []
+        for gt in ((hin, w), hin.float() @ w.float().t()):
+            st = torch.zeros(2, heads, mo.mlstm_state(dim, vdim), device="cuda")
+            st[..., :dim * vdim + dim + 1] = finals[0][:2]
+            ys.append(mo.rows_buffer(2, heads * vdim, dtype, "cuda"))
+            mo.mlstm(padded(proj[2][:2]), gt, bias, weight, st, dev([1, 0]), None, None, dev([9, 9]), heads, dim, vdim, cap, 1e-4, ys[-1])
+        close(ys[0], ys[1], 1e-2 if dtype == BF else 1e-4)
     idle = torch.zeros(2, heads, mo.mlstm_state(dim, vdim), device="cuda")
     y = torch.ones(1, heads * vdim, dtype=dtype, device="cuda")
     mo.mlstm(padded(proj[0]), padded(gates[0]), bias, weight, idle, dev([-1]), None, None, dev([0]), heads, dim, vdim, cap, 1e-4, y)
