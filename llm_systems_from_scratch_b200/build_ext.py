@@ -5,8 +5,9 @@ ctypes, so no PyTorch headers are needed and a full rebuild takes seconds.  The 
 object is written next to this file (``_b200_kernels.so``): it is git-ignored but
 travels with the source tree to the GPU machine.
 
-``build_serving`` compiles only what serving needs (without the backward kernels) into ``_b200_serving.so``, for a
-fresh checkout whose first command serves a model; objects are shared, so a full build later compiles the rest.
+``build_serving`` compiles only what serving one kind of model needs (no backward kernels, no other model's mixers) into
+``_b200_serving.so``, for a fresh checkout whose first command serves a model; objects are shared, so a full build later
+compiles the rest.
 
 Usage:  python -m llm_systems_from_scratch_b200.build_ext [--force] [--verbose]
 """
@@ -26,6 +27,9 @@ BUILD_DIR = PKG_DIR / "csrc" / "build"
 LIB_PATH = PKG_DIR / "_b200_kernels.so"
 SERVING_LIB_PATH = PKG_DIR / "_b200_serving.so"
 NOT_FOR_SERVING = {"flash_attn_bwd.cu"}     # training only (comm_kernels.cu holds host code of the GEMMs)
+# kernels that belong to single mixers; a model class names those it uses (KERNELS)
+MIXERS = {"flash_attn_fwd.cu", "latent_attention.cu", "latent_decode_tc.cu", "retention.cu", "grouped_attention.cu",
+          "grouped_prefill.cu", "mlstm.cu"}
 HOST_SRC = CSRC / "host" / "host_runtime.cpp"
 HOST_LIB_PATH = PKG_DIR / "_b200_host.so"
 
@@ -133,12 +137,14 @@ def build(force: bool = False, verbose: bool = False) -> Path:
     return LIB_PATH
 
 
-def build_serving() -> Path:
-    """The library a serving command loads: the full one if it has been built, else the serving kernels alone."""
+def build_serving(mixers=None) -> Path:
+    """The library a serving command loads: the full one if it has been built, else the serving kernels alone, those of
+    ``mixers`` (source names out of ``MIXERS``; None: all) among them."""
     build_host()
     if LIB_PATH.exists():
         return LIB_PATH
-    srcs = [s for s in sources() if s.name not in NOT_FOR_SERVING]
+    left_out = NOT_FOR_SERVING | (set() if mixers is None else MIXERS - set(mixers))
+    srcs = [s for s in sources() if s.name not in left_out]
     stamp, digest = BUILD_DIR / "serving_stamp.txt", _digest(srcs + headers())
     if not (SERVING_LIB_PATH.exists() and stamp.exists() and stamp.read_text() == digest):
         _compile_and_link(srcs, SERVING_LIB_PATH)

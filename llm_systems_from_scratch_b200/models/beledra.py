@@ -106,6 +106,8 @@ class Layer:
 
 
 class Beledra(LayeredModel):
+    KERNELS = ("grouped_attention.cu", "grouped_prefill.cu", "mlstm.cu")
+
     def __init__(self, config: dict, tensors, dtype=torch.bfloat16, device="cuda"):
         """``tensors[name]`` gives a tensor in its stored layout (a dict or a ``SafetensorsFile``)."""
         super().__init__(dtype, device)

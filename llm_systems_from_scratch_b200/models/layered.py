@@ -28,6 +28,7 @@ def need(d: dict, keys, where: str):
 
 class LayeredModel:
     GPU_DTYPES = (torch.bfloat16, torch.float32)
+    KERNELS = None                    # CUDA sources of its mixers (build_ext.MIXERS); None: all of them
     DEFAULT_CONTEXT = 4096            # positions an engine serves unless it is told otherwise; the designs have no limit
 
     def __init__(self, dtype, device):

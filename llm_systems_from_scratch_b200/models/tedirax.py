@@ -99,6 +99,8 @@ class Layer:
 
 
 class Tedirax(LayeredModel):
+    KERNELS = ("flash_attn_fwd.cu", "latent_attention.cu", "latent_decode_tc.cu", "retention.cu")
+
     def __init__(self, config: dict, tensors, dtype=torch.bfloat16, device="cuda"):
         """``tensors[name]`` gives a tensor in its stored layout (a dict or a ``SafetensorsFile``)."""
         super().__init__(dtype, device)

@@ -46,7 +46,10 @@ def _lib():
             "b200_mlstm": [P, L, P, L, P, L, P, L, I, P, P, P, L, P, P, P, P, I, I, I, I, I, I, I, F, F, I, I, P, P],
             "b200_retention_recurrent": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
         }.items():
-            fn = getattr(lib, name)
+            fn = getattr(lib, name, None)
+            if fn is None:                 # a serving library holds the mixers of one model
+                _req(native.lib_path().stem == "_b200_serving", f"symbol {name} is missing from {native.lib_path()}")
+                continue
             fn.argtypes, fn.restype = args, ctypes.c_int
         _declared = True
     return lib

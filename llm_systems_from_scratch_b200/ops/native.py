@@ -34,13 +34,13 @@ def lib_path() -> Path:
     return _LIB_PATH
 
 
-def load_serving():
+def load_serving(mixers=None):
     """Load the library for serving: the full one if it is there, else one of the serving kernels alone, built if need be
-    (``build_ext.build_serving``).  Training then needs a process of its own."""
+    (``build_ext.build_serving``).  Training, and models with other mixers, then need a process of their own."""
     global _LIB_PATH
     if _LIB is None:
         from ..build_ext import build_serving
-        _LIB_PATH = build_serving()
+        _LIB_PATH = build_serving(mixers)
     return load()
 
 

@@ -69,11 +69,12 @@ def main(argv=None) -> int:
     if not torch.cuda.is_available():
         raise RuntimeError("trace_run needs a CUDA device")
     from ..models.registry import model_class, read_config
-    if args.dtype == "float32" and torch.float32 not in getattr(model_class(read_config(args.model)), "GPU_DTYPES", ()):
+    cls = model_class(read_config(args.model))
+    if args.dtype == "float32" and torch.float32 not in getattr(cls, "GPU_DTYPES", ()):
         print("this model is served in bfloat16 only", file=sys.stderr)
         return 3
     from ..ops import native
-    native.load_serving()
+    native.load_serving(getattr(cls, "KERNELS", None))
     engine = open_engine(args.model, getattr(torch, args.dtype), args.max_tokens)
     replay(engine, sys.stdin, args.out)
     return 0

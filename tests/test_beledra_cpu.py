@@ -255,3 +255,17 @@ def test_generate_and_serve_commands(tmp_path, capsys):
     serve.main(["--config", str(tmp_path / "s.yaml"), "--offline"])
     rec = json.loads(capsys.readouterr().out.strip().splitlines()[-1])
     assert rec["requests"] == 5 and rec["model"] == "Beledra" and rec["output_tokens"] > 0
+
+
+def test_serving_configuration_and_kernel_sources():
+    import os
+    from llm_systems_from_scratch_b200 import build_ext
+    from llm_systems_from_scratch_b200.models.registry import MODELS
+    from llm_systems_from_scratch_b200.utils.config import load_config, validate
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    cfg = validate(load_config(os.path.join(root, "configures", "serve_beledra.yaml")), require_dataset=False)
+    layers = BeledraConfig.from_dict(cfg["model"]).layers
+    assert len(layers) == 24 and all(la.mixer.get("kv_from") in (None, i - 2) for i, la in enumerate(layers))
+    names = {s.name for s in build_ext.sources()}
+    assert build_ext.MIXERS <= names
+    assert all(set(getattr(m, "KERNELS", None) or ()) <= build_ext.MIXERS for m in MODELS.values())
