@@ -119,7 +119,8 @@ __global__ void __launch_bounds__(256) grouped_prep_kernel(const GroupedPrepPara
   }
 }
 
-// The same for sizes in whole pieces of 8 elements: LPV lanes own a vector, one piece each, in ROWS rows one after the other.
+// The same for sizes in whole pieces of 8 elements: LPV lanes own a vector, one piece each; a thread owns the same columns of UNITS
+// vectors of one row, so it loads the angles once.
 template <typename T>
 struct Piece {                    // 8 elements as they are stored
   uint4 v[sizeof(T) / 2];
@@ -147,38 +148,59 @@ __device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
   *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
 }
 
-template <typename T, int LPV, int ROWS>
+template <typename T, int LPV, int UNITS>
 __global__ void __launch_bounds__(512, 2) grouped_prep_pieces_kernel(const GroupedPrepParams p) {
   pdl_sync();
-  const int piece = threadIdx.x % LPV, c = piece * 8;
+  const int row = blockIdx.x, piece = threadIdx.x % LPV, c = piece * 8;
   const int nq = p.heads * p.maps, nk = p.wk != nullptr ? p.kv_heads * p.maps : 0, nv = p.wk != nullptr ? p.kv_heads : 0;
-  const int v = blockIdx.y * (blockDim.x / LPV) + threadIdx.x / LPV;             // this thread's vector in every row
-  const bool query = v < nq, value = v >= nq + nk, mine = v < nq + nk + nv;
-  const int row0 = blockIdx.x * ROWS, n = min(ROWS, p.rows - row0);
-  const int src_off = value ? (nq + nk) * p.dim + (v - nq - nk) * p.vdim : v * p.dim;      // the keys follow the queries
-  const int len = value ? p.vdim : p.dim;
-  const T* src = reinterpret_cast<const T*>(p.proj) + row0 * p.ld + src_off;
+  const int per = blockDim.x / LPV, v0 = blockIdx.y * per * UNITS + threadIdx.x / LPV;       // vectors v0, v0 + per, ...
+  const T* src = reinterpret_cast<const T*>(p.proj) + (long long)row * p.ld;
   const int half = p.rot / 2, shift = half / 8;
-  const bool low = c < half, turned = c < p.rot && !value;
+  const bool low = c < half, turned = c < p.rot;
   const int partner = turned ? (low ? piece + shift : piece - shift) : piece;    // lane that holds the other half of the pairs
   const uint32_t lanes = LPV == 32 ? 0xffffffffu : (((1u << (LPV & 31)) - 1u) << ((threadIdx.x & 31) / LPV * LPV));
-  Piece<T> raw[ROWS];
+  auto offset = [&](int v) { return v >= nq + nk ? (nq + nk) * p.dim + (v - nq - nk) * p.vdim : v * p.dim; };    // q | k | v
+  Piece<T> raw[UNITS];
 #pragma unroll
-  for (int i = 0; i < ROWS; ++i) {                               // all rows are requested before the first is worked on
+  for (int u = 0; u < UNITS; ++u) {                              // everything is requested before the first vector is worked on
+    const int v = v0 + u * per;
 #pragma unroll
-    for (int j = 0; j < (int)sizeof(T) / 2; ++j) raw[i].v[j] = make_uint4(0, 0, 0, 0);
-    if (i < n && mine && c < len) raw[i] = load_piece(src + i * p.ld + c);
+    for (int j = 0; j < (int)sizeof(T) / 2; ++j) raw[u].v[j] = make_uint4(0, 0, 0, 0);
+    if (v < nq + nk + nv && c < (v >= nq + nk ? p.vdim : p.dim)) raw[u] = load_piece(src + offset(v) + c);
   }
-  float w[8];
+  float cs[8], sn[8];
 #pragma unroll
-  for (int j = 0; j < 8; ++j) w[j] = 0.f;
-  if (mine && !value && c < p.dim) unpack(load_piece(reinterpret_cast<const T*>(query ? p.wq : p.wk) + c), w);
+  for (int j = 0; j < 8; ++j) cs[j] = sn[j] = 0.f;
+  if (turned) {
+    int at = p.positions[row];
+    if (at < 0 || at >= p.ctx) {
+      if (threadIdx.x == 0) report_bad_arg(p.status, 14);
+      at = 0;
+    }
+    const float* tab = p.cos_sin + (long long)at * half + (low ? c : c - half);
+    unpack(load_piece(tab), cs);
+    unpack(load_piece(tab + (long long)p.ctx * half), sn);
+    if (low) {
 #pragma unroll
-  for (int i = 0; i < ROWS; ++i) {
-    if (i >= n) break;
+      for (int j = 0; j < 8; ++j) sn[j] = -sn[j];
+    }
+  }
+  const long long slot = p.slots[row];
+  const bool keep = slot >= 0 && slot < p.num_slots;             // a padding row of the batch has no slot
+  if (nk > 0 && slot >= p.num_slots && threadIdx.x == 0) report_bad_arg(p.status, 13);
+  T* cache = reinterpret_cast<T*>(p.cache) + (keep ? slot : 0) * ((long long)p.kv_heads * (p.maps * p.kp + p.vp));
+#pragma unroll
+  for (int u = 0; u < UNITS; ++u) {
+    const int v = v0 + u * per;
+    if (v >= nq + nk + nv) break;
+    const bool query = v < nq, value = v >= nq + nk;
     float f[8];
-    unpack(raw[i], f);
+    unpack(raw[u], f);
     if (!value) {
+      float w[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) w[j] = 0.f;
+      if (c < p.dim) unpack(load_piece(reinterpret_cast<const T*>(query ? p.wq : p.wk) + c), w);
       float ss = 0.f;
 #pragma unroll
       for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
@@ -188,44 +210,24 @@ __global__ void __launch_bounds__(512, 2) grouped_prep_pieces_kernel(const Group
 #pragma unroll
       for (int j = 0; j < 8; ++j) f[j] *= r * w[j];
       if (p.rot > 0) {
-        float o[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) o[j] = __shfl_sync(lanes, f[j], partner, LPV);
-        if (turned) {
-          int at = p.positions[row0 + i];
-          if (at < 0 || at >= p.ctx) {
-            if (piece == 0) report_bad_arg(p.status, 14);
-            at = 0;
-          }
-          float cs[8], sn[8];
-          const float* tab = p.cos_sin + (long long)at * half + (low ? c : c - half);
-          unpack(load_piece(tab), cs);
-          unpack(load_piece(tab + (long long)p.ctx * half), sn);
-          const float sign = low ? -1.f : 1.f;
-#pragma unroll
-          for (int j = 0; j < 8; ++j) f[j] = fmaf(f[j], cs[j], sign * o[j] * sn[j]);
+        for (int j = 0; j < 8; ++j) {
+          const float o = __shfl_sync(lanes, f[j], partner, LPV);
+          if (turned) f[j] = fmaf(f[j], cs[j], o * sn[j]);
         }
       }
     }
-    if (!mine) continue;
     if (query) {
-      T* dst = reinterpret_cast<T*>(p.q) + ((long long)(row0 + i) * nq + v) * p.qp;
-      if (c < p.qp) store8(dst + c, f);                          // lanes past dim: zeros, the pad behind the vector
+      if (c < p.qp) store8(reinterpret_cast<T*>(p.q) + ((long long)row * nq + v) * p.qp + c, f);    // lanes past dim: zeros, the pad
       continue;
     }
-    const long long slot = p.slots[row0 + i];
-    if (slot < 0) continue;                                      // padding row of the batch
-    if (slot >= p.num_slots) {
-      if (piece == 0) report_bad_arg(p.status, 13);
-      continue;
-    }
-    T* dst = reinterpret_cast<T*>(p.cache) + slot * ((long long)p.kv_heads * (p.maps * p.kp + p.vp)) +
-             (value ? nk * p.kp + (v - nq - nk) * p.vp : (v - nq) * p.kp);
-    if (c < len) store8(dst + c, f);
+    if (!keep) continue;
+    T* dst = cache + (value ? nk * p.kp + (v - nq - nk) * p.vp : (v - nq) * p.kp);
+    if (c < (value ? p.vdim : p.dim)) store8(dst + c, f);
     if (value)
       for (int e = c + LPV * 8; e < p.vdim; e += LPV * 8) {      // values longer than a key: copied
         float g[8];
-        unpack(load_piece(src + i * p.ld + e), g);
+        unpack(load_piece(src + offset(v) + e), g);
         store8(dst + e, g);
       }
   }
@@ -233,15 +235,14 @@ __global__ void __launch_bounds__(512, 2) grouped_prep_pieces_kernel(const Group
 
 template <typename T, int LPV>
 static void launch_prep_lanes(const GroupedPrepParams& p, int vectors, cudaStream_t st) {
-  int threads = (vectors * LPV + 31) / 32 * 32;
-  if (threads > 512) {                                           // several blocks of equal size per row
-    const int blocks = (threads + 511) / 512;
-    threads = (threads / blocks + 31) / 32 * 32;
-  }
-  const int per = threads / LPV;
-  const unsigned ny = (unsigned)((vectors + per - 1) / per);
-  if (p.rows >= 148 * 16) launch_dep(grouped_prep_pieces_kernel<T, LPV, 4>, dim3((p.rows + 3) / 4, ny), threads, 0, st, p);
-  else launch_dep(grouped_prep_pieces_kernel<T, LPV, 1>, dim3(p.rows, ny), threads, 0, st, p);
+  const bool many = p.rows >= 148 * 16;                          // few rows: their vectors spread over the SMs
+  const int units = many ? 4 : 1;
+  int threads = ((vectors + units - 1) / units * LPV + 31) / 32 * 32;
+  if (threads > 512) threads = 256;
+  const int per = threads / LPV * units;
+  const dim3 grid(p.rows, (unsigned)((vectors + per - 1) / per));
+  if (many) launch_dep(grouped_prep_pieces_kernel<T, LPV, 4>, grid, threads, 0, st, p);
+  else launch_dep(grouped_prep_pieces_kernel<T, LPV, 1>, grid, threads, 0, st, p);
 }
 
 template <typename T>
