@@ -16,7 +16,9 @@
 //
 // WINDOW instances (b200_flash_window_fwd) serve portions of prompts under a sliding window: queries and keys come from
 // separate matrices, a sequence has more keys than queries (the earlier tokens its first queries can still see), tile X
-// walks only the key tiles its window touches, and the epilogue can multiply with sigmoid(gate).
+// walks only the key tiles its window touches, and the epilogue can multiply with sigmoid(gate), element by element or per head.
+// ROPE instances have one more 64-column panel of queries and keys: rotated parts, whose keys are shared by all heads and come from a
+// matrix of their own.  With heads of 128 the second stage of values makes room for them.
 #include "ptx.cuh"
 
 namespace b200 {
@@ -97,7 +99,10 @@ struct FlashFwdParams {
   // WINDOW instances only
   const int* cu_k;       // (batch+1) row offsets of the keys; queries are the last positions of their sequence's keys
   int window;            // a query sees the `window` keys up to and including its own position
-  int vdim;              // columns of a head that are written (<= DH)
+  int dim, vdim;         // columns of a head's queries and keys; columns that are written (<= DH)
+  int q_step, k_step, v_step, v_off;    // columns from head to head of queries, keys, values; first column of the values
+  int head_gate;         // gate has one column per head
+  int rot, qr_col, qr_step, kr_col;     // ROPE: columns of the rotated part, where they are in the queries and in tm_kr
   long long ld_o;
   const __nv_bfloat16* gate;   // optional (rows, heads * vdim), row pitch ld_gate
   long long ld_gate;
@@ -113,23 +118,27 @@ struct FlashFwdParams {
       p.trace[((role) * 64 + (step)) * 8 + (slot)] = clock64();                              \
   } while (0)
 
-template <int DH>
+template <int DH, bool ROPE>
 struct FlashFwdSmem {
   static constexpr int PANELS = DH / 64;              // 64-column (128-byte) panels per tile
-  static constexpr int TILE_BYTES = 128 * DH * 2;     // Q, K or V tile
+  static constexpr int TILE_BYTES = 128 * DH * 2;     // V tile
+  static constexpr int QK_BYTES = TILE_BYTES + (ROPE ? 16384 : 0);      // Q or K tile
+  static constexpr int V_STAGES = ROPE && DH == 128 ? 1 : 2;
   static constexpr int OFF_Q = 0;                     // Q_A, Q_B
-  static constexpr int OFF_K = OFF_Q + 2 * TILE_BYTES;
-  static constexpr int OFF_V = OFF_K + 2 * TILE_BYTES;
-  static constexpr int OFF_BAR = OFF_V + 2 * TILE_BYTES;
+  static constexpr int OFF_K = OFF_Q + 2 * QK_BYTES;
+  static constexpr int OFF_V = OFF_K + 2 * QK_BYTES;
+  static constexpr int OFF_BAR = OFF_V + V_STAGES * TILE_BYTES;
   static constexpr int NUM_BARS = 1 + 4 + 4 + 2 + 4 + 2;  // q, k full/empty, v full/empty, s_full[2], p_full[2][2], o_full[2]
   static constexpr int TOTAL = OFF_BAR + NUM_BARS * 8 + 16 + 1024;
 };
 
-template <int DH, bool WINDOW>
+template <int DH, bool WINDOW, bool ROPE>
 __global__ void __launch_bounds__(FA_THREADS, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_constant__ CUtensorMap tm_kv,
-                 const FlashFwdParams p) {
-  using L = FlashFwdSmem<DH>;
+                 const __grid_constant__ CUtensorMap tm_kr, const FlashFwdParams p) {
+  static_assert(WINDOW || !ROPE, "");
+  using L = FlashFwdSmem<DH, ROPE>;
+  constexpr int VS = L::V_STAGES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR);
@@ -194,6 +203,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
     fence_barrier_init();
     prefetch_tensormap(&tm_qkv);
     if (WINDOW) prefetch_tensormap(&tm_kv);
+    if (ROPE) prefetch_tensormap(&tm_kr);
   }
   if (warp == 1) {
     tmem_alloc(tmem_holder, 512);
@@ -205,33 +215,43 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
   const uint32_t tmem_base = *tmem_holder;
   // columns: S_A [0,128)  S_B [128,256)  O_A [256,256+DH)  O_B [384,384+DH); P_X overlays the first 64 columns of S_X
 
-  const int col_q = h * DH, col_k = (WINDOW ? 0 : p.d) + h * DH, col_v = (WINDOW ? p.d : 2 * p.d) + h * DH;
+  const int col_q = h * (WINDOW ? p.q_step : DH), col_k = WINDOW ? h * p.k_step : p.d + h * DH,
+            col_v = WINDOW ? p.v_off + h * p.v_step : 2 * p.d + h * DH;
+  const int pd = WINDOW ? (p.dim + 63) / 64 : L::PANELS;                // panels of queries and keys that are loaded
+  const int ksteps = WINDOW ? (p.dim + 15) / 16 : DH / 16;
   const CUtensorMap* const map_kv = WINDOW ? &tm_kv : &tm_qkv;
 
   if (warp == 0) {
     if (active && elect_one()) {   // elect.sync keeps the issuing code warp-uniform (descriptors in uniform registers)
       // rows past the end of the tensor are zero-filled by TMA; rows of a following packed sequence are masked or unused
-      mbar_expect_tx(q_full, 2 * L::TILE_BYTES);
+      const uint32_t qk_bytes = (uint32_t)(pd + (ROPE ? 1 : 0)) * 16384u;
+      mbar_expect_tx(q_full, 2 * qk_bytes);
 #pragma unroll
-      for (int x = 0; x < 2; ++x)
+      for (int x = 0; x < 2; ++x) {
 #pragma unroll
         for (int pn = 0; pn < L::PANELS; ++pn)
-          tma_load_2d(smem + L::OFF_Q + x * L::TILE_BYTES + pn * 16384, &tm_qkv, q_full, col_q + pn * 64,
-                      row_base + q0_t[x]);
+          if (pn < pd)
+            tma_load_2d(smem + L::OFF_Q + x * L::QK_BYTES + pn * 16384, &tm_qkv, q_full, col_q + pn * 64, row_base + q0_t[x]);
+        if (ROPE)
+          tma_load_2d(smem + L::OFF_Q + x * L::QK_BYTES + L::TILE_BYTES, &tm_qkv, q_full, p.qr_col + h * p.qr_step, row_base + q0_t[x]);
+      }
       for (int j = j0; j < n_kv; ++j) {
         const int st = (j - j0) & 1;
         const uint32_t ph = ((j - j0) >> 1) & 1;
         const int krow = key_base + j * FA_BK;
         if (!mbar_wait(&k_empty[st], ph ^ 1, abort_word)) { *abort_word = ERR_WAIT_EMPTY; break; }
-        mbar_expect_tx(&k_full[st], L::TILE_BYTES);
+        mbar_expect_tx(&k_full[st], qk_bytes);
 #pragma unroll
         for (int pn = 0; pn < L::PANELS; ++pn)
-          tma_load_2d(smem + L::OFF_K + st * L::TILE_BYTES + pn * 16384, map_kv, &k_full[st], col_k + pn * 64, krow);
-        if (!mbar_wait(&v_empty[st], ph ^ 1, abort_word)) { *abort_word = ERR_WAIT_EMPTY; break; }
-        mbar_expect_tx(&v_full[st], L::TILE_BYTES);
+          if (pn < pd)
+            tma_load_2d(smem + L::OFF_K + st * L::QK_BYTES + pn * 16384, map_kv, &k_full[st], col_k + pn * 64, krow);
+        if (ROPE) tma_load_2d(smem + L::OFF_K + st * L::QK_BYTES + L::TILE_BYTES, &tm_kr, &k_full[st], p.kr_col, krow);
+        const int sv = (j - j0) % VS;
+        if (!mbar_wait(&v_empty[sv], (((j - j0) / VS) & 1) ^ 1, abort_word)) { *abort_word = ERR_WAIT_EMPTY; break; }
+        mbar_expect_tx(&v_full[sv], L::TILE_BYTES);
 #pragma unroll
         for (int pn = 0; pn < L::PANELS; ++pn)
-          tma_load_2d(smem + L::OFF_V + st * L::TILE_BYTES + pn * 16384, map_kv, &v_full[st], col_v + pn * 64, krow);
+          tma_load_2d(smem + L::OFF_V + sv * L::TILE_BYTES + pn * 16384, map_kv, &v_full[sv], col_v + pn * 64, krow);
       }
     }
   } else if (warp == 1) {
@@ -241,12 +261,22 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
       constexpr uint32_t idesc_qk = make_idesc_bf16(128, FA_BK, false, false);
       constexpr uint32_t idesc_pv = make_idesc_bf16(128, DH, false, true);
       auto issue_s = [&](int x, int j) {   // S_X(j) = Q_X K_j^T
-        const uint64_t q_desc = make_smem_desc(smem_u32(smem + L::OFF_Q + x * L::TILE_BYTES), 16, 1024);
-        const uint64_t k_desc = make_smem_desc(smem_u32(smem + L::OFF_K + ((j - j0) & 1) * L::TILE_BYTES), 16, 1024);
+        const uint64_t q_desc = make_smem_desc(smem_u32(smem + L::OFF_Q + x * L::QK_BYTES), 16, 1024);
+        const uint64_t k_desc = make_smem_desc(smem_u32(smem + L::OFF_K + ((j - j0) & 1) * L::QK_BYTES), 16, 1024);
+        if (ROPE) {
+          const int rsteps = (p.rot + 15) / 16;
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            if (k >= rsteps) break;
+            const uint32_t off = (L::TILE_BYTES + k * 32) >> 4;
+            umma_f16_ss(tmem_base + x * 128, q_desc + off, k_desc + off, idesc_qk, k > 0 ? 1u : 0u);
+          }
+        }
 #pragma unroll
         for (int k = 0; k < DH / 16; ++k) {
+          if (WINDOW && k >= ksteps) break;
           const uint32_t off = ((k / 4) * 16384 + (k % 4) * 32) >> 4;
-          umma_f16_ss(tmem_base + x * 128, q_desc + off, k_desc + off, idesc_qk, k > 0 ? 1u : 0u);
+          umma_f16_ss(tmem_base + x * 128, q_desc + off, k_desc + off, idesc_qk, (ROPE || k > 0) ? 1u : 0u);
         }
         umma_commit(&s_full[x]);
       };
@@ -254,7 +284,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
       // A = P from tensor memory (16 keys = 8 packed columns), B = V MN-major (dh contiguous, keys are rows of
       // 128 B): 16 keys = 2048 B; dh panels 16384 B apart.
       auto issue_pv = [&](int x, int j, int half) {
-        const uint64_t v_desc = make_smem_desc(smem_u32(smem + L::OFF_V + ((j - j0) & 1) * L::TILE_BYTES), 16384, 1024);
+        const uint64_t v_desc = make_smem_desc(smem_u32(smem + L::OFF_V + ((j - j0) % VS) * L::TILE_BYTES), 16384, 1024);
 #pragma unroll
         for (int kk = 0; kk < FA_BK / 32; ++kk) {
           const int k = half * (FA_BK / 32) + kk;
@@ -271,13 +301,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
         umma_commit(&k_empty[0]);
       }
       for (int j = j0; j < n_kv && ok; ++j) {
-        const int st = (j - j0) & 1;
-        const uint32_t ph = ((j - j0) >> 1) & 1;
+        const int st = (j - j0) & 1, sv = (j - j0) % VS;
+        const uint32_t pv = ((j - j0) / VS) & 1;
         bool v_ready = false, k_ready = false;
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
           if (j >= lo_t[x] && j < n_kv_t[x]) {
-            ok = mbar_wait(&p_full[2 * x], (j - lo_t[x]) & 1, abort_word) && (v_ready || mbar_wait(&v_full[st], ph, abort_word));
+            ok = mbar_wait(&p_full[2 * x], (j - lo_t[x]) & 1, abort_word) && (v_ready || mbar_wait(&v_full[sv], pv, abort_word));
             if (!ok) break;
             v_ready = true;
             tc_fence_after();
@@ -289,7 +319,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
             issue_pv(x, j, 1);
             FWD_TRACE(1, j, x * 4 + 1);
           }
-          if (x == 1) umma_commit(&v_empty[st]);   // both tiles are done with V_j
+          if (x == 1) umma_commit(&v_empty[sv]);   // both tiles are done with V_j
           if (j + 1 >= lo_t[x] && j + 1 < n_kv_t[x]) {
             ok = k_ready || mbar_wait(&k_full[st ^ 1], ((j + 1 - j0) >> 1) & 1, abort_word);
             if (!ok) break;
@@ -320,7 +350,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
     float m_run = -INFINITY;                    // running reference max in scaled log2 units
     float l_run = 0.f;                          // running row sum relative to m_run
     bool ok = true;
-    if (WINDOW && p.gate != nullptr && q_idx < seq_len) {      // the epilogue's gate row into L2
+    if (WINDOW && p.gate != nullptr && !p.head_gate && q_idx < seq_len) {      // the epilogue's gate row into L2
       const __nv_bfloat16* grow = p.gate + (long long)(row_base + q_idx) * p.ld_gate + h * p.vdim;
       for (int i = 0; i < p.vdim; i += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(grow + i));
     }
@@ -437,8 +467,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
     if (ok && n_kv_x > 0) ok = mbar_wait(&o_full[x], 0, abort_word);
     if (ok && n_kv_x > 0) {
       tc_fence_after();
-      const float inv_l = 1.f / l_run;
+      float inv_l = 1.f / l_run;
       const bool valid = q_idx < seq_len;
+      if (WINDOW && p.head_gate && valid) inv_l *= fa_sigmoid(__bfloat162float(p.gate[(long long)(row_base + q_idx) * p.ld_gate + h]));
       __nv_bfloat16* orow = WINDOW ? p.o + (long long)(row_base + q_idx) * p.ld_o + h * p.vdim
                                    : p.o + (size_t)(row_base + q_idx) * p.d + h * DH;
 #pragma unroll 1
@@ -449,7 +480,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
         if (WINDOW) {
           if (valid && c * 32 < p.vdim) {      // no early continue: the next tensor-memory load needs the whole warp
             const __nv_bfloat16* grow =
-                p.gate != nullptr ? p.gate + (long long)(row_base + q_idx) * p.ld_gate + h * p.vdim + c * 32 : nullptr;
+                p.gate != nullptr && !p.head_gate ? p.gate + (long long)(row_base + q_idx) * p.ld_gate + h * p.vdim + c * 32 : nullptr;
             const int n = min(32, p.vdim - c * 32);
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
@@ -514,17 +545,18 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tm_qkv, const __grid_consta
   }
 }
 
-template <int DH, bool WINDOW>
-static int launch_flash_fwd(const CUtensorMap& tm, const CUtensorMap& tm_kv, const FlashFwdParams& p, cudaStream_t stream) {
-  using L = FlashFwdSmem<DH>;
-  auto kern = flash_fwd_kernel<DH, WINDOW>;
+template <int DH, bool WINDOW, bool ROPE = false>
+static int launch_flash_fwd(const CUtensorMap& tm, const CUtensorMap& tm_kv, const FlashFwdParams& p, cudaStream_t stream,
+                            const CUtensorMap* tm_kr = nullptr) {
+  using L = FlashFwdSmem<DH, ROPE>;
+  auto kern = flash_fwd_kernel<DH, WINDOW, ROPE>;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL) != cudaSuccess) return -3;
     configured = true;
   }
   const int grid = p.batch * p.heads * ((p.n_qblk + 1) / 2);   // one CTA per pair of query tiles
-  kern<<<grid, FA_THREADS, L::TOTAL, stream>>>(tm, tm_kv, p);
+  kern<<<grid, FA_THREADS, L::TOTAL, stream>>>(tm, tm_kv, tm_kr != nullptr ? *tm_kr : tm_kv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -583,31 +615,48 @@ extern "C" int b200_flash_varlen_fwd(const void* qkv, void* o, const int* cu_seq
   return dh == 64 ? launch_flash_fwd<64, false>(tm, tm, p, stream) : launch_flash_fwd<128, false>(tm, tm, p, stream);
 }
 
-// Portions of prompts under a sliding window.  q: (total_q, heads * dh), kv: (total_k, 2 * heads * dh) = K | V, heads padded
-// with zero columns to dh = 64 or 128; cu_q / cu_k: (batch + 1) row offsets on the device; query i of a sequence with Lq
-// queries and Lk keys sits at key position i + Lk - Lq and sees the `window` keys up to it (window <= 0: all of them).
-// o: (total_q, heads * vdim), row pitch ld_o, multiplied by sigmoid(gate) when gate is given.  scale must be positive.
-extern "C" int b200_flash_window_fwd(const void* q, const void* kv, void* o, const void* gate, const int* cu_q,
-                                     const int* cu_k, int batch, int max_q, int total_q, int total_k, int heads, int dh,
-                                     int vdim, int window, float scale, long long ld_q, long long ld_kv, long long ld_o,
-                                     long long ld_gate, uint32_t* status, cudaStream_t stream) {
-  if ((dh != 64 && dh != 128) || vdim <= 0 || vdim > dh || !(scale > 0.f)) return -10;
-  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv)) & 15 || ld_q % 8 || ld_kv % 8) return -10;
+// Portions of prompts under a sliding window.  q: (total_q, q_cols), kv: (total_k, kv_cols); a head's queries, keys and values are dim,
+// dim and vdim columns (at most 128; more than 64 take the instance for 128) at h * q_step, h * k_step and v_off + h * v_step (steps and
+// offsets multiples of 8).  Columns are loaded in boxes of 64 and multiplied 16 at a time: up to the next multiple of 16 they must be
+// finite, and zero in q or k.  cu_q / cu_k: (batch + 1) row offsets on the device; query i of a sequence with Lq queries and Lk keys
+// sits at key position i + Lk - Lq and sees the `window` keys up to it (window <= 0: all of them).
+// rot > 0 (at most 64): the score gains rotated parts, rot columns of q at qr_col + h * qr_step and of kr (total_k, kr_cols) at kr_col,
+// the latter for all heads; the same rules.
+// o: (total_q, heads * vdim), row pitch ld_o, multiplied by sigmoid(gate) when gate is given: (total_q, heads * vdim), or
+// (total_q, heads) with head_gate.  scale must be positive.
+struct FlashWindowShape {        // passed by pointer through the C interface: the field order is part of it
+  long long ld_q, ld_kv, ld_kr, ld_o, ld_gate;
+  int q_cols, kv_cols, kr_cols, heads, dim, vdim, q_step, k_step, v_step, v_off, rot, qr_col, qr_step, kr_col, window, head_gate;
+  float scale;
+};
+
+extern "C" int b200_flash_window_fwd(const void* q, const void* kv, const void* kr, void* o, const void* gate, const int* cu_q,
+                                     const int* cu_k, int batch, int max_q, int total_q, int total_k, const FlashWindowShape* s,
+                                     uint32_t* status, cudaStream_t stream) {
+  const int dh = s->dim > 64 || s->vdim > 64 ? 128 : 64;
+  if (s->heads <= 0 || s->dim <= 0 || s->dim > 128 || s->vdim <= 0 || s->vdim > 128 || !(s->scale > 0.f)) return -10;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(kr)) & 15 || s->ld_q % 8 ||
+      s->ld_kv % 8 || (s->q_step | s->k_step | s->v_step | s->v_off) % 8)
+    return -10;
+  if (s->rot < 0 || s->rot > 64 || (s->rot > 0 && (kr == nullptr || s->ld_kr % 8 || (s->qr_col | s->qr_step | s->kr_col) % 8))) return -10;
   if (batch <= 0 || total_q <= 0) return 0;
-  const int d = heads * dh;
-  CUtensorMap tm, tm_kv;
-  if (make_tmap_bf16_2d(&tm, q, (uint64_t)total_q, (uint64_t)d, (uint64_t)ld_q, 64, 128)) return -20;
-  if (make_tmap_bf16_2d(&tm_kv, kv, (uint64_t)total_k, (uint64_t)2 * d, (uint64_t)ld_kv, 64, 128)) return -21;
+  CUtensorMap tm, tm_kv, tm_kr;
+  if (make_tmap_bf16_2d(&tm, q, (uint64_t)total_q, (uint64_t)s->q_cols, (uint64_t)s->ld_q, 64, 128)) return -20;
+  if (make_tmap_bf16_2d(&tm_kv, kv, (uint64_t)total_k, (uint64_t)s->kv_cols, (uint64_t)s->ld_kv, 64, 128)) return -21;
+  if (s->rot > 0 && make_tmap_bf16_2d(&tm_kr, kr, (uint64_t)total_k, (uint64_t)s->kr_cols, (uint64_t)s->ld_kr, 64, 128)) return -22;
   FlashFwdParams p = {};
   p.o = (__nv_bfloat16*)o; p.cu_seqlens = cu_q; p.cu_k = cu_k;
-  p.batch = batch; p.seq = max_q; p.heads = heads; p.d = d;
+  p.batch = batch; p.seq = max_q; p.heads = s->heads; p.d = s->heads * dh;
   p.n_qblk = (max_q + FA_BQ - 1) / FA_BQ;
-  p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = window > 0 ? window : (1 << 30);
-  p.vdim = vdim; p.ld_o = ld_o;
-  p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate;
-  p.out_vec = vdim % 8 == 0 && ld_o % 8 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0;
-  p.gate_vec = vdim % 8 == 0 && ld_gate % 8 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0;
+  p.scale_log2 = s->scale * 1.4426950408889634f;
+  p.window = s->window > 0 ? s->window : (1 << 30);
+  p.dim = s->dim; p.vdim = s->vdim; p.q_step = s->q_step; p.k_step = s->k_step; p.v_step = s->v_step; p.v_off = s->v_off;
+  p.rot = s->rot; p.qr_col = s->qr_col; p.qr_step = s->qr_step; p.kr_col = s->kr_col;
+  p.ld_o = s->ld_o; p.gate = (const __nv_bfloat16*)gate; p.ld_gate = s->ld_gate; p.head_gate = gate != nullptr && s->head_gate;
+  p.out_vec = s->vdim % 8 == 0 && s->ld_o % 8 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0;
+  p.gate_vec = s->vdim % 8 == 0 && s->ld_gate % 8 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0;
   p.status = status;
+  if (s->rot > 0)
+    return dh == 64 ? launch_flash_fwd<64, true, true>(tm, tm_kv, p, stream, &tm_kr) : launch_flash_fwd<128, true, true>(tm, tm_kv, p, stream, &tm_kr);
   return dh == 64 ? launch_flash_fwd<64, true>(tm, tm_kv, p, stream) : launch_flash_fwd<128, true>(tm, tm_kv, p, stream);
 }

@@ -18,6 +18,7 @@ enum GemmEpilogue : int {
   // (M x 2N, bf16) and C (M x 2N, bf16) receives d(gate) | d(up).
   EPI_SWIGLU_BWD = 4,
   // C = bf16(acc * sigmoid(R)): the output gate of an attention layer, R bf16 of C's shape.
+  // (With GemmParams::head_gate R has one column per problem instead.)
   EPI_BF16_GATE = 5,
   // Flag or-ed into the epilogue code by the caller (CTA-pair kernel): output columns from N up to the next 16-byte
   // boundary lie inside the row pitch and may be overwritten with zeros.
@@ -26,6 +27,21 @@ enum GemmEpilogue : int {
   // before this one on the stream (inference weights), so its first tiles may be requested before that kernel ends.
   EPI_B_STABLE = 0x200,
 };
+
+// What becomes of an accumulator before the epilogue code above: act(alpha * (acc + bias[n])).  Passed by pointer through the C
+// interface: the field order is part of it.
+enum GemmAct : int { ACT_NONE = 0, ACT_GELU = 1, ACT_CAP = 2 };     // gelu with erf; cap * tanh(v / cap)
+struct GemmFinish {
+  const float* bias;           // (N) or null
+  float alpha, cap;
+  int act;
+};
+
+__device__ __forceinline__ float finish_act(float v, int act, float cap) {
+  if (act == ACT_GELU) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+  if (act == ACT_CAP) return cap * tanhf(v / cap);
+  return v;
+}
 
 // Optional all-gather carried by a GEMM launch: while the MMA warps work, two copy warps per CTA pull
 // the weight shards of the *next* FSDP unit from every peer GPU into a local buffer (plain 16-byte peer
@@ -81,6 +97,9 @@ struct GemmParams {
   const int* tile_group;
   int group_rows;
   int batch, a_step, c_step;
+  int head_gate;              // EPI_BF16_GATE: R is (M, batch), one gate per problem
+  int finished;               // `finish` applies
+  GemmFinish finish;
   int relu;                   // gated instances of the single-CTA kernel: relu(gate) * up instead of silu(gate) * up
   int splits;
   float* ws;                  // splits * tiles partial tiles of BM x BN floats
@@ -122,12 +141,46 @@ __device__ __forceinline__ void epilogue_rope(const GemmParams& p, int row, int 
   }
 }
 
+// `ncols` (at most 32) accumulators of one row, starting with output column col0.
+__device__ __forceinline__ void epilogue_finish(const GemmParams& p, int col0, int ncols, uint32_t (&acc)[32]) {
+  if (p.finish.bias != nullptr) {
+    const float* b = p.finish.bias + col0;
+    if (ncols >= 32 && (reinterpret_cast<uintptr_t>(b) & 15) == 0) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float4 v = __ldg(reinterpret_cast<const float4*>(b) + j);
+        acc[4 * j] = __float_as_uint(__uint_as_float(acc[4 * j]) + v.x);
+        acc[4 * j + 1] = __float_as_uint(__uint_as_float(acc[4 * j + 1]) + v.y);
+        acc[4 * j + 2] = __float_as_uint(__uint_as_float(acc[4 * j + 2]) + v.z);
+        acc[4 * j + 3] = __float_as_uint(__uint_as_float(acc[4 * j + 3]) + v.w);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 32; ++j)
+        if (j < ncols) acc[j] = __float_as_uint(__uint_as_float(acc[j]) + __ldg(b + j));
+    }
+  }
+  if (p.finish.act == ACT_NONE) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) acc[j] = __float_as_uint(__uint_as_float(acc[j]) * p.finish.alpha);
+  } else if (p.finish.act == ACT_GELU) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) acc[j] = __float_as_uint(finish_act(__uint_as_float(acc[j]) * p.finish.alpha, ACT_GELU, 0.f));
+  } else {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) acc[j] = __float_as_uint(finish_act(__uint_as_float(acc[j]) * p.finish.alpha, ACT_CAP, p.finish.cap));
+  }
+}
+
+__device__ __forceinline__ float gate_of(float g) { return __fdividef(1.f, 1.f + __expf(-g)); }
+
 // One 32-column chunk of one output row.  `coff` shifts the columns of C and R (one of several problems side by side).
 __device__ __forceinline__ void epilogue_store(const GemmParams& p, int row, int col0, uint32_t (&acc)[32],
                                                int coff = 0) {
   if (row >= p.M) return;
   const int ncols = min(32, p.N - col0);
   if (ncols <= 0) return;
+  if (p.finished) epilogue_finish(p, col0, ncols, acc);
   if (p.rope_cs != nullptr && col0 < 2 * p.rope_d && ncols == 32) epilogue_rope(p, row, col0, acc);
   if (p.epi == EPI_SWIGLU_BWD) {
     // as the stand-alone kernel (fast division apart): dh is rounded to bf16 first, gate and up are read as bf16
@@ -156,11 +209,17 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, int row, int
     }
     return;
   }
+  if (p.epi == EPI_BF16_GATE && p.head_gate) {
+    const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.R) + (long long)row * p.ldr;
+    const float g = gate_of(__bfloat162float(r[coff / p.c_step]));
+#pragma unroll
+    for (int j = 0; j < 32; ++j) acc[j] = __float_as_uint(__uint_as_float(acc[j]) * g);
+  }
   if (p.epi == EPI_BF16 || p.epi == EPI_BF16_RES || p.epi == EPI_BF16_GATE) {
     __nv_bfloat16* c = reinterpret_cast<__nv_bfloat16*>(p.C) + (long long)row * p.ldc + coff + col0;
     const bool vec_ok = (ncols == 32) && ((p.ldc & 7) == 0) && ((coff & 7) == 0) &&
                         ((reinterpret_cast<uintptr_t>(p.C) & 15) == 0);
-    if (p.epi == EPI_BF16_GATE) {
+    if (p.epi == EPI_BF16_GATE && !p.head_gate) {
       const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.R) + (long long)row * p.ldr + coff + col0;
       if (vec_ok && (p.ldr & 7) == 0 && (reinterpret_cast<uintptr_t>(p.R) & 15) == 0) {
 #pragma unroll

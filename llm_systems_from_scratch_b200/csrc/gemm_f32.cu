@@ -1,7 +1,7 @@
 // fp32 GEMM on the FMA pipes, D[m, n] = sum_k A[m, k] B[n, k], for models that run in 32-bit: the tensor cores have no
 // full fp32 mode.  Same three problem kinds as the bf16 kernel (one problem, one group of B rows per 128-row tile of A,
 // or one problem per head side by side); no alignment requirements.
-#include "typed.cuh"
+#include "gemm_common.cuh"
 
 namespace b200 {
 
@@ -15,6 +15,8 @@ struct GemmF32Params {
   int accumulate;
   const int* tile_group;       // per 128 rows of A
   int group_rows, a_step, c_step;
+  int finished;
+  GemmFinish finish;
 };
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
@@ -58,7 +60,9 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (m < p.M && n < p.N) {
         float* c = C + (long long)m * p.ldc + n;
-        *c = p.accumulate ? *c + acc[i][j] : acc[i][j];
+        float v = acc[i][j];
+        if (p.finished) v = finish_act(p.finish.alpha * (v + (p.finish.bias != nullptr ? p.finish.bias[n] : 0.f)), p.finish.act, p.finish.cap);
+        *c = p.accumulate ? *c + v : v;
       }
     }
 }
@@ -68,15 +72,17 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Params p) {
 using namespace b200;
 
 // accumulate: C += A B^T.  tile_group / batch as in b200_gemm_bf16_grouped (batch <= 1 and no tile_group: one problem).
+// finish: null, or what to do with the sums first (a bias is that of a single problem).
 extern "C" int b200_gemm_f32(const float* A, const float* B, float* C, int M, int N, int K, long long lda, long long ldb,
                              long long ldc, int accumulate, const int* tile_group, int group_rows, int batch, int a_step,
-                             int c_step, cudaStream_t st) {
+                             int c_step, const GemmFinish* finish, cudaStream_t st) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if (tile_group != nullptr && (batch > 1 || M % 128)) return -12;
   GemmF32Params p;
   p.A = A; p.B = B; p.C = C; p.M = M; p.N = N; p.K = K; p.lda = lda; p.ldb = ldb; p.ldc = ldc;
   p.accumulate = accumulate; p.tile_group = tile_group;
-  p.group_rows = group_rows; p.a_step = a_step; p.c_step = c_step;
+  p.group_rows = group_rows; p.a_step = a_step; p.c_step = c_step; p.finished = finish != nullptr;
+  if (finish != nullptr) p.finish = *finish;
   const dim3 grid((N + SG_TILE - 1) / SG_TILE, (M + SG_TILE - 1) / SG_TILE, batch > 1 ? batch : 1);
   if (grid.y > 65535 || grid.z > 65535) return -13;
   launch_dep(gemm_f32_kernel, grid, 256, 0, st, p);

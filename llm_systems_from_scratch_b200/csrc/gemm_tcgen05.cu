@@ -453,7 +453,7 @@ using namespace b200;
 static int gemm_bf16_impl(const void* A, const void* B, void* C, const void* R, int M, int N, int K, long long lda,
                           long long ldb, long long ldc, long long ldr, int a_mn, int b_mn, int epi, int bn_hint,
                           int max_ctas, int splits, float* ws, uint32_t* tile_counters, uint32_t* status,
-                          cudaStream_t stream) {
+                          cudaStream_t stream, const GemmFinish* finish = nullptr) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15) || (lda & 7) || (ldb & 7))
     return -10;
@@ -515,7 +515,9 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, const void* R, 
   p.swiglu_f = 0; p.H = nullptr; p.ldh = 0;
   p.splits = splits > 1 ? splits : 1; p.ws = ws; p.tile_counters = tile_counters;
   p.b_early = b_early;
-  p.tile_group = nullptr; p.group_rows = 0; p.batch = 1; p.a_step = p.c_step = 0; p.relu = 0;
+  p.tile_group = nullptr; p.group_rows = 0; p.batch = 1; p.a_step = p.c_step = 0; p.relu = 0; p.head_gate = 0;
+  p.finished = finish != nullptr;
+  if (finish != nullptr) p.finish = *finish;
 
 #define DISPATCH(BN_)                                                                    \
   if (a_mn && b_mn) return launch_gemm<BN_, true, true>(tmA, tmB, p, max_ctas, stream);   \
@@ -534,6 +536,14 @@ extern "C" int b200_gemm_bf16(const void* A, const void* B, void* C, const void*
                               int epi, int bn_hint, int max_ctas, uint32_t* status, cudaStream_t stream) {
   return gemm_bf16_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, a_mn, b_mn, epi, bn_hint, max_ctas, 1, nullptr,
                         nullptr, status, stream);
+}
+
+// K-major operands, epi 0, 1 or 3, accumulators finished first (see GemmFinish).
+extern "C" int b200_gemm_bf16_finish(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
+                                     long long ldc, int epi, const GemmFinish* finish, uint32_t* status, cudaStream_t stream) {
+  const int base = epi & ~EPI_B_STABLE;
+  if (base != EPI_BF16 && base != EPI_F32 && base != EPI_F32_ACC) return -11;
+  return gemm_bf16_impl(A, B, C, nullptr, M, N, K, lda, ldb, ldc, 0, 0, 0, epi, 0, 0, 1, nullptr, nullptr, status, stream, finish);
 }
 
 // Tile width and number of K slices for a GEMM with at most two rows of tiles (decode: M <= 256, weights streamed
@@ -575,10 +585,10 @@ extern "C" int b200_gemm_splitk_counters(void) { return 4 * num_sms() * 4; }
 // b200_gemm_bf16 for K-major operands and M <= 256 with K split over CTAs (see b200_gemm_splitk_plan).  `ws` and
 // `tile_counters` are scratch of the sizes above; the counters must be zero on entry and are zero again on exit.
 // One launch at a time may use a given workspace (launches on one stream are ordered; other streams need their own).
-extern "C" int b200_gemm_bf16_splitk(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
-                                     long long lda, long long ldb, long long ldc, long long ldr, int epi, float* ws,
-                                     long long ws_floats, uint32_t* tile_counters, int n_counters, uint32_t* status,
-                                     cudaStream_t stream) {
+static int splitk_impl(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
+                       long long lda, long long ldb, long long ldc, long long ldr, int epi, float* ws,
+                       long long ws_floats, uint32_t* tile_counters, int n_counters, uint32_t* status,
+                       cudaStream_t stream, const GemmFinish* finish) {
   int bn = 0, splits = 1;
   b200_gemm_splitk_plan(M, N, K, &bn, &splits);
   const long long tiles = (long long)((M + BM - 1) / BM) * ((N + bn - 1) / bn);
@@ -588,9 +598,22 @@ extern "C" int b200_gemm_bf16_splitk(const void* A, const void* B, void* C, cons
   const int base_epi = epi & ~EPI_B_STABLE;
   if (base_epi != EPI_BF16 && base_epi != EPI_F32 && base_epi != EPI_BF16_RES && base_epi != EPI_F32_ACC) return -11;
   if (splits <= 1)
-    return gemm_bf16_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, 0, 0, epi, 0, 0, 1, nullptr, nullptr, status, stream);
+    return gemm_bf16_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, 0, 0, epi, 0, 0, 1, nullptr, nullptr, status, stream, finish);
   return gemm_bf16_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, 0, 0, epi, bn, 0, splits, ws, tile_counters, status,
-                        stream);
+                        stream, finish);
+}
+
+extern "C" int b200_gemm_bf16_splitk(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
+                                     long long lda, long long ldb, long long ldc, long long ldr, int epi, float* ws,
+                                     long long ws_floats, uint32_t* tile_counters, int n_counters, uint32_t* status,
+                                     cudaStream_t stream) {
+  return splitk_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, epi, ws, ws_floats, tile_counters, n_counters, status, stream, nullptr);
+}
+
+extern "C" int b200_gemm_bf16_splitk_finish(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
+                                            long long ldc, int epi, const GemmFinish* finish, float* ws, long long ws_floats,
+                                            uint32_t* tile_counters, int n_counters, uint32_t* status, cudaStream_t stream) {
+  return splitk_impl(A, B, C, nullptr, M, N, K, lda, ldb, ldc, 0, epi, ws, ws_floats, tile_counters, n_counters, status, stream, finish);
 }
 
 // Several GEMMs in one launch, K-major bf16 operands (see GemmParams):
@@ -600,12 +623,13 @@ extern "C" int b200_gemm_bf16_splitk(const void* A, const void* B, void* C, cons
 //   tile_group == null: `batch` problems side by side: problem g multiplies A[:, g * a_step : g * a_step + K] with
 //     B[g * group_rows : g * group_rows + N, :] into C[:, g * c_step : g * c_step + N].  a_step must be a multiple of 8.
 //     With `swiglu` B has the 2 N rows of one gated feed-forward per problem, as above (any M).
-// swiglu: 0 off, 1 silu(gate) * up, 2 relu(gate) * up.
+// swiglu: 0 off, 1 silu(gate) * up, 2 relu(gate) * up.  head_gate: with epi 5, R (M, batch) holds one gate per problem.
+// finish: null, or what to do with the accumulators first (not with swiglu).
 // Columns of A past a problem's K (up to the next multiple of 64) are multiplied with zeros, so they must be finite.
 extern "C" int b200_gemm_bf16_grouped(const void* A, const void* B, void* C, const void* R, int M, int N, int K,
                                       long long lda, long long ldb, long long ldc, long long ldr, const int* tile_group,
                                       int n_groups, int group_rows, int batch, int a_step, int c_step, int swiglu,
-                                      int epi, uint32_t* status, cudaStream_t stream) {
+                                      int epi, int head_gate, const GemmFinish* finish, uint32_t* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15) || (lda & 7) || (ldb & 7))
     return -10;
@@ -614,9 +638,11 @@ extern "C" int b200_gemm_bf16_grouped(const void* A, const void* B, void* C, con
   epi &= ~EPI_B_STABLE;
   if (epi != EPI_BF16 && epi != EPI_F32 && epi != EPI_BF16_GATE) return -11;
   if (epi == EPI_BF16_GATE && (R == nullptr || rows)) return -11;
+  if (head_gate && c_step <= 0) return -11;
   if (rows && ((M % BM) || n_groups <= 0 || group_rows != (swiglu ? 2 * N : N))) return -12;
   if (!rows && (batch <= 0 || (a_step & 7) || group_rows < (swiglu ? 2 * N : N))) return -12;
-  if (swiglu < 0 || swiglu > 2 || (swiglu && epi != EPI_BF16)) return -12;
+  if (swiglu < 0 || swiglu > 2 || (swiglu && (epi != EPI_BF16 || finish != nullptr))) return -12;
+  if (finish != nullptr && finish->bias != nullptr && (rows || batch > 1)) return -12;
   const int sms = num_sms();
   const long long mt = (M + BM - 1) / BM, problems = rows ? 1 : batch;
   int bn = 64;
@@ -648,6 +674,8 @@ extern "C" int b200_gemm_bf16_grouped(const void* A, const void* B, void* C, con
   p.splits = 1; p.ws = nullptr; p.tile_counters = nullptr;
   p.b_early = b_early;
   p.tile_group = tile_group; p.group_rows = group_rows; p.batch = rows ? 1 : batch; p.a_step = a_step; p.c_step = c_step; p.relu = swiglu == 2;
+  p.head_gate = head_gate; p.finished = finish != nullptr;
+  if (finish != nullptr) p.finish = *finish;
   if (!rows && swiglu) {
     if (bn == 256) return launch_gemm<256, false, false, GROUP_COLS, true>(tmA, tmB, p, 0, stream);
     if (bn == 128) return launch_gemm<128, false, false, GROUP_COLS, true>(tmA, tmB, p, 0, stream);

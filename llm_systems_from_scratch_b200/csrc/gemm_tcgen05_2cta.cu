@@ -497,11 +497,16 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
           if (out_f32) {
             tmem_ld_32x32(taddr + c * 32, o);
             tmem_ld_wait();
+            if (p.finished) epilogue_finish(p, col, p.N - col, o);
           } else {
             uint32_t r0[32], r1[32];
             tmem_ld_32x32(taddr + c * 64, r0);
             tmem_ld_32x32(taddr + c * 64 + 32, r1);
             tmem_ld_wait();
+            if (p.finished) {
+              epilogue_finish(p, col, p.N - col, r0);
+              epilogue_finish(p, col + 32, p.N - col - 32, r1);
+            }
             if (p.rope_cs != nullptr && col < 2 * p.rope_d) {      // N = 3 * rope_d, heads are multiples of 32 columns
               epilogue_rope(p, row, col, r0);
               epilogue_rope(p, row, col + 32, r1);
@@ -619,7 +624,7 @@ static int gemm_pair_impl(const void* A, const void* B, void* C, const void* R, 
                           const GatherTask* gather, const uint32_t* wait_counter, uint32_t wait_value,
                           uint32_t* status, cudaStream_t stream, const float* rope_cs = nullptr, int rope_seq = 0,
                           int rope_d = 0, int rope_dh = 0, int rope_ctx = 0, int swiglu_f = 0, void* H = nullptr,
-                          long long ldh = 0, const ReduceTask* reduce = nullptr) {
+                          long long ldh = 0, const ReduceTask* reduce = nullptr, const GemmFinish* finish = nullptr) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15) || (lda & 7) || (ldb & 7))
     return -10;
@@ -644,7 +649,9 @@ static int gemm_pair_impl(const void* A, const void* B, void* C, const void* R, 
   else { p.gather.dst = nullptr; p.gather.done = nullptr; p.gather.shard_vec = 0; p.gather.world = 0; p.gather.rank = 0; }
   if (reduce != nullptr) p.reduce = *reduce;
   else p.reduce.n = 0;
-  p.splits = 1; p.ws = nullptr; p.tile_counters = nullptr; p.b_early = 0;
+  p.splits = 1; p.ws = nullptr; p.tile_counters = nullptr; p.b_early = 0; p.head_gate = 0;
+  p.finished = finish != nullptr;
+  if (finish != nullptr) p.finish = *finish;
   p.wait_counter = wait_counter; p.wait_value = wait_value; p.wait_limit_ns = g_counter_wait_limit_ns;
   p.rope_cs = rope_cs; p.rope_seq = rope_seq; p.rope_d = rope_d; p.rope_dh = rope_dh; p.rope_ctx = rope_ctx;
   p.swiglu_f = swiglu_f; p.H = H; p.ldh = ldh;
@@ -693,6 +700,14 @@ extern "C" int b200_gemm_bf16_pair(const void* A, const void* B, void* C, const 
                                    long long lda, long long ldb, long long ldc, long long ldr, int a_mn, int b_mn,
                                    int epi, uint32_t* status, cudaStream_t stream) {
   return gemm_pair_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, a_mn, b_mn, epi, nullptr, nullptr, 0, status, stream);
+}
+
+// K-major operands, epi 0, 1 or 3, accumulators finished first (see GemmFinish).
+extern "C" int b200_gemm_bf16_pair_finish(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
+                                          long long ldc, int epi, const GemmFinish* finish, uint32_t* status, cudaStream_t stream) {
+  if (epi != EPI_BF16 && epi != EPI_F32 && epi != EPI_F32_ACC) return -11;
+  return gemm_pair_impl(A, B, C, nullptr, M, N, K, lda, ldb, ldc, 0, 0, 0, epi, nullptr, nullptr, 0, status, stream, nullptr, 0, 0, 0,
+                        0, 0, nullptr, 0, nullptr, finish);
 }
 
 // The same GEMM carrying an all-gather: while the tensor cores work, copy warps pull `shard_bytes` from each

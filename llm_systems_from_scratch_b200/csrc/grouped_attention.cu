@@ -1,6 +1,7 @@
 // Softmax attention of grouped heads over a paged cache: query head h reads key/value head h / (heads / kv_heads), under a
-// sliding window (position i sees the `window` positions up to and including i), with an optional bias per distance and,
-// for differential attention, two maps per head over the same values:
+// sliding window (position i sees the `window` positions up to and including i, and the first `keep` positions of the sequence), with
+// optional parts: scores capped softly (cap tanh(score / cap)), a bias per distance, a sink per head (exp(sink) joins the softmax's
+// denominator) and, for differential attention, two maps per head over the same values:
 //     o = a_1 - difference * a_2,   o <- o / rms(o) * out_scale
 // and an optional gate, o * sigmoid(g).  This file: norm, rotation and append; the general kernel (any size, bf16 or fp32);
 // decode on mma.sync.  Portions of prompts: grouped_prefill.cu.
@@ -253,6 +254,129 @@ static void launch_prep_pieces(const GroupedPrepParams& p, cudaStream_t st) {
   else launch_prep_lanes<T, 32>(p, vectors, st);
 }
 
+// Norm over the whole projection: the queries of all heads share one root mean square, so do the keys; weights of the projections'
+// sizes.  One block per row, pieces of VEC elements per thread, the first KEEP of them in registers between the passes.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(512) grouped_prep_whole_kernel(const GroupedPrepParams p) {
+  pdl_sync();
+  __shared__ float red[2][16];
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool own = p.wk != nullptr;
+  const int nq = p.heads * p.dim, nk = own ? p.kv_heads * p.dim : 0, nv = own ? p.kv_heads * p.vdim : 0;
+  const T* src = reinterpret_cast<const T*>(p.proj) + (long long)row * p.ld;
+  const int step = blockDim.x * VEC, total = nq + nk + nv;
+  auto load = [&](int c, float (&f)[VEC]) __attribute__((always_inline)) {
+    if constexpr (VEC == 8) unpack(load_piece(src + c), f);
+    else f[0] = to_f(src[c]);
+  };
+  constexpr int KEEP = 3;
+  float keep[KEEP][VEC], sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * VEC + j * step;
+    if (c < total) load(c, keep[j]);
+  }
+  auto square = [&](int c, const float (&f)[VEC]) __attribute__((always_inline)) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(f[i], f[i], ss);
+    if (c < nq) sq += ss;
+    else if (c < nq + nk) sk += ss;
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * VEC + j * step;
+    if (c < nq + nk) square(c, keep[j]);
+  }
+  for (int c = threadIdx.x * VEC + KEEP * step; c < nq + nk; c += step) {
+    float f[VEC];
+    load(c, f);
+    square(c, f);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    sk += __shfl_xor_sync(0xffffffffu, sk, o);
+  }
+  if (lane == 0) {
+    red[0][warp] = sq;
+    red[1][warp] = sk;
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) {
+    sq += red[0][w];
+    sk += red[1][w];
+  }
+  const float rq = rsqrtf(sq / (float)nq + p.eps), rk = own ? rsqrtf(sk / (float)nk + p.eps) : 0.f;
+  int pos = p.positions[row];
+  if (p.rot > 0 && (pos < 0 || pos >= p.ctx)) {
+    if (threadIdx.x == 0) report_bad_arg(p.status, 23);
+    pos = 0;
+  }
+  const long long slot = p.slots[row];
+  const bool live = slot >= 0 && slot < p.num_slots;             // a padding row of the batch has no slot
+  if (own && slot >= p.num_slots && threadIdx.x == 0) report_bad_arg(p.status, 24);
+  T* cache = reinterpret_cast<T*>(p.cache) + (live ? slot : 0) * ((long long)p.kv_heads * (p.kp + p.vp));
+  T* q = reinterpret_cast<T*>(p.q) + (long long)row * p.heads * p.qp;
+  const int half = p.rot / 2;
+  auto finish = [&](int c, float (&f)[VEC]) __attribute__((always_inline)) {
+    T* dst;
+    if (c < nq + nk) {
+      const bool query = c < nq;
+      const int at = query ? c : c - nq, v = at / p.dim, e = at - v * p.dim;
+      const T* w = reinterpret_cast<const T*>(query ? p.wq : p.wk) + at;
+      const float r = query ? rq : rk;
+      float g[VEC];
+      if constexpr (VEC == 8) unpack(load_piece(w), g);
+      else g[0] = to_f(*w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) f[i] *= r * g[i];
+      if (e < p.rot) {
+        const bool low = e < half;
+        const int to = low ? half : -half;
+        float o[VEC];
+        load(c + to, o);
+        if constexpr (VEC == 8) unpack(load_piece(w + to), g);
+        else g[0] = to_f(w[to]);
+        const float* cs = p.cos_sin + (long long)pos * half + (low ? e : e - half);
+        const float* sn = cs + (long long)p.ctx * half;
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          const float other = o[i] * r * g[i];
+          f[i] = low ? f[i] * cs[i] - other * sn[i] : f[i] * cs[i] + other * sn[i];
+        }
+      }
+      dst = query ? q + v * p.qp + e : cache + v * p.kp + e;
+    } else {
+      const int at = c - nq - nk, v = at / p.vdim;
+      dst = cache + p.kv_heads * p.kp + v * p.vp + (at - v * p.vdim);
+    }
+    if (c < nq || live) {
+      if constexpr (VEC == 8) store8(dst, f);
+      else from_f(*dst, f[0]);
+    }
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * VEC + j * step;
+    if (c < total) finish(c, keep[j]);
+  }
+  for (int c = threadIdx.x * VEC + KEEP * step; c < total; c += step) {
+    float f[VEC];
+    load(c, f);
+    finish(c, f);
+  }
+  // the pads behind every vector
+  auto pad = [&](T* base, int vectors, int pitch, int len) {
+    const int n = pitch - len;
+    for (int i = threadIdx.x; i < vectors * n; i += blockDim.x) from_f(base[(i / n) * pitch + len + i % n], 0.f);
+  };
+  if (p.qp > p.dim) pad(q, p.heads, p.qp, p.dim);
+  if (own && live && p.kp > p.dim) pad(cache, p.kv_heads, p.kp, p.dim);
+  if (own && live && p.vp > p.vdim) pad(cache + p.kv_heads * p.kp, p.kv_heads, p.vp, p.vdim);
+}
+
 // ------------------------------------------------------------------------------------------------------ general form
 // One warp per (row, head), keys one after the other; any size, T = bf16 or fp32.  row_seq[row] names the row's line of
 // `tables` (null: line `row`).
@@ -292,8 +416,9 @@ __global__ void __launch_bounds__(128) grouped_rows_kernel(const GroupedRowsPara
   const int width = s.kv_heads * (s.maps * s.kp + s.vp);
   if (live) {
     const int* table = p.tables + (long long)seq * p.max_pages;
-    const int lo = max(0, pos - s.window + 1);
-    for (int j = lo; j <= pos; ++j) {
+    const int lo = max(0, pos - s.window + 1), kept = min(s.keep, lo);
+    for (int n = lo - kept; n <= pos; ++n) {
+      const int j = n < lo ? n - (lo - kept) : n;                 // the kept positions, then the window
       const int pg = j / p.page_size;
       const int page = pg < p.max_pages ? table[pg] : -1;
       if ((unsigned)page >= (unsigned)p.num_pages) {
@@ -309,7 +434,9 @@ __global__ void __launch_bounds__(128) grouped_rows_kernel(const GroupedRowsPara
         for (int i = lane; i < s.dim; i += 32) sc = fmaf(qs[m * s.dim + i], to_f(k[i]), sc);
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) sc += __shfl_xor_sync(0xffffffffu, sc, o);
-        sc = sc * s.scale + b;
+        sc *= s.scale;
+        if (s.softcap > 0.f) sc = s.softcap * tanhf(sc / s.softcap);
+        sc += b;
         const float mn = fmaxf(mx[m], sc);
         const float a = expf(mx[m] - mn), e = expf(sc - mn);      // first key: exp(-inf) = 0
         l[m] = l[m] * a + e;
@@ -317,6 +444,12 @@ __global__ void __launch_bounds__(128) grouped_rows_kernel(const GroupedRowsPara
         mx[m] = mn;
       }
     }
+  }
+  if (s.sink != nullptr && live) {
+    const float mn = fmaxf(mx[0], s.sink[h]);
+    const float a = expf(mx[0] - mn);
+    l[0] = l[0] * a + expf(s.sink[h] - mn);
+    for (int c = lane; c < s.vdim; c += 32) acc[c] *= a;
   }
   const float i0 = l[0] > 0.f ? 1.f / l[0] : 0.f, i1 = l[1] > 0.f ? s.difference / l[1] : 0.f;
   float ss = 0.f;
@@ -423,6 +556,11 @@ __device__ __forceinline__ void grouped_finish(const GroupedShape& s, int lane, 
   }
 }
 
+// Denominator l relative to the maximum m (log2 units; -inf: no key), with the sink in it.
+__device__ __forceinline__ void add_sink(float sink, float m, float& l) {
+  if (m != -INFINITY) l += exp2f(fminf(fmaf(sink, LOG2E, -m), 126.f));      // a sink that far above every key takes all the weight
+}
+
 template <int KT, int VT>
 __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const GroupedDecodeParams p) {
   using L = GroupedDecodeSmem<KT, VT>;
@@ -451,15 +589,18 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
   const int pos = p.positions[row];
   const bool live = p.slots[row] >= 0 && pos >= 0;
   const int lo = live ? max(0, pos - s.window + 1) : 0;
-  const int first = lo / GD_TOK, total = live ? pos / GD_TOK + 1 - first : 0;       // tiles start at multiples of 16 tokens
+  // tiles of 16 tokens, starting at multiples of 16: those of the kept tokens in front of the window's first tile, then the window's
+  const int first = lo / GD_TOK, kept = min((s.keep + GD_TOK - 1) / GD_TOK, first);
+  const int total = live ? kept + pos / GD_TOK + 1 - first : 0;
+  auto token = [&](int tile) { return (tile < kept ? tile : first + tile - kept) * GD_TOK; };
   const int per = (total + p.splits - 1) / p.splits;
   const int i0 = min(total, split * per), tiles = min(total, i0 + per) - i0;
   const int* table = p.tables + (long long)row * p.max_pages;
 
   auto look_up = [&](int i) -> long long {     // cache row of this lane's token of tile i0 + i of this split; -1: none
     if (i >= tiles) return -1;
-    const int t = (first + i0 + i) * GD_TOK + (lane & 15);
-    if (t < lo || t > pos) return -1;
+    const int t = token(i0 + i) + (lane & 15);
+    if ((t < lo && t >= s.keep) || t > pos) return -1;
     const int pg = t / p.page_size;
     const int page = pg < p.max_pages ? table[pg] : -1;
     if ((unsigned)page < (unsigned)p.num_pages) return (long long)page * p.page_size + t % p.page_size;
@@ -499,7 +640,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
   for (int j = 0; j < VT; ++j)
 #pragma unroll
     for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
-  const float scale_log2 = s.scale * 1.4426950408889634f;
+  const float scale_log2 = s.scale * LOG2E, slope = s.softcap > 0.f ? 2.f * LOG2E * s.scale / s.softcap : 0.f;
   const float* bias[2] = {nullptr, nullptr};
   if (p.bias != nullptr) {
 #pragma unroll
@@ -508,7 +649,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
 
   float bn[2][4];                                      // bias of the tile after the one at work
   auto load_bias = [&](int i) {
-    const int t = (first + i0 + i) * GD_TOK + (lane & 3) * 2;
+    const int t = token(i0 + i) + (lane & 3) * 2;
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
@@ -534,16 +675,16 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
       gd_mma(sc[0], qf[kk], b[0], b[1]);
       gd_mma(sc[1], qf[kk], b[2], b[3]);
     }
-    const int t0 = (first + i0 + i) * GD_TOK + (lane & 3) * 2;
+    const int t0 = token(i0 + i) + (lane & 3) * 2;
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = t0 + n * 8 + (e & 1);
-        float x = sc[n][e] * scale_log2;
-        const bool seen = t >= lo && t <= pos;
-        if (p.bias != nullptr) x = fmaf(bn[n][e], 1.4426950408889634f, x);
+        float x = s.softcap > 0.f ? capped_log2(sc[n][e], slope, s.softcap * LOG2E) : sc[n][e] * scale_log2;
+        const bool seen = (t >= lo || t < s.keep) && t <= pos;
+        if (p.bias != nullptr) x = fmaf(bn[n][e], LOG2E, x);
         x = seen ? x : -INFINITY;
         sc[n][e] = x;
         mx[e >> 1] = fmaxf(mx[e >> 1], x);
@@ -647,6 +788,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
         for (int c = lane; c < s.vdim; c += 32) p.part_o[at * s.vdim + c] = sum(mp, c);
       }
     } else {
+      if (s.sink != nullptr) add_sink(s.sink[h], m[0], l[0]);
       const float inv[2] = {l[0] > 0.f ? 1.f / l[0] : 0.f, l[1] > 0.f ? 1.f / l[1] : 0.f};
       grouped_finish(s, lane, p.o + (long long)row * p.ld_o + h * s.vdim,
                      p.gate != nullptr ? p.gate + (long long)row * p.ld_gate + h * s.vdim : nullptr, [&](int mp, int c) {
@@ -677,6 +819,7 @@ __global__ void __launch_bounds__(128) grouped_merge_kernel(const GroupedDecodeP
     for (int i = 0; i < p.splits; ++i) gm[mp] = fmaxf(gm[mp], ml[i * 2]);
     float l = 0.f;
     for (int i = 0; i < p.splits; ++i) l += ml[i * 2] == -INFINITY ? 0.f : ml[i * 2 + 1] * exp2f(ml[i * 2] - gm[mp]);
+    if (mp == 0 && s.sink != nullptr) add_sink(s.sink[h], gm[0], l);
     inv[mp] = l > 0.f ? 1.f / l : 0.f;
   }
   grouped_finish(s, lane, p.o + (long long)row * p.ld_o + h * s.vdim,
@@ -737,6 +880,34 @@ extern "C" int b200_grouped_prep(const void* proj, long long ld, void* q, void* 
   } else {
     if (vec) launch_dep(grouped_prep_kernel<__nv_bfloat16, 4>, grid, warps * 32, 0, st, p);
     else launch_dep(grouped_prep_kernel<__nv_bfloat16, 1>, grid, warps * 32, 0, st, p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// As b200_grouped_prep for one map, with one norm over all queries and one over all keys: wq (heads * dim), wk (kv_heads * dim).
+extern "C" int b200_grouped_prep_whole(const void* proj, long long ld, void* q, void* cache, const void* wq, const void* wk,
+                                       const float* cos_sin, const int* positions, const long long* slots, int rows, int rot, int ctx,
+                                       long long num_slots, const GroupedShape* s, int f32, uint32_t* status, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (!shape_ok(*s) || s->maps != 1 || rot < 0 || rot > s->dim || (rot & 1) || (rot > 0 && cos_sin == nullptr) || wq == nullptr) return -10;
+  GroupedPrepParams p;
+  p.proj = proj; p.ld = ld; p.q = q; p.cache = cache; p.wq = wq; p.wk = wk; p.cos_sin = cos_sin; p.positions = positions;
+  p.slots = slots; p.rows = rows; p.heads = s->heads; p.kv_heads = s->kv_heads; p.maps = 1; p.dim = s->dim;
+  p.vdim = s->vdim; p.qp = s->qp; p.kp = s->kp; p.vp = s->vp; p.rot = rot; p.ctx = ctx; p.num_slots = num_slots;
+  p.eps = s->eps; p.status = status;
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) |
+                         reinterpret_cast<uintptr_t>(wq) | reinterpret_cast<uintptr_t>(wk);
+  const bool vec = s->dim % 8 == 0 && s->vdim % 8 == 0 && (rot / 2) % 8 == 0 && ld % 8 == 0 && (ptrs & 15) == 0;
+  const int pieces = (s->heads * s->dim + (wk != nullptr ? s->kv_heads * (s->dim + s->vdim) : 0)) / (vec ? 8 : 1);
+  int threads = ((pieces + 1) / 2 + 31) / 32 * 32;
+  if (threads > 512) threads = 512;
+  if (rows < 148 * 2) threads = min(512, (pieces + 31) / 32 * 32);
+  if (f32) {
+    if (vec) launch_dep(grouped_prep_whole_kernel<float, 8>, rows, threads, 0, st, p);
+    else launch_dep(grouped_prep_whole_kernel<float, 1>, rows, threads, 0, st, p);
+  } else {
+    if (vec) launch_dep(grouped_prep_whole_kernel<__nv_bfloat16, 8>, rows, threads, 0, st, p);
+    else launch_dep(grouped_prep_whole_kernel<__nv_bfloat16, 1>, rows, threads, 0, st, p);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -8,13 +8,23 @@ namespace b200 {
 struct GroupedShape {
   int heads, kv_heads, maps, dim, vdim;
   int qp, kp, vp;               // pitches of a query vector, a cached key, a cached value
-  int window;
-  float scale, eps, difference, out_scale;
+  int window, keep;             // position i sees j if i - j < window or j < keep
+  float scale, eps, difference, out_scale, softcap;      // softcap 0: none
+  const float* sink;            // (heads) or null: exp(sink) joins the denominator (one map)
 };
 
 inline bool shape_ok(const GroupedShape& s) {
   return s.heads > 0 && s.kv_heads > 0 && s.heads % s.kv_heads == 0 && (s.maps == 1 || s.maps == 2) && s.dim > 0 && s.vdim > 0 &&
-         s.qp >= s.kp && s.kp >= s.dim && s.vp >= s.vdim && s.qp % 8 == 0 && s.kp % 8 == 0 && s.vp % 8 == 0 && s.window > 0;
+         s.qp >= s.kp && s.kp >= s.dim && s.vp >= s.vdim && s.qp % 8 == 0 && s.kp % 8 == 0 && s.vp % 8 == 0 && s.window > 0 && s.keep >= 0 &&
+         s.softcap >= 0.f && (s.sink == nullptr || s.maps == 1);
+}
+
+constexpr float LOG2E = 1.4426950408889634f;
+
+// cap tanh(x / cap) log2(e) for x = score * scale: tanh(z) = 1 - 2 / (1 + exp(2 z)), whose error is one of rounding in the result's own
+// scale.  slope = 2 log2(e) scale / cap, top = cap log2(e).
+__device__ __forceinline__ float capped_log2(float score, float slope, float top) {
+  return fmaf(-2.f * top, __fdividef(1.f, 1.f + exp2f(score * slope)), top);
 }
 
 }  // namespace b200

@@ -8,6 +8,8 @@
 // Key tiles of 128 positions start at multiples of 128 and are copied as one TMA box per page and 64 columns (a box may bring
 // columns of the next head: the query's pad is zero, and outputs past vdim are not stored).  Value rows past the request's
 // last token are zeroed in shared memory before the product.
+// A CTA walks the tiles of the kept first positions (both query tiles see them), then those of its window.
+//   CAP   scores are capped softly in the second pass (the cap is monotone, so the row maximum is taken of the raw scores)
 //   BIAS  a table per head and distance (shared memory) is added to the scaled scores, which go back to tensor memory for the
 //         second pass; distances from the table's last entry on read that entry
 #include "grouped_attention.cuh"
@@ -33,6 +35,8 @@ struct GroupedPrefillParams {
 constexpr int GP_THREADS = 64 + 256;      // TMA warp, MMA warp, 4 + 4 softmax warps
 constexpr int GP_LUT_PAD = 254;           // table entries in front of distance 0 (keys of a tile that lie behind a query)
 
+enum GroupedScores : int { SCORES_PLAIN = 0, SCORES_BIAS = 1, SCORES_CAP = 2 };
+
 template <int P, bool BIAS>
 struct GroupedPrefillSmem {
   static constexpr int TILE = 128 * 64 * P * 2;
@@ -47,6 +51,11 @@ struct GroupedPrefillSmem {
 __device__ __forceinline__ float gp_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float gp_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
 __device__ __forceinline__ float gp_sigmoid(float g) {     // (1 + tanh(g / 2)) / 2, one special-function instruction
@@ -107,9 +116,10 @@ __device__ __forceinline__ void gp_store(const GroupedPrefillParams& p, __nv_bfl
   }
 }
 
-template <int P, int MAPS, bool BIAS>
+template <int P, int MAPS, int SCORES>
 __global__ void __launch_bounds__(GP_THREADS, 1)
 grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv, const GroupedPrefillParams p) {
+  constexpr bool BIAS = SCORES == SCORES_BIAS, CAP = SCORES == SCORES_CAP;
   using L = GroupedPrefillSmem<P, BIAS>;
   extern __shared__ uint8_t gp_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(gp_raw) + 1023) & ~uintptr_t(1023));
@@ -156,8 +166,8 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
   const int row_base = p.cu[b], seq_len = p.cu[b + 1] - row_base;
   const int shift = seq_len > 0 ? p.positions[row_base] : 0;            // position of query 0
   const int last_pos = shift + seq_len - 1;
-  // tile X covers queries [q0[X], q0[X] + 128) and key tiles lo_t[X] .. n_kv_t[X] - 1; A's range starts and ends no later than
-  // B's and the two leave no gap
+  // tile X covers queries [q0[X], q0[X] + 128) and walks the steps lo_t[X] .. n_kv_t[X] - 1; A's range starts and ends no later than
+  // B's and the two leave no gap.  Step j is key tile j + (j < kept ? 0 : skip): with kept positions, B starts with them as A does.
   const int q0_t[2] = {MAPS == 1 ? blk * 256 : blk * 128, MAPS == 1 ? blk * 256 + 128 : blk * 128};
   int n_kv_t[2], lo_t[2];
 #pragma unroll
@@ -165,7 +175,16 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     n_kv_t[x] = q0_t[x] < seq_len ? (min(q0_t[x] + 128, seq_len) + shift + 127) / 128 : 0;
     lo_t[x] = n_kv_t[x] > 0 ? max(0, q0_t[x] + shift - s.window + 1) / 128 : 0;
   }
+  const int kept = min((s.keep + 127) / 128, lo_t[0]), skip = kept > 0 ? lo_t[0] - kept : 0;
+  if (s.keep > 0) {
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      n_kv_t[x] -= n_kv_t[x] > 0 ? skip : 0;
+      lo_t[x] = 0;
+    }
+  }
   const int n_kv = max(n_kv_t[0], n_kv_t[1]), j0 = lo_t[0];
+  auto key_tile = [&](int j) { return j < kept ? j : j + skip; };
   const bool active = n_kv > 0;
   if (BIAS && active) {
     const float* row = p.bias + (long long)h * p.bias_len;
@@ -198,7 +217,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         const int i = j - j0;
         int page = 0;
         if (lane < pages) {
-          const int pg = min(j * pages + lane, last_page);              // past the end: something valid
+          const int pg = min(key_tile(j) * pages + lane, last_page);              // past the end: something valid
           page = pg < p.max_pages ? p.tables[(long long)b * p.max_pages + pg] : -1;
           if ((unsigned)page >= (unsigned)p.num_pages) {
             report_bad_arg(p.status, 19);
@@ -312,6 +331,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     const uint32_t tm_s = tmem_base + x * 128 + lane_addr;
     const uint32_t tm_o = tmem_base + 256 + x * 128 + lane_addr;
     const float scale2 = BIAS ? 1.f : p.scale_log2;       // of what the second pass finds in tensor memory
+    const float slope = CAP ? 2.f * p.scale_log2 / s.softcap : 0.f, top = s.softcap * LOG2E;      // see capped_log2
     float m_run = -INFINITY, l_run = 0.f;                 // running reference max in scaled log2 units, row sum relative to it
     bool ok = true;
     const __nv_bfloat16* grow = p.gate != nullptr && q_idx < seq_len ? p.gate + (long long)(row_base + q_idx) * p.ld_gate + h * s.vdim : nullptr;
@@ -320,13 +340,14 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     for (int j = lo_x; j < n_kv_x; ++j) {
       if (!mbar_wait(&s_full[x], (j - lo_x) & 1, abort_word)) { ok = false; break; }
       tc_fence_after();
-      const int k0 = j * 128;
+      const int k0 = key_tile(j) * 128;
       // tile touches the diagonal or the lower edge of the window (warp-uniform)
       const bool edge = (k0 + 127 > q0 + shift) || (k0 <= q0 + 127 + shift - s.window);
+      const int kept_e = min(s.keep - k0, q_key - k0 + 1);      // keys k0 + e with e below are visible wherever the window is
       // Key k0 + e is visible iff e - first <= span as unsigned numbers (one comparison for both edges of the window).
       const int first = q_key - s.window + 1 - k0;
       const uint32_t span = (uint32_t)(s.window - 1);
-      auto hidden = [&](int e) { return (uint32_t)(e - first) > span; };
+      auto hidden = [&](int e) { return (uint32_t)(e - first) > span && e >= kept_e; };
       float mx = -INFINITY;
       // pass 1: row maximum (plain: over the raw scores; BIAS: scores in log2 units with the bias, written back)
       const float* bp = nullptr;
@@ -361,7 +382,8 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       };
       if (edge) row_max(true);
       else row_max(false);
-      if (!BIAS) mx *= p.scale_log2;
+      if (CAP) mx = capped_log2(mx, slope, top);             // (no key: -cap, below or equal to what any key would give)
+      else if (!BIAS) mx *= p.scale_log2;
       // Lazy rescale: keep the old reference max unless it moved by more than 8 (a factor 256).
       float m_new = m_run;
       if (mx > m_run + 8.f) m_new = mx;
@@ -408,7 +430,13 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
             float x0, x1;
-            gp_fma2(x0, x1, __uint_as_float(sc[i]), __uint_as_float(sc[i + 1]), scale2, -m_ref);
+            if (CAP) {
+              x0 = gp_exp2(__uint_as_float(sc[i]) * slope);
+              x1 = gp_exp2(__uint_as_float(sc[i + 1]) * slope);
+              gp_fma2(x0, x1, gp_rcp(1.f + x0), gp_rcp(1.f + x1), -2.f * top, top - m_ref);
+            } else {
+              gp_fma2(x0, x1, __uint_as_float(sc[i]), __uint_as_float(sc[i + 1]), scale2, -m_ref);
+            }
             float e0 = gp_exp2(x0), e1 = gp_exp2(x1);
             if (!BIAS && masked) {                       // (BIAS: hidden keys are -inf already)
               e0 = hidden(c * 32 + i) ? 0.f : e0;
@@ -438,6 +466,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       if (ok && n_kv_x > 0) ok = mbar_wait(&o_full[x], 0, abort_word);
       if (ok && n_kv_x > 0) {
         tc_fence_after();
+        if (s.sink != nullptr) l_run += gp_exp2(fminf(fmaf(s.sink[h], LOG2E, -m_run), 126.f));
         const float inv_l = 1.f / l_run;
 #pragma unroll 1
         for (int c = 0; c < 2 * P; ++c) {
@@ -505,10 +534,10 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
   }
 }
 
-template <int P, int MAPS, bool BIAS>
+template <int P, int MAPS, int SCORES>
 static int launch_grouped_prefill(const CUtensorMap& tm_q, const CUtensorMap& tm_kv, const GroupedPrefillParams& p, cudaStream_t st) {
-  const int smem = GroupedPrefillSmem<P, BIAS>::total(p.bias_len);
-  auto kern = grouped_prefill_kernel<P, MAPS, BIAS>;
+  const int smem = GroupedPrefillSmem<P, SCORES == SCORES_BIAS>::total(p.bias_len);
+  auto kern = grouped_prefill_kernel<P, MAPS, SCORES>;
   static int configured = 0;
   if (smem > configured) {
     if (smem > 232448 || cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
@@ -526,7 +555,7 @@ using namespace b200;
 
 // q: (total_q, heads * maps * qp) with qp a multiple of 64, portion b in rows cu[b] .. cu[b + 1] - 1 (at most max_q of them), its first
 // query at position positions[cu[b]]; line b of the tables holds its pages.  dim and vdim up to 128, page_size a divisor of 128 of
-// at least 8, scale positive unless there is a bias, bias_len at most B200_GROUPED_BIAS_MAX.
+// at least 8, a softcap only for one map and without a bias, scale positive unless there is a bias, bias_len at most B200_GROUPED_BIAS_MAX.
 constexpr int B200_GROUPED_BIAS_MAX = 6000;
 
 extern "C" int b200_grouped_prefill(const void* q, const void* cache, void* o, long long ld_o, const void* gate, long long ld_gate,
@@ -536,6 +565,7 @@ extern "C" int b200_grouped_prefill(const void* q, const void* cache, void* o, l
   if (portions <= 0 || total_q <= 0) return 0;
   if (!shape_ok(*s) || s->dim > 128 || s->vdim > 128 || s->qp % 64 || page_size < 8 || 128 % page_size || max_q <= 0) return -10;
   if (bias != nullptr ? (bias_len <= 0 || bias_len > B200_GROUPED_BIAS_MAX) : !(s->scale > 0.f)) return -11;
+  if (s->softcap > 0.f && (bias != nullptr || s->maps != 1)) return -12;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15) return -10;
   const uint64_t qw = (uint64_t)s->heads * s->maps * s->qp, width = (uint64_t)s->kv_heads * (s->maps * s->kp + s->vp);
   CUtensorMap tm_q, tm_kv;
@@ -549,13 +579,15 @@ extern "C" int b200_grouped_prefill(const void* q, const void* cache, void* o, l
   p.out_vec = s->vdim % 8 == 0 && ld_o % 8 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0;
   p.gate_vec = s->vdim % 8 == 0 && ld_gate % 8 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0;
   const bool wide = s->dim > 64 || s->vdim > 64;
-#define GROUPED_PREFILL(MAPS, BIAS) \
-  return wide ? launch_grouped_prefill<2, MAPS, BIAS>(tm_q, tm_kv, p, st) : launch_grouped_prefill<1, MAPS, BIAS>(tm_q, tm_kv, p, st)
+#define GROUPED_PREFILL(MAPS, SCORES)                                          \
+  return wide ? launch_grouped_prefill<2, MAPS, SCORES>(tm_q, tm_kv, p, st)    \
+              : launch_grouped_prefill<1, MAPS, SCORES>(tm_q, tm_kv, p, st)
   if (s->maps == 1) {
-    if (bias != nullptr) GROUPED_PREFILL(1, true);
-    GROUPED_PREFILL(1, false);
+    if (bias != nullptr) GROUPED_PREFILL(1, SCORES_BIAS);
+    if (s->softcap > 0.f) GROUPED_PREFILL(1, SCORES_CAP);
+    GROUPED_PREFILL(1, SCORES_PLAIN);
   }
-  if (bias != nullptr) GROUPED_PREFILL(2, true);
-  GROUPED_PREFILL(2, false);
+  if (bias != nullptr) GROUPED_PREFILL(2, SCORES_BIAS);
+  GROUPED_PREFILL(2, SCORES_PLAIN);
 #undef GROUPED_PREFILL
 }

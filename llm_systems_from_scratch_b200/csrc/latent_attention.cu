@@ -3,7 +3,11 @@
 // GEMM per head): score = q'_h . c * scale, and sum_j p_j c_j goes through W_uv,h afterwards.  Every cached byte is then
 // read once for all heads.  The mask is a sliding window: position i sees the `window` positions up to and including i.
 //
-// Cache layout per layer run: (num_pages, page_size, width), width = latent size rounded up to 8 elements, zero padded.
+// A rotated key part shared by all heads may follow the latent: the score gains q_rot,h . k_rot, so a query in latent space is
+// [q'_h, q_rot,h], a cached vector [c, k_rot], and only c is summed up.
+//
+// Cache layout per layer run: (num_pages, page_size, width), width = vwidth + rotated part, each rounded up to 8 elements, zero padded
+// (vwidth: the latent).
 #include "typed.cuh"
 
 namespace b200 {
@@ -71,6 +75,117 @@ __global__ void __launch_bounds__(256) latent_norm_append_kernel(
   }
 }
 
+// Rotation of interleaved pairs (elements 2i and 2i + 1) and append.  One block per row: warp 0 norms the latent and rotates the key
+// part on their way to the cache, the other warps rotate the heads' query parts: for the first `absorbed` rows behind the queries in
+// latent space, for the others in place.
+struct LatentRotateParams {
+  void* q;                     // (rows, ld_q)
+  const void* kv;              // (rows, ld_kv)
+  long long ld_q, ld_kv;
+  int q_col, q_pitch;          // rotated part of head h: columns q_col + h * q_pitch ... of q
+  int kv_col;                  // the latent's first column of kv, negative: no latent here
+  int k_col;                   // the key part's first column of kv, negative: none
+  const void* wkv;
+  void* ql;                    // (absorbed, heads * width)
+  void* cache;
+  const float* cos_sin;        // (2, ctx, rot / 2)
+  const int* positions;
+  const long long* slots;
+  int rows, absorbed, heads, kv_rank, vwidth, width, rot, ctx;
+  long long num_slots;
+  float eps;
+  uint32_t* status;
+};
+
+// VEC elements (whole pairs) of a rotated vector: src -> dst
+template <typename T, int VEC>
+__device__ __forceinline__ void rotate_pairs(const T* src, T* dst, const float* cs, const float* sn) {
+  float f[VEC];
+  if constexpr (VEC == 4) {
+    load_vec<4>(src, f);
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) f[i] = to_f(src[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < VEC; i += 2) {
+    const float c = cs[i / 2], s = sn[i / 2], u = f[i], v = f[i + 1];
+    f[i] = u * c - v * s;
+    f[i + 1] = v * c + u * s;
+  }
+  if constexpr (VEC == 4) {
+    store_vec<4>(dst, f);
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) from_f(dst[i], f[i]);
+  }
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) latent_rotate_kernel(const LatentRotateParams p) {
+  pdl_sync();
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  T* pr = reinterpret_cast<T*>(p.q) + (long long)row * p.ld_q;
+  const T* kr = reinterpret_cast<const T*>(p.kv) + (long long)row * p.ld_kv;
+  int pos = p.positions[row];
+  if (pos < 0 || pos >= p.ctx) {
+    if (threadIdx.x == 0) report_bad_arg(p.status, 21);
+    pos = 0;
+  }
+  const int half = p.rot / 2;
+  const float* cs = p.cos_sin + (long long)pos * half;
+  const float* sn = cs + (long long)p.ctx * half;
+  if (warp > 0) {
+    const int per = p.rot / VEC, total = p.heads * per;
+    for (int i = threadIdx.x - 32; i < total; i += blockDim.x - 32) {
+      const int h = i / per, c = (i - h * per) * VEC;
+      T* src = pr + p.q_col + h * p.q_pitch + c;
+      T* dst = row < p.absorbed ? reinterpret_cast<T*>(p.ql) + ((long long)row * p.heads + h) * p.width + p.vwidth + c : src;
+      rotate_pairs<T, VEC>(src, dst, cs + c / 2, sn + c / 2);
+    }
+    const int pad = p.width - p.vwidth - p.rot;
+    if (row < p.absorbed)
+      for (int i = threadIdx.x - 32; i < p.heads * pad; i += blockDim.x - 32)
+        from_f(reinterpret_cast<T*>(p.ql)[((long long)row * p.heads + i / pad) * p.width + p.vwidth + p.rot + i % pad], 0.f);
+    return;
+  }
+  const long long slot = p.slots[row];
+  if (slot < 0) return;                       // padding row of the batch
+  if (slot >= p.num_slots) {
+    if (lane == 0) report_bad_arg(p.status, 22);
+    return;
+  }
+  T* dst = reinterpret_cast<T*>(p.cache) + slot * p.width;
+  if (p.k_col >= 0) {
+    for (int c = lane * VEC; c < p.rot; c += 32 * VEC) rotate_pairs<T, VEC>(kr + p.k_col + c, dst + p.vwidth + c, cs + c / 2, sn + c / 2);
+    for (int c = p.vwidth + p.rot + lane; c < p.width; c += 32) from_f(dst[c], 0.f);
+  }
+  if (p.kv_col < 0) return;
+  constexpr int LV = VEC == 4 ? 4 : 1;
+  const T* src = kr + p.kv_col;
+  float ss = 0.f;
+#pragma unroll 4
+  for (int c = lane * LV; c < p.kv_rank; c += 32 * LV) {
+    float f[LV];
+    load_vec<LV>(src + c, f);
+#pragma unroll
+    for (int i = 0; i < LV; ++i) ss += f[i] * f[i];
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float r = rsqrtf(ss / (float)p.kv_rank + p.eps);
+#pragma unroll 4
+  for (int c = lane * LV; c < p.kv_rank; c += 32 * LV) {
+    float f[LV], g[LV];
+    load_vec<LV>(src + c, f);
+    load_vec<LV>(reinterpret_cast<const T*>(p.wkv) + c, g);
+#pragma unroll
+    for (int i = 0; i < LV; ++i) f[i] = f[i] * r * g[i];
+    store_vec<LV>(dst + c, f);
+  }
+  for (int c = p.kv_rank + lane; c < p.vwidth; c += 32) from_f(dst[c], 0.f);
+}
+
 // Latents of the keys that the portions of a step can see, packed for the prefill kernel:
 //   out[cu_k[b] + i] = latent of position first_k[b] + i of portion b
 template <typename T>
@@ -102,12 +217,12 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(
 }
 
 // General form, any head count, any width, T = bf16 or fp32: one warp per (row, head), keys one after the other.
-// q / o: (rows, heads * width).  row_seq[row] names the row's line of `tables`.
+// q: (rows, heads * width), o: (rows, heads * vwidth).  row_seq[row] names the row's line of `tables`.
 template <typename T>
 __global__ void __launch_bounds__(128) latent_attn_rows_kernel(
     const T* __restrict__ q, const T* __restrict__ cache, T* __restrict__ o, const int* __restrict__ row_seq,
     const int* __restrict__ positions, const long long* __restrict__ slots, const int* __restrict__ tables, int seqs,
-    int rows, int heads, int width, int max_pages, int page_size, int num_pages, int window, float scale,
+    int rows, int heads, int width, int vwidth, int max_pages, int page_size, int num_pages, int window, float scale,
     uint32_t* __restrict__ status) {
   pdl_sync();
   extern __shared__ float lsm[];
@@ -118,7 +233,7 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(
   float* qs = lsm + warp * 2 * width;
   float* acc = qs + width;
   const T* qr = q + ((long long)row * heads + h) * width;
-  T* orow = o + ((long long)row * heads + h) * width;
+  T* orow = o + ((long long)row * heads + h) * vwidth;
   for (int c = lane; c < width; c += 32) { qs[c] = to_f(qr[c]) * scale; acc[c] = 0.f; }
   float m = -INFINITY, l = 0.f;
   const int seq = row_seq != nullptr ? row_seq[row] : row;
@@ -142,12 +257,12 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(
       const float mn = fmaxf(m, s);
       const float a = expf(m - mn), e = expf(s - mn);      // first key: exp(-inf) = 0
       l = l * a + e;
-      for (int i = lane; i < width; i += 32) acc[i] = acc[i] * a + e * to_f(c[i]);
+      for (int i = lane; i < vwidth; i += 32) acc[i] = acc[i] * a + e * to_f(c[i]);
       m = mn;
     }
   }
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int c = lane; c < width; c += 32) from_f(orow[c], acc[c] * inv);
+  for (int c = lane; c < vwidth; c += 32) from_f(orow[c], acc[c] * inv);
 }
 
 // ------------------------------------------------------------------------------- decode, bf16, on the tensor cores
@@ -188,29 +303,30 @@ __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
 struct LatentDecodeParams {
   const __nv_bfloat16* q;       // (rows, heads * width)
   const __nv_bfloat16* cache;
-  __nv_bfloat16* o;             // (rows, heads * width)
-  float* part_o;                // (rows, heads, splits, width) when splits > 1
+  __nv_bfloat16* o;             // (rows, heads * vwidth)
+  float* part_o;                // (rows, heads, splits, vwidth) when splits > 1
   float* part_ml;               // (rows, heads, splits, 2)
   const int* positions;
   const long long* slots;
   const int* tables;            // line i for row i
-  int rows, heads, width, max_pages, page_size, num_pages, window, splits;
+  int rows, heads, width, vwidth, max_pages, page_size, num_pages, window, splits;
   float scale_log2;
   uint32_t* status;
 };
 
-template <int NT>
+template <int KT>
 struct LatentDecodeSmem {
-  static constexpr int KP = NT * 64;            // latent columns, padded
+  static constexpr int KP = KT * 64;            // columns of a cached vector, padded
   static constexpr int PITCH = KP + 8;          // an odd number of 16-byte pieces: ldmatrix without bank conflicts
   static constexpr int bytes(int hg) {
     return LD_STAGES * LD_BT * PITCH * 2 + hg * 16 * (2 * (LD_BT + 4) * 4 + (LD_BT + 8) * 2 + 8);
   }
 };
 
-template <int NT, int HG>
-__global__ void __launch_bounds__(256 * HG, HG == 1 ? 2 : 1) latent_decode_kernel(const LatentDecodeParams p) {
-  using L = LatentDecodeSmem<NT>;
+// KT, NT: 64-column pieces of a cached vector and of the part of it that is summed up
+template <int KT, int NT, int HG>
+__global__ void __launch_bounds__(256 * HG, HG == 1 && KT <= 8 ? 2 : 1) latent_decode_kernel(const LatentDecodeParams p) {
+  using L = LatentDecodeSmem<KT>;
   constexpr int KP = L::KP, PITCH = L::PITCH, M = HG * 16, SP = LD_BT + 4, PP = LD_BT + 8, THREADS = 256 * HG;
   constexpr int ROWS = LD_BT / (8 * HG);                                    // token rows a warp copies per tile
   extern __shared__ __align__(16) uint8_t ld_smem[];
@@ -284,12 +400,12 @@ __global__ void __launch_bounds__(256 * HG, HG == 1 ? 2 : 1) latent_decode_kerne
   long long next_src = LD_STAGES - 1 < tiles ? look_up(LD_STAGES - 1) : -1;
   asm volatile("cp.async.wait_group %0;" ::"n"(LD_STAGES - 1) : "memory");  // the queries have landed
   __syncthreads();
-  uint32_t qf[NT * 2][4];                  // A fragments of this group's 16 heads, this warp's half of the columns
+  uint32_t qf[KT * 2][4];                  // A fragments of this group's 16 heads, this warp's half of the columns
   {
     const uint32_t a_addr = smem_u32(sc + ((LD_STAGES - 1) * LD_BT + grp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PITCH +
-                                     kh * NT * 32 + (lane >> 4) * 8);
+                                     kh * KT * 32 + (lane >> 4) * 8);
 #pragma unroll
-    for (int k = 0; k < NT * 2; ++k) ldsm_x4(qf[k], a_addr + k * 32);
+    for (int k = 0; k < KT * 2; ++k) ldsm_x4(qf[k], a_addr + k * 32);
   }
   float acc[NT][4];
 #pragma unroll
@@ -310,9 +426,9 @@ __global__ void __launch_bounds__(256 * HG, HG == 1 ? 2 : 1) latent_decode_kerne
     const __nv_bfloat16* c = sc + (it % LD_STAGES) * LD_BT * PITCH;
     // ---- scores of 8 tokens for the group's heads
     float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-    const uint32_t b_addr = smem_u32(c + (tq * 8 + (lane & 7)) * PITCH + kh * NT * 32 + (lane >> 3) * 8);
+    const uint32_t b_addr = smem_u32(c + (tq * 8 + (lane & 7)) * PITCH + kh * KT * 32 + (lane >> 3) * 8);
 #pragma unroll
-    for (int k = 0; k < NT; ++k) {
+    for (int k = 0; k < KT; ++k) {
       uint32_t b[4];
       ldsm_x4(b, b_addr + k * 64);
       mma_bf16(s0, qf[2 * k], b[0], b[1]);
@@ -388,13 +504,13 @@ __global__ void __launch_bounds__(256 * HG, HG == 1 ? 2 : 1) latent_decode_kerne
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       const int col = wq * (NT * 8) + j * 8 + (lane & 3) * 2;
-      if (col >= p.width) continue;
+      if (col >= p.vwidth) continue;
       const float x = acc[j][half * 2], y = acc[j][half * 2 + 1];
       if (p.splits > 1)
-        *reinterpret_cast<float2*>(p.part_o + (((long long)row * p.heads + h0 + r) * p.splits + split) * p.width + col) =
+        *reinterpret_cast<float2*>(p.part_o + (((long long)row * p.heads + h0 + r) * p.splits + split) * p.vwidth + col) =
             make_float2(x, y);
       else
-        *reinterpret_cast<uint32_t*>(p.o + ((long long)row * p.heads + h0 + r) * p.width + col) = pack_bf16x2(x * inv, y * inv);
+        *reinterpret_cast<uint32_t*>(p.o + ((long long)row * p.heads + h0 + r) * p.vwidth + col) = pack_bf16x2(x * inv, y * inv);
     }
   }
 }
@@ -426,10 +542,10 @@ void launch_latent_merge(const float* part_o, const float* part_ml, __nv_bfloat1
   launch_dep(latent_merge_kernel, items, 128, 0, st, part_o, part_ml, o, splits, width);
 }
 
-template <int NT, int HG>
+template <int KT, int NT, int HG>
 static int launch_latent_decode(const LatentDecodeParams& p, cudaStream_t st) {
-  constexpr int smem = LatentDecodeSmem<NT>::bytes(HG);
-  auto kern = latent_decode_kernel<NT, HG>;
+  constexpr int smem = LatentDecodeSmem<KT>::bytes(HG);
+  auto kern = latent_decode_kernel<KT, NT, HG>;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -3;
@@ -437,8 +553,13 @@ static int launch_latent_decode(const LatentDecodeParams& p, cudaStream_t st) {
   }
   launch_dep(kern, dim3(p.rows, (p.heads + HG * 16 - 1) / (HG * 16), p.splits), 256 * HG, smem, st, p);
   if (p.splits > 1)
-    launch_latent_merge(p.part_o, p.part_ml, p.o, p.rows * p.heads, p.splits, p.width, st);
+    launch_latent_merge(p.part_o, p.part_ml, p.o, p.rows * p.heads, p.splits, p.vwidth, st);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <int KT, int NT>
+static int launch_latent_decode_heads(const LatentDecodeParams& p, cudaStream_t st) {
+  return p.heads > 16 ? launch_latent_decode<KT, NT, 2>(p, st) : launch_latent_decode<KT, NT, 1>(p, st);
 }
 
 }  // namespace b200
@@ -471,6 +592,36 @@ extern "C" int b200_latent_norm_append(const void* proj, long long ld_proj, cons
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
+// See LatentRotateParams.  kv_rank <= vwidth <= width - rot; kv_col, k_col negative: the cache keeps what it has.
+extern "C" int b200_latent_rotate(void* q, long long ld_q, const void* kv, long long ld_kv, int q_col, int q_pitch, int kv_col, int k_col, const void* wkv, void* ql,
+                                  int absorbed, void* cache, const float* cos_sin, const int* positions, const long long* slots,
+                                  int rows, int heads, int kv_rank, int vwidth, int width, int rot, int ctx, long long num_slots,
+                                  float eps, int f32, uint32_t* status, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (heads <= 0 || rot <= 0 || (rot & 1) || q_pitch < rot || kv_rank <= 0 || vwidth < kv_rank || width < vwidth + rot ||
+      cos_sin == nullptr || ((kv_col >= 0 || k_col >= 0) && kv == nullptr) || (kv_col >= 0 && wkv == nullptr) || (absorbed > 0 && ql == nullptr))
+    return -10;
+  LatentRotateParams p;
+  p.q = q; p.ld_q = ld_q; p.kv = kv; p.ld_kv = ld_kv; p.q_col = q_col; p.q_pitch = q_pitch; p.kv_col = kv_col; p.k_col = k_col; p.wkv = wkv; p.ql = ql;
+  p.cache = cache; p.cos_sin = cos_sin; p.positions = positions; p.slots = slots; p.rows = rows; p.absorbed = absorbed;
+  p.heads = heads; p.kv_rank = kv_rank; p.vwidth = vwidth; p.width = width; p.rot = rot; p.ctx = ctx; p.num_slots = num_slots;
+  p.eps = eps; p.status = status;
+  const bool vec = (rot | kv_rank | q_pitch | q_col | vwidth | width) % 4 == 0 && (kv_col < 0 || kv_col % 4 == 0) &&
+                   (k_col < 0 || k_col % 4 == 0) && (ld_q | ld_kv) % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(ql) | reinterpret_cast<uintptr_t>(cache) |
+                     reinterpret_cast<uintptr_t>(wkv)) & 15) == 0;
+  int threads = 32 + (heads * (rot / (vec ? 4 : 2)) + 31) / 32 * 32;
+  if (threads > 256) threads = 256;
+  if (f32) {
+    if (vec) launch_dep(latent_rotate_kernel<float, 4>, rows, threads, 0, st, p);
+    else launch_dep(latent_rotate_kernel<float, 2>, rows, threads, 0, st, p);
+  } else {
+    if (vec) launch_dep(latent_rotate_kernel<__nv_bfloat16, 4>, rows, threads, 0, st, p);
+    else launch_dep(latent_rotate_kernel<__nv_bfloat16, 2>, rows, threads, 0, st, p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
 // bf16 caches only (the packed latents feed the tensor-core prefill).
 extern "C" int b200_latent_gather(const void* cache, void* out, const int* cu_k, const int* first_k, const int* tables,
                                   int portions, int total_rows, int max_pages, int page_size, int num_pages, int width,
@@ -487,11 +638,11 @@ extern "C" int b200_latent_gather(const void* cache, void* out, const int* cu_k,
 
 // window <= 0: no window.  row_seq null: row i uses line i of the tables.
 extern "C" int b200_latent_attn_rows(const void* q, const void* cache, void* o, const int* row_seq, const int* positions,
-                                     const long long* slots, const int* tables, int seqs, int rows, int heads, int width,
+                                     const long long* slots, const int* tables, int seqs, int rows, int heads, int width, int vwidth,
                                      int max_pages, int page_size, int num_pages, int window, float scale, int f32,
                                      uint32_t* status, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (heads <= 0 || width <= 0 || page_size <= 0 || width > 6144) return -10;
+  if (heads <= 0 || width <= 0 || vwidth <= 0 || vwidth > width || page_size <= 0 || width > 6144) return -10;
   const unsigned grid = (unsigned)(((long long)rows * heads + 3) / 4);
   const size_t smem = 4ull * 2 * width * sizeof(float);
   if (f32) {
@@ -499,36 +650,39 @@ extern "C" int b200_latent_attn_rows(const void* q, const void* cache, void* o, 
                                                  (int)smem) != cudaSuccess)
       return -3;
     launch_dep(latent_attn_rows_kernel<float>, grid, 128, smem, st, (const float*)q, (const float*)cache, (float*)o, row_seq,
-               positions, slots, tables, seqs, rows, heads, width, max_pages, page_size, num_pages, window, scale, status);
+               positions, slots, tables, seqs, rows, heads, width, vwidth, max_pages, page_size, num_pages, window, scale, status);
   } else {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(latent_attn_rows_kernel<__nv_bfloat16>,
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return -3;
     launch_dep(latent_attn_rows_kernel<__nv_bfloat16>, grid, 128, smem, st, (const __nv_bfloat16*)q,
                (const __nv_bfloat16*)cache, (__nv_bfloat16*)o, row_seq, positions, slots, tables, seqs, rows, heads, width,
-               max_pages, page_size, num_pages, window, scale, status);
+               vwidth, max_pages, page_size, num_pages, window, scale, status);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-// Decode on the tensor cores: bf16, one query row per line of the tables, width a multiple of 8 up to 512.  splits > 1 needs
-// part_o (rows * heads * splits * width floats) and part_ml (rows * heads * splits * 2 floats).
+// Decode on the tensor cores: bf16, one query row per line of the tables, width and vwidth multiples of 8, vwidth up to 512, width up to
+// 576.  splits > 1 needs part_o (rows * heads * splits * vwidth floats) and part_ml (rows * heads * splits * 2 floats).
 extern "C" int b200_latent_decode(const void* q, const void* cache, void* o, float* part_o, float* part_ml,
                                   const int* positions, const long long* slots, const int* tables, int rows, int heads,
-                                  int width, int max_pages, int page_size, int num_pages, int window, int splits,
+                                  int width, int vwidth, int max_pages, int page_size, int num_pages, int window, int splits,
                                   float scale, uint32_t* status, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (width % 8 || width <= 0 || width > 512 || heads <= 0 || page_size <= 0 || splits < 1 || splits > 65535) return -10;
+  if (width % 8 || vwidth % 8 || vwidth <= 0 || vwidth > 512 || width < vwidth || width > 576 || heads <= 0 || page_size <= 0 ||
+      splits < 1 || splits > 65535)
+    return -10;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(o)) & 15) return -10;
   if (splits > 1 && (part_o == nullptr || part_ml == nullptr)) return -11;
   LatentDecodeParams p;
   p.q = (const __nv_bfloat16*)q; p.cache = (const __nv_bfloat16*)cache; p.o = (__nv_bfloat16*)o;
   p.part_o = part_o; p.part_ml = part_ml; p.positions = positions; p.slots = slots; p.tables = tables;
-  p.rows = rows; p.heads = heads; p.width = width; p.max_pages = max_pages; p.page_size = page_size;
+  p.rows = rows; p.heads = heads; p.width = width; p.vwidth = vwidth; p.max_pages = max_pages; p.page_size = page_size;
   p.num_pages = num_pages; p.window = window; p.splits = splits; p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
-  const bool wide = heads > 16;
-  if (width <= 128) return wide ? launch_latent_decode<2, 2>(p, st) : launch_latent_decode<2, 1>(p, st);
-  if (width <= 256) return wide ? launch_latent_decode<4, 2>(p, st) : launch_latent_decode<4, 1>(p, st);
-  return wide ? launch_latent_decode<8, 2>(p, st) : launch_latent_decode<8, 1>(p, st);
+  if (width <= 128) return launch_latent_decode_heads<2, 2>(p, st);
+  if (width <= 256) return launch_latent_decode_heads<4, 4>(p, st);
+  if (width <= 320 && vwidth <= 256) return launch_latent_decode_heads<5, 4>(p, st);
+  if (width <= 512) return launch_latent_decode_heads<8, 8>(p, st);
+  return launch_latent_decode_heads<9, 8>(p, st);
 }

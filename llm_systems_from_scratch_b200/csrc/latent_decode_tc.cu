@@ -5,6 +5,8 @@
 // does.  Here the TOKENS are the M dimension, so the heads only have to fill N (16, 32 or 64):
 //     S^T (128 tokens x heads)        = C (tokens x latent)  Q^T            A = C, K-major
 //     O^T (128 latent dims x heads)  += C^T (latent x tokens) P^T           A = C, MN-major, the same shared memory
+// A rotated key part behind the latent (up to 64 columns) is a stage of its own that only takes part in the scores.  It comes first in
+// a tile, so that its place in the ring is free again before the tile's last latents need one.
 // One CTA = one request and one split of its window, in tiles of 128 tokens that start on page borders.
 //   warp 0      TMA producer: pages -> a ring of stages of 128 tokens x 128 latent columns (one box per page and 64 columns;
 //               the lanes issue one page each; pages of 64 tokens keep the number of boxes small)
@@ -21,13 +23,13 @@ int make_tmap_bf16_2d(CUtensorMap* tm, const void* ptr, uint64_t rows, uint64_t 
 
 struct LatentTcParams {
   const __nv_bfloat16* q;       // (rows, heads * width)
-  __nv_bfloat16* o;             // (rows, heads * width)
-  float* part_o;                // (rows, heads, splits, width) when splits > 1
+  __nv_bfloat16* o;             // (rows, heads * vwidth)
+  float* part_o;                // (rows, heads, splits, vwidth) when splits > 1
   float* part_ml;               // (rows, heads, splits, 2)
   const int* positions;
   const long long* slots;
   const int* tables;
-  int rows, heads, width, max_pages, page_size, num_pages, window, splits;
+  int rows, heads, width, vwidth, max_pages, page_size, num_pages, window, splits;
   float scale_log2;
   uint32_t* status;
 };
@@ -46,8 +48,8 @@ template <int HN>
 struct LatentTcSmem {
   static constexpr int STAGES = HN == 16 ? 6 : (HN == 32 ? 5 : 4);
   static constexpr int STAGE = 32768;                    // two panels of 128 tokens x 64 latent columns
-  static constexpr int OFF_Q = STAGES * STAGE;           // panels of HN rows x 128 bytes, up to 8
-  static constexpr int OFF_P = OFF_Q + 8 * HN * 128;     // two panels of HN rows x 64 tokens
+  static constexpr int OFF_Q = STAGES * STAGE;           // panels of HN rows x 128 bytes, up to 9
+  static constexpr int OFF_P = OFF_Q + 9 * HN * 128;     // two panels of HN rows x 64 tokens
   static constexpr int OFF_MAX = OFF_P + 2 * HN * 128;   // [4][HN] floats
   static constexpr int OFF_RUN = OFF_MAX + 4 * HN * 4;   // m [HN], alpha [HN], need
   static constexpr int OFF_BAR = OFF_RUN + 2 * HN * 4 + 16;
@@ -147,15 +149,15 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Late
   const int total = live ? (pos + 1 - base + LT_TILE - 1) / LT_TILE : 0;
   const int per = (total + p.splits - 1) / p.splits;
   const int i0 = min(total, split * per), tiles = min(total, i0 + per) - i0;
-  const int nb = p.width / 128;                                 // stages per tile
+  const int nv = p.vwidth / 128, nr = p.width > p.vwidth ? 1 : 0, nb = nv + nr;      // stages per tile: rotated part, latents
   const int t_first = base + i0 * LT_TILE;
 
   if (warp >= 2) {                                              // queries: HN rows, zero beyond the heads
-    const int vecs = p.width / 8;
+    const int vecs = (p.width + 63) / 64 * 8;                   // whole panels, zero beyond the width
     for (int i = threadIdx.x - 64; i < HN * vecs; i += LT_SOFTMAX) {
       const int h = i / vecs, v = i - h * vecs;
       uint4 x = make_uint4(0, 0, 0, 0);
-      if (h < p.heads) x = *reinterpret_cast<const uint4*>(p.q + ((long long)row * p.heads + h) * p.width + v * 8);
+      if (h < p.heads && v * 8 < p.width) x = *reinterpret_cast<const uint4*>(p.q + ((long long)row * p.heads + h) * p.width + v * 8);
       *reinterpret_cast<uint4*>(smem + L::OFF_Q + (v >> 3) * (HN * 128) + h * 128 + (((v & 7) ^ (h & 7)) << 4)) = x;
     }
     if (threadIdx.x - 64 < HN) srun[threadIdx.x - 64] = -INFINITY;
@@ -188,12 +190,14 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Late
           ok = false;
           break;
         }
-        if (lane == 0) mbar_expect_tx(&full[st], L::STAGE);
+        const bool rot = b < nr;
+        if (lane == 0) mbar_expect_tx(&full[st], rot ? L::STAGE / 2 : L::STAGE);
         __syncwarp();
         if (lane < pages) {
           uint8_t* dst = smem + st * L::STAGE + lane * p.page_size * 128;
-          tma_load_2d(dst, &tm_cache, &full[st], b * 128, page * p.page_size);
-          tma_load_2d(dst + 16384, &tm_cache, &full[st], b * 128 + 64, page * p.page_size);
+          const int col = rot ? p.vwidth : (b - nr) * 128;
+          tma_load_2d(dst, &tm_cache, &full[st], col, page * p.page_size);
+          if (!rot) tma_load_2d(dst + 16384, &tm_cache, &full[st], col + 64, page * p.page_size);
         }
         __syncwarp();
       }
@@ -210,11 +214,16 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Late
           if (!ok) break;
           tc_fence_after();
           const uint64_t c = make_smem_desc(smem_u32(smem + st * L::STAGE), 16, 1024);
-          const uint64_t q = make_smem_desc(smem_u32(smem + L::OFF_Q + b * 2 * HN * 128), 16, 1024);
+          const bool rot = b < nr;
+          const uint64_t q = make_smem_desc(smem_u32(smem + L::OFF_Q + (rot ? nv : b - nr) * 2 * HN * 128), 16, 1024);
+          const int ksteps = rot ? (p.width - p.vwidth + 15) / 16 : 8;
 #pragma unroll
-          for (int k = 0; k < 8; ++k)
+          for (int k = 0; k < 8; ++k) {
+            if (k >= ksteps) break;
             umma_f16_ss(tmem, c + (uint32_t)(((k / 4) * 16384 + (k % 4) * 32) >> 4),
                         q + (uint32_t)(((k / 4) * HN * 128 + (k % 4) * 32) >> 4), id_s, (b | k) ? 1u : 0u);
+          }
+          if (rot) umma_commit(&empty[st]);
         }
         if (!ok) break;
         umma_commit(s_full);
@@ -222,8 +231,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Late
         if (!ok) break;
         tc_fence_after();
         const uint64_t pt = make_smem_desc(smem_u32(smem + L::OFF_P), 16, 1024);
-        for (int b = 0; b < nb; ++b) {
-          const int st = (i * nb + b) % ST;
+        for (int b = 0; b < nv; ++b) {
+          const int st = (i * nb + nr + b) % ST;
           const uint64_t ct = make_smem_desc(smem_u32(smem + st * L::STAGE), 16384, 1024);
 #pragma unroll
           for (int k = 0; k < 8; ++k)
@@ -264,8 +273,8 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Late
       if (!mbar_wait(s_full, i & 1, abort_word)) { ok = false; *abort_word = ERR_WAIT_MISC; }
       tc_fence_after();
       if (t > pos) {                   // never written by this request: zero, so that it cannot reach O even as 0 * NaN
-        for (int b = 0; b < nb; ++b) {
-          uint8_t* c = smem + ((i * nb + b) % ST) * L::STAGE + half * 16384 + r * 128;
+        for (int b = 0; b < nv; ++b) {
+          uint8_t* c = smem + ((i * nb + nr + b) % ST) * L::STAGE + half * 16384 + r * 128;
 #pragma unroll
           for (int v = 0; v < 8; ++v) *reinterpret_cast<uint4*>(c + v * 16) = make_uint4(0, 0, 0, 0);
         }
@@ -309,7 +318,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Late
         *reinterpret_cast<__nv_bfloat16*>(p_base + h * 128 + ((p_piece ^ (h & 7)) << 4)) = __float2bfloat16(e);
       }
       if (need && i > 0) {             // S^T(i) was issued after the products of tile i - 1, so those are complete
-        for (int b = 0; b < nb; ++b)
+        for (int b = 0; b < nv; ++b)
 #pragma unroll
           for (int c = 0; c < HH / 8; ++c) {
             uint32_t raw[8];
@@ -344,7 +353,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Late
     softmax_barrier();
     if (tiles > 0 && !mbar_wait(o_full, 0, abort_word)) { ok = false; *abort_word = ERR_WAIT_TMEM_FULL; }
     tc_fence_after();
-    for (int b = 0; b < nb; ++b) {
+    for (int b = 0; b < nv; ++b) {
       float x[HH];
       if (tiles > 0 && ok) {
         load_cols(HN * (1 + b) + hb, x);
@@ -357,9 +366,9 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Late
         const int h = hb + j;
         if (h >= p.heads) break;
         if (p.splits > 1)
-          p.part_o[(((long long)row * p.heads + h) * p.splits + split) * p.width + b * 128 + r] = x[j];
+          p.part_o[(((long long)row * p.heads + h) * p.splits + split) * p.vwidth + b * 128 + r] = x[j];
         else
-          p.o[((long long)row * p.heads + h) * p.width + b * 128 + r] = __float2bfloat16(x[j] * salpha[h]);
+          p.o[((long long)row * p.heads + h) * p.vwidth + b * 128 + r] = __float2bfloat16(x[j] * salpha[h]);
       }
     }
   }
@@ -391,7 +400,7 @@ static int launch_latent_tc(const CUtensorMap& tm, const LatentTcParams& p, cuda
     configured = true;
   }
   launch_dep(kern, dim3(p.rows, p.splits), LT_THREADS, LatentTcSmem<HN>::TOTAL, st, tm, p);
-  if (p.splits > 1) launch_latent_merge(p.part_o, p.part_ml, p.o, p.rows * p.heads, p.splits, p.width, st);
+  if (p.splits > 1) launch_latent_merge(p.part_o, p.part_ml, p.o, p.rows * p.heads, p.splits, p.vwidth, st);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -399,14 +408,14 @@ static int launch_latent_tc(const CUtensorMap& tm, const LatentTcParams& p, cuda
 
 using namespace b200;
 
-// As b200_latent_decode, for widths that are multiples of 128 up to 512, at most 64 heads and page sizes 8 .. 128 that
-// divide 128.
+// As b200_latent_decode, for vwidths that are multiples of 128 up to 512, widths up to 64 above, at most 64 heads and page sizes
+// 8 .. 128 that divide 128.
 extern "C" int b200_latent_decode_tc(const void* q, const void* cache, void* o, float* part_o, float* part_ml,
                                      const int* positions, const long long* slots, const int* tables, int rows, int heads,
-                                     int width, int max_pages, int page_size, int num_pages, int window, int splits,
+                                     int width, int vwidth, int max_pages, int page_size, int num_pages, int window, int splits,
                                      float scale, uint32_t* status, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (width % 128 || width <= 0 || width > 512 || heads <= 0 || heads > 64 || page_size < 8 || page_size > 128 ||
+  if (vwidth % 128 || vwidth <= 0 || vwidth > 512 || width % 8 || width < vwidth || width > vwidth + 64 || heads <= 0 || heads > 64 || page_size < 8 || page_size > 128 ||
       128 % page_size || splits < 1 || splits > 65535)
     return -10;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(o)) & 15) return -10;
@@ -416,7 +425,7 @@ extern "C" int b200_latent_decode_tc(const void* q, const void* cache, void* o, 
     return -20;
   LatentTcParams p;
   p.q = (const __nv_bfloat16*)q; p.o = (__nv_bfloat16*)o; p.part_o = part_o; p.part_ml = part_ml;
-  p.positions = positions; p.slots = slots; p.tables = tables; p.rows = rows; p.heads = heads; p.width = width;
+  p.positions = positions; p.slots = slots; p.tables = tables; p.rows = rows; p.heads = heads; p.width = width; p.vwidth = vwidth;
   p.max_pages = max_pages; p.page_size = page_size; p.num_pages = num_pages; p.window = window; p.splits = splits;
   p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   if (heads <= 16) return launch_latent_tc<16>(tm, p, st);

@@ -6,20 +6,28 @@
 namespace b200 {
 
 struct ResidualNormParams {
-  // source of the row: the embedding table (tokens != null, written to x) or x itself
+  // source of the row: the embedding table times embed_scale (tokens != null, written to x) or x itself
   const long long* tokens;
   const void* embed;
   int vocab;
+  float embed_scale;
   float* x;                  // (rows, d) fp32 residual stream
   const long long* row_index;  // optional: output row i reads residual row row_index[i] and x is not written
-  // optional expert outputs that belong to the row: x += yscale * sum_k y[ypos[row, k]]
+  // optional expert outputs that belong to the row: x += yscale * sum_k yweight[row, k] * y[ypos[row, k]] (yweight null: ones).
+  // A choice with ypos = -2 stands for the experts' input z[row] itself; s[row], times sigmoid(sgate[row]), is an expert's output
+  // that every row receives.
   const void* y;
   const int* ypos;
+  const float* yweight;
   int ytop, y_rows;
   float yscale;
   long long ld_y;
-  // norm: h = x / rms(x) * w (h == null: only the residual is updated)
+  const void *z, *s;
+  const float* sgate;
+  long long ld_z, ld_s, ld_sgate;
+  // norm: h = x / rms(x) * (w + w_offset) (h == null: only the residual is updated)
   const void* w;
+  float w_offset;
   void* h;
   long long ld_h;
   float eps;
@@ -31,6 +39,30 @@ struct ResidualNormParams {
   int rows, x_rows, d;
   uint32_t* status;
 };
+
+// What the experts add to columns c .. c + VEC - 1 of residual row `src`, without yscale.
+template <typename T, int VEC>
+__device__ __forceinline__ void expert_sum(const ResidualNormParams& p, long long src, int c, float share, float (&s)[VEC]) {
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) s[i] = 0.f;
+  float g[VEC];
+  for (int k = 0; k < p.ytop; ++k) {
+    const int pos = p.ypos[src * p.ytop + k];
+    const T* from;
+    if (pos >= 0 && pos < p.y_rows) from = reinterpret_cast<const T*>(p.y) + (long long)pos * p.ld_y;
+    else if (pos == -2 && p.z != nullptr) from = reinterpret_cast<const T*>(p.z) + src * p.ld_z;
+    else continue;                          // a padding row of the batch
+    const float a = p.yweight != nullptr ? p.yweight[src * p.ytop + k] : 1.f;
+    load_vec<VEC>(from + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s[i] = fmaf(a, g[i], s[i]);
+  }
+  if (p.s != nullptr) {
+    load_vec<VEC>(reinterpret_cast<const T*>(p.s) + src * p.ld_s + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s[i] = fmaf(share, g[i], s[i]);
+  }
+}
 
 // One block per row; every thread keeps to its own columns, so the second pass re-reads what the thread itself wrote.
 template <typename T, int VEC>
@@ -57,26 +89,23 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormPa
     er = reinterpret_cast<const T*>(p.embed) + tok * p.d;
   }
   const bool changed = (er != nullptr || p.y != nullptr) && p.row_index == nullptr;
+  const float share = p.s != nullptr ? (p.sgate != nullptr ? 1.f / (1.f + expf(-p.sgate[src * p.ld_sgate])) : 1.f) : 0.f;
   constexpr int KEEP = 4;                 // column groups of a thread that stay in registers between the passes
   float keep[KEEP][VEC];
   float ss = 0.f;
   int n = 0;
   for (int c = threadIdx.x * VEC; c < p.d; c += blockDim.x * VEC, ++n) {
     float f[VEC];
-    if (er != nullptr) load_vec<VEC>(er + c, f);
-    else load_vec<VEC>(xr + c, f);
+    if (er != nullptr) {
+      load_vec<VEC>(er + c, f);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) f[i] *= p.embed_scale;
+    } else {
+      load_vec<VEC>(xr + c, f);
+    }
     if (p.y != nullptr) {
       float s[VEC];
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) s[i] = 0.f;
-      for (int k = 0; k < p.ytop; ++k) {
-        const int pos = p.ypos[src * p.ytop + k];
-        if (pos < 0 || pos >= p.y_rows) continue;            // a padding row of the batch
-        float g[VEC];
-        load_vec<VEC>(reinterpret_cast<const T*>(p.y) + (long long)pos * p.ld_y + c, g);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) s[i] += g[i];
-      }
+      expert_sum<T, VEC>(p, src, c, share, s);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) f[i] += p.yscale * s[i];
     }
@@ -108,21 +137,13 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormPa
     } else {                              // a gathered row with expert outputs: not stored, so added up again
       load_vec<VEC>(xr + c, f);
       float s[VEC];
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) s[i] = 0.f;
-      for (int k = 0; k < p.ytop; ++k) {
-        const int pos = p.ypos[src * p.ytop + k];
-        if (pos < 0 || pos >= p.y_rows) continue;
-        load_vec<VEC>(reinterpret_cast<const T*>(p.y) + (long long)pos * p.ld_y + c, g);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) s[i] += g[i];
-      }
+      expert_sum<T, VEC>(p, src, c, share, s);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) f[i] += p.yscale * s[i];
     }
     load_vec<VEC>(reinterpret_cast<const T*>(p.w) + c, g);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) f[i] = f[i] * r * g[i];
+    for (int i = 0; i < VEC; ++i) f[i] = f[i] * r * (g[i] + p.w_offset);
     store_vec<VEC>(hr + c, f);
     if (p.xg != nullptr) {
       for (int k = 0; k < p.gtop; ++k) {
@@ -312,16 +333,16 @@ __global__ void glu_any_kernel(const T* __restrict__ gu, T* __restrict__ h, long
   }
 }
 
-// o *= sigmoid(g), element by element.
+// o *= sigmoid(g), a gate for every `per` columns.
 template <typename T>
-__global__ void gate_sigmoid_kernel(T* __restrict__ o, const T* __restrict__ g, long long rows, int n, long long ld_o,
+__global__ void gate_sigmoid_kernel(T* __restrict__ o, const T* __restrict__ g, long long rows, int n, int per, long long ld_o,
                                     long long ld_g) {
   pdl_sync();
   const long long total = rows * n;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / n;
     const int c = (int)(i - r * n);
-    const float s = 1.f / (1.f + expf(-to_f(g[r * ld_g + c])));
+    const float s = 1.f / (1.f + expf(-to_f(g[r * ld_g + c / per])));
     from_f(o[r * ld_o + c], to_f(o[r * ld_o + c]) * s);
   }
 }
@@ -336,26 +357,41 @@ static int blocks_for(long long work, int threads) {
 
 using namespace b200;
 
+// What the experts add, passed by pointer through the C interface: the field order is part of it.
+struct ExpertOutputs {
+  const void* y;
+  const int* ypos;
+  const float* yweight;
+  const void *z, *s;
+  const float* sgate;
+  long long ld_y, ld_z, ld_s, ld_sgate;
+  int ytop, y_rows;
+  float yscale;
+};
+
 // See ResidualNormParams.  f32 != 0: T = float, else bf16.
-extern "C" int b200_residual_norm(const long long* tokens, const void* embed, int vocab, float* x,
-                                  const long long* row_index, const void* y, const int* ypos, int ytop, int y_rows,
-                                  float yscale, long long ld_y, const void* w, void* h, long long ld_h, float eps,
-                                  void* xg, const int* gpos, int gtop, int xg_rows, long long ld_xg, int rows,
-                                  int x_rows, int d, int f32, uint32_t* status, cudaStream_t st) {
+extern "C" int b200_residual_norm(const long long* tokens, const void* embed, int vocab, float embed_scale, float* x,
+                                  const long long* row_index, const ExpertOutputs* ex, const void* w, float w_offset, void* h,
+                                  long long ld_h, float eps, void* xg, const int* gpos, int gtop, int xg_rows, long long ld_xg,
+                                  int rows, int x_rows, int d, int f32, uint32_t* status, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (d <= 0 || x == nullptr || (h != nullptr && w == nullptr) || (tokens != nullptr && embed == nullptr) ||
-      (y != nullptr && ypos == nullptr) || (xg != nullptr && (gpos == nullptr || h == nullptr)) ||
+      (ex != nullptr && (ex->y == nullptr || ex->ypos == nullptr)) || (xg != nullptr && (gpos == nullptr || h == nullptr)) ||
       (tokens != nullptr && row_index != nullptr))
     return -10;
-  ResidualNormParams p;
-  p.tokens = tokens; p.embed = embed; p.vocab = vocab; p.x = x; p.row_index = row_index;
-  p.y = y; p.ypos = ypos; p.ytop = ytop; p.y_rows = y_rows; p.yscale = yscale; p.ld_y = ld_y;
-  p.w = w; p.h = h; p.ld_h = ld_h; p.eps = eps;
+  ResidualNormParams p = {};
+  p.tokens = tokens; p.embed = embed; p.vocab = vocab; p.embed_scale = embed_scale; p.x = x; p.row_index = row_index;
+  if (ex != nullptr) {
+    p.y = ex->y; p.ypos = ex->ypos; p.yweight = ex->yweight; p.ytop = ex->ytop; p.y_rows = ex->y_rows; p.yscale = ex->yscale;
+    p.ld_y = ex->ld_y; p.z = ex->z; p.ld_z = ex->ld_z; p.s = ex->s; p.ld_s = ex->ld_s; p.sgate = ex->sgate; p.ld_sgate = ex->ld_sgate;
+  }
+  p.w = w; p.w_offset = w_offset; p.h = h; p.ld_h = ld_h; p.eps = eps;
   p.xg = xg; p.gpos = gpos; p.gtop = gtop; p.xg_rows = xg_rows; p.ld_xg = ld_xg;
   p.rows = rows; p.x_rows = x_rows; p.d = d; p.status = status;
-  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(embed) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) |
-                         reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(xg);
-  const bool vec = d % 4 == 0 && ld_y % 4 == 0 && ld_h % 4 == 0 && ld_xg % 4 == 0 && (ptrs & 15) == 0;
+  const uintptr_t ptrs = reinterpret_cast<uintptr_t>(embed) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(p.y) |
+                         reinterpret_cast<uintptr_t>(p.z) | reinterpret_cast<uintptr_t>(p.s) | reinterpret_cast<uintptr_t>(w) |
+                         reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(xg);
+  const bool vec = d % 4 == 0 && (p.ld_y | p.ld_z | p.ld_s | ld_h | ld_xg) % 4 == 0 && (ptrs & 15) == 0;
   const int per = vec ? 4 : 1;
   int threads = ((d + per - 1) / per + 31) / 32 * 32;
   if (threads > 256) threads = 256;
@@ -430,13 +466,14 @@ extern "C" int b200_glu_any(const void* gu, void* h, long long rows, int F, long
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-extern "C" int b200_gate_sigmoid(void* o, const void* g, long long rows, int n, long long ld_o, long long ld_g, int f32,
+extern "C" int b200_gate_sigmoid(void* o, const void* g, long long rows, int n, int per, long long ld_o, long long ld_g, int f32,
                                  cudaStream_t st) {
   if (rows <= 0) return 0;
+  if (per <= 0) return -10;
   const int b = blocks_for(rows * n, 256);
-  if (f32) launch_dep(gate_sigmoid_kernel<float>, b, 256, 0, st, (float*)o, (const float*)g, rows, n, ld_o, ld_g);
+  if (f32) launch_dep(gate_sigmoid_kernel<float>, b, 256, 0, st, (float*)o, (const float*)g, rows, n, per, ld_o, ld_g);
   else
     launch_dep(gate_sigmoid_kernel<__nv_bfloat16>, b, 256, 0, st, (__nv_bfloat16*)o, (const __nv_bfloat16*)g, rows, n,
-               ld_o, ld_g);
+               per, ld_o, ld_g);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }

@@ -1,0 +1,230 @@
+// Mixture of experts with a learned router: choice of experts per row, then the rows sorted by expert into 128-row tiles.
+//
+// The router's logits come out of a GEMM in fp32.  moe_route takes the softmax over all outputs of a row, chooses the `top` outputs
+// with the largest score + correction and weighs them with their share of the scores; outputs from `experts` on are identities (the
+// experts' input itself) and need no expert row.  A chosen expert's place among the rows that chose it comes from a counter per
+// expert (counted per block in shared memory first).  moe_dispatch turns the counters into tiles (every block does the short prefix
+// sum itself), writes where each choice's row went and copies the rows there.  Which row of a tile a token gets depends on the
+// order of the atomics; what is computed for it does not.
+#include "typed.cuh"
+
+namespace b200 {
+
+constexpr int ROUTE_TILE = 128;            // rows of an expert tile (mixer_elementwise.cu: PLAN_TILE)
+constexpr int ROUTE_WARPS = 8;
+constexpr int ROUTE_ROWS = 4;              // rows of a warp
+
+struct RouteParams {
+  const float* z;              // (rows, ld_z): logits of experts + identities
+  long long ld_z;
+  const float* correction;     // (outputs)
+  const long long* slots;      // negative = padding row
+  int* choice;                 // (rows, top): chosen output, -1 for a padding row
+  int* rank;                   // (rows, top): place among the rows of the chosen expert
+  float* weight;               // (rows, top)
+  int* count;                  // (experts), zero before the launch
+  int rows, experts, outputs, top;
+};
+
+// One warp per row at a time; shared memory: per warp the scores and the choice scores, per block a counter and a base per expert.
+__global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(const RouteParams p) {
+  pdl_sync();
+  extern __shared__ float rsm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* s = rsm + warp * 2 * p.outputs;
+  float* key = s + p.outputs;
+  int* local = reinterpret_cast<int*>(rsm + ROUTE_WARPS * 2 * p.outputs);
+  int* base = local + p.experts;
+  int* picked = base + p.experts;            // [ROUTE_WARPS * ROUTE_ROWS][top][2]: expert, place within the block
+  for (int e = threadIdx.x; e < p.experts; e += blockDim.x) local[e] = 0;
+  __syncthreads();
+  const int row0 = (blockIdx.x * ROUTE_WARPS + warp) * ROUTE_ROWS;
+  for (int r = 0; r < ROUTE_ROWS && row0 + r < p.rows; ++r) {
+    const int row = row0 + r;
+    int* mine = picked + (warp * ROUTE_ROWS + r) * p.top * 2;
+    if (p.slots[row] < 0) {
+      for (int k = lane; k < p.top; k += 32) {
+        mine[2 * k] = -1;
+        p.choice[(long long)row * p.top + k] = -1;
+        p.weight[(long long)row * p.top + k] = 0.f;
+      }
+      continue;
+    }
+    const float* z = p.z + (long long)row * p.ld_z;
+    float mx = -INFINITY;
+    for (int e = lane; e < p.outputs; e += 32) mx = fmaxf(mx, s[e] = z[e]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    float sum = 0.f;
+    for (int e = lane; e < p.outputs; e += 32) sum += s[e] = expf(s[e] - mx);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    for (int e = lane; e < p.outputs; e += 32) {
+      s[e] /= sum;
+      key[e] = s[e] + p.correction[e];
+    }
+    __syncwarp();
+    float total = 0.f;
+    for (int k = 0; k < p.top; ++k) {        // a lane looks after outputs lane, lane + 32, ...; ties go to the lower index
+      float best = -INFINITY;
+      int at = p.outputs;
+      for (int e = lane; e < p.outputs; e += 32)
+        if (key[e] > best) {
+          best = key[e];
+          at = e;
+        }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ob > best || (ob == best && oa < at)) {
+          best = ob;
+          at = oa;
+        }
+      }
+      if (at >= p.outputs) at = 0;           // not a number anywhere: something valid
+      total += s[at];
+      __syncwarp();
+      if (lane == (at & 31)) key[at] = -INFINITY;
+      if (lane == 0) {
+        mine[2 * k] = at;
+        if (at < p.experts) mine[2 * k + 1] = atomicAdd(&local[at], 1);
+      }
+      __syncwarp();
+    }
+    for (int k = lane; k < p.top; k += 32) {
+      p.choice[(long long)row * p.top + k] = mine[2 * k];
+      p.weight[(long long)row * p.top + k] = s[mine[2 * k]] / (total + 1e-20f);
+    }
+    __syncwarp();
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < p.experts; e += blockDim.x) base[e] = local[e] > 0 ? atomicAdd(&p.count[e], local[e]) : 0;
+  __syncthreads();
+  const int first = blockIdx.x * ROUTE_WARPS * ROUTE_ROWS;
+  const int n = min(ROUTE_WARPS * ROUTE_ROWS, p.rows - first) * p.top;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const int e = picked[2 * i];
+    p.rank[(long long)first * p.top + i] = e >= 0 && e < p.experts ? base[e] + picked[2 * i + 1] : -1;
+  }
+}
+
+struct DispatchParams {
+  const void* h;               // (rows, ld_h), `vecs` 16-byte pieces (or `d` elements) of a row are copied
+  long long ld_h;
+  void* xg;                    // (tiles * 128, ld_xg)
+  long long ld_xg;
+  const int *choice, *rank, *count;
+  int* pos;                    // (rows, top): row of xg, -2 identity, -1 none
+  int* tile_group;             // (tiles): expert, -1 = not used
+  int rows, experts, top, tiles, d;
+};
+
+// E: an element, or 16 bytes of them.  One warp per row.
+template <typename E>
+__global__ void __launch_bounds__(256) moe_dispatch_kernel(const DispatchParams p) {
+  pdl_sync();
+  extern __shared__ int start[];             // [experts + 1]: first tile of every expert
+  __shared__ int warp_sum[8];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int carry = 0;
+  for (int e0 = 0; e0 < p.experts; e0 += 256) {
+    const int e = e0 + threadIdx.x;
+    const int n = e < p.experts ? (p.count[e] + ROUTE_TILE - 1) / ROUTE_TILE : 0;
+    int x = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int y = __shfl_up_sync(0xffffffffu, x, o);
+      if (lane >= o) x += y;
+    }
+    if (lane == 31) warp_sum[warp] = x;
+    __syncthreads();
+    int before = carry;
+    for (int w = 0; w < 8; ++w) {
+      if (w < warp) before += warp_sum[w];
+      carry += warp_sum[w];
+    }
+    if (e < p.experts) start[e] = before + x - n;
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) start[p.experts] = carry;
+  __syncthreads();
+  if (blockIdx.x == 0) {
+    for (int e = warp; e < p.experts; e += 8)
+      for (int t = start[e] + lane; t < start[e + 1] && t < p.tiles; t += 32) p.tile_group[t] = e;
+    for (int t = carry + threadIdx.x; t < p.tiles; t += 256) p.tile_group[t] = -1;
+  }
+  const int row = blockIdx.x * 8 + warp;
+  if (row >= p.rows) return;
+  const E* src = reinterpret_cast<const E*>(p.h) + row * p.ld_h;
+  for (int k0 = 0; k0 < p.top; k0 += 32) {
+    const int k = k0 + lane, n = min(32, p.top - k0);
+    int to = -1;
+    if (k < p.top) {
+      const int e = p.choice[(long long)row * p.top + k];
+      if (e >= p.experts) to = -2;
+      else if (e >= 0) {
+        to = start[e] * ROUTE_TILE + p.rank[(long long)row * p.top + k];
+        if (to >= p.tiles * ROUTE_TILE) to = -1;
+      }
+      p.pos[(long long)row * p.top + k] = to;
+    }
+    for (int c0 = 0; c0 < p.d; c0 += 128) {
+      E v[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (c0 + i * 32 + lane < p.d) v[i] = src[c0 + i * 32 + lane];
+      for (int j = 0; j < n; ++j) {
+        const int at = __shfl_sync(0xffffffffu, to, j);
+        if (at < 0) continue;
+        E* dst = reinterpret_cast<E*>(p.xg) + at * p.ld_xg;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (c0 + i * 32 + lane < p.d) dst[c0 + i * 32 + lane] = v[i];
+      }
+    }
+  }
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+// `count` (experts ints) must be zero; identities are the outputs from `experts` on.
+extern "C" int b200_moe_route(const float* z, long long ld_z, const float* correction, const long long* slots, int* choice, int* rank,
+                              float* weight, int* count, int rows, int experts, int outputs, int top, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (experts <= 0 || outputs < experts || top <= 0 || top > outputs) return -10;
+  RouteParams p;
+  p.z = z; p.ld_z = ld_z; p.correction = correction; p.slots = slots; p.choice = choice; p.rank = rank; p.weight = weight; p.count = count;
+  p.rows = rows; p.experts = experts; p.outputs = outputs; p.top = top;
+  const size_t smem = (size_t)ROUTE_WARPS * 2 * outputs * 4 + 2ull * experts * 4 + (size_t)ROUTE_WARPS * ROUTE_ROWS * top * 8;
+  if (smem > 200 * 1024) return -12;
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    return -3;
+  launch_dep(moe_route_kernel, (unsigned)((rows + ROUTE_WARPS * ROUTE_ROWS - 1) / (ROUTE_WARPS * ROUTE_ROWS)), ROUTE_WARPS * 32, smem, st, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// h (rows, d) of `elem`-byte elements, copied to its places in xg (tiles * 128, ld_xg).
+extern "C" int b200_moe_dispatch(const void* h, long long ld_h, void* xg, long long ld_xg, const int* choice, const int* rank,
+                                 const int* count, int* pos, int* tile_group, int rows, int experts, int top, int tiles, int d, int elem,
+                                 cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (experts <= 0 || experts > 4096 || top <= 0 || tiles <= 0 || d <= 0 || (elem != 2 && elem != 4)) return -10;
+  DispatchParams p;
+  p.h = h; p.ld_h = ld_h; p.xg = xg; p.ld_xg = ld_xg; p.choice = choice; p.rank = rank; p.count = count; p.pos = pos;
+  p.tile_group = tile_group; p.rows = rows; p.experts = experts; p.top = top; p.tiles = tiles; p.d = d;
+  const unsigned grid = (unsigned)((rows + 7) / 8);
+  const size_t smem = (experts + 1) * sizeof(int);
+  const int per = 16 / elem;
+  if (d % per == 0 && ld_h % per == 0 && ld_xg % per == 0 && ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(xg)) & 15) == 0) {
+    p.d = d / per; p.ld_h = ld_h / per; p.ld_xg = ld_xg / per;
+    launch_dep(moe_dispatch_kernel<uint4>, grid, 256, smem, st, p);
+  } else if (elem == 2) {
+    launch_dep(moe_dispatch_kernel<uint16_t>, grid, 256, smem, st, p);
+  } else {
+    launch_dep(moe_dispatch_kernel<uint32_t>, grid, 256, smem, st, p);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}

@@ -1,4 +1,4 @@
-"""What models made of listed layers have in common (``tedirax.py``, ``beledra.py``): configuration checks, loading from a
+"""What models made of listed layers have in common (``tedirax.py``, ``beledra.py``, ``genedra.py``): configuration checks, loading from a
 folder, random weights, generation through the serving engine.
 
 A subclass reads its configuration, packs its weights into ``layers`` / ``runs`` (objects with a ``mixer`` from ``mixers.py``

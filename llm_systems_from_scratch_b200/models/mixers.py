@@ -6,8 +6,10 @@ input become one product; heads are padded to what the kernels tile by) and runs
 * a mixer is called with its input rows ``h``, the fp32 residual stream ``x``, the ``StepBatch`` and its own part of the
   cache (``cache_spec()`` says what that is).  It adds its output to ``x`` in the epilogue of its output projection, or
   returns it when ``x`` is None (designs that norm a sublayer's output before they add it)
-* a feed-forward returns outputs that the next pass over the residual stream adds (``ops.mixer_ops.residual_norm``,
-  ``add_normed``)
+* a feed-forward does the same, or returns outputs that the next pass over the residual stream adds (``ops.mixer_ops``:
+  ``residual_norm``, ``add_normed``)
+
+What a sublayer adds to ``x`` it multiplies with its ``gain``.
 
 ``get(name)`` gives a weight in its stored layout ([out, in])."""
 from __future__ import annotations
@@ -35,82 +37,134 @@ def _expect(name: str, t, *shape):
     return t
 
 
-def _project(y, w_o, x):
+def _project(y, w_o, x, gain: float = 1.0, bias=None):
     """The output projection, into the residual stream or returned."""
-    return mo.linear(y, w_o) if x is None else mo.linear(y, w_o, out=x, accumulate=True)
+    return mo.linear(y, w_o, bias=bias) if x is None else mo.linear(y, w_o, out=x, accumulate=True, alpha=gain, bias=bias)
+
+
+def _align(n: int, to: int) -> int:
+    return -(-n // to) * to
+
+
+def _row_pad(w, to: int):
+    """Zero rows up to ``to``."""
+    return w if w.shape[0] == to else torch.cat((w, torch.zeros((to - w.shape[0], w.shape[1]), dtype=w.dtype, device=w.device)))
 
 
 class LatentAttention:
-    """Attention whose keys and values are linear images of one cached latent per token; no positions.
+    """Attention whose keys and values are linear images of one cached latent per token.
 
-    q = W_uq rms_norm(W_dq h), c = rms_norm(W_dkv h), k_h = W_uk,h c, v_h = W_uv,h c, softmax(scale q.k) over the last
-    ``window`` positions (0 = all), heads multiplied by sigmoid(W_g h), then W_o.  The cache holds c alone."""
+    q = W_uq rms_norm(W_dq h), or W_q h without a ``q_rank``; c = rms_norm(W_dkv h), k_h = W_uk,h c, v_h = W_uv,h c,
+    softmax(scale q.k) over the last ``window`` positions (0 = all), heads multiplied by sigmoid(W_g h) (``gate``: "elements", or
+    one number per head: "heads"), then W_o.  The cache holds c.  Optional parts:
 
-    def __init__(self, get, width: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, window: int,
-                 eps: float, dtype, device):
+    * ``rot_dim`` / ``rope``: every head's query has rot_dim more rows, which are rotated (interleaved pairs); W_dkv has rot_dim more
+      rows, a rotated key part shared by all heads, cached behind c
+    * ``kv_from``: latents and key parts of that earlier layer run instead of its own"""
+
+    def __init__(self, get, width: int, heads: int, dim: int, vdim: int, q_rank: int | None, kv_rank: int, scale: float, window: int,
+                 eps: float, dtype, device, rot_dim: int = 0, rope=None, kv_from: int | None = None, gate: str = "elements",
+                 gain: float = 1.0):
+        if rot_dim % 2 or (rot_dim and rope is None):
+            raise ValueError("the rotated dimensions come in pairs and need angles")
+        if gate not in ("elements", "heads"):
+            raise ValueError(f"unknown gate {gate!r}")
         self.heads, self.dim, self.vdim, self.q_rank, self.kv_rank = heads, dim, vdim, q_rank, kv_rank
+        self.rot, self.rope, self.kv_from, self.gain = int(rot_dim), rope, kv_from, float(gain)
         self.scale, self.window, self.eps = float(scale), int(window), float(eps)
-        self.latent = mo.pitch(kv_rank)                  # cached vector, zero padded
+        self.latent, self.rp = mo.pitch(kv_rank), mo.pitch(rot_dim)             # cached parts, zero padded
+        self.cached = self.latent + self.rp
         w = lambda name, *shape: _expect(name, get(name), *shape)
-        dq, dkv = w("dq", q_rank, width), w("dkv", kv_rank, width)
-        uq, uk = w("uq", heads * dim, q_rank), w("uk", heads * dim, kv_rank)
-        uv, g = w("uv", heads * vdim, kv_rank), w("g", heads * vdim, width)
-        o = w("o", width, heads * vdim)
         pack = lambda t: mo.padded_weight(t, dtype, device)
-        # the tensor-core prefill takes heads of 64 or 128; elsewhere a head only has to start on a 16-byte boundary
-        self.flash_dim = 0 if max(dim, vdim) > 128 else (64 if max(dim, vdim) <= 64 else 128)
-        if dtype != torch.bfloat16 or torch.device(device).type != "cuda" or scale <= 0:
-            self.flash_dim = 0
-        self.qdim = self.flash_dim or mo.pitch(dim)
-        self.w_in = pack(torch.cat((dq, dkv, g)))
-        self.w_uq = pack(_head_pad(uq, heads, dim, self.qdim))
-        ukt = torch.zeros((heads, self.latent, self.qdim), dtype=uk.dtype, device=uk.device)        # q_h -> latent space: W_uk,h^T
+        # the tensor-core prefill takes heads up to 128 whose columns are multiplied 16 at a time; elsewhere a head only has to start on
+        # a 16-byte boundary
+        self.tiles = (dtype == torch.bfloat16 and torch.device(device).type == "cuda" and max(dim, vdim) <= 128 and rot_dim <= 64
+                      and scale > 0)
+        self.qp, self.vp = _align(dim, 16) if self.tiles else mo.pitch(dim), mo.pitch(vdim)
+        # queries: the unrotated parts of all heads, then the rotated ones
+        own = w("uq", heads * (dim + rot_dim), q_rank) if q_rank is not None else w("q", heads * (dim + rot_dim), width)
+        own = own.view(heads, dim + rot_dim, -1)
+        q = _head_pad(own[:, :dim].reshape(heads * dim, -1), heads, dim, self.qp)
+        if rot_dim:
+            q = torch.cat((q, _head_pad(own[:, dim:].reshape(heads * rot_dim, -1), heads, rot_dim, self.rp)))
+        parts, at = [], 0
+        self.w_uq = self.n_q = None
+        if q_rank is not None:
+            parts.append(w("dq", q_rank, width))
+            self.w_uq, self.n_q = pack(q), w("dq.norm", q_rank).to(device=device, dtype=dtype).contiguous()
+        else:
+            parts.append(q)
+        self.kv_col = self.k_col = self.n_kv = None
+        if kv_from is None:
+            dkv = w("dkv", kv_rank + rot_dim, width)
+            self.kv_col = sum(len(p) for p in parts)
+            parts.append(dkv[:kv_rank])
+            if rot_dim:
+                parts[-1] = _row_pad(parts[-1], self.latent)
+                self.k_col = self.kv_col + self.latent
+                parts.append(_row_pad(dkv[kv_rank:], self.rp))
+            self.n_kv = w("dkv.norm", kv_rank).to(device=device, dtype=dtype).contiguous()
+        self.gate_col = sum(len(p) for p in parts)
+        parts.append(w("g", heads * vdim if gate == "elements" else heads, width))
+        self.w_in = pack(torch.cat(parts))
+        uk, uv = w("uk", heads * dim, kv_rank), w("uv", heads * vdim, kv_rank)
+        ukt = torch.zeros((heads, self.latent, self.qp), dtype=uk.dtype, device=uk.device)        # q_h -> latent space: W_uk,h^T
         ukt[:, :kv_rank, :dim] = uk.view(heads, dim, kv_rank).transpose(1, 2)
-        self.w_ukt = pack(ukt.reshape(heads * self.latent, self.qdim))
+        self.w_ukt = pack(ukt.reshape(heads * self.latent, self.qp))
         uvp = torch.zeros((heads * vdim, self.latent), dtype=uv.dtype, device=uv.device)
         uvp[:, :kv_rank] = uv
         self.w_uv = pack(uvp)
-        if self.flash_dim:
-            kv = torch.zeros((2 * heads * self.flash_dim, self.latent), dtype=uk.dtype, device=uk.device)
-            kv[:heads * self.flash_dim, :kv_rank] = _head_pad(uk, heads, dim, self.flash_dim)
-            kv[heads * self.flash_dim:, :kv_rank] = _head_pad(uv, heads, vdim, self.flash_dim)
+        if self.tiles:
+            kv = torch.zeros((heads * (self.qp + self.vp), self.latent), dtype=uk.dtype, device=uk.device)
+            kv[:heads * self.qp, :kv_rank] = _head_pad(uk, heads, dim, self.qp)
+            kv[heads * self.qp:, :kv_rank] = _head_pad(uv, heads, vdim, self.vp)
             self.w_ukv = pack(kv)
-        self.w_o = pack(o)
-        self.n_q = w("dq.norm", q_rank).to(device=device, dtype=dtype).contiguous()
-        self.n_kv = w("dkv.norm", kv_rank).to(device=device, dtype=dtype).contiguous()
+        self.w_o = pack(w("o", width, heads * vdim))
 
     def cache_spec(self):
-        return PagedSpec(self.latent)
+        return PagedSpec(self.cached) if self.kv_from is None else SharedSpec(self.kv_from)
 
     def __call__(self, h, x, batch, cache):
-        heads, n = self.heads, batch.n_single
+        heads, n, rows = self.heads, batch.n_single, batch.n_rows
         proj = mo.linear(h, self.w_in)
-        cq = mo.latent_norm_append(proj, self.n_q, self.n_kv, self.eps, cache, batch.slots)
-        q = mo.linear(cq, self.w_uq)
-        gate = proj[:, self.q_rank + self.kv_rank:]
-        o = mo.rows_buffer(h.shape[0], heads * self.vdim, h.dtype, h.device)
+        q = proj
+        if self.q_rank is not None:
+            cq = mo.latent_norm_append(proj, self.n_q, self.n_kv, self.eps, cache, batch.slots)
+            q = mo.linear(cq, self.w_uq)
+        gate = proj[:, self.gate_col:]
+        o = mo.rows_buffer(rows, heads * self.vdim, h.dtype, h.device)
+        absorbed = n if self.tiles else rows             # rows whose queries move into latent space
+        ql = None
+        if absorbed:
+            ql = torch.empty((absorbed, heads * self.cached), dtype=h.dtype, device=h.device)
+            mo.gemm_heads(q[:absorbed], self.w_ukt, heads, self.qp, self.latent, out=ql, c_step=self.cached)
+        if self.rot:
+            mo.latent_rotate(q, heads * self.qp, self.rp, proj, self.kv_col if self.q_rank is None else None, self.k_col, self.n_kv, ql,
+                             cache, self.rope.table, batch.positions, batch.slots, heads, self.kv_rank, self.latent, self.rot, self.eps)
         if n:
-            ql = mo.gemm_heads(q[:n], self.w_ukt, heads, self.qdim, self.latent)
-            ol = mo.latent_decode(ql, cache, batch.positions[:n], batch.slots[:n], batch.tables[:n], heads, self.window, self.scale)
+            ol = mo.latent_decode(ql[:n], cache, batch.positions[:n], batch.slots[:n], batch.tables[:n], heads, self.window, self.scale,
+                                  vwidth=self.latent)
             mo.gemm_heads(ol, self.w_uv, heads, self.latent, self.vdim, out=o[:n], gate=gate[:n])
-        if batch.n_rows > n:
-            self._portions(q[n:], gate[n:], o[n:], batch, cache, slice(n, batch.n_rows))
-        return _project(o, self.w_o, x)
+        if rows > n and self.tiles:
+            self._portions(q[n:], gate[n:], o[n:], batch, cache)
+        elif rows > n:
+            ol = mo.latent_attention_rows(ql[n:], cache, batch.row_seq[n:], batch.positions[n:], batch.slots[n:], batch.tables, heads,
+                                          self.window, self.scale, self.latent)
+            mo.gemm_heads(ol, self.w_uv, heads, self.latent, self.vdim, out=o[n:], gate=gate[n:])
+        return _project(o, self.w_o, x, self.gain)
 
-    def _portions(self, q, gate, o, batch, cache, rows: slice):
+    def _portions(self, q, gate, o, batch, cache):
+        """Keys and values of everything the portions can see, expanded from the cached latents."""
         heads = self.heads
-        if self.flash_dim:
-            # keys and values of everything the portions can see, expanded from the cached latents
-            cu_k, first, total, _ = batch.key_ranges(self.window)
-            c = mo.latent_gather(cache, cu_k, first, batch.tables[batch.n_single:], total)
-            kv = mo.linear(c, self.w_ukv)
-            mo.window_attention(q, kv, batch.cu, cu_k, batch.max_portion, heads, self.flash_dim, self.vdim, self.window,
-                                self.scale, o, gate)
-            return
-        ql = mo.gemm_heads(q, self.w_ukt, heads, self.qdim, self.latent)
-        ol = mo.latent_attention_rows(ql, cache, batch.row_seq[rows], batch.positions[rows], batch.slots[rows], batch.tables,
-                                      heads, self.window, self.scale)
-        mo.gemm_heads(ol, self.w_uv, heads, self.latent, self.vdim, out=o, gate=gate)
+        cu_k, first, total, _ = batch.key_ranges(self.window)
+        key = (cache.data_ptr(), self.window)            # layers that share a cache share its packed rows
+        if key not in batch.gathered:
+            batch.gathered[key] = mo.latent_gather(cache, cu_k, first, batch.tables[batch.n_single:], total)
+        c = batch.gathered[key]
+        kv = mo.linear(c[:, :self.latent], self.w_ukv)
+        rot = (c, self.rot, heads * self.qp, self.rp, self.latent) if self.rot else None
+        mo.window_attention(q, kv, batch.cu, cu_k, batch.max_portion, heads, self.dim, self.vdim, self.window, self.scale, o, gate,
+                            (self.qp, self.qp, self.vp, heads * self.qp), rot)
 
 
 class Retention:
@@ -202,9 +256,13 @@ class MatrixMemory:
 class GroupedAttention:
     """Softmax attention of grouped heads under a sliding window: query head h reads key/value head h // (heads / kv_heads).
 
-    Queries and keys are RMS-normed per head (weights ``q.norm`` / ``k.norm``), rotated in their first ``rot_dims`` dimensions
-    (``rope``), scored with ``scale``.  Optional parts:
+    Queries and keys are RMS-normed (weights ``q.norm`` / ``k.norm``; ``norm`` "head": per head, "projection": over all heads at
+    once), rotated in their first ``rot_dims`` dimensions (``rope``), scored with ``scale``.  Optional parts:
 
+    * ``keep``: the first ``keep`` positions of a sequence stay visible whatever the window
+    * ``softcap``: scores are capped softly, cap tanh(score / cap)
+    * ``sink``: exp(sink_h), a number per head, joins the softmax's denominator
+    * ``biased``: q, k, v and o have biases (``q.b`` ...)
     * ``bias_max``: a table ``rel`` (buckets, heads) adds a bias per distance to the scaled scores, exact for near keys and
       logarithmic up to ``bias_max``
     * ``difference`` (with ``out_scale``): two maps per head over the same values (queries and keys have twice the rows, laid
@@ -216,23 +274,34 @@ class GroupedAttention:
 
     def __init__(self, get, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, eps: float,
                  dtype, device, bias_max: float | None = None, rope=None, rot_dims: int = 0, difference: float | None = None,
-                 out_scale: float = 1.0, gated: bool = False, kv_from: int | None = None):
-        self.gated, self.kv_from, self.rope = gated, kv_from, rope
+                 out_scale: float = 1.0, gated: bool = False, kv_from: int | None = None, keep: int = 0, softcap: float | None = None,
+                 sink: bool = False, biased: bool = False, norm: str = "head", gain: float = 1.0):
+        self.gated, self.kv_from, self.rope, self.gain = gated, kv_from, rope, float(gain)
         if heads % kv_heads:
             raise ValueError("the query heads must share the key heads evenly")
         if rot_dims % 2 or rot_dims > dim:
             raise ValueError("the rotated dimensions must be even in number and fit the head")
+        if norm not in ("head", "projection"):
+            raise ValueError(f"unknown norm {norm!r}")
         maps = 1 if difference is None else 2
+        if maps == 2 and (sink or norm == "projection"):
+            raise ValueError("sinks and norms over a projection are those of a single map")
         w = lambda name, *shape: _expect(name, get(name), *shape)
-        parts = [w("q", heads * maps * dim, width)]
+        rows = {"q": heads * maps * dim}
         if kv_from is None:
-            parts += [w("k", kv_heads * maps * dim, width), w("v", kv_heads * vdim, width)]
+            rows.update({"k": kv_heads * maps * dim, "v": kv_heads * vdim})
         if gated:
-            parts.append(w("g", heads * vdim, width))
-        self.w_in = mo.padded_weight(torch.cat(parts), dtype, device)
+            rows["g"] = heads * vdim
+        self.w_in = mo.padded_weight(torch.cat([w(name, n, width) for name, n in rows.items()]), dtype, device)
         self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
-        vec = lambda name: w(name, dim).to(device=device, dtype=dtype).contiguous()
-        self.n_q, self.n_k = vec("q.norm"), vec("k.norm") if kv_from is None else None
+        f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+        self.b_in = self.b_o = None
+        if biased:
+            none = lambda n: torch.zeros(n, dtype=get("q.b").dtype, device=get("q.b").device)
+            self.b_in = f32(torch.cat([none(n) if name == "g" else w(name + ".b", n) for name, n in rows.items()]))
+            self.b_o = f32(w("o.b", width))
+        vec = lambda name, n: w(name, dim if norm == "head" else n * dim).to(device=device, dtype=dtype).contiguous()
+        self.n_q, self.n_k = vec("q.norm", heads), vec("k.norm", kv_heads) if kv_from is None else None
         bias = None
         if bias_max is not None:
             rel = get("rel")
@@ -240,7 +309,8 @@ class GroupedAttention:
                 raise ValueError(f"rel has shape {tuple(rel.shape)}, expected {heads} columns")
             bias = distance_table(rel, bias_max, window).to(device)
         self.shape = mo.AttentionShape(heads, kv_heads, maps, dim, vdim, rot_dims, float(scale), int(window), float(eps),
-                                       float(difference or 0.0), float(out_scale), bias)
+                                       float(difference or 0.0), float(out_scale), bias, int(keep), float(softcap or 0.0),
+                                       f32(w("sink", heads)) if sink else None, norm == "projection")
         self.tensor_cores = torch.device(device).type == "cuda" and mo.attention_tiles(self.shape, dtype)
 
     def cache_spec(self):
@@ -248,7 +318,7 @@ class GroupedAttention:
 
     def __call__(self, h, x, batch, cache):
         s, n = self.shape, batch.n_single
-        proj = mo.linear(h, self.w_in)
+        proj = mo.linear(h, self.w_in, bias=self.b_in)
         q = mo.attention_prepare(proj, s, self.n_q, self.n_k, self.rope.table if self.rope is not None else None,
                                  batch.positions, batch.slots, cache)
         o = mo.rows_buffer(h.shape[0], s.heads * s.vdim, h.dtype, h.device)
@@ -265,7 +335,7 @@ class GroupedAttention:
             else:
                 mo.attention_rows(q[rest], s, cache, batch.row_seq[rest], batch.positions[rest], batch.slots[rest],
                                   batch.tables, o[rest], part(rest))
-        return _project(o, self.w_o, x)
+        return _project(o, self.w_o, x, self.gain, self.b_o)
 
 
 def distance_bucket(n: int, rows: int, far: float) -> int:
@@ -294,7 +364,8 @@ class RotaryTable:
     """cos and sin of position * frequency, rounded once from double precision: (2, positions, dims / 2) fp32.  One per rotation,
     shared by the layers that use it; the engine sizes it to its longest context.
 
-    The frequencies are base^(-2 i / dims).  ``scaling`` (factor, original, fast, slow) interpolates them as YaRN does: pairs
+    The frequencies are base^(-2 i / dims).  ``scaling`` with a ``factor`` alone divides all of them by it; with (factor, original, fast,
+    slow) it interpolates them as YaRN does: pairs
     that turn more than ``fast`` times within ``original`` positions stay, those that turn less than ``slow`` times are slowed
     down by ``factor``, a linear ramp between; cos and sin are multiplied by 0.1 ln(factor) + 1."""
 
@@ -303,7 +374,9 @@ class RotaryTable:
         self.table = None
         self.freq = self.base ** (-2.0 * torch.arange(self.dims // 2, dtype=torch.float64) / self.dims)
         self.gain = 1.0
-        if scaling is not None:
+        if scaling is not None and set(scaling) == {"factor"}:
+            self.freq = self.freq / scaling["factor"]
+        elif scaling is not None:
             pair = lambda turns: self.dims * math.log(scaling["original"] / (2 * math.pi * turns)) / (2 * math.log(self.base))
             lo, hi = max(math.floor(pair(scaling["fast"])), 0), min(math.ceil(pair(scaling["slow"])), self.dims - 1)
             ramp = ((torch.arange(self.dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
@@ -319,14 +392,14 @@ class RotaryTable:
 class GatedFeedForward:
     """W_down (act(W_gate h) * (W_up h)), ``act`` "silu" or "relu"."""
 
-    def __init__(self, get, width: int, ff: int, act: str, dtype, device):
-        self.ff, self.act = ff, act
+    def __init__(self, get, width: int, ff: int, act: str, dtype, device, gain: float = 1.0):
+        self.ff, self.act, self.gain = ff, act, float(gain)
         gu = torch.cat((_expect("gate", get("gate"), ff, width), _expect("up", get("up"), ff, width)))
         self.w_gu = mo.padded_weight(gu, dtype, device)                           # gate rows first
         self.w_down = mo.padded_weight(_expect("down", get("down"), width, ff), dtype, device)
 
-    def __call__(self, h):
-        return mo.linear(mo.glu(h, self.w_gu, self.ff, self.act), self.w_down)
+    def __call__(self, h, x=None):
+        return _project(mo.glu(h, self.w_gu, self.ff, self.act), self.w_down, x, self.gain)
 
 
 class TableExperts:
@@ -353,3 +426,41 @@ class TableExperts:
     def __call__(self, xg, tile_group):
         hidden = mo.gemm_rows(xg, self.w_gu, tile_group, self.ff, swiglu=True)
         return mo.gemm_rows(hidden, self.w_down, tile_group, self.width, swiglu=False)
+
+
+class RoutedExperts:
+    """Experts W_down gelu(W_up h) chosen by a learned router.
+
+    The router's softmax runs over ``experts`` + ``identity`` outputs; the last ``identity`` of them stand for h itself.  The ``top``
+    outputs with the largest score + ``correction`` are chosen and weighted by their share of the chosen scores.  ``shared``: rows of
+    an expert that every token uses, times sigmoid of one number per token (``shared.sg``, a row of the router's product).
+
+    A step's rows are sorted by chosen expert into 128-row tiles for the grouped products; what comes out is added up by the next pass
+    over the residual stream (``ops.mixer_ops.ExpertOutputs``)."""
+
+    def __init__(self, get, width: int, ff: int, experts: int, top: int, identity: int, shared: int | None, dtype, device,
+                 gain: float = 1.0):
+        if not 0 < top <= experts + identity:
+            raise ValueError(f"{top} of {experts + identity} outputs cannot be chosen")
+        self.width, self.ff, self.experts, self.top, self.identity, self.gain = width, ff, experts, top, identity, float(gain)
+        w = lambda name, *shape: _expect(name, get(name), *shape)
+        pack = lambda *ts: mo.padded_weight(torch.cat(ts), dtype, device)
+        self.shared = shared is not None
+        router = [w("router", experts + identity, width)]
+        if self.shared:
+            router.append(w("shared.sg", 1, width))
+            self.w_shared_up, self.w_shared_down = pack(w("shared.up", shared, width)), pack(w("shared.down", width, shared))
+        self.w_router = pack(*router)
+        self.correction = w("correction", experts + identity).to(device=device, dtype=torch.float32).contiguous()
+        self.w_up = pack(*[w(f"e{e}.up", ff, width) for e in range(experts)])
+        self.w_down = pack(*[w(f"e{e}.down", width, ff) for e in range(experts)])
+
+    def __call__(self, h, slots, count):
+        """``count``: (experts,) int32 of zeros."""
+        outputs = self.experts + self.identity
+        z = mo.linear(h, self.w_router, out_dtype=torch.float32)                   # what is routed by is 32-bit
+        choice, rank, weight = mo.moe_route(z[:, :outputs], self.correction, slots, self.experts, self.top, count)
+        xg, pos, groups = mo.moe_dispatch(h, choice, rank, count)
+        y = mo.gemm_rows(mo.gemm_rows(xg, self.w_up, groups, self.ff, False, "gelu"), self.w_down, groups, self.width, False)
+        s = mo.linear(mo.linear(h, self.w_shared_up, act="gelu"), self.w_shared_down) if self.shared else None
+        return mo.ExpertOutputs(y, pos, self.gain, weight, h, s, z[:, outputs] if self.shared else None)

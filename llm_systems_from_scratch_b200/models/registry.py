@@ -10,10 +10,11 @@ import os
 import torch
 
 from .beledra import Beledra
+from .genedra import Genedra
 from .tedirax import Tedirax
 from .transformer import TransformerLM
 
-MODELS = {"TransformerLM": TransformerLM, "Tedirax": Tedirax, "Beledra": Beledra}
+MODELS = {"TransformerLM": TransformerLM, "Tedirax": Tedirax, "Beledra": Beledra, "Genedra": Genedra}
 
 
 def model_class(config: dict):

@@ -1,4 +1,4 @@
-"""Ops of the layered decoders (mixers, token-table experts, 32-bit residual stream): CUDA tensors go to the sm_100a
+"""Ops of the layered decoders (mixers, experts, 32-bit residual stream): CUDA tensors go to the sm_100a
 kernels, CPU tensors to the PyTorch statements in ``mixer_torch``.  Activations are bf16 (serving) or fp32 (a model run
 in 32-bit); the residual stream, scores, norms and recurrent states are fp32 either way.
 
@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
+from typing import NamedTuple
 
 import torch
 
@@ -24,22 +25,26 @@ def _lib():
     if not _declared:
         P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
         for name, args in {
-            "b200_residual_norm": [P, P, I, P, P, P, P, I, I, F, L, P, P, L, F, P, P, I, I, L, I, I, I, I, P, P],
+            "b200_residual_norm": [P, P, I, F, P, P, P, P, F, P, L, F, P, P, I, I, L, I, I, I, I, P, P],
             "b200_moe_plan": [P, P, I, I, I, P, P, P, P, L, P, I, P, P],
             "b200_moe_plan_layers": [],
             "b200_add_normed": [P, P, I, P, P, L, P, P, L, F, I, I, I, P, P],
             "b200_glu_any": [P, P, L, I, L, L, I, I, P],
-            "b200_gate_sigmoid": [P, P, L, I, L, L, I, P],
-            "b200_gemm_f32": [P, P, P, I, I, I, L, L, L, I, P, I, I, I, I, P],
-            "b200_gemm_bf16_grouped": [P, P, P, P, I, I, I, L, L, L, L, P, I, I, I, I, I, I, I, P, P],
+            "b200_gate_sigmoid": [P, P, L, I, I, L, L, I, P],
+            "b200_gemm_f32": [P, P, P, I, I, I, L, L, L, I, P, I, I, I, I, P, P],
+            "b200_gemm_bf16_grouped": [P, P, P, P, I, I, I, L, L, L, L, P, I, I, I, I, I, I, I, I, P, P, P],
+            "b200_moe_route": [P, L, P, P, P, P, P, P, I, I, I, I, P],
+            "b200_moe_dispatch": [P, L, P, L, P, P, P, P, P, I, I, I, I, I, I, P],
             "b200_latent_norm_append": [P, L, P, P, P, L, P, P, I, I, I, I, L, F, I, P, P],
             "b200_latent_gather": [P, P, P, P, P, I, I, I, I, I, I, P, P],
-            "b200_latent_attn_rows": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
-            "b200_latent_decode": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
-            "b200_latent_decode_tc": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
-            "b200_flash_window_fwd": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, L, L, L, L, P, P],
+            "b200_latent_rotate": [P, L, P, L, I, I, I, I, P, P, I, P, P, P, P, I, I, I, I, I, I, I, L, F, I, P, P],
+            "b200_latent_attn_rows": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, P],
+            "b200_latent_decode": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
+            "b200_latent_decode_tc": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
+            "b200_flash_window_fwd": [P, P, P, P, P, P, P, I, I, I, I, P, P, P],
             "b200_retention_chunk": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
             "b200_grouped_prep": [P, L, P, P, P, P, P, P, P, I, I, I, L, P, I, P, P],
+            "b200_grouped_prep_whole": [P, L, P, P, P, P, P, P, P, I, I, I, L, P, I, P, P],
             "b200_grouped_rows": [P, P, P, L, P, L, P, I, P, P, P, P, I, I, I, I, I, P, I, P, P],
             "b200_grouped_decode": [P, P, P, L, P, L, P, I, P, P, P, P, P, I, I, I, I, I, P, P, P],
             "b200_grouped_prefill": [P, P, P, L, P, L, P, I, P, P, P, I, I, I, I, I, I, P, P, P],
@@ -77,42 +82,62 @@ def padded_weight(w, dtype, device):
 
 
 # --------------------------------------------------------------------------------- matrix products
-def linear(a, w, out=None, accumulate=False, out_dtype=None):
-    """a (R, K) @ w (N, K)^T.  ``accumulate`` adds to an fp32 ``out``."""
+ACTS = {None: 0, "gelu": 1, "cap": 2}
+
+
+def _finish(bias, alpha, act, cap):
+    """What becomes of a product's sums, or None if nothing does."""
+    _req(act in ACTS and (act != "cap" or cap > 0.0), "unknown activation")
+    if bias is None and alpha == 1.0 and act is None:
+        return None
+    _req(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous()), "a bias is contiguous fp32")
+    return native.GemmFinish(_ptr(bias), float(alpha), float(cap), ACTS[act])
+
+
+def _ref(struct):
+    return None if struct is None else ctypes.byref(struct)
+
+
+def linear(a, w, out=None, accumulate=False, out_dtype=None, bias=None, alpha: float = 1.0, act: str | None = None, cap: float = 0.0):
+    """act(alpha * (a (R, K) @ w (N, K)^T + bias)), bias fp32.  ``accumulate`` adds to an fp32 ``out``; act: "gelu" (with erf),
+    "cap" (cap * tanh(v / cap)) or nothing."""
     if out is None:
         out = rows_buffer(a.shape[0], w.shape[0], out_dtype or a.dtype, a.device)
     if not a.is_cuda:
-        r = a.float() @ w.float().t()
+        r = mixer_torch.finish(a.float() @ w.float().t(), bias, alpha, act, cap)
         out.copy_(out + r if accumulate else r)
         return out
+    _req(bias is None or bias.numel() == w.shape[0], "bad bias")
+    finish = _finish(bias, alpha, act, cap)
     if a.dtype == torch.bfloat16:
-        return native.gemm(a, w, "nt", out=out, accumulate=accumulate, b_stable=True)
+        return native.gemm(a, w, "nt", out=out, accumulate=accumulate, b_stable=True, finish=finish)
     _req(out.dtype == torch.float32 and w.dtype == torch.float32 and a.shape[1] == w.shape[1], "fp32 product of fp32 operands")
     _check(_lib().b200_gemm_f32(_ptr(a), _ptr(w), _ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0), w.stride(0),
-                                out.stride(0), int(accumulate), None, 0, 1, 0, 0, _stream()), "gemm_f32")
+                                out.stride(0), int(accumulate), None, 0, 1, 0, 0, _ref(finish), _stream()), "gemm_f32")
     return out
 
 
-def gemm_rows(a, w, tile_group, n: int, swiglu: bool):
+def gemm_rows(a, w, tile_group, n: int, swiglu: bool, act: str | None = None):
     """Every 128-row tile t of a (P, K) times the rows of w that belong to group tile_group[t] (negative: skipped, the
     rows of the result stay undefined).  ``swiglu``: a group has 2 n rows, gate rows first, and the result is
-    silu(gate) * up; otherwise n rows."""
+    silu(gate) * up; otherwise n rows and ``act`` of the product."""
     rows = 2 * n if swiglu else n
     if not a.is_cuda:
-        return mixer_torch.gemm_rows(a, w, tile_group, rows, n, swiglu)
+        return mixer_torch.gemm_rows(a, w, tile_group, rows, n, swiglu, act)
     lib = _lib()
     p, k = a.shape
     _req(tile_group.dtype == torch.int32 and tile_group.is_contiguous() and tile_group.numel() * TILE >= p and p % TILE == 0
-         and w.shape[0] % rows == 0 and w.shape[1] == k, "bad grouped product")
+         and w.shape[0] % rows == 0 and w.shape[1] == k and not (swiglu and act), "bad grouped product")
+    finish = _finish(None, 1.0, act, 0.0)
     if a.dtype == torch.bfloat16:
         out = rows_buffer(p, n, a.dtype, a.device)
         _check(lib.b200_gemm_bf16_grouped(_ptr(a), _ptr(w), _ptr(out), None, p, n, k, a.stride(0), w.stride(0), out.stride(0),
-                                          0, _ptr(tile_group), w.shape[0] // rows, rows, 1, 0, 0, int(swiglu), 0,
+                                          0, _ptr(tile_group), w.shape[0] // rows, rows, 1, 0, 0, int(swiglu), 0, 0, _ref(finish),
                                           _ptr(native.status_word(a.device)), _stream()), "gemm_grouped")
         return out
     out = rows_buffer(p, rows, a.dtype, a.device)
     _check(lib.b200_gemm_f32(_ptr(a), _ptr(w), _ptr(out), p, rows, k, a.stride(0), w.stride(0), out.stride(0), 0,
-                             _ptr(tile_group), rows, 1, 0, 0, _stream()), "gemm_f32")
+                             _ptr(tile_group), rows, 1, 0, 0, _ref(finish), _stream()), "gemm_f32")
     if not swiglu:
         return out
     h = rows_buffer(p, n, a.dtype, a.device)
@@ -130,7 +155,7 @@ def glu(a, w, n: int, act: str):
     m, k = a.shape
     if a.dtype == torch.bfloat16:
         _check(lib.b200_gemm_bf16_grouped(_ptr(a), _ptr(w), _ptr(out), None, m, n, k, a.stride(0), w.stride(0), out.stride(0), 0, None,
-                                          0, 2 * n, 1, 0, 0, 2 if act == "relu" else 1, native.EPI_B_STABLE,
+                                          0, 2 * n, 1, 0, 0, 2 if act == "relu" else 1, native.EPI_B_STABLE, 0, None,
                                           _ptr(native.status_word(a.device)), _stream()), "gemm_glu")
         return out
     gu = linear(a, w)
@@ -138,56 +163,99 @@ def glu(a, w, n: int, act: str):
     return out
 
 
-def gemm_heads(a, w, heads: int, k: int, n: int, out=None, gate=None):
-    """One product per head, side by side: out[:, h n : (h+1) n] = a[:, h k : (h+1) k] @ w_h^T, w_h = rows
-    [h w.shape[0] / heads, ...) of w; ``gate`` multiplies with sigmoid(gate), element by element."""
+def gemm_heads(a, w, heads: int, k: int, n: int, out=None, gate=None, a_step: int | None = None, c_step: int | None = None):
+    """One product per head, side by side: out[:, h c_step : h c_step + n] = a[:, h a_step : h a_step + k] @ w_h^T, w_h = rows
+    [h w.shape[0] / heads, ...) of w (the steps are k and n unless given); ``gate`` multiplies with sigmoid(gate), element by
+    element or, with one column per head, head by head."""
+    a_step, c_step = a_step or k, c_step or n
     if out is None:
         out = rows_buffer(a.shape[0], heads * n, a.dtype, a.device)
     if not a.is_cuda:
-        return mixer_torch.gemm_heads(a, w, heads, k, n, out, gate)
+        return mixer_torch.gemm_heads(a, w, heads, k, n, out, gate, a_step, c_step)
     lib = _lib()
-    _req(w.shape[0] % heads == 0 and w.shape[1] == k and a.shape[1] >= heads * k and out.shape[1] >= heads * n, "bad head product")
+    _req(w.shape[0] % heads == 0 and w.shape[1] == k and a.shape[1] >= (heads - 1) * a_step + k
+         and out.shape[1] >= (heads - 1) * c_step + n, "bad head product")
+    by_head = gate is not None and gate.shape[1] == heads
+    _req(gate is None or by_head or (gate.shape[1] >= heads * n and c_step == n), "bad gate")
     if a.dtype == torch.bfloat16:
-        _req(k % 8 == 0, "a head's columns must start on a 16-byte boundary")
+        _req(k % 8 == 0 and a_step % 8 == 0, "a head's columns must start on a 16-byte boundary")
         epi = (5 if gate is not None else 0) | native.EPI_B_STABLE
         _check(lib.b200_gemm_bf16_grouped(_ptr(a), _ptr(w), _ptr(out), _ptr(gate), a.shape[0], n, k, a.stride(0), w.stride(0),
                                           out.stride(0), 0 if gate is None else gate.stride(0), None, 0, w.shape[0] // heads,
-                                          heads, k, n, 0, epi, _ptr(native.status_word(a.device)), _stream()), "gemm_heads")
+                                          heads, a_step, c_step, 0, epi, int(by_head), None, _ptr(native.status_word(a.device)),
+                                          _stream()), "gemm_heads")
         return out
     _check(lib.b200_gemm_f32(_ptr(a), _ptr(w), _ptr(out), a.shape[0], n, k, a.stride(0), w.stride(0), out.stride(0), 0, None,
-                             w.shape[0] // heads, heads, k, n, _stream()), "gemm_f32")
+                             w.shape[0] // heads, heads, a_step, c_step, None, _stream()), "gemm_f32")
     if gate is not None:
         gate_sigmoid_(out, gate)
     return out
 
 
 def gate_sigmoid_(o, gate):
+    """o (R, n) times sigmoid(gate (R, m)), every gate for n / m columns."""
+    n, m = o.shape[1], gate.shape[1]
+    _req(n % m == 0 and o.shape[0] == gate.shape[0] and o.dtype == gate.dtype, "gate and output must match")
     if not o.is_cuda:
-        return o.mul_(torch.sigmoid(gate.float()).to(o.dtype))
-    _req(o.shape == gate.shape and o.dtype == gate.dtype, "gate and output must match")
-    _check(_lib().b200_gate_sigmoid(_ptr(o), _ptr(gate), o.shape[0], o.shape[1], o.stride(0), gate.stride(0), _f32(o),
+        return o.mul_(torch.sigmoid(gate.float()).repeat_interleave(n // m, 1).to(o.dtype))
+    _check(_lib().b200_gate_sigmoid(_ptr(o), _ptr(gate), o.shape[0], n, n // m, o.stride(0), gate.stride(0), _f32(o),
                                     _stream()), "gate_sigmoid")
     return o
 
 
 # ------------------------------------------------------------------------------- residual and norm
-def residual_norm(x, w=None, eps: float = 0.0, tokens=None, embed=None, row_index=None, pending=None, scatter=None):
+class ExpertOutputs(NamedTuple):
+    """What the experts of a layer add to the residual stream: x += scale * (sum_k weight[row, k] * y[pos[row, k]] + sigmoid(sgate[row])
+    * s[row]); a choice with pos -2 stands for the experts' input z[row], -1 for none; without ``weight`` all weights are one."""
+    y: torch.Tensor
+    pos: torch.Tensor                        # (R, top) int32
+    scale: float
+    weight: torch.Tensor | None = None       # (R, top) fp32
+    z: torch.Tensor | None = None
+    s: torch.Tensor | None = None
+    sgate: torch.Tensor | None = None        # (R,) fp32, any stride
+
+
+class _NativeOutputs(ctypes.Structure):
+    """csrc/mixer_elementwise.cu: ExpertOutputs"""
+    _fields_ = [(n, ctypes.c_void_p) for n in ("y", "ypos", "yweight", "z", "s", "sgate")] + \
+               [(n, ctypes.c_longlong) for n in ("ld_y", "ld_z", "ld_s", "ld_sgate")] + \
+               [("ytop", ctypes.c_int), ("y_rows", ctypes.c_int), ("yscale", ctypes.c_float)]
+
+
+def _expert_outputs(ex: ExpertOutputs, x, act_dtype):
+    rows, d = x.shape
+    fits = lambda t, n: t is None or (t.dtype == act_dtype and t.shape == (n, d) and t.stride(1) == 1)
+    _req(fits(ex.y, ex.y.shape[0]) and fits(ex.z, rows) and fits(ex.s, rows) and ex.pos.dtype == torch.int32
+         and ex.pos.is_contiguous() and ex.pos.shape[0] == rows, "bad expert outputs")
+    _req(ex.weight is None or (ex.weight.dtype == torch.float32 and ex.weight.is_contiguous() and ex.weight.shape == ex.pos.shape),
+         "bad expert weights")
+    _req(ex.sgate is None or (ex.sgate.dtype == torch.float32 and ex.sgate.shape == (rows,)), "bad gate")
+    pitch_of = lambda t: 0 if t is None else t.stride(0)
+    return _NativeOutputs(_ptr(ex.y), _ptr(ex.pos), _ptr(ex.weight), _ptr(ex.z), _ptr(ex.s), _ptr(ex.sgate), pitch_of(ex.y),
+                          pitch_of(ex.z), pitch_of(ex.s), pitch_of(ex.sgate), ex.pos.shape[1], ex.y.shape[0], float(ex.scale))
+
+
+def residual_norm(x, w=None, eps: float = 0.0, tokens=None, embed=None, row_index=None, pending=None, scatter=None,
+                  embed_scale: float = 1.0, w_offset: float = 0.0):
     """One pass over the fp32 residual stream x (R, d):
 
-    * ``tokens`` / ``embed``: x = embed[tokens] first
-    * ``pending`` = (y, pos (R, top), scale): x += scale * sum_k y[pos[row, k]] (expert outputs; -1 = none)
-    * ``w``: h = x / rms(x) * w, returned in w's dtype (no ``w``: only x is updated)
+    * ``tokens`` / ``embed``: x = embed[tokens] * embed_scale first
+    * ``pending``: ``ExpertOutputs`` (or its first three fields) to add to x
+    * ``w``: h = x / rms(x) * (w + w_offset), returned in w's dtype (no ``w``: only x is updated)
     * ``row_index``: h for these rows of x only, x itself stays as it is
     * ``scatter`` = (pos (R, top), rows): also returns the normed rows at the places the experts read them from
 
     Returns (h, scattered)."""
+    if pending is not None:
+        pending = ExpertOutputs(*pending)
     if not x.is_cuda:
-        return mixer_torch.residual_norm(x, tokens, embed, row_index, pending, w, eps, scatter)
+        return mixer_torch.residual_norm(x, tokens, embed, row_index, pending, w, eps, scatter, embed_scale, w_offset)
     lib = _lib()
     _req(x.dtype == torch.float32 and x.is_contiguous(), "the residual stream is contiguous fp32")
     d = x.shape[1]
     rows = x.shape[0] if row_index is None else row_index.numel()
-    act = w if w is not None else (embed if embed is not None else pending[0])
+    act = w if w is not None else (embed if embed is not None else pending.y)
     h = xg = None
     if w is not None:
         _req(w.numel() == d and w.is_contiguous(), "bad norm weight")
@@ -197,20 +265,14 @@ def residual_norm(x, w=None, eps: float = 0.0, tokens=None, embed=None, row_inde
              and embed.dtype == act.dtype, "bad embedding")
     if row_index is not None:
         _req(row_index.dtype == torch.int64 and row_index.is_contiguous(), "row_index must be int64")
-    y = ypos = None
-    scale = 1.0
-    if pending is not None:
-        y, ypos, scale = pending
-        _req(y.dtype == act.dtype and y.shape[1] == d and ypos.dtype == torch.int32 and ypos.is_contiguous()
-             and ypos.shape[0] == x.shape[0], "bad expert outputs")
+    ex = None if pending is None else _expert_outputs(pending, x, act.dtype)
     gpos, g_rows = scatter if scatter is not None else (None, 0)
     if scatter is not None:
         _req(gpos.dtype == torch.int32 and gpos.is_contiguous() and gpos.shape[0] == rows, "bad expert positions")
         xg = rows_buffer(g_rows, d, w.dtype, x.device)
     _check(lib.b200_residual_norm(
-        _ptr(tokens), _ptr(embed), 0 if embed is None else embed.shape[0], _ptr(x), _ptr(row_index), _ptr(y), _ptr(ypos),
-        0 if ypos is None else ypos.shape[1], 0 if y is None else y.shape[0], float(scale), 0 if y is None else y.stride(0),
-        _ptr(w), _ptr(h), 0 if h is None else h.stride(0), float(eps), _ptr(xg), _ptr(gpos),
+        _ptr(tokens), _ptr(embed), 0 if embed is None else embed.shape[0], float(embed_scale), _ptr(x), _ptr(row_index), _ref(ex),
+        _ptr(w), float(w_offset), _ptr(h), 0 if h is None else h.stride(0), float(eps), _ptr(xg), _ptr(gpos),
         0 if gpos is None else gpos.shape[1], g_rows, 0 if xg is None else xg.stride(0), rows, x.shape[0], d, _f32(act),
         _ptr(native.status_word(x.device)), _stream()), "residual_norm")
     return h, xg
@@ -268,6 +330,40 @@ def moe_plan(tokens, slots, tables, experts):
     return ([pos[i, :rows * t.shape[1]].view(rows, t.shape[1]) for i, t in enumerate(tables)], [group[i] for i in range(len(tables))])
 
 
+def moe_route(z, correction, slots, experts: int, top: int, count):
+    """Choose experts by score: z (R, outputs) fp32 logits of the experts and, behind them, of identities; scores are their softmax.  The
+    ``top`` outputs with the largest score + correction are chosen and weighted by their share of the chosen scores.  ``count``
+    (experts,) int32, zero on entry, receives the rows per expert.  Returns choice (-1 in padding rows), rank among the expert's
+    rows, weight, each (R, top)."""
+    rows, outputs = z.shape
+    if not z.is_cuda:
+        return mixer_torch.moe_route(z, correction, slots, experts, top, count)
+    _req(z.dtype == torch.float32 and z.stride(1) == 1 and correction.dtype == torch.float32 and correction.numel() == outputs
+         and correction.is_contiguous() and count.dtype == torch.int32 and count.is_contiguous() and count.numel() == experts
+         and slots.dtype == torch.int64 and slots.numel() == rows and 0 < top <= outputs and experts <= outputs, "bad router inputs")
+    choice, rank = (torch.empty((rows, top), dtype=torch.int32, device=z.device) for _ in range(2))
+    weight = torch.empty((rows, top), dtype=torch.float32, device=z.device)
+    _check(_lib().b200_moe_route(_ptr(z), z.stride(0), _ptr(correction), _ptr(slots), _ptr(choice), _ptr(rank), _ptr(weight),
+                                 _ptr(count), rows, experts, outputs, top, _stream()), "moe_route")
+    return choice, rank, weight
+
+
+def moe_dispatch(h, choice, rank, count):
+    """Rows of h sorted by chosen expert into 128-row tiles.  Returns them (tiles * 128, d), where each choice went, pos (R, top) int32
+    (-2: an identity, -1: none), and the expert of every tile, tile_group (tiles,) int32."""
+    (rows, top), experts = choice.shape, count.numel()
+    tiles = plan_tiles(rows, experts, top)
+    if not h.is_cuda:
+        return mixer_torch.moe_dispatch(h, choice, rank, count, tiles)
+    _req(h.stride(1) == 1 and h.shape[0] == rows and choice.dtype == torch.int32 and rank.dtype == torch.int32, "bad expert rows")
+    xg = rows_buffer(tiles * TILE, h.shape[1], h.dtype, h.device)
+    pos = torch.empty((rows, top), dtype=torch.int32, device=h.device)
+    group = torch.empty((tiles,), dtype=torch.int32, device=h.device)
+    _check(_lib().b200_moe_dispatch(_ptr(h), h.stride(0), _ptr(xg), xg.stride(0), _ptr(choice), _ptr(rank), _ptr(count), _ptr(pos),
+                                    _ptr(group), rows, experts, top, tiles, h.shape[1], h.element_size(), _stream()), "moe_dispatch")
+    return xg, pos, group
+
+
 # -------------------------------------------------------------------------------- latent attention
 def latent_norm_append(proj, wq, wkv, eps: float, cache, slots):
     """Norm of both latents in proj (columns [0, q_rank) and [q_rank, q_rank + kv_rank)): returns the query latent and
@@ -285,23 +381,47 @@ def latent_norm_append(proj, wq, wkv, eps: float, cache, slots):
     return cq
 
 
-def latent_attention_rows(q, cache, row_seq, positions, slots, tables, heads: int, window: int, scale: float):
-    """q (R, heads * width) in latent space against the paged latents; every row has its own position and line of
-    ``tables`` (``row_seq`` None: line i for row i).  window 0 = none.  Returns (R, heads * width)."""
+def latent_rotate(q, q_col: int, q_pitch: int, kv, kv_col: int | None, k_col: int | None, wkv, ql, cache, cos_sin, positions, slots,
+                  heads: int, kv_rank: int, vwidth: int, rot: int, eps: float):
+    """Rotation (interleaved pairs) and append: the heads' rotated query parts are columns q_col + h * q_pitch ... of ``q``; those of
+    the first rows go behind the queries in latent space, ``ql`` (rows, heads * width), the others stay in place.  The latent at
+    column ``kv_col`` of ``kv`` (None: no latent here) is normed and, with the rotated key part at ``k_col`` (None: none), written to
+    its cache slot: latent, then from column ``vwidth`` on the key part."""
+    n = 0 if ql is None else ql.shape[0]
     if not q.is_cuda:
-        return mixer_torch.latent_attention(q, cache, row_seq, positions, slots, tables, heads, window, scale)
+        return mixer_torch.latent_rotate(q, q_col, q_pitch, kv, kv_col, k_col, wkv, ql, cache, cos_sin, positions, slots, heads,
+                                         kv_rank, vwidth, rot, eps)
+    width = cache.shape[-1]
+    _req(cache.is_contiguous() and cache.dtype == q.dtype and slots.dtype == torch.int64 and slots.numel() == q.shape[0]
+         and positions.dtype == torch.int32 and q.stride(1) == 1 and kv.stride(1) == 1 and kv.dtype == q.dtype
+         and kv.shape[0] == q.shape[0], "bad latent cache or rows")
+    _req(cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[2] == rot // 2, "bad rotary table")
+    _req(ql is None or (ql.is_contiguous() and ql.dtype == q.dtype and ql.shape[1] == heads * width), "bad latent queries")
+    _check(_lib().b200_latent_rotate(
+        _ptr(q), q.stride(0), _ptr(kv), kv.stride(0), q_col, q_pitch, -1 if kv_col is None else kv_col, -1 if k_col is None else k_col, _ptr(wkv), _ptr(ql),
+        n, _ptr(cache), _ptr(cos_sin), _ptr(positions), _ptr(slots), q.shape[0], heads, kv_rank, vwidth, width, rot, cos_sin.shape[1],
+        cache.shape[0] * cache.shape[1], float(eps), _f32(q), _ptr(native.status_word(q.device)), _stream()), "latent_rotate")
+
+
+def latent_attention_rows(q, cache, row_seq, positions, slots, tables, heads: int, window: int, scale: float, vwidth: int | None = None):
+    """q (R, heads * width) in latent space against the paged latents; every row has its own position and line of
+    ``tables`` (``row_seq`` None: line i for row i).  window 0 = none.  Returns (R, heads * vwidth): what is summed up are the first
+    ``vwidth`` columns of a cached vector (all of them unless given)."""
+    vwidth = vwidth or cache.shape[-1]
+    if not q.is_cuda:
+        return mixer_torch.latent_attention(q, cache, row_seq, positions, slots, tables, heads, window, scale, vwidth)
     _req(q.is_contiguous() and cache.is_contiguous() and q.dtype == cache.dtype and q.shape[1] == heads * cache.shape[-1],
          "bad latent queries")
     _req(tables.dtype == torch.int32 and tables.is_contiguous() and positions.dtype == torch.int32, "bad tables")
-    out = torch.empty_like(q)
+    out = torch.empty((q.shape[0], heads * vwidth), dtype=q.dtype, device=q.device)
     _check(_lib().b200_latent_attn_rows(_ptr(q), _ptr(cache), _ptr(out), _ptr(row_seq), _ptr(positions), _ptr(slots),
-                                        _ptr(tables), tables.shape[0], q.shape[0], heads, cache.shape[-1], tables.shape[1],
+                                        _ptr(tables), tables.shape[0], q.shape[0], heads, cache.shape[-1], vwidth, tables.shape[1],
                                         cache.shape[1], cache.shape[0], window, float(scale), _f32(q),
                                         _ptr(native.status_word(q.device)), _stream()), "latent_attn_rows")
     return out
 
 
-DECODE_MAX_WIDTH = 512           # latents the tensor-core decode kernel holds in shared memory
+DECODE_MAX_WIDTH, DECODE_MAX_KEY = 512, 576      # what the tensor-core decode kernels sum up, and score, of a cached vector
 DECODE_TILE = 32
 
 
@@ -330,17 +450,21 @@ def latent_splits_tc(rows: int, keys: int, sms: int = 148) -> int:
     return best
 
 
-def latent_decode(q, cache, positions, slots, tables, heads: int, window: int, scale: float, splits: int = 0, kernel: str = "auto"):
+def latent_decode(q, cache, positions, slots, tables, heads: int, window: int, scale: float, splits: int = 0, kernel: str = "auto",
+                  vwidth: int | None = None):
     """``latent_attention_rows`` for one query row per request: line i of ``tables`` belongs to row i.  ``kernel``: "tcgen05"
-    (widths that are multiples of 128, up to 64 heads, pages that divide 128), "mma" (any width up to 512), "rows"; "auto"
-    takes the first that fits, and "mma" for small batches, whose CTAs it spreads over the SMs with shorter chains."""
+    (vwidths that are multiples of 128, up to 64 columns behind them, up to 64 heads, pages that divide 128), "mma" (any width up to
+    ``DECODE_MAX_KEY``), "rows"; "auto" takes the first that fits, and "mma" for small batches, whose CTAs it spreads over the SMs
+    with shorter chains."""
     width, page = cache.shape[-1], cache.shape[1]
+    vwidth = vwidth or width
     if kernel == "auto":
-        fits = q.is_cuda and q.dtype == torch.bfloat16 and width <= DECODE_MAX_WIDTH
-        tc = fits and width % 128 == 0 and heads <= 64 and page >= 8 and 128 % page == 0 and q.shape[0] * max(heads, 16) >= 1024
+        fits = q.is_cuda and q.dtype == torch.bfloat16 and vwidth <= DECODE_MAX_WIDTH and width <= DECODE_MAX_KEY
+        tc = (fits and vwidth % 128 == 0 and width <= vwidth + 64 and heads <= 64 and page >= 8 and 128 % page == 0
+              and q.shape[0] * max(heads, 16) >= 1024)
         kernel = "tcgen05" if tc else ("mma" if fits else "rows")
     if kernel == "rows":
-        return latent_attention_rows(q, cache, None, positions, slots, tables, heads, window, scale)
+        return latent_attention_rows(q, cache, None, positions, slots, tables, heads, window, scale, vwidth)
     rows = q.shape[0]
     _req(q.is_contiguous() and cache.is_contiguous() and q.shape[1] == heads * width and tables.shape[0] >= rows, "bad latent queries")
     _req(q.dtype == torch.bfloat16 and cache.dtype == q.dtype, "bf16 queries and latents")
@@ -351,11 +475,11 @@ def latent_decode(q, cache, positions, slots, tables, heads: int, window: int, s
         fn, splits = _lib().b200_latent_decode_tc, splits or latent_splits_tc(rows, keys)
     else:
         fn, splits = _lib().b200_latent_decode, splits or latent_splits(rows, heads, keys)
-    out = torch.empty_like(q)
-    part = torch.empty(rows * heads * splits * (width + 2) if splits > 1 else 0, dtype=torch.float32, device=q.device)
-    ml = part[rows * heads * splits * width:]
+    out = torch.empty((rows, heads * vwidth), dtype=q.dtype, device=q.device)
+    part = torch.empty(rows * heads * splits * (vwidth + 2) if splits > 1 else 0, dtype=torch.float32, device=q.device)
+    ml = part[rows * heads * splits * vwidth:]
     _check(fn(_ptr(q), _ptr(cache), _ptr(out), _ptr(part), _ptr(ml), _ptr(positions), _ptr(slots), _ptr(tables), rows, heads, width,
-              tables.shape[1], page, cache.shape[0], window, splits, float(scale), _ptr(native.status_word(q.device)), _stream()),
+              vwidth, tables.shape[1], page, cache.shape[0], window, splits, float(scale), _ptr(native.status_word(q.device)), _stream()),
            "latent_decode" if splits > 1 else "latent_decode_one")
     return out
 
@@ -372,17 +496,38 @@ def latent_gather(cache, cu_k, first_k, tables, total: int):
     return out
 
 
-def window_attention(q, kv, cu_q, cu_k, max_q: int, heads: int, head_dim: int, vdim: int, window: int, scale: float, out, gate=None):
-    """Softmax attention of packed portions under a sliding window on the tensor cores: q (Rq, heads * head_dim), kv (Rk, 2 *
-    heads * head_dim) = K | V with zero columns up to head_dim (64 or 128); the queries of a portion are the last
-    positions of its keys.  out (Rq, heads * vdim), times sigmoid(gate)."""
+class _WindowShape(ctypes.Structure):
+    """csrc/flash_attn_fwd.cu: FlashWindowShape"""
+    _fields_ = [(n, ctypes.c_longlong) for n in ("ld_q", "ld_kv", "ld_kr", "ld_o", "ld_gate")] + \
+               [(n, ctypes.c_int) for n in ("q_cols", "kv_cols", "kr_cols", "heads", "dim", "vdim", "q_step", "k_step", "v_step", "v_off",
+                                            "rot", "qr_col", "qr_step", "kr_col", "window", "head_gate")] + [("scale", ctypes.c_float)]
+
+
+def window_attention(q, kv, cu_q, cu_k, max_q: int, heads: int, dim: int, vdim: int, window: int, scale: float, out, gate=None,
+                     steps=None, rot=None):
+    """Softmax attention of packed portions under a sliding window (0 = none) on the tensor cores: a head's queries are ``dim`` columns of
+    q (Rq, ...), its keys and values ``dim`` and ``vdim`` columns of kv (Rk, ...), up to 128 each; the queries of a portion are the
+    last positions of its keys.  ``steps`` = (q_step, k_step, v_step, v_off): head h starts at columns h q_step, h k_step,
+    v_off + h v_step (default: heads of ``dim`` columns side by side, all keys before all values); columns from ``dim`` up to the next
+    multiple of 16 must be finite, and zero in q or kv.  ``rot`` = (kr (Rk, ...), dims, qr_col, qr_step, kr_col): the scores gain
+    rotated parts, ``dims`` (up to 64) columns of q at qr_col + h qr_step and of kr, for all heads, at kr_col.
+    out (Rq, heads * vdim), times sigmoid(gate), element by element or with a column per head."""
+    q_step, k_step, v_step, v_off = steps or (dim, dim, dim, heads * dim)
+    kr, dims, qr_col, qr_step, kr_col = rot or (None, 0, 0, 0, 0)
     _req(q.dtype == torch.bfloat16 and kv.dtype == torch.bfloat16 and q.stride(1) == 1 and kv.stride(1) == 1, "bf16 queries and keys")
-    _req(q.shape[1] == heads * head_dim and kv.shape[1] == 2 * heads * head_dim and out.shape == (q.shape[0], heads * vdim), "bad shapes")
+    _req(q.shape[1] >= (heads - 1) * q_step + dim and kv.shape[1] >= max((heads - 1) * k_step + dim, v_off + (heads - 1) * v_step + vdim)
+         and out.shape == (q.shape[0], heads * vdim), "bad shapes")
+    _req(kr is None or (kr.dtype == torch.bfloat16 and kr.stride(1) == 1 and kr.shape[0] == kv.shape[0] and kr.shape[1] >= kr_col + dims
+                        and q.shape[1] >= qr_col + (heads - 1) * qr_step + dims), "bad rotated parts")
+    _req(gate is None or gate.shape in ((q.shape[0], heads), tuple(out.shape)), "bad gate")
     _req(cu_q.dtype == torch.int32 and cu_k.dtype == torch.int32 and cu_q.numel() == cu_k.numel(), "bad row offsets")
+    by_head = gate is not None and gate.shape[1] == heads
+    shape = _WindowShape(q.stride(0), kv.stride(0), 0 if kr is None else kr.stride(0), out.stride(0), 0 if gate is None else gate.stride(0),
+                         q.shape[1], kv.shape[1], 0 if kr is None else kr.shape[1], heads, dim, vdim, q_step, k_step, v_step, v_off,
+                         dims, qr_col, qr_step, kr_col, window, int(by_head), float(scale))
     _check(_lib().b200_flash_window_fwd(
-        _ptr(q), _ptr(kv), _ptr(out), _ptr(gate), _ptr(cu_q), _ptr(cu_k), cu_q.numel() - 1, max_q, q.shape[0], kv.shape[0], heads,
-        head_dim, vdim, window, float(scale), q.stride(0), kv.stride(0), out.stride(0), 0 if gate is None else gate.stride(0),
-        _ptr(native.status_word(q.device)), _stream()), "flash_window_fwd")
+        _ptr(q), _ptr(kv), _ptr(kr), _ptr(out), _ptr(gate), _ptr(cu_q), _ptr(cu_k), cu_q.numel() - 1, max_q, q.shape[0], kv.shape[0],
+        ctypes.byref(shape), _ptr(native.status_word(q.device)), _stream()), "flash_window_fwd")
     return out
 
 
@@ -492,7 +637,8 @@ def mlstm(proj, gates, gate_bias, weight, state, state_slots, cu, spans, positio
 @dataclass
 class AttentionShape:
     """Sizes and constants of one grouped attention (``models.mixers.GroupedAttention``); ``bias`` (heads, n) fp32 holds the bias
-    per distance, distances from n - 1 on read its last column."""
+    per distance, distances from n - 1 on read its last column.  ``softcap`` 0: scores are not capped; ``sink`` (heads,) fp32 or None;
+    ``whole_norm``: one norm over all queries (and keys) of a token instead of one per head."""
     heads: int
     kv_heads: int
     maps: int
@@ -505,6 +651,10 @@ class AttentionShape:
     difference: float = 0.0
     out_scale: float = 1.0
     bias: torch.Tensor | None = None
+    keep: int = 0
+    softcap: float = 0.0
+    sink: torch.Tensor | None = None
+    whole_norm: bool = False
 
     @property
     def q_pitch(self) -> int:
@@ -526,15 +676,16 @@ class AttentionShape:
 
 class _NativeShape(ctypes.Structure):
     """csrc/grouped_attention.cuh: GroupedShape"""
-    _fields_ = [(n, ctypes.c_int) for n in ("heads", "kv_heads", "maps", "dim", "vdim", "qp", "kp", "vp", "window")] + \
-               [(n, ctypes.c_float) for n in ("scale", "eps", "difference", "out_scale")]
+    _fields_ = [(n, ctypes.c_int) for n in ("heads", "kv_heads", "maps", "dim", "vdim", "qp", "kp", "vp", "window", "keep")] + \
+               [(n, ctypes.c_float) for n in ("scale", "eps", "difference", "out_scale", "softcap")] + [("sink", ctypes.c_void_p)]
 
 
 def _native_shape(s: AttentionShape):
     got = s.__dict__.get("_native")
     if got is None:
         got = s.__dict__["_native"] = _NativeShape(s.heads, s.kv_heads, s.maps, s.dim, s.vdim, s.q_pitch, s.k_pitch, s.v_pitch,
-                                                   s.window, s.scale, s.eps, s.difference, s.out_scale)
+                                                   s.window, s.keep, s.scale, s.eps, s.difference, s.out_scale, s.softcap,
+                                                   _ptr(s.sink))
     return ctypes.byref(got)
 
 
@@ -545,6 +696,8 @@ def attention_tiles(s: AttentionShape, dtype) -> bool:
     """Whether portions of prompts run on the tensor-core kernel."""
     if dtype != torch.bfloat16 or s.dim > 128 or s.vdim > 128:
         return False
+    if s.softcap > 0 and (s.bias is not None or s.maps != 1):
+        return False
     return s.scale > 0 if s.bias is None else s.bias.shape[1] <= BIAS_MAX
 
 
@@ -553,7 +706,7 @@ def attention_pages(page_size: int) -> bool:
 
 
 def attention_prepare(proj, s: AttentionShape, wq, wk, cos_sin, positions, slots, cache):
-    """Queries of ``proj`` (q | k | v | ..., or q | ... without ``wk``) normed and rotated, (R, heads * maps * q_pitch) with zeros
+    """Queries of ``proj`` (q | k | v | ..., or q | ... without ``wk``) normed (per head, or over all of them) and rotated, (R, heads * maps * q_pitch) with zeros
     behind every head; keys, likewise, and values go to their cache slots (negative slot: not written)."""
     q = torch.empty((proj.shape[0], s.heads * s.maps * s.q_pitch), dtype=proj.dtype, device=proj.device)
     if not proj.is_cuda:
@@ -561,7 +714,11 @@ def attention_prepare(proj, s: AttentionShape, wq, wk, cos_sin, positions, slots
     _req(cache.is_contiguous() and cache.dtype == proj.dtype and cache.shape[-1] == s.cache_width and slots.dtype == torch.int64
          and slots.numel() == proj.shape[0] and positions.dtype == torch.int32 and wq.dtype == proj.dtype, "bad cache or rows")
     _req(s.rot == 0 or (cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[2] == s.rot // 2), "bad rotary table")
-    _check(_lib().b200_grouped_prep(_ptr(proj), proj.stride(0), _ptr(q), _ptr(cache), _ptr(wq), _ptr(wk), _ptr(cos_sin),
+    norm = lambda n: s.dim if not s.whole_norm else n * s.dim
+    _req(wq.numel() == norm(s.heads) and wq.is_contiguous() and (wk is None or (wk.numel() == norm(s.kv_heads) and wk.is_contiguous())),
+         "bad norm weights")
+    fn = _lib().b200_grouped_prep_whole if s.whole_norm else _lib().b200_grouped_prep
+    _check(fn(_ptr(proj), proj.stride(0), _ptr(q), _ptr(cache), _ptr(wq), _ptr(wk), _ptr(cos_sin),
                                     _ptr(positions), _ptr(slots), proj.shape[0], s.rot, cos_sin.shape[1] if s.rot else 0,
                                     cache.shape[0] * cache.shape[1], _native_shape(s), _f32(proj),
                                     _ptr(native.status_word(proj.device)), _stream()), "grouped_prep")
@@ -606,7 +763,7 @@ def attention_decode(q, s: AttentionShape, cache, positions, slots, tables, out,
     fits = q.is_cuda and q.dtype == torch.bfloat16 and s.maps * s.k_pitch <= 256 and s.v_pitch <= 128
     if not fits:
         return attention_rows(q, s, cache, None, positions, slots, tables, out, gate)
-    rows, keys = q.shape[0], min(s.window, tables.shape[1] * cache.shape[1])
+    rows, keys = q.shape[0], min(s.window + s.keep, tables.shape[1] * cache.shape[1])
     _req(tables.shape[0] >= rows, "bad tables")
     args = _attention_args(q, s, cache, positions, tables, out, gate)
     splits = splits or attention_splits(s, rows, keys)

@@ -7,20 +7,34 @@ import torch
 TILE = 128
 
 
-def residual_norm(x, tokens, embed, row_index, pending, w, eps, scatter):
-    src = x if tokens is None else embed[tokens.long()].float()
+def finish(r, bias, alpha, act, cap):
+    r = alpha * (r if bias is None else r + bias)
+    if act == "gelu":
+        return torch.nn.functional.gelu(r)
+    return cap * torch.tanh(r / cap) if act == "cap" else r
+
+
+def residual_norm(x, tokens, embed, row_index, pending, w, eps, scatter, embed_scale, w_offset):
+    src = x if tokens is None else embed[tokens.long()].float() * embed_scale
+    pick = (lambda t: t) if row_index is None else (lambda t: t[row_index.long()])
     if row_index is not None:
         src = x[row_index.long()]
     if pending is not None:
-        y, pos, scale = pending
-        rows = pos if row_index is None else pos[row_index.long()]
-        live = rows >= 0
-        src = src + scale * (y.float()[rows.clamp(min=0).long()] * live.unsqueeze(-1)).sum(1)
+        rows = pick(pending.pos)
+        weight = (rows >= 0).float() if pending.weight is None else pick(pending.weight)
+        part = pending.y.float()[rows.clamp(min=0).long()].masked_fill((rows < 0).unsqueeze(-1), 0.0)
+        if pending.z is not None:
+            part = torch.where((rows == -2).unsqueeze(-1), pick(pending.z).float().unsqueeze(1), part)
+        total = (part * weight.unsqueeze(-1)).sum(1)
+        if pending.s is not None:
+            share = 1.0 if pending.sgate is None else torch.sigmoid(pick(pending.sgate)).unsqueeze(1)
+            total = total + share * pick(pending.s).float()
+        src = src + pending.scale * total
     if row_index is None:
         x.copy_(src)
     if w is None:
         return None, None
-    h = (src * torch.rsqrt(src.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(w.dtype)
+    h = (src * torch.rsqrt(src.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + w_offset)).to(w.dtype)
     if scatter is None:
         return h, None
     pos, rows = scatter
@@ -66,7 +80,37 @@ def moe_plan(tokens, slots, tables, experts, tiles):
     return pos, groups
 
 
-def gemm_rows(a, w, tile_group, group_rows, n, swiglu):
+def moe_route(z, correction, slots, experts, top, count):
+    s = torch.softmax(z, -1)
+    choice = torch.topk(s + correction, top, dim=-1).indices
+    weight = s.gather(1, choice)
+    weight = weight / (weight.sum(-1, keepdim=True) + 1e-20)
+    choice, rank = choice.to(torch.int32), torch.full(choice.shape, -1, dtype=torch.int32)
+    choice[slots < 0], weight[slots < 0] = -1, 0.0
+    for r in range(z.shape[0]):
+        for k, e in enumerate(choice[r].tolist()):
+            if 0 <= e < experts:
+                rank[r, k] = count[e]
+                count[e] += 1
+    return choice, rank, weight
+
+
+def moe_dispatch(h, choice, rank, count, tiles):
+    used = -(-count // TILE)
+    start = torch.cumsum(used, 0) - used
+    group = torch.full((tiles,), -1, dtype=torch.int32)
+    for e, n in enumerate(used.tolist()):
+        group[int(start[e]):int(start[e]) + n] = e
+    known = (choice >= 0) & (choice < count.numel())
+    pos = torch.where(known, start[choice.clamp(0, count.numel() - 1).long()].to(torch.int32) * TILE + rank, -1).to(torch.int32)
+    pos[choice >= count.numel()] = -2
+    xg = torch.zeros((tiles * TILE, h.shape[1]), dtype=h.dtype)
+    for k in range(choice.shape[1]):
+        xg[pos[known[:, k], k].long()] = h[known[:, k]]
+    return xg, pos, group
+
+
+def gemm_rows(a, w, tile_group, group_rows, n, swiglu, act):
     out = torch.zeros((a.shape[0], n), dtype=a.dtype)
     for t, e in enumerate(tile_group.tolist()):
         if e < 0:
@@ -74,18 +118,44 @@ def gemm_rows(a, w, tile_group, group_rows, n, swiglu):
         r = a[t * TILE:(t + 1) * TILE].float() @ w[e * group_rows:(e + 1) * group_rows].float().t()
         if swiglu:
             r = torch.nn.functional.silu(r[:, :n]) * r[:, n:]
+        r = finish(r, None, 1.0, act, 0.0)
         out[t * TILE:(t + 1) * TILE] = r.to(a.dtype)
     return out
 
 
-def gemm_heads(a, w, heads, k, n, out, gate):
+def gemm_heads(a, w, heads, k, n, out, gate, a_step, c_step):
     group = w.shape[0] // heads
     for h in range(heads):
-        r = a[:, h * k:(h + 1) * k].float() @ w[h * group:h * group + n, :k].float().t()
+        r = a[:, h * a_step:h * a_step + k].float() @ w[h * group:h * group + n, :k].float().t()
         if gate is not None:
-            r = r * torch.sigmoid(gate[:, h * n:(h + 1) * n].float())
-        out[:, h * n:(h + 1) * n] = r.to(out.dtype)
+            g = gate[:, h:h + 1] if gate.shape[1] == heads else gate[:, h * n:(h + 1) * n]
+            r = r * torch.sigmoid(g.float())
+        out[:, h * c_step:h * c_step + n] = r.to(out.dtype)
     return out
+
+
+def latent_rotate(proj, q_col, q_pitch, kv, kv_col, k_col, wkv, ql, cache, cos_sin, positions, slots, heads, kv_rank, vwidth, rot, eps):
+    c, sn = cos_sin[0, positions.long()], cos_sin[1, positions.long()]
+
+    def turned(t):                                   # (R, ..., rot): pairs (2i, 2i + 1)
+        shape = (-1, *[1] * (t.dim() - 2), rot // 2)
+        u, v, cc, ss = t[..., 0::2].float(), t[..., 1::2].float(), c.view(shape), sn.view(shape)
+        return torch.stack((u * cc - v * ss, v * cc + u * ss), -1).flatten(-2)
+    live, n, width = slots >= 0, 0 if ql is None else ql.shape[0], cache.shape[-1]
+    flat = cache.view(-1, width)
+    if k_col is not None:
+        flat[slots[live], vwidth:] = 0
+        flat[slots[live], vwidth:vwidth + rot] = turned(kv[:, k_col:k_col + rot])[live].to(cache.dtype)
+    if kv_col is not None:
+        t = kv[live, kv_col:kv_col + kv_rank].float()
+        flat[slots[live], kv_rank:vwidth] = 0
+        flat[slots[live], :kv_rank] = (t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * wkv.float()).to(cache.dtype)
+    parts = turned(torch.stack([proj[:, q_col + h * q_pitch:q_col + h * q_pitch + rot] for h in range(heads)], 1)).to(proj.dtype)
+    if n:
+        ql.view(n, heads, width)[..., vwidth:] = 0
+        ql.view(n, heads, width)[..., vwidth:vwidth + rot] = parts[:n]
+    for h in range(heads):
+        proj[n:, q_col + h * q_pitch:q_col + h * q_pitch + rot] = parts[n:, h]
 
 
 def latent_norm_append(proj, wq, wkv, eps, cache, slots, cq):
@@ -98,9 +168,9 @@ def latent_norm_append(proj, wq, wkv, eps, cache, slots, cq):
     return cq
 
 
-def latent_attention(q, cache, row_seq, positions, slots, tables, heads, window, scale):
+def latent_attention(q, cache, row_seq, positions, slots, tables, heads, window, scale, vwidth):
     width, page = cache.shape[-1], cache.shape[1]
-    out = torch.zeros_like(q)
+    out = torch.zeros((q.shape[0], heads * vwidth), dtype=q.dtype)
     flat = cache.view(-1, width)
     for r in range(q.shape[0]):
         if slots[r] < 0:
@@ -110,7 +180,7 @@ def latent_attention(q, cache, row_seq, positions, slots, tables, heads, window,
         line = tables[int(row_seq[r]) if row_seq is not None else r].long()
         c = flat[line[j // page] * page + j % page].float()
         s = torch.einsum("hw,jw->hj", q[r].float().view(heads, width), c) * scale
-        out[r] = torch.einsum("hj,jw->hw", torch.softmax(s, -1), c).reshape(-1).to(q.dtype)
+        out[r] = torch.einsum("hj,jw->hw", torch.softmax(s, -1), c[:, :vwidth]).reshape(-1).to(q.dtype)
     return out
 
 
@@ -180,8 +250,8 @@ def attention_prepare(proj, s, wq, wk, cos_sin, positions, slots, cache, q):
     half = s.rot // 2
 
     def vectors(cols, n, w):
-        t = cols.float().reshape(-1, n, s.dim)
-        t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + s.eps) * w.float()
+        t = cols.float() if s.whole_norm else cols.float().reshape(-1, n, s.dim)
+        t = (t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + s.eps) * w.float()).reshape(-1, n, s.dim)
         if half:
             c, sn = cos_sin[0, positions.long()][:, None], cos_sin[1, positions.long()][:, None]
             u, v = t[..., :half], t[..., half:s.rot]
@@ -207,15 +277,20 @@ def attention_rows(q, s, cache, row_seq, positions, slots, tables, out, gate):
             out[r] = 0
             continue
         p = int(positions[r])
-        j = torch.arange(max(0, p - s.window + 1), p + 1)
+        lo = max(0, p - s.window + 1)
+        j = torch.cat((torch.arange(min(s.keep, lo)), torch.arange(lo, p + 1)))
         line = tables[int(row_seq[r]) if row_seq is not None else r].long()
         c = flat[line[j // page] * page + j % page].float()
         k = c[:, :keys].view(-1, s.kv_heads, s.maps, s.k_pitch)[..., :s.dim].repeat_interleave(rep, 1)
         v = c[:, keys:].view(-1, s.kv_heads, s.v_pitch)[..., :s.vdim].repeat_interleave(rep, 1)
         score = torch.einsum("hmd,jhmd->hmj", q[r].float().view(s.heads, s.maps, s.q_pitch)[..., :s.dim], k) * s.scale
+        if s.softcap:
+            score = s.softcap * torch.tanh(score / s.softcap)
         if s.bias is not None:
             score = score + s.bias[:, (p - j).clamp(max=s.bias.shape[1] - 1)][:, None]
-        o = torch.einsum("hmj,jhe->hme", torch.softmax(score, -1), v)
+        if s.sink is not None:
+            score = torch.cat((score, s.sink.view(-1, 1, 1).expand(-1, s.maps, 1)), -1)
+        o = torch.einsum("hmj,jhe->hme", torch.softmax(score, -1)[..., :len(j)], v)
         if s.maps == 2:
             o = o[:, 0] - s.difference * o[:, 1]
             o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + s.eps) * s.out_scale

@@ -84,6 +84,9 @@ def _declare(lib):
         "b200_gemm_bf16_pair": [P, P, P, P, I, I, I, L, L, L, L, I, I, I, P, P],
         "b200_gemm_bf16_pair_gather": [P, P, P, P, I, I, I, L, L, L, L, I, I, I, P, P, ctypes.c_ulonglong, I, I, P, P,
                                        P, ctypes.c_uint, P, P],
+        "b200_gemm_bf16_finish": [P, P, P, I, I, I, L, L, L, I, P, P, P],
+        "b200_gemm_bf16_pair_finish": [P, P, P, I, I, I, L, L, L, I, P, P, P],
+        "b200_gemm_bf16_splitk_finish": [P, P, P, I, I, I, L, L, L, I, P, P, L, P, I, P, P],
         "b200_gemm_bf16_splitk": [P, P, P, P, I, I, I, L, L, L, L, I, P, L, P, I, P, P],
         "b200_gemm_splitk_plan": [I, I, I, P, P],
         "b200_gemm_splitk_counters": [],
@@ -208,6 +211,11 @@ EPI_PAD_WRITABLE = 0x100
 EPI_B_STABLE = 0x200
 
 
+class GemmFinish(ctypes.Structure):
+    """csrc/gemm_common.cuh: GemmFinish.  act(alpha * (sum + bias)); act 0 none, 1 gelu, 2 cap * tanh(v / cap)."""
+    _fields_ = [("bias", c_void_p), ("alpha", c_float), ("cap", c_float), ("act", c_int)]
+
+
 # Problems at least this large (rows of the output) run on CTA pairs (cta_group::2, 256 x 256 tiles).
 PAIR_MIN_M = int(os.environ.get("B200_GEMM_PAIR_MIN_M", "1024"))
 FUSE_ROPE = os.environ.get("B200_FUSE_ROPE", "1") == "1"                # RoPE in the QKV GEMM epilogue
@@ -268,7 +276,7 @@ def _gemm_pair_tasks(lib, a, b, out, r, m, n, k, lda, ldb, ldc, ldr, a_mn, b_mn,
 
 
 def gemm(a, b, layout: str, out=None, out_dtype=None, residual=None, accumulate=False, bn_hint=0, max_ctas=0,
-         pair=None, gather=None, pad_writable=False, reduce=None, b_stable=False):
+         pair=None, gather=None, pad_writable=False, reduce=None, b_stable=False, finish=None):
     """bf16 tensor-core GEMM (tcgen05).  layout 'nt' | 'nn' | 'tn' as in ``torch_impl.gemm``.
 
     ``pair`` forces (True) or forbids (False) the CTA-pair kernel; by default large problems use it.
@@ -280,8 +288,11 @@ def gemm(a, b, layout: str, out=None, out_dtype=None, residual=None, accumulate=
     launch), so the weights' DRAM latency overlaps the predecessor's tail.
     ``pad_writable``: ``out`` is a column slice of a wider buffer and the columns from N up to the next 16-byte
     boundary (inside the row pitch) may be overwritten with zeros; this lets a row count that is not a multiple of
-    16 bytes (a vocabulary of 50,257) use the TMA-store epilogue."""
+    16 bytes (a vocabulary of 50,257) use the TMA-store epilogue.
+    ``finish``: a ``GemmFinish``, what becomes of the sums before they are stored or added (layout 'nt')."""
     lib = load()
+    if finish is not None:
+        _req(layout == "nt" and residual is None and gather is None and reduce is None, "a finished product is a plain one")
     _req(a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16, "gemm inputs must be bf16")
     _rowmajor(a, "a")
     _rowmajor(b, "b")
@@ -344,6 +355,10 @@ def gemm(a, b, layout: str, out=None, out_dtype=None, residual=None, accumulate=
         if carry_reduce is not None:
             carry_reduce.mark_done()
         return out
+    if pair and finish is not None:
+        _check(lib.b200_gemm_bf16_pair_finish(_ptr(a), _ptr(b), _ptr(out), m, n, k, lda, ldb, out.stride(0), epi & ~EPI_PAD_WRITABLE,
+                                              ctypes.byref(finish), _ptr(status_word(a.device)), _stream()), "b200_gemm_bf16_pair")
+        return out
     if pair:
         rc = lib.b200_gemm_bf16_pair(_ptr(a), _ptr(b), _ptr(out), _ptr(residual), m, n, k, lda, ldb, out.stride(0),
                                      ldr, a_mn, b_mn, epi, _ptr(status_word(a.device)), _stream())
@@ -355,11 +370,20 @@ def gemm(a, b, layout: str, out=None, out_dtype=None, residual=None, accumulate=
         scratch = _splitk_scratch(a.device)
         if scratch is not None:
             ws, counters = scratch
+            if finish is not None:
+                _check(lib.b200_gemm_bf16_splitk_finish(
+                    _ptr(a), _ptr(b), _ptr(out), m, n, k, lda, ldb, out.stride(0), epi, ctypes.byref(finish), _ptr(ws), ws.numel(),
+                    _ptr(counters), counters.numel(), _ptr(status_word(a.device)), _stream()), "b200_gemm_bf16_splitk")
+                return out
             rc = lib.b200_gemm_bf16_splitk(_ptr(a), _ptr(b), _ptr(out), _ptr(residual), m, n, k, lda, ldb, out.stride(0),
                                            ldr, epi, _ptr(ws), ws.numel(), _ptr(counters), counters.numel(),
                                            _ptr(status_word(a.device)), _stream())
             _check(rc, "b200_gemm_bf16_splitk")
             return out
+    if finish is not None:
+        _check(lib.b200_gemm_bf16_finish(_ptr(a), _ptr(b), _ptr(out), m, n, k, lda, ldb, out.stride(0), epi, ctypes.byref(finish),
+                                         _ptr(status_word(a.device)), _stream()), "b200_gemm_bf16")
+        return out
     rc = lib.b200_gemm_bf16(_ptr(a), _ptr(b), _ptr(out), _ptr(residual), m, n, k, lda, ldb, out.stride(0), ldr,
                             a_mn, b_mn, epi, bn_hint, max_ctas, _ptr(status_word(a.device)), _stream())
     _check(rc, "b200_gemm_bf16")

@@ -127,12 +127,13 @@ class LayeredBackend:
 
     def stream(self, batch):
         """The residual stream of a step, not yet written."""
+        batch.gathered.clear()
         return torch.empty((batch.n_rows, self.model.config.width), dtype=torch.float32, device=self.device)
 
-    def head(self, h):
-        """(rows, vocabulary) fp32 of normed rows."""
+    def head(self, h, cap: float | None = None):
+        """(rows, vocabulary) fp32 of normed rows; ``cap``: capped softly."""
         out = torch.empty((h.shape[0], mo.pitch(self.vocab)), dtype=torch.float32, device=self.device)
-        mo.linear(h, self.model.head, out=out[:, :self.vocab])
+        mo.linear(h, self.model.head, out=out[:, :self.vocab], act="cap" if cap else None, cap=cap or 0.0)
         return out
 
 
@@ -209,6 +210,51 @@ class PostNormLayers(LayeredBackend):
         """(rows, vocabulary) fp32."""
         h, _ = mo.residual_norm(x, self.model.final_norm, self.model.config.eps, row_index=rows)
         return self.head(h)
+
+
+class PreNormLayers(LayeredBackend):
+    """Sublayers one after the other, each reading a norm of the residual stream and adding its output times a gain
+    (``models/genedra.py``).  Products add into the stream in their epilogues; the outputs of experts are added by the pass that
+    makes the next sublayer's input."""
+
+    def __init__(self, model):
+        super().__init__(model)
+        self.counters = [layer.mlp.experts for layer in model.layers if layer.routed]
+
+    def forward(self, batch, trace=None):
+        """``trace``: a list that receives the residual stream after every layer run (a copy; for tests)."""
+        m, cfg = self.model, self.model.config
+        x = self.stream(batch)
+        counts = None
+        if self.counters:
+            counts = iter(torch.zeros(sum(self.counters), dtype=torch.int32, device=self.device).split(self.counters))
+        start = dict(tokens=batch.tokens, embed=m.embed, embed_scale=cfg.embed_scale)
+        pending = None
+        for run, layer in enumerate(m.runs):
+            h, _ = mo.residual_norm(x, layer.norm1, cfg.eps, pending=pending, w_offset=1.0, **start)
+            start, pending = {}, None
+            layer.mixer(h, x, batch, self.cache.entries[run])
+            if layer.mlp is not None:
+                h, _ = mo.residual_norm(x, layer.norm2, cfg.eps, w_offset=1.0)
+                if layer.routed:
+                    pending = layer.mlp(h, batch.slots, next(counts))
+                else:
+                    layer.mlp(h, x)
+            if trace is not None:
+                if pending is not None:
+                    mo.residual_norm(x, pending=pending)
+                    pending = None
+                trace.append(x.clone())
+        if start:
+            mo.residual_norm(x, **start)
+        return x, pending
+
+    def logits(self, hidden, rows=None):
+        """(rows, vocabulary) fp32."""
+        x, pending = hidden
+        m = self.model
+        h, _ = mo.residual_norm(x, m.final_norm, m.config.eps, row_index=rows, pending=pending, w_offset=1.0)
+        return self.head(h, m.config.logit_softcap)
 
 
 def wanted_index(rows: np.ndarray, device) -> torch.Tensor:

@@ -25,6 +25,7 @@ class StepBatch:
     portions: list = field(default_factory=list)     # (start position, tokens) of every portion
     splits: int = 0                      # context splits of the decode attention (0 = choose)
     order: list = field(default_factory=list)        # entry index of each sequence, as the caller listed them
+    gathered: dict = field(default_factory=dict)     # packed cache rows of this pass over the layers, for layers that share a cache
     _ranges: dict = field(default_factory=dict)
 
     @property

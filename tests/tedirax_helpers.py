@@ -98,7 +98,8 @@ def feed(engine, seqs, schedule, poison=False):
     if poison:
         # nothing may be read that was not written by its own request (the zero padding of a latent is not data)
         for run, e in zip(engine.backend.model.runs, engine.cache.entries):
-            e[..., :getattr(run.mixer, "kv_rank", e.shape[-1])] = float("nan")
+            pad = hasattr(run.mixer, "kv_rank") and not run.mixer.rot
+            e[..., :run.mixer.kv_rank if pad else e.shape[-1]] = float("nan")
     at, live, got = [0] * len(seqs), {}, [[] for _ in seqs]
     for step in schedule:
         entries = []
