@@ -543,6 +543,7 @@ extern "C" int b200_gemm_bf16_finish(const void* A, const void* B, void* C, int 
                                      long long ldc, int epi, const GemmFinish* finish, uint32_t* status, cudaStream_t stream) {
   const int base = epi & ~EPI_B_STABLE;
   if (base != EPI_BF16 && base != EPI_F32 && base != EPI_F32_ACC) return -11;
+  if (finish != nullptr && finish->act == ACT_GELU && base != EPI_BF16) return -11;
   return gemm_bf16_impl(A, B, C, nullptr, M, N, K, lda, ldb, ldc, 0, 0, 0, epi, 0, 0, 1, nullptr, nullptr, status, stream, finish);
 }
 
@@ -597,6 +598,7 @@ static int splitk_impl(const void* A, const void* B, void* C, const void* R, int
     return -12;
   const int base_epi = epi & ~EPI_B_STABLE;
   if (base_epi != EPI_BF16 && base_epi != EPI_F32 && base_epi != EPI_BF16_RES && base_epi != EPI_F32_ACC) return -11;
+  if (finish != nullptr && finish->act == ACT_GELU && base_epi != EPI_BF16) return -11;
   if (splits <= 1)
     return gemm_bf16_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, 0, 0, epi, 0, 0, 1, nullptr, nullptr, status, stream, finish);
   return gemm_bf16_impl(A, B, C, R, M, N, K, lda, ldb, ldc, ldr, 0, 0, epi, bn, 0, splits, ws, tile_counters, status,
@@ -643,6 +645,7 @@ extern "C" int b200_gemm_bf16_grouped(const void* A, const void* B, void* C, con
   if (!rows && (batch <= 0 || (a_step & 7) || group_rows < (swiglu ? 2 * N : N))) return -12;
   if (swiglu < 0 || swiglu > 2 || (swiglu && (epi != EPI_BF16 || finish != nullptr))) return -12;
   if (finish != nullptr && finish->bias != nullptr && (rows || batch > 1)) return -12;
+  if (finish != nullptr && finish->act == ACT_GELU && epi != EPI_BF16) return -12;
   const int sms = num_sms();
   const long long mt = (M + BM - 1) / BM, problems = rows ? 1 : batch;
   int bn = 64;

@@ -706,6 +706,7 @@ extern "C" int b200_gemm_bf16_pair(const void* A, const void* B, void* C, const 
 extern "C" int b200_gemm_bf16_pair_finish(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
                                           long long ldc, int epi, const GemmFinish* finish, uint32_t* status, cudaStream_t stream) {
   if (epi != EPI_BF16 && epi != EPI_F32 && epi != EPI_F32_ACC) return -11;
+  if (finish != nullptr && finish->act == ACT_GELU && epi != EPI_BF16) return -11;
   return gemm_pair_impl(A, B, C, nullptr, M, N, K, lda, ldb, ldc, 0, 0, 0, epi, nullptr, nullptr, 0, status, stream, nullptr, 0, 0, 0,
                         0, 0, nullptr, 0, nullptr, finish);
 }

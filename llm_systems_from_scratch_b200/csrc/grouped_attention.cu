@@ -257,7 +257,7 @@ static void launch_prep_pieces(const GroupedPrepParams& p, cudaStream_t st) {
 // Norm over the whole projection: the queries of all heads share one root mean square, so do the keys; weights of the projections'
 // sizes.  One block per row, pieces of VEC elements per thread, the first KEEP of them in registers between the passes.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(512) grouped_prep_whole_kernel(const GroupedPrepParams p) {
+__global__ void __launch_bounds__(512, 2) grouped_prep_whole_kernel(const GroupedPrepParams p) {
   pdl_sync();
   __shared__ float red[2][16];
   const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -265,17 +265,21 @@ __global__ void __launch_bounds__(512) grouped_prep_whole_kernel(const GroupedPr
   const int nq = p.heads * p.dim, nk = own ? p.kv_heads * p.dim : 0, nv = own ? p.kv_heads * p.vdim : 0;
   const T* src = reinterpret_cast<const T*>(p.proj) + (long long)row * p.ld;
   const int step = blockDim.x * VEC, total = nq + nk + nv;
-  auto load = [&](int c, float (&f)[VEC]) __attribute__((always_inline)) {
-    if constexpr (VEC == 8) unpack(load_piece(src + c), f);
-    else f[0] = to_f(src[c]);
+  auto load = [&](const T* from, float (&f)[VEC]) __attribute__((always_inline)) {
+    if constexpr (VEC == 8) unpack(load_piece(from), f);
+    else f[0] = to_f(*from);
   };
-  constexpr int KEEP = 3;
+  constexpr int KEEP = 2;
   float keep[KEEP][VEC], sq = 0.f, sk = 0.f;
 #pragma unroll
   for (int j = 0; j < KEEP; ++j) {
     const int c = threadIdx.x * VEC + j * step;
-    if (c < total) load(c, keep[j]);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) keep[j][i] = 0.f;
+    if (c < total) load(src + c, keep[j]);
   }
+  int pos = p.positions[row];
+  const long long slot = p.slots[row];
   auto square = [&](int c, const float (&f)[VEC]) __attribute__((always_inline)) {
     float ss = 0.f;
 #pragma unroll
@@ -284,13 +288,10 @@ __global__ void __launch_bounds__(512) grouped_prep_whole_kernel(const GroupedPr
     else if (c < nq + nk) sk += ss;
   };
 #pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    const int c = threadIdx.x * VEC + j * step;
-    if (c < nq + nk) square(c, keep[j]);
-  }
+  for (int j = 0; j < KEEP; ++j) square(threadIdx.x * VEC + j * step, keep[j]);
   for (int c = threadIdx.x * VEC + KEEP * step; c < nq + nk; c += step) {
     float f[VEC];
-    load(c, f);
+    load(src + c, f);
     square(c, f);
   }
 #pragma unroll
@@ -309,53 +310,64 @@ __global__ void __launch_bounds__(512) grouped_prep_whole_kernel(const GroupedPr
     sk += red[1][w];
   }
   const float rq = rsqrtf(sq / (float)nq + p.eps), rk = own ? rsqrtf(sk / (float)nk + p.eps) : 0.f;
-  int pos = p.positions[row];
   if (p.rot > 0 && (pos < 0 || pos >= p.ctx)) {
     if (threadIdx.x == 0) report_bad_arg(p.status, 23);
     pos = 0;
   }
-  const long long slot = p.slots[row];
   const bool live = slot >= 0 && slot < p.num_slots;             // a padding row of the batch has no slot
   if (own && slot >= p.num_slots && threadIdx.x == 0) report_bad_arg(p.status, 24);
   T* cache = reinterpret_cast<T*>(p.cache) + (live ? slot : 0) * ((long long)p.kv_heads * (p.kp + p.vp));
   T* q = reinterpret_cast<T*>(p.q) + (long long)row * p.heads * p.qp;
   const int half = p.rot / 2;
   auto finish = [&](int c, float (&f)[VEC]) __attribute__((always_inline)) {
-    T* dst;
-    if (c < nq + nk) {
-      const bool query = c < nq;
-      const int at = query ? c : c - nq, v = at / p.dim, e = at - v * p.dim;
-      const T* w = reinterpret_cast<const T*>(query ? p.wq : p.wk) + at;
-      const float r = query ? rq : rk;
+    const bool query = c < nq, vector = c < nq + nk;
+    const int at = query ? c : c - nq, v = vector ? at / p.dim : 0, e = at - v * p.dim;
+    const T* w = reinterpret_cast<const T*>(query ? p.wq : p.wk) + at;
+    const float r = query ? rq : rk;
+    const bool turned = vector && e < p.rot, low = e < half;
+    if (vector) {
       float g[VEC];
-      if constexpr (VEC == 8) unpack(load_piece(w), g);
-      else g[0] = to_f(*w);
+      load(w, g);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) f[i] *= r * g[i];
-      if (e < p.rot) {
-        const bool low = e < half;
-        const int to = low ? half : -half;
-        float o[VEC];
-        load(c + to, o);
-        if constexpr (VEC == 8) unpack(load_piece(w + to), g);
-        else g[0] = to_f(w[to]);
-        const float* cs = p.cos_sin + (long long)pos * half + (low ? e : e - half);
-        const float* sn = cs + (long long)p.ctx * half;
+    }
+    if (p.rot > 0) {
+      const int to = low ? half : -half;
+      float o[VEC];
+      if (turned) {                          // the other half of the pair, normed again
+        float g[VEC];
+        load(src + c + to, o);
+        load(w + to, g);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) {
-          const float other = o[i] * r * g[i];
-          f[i] = low ? f[i] * cs[i] - other * sn[i] : f[i] * cs[i] + other * sn[i];
-        }
+        for (int i = 0; i < VEC; ++i) o[i] *= r * g[i];
       }
-      dst = query ? q + v * p.qp + e : cache + v * p.kp + e;
+      if (turned) {
+        const float* cp = p.cos_sin + (long long)pos * half + (low ? e : e - half);
+        const float* sp = cp + (long long)p.ctx * half;
+        float cs[VEC], sn[VEC];
+        if constexpr (VEC == 8) {
+          unpack(load_piece(cp), cs);
+          unpack(load_piece(sp), sn);
+        } else {
+          cs[0] = *cp;
+          sn[0] = *sp;
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) f[i] = low ? f[i] * cs[i] - o[i] * sn[i] : f[i] * cs[i] + o[i] * sn[i];
+      }
+    }
+    if (!query && !live) return;
+    T* dst;
+    if (query) {
+      dst = q + v * p.qp + e;
+    } else if (vector) {
+      dst = cache + v * p.kp + e;
     } else {
-      const int at = c - nq - nk, v = at / p.vdim;
-      dst = cache + p.kv_heads * p.kp + v * p.vp + (at - v * p.vdim);
+      const int a = c - nq - nk, n = a / p.vdim;
+      dst = cache + p.kv_heads * p.kp + n * p.vp + (a - n * p.vdim);
     }
-    if (c < nq || live) {
-      if constexpr (VEC == 8) store8(dst, f);
-      else from_f(*dst, f[0]);
-    }
+    if constexpr (VEC == 8) store8(dst, f);
+    else from_f(*dst, f[0]);
   };
 #pragma unroll
   for (int j = 0; j < KEEP; ++j) {
@@ -364,7 +376,7 @@ __global__ void __launch_bounds__(512) grouped_prep_whole_kernel(const GroupedPr
   }
   for (int c = threadIdx.x * VEC + KEEP * step; c < total; c += step) {
     float f[VEC];
-    load(c, f);
+    load(src + c, f);
     finish(c, f);
   }
   // the pads behind every vector
@@ -375,6 +387,132 @@ __global__ void __launch_bounds__(512) grouped_prep_whole_kernel(const GroupedPr
   if (p.qp > p.dim) pad(q, p.heads, p.qp, p.dim);
   if (own && live && p.kp > p.dim) pad(cache, p.kv_heads, p.kp, p.dim);
   if (own && live && p.vp > p.vdim) pad(cache + p.kv_heads * p.kp, p.kv_heads, p.vp, p.vdim);
+}
+
+// The same where a thread's pieces of 8 elements have the same place in their vectors (dim a power of two up to 256): weights and angles are
+// requested with the pieces, before the block waits for its sums, the angles once, and the other half of a rotated pair comes
+// from the lane that holds it.
+template <typename T>
+__global__ void __launch_bounds__(512, 2) grouped_prep_whole_pieces_kernel(const GroupedPrepParams p) {
+  pdl_sync();
+  __shared__ float red[2][16];
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool own = p.wk != nullptr;
+  const int nq = p.heads * p.dim, nk = own ? p.kv_heads * p.dim : 0, total = nq + nk + (own ? p.kv_heads * p.vdim : 0);
+  const T* src = reinterpret_cast<const T*>(p.proj) + (long long)row * p.ld;
+  const int step = blockDim.x * 8, c0 = threadIdx.x * 8, e = c0 & (p.dim - 1);      // e: place in the vector
+  const int half = p.rot / 2;
+  const bool turned = e < p.rot, low = e < half;
+  const int from = turned ? lane + (low ? half : -half) / 8 : lane;
+  auto weights = [&](int c) { return c < nq ? reinterpret_cast<const T*>(p.wq) + c : reinterpret_cast<const T*>(p.wk) + (c - nq); };
+  constexpr int KEEP = 2;
+  Piece<T> raw[KEEP], w[KEEP];
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+#pragma unroll
+    for (int i = 0; i < (int)sizeof(T) / 2; ++i) raw[j].v[i] = w[j].v[i] = make_uint4(0, 0, 0, 0);
+    if (c0 + j * step < total) raw[j] = load_piece(src + c0 + j * step);
+  }
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if (c0 + j * step < nq + nk) w[j] = load_piece(weights(c0 + j * step));
+  int pos = p.positions[row];
+  const long long slot = p.slots[row];
+  if (p.rot > 0 && (pos < 0 || pos >= p.ctx)) {
+    if (threadIdx.x == 0) report_bad_arg(p.status, 23);
+    pos = 0;
+  }
+  float cs[8], sn[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) cs[i] = sn[i] = 0.f;
+  if (turned) {
+    const float* cp = p.cos_sin + (long long)pos * half + (low ? e : e - half);
+    unpack(load_piece(cp), cs);
+    unpack(load_piece(cp + (long long)p.ctx * half), sn);
+    if (low) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) sn[i] = -sn[i];
+    }
+  }
+  float sq = 0.f, sk = 0.f;
+  auto square = [&](int c, const Piece<T>& r) __attribute__((always_inline)) {
+    float f[8], ss = 0.f;
+    unpack(r, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss = fmaf(f[i], f[i], ss);
+    if (c < nq) sq += ss;
+    else if (c < nq + nk) sk += ss;
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) square(c0 + j * step, raw[j]);
+  for (int c = c0 + KEEP * step; c < nq + nk; c += step) square(c, load_piece(src + c));
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    sk += __shfl_xor_sync(0xffffffffu, sk, o);
+  }
+  if (lane == 0) {
+    red[0][warp] = sq;
+    red[1][warp] = sk;
+  }
+  __syncthreads();
+  sq = lane < (int)(blockDim.x >> 5) ? red[0][lane & 15] : 0.f;
+  sk = lane < (int)(blockDim.x >> 5) ? red[1][lane & 15] : 0.f;
+#pragma unroll
+  for (int o = 8; o > 0; o >>= 1) {
+    sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    sk += __shfl_xor_sync(0xffffffffu, sk, o);
+  }
+  sq = __shfl_sync(0xffffffffu, sq, 0);
+  sk = __shfl_sync(0xffffffffu, sk, 0);
+  const float rq = rsqrtf(sq / (float)nq + p.eps), rk = own ? rsqrtf(sk / (float)nk + p.eps) : 0.f;
+  const bool live = slot >= 0 && slot < p.num_slots;             // a padding row of the batch has no slot
+  if (own && slot >= p.num_slots && threadIdx.x == 0) report_bad_arg(p.status, 24);
+  T* cache = reinterpret_cast<T*>(p.cache) + (live ? slot : 0) * ((long long)p.kv_heads * (p.kp + p.vp));
+  T* q = reinterpret_cast<T*>(p.q) + (long long)row * p.heads * p.qp;
+  auto finish = [&](int c, const Piece<T>& r, const Piece<T>& wr) __attribute__((always_inline)) {      // all lanes of a warp together
+    const bool query = c < nq, vector = c < nq + nk;
+    const int at = query ? c : c - nq, v = vector ? at / p.dim : 0;
+    float f[8];
+    unpack(r, f);
+    if (vector) {
+      float g[8];
+      unpack(wr, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] *= (query ? rq : rk) * g[i];
+    }
+    if (p.rot > 0) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float o = __shfl_sync(0xffffffffu, f[i], from);
+        if (turned && vector) f[i] = fmaf(f[i], cs[i], o * sn[i]);
+      }
+    }
+    if (c >= total || (!query && !live)) return;
+    if (query) {
+      store8(q + v * p.qp + e, f);
+    } else if (vector) {
+      store8(cache + v * p.kp + e, f);
+    } else {
+      const int a = c - nq - nk, n = a / p.vdim;
+      store8(cache + p.kv_heads * p.kp + n * p.vp + (a - n * p.vdim), f);
+    }
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if (__any_sync(0xffffffffu, c0 + j * step < total)) finish(c0 + j * step, raw[j], w[j]);
+  for (int k = KEEP * step; k < total; k += step) {
+    const int c = c0 + k;
+    Piece<T> r, wr;
+#pragma unroll
+    for (int i = 0; i < (int)sizeof(T) / 2; ++i) r.v[i] = wr.v[i] = make_uint4(0, 0, 0, 0);
+    if (c < total) r = load_piece(src + c);
+    if (c < nq + nk) wr = load_piece(weights(c));
+    finish(c, r, wr);
+  }
+  if (p.qp > p.dim)                          // a query's pitch is 64 at least
+    for (int i = threadIdx.x; i < p.heads * (p.qp - p.dim); i += blockDim.x)
+      from_f(q[(i / (p.qp - p.dim)) * p.qp + p.dim + i % (p.qp - p.dim)], 0.f);
 }
 
 // ------------------------------------------------------------------------------------------------------ general form
@@ -900,15 +1038,20 @@ extern "C" int b200_grouped_prep_whole(const void* proj, long long ld, void* q, 
   const bool vec = s->dim % 8 == 0 && s->vdim % 8 == 0 && (rot / 2) % 8 == 0 && ld % 8 == 0 && (ptrs & 15) == 0;
   const int pieces = (s->heads * s->dim + (wk != nullptr ? s->kv_heads * (s->dim + s->vdim) : 0)) / (vec ? 8 : 1);
   int threads = ((pieces + 1) / 2 + 31) / 32 * 32;
+  if (rows < 148 * 2) threads = (pieces + 31) / 32 * 32;
   if (threads > 512) threads = 512;
-  if (rows < 148 * 2) threads = min(512, (pieces + 31) / 32 * 32);
+  const int lanes = s->dim / 8;
+  const bool same = vec && lanes <= 32 && (lanes & (lanes - 1)) == 0 && (reinterpret_cast<uintptr_t>(cos_sin) & 15) == 0;
+#define PREP_WHOLE(T)                                                                                  \
+  if (same) launch_dep(grouped_prep_whole_pieces_kernel<T>, rows, threads, 0, st, p);                 \
+  else if (vec) launch_dep(grouped_prep_whole_kernel<T, 8>, rows, threads, 0, st, p);                 \
+  else launch_dep(grouped_prep_whole_kernel<T, 1>, rows, threads, 0, st, p)
   if (f32) {
-    if (vec) launch_dep(grouped_prep_whole_kernel<float, 8>, rows, threads, 0, st, p);
-    else launch_dep(grouped_prep_whole_kernel<float, 1>, rows, threads, 0, st, p);
+    PREP_WHOLE(float);
   } else {
-    if (vec) launch_dep(grouped_prep_whole_kernel<__nv_bfloat16, 8>, rows, threads, 0, st, p);
-    else launch_dep(grouped_prep_whole_kernel<__nv_bfloat16, 1>, rows, threads, 0, st, p);
+    PREP_WHOLE(__nv_bfloat16);
   }
+#undef PREP_WHOLE
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 

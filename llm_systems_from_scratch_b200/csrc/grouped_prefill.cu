@@ -9,7 +9,8 @@
 // columns of the next head: the query's pad is zero, and outputs past vdim are not stored).  Value rows past the request's
 // last token are zeroed in shared memory before the product.
 // A CTA walks the tiles of the kept first positions (both query tiles see them), then those of its window.
-//   CAP   scores are capped softly in the second pass (the cap is monotone, so the row maximum is taken of the raw scores)
+//   CAP   scores are capped softly in the second pass (the cap is monotone, so the row maximum is taken of the raw scores); a tile
+//         whose scores stay below the cap evaluates tanh as a polynomial, others take capped_log2
 //   BIAS  a table per head and distance (shared memory) is added to the scaled scores, which go back to tensor memory for the
 //         second pass; distances from the table's last entry on read that entry
 #include "grouped_attention.cuh"
@@ -81,6 +82,25 @@ __device__ __forceinline__ void gp_add2(float& d0, float& d1, float a0, float a1
       "add.rn.f32x2 rd, rd, ra;\n\tmov.b64 {%0, %1}, rd;\n\t}"
       : "+f"(d0), "+f"(d1)
       : "f"(a0), "f"(a1));
+}
+// top tanh(z) - m for z = score * slope / (2 log2 e), |z| <= 1: tanh(z) = z Q(z^2), Q of degree 5 fitted by weighted least squares (error
+// 3e-7).  k = z per score.
+__device__ __forceinline__ void gp_tanh2(float& d0, float& d1, float s0, float s1, float k, float top, float m) {
+  constexpr float c[6] = {0.99999684f, -0.33324003f, 0.13253525f, -0.050972860f, 0.016114177f, -0.0028394643f};
+  const float2 z = __fmul2_rn(make_float2(s0, s1), make_float2(k, k));
+  const float2 t = __fmul2_rn(z, z);
+  float2 q = make_float2(c[5], c[5]);
+#pragma unroll
+  for (int i = 4; i >= 0; --i) q = __ffma2_rn(q, t, make_float2(c[i], c[i]));
+  q = __fmul2_rn(q, z);
+  q = __ffma2_rn(q, make_float2(top, top), make_float2(-m, -m));
+  d0 = q.x;
+  d1 = q.y;
+}
+__device__ __forceinline__ float gp_min3(float a, float b, float c) {
+  float r;
+  asm("min.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c));
+  return r;
 }
 __device__ __forceinline__ void gp_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }   // the softmax threads
 
@@ -332,6 +352,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     const uint32_t tm_o = tmem_base + 256 + x * 128 + lane_addr;
     const float scale2 = BIAS ? 1.f : p.scale_log2;       // of what the second pass finds in tensor memory
     const float slope = CAP ? 2.f * p.scale_log2 / s.softcap : 0.f, top = s.softcap * LOG2E;      // see capped_log2
+    const float part = slope / (2.f * LOG2E);             // a score's part of the cap
     float m_run = -INFINITY, l_run = 0.f;                 // running reference max in scaled log2 units, row sum relative to it
     bool ok = true;
     const __nv_bfloat16* grow = p.gate != nullptr && q_idx < seq_len ? p.gate + (long long)(row_base + q_idx) * p.ld_gate + h * s.vdim : nullptr;
@@ -348,7 +369,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       const int first = q_key - s.window + 1 - k0;
       const uint32_t span = (uint32_t)(s.window - 1);
       auto hidden = [&](int e) { return (uint32_t)(e - first) > span && e >= kept_e; };
-      float mx = -INFINITY;
+      float mx = -INFINITY, mn = INFINITY;
       // pass 1: row maximum (plain: over the raw scores; BIAS: scores in log2 units with the bias, written back)
       const float* bp = nullptr;
       if (BIAS) {
@@ -375,6 +396,13 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
           }
 #pragma unroll
           for (int i = 0; i < 32; i += 2) mx = gp_max3(mx, __uint_as_float(cur[i]), __uint_as_float(cur[i + 1]));
+          if (CAP) {
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) {
+              const bool h0 = masked && hidden(c * 32 + i), h1 = masked && hidden(c * 32 + i + 1);
+              mn = gp_min3(mn, h0 ? INFINITY : __uint_as_float(cur[i]), h1 ? INFINITY : __uint_as_float(cur[i + 1]));
+            }
+          }
           if (c < 3) tmem_ld_wait();
           if (BIAS) tmem_st_32x32(tm_s + c * 32, cur);
         }
@@ -382,6 +410,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       };
       if (edge) row_max(true);
       else row_max(false);
+      const bool low = CAP && !__any_sync(0xffffffffu, fmaxf(mx, -mn) * part > 1.f);      // every score of the tile is below the cap
       if (CAP) mx = capped_log2(mx, slope, top);             // (no key: -cap, below or equal to what any key would give)
       else if (!BIAS) mx *= p.scale_log2;
       // Lazy rescale: keep the old reference max unless it moved by more than 8 (a factor 256).
@@ -417,7 +446,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       // which this thread has already read.  (A row whose window starts in a later tile has seen no key yet.)
       const float m_ref = m_new == -INFINITY ? 0.f : m_new;
       float sum = 0.f, sum1 = 0.f;
-      auto weights = [&](const bool masked) __attribute__((always_inline)) {
+      auto weights = [&](const bool masked, const bool poly) __attribute__((always_inline)) {
         uint32_t sa[32], sb[32];
         tmem_ld_32x32(tm_s, sa);
         tmem_ld_wait();
@@ -430,7 +459,9 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
             float x0, x1;
-            if (CAP) {
+            if (CAP && poly) {
+              gp_tanh2(x0, x1, __uint_as_float(sc[i]), __uint_as_float(sc[i + 1]), part, top, m_ref);
+            } else if (CAP) {
               x0 = gp_exp2(__uint_as_float(sc[i]) * slope);
               x1 = gp_exp2(__uint_as_float(sc[i + 1]) * slope);
               gp_fma2(x0, x1, gp_rcp(1.f + x0), gp_rcp(1.f + x1), -2.f * top, top - m_ref);
@@ -454,8 +485,13 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
           }
         }
       };
-      if (!BIAS && edge) weights(true);
-      else weights(false);
+      if (CAP && low) {
+        if (edge) weights(true, true);
+        else weights(false, true);
+      } else {
+        if (!BIAS && edge) weights(true, false);
+        else weights(false, false);
+      }
       l_run = l_run * (need ? alpha : 1.f) + (sum + sum1);
       m_run = m_new;
     }

@@ -100,6 +100,20 @@ struct LatentRotateParams {
 // VEC elements (whole pairs) of a rotated vector: src -> dst
 template <typename T, int VEC>
 __device__ __forceinline__ void rotate_pairs(const T* src, T* dst, const float* cs, const float* sn) {
+  if constexpr (VEC == 8) {                   // bf16, 16 bytes
+    const uint4 raw = *reinterpret_cast<const uint4*>(src);
+    const float4 c = *reinterpret_cast<const float4*>(cs), s = *reinterpret_cast<const float4*>(sn);
+    const uint32_t in[4] = {raw.x, raw.y, raw.z, raw.w};
+    const float cc[4] = {c.x, c.y, c.z, c.w}, ss[4] = {s.x, s.y, s.z, s.w};
+    uint32_t out[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 v = unpack_bf16x2(in[i]);
+      out[i] = pack_bf16x2(v.x * cc[i] - v.y * ss[i], v.y * cc[i] + v.x * ss[i]);
+    }
+    *reinterpret_cast<uint4*>(dst) = make_uint4(out[0], out[1], out[2], out[3]);
+    return;
+  }
   float f[VEC];
   if constexpr (VEC == 4) {
     load_vec<4>(src, f);
@@ -161,7 +175,7 @@ __global__ void __launch_bounds__(256) latent_rotate_kernel(const LatentRotatePa
     for (int c = p.vwidth + p.rot + lane; c < p.width; c += 32) from_f(dst[c], 0.f);
   }
   if (p.kv_col < 0) return;
-  constexpr int LV = VEC == 4 ? 4 : 1;
+  constexpr int LV = VEC >= 4 ? 4 : 1;
   const T* src = kr + p.kv_col;
   float ss = 0.f;
 #pragma unroll 4
@@ -610,9 +624,13 @@ extern "C" int b200_latent_rotate(void* q, long long ld_q, const void* kv, long 
                    (k_col < 0 || k_col % 4 == 0) && (ld_q | ld_kv) % 4 == 0 &&
                    ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(ql) | reinterpret_cast<uintptr_t>(cache) |
                      reinterpret_cast<uintptr_t>(wkv)) & 15) == 0;
-  int threads = 32 + (heads * (rot / (vec ? 4 : 2)) + 31) / 32 * 32;
+  const bool wide = vec && !f32 && (rot | q_pitch | q_col | vwidth | width) % 8 == 0 && (k_col < 0 || k_col % 8 == 0) && (ld_q | ld_kv) % 8 == 0 &&
+                    (reinterpret_cast<uintptr_t>(cos_sin) & 15) == 0;
+  int threads = 32 + (heads * (rot / (wide ? 8 : (vec ? 4 : 2))) + 31) / 32 * 32;
   if (threads > 256) threads = 256;
-  if (f32) {
+  if (wide) {
+    launch_dep(latent_rotate_kernel<__nv_bfloat16, 8>, rows, threads, 0, st, p);
+  } else if (f32) {
     if (vec) launch_dep(latent_rotate_kernel<float, 4>, rows, threads, 0, st, p);
     else launch_dep(latent_rotate_kernel<float, 2>, rows, threads, 0, st, p);
   } else {

@@ -40,33 +40,10 @@ struct ResidualNormParams {
   uint32_t* status;
 };
 
-// What the experts add to columns c .. c + VEC - 1 of residual row `src`, without yscale.
+// One block per row.  A thread keeps KEEP groups of its columns in registers between the passes, and requests all of them before it
+// works on the first; columns of wider rows are read (and, where experts add to a row that is not stored, added up) again.
 template <typename T, int VEC>
-__device__ __forceinline__ void expert_sum(const ResidualNormParams& p, long long src, int c, float share, float (&s)[VEC]) {
-#pragma unroll
-  for (int i = 0; i < VEC; ++i) s[i] = 0.f;
-  float g[VEC];
-  for (int k = 0; k < p.ytop; ++k) {
-    const int pos = p.ypos[src * p.ytop + k];
-    const T* from;
-    if (pos >= 0 && pos < p.y_rows) from = reinterpret_cast<const T*>(p.y) + (long long)pos * p.ld_y;
-    else if (pos == -2 && p.z != nullptr) from = reinterpret_cast<const T*>(p.z) + src * p.ld_z;
-    else continue;                          // a padding row of the batch
-    const float a = p.yweight != nullptr ? p.yweight[src * p.ytop + k] : 1.f;
-    load_vec<VEC>(from + c, g);
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) s[i] = fmaf(a, g[i], s[i]);
-  }
-  if (p.s != nullptr) {
-    load_vec<VEC>(reinterpret_cast<const T*>(p.s) + src * p.ld_s + c, g);
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) s[i] = fmaf(share, g[i], s[i]);
-  }
-}
-
-// One block per row; every thread keeps to its own columns, so the second pass re-reads what the thread itself wrote.
-template <typename T, int VEC>
-__global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormParams p) {
+__global__ void __launch_bounds__(256, 3) residual_norm_kernel(const ResidualNormParams p) {
   pdl_sync();
   __shared__ float red[32];
   const int row = blockIdx.x;
@@ -90,58 +67,70 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormPa
   }
   const bool changed = (er != nullptr || p.y != nullptr) && p.row_index == nullptr;
   const float share = p.s != nullptr ? (p.sgate != nullptr ? 1.f / (1.f + expf(-p.sgate[src * p.ld_sgate])) : 1.f) : 0.f;
-  constexpr int KEEP = 4;                 // column groups of a thread that stay in registers between the passes
-  float keep[KEEP][VEC];
-  float ss = 0.f;
-  int n = 0;
-  for (int c = threadIdx.x * VEC; c < p.d; c += blockDim.x * VEC, ++n) {
-    float f[VEC];
-    if (er != nullptr) {
-      load_vec<VEC>(er + c, f);
+  constexpr int KEEP = 4;
+  const int step = blockDim.x * VEC, c0 = threadIdx.x * VEC;
+  // columns of the first GROUPS groups, from c on, as the sublayers have left them
+  auto gather = [&](int c, auto& f) __attribute__((always_inline)) {
+    constexpr int GROUPS = sizeof(f) / sizeof(f[0]);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) f[i] *= p.embed_scale;
-    } else {
-      load_vec<VEC>(xr + c, f);
-    }
-    if (p.y != nullptr) {
-      float s[VEC];
-      expert_sum<T, VEC>(p, src, c, share, s);
+    for (int j = 0; j < GROUPS; ++j) {
+      if (c + j * step >= p.d) break;
+      if (er != nullptr) {
+        load_vec<VEC>(er + c + j * step, f[j]);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) f[i] += p.yscale * s[i];
-    }
-    if (changed) store_vec<VEC>(xr + c, f);
-#pragma unroll
-    for (int j = 0; j < KEEP; ++j)
-      if (j == n) {
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) keep[j][i] = f[i];
+        for (int i = 0; i < VEC; ++i) f[j][i] *= p.embed_scale;
+      } else {
+        load_vec<VEC>(xr + c + j * step, f[j]);
       }
+    }
+    if (p.y == nullptr) return;
+    auto add = [&](const T* from, float a) __attribute__((always_inline)) {
+      float g[GROUPS][VEC];
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) ss += f[i] * f[i];
+      for (int j = 0; j < GROUPS; ++j)
+        if (c + j * step < p.d) load_vec<VEC>(from + c + j * step, g[j]);
+#pragma unroll
+      for (int j = 0; j < GROUPS; ++j)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) f[j][i] = fmaf(a, g[j][i], f[j][i]);
+    };
+    if (p.s != nullptr) add(reinterpret_cast<const T*>(p.s) + src * p.ld_s, p.yscale * share);
+#pragma unroll 1
+    for (int k = 0; k < p.ytop; ++k) {
+      const int pos = p.ypos[src * p.ytop + k];
+      const float a = p.yscale * (p.yweight != nullptr ? p.yweight[src * p.ytop + k] : 1.f);
+      if (pos >= 0 && pos < p.y_rows) add(reinterpret_cast<const T*>(p.y) + (long long)pos * p.ld_y, a);
+      else if (pos == -2 && p.z != nullptr) add(reinterpret_cast<const T*>(p.z) + src * p.ld_z, a);
+      // else: a padding row of the batch
+    }
+  };
+  float keep[KEEP][VEC], ss = 0.f;
+  gather(c0, keep);
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    if (c0 + j * step >= p.d) break;
+    if (changed) store_vec<VEC>(xr + c0 + j * step, keep[j]);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(keep[j][i], keep[j][i], ss);
+  }
+  for (int c = c0 + KEEP * step; c < p.d; c += step) {
+    float f[1][VEC];
+    gather(c, f);
+    if (changed) store_vec<VEC>(xr + c, f[0]);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(f[0][i], f[0][i], ss);
   }
   if (p.h == nullptr) return;
+  const T* w = reinterpret_cast<const T*>(p.w);
+  Raw<T, VEC> wk[KEEP];                      // requested before the block waits for its sum
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if (c0 + j * step < p.d) wk[j] = *reinterpret_cast<const Raw<T, VEC>*>(w + c0 + j * step);
   const float r = rsqrtf(block_total(ss, red) / (float)p.d + p.eps);
   T* hr = reinterpret_cast<T*>(p.h) + (long long)row * p.ld_h;
-  n = 0;
-  for (int c = threadIdx.x * VEC; c < p.d; c += blockDim.x * VEC, ++n) {
-    float f[VEC], g[VEC];
-    if (n < KEEP) {
-#pragma unroll
-      for (int j = 0; j < KEEP; ++j)
-        if (j == n) {
-#pragma unroll
-          for (int i = 0; i < VEC; ++i) f[i] = keep[j][i];
-        }
-    } else if (changed || p.y == nullptr) {
-      load_vec<VEC>(xr + c, f);
-    } else {                              // a gathered row with expert outputs: not stored, so added up again
-      load_vec<VEC>(xr + c, f);
-      float s[VEC];
-      expert_sum<T, VEC>(p, src, c, share, s);
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) f[i] += p.yscale * s[i];
-    }
-    load_vec<VEC>(reinterpret_cast<const T*>(p.w) + c, g);
+  auto finish = [&](int c, const Raw<T, VEC>& wr, float (&f)[VEC]) __attribute__((always_inline)) {
+    float g[VEC];
+    load_vec<VEC>(wr.v, g);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) f[i] = f[i] * r * (g[i] + p.w_offset);
     store_vec<VEC>(hr + c, f);
@@ -151,6 +140,15 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const ResidualNormPa
         if (pos >= 0 && pos < p.xg_rows) store_vec<VEC>(reinterpret_cast<T*>(p.xg) + (long long)pos * p.ld_xg + c, f);
       }
     }
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if (c0 + j * step < p.d) finish(c0 + j * step, wk[j], keep[j]);
+  for (int c = c0 + KEEP * step; c < p.d; c += step) {
+    float f[1][VEC];
+    if (changed) load_vec<VEC>(xr + c, f[0]);
+    else gather(c, f);
+    finish(c, *reinterpret_cast<const Raw<T, VEC>*>(w + c), f[0]);
   }
 }
 
@@ -392,7 +390,8 @@ extern "C" int b200_residual_norm(const long long* tokens, const void* embed, in
                          reinterpret_cast<uintptr_t>(p.z) | reinterpret_cast<uintptr_t>(p.s) | reinterpret_cast<uintptr_t>(w) |
                          reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(xg);
   const bool vec = d % 4 == 0 && (p.ld_y | p.ld_z | p.ld_s | ld_h | ld_xg) % 4 == 0 && (ptrs & 15) == 0;
-  const int per = vec ? 4 : 1;
+  const int groups = rows >= 148 * 8 ? 4 : 1;        // of a thread: many rows share an SM, few have all of its threads
+  const int per = (vec ? 4 : 1) * groups;
   int threads = ((d + per - 1) / per + 31) / 32 * 32;
   if (threads > 256) threads = 256;
   if (f32) {

@@ -40,6 +40,11 @@ __device__ __forceinline__ void store_vec(__nv_bfloat16* p, const float (&f)[VEC
   else *p = __float2bfloat16(f[0]);
 }
 
+template <typename T, int VEC>
+struct alignas(sizeof(T) * VEC) Raw {       // VEC elements as they are stored
+  T v[VEC];
+};
+
 // Sum over the block (blockDim.x a multiple of 32, at most 1024); every thread receives it.  `red`: 32 floats.
 __device__ __forceinline__ float block_total(float v, float* red) {
 #pragma unroll

@@ -436,7 +436,10 @@ class RoutedExperts:
     an expert that every token uses, times sigmoid of one number per token (``shared.sg``, a row of the router's product).
 
     A step's rows are sorted by chosen expert into 128-row tiles for the grouped products; what comes out is added up by the next pass
-    over the residual stream (``ops.mixer_ops.ExpertOutputs``)."""
+    over the residual stream (``ops.mixer_ops.ExpertOutputs``).  In steps of few rows the shared expert is part of the grouped
+    products too, if its rows are a multiple of the experts': in pieces of their size, which add up to it."""
+
+    FOLD_ROWS = 256            # the largest step in which the shared expert joins the others
 
     def __init__(self, get, width: int, ff: int, experts: int, top: int, identity: int, shared: int | None, dtype, device,
                  gain: float = 1.0):
@@ -446,21 +449,33 @@ class RoutedExperts:
         w = lambda name, *shape: _expect(name, get(name), *shape)
         pack = lambda *ts: mo.padded_weight(torch.cat(ts), dtype, device)
         self.shared = shared is not None
-        router = [w("router", experts + identity, width)]
+        self.folds = shared // ff if self.shared and shared % ff == 0 else 0          # pieces of the shared expert among the others
+        router, up = [w("router", experts + identity, width)], [w(f"e{e}.up", ff, width) for e in range(experts)]
+        down = [w(f"e{e}.down", width, ff) for e in range(experts)]
         if self.shared:
             router.append(w("shared.sg", 1, width))
-            self.w_shared_up, self.w_shared_down = pack(w("shared.up", shared, width)), pack(w("shared.down", width, shared))
-        self.w_router = pack(*router)
+            s_up, s_down = w("shared.up", shared, width), w("shared.down", width, shared)
+            up += list(s_up.split(ff)) if self.folds else []
+            down += list(s_down.split(ff, 1)) if self.folds else []
+        self.w_router, self.w_up, self.w_down = pack(*router), pack(*up), pack(*down)
+        if self.shared:
+            self.w_shared_up = self.w_up[experts * ff:] if self.folds else pack(s_up)
+            self.w_shared_down = self.w_down[experts * width:] if self.folds == 1 else pack(s_down)
         self.correction = w("correction", experts + identity).to(device=device, dtype=torch.float32).contiguous()
-        self.w_up = pack(*[w(f"e{e}.up", ff, width) for e in range(experts)])
-        self.w_down = pack(*[w(f"e{e}.down", width, ff) for e in range(experts)])
 
     def __call__(self, h, slots, count):
         """``count``: (experts,) int32 of zeros."""
-        outputs = self.experts + self.identity
-        z = mo.linear(h, self.w_router, out_dtype=torch.float32)                   # what is routed by is 32-bit
-        choice, rank, weight = mo.moe_route(z[:, :outputs], self.correction, slots, self.experts, self.top, count)
-        xg, pos, groups = mo.moe_dispatch(h, choice, rank, count)
+        outputs, rows = self.experts + self.identity, h.shape[0]
+        fold = self.folds if rows <= self.FOLD_ROWS else 0
+        cols = outputs + (fold > 0)
+        if mo.routes_rows(rows, self.w_router):
+            z, choice, rank, weight = mo.moe_route_rows(h, self.w_router, self.correction, slots, self.experts, self.top, count, fold)
+        else:
+            z = mo.linear(h, self.w_router, out_dtype=torch.float32)               # what is routed by is 32-bit
+            choice, rank, weight = mo.moe_route(z[:, :cols], self.correction, slots, self.experts, self.top, count, fold)
+        xg, pos, groups = mo.moe_dispatch(h, choice, rank, count, fold)
         y = mo.gemm_rows(mo.gemm_rows(xg, self.w_up, groups, self.ff, False, "gelu"), self.w_down, groups, self.width, False)
-        s = mo.linear(mo.linear(h, self.w_shared_up, act="gelu"), self.w_shared_down) if self.shared else None
-        return mo.ExpertOutputs(y, pos, self.gain, weight, h, s, z[:, outputs] if self.shared else None)
+        if fold or not self.shared:
+            return mo.ExpertOutputs(y, pos, self.gain, weight, h)
+        s = mo.linear(mo.linear(h, self.w_shared_up, act="gelu"), self.w_shared_down)
+        return mo.ExpertOutputs(y, pos, self.gain, weight, h, s, z[:, outputs])

@@ -61,6 +61,9 @@ def build(kind: str, s: dict):
     if kind == "Beledra":
         from .bench_beledra import beledra_config
         return build_model(beledra_config(s))
+    if kind == "Genedra":
+        from .bench_genedra import genedra_config
+        return build_model(genedra_config(s))
     return build_model(dict(vocab_size=s["vocab"], context_length=4096, d_model=s["width"], num_layers=s["runs"],
                             num_heads=s["heads"], d_ff=s["ff"], rope_theta=10000.0))
 
@@ -374,12 +377,16 @@ def _decode_kernels(s, t, b):
 
 
 def run(sizes, steps: int = 10, warmup: int = 3, per_kernel: bool = True, model: str = "Tedirax"):
-    """One record per size: Tedirax beside the TransformerLM, or Beledra beside both."""
+    """One record per size: Tedirax beside the TransformerLM, Beledra beside both, or Genedra beside all three."""
     for size in sizes:
         if model == "Beledra":
             from . import bench_beledra
             rec = models(size, steps, warmup, ("Beledra", "Tedirax", "TransformerLM"))
             more = bench_beledra.kernels
+        elif model == "Genedra":
+            from . import bench_genedra
+            rec = models(size, steps, warmup, ("Genedra", "Tedirax", "Beledra", "TransformerLM"))
+            more = bench_genedra.kernels
         else:
             rec, more = models(size, steps, warmup), kernels
         if per_kernel:

@@ -33,8 +33,9 @@ def _lib():
             "b200_gate_sigmoid": [P, P, L, I, I, L, L, I, P],
             "b200_gemm_f32": [P, P, P, I, I, I, L, L, L, I, P, I, I, I, I, P, P],
             "b200_gemm_bf16_grouped": [P, P, P, P, I, I, I, L, L, L, L, P, I, I, I, I, I, I, I, I, P, P, P],
-            "b200_moe_route": [P, L, P, P, P, P, P, P, I, I, I, I, P],
-            "b200_moe_dispatch": [P, L, P, L, P, P, P, P, P, I, I, I, I, I, I, P],
+            "b200_moe_route": [P, L, P, P, P, P, P, P, I, I, I, I, I, P],
+            "b200_moe_route_rows": [P, L, P, L, I, I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, P],
+            "b200_moe_dispatch": [P, L, P, L, P, P, P, P, P, I, I, I, I, I, I, I, P],
             "b200_latent_norm_append": [P, L, P, P, P, L, P, P, I, I, I, I, L, F, I, P, P],
             "b200_latent_gather": [P, P, P, P, P, I, I, I, I, I, I, P, P],
             "b200_latent_rotate": [P, L, P, L, I, I, I, I, P, P, I, P, P, P, P, I, I, I, I, I, I, I, L, F, I, P, P],
@@ -99,8 +100,8 @@ def _ref(struct):
 
 
 def linear(a, w, out=None, accumulate=False, out_dtype=None, bias=None, alpha: float = 1.0, act: str | None = None, cap: float = 0.0):
-    """act(alpha * (a (R, K) @ w (N, K)^T + bias)), bias fp32.  ``accumulate`` adds to an fp32 ``out``; act: "gelu" (with erf),
-    "cap" (cap * tanh(v / cap)) or nothing."""
+    """act(alpha * (a (R, K) @ w (N, K)^T + bias)), bias fp32.  ``accumulate`` adds to an fp32 ``out``; act: "gelu" (with erf; stored in
+    the activation type), "cap" (cap * tanh(v / cap)) or nothing."""
     if out is None:
         out = rows_buffer(a.shape[0], w.shape[0], out_dtype or a.dtype, a.device)
     if not a.is_cuda:
@@ -298,9 +299,10 @@ def add_normed(x, y=None, w=None, eps: float = 0.0, tokens=None, embed=None):
 
 
 # ------------------------------------------------------------------------------ mixture of experts
-def plan_tiles(rows: int, experts: int, top: int) -> int:
-    """Row tiles that ``rows`` tokens can need at most: every expert in use leaves one tile partly empty."""
-    return min(experts, rows * top) + rows * top // TILE
+def plan_tiles(rows: int, experts: int, top: int, always: int = 0) -> int:
+    """Row tiles that ``rows`` tokens can need at most: every expert in use leaves one tile partly empty, and each of the ``always``
+    experts receives all rows."""
+    return min(experts, rows * top) + rows * top // TILE + always * -(-rows // TILE)
 
 
 def moe_plan(tokens, slots, tables, experts):
@@ -330,37 +332,64 @@ def moe_plan(tokens, slots, tables, experts):
     return ([pos[i, :rows * t.shape[1]].view(rows, t.shape[1]) for i, t in enumerate(tables)], [group[i] for i in range(len(tables))])
 
 
-def moe_route(z, correction, slots, experts: int, top: int, count):
+def moe_route(z, correction, slots, experts: int, top: int, count, always: int = 0):
     """Choose experts by score: z (R, outputs) fp32 logits of the experts and, behind them, of identities; scores are their softmax.  The
     ``top`` outputs with the largest score + correction are chosen and weighted by their share of the chosen scores.  ``count``
-    (experts,) int32, zero on entry, receives the rows per expert.  Returns choice (-1 in padding rows), rank among the expert's
-    rows, weight, each (R, top)."""
-    rows, outputs = z.shape
+    (experts,) int32, zero on entry, receives the rows per expert.  ``always``: that many weights sigmoid(z[:, outputs]) more per row
+    (z has one more column).  Returns choice (-1 in padding rows) and rank among the expert's rows, (R, top), and weight
+    (R, top + always)."""
+    rows, outputs = z.shape[0], correction.numel()
+    _req(z.shape[1] == outputs + (always > 0) and 0 < top <= outputs and experts <= outputs, "bad router sizes")
     if not z.is_cuda:
-        return mixer_torch.moe_route(z, correction, slots, experts, top, count)
-    _req(z.dtype == torch.float32 and z.stride(1) == 1 and correction.dtype == torch.float32 and correction.numel() == outputs
-         and correction.is_contiguous() and count.dtype == torch.int32 and count.is_contiguous() and count.numel() == experts
-         and slots.dtype == torch.int64 and slots.numel() == rows and 0 < top <= outputs and experts <= outputs, "bad router inputs")
-    choice, rank = (torch.empty((rows, top), dtype=torch.int32, device=z.device) for _ in range(2))
-    weight = torch.empty((rows, top), dtype=torch.float32, device=z.device)
+        return mixer_torch.moe_route(z, correction, slots, experts, top, count, always)
+    _req(z.dtype == torch.float32 and z.stride(1) == 1, "bad logits")
+    choice, rank, weight = _route_buffers(rows, top, always, correction, slots, experts, count)
     _check(_lib().b200_moe_route(_ptr(z), z.stride(0), _ptr(correction), _ptr(slots), _ptr(choice), _ptr(rank), _ptr(weight),
-                                 _ptr(count), rows, experts, outputs, top, _stream()), "moe_route")
+                                 _ptr(count), rows, experts, outputs, top, always, _stream()), "moe_route")
     return choice, rank, weight
 
 
-def moe_dispatch(h, choice, rank, count):
-    """Rows of h sorted by chosen expert into 128-row tiles.  Returns them (tiles * 128, d), where each choice went, pos (R, top) int32
-    (-2: an identity, -1: none), and the expert of every tile, tile_group (tiles,) int32."""
+def _route_buffers(rows, top, always, correction, slots, experts, count):
+    _req(correction.dtype == torch.float32 and correction.is_contiguous() and count.dtype == torch.int32 and count.is_contiguous()
+         and count.numel() == experts and slots.dtype == torch.int64 and slots.numel() == rows, "bad router inputs")
+    choice, rank = (torch.empty((rows, top), dtype=torch.int32, device=correction.device) for _ in range(2))
+    return choice, rank, torch.empty((rows, top + always), dtype=torch.float32, device=correction.device)
+
+
+ROUTE_ROWS, ROUTE_BYTES = 256, 32 << 20          # rows, and bytes of the router read once per row, up to which one kernel does it all
+
+
+def routes_rows(rows: int, w) -> bool:
+    """Whether a step of this many rows is routed by ``moe_route_rows``."""
+    return w.is_cuda and rows <= ROUTE_ROWS and rows * w.numel() * w.element_size() <= ROUTE_BYTES and 3 * w.shape[0] + w.shape[1] <= 12000
+
+
+def moe_route_rows(h, w, correction, slots, experts: int, top: int, count, always: int = 0):
+    """``moe_route`` of the few rows of a decode step with the router's product, z = h w^T in fp32.  Returns z too."""
+    (rows, d), columns = h.shape, w.shape[0]
+    _req(h.is_cuda and h.dtype == w.dtype and h.stride(1) == 1 and w.shape[1] == d and columns >= correction.numel() + (always > 0), "bad router")
+    z = torch.empty((rows, columns), dtype=torch.float32, device=h.device)
+    choice, rank, weight = _route_buffers(rows, top, always, correction, slots, experts, count)
+    _check(_lib().b200_moe_route_rows(_ptr(h), h.stride(0), _ptr(w), w.stride(0), d, columns, _ptr(z), columns, _ptr(correction), _ptr(slots),
+                                      _ptr(choice), _ptr(rank), _ptr(weight), _ptr(count), rows, experts, correction.numel(), top, always,
+                                      _f32(h), _stream()), "moe_route_rows")
+    return z, choice, rank, weight
+
+
+def moe_dispatch(h, choice, rank, count, always: int = 0):
+    """Rows of h sorted by chosen expert into 128-row tiles, then all rows for each of the ``always`` further experts.  Returns them
+    (tiles * 128, d), where each choice went, pos (R, top + always) int32 (-2: an identity, -1: none), and the expert of every tile,
+    tile_group (tiles,) int32."""
     (rows, top), experts = choice.shape, count.numel()
-    tiles = plan_tiles(rows, experts, top)
+    tiles = plan_tiles(rows, experts, top, always)
     if not h.is_cuda:
-        return mixer_torch.moe_dispatch(h, choice, rank, count, tiles)
+        return mixer_torch.moe_dispatch(h, choice, rank, count, always, tiles)
     _req(h.stride(1) == 1 and h.shape[0] == rows and choice.dtype == torch.int32 and rank.dtype == torch.int32, "bad expert rows")
     xg = rows_buffer(tiles * TILE, h.shape[1], h.dtype, h.device)
-    pos = torch.empty((rows, top), dtype=torch.int32, device=h.device)
+    pos = torch.empty((rows, top + always), dtype=torch.int32, device=h.device)
     group = torch.empty((tiles,), dtype=torch.int32, device=h.device)
     _check(_lib().b200_moe_dispatch(_ptr(h), h.stride(0), _ptr(xg), xg.stride(0), _ptr(choice), _ptr(rank), _ptr(count), _ptr(pos),
-                                    _ptr(group), rows, experts, top, tiles, h.shape[1], h.element_size(), _stream()), "moe_dispatch")
+                                    _ptr(group), rows, experts, top, always, tiles, h.shape[1], h.element_size(), _stream()), "moe_dispatch")
     return xg, pos, group
 
 

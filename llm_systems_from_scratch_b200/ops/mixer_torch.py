@@ -80,11 +80,14 @@ def moe_plan(tokens, slots, tables, experts, tiles):
     return pos, groups
 
 
-def moe_route(z, correction, slots, experts, top, count):
-    s = torch.softmax(z, -1)
+def moe_route(z, correction, slots, experts, top, count, always):
+    outputs = correction.numel()
+    s = torch.softmax(z[:, :outputs], -1)
     choice = torch.topk(s + correction, top, dim=-1).indices
     weight = s.gather(1, choice)
     weight = weight / (weight.sum(-1, keepdim=True) + 1e-20)
+    if always:
+        weight = torch.cat((weight, torch.sigmoid(z[:, outputs:]).expand(-1, always)), 1)
     choice, rank = choice.to(torch.int32), torch.full(choice.shape, -1, dtype=torch.int32)
     choice[slots < 0], weight[slots < 0] = -1, 0.0
     for r in range(z.shape[0]):
@@ -95,18 +98,22 @@ def moe_route(z, correction, slots, experts, top, count):
     return choice, rank, weight
 
 
-def moe_dispatch(h, choice, rank, count, tiles):
-    used = -(-count // TILE)
+def moe_dispatch(h, choice, rank, count, always, tiles):
+    rows, experts = len(h), count.numel()
+    used = -(-torch.cat((count, torch.full((always,), rows, dtype=count.dtype))) // TILE)
     start = torch.cumsum(used, 0) - used
     group = torch.full((tiles,), -1, dtype=torch.int32)
     for e, n in enumerate(used.tolist()):
         group[int(start[e]):int(start[e]) + n] = e
-    known = (choice >= 0) & (choice < count.numel())
-    pos = torch.where(known, start[choice.clamp(0, count.numel() - 1).long()].to(torch.int32) * TILE + rank, -1).to(torch.int32)
-    pos[choice >= count.numel()] = -2
+    known = (choice >= 0) & (choice < experts)
+    pos = torch.where(known, start[choice.clamp(0, experts - 1).long()].to(torch.int32) * TILE + rank, -1).to(torch.int32)
+    pos[choice >= experts] = -2
+    more = torch.arange(rows)[:, None] + start[None, experts:] * TILE
+    pos = torch.cat((pos, torch.where(choice[:, :1] >= 0, more, -1).to(torch.int32)), 1)
     xg = torch.zeros((tiles * TILE, h.shape[1]), dtype=h.dtype)
-    for k in range(choice.shape[1]):
-        xg[pos[known[:, k], k].long()] = h[known[:, k]]
+    for k in range(pos.shape[1]):
+        live = pos[:, k] >= 0
+        xg[pos[live, k].long()] = h[live]
     return xg, pos, group
 
 

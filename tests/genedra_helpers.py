@@ -44,7 +44,7 @@ CONFIGS = {
                   eps=1e-4, embed=1.0, mult=1.0, cap=7.0),
     # sizes the tensor-core kernels take
     "tiles": config(203, 96, [latent(6, 40, 56, 72, 24, mlp=moe(40, 6, 2, 1, 24)), attention(6, 2, 48, 24, 33, 5, 8.0, 16, mlp=dense(72)),
-                              latent(3, 72, 40, 72, 24, kv_from=0, mlp=moe(24, 3, 4, 2, 56)), attention(4, 1, 24, 72, 70, 1, 50.0, 8)]),
+                              latent(3, 72, 40, 72, 24, kv_from=0, mlp=moe(24, 3, 4, 2, 24)), attention(4, 1, 24, 72, 70, 1, 50.0, 8)]),
     # heads of 128 with 64 rotated dimensions more, more heads than one group of the decode kernels, windows and kept tokens of
     # several key tiles
     "wide": config(160, 128, [latent(20, 128, 128, 128, 64, mlp=moe(64, 8, 3, 2, 40)),

@@ -163,6 +163,14 @@ def test_routing_and_dispatch():
     assert (pos[choice >= experts] == -2).all() and (pos[~live] == -1).all()
     r, k = ((choice >= 0) & (choice < experts)).nonzero(as_tuple=True)
     assert torch.equal(xg[pos[r, k].long()], h[r])
+    # two more experts that every row uses, weighted by one more logit
+    z2 = torch.cat((z, randn(rows, 1, seed=4)), 1)
+    choice, rank, weight = mo.moe_route(z2, corr, slots, experts, top, count.zero_(), 2)
+    assert torch.allclose(weight[live, top:], torch.sigmoid(z2[live, -1:]).expand(-1, 2)) and float(weight[~live].abs().sum()) == 0.0
+    xg, more, group = mo.moe_dispatch(h, choice, rank, count, 2)
+    assert torch.equal(more[:, :top], pos) and (more[~live] == -1).all()
+    for a in range(2):
+        assert (group[(more[live, top + a] // mo.TILE).long()] == experts + a).all() and torch.equal(xg[more[live, top + a].long()], h[live])
 
 
 def test_expert_outputs_join_the_residual_stream():

@@ -162,21 +162,49 @@ def test_routing_and_dispatch(dtype, rows, experts, identity, top, d):
     slots = torch.zeros(rows, dtype=torch.int64, device="cuda")
     slots[3::11] = -1
     live = (slots >= 0).cpu()
-    count = torch.zeros(experts, dtype=torch.int32, device="cuda")
-    choice, rank, weight = mo.moe_route(wide, corr.cuda(), slots, experts, top, count)
     want, wweight = O.route(z.double(), torch.eye(n, dtype=torch.float64), corr.double(), top)
-    assert torch.equal(choice.cpu()[live], want.int()[live]) and (choice.cpu()[~live] == -1).all()
-    close(weight[live.cuda()], wweight[live], 1e-6)
     h = padded(randn(rows, d, seed=3, dtype=dtype))
-    xg, pos, group = mo.moe_dispatch(h, choice, rank, count)
+    for always in (0, 2):                                  # experts that every row uses
+        count = torch.zeros(experts, dtype=torch.int32, device="cuda")
+        logits = wide if not always else torch.cat((wide, randn(rows, 1, seed=4)), 1)
+        choice, rank, weight = mo.moe_route(logits, corr.cuda(), slots, experts, top, count, always)
+        assert torch.equal(choice.cpu()[live], want.int()[live]) and (choice.cpu()[~live] == -1).all()
+        share = torch.sigmoid(logits[:, n:].double().cpu()).expand(-1, always) if always else torch.zeros(rows, 0, dtype=torch.float64)
+        close(weight[live.cuda()], torch.cat((wweight, share), 1)[live], 1e-6)
+        dispatched(mo, h, choice, rank, count, live, experts, top, always)
+
+
+def dispatched(mo, h, choice, rank, count, live, experts, top, always):
+    xg, pos, group = mo.moe_dispatch(h, choice, rank, count, always)
     choice, pos, group, count, xg, h = (t.cpu() for t in (choice, pos, group, count, xg, h))
-    assert (pos[choice >= experts] == -2).all() and (pos[~live] == -1).all()
+    for a in range(always):
+        mine = pos[live, top + a]
+        assert (group[(mine // mo.TILE).long()] == experts + a).all() and torch.equal(xg[mine.long()], h[live])
+    assert (pos[:, :top][choice >= experts] == -2).all() and (pos[~live] == -1).all()
+    pos = pos[:, :top]
     for e in range(experts):
         used = pos[choice == e]
         assert used.unique().numel() == used.numel() == int(count[e]) and (group[(used // mo.TILE).long()] == e).all()
-    assert int((group >= 0).sum()) == sum(-(-int(c) // mo.TILE) for c in count)
+    assert int((group >= 0).sum()) == sum(-(-int(c) // mo.TILE) for c in count) + always * -(-len(h) // mo.TILE)
     r, k = ((choice >= 0) & (choice < experts)).nonzero(as_tuple=True)
     assert torch.equal(xg[pos[r, k].long()], h[r])
+
+
+@pytest.mark.parametrize("dtype", [BF, F32])
+@pytest.mark.parametrize("rows,experts,identity,top,d,always", [(1, 3, 1, 1, 5, 0), (33, 12, 3, 4, 44, 1), (128, 64, 8, 6, 320, 2), (70, 300, 0, 9, 2048, 0)])
+def test_few_rows_are_routed_with_the_product(dtype, rows, experts, identity, top, d, always):
+    mo = mops()
+    n = experts + identity
+    h, w = padded(randn(rows, d, seed=1, dtype=dtype)), mo.padded_weight(randn(n + 1, d, seed=2, dtype=dtype, scale=2 * d ** -0.5), dtype, "cuda")
+    corr, slots = 0.02 * randn(n, seed=3), torch.zeros(rows, dtype=torch.int64, device="cuda")
+    slots[5::7] = -1
+    live = (slots >= 0).cpu()
+    count, again = torch.zeros(experts, dtype=torch.int32, device="cuda"), torch.zeros(experts, dtype=torch.int32, device="cuda")
+    z, choice, rank, weight = mo.moe_route_rows(h, w, corr, slots, experts, top, count, always)
+    close(z, h.double() @ w.double().t(), 1e-5)
+    c2, _, w2 = mo.moe_route(z[:, :n + (always > 0)], corr, slots, experts, top, again, always)
+    assert torch.equal(choice, c2) and torch.equal(count, again) and torch.equal(weight[live.cuda()], w2[live.cuda()])
+    dispatched(mo, h, choice, rank, count, live, experts, top, always)
 
 
 def test_correction_changes_the_choice_but_not_the_weights():
