@@ -1,9 +1,9 @@
 // Softmax attention of grouped heads over a paged cache: query head h reads key/value head h / (heads / kv_heads), under a
-// sliding window (position i sees the `window` positions up to and including i, and the first `keep` positions of the sequence), with
-// optional parts: scores capped softly (cap tanh(score / cap)), a bias per distance, a sink per head (exp(sink) joins the softmax's
-// denominator) and, for differential attention, two maps per head over the same values:
+// sliding window (position i sees the `window` positions up to and including i, and the first `keep` positions of the sequence) or inside
+// chunks of `window` positions counted from the sequence's first, with optional parts: scores capped softly (cap tanh(score / cap)), a bias
+// per distance from a table or linear in it, a sink per head (exp(sink) joins the softmax's denominator) and, for differential attention, two maps per head over the same values:
 //     o = a_1 - difference * a_2,   o <- o / rms(o) * out_scale
-// and an optional gate, o * sigmoid(g).  This file: norm, rotation and append; the general kernel (any size, bf16 or fp32);
+// and an optional gate, o * sigmoid(g), per element or per head.  This file: norm, rotation and append; the general kernel (any size, bf16 or fp32);
 // decode on mma.sync.  Portions of prompts: grouped_prefill.cu.
 //
 // Cache row of a token: kv_heads x maps keys of kp elements, then kv_heads values of vp elements (kp, vp: dim, vdim rounded
@@ -122,33 +122,6 @@ __global__ void __launch_bounds__(256) grouped_prep_kernel(const GroupedPrepPara
 
 // The same for sizes in whole pieces of 8 elements: LPV lanes own a vector, one piece each; a thread owns the same columns of UNITS
 // vectors of one row, so it loads the angles once.
-template <typename T>
-struct Piece {                    // 8 elements as they are stored
-  uint4 v[sizeof(T) / 2];
-};
-__device__ __forceinline__ void unpack(const Piece<__nv_bfloat16>& r, float (&f)[8]) {
-  const float2 a = unpack_bf16x2(r.v[0].x), b = unpack_bf16x2(r.v[0].y), c = unpack_bf16x2(r.v[0].z), d = unpack_bf16x2(r.v[0].w);
-  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
-}
-__device__ __forceinline__ void unpack(const Piece<float>& r, float (&f)[8]) {
-  f[0] = __uint_as_float(r.v[0].x); f[1] = __uint_as_float(r.v[0].y); f[2] = __uint_as_float(r.v[0].z); f[3] = __uint_as_float(r.v[0].w);
-  f[4] = __uint_as_float(r.v[1].x); f[5] = __uint_as_float(r.v[1].y); f[6] = __uint_as_float(r.v[1].z); f[7] = __uint_as_float(r.v[1].w);
-}
-template <typename T>
-__device__ __forceinline__ Piece<T> load_piece(const T* p) {
-  Piece<T> r;
-#pragma unroll
-  for (int j = 0; j < (int)sizeof(T) / 2; ++j) r.v[j] = reinterpret_cast<const uint4*>(p)[j];
-  return r;
-}
-__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
-  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
-}
-__device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
-  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
-}
-
 template <typename T, int LPV, int UNITS>
 __global__ void __launch_bounds__(512, 2) grouped_prep_pieces_kernel(const GroupedPrepParams p) {
   pdl_sync();
@@ -554,7 +527,8 @@ __global__ void __launch_bounds__(128) grouped_rows_kernel(const GroupedRowsPara
   const int width = s.kv_heads * (s.maps * s.kp + s.vp);
   if (live) {
     const int* table = p.tables + (long long)seq * p.max_pages;
-    const int lo = max(0, pos - s.window + 1), kept = min(s.keep, lo);
+    const int lo = max(0, first_seen(s, pos)), kept = min(s.keep, lo);
+    const float slope = s.slopes != nullptr ? s.slopes[h] : 0.f;
     for (int n = lo - kept; n <= pos; ++n) {
       const int j = n < lo ? n - (lo - kept) : n;                 // the kept positions, then the window
       const int pg = j / p.page_size;
@@ -565,7 +539,7 @@ __global__ void __launch_bounds__(128) grouped_rows_kernel(const GroupedRowsPara
       }
       const T* c = reinterpret_cast<const T*>(p.cache) + ((long long)page * p.page_size + j % p.page_size) * width;
       const T* v = c + s.kv_heads * s.maps * s.kp + g * s.vp;
-      const float b = p.bias != nullptr ? p.bias[h * p.bias_len + min(pos - j, p.bias_len - 1)] : 0.f;
+      const float b = (p.bias != nullptr ? p.bias[h * p.bias_len + min(pos - j, p.bias_len - 1)] : 0.f) - slope * (float)(pos - j);
       for (int m = 0; m < s.maps; ++m) {
         const T* k = c + (g * s.maps + m) * s.kp;
         float sc = 0.f;
@@ -604,10 +578,10 @@ __global__ void __launch_bounds__(128) grouped_rows_kernel(const GroupedRowsPara
     f = rsqrtf(ss / (float)s.vdim + s.eps) * s.out_scale;
   }
   T* orow = reinterpret_cast<T*>(p.o) + (long long)row * p.ld_o + h * s.vdim;
-  const T* grow = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + (long long)row * p.ld_gate + h * s.vdim : nullptr;
+  const T* grow = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + (long long)row * p.ld_gate + gate_column(s, h) : nullptr;
   for (int c = lane; c < s.vdim; c += 32) {
     float o = acc[c] * f;
-    if (grow != nullptr) o /= 1.f + expf(-to_f(grow[c]));
+    if (grow != nullptr) o /= 1.f + expf(-to_f(grow[s.head_gate ? 0 : c]));
     from_f(orow[c], live ? o : 0.f);
   }
 }
@@ -689,7 +663,7 @@ __device__ __forceinline__ void grouped_finish(const GroupedShape& s, int lane, 
     const int c = lane + i * 32;
     if (c >= s.vdim) break;
     float x = o[i] * f;
-    if (grow != nullptr) x *= sigmoid_f(__bfloat162float(grow[c]));
+    if (grow != nullptr) x *= sigmoid_f(__bfloat162float(grow[s.head_gate ? 0 : c]));
     orow[c] = __float2bfloat16(x);
   }
 }
@@ -726,7 +700,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
   pdl_sync();
   const int pos = p.positions[row];
   const bool live = p.slots[row] >= 0 && pos >= 0;
-  const int lo = live ? max(0, pos - s.window + 1) : 0;
+  const int lo = live ? max(0, first_seen(s, pos)) : 0;
   // tiles of 16 tokens, starting at multiples of 16: those of the kept tokens in front of the window's first tile, then the window's
   const int first = lo / GD_TOK, kept = min((s.keep + GD_TOK - 1) / GD_TOK, first);
   const int total = live ? kept + pos / GD_TOK + 1 - first : 0;
@@ -785,6 +759,11 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
     for (int i = 0; i < 2; ++i) bias[i] = p.bias + (long long)(h0 + min(((lane >> 2) + i * 8) / s.maps, nh - 1)) * p.bias_len;
   }
 
+  float slope2[2] = {0.f, 0.f};                        // log2 units per token, of this lane's two query vectors
+  if (s.slopes != nullptr) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) slope2[i] = LOG2E * s.slopes[h0 + min((lane >> 2) + i * 8, nh - 1)];
+  }
   float bn[2][4];                                      // bias of the tile after the one at work
   auto load_bias = [&](int i) {
     const int t = token(i0 + i) + (lane & 3) * 2;
@@ -823,6 +802,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
         float x = s.softcap > 0.f ? capped_log2(sc[n][e], slope, s.softcap * LOG2E) : sc[n][e] * scale_log2;
         const bool seen = (t >= lo || t < s.keep) && t <= pos;
         if (p.bias != nullptr) x = fmaf(bn[n][e], LOG2E, x);
+        else x = fmaf(slope2[e >> 1], (float)(t - pos), x);
         x = seen ? x : -INFINITY;
         sc[n][e] = x;
         mx[e >> 1] = fmaxf(mx[e >> 1], x);
@@ -929,7 +909,7 @@ __global__ void __launch_bounds__(GD_WARPS * 32) grouped_decode_kernel(const Gro
       if (s.sink != nullptr) add_sink(s.sink[h], m[0], l[0]);
       const float inv[2] = {l[0] > 0.f ? 1.f / l[0] : 0.f, l[1] > 0.f ? 1.f / l[1] : 0.f};
       grouped_finish(s, lane, p.o + (long long)row * p.ld_o + h * s.vdim,
-                     p.gate != nullptr ? p.gate + (long long)row * p.ld_gate + h * s.vdim : nullptr, [&](int mp, int c) {
+                     p.gate != nullptr ? p.gate + (long long)row * p.ld_gate + gate_column(s, h) : nullptr, [&](int mp, int c) {
                        float v = 0.f;                  // constant map index: the factors stay in registers
 #pragma unroll
                        for (int w = 0; w < GD_WARPS; ++w)
@@ -961,7 +941,7 @@ __global__ void __launch_bounds__(128) grouped_merge_kernel(const GroupedDecodeP
     inv[mp] = l > 0.f ? 1.f / l : 0.f;
   }
   grouped_finish(s, lane, p.o + (long long)row * p.ld_o + h * s.vdim,
-                 p.gate != nullptr ? p.gate + (long long)row * p.ld_gate + h * s.vdim : nullptr, [&](int mp, int c) {
+                 p.gate != nullptr ? p.gate + (long long)row * p.ld_gate + gate_column(s, h) : nullptr, [&](int mp, int c) {
                    const float* ml = p.part_ml + (base + mp * p.splits) * 2;
                    const float* po = p.part_o + (base + mp * p.splits) * s.vdim + c;
                    const float m = mp ? gm[1] : gm[0];

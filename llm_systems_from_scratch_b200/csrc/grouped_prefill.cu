@@ -11,6 +11,7 @@
 // A CTA walks the tiles of the kept first positions (both query tiles see them), then those of its window.
 //   CAP   scores are capped softly in the second pass (the cap is monotone, so the row maximum is taken of the raw scores); a tile
 //         whose scores stay below the cap evaluates tanh as a polynomial, others take capped_log2
+//   SLOPE slope * distance comes off the scaled score in both passes (two fused multiply-adds per score, nothing is written back)
 //   BIAS  a table per head and distance (shared memory) is added to the scaled scores, which go back to tensor memory for the
 //         second pass; distances from the table's last entry on read that entry
 #include "grouped_attention.cuh"
@@ -36,7 +37,7 @@ struct GroupedPrefillParams {
 constexpr int GP_THREADS = 64 + 256;      // TMA warp, MMA warp, 4 + 4 softmax warps
 constexpr int GP_LUT_PAD = 254;           // table entries in front of distance 0 (keys of a tile that lie behind a query)
 
-enum GroupedScores : int { SCORES_PLAIN = 0, SCORES_BIAS = 1, SCORES_CAP = 2 };
+enum GroupedScores : int { SCORES_PLAIN = 0, SCORES_BIAS = 1, SCORES_CAP = 2, SCORES_SLOPE = 3 };
 
 template <int P, bool BIAS>
 struct GroupedPrefillSmem {
@@ -110,7 +111,11 @@ __device__ __forceinline__ void gp_store(const GroupedPrefillParams& p, __nv_bfl
 #pragma unroll
   for (int q = 0; q < 4; ++q) {
     if (q * 8 >= n) break;
-    if (grow != nullptr && p.gate_vec && q * 8 + 8 <= n) {
+    if (grow != nullptr && p.s.head_gate) {
+      const float a = gp_sigmoid(__bfloat162float(*grow));
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[q * 8 + i] *= a;
+    } else if (grow != nullptr && p.gate_vec && q * 8 + 8 <= n) {
       const uint4 gv = *reinterpret_cast<const uint4*>(grow + col + q * 8);
       const uint32_t gg[4] = {gv.x, gv.y, gv.z, gv.w};
 #pragma unroll
@@ -139,7 +144,7 @@ __device__ __forceinline__ void gp_store(const GroupedPrefillParams& p, __nv_bfl
 template <int P, int MAPS, int SCORES>
 __global__ void __launch_bounds__(GP_THREADS, 1)
 grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv, const GroupedPrefillParams p) {
-  constexpr bool BIAS = SCORES == SCORES_BIAS, CAP = SCORES == SCORES_CAP;
+  constexpr bool BIAS = SCORES == SCORES_BIAS, CAP = SCORES == SCORES_CAP, SLOPE = SCORES == SCORES_SLOPE;
   using L = GroupedPrefillSmem<P, BIAS>;
   extern __shared__ uint8_t gp_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(gp_raw) + 1023) & ~uintptr_t(1023));
@@ -193,7 +198,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     n_kv_t[x] = q0_t[x] < seq_len ? (min(q0_t[x] + 128, seq_len) + shift + 127) / 128 : 0;
-    lo_t[x] = n_kv_t[x] > 0 ? max(0, q0_t[x] + shift - s.window + 1) / 128 : 0;
+    lo_t[x] = n_kv_t[x] > 0 ? max(0, first_seen(s, q0_t[x] + shift)) / 128 : 0;
   }
   const int kept = min((s.keep + 127) / 128, lo_t[0]), skip = kept > 0 ? lo_t[0] - kept : 0;
   if (s.keep > 0) {
@@ -355,19 +360,22 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     const float part = slope / (2.f * LOG2E);             // a score's part of the cap
     float m_run = -INFINITY, l_run = 0.f;                 // running reference max in scaled log2 units, row sum relative to it
     bool ok = true;
-    const __nv_bfloat16* grow = p.gate != nullptr && q_idx < seq_len ? p.gate + (long long)(row_base + q_idx) * p.ld_gate + h * s.vdim : nullptr;
-    if (grow != nullptr)                                  // the epilogue's gate row into L2
+    const __nv_bfloat16* grow = p.gate != nullptr && q_idx < seq_len ? p.gate + (long long)(row_base + q_idx) * p.ld_gate + gate_column(s, h) : nullptr;
+    const int from = first_seen(s, q_key), from_last = first_seen(s, q0 + 127 + shift);     // of this row, of the tile's last one
+    const float slope2 = SLOPE ? s.slopes[h] * LOG2E : 0.f;                                 // log2 units per token
+    if (grow != nullptr && !s.head_gate)                                  // the epilogue's gate row into L2
       for (int i = 0; i < s.vdim; i += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(grow + i));
     for (int j = lo_x; j < n_kv_x; ++j) {
       if (!mbar_wait(&s_full[x], (j - lo_x) & 1, abort_word)) { ok = false; break; }
       tc_fence_after();
       const int k0 = key_tile(j) * 128;
       // tile touches the diagonal or the lower edge of the window (warp-uniform)
-      const bool edge = (k0 + 127 > q0 + shift) || (k0 <= q0 + 127 + shift - s.window);
+      const bool edge = (k0 + 127 > q0 + shift) || (k0 < from_last);
       const int kept_e = min(s.keep - k0, q_key - k0 + 1);      // keys k0 + e with e below are visible wherever the window is
       // Key k0 + e is visible iff e - first <= span as unsigned numbers (one comparison for both edges of the window).
-      const int first = q_key - s.window + 1 - k0;
-      const uint32_t span = (uint32_t)(s.window - 1);
+      const int first = from - k0;
+      const uint32_t span = (uint32_t)(q_key - from);
+      const float base = SLOPE ? slope2 * (float)(k0 - q_key) : 0.f;      // of the tile's first key
       auto hidden = [&](int e) { return (uint32_t)(e - first) > span && e >= kept_e; };
       float mx = -INFINITY, mn = INFINITY;
       // pass 1: row maximum (plain: over the raw scores; BIAS: scores in log2 units with the bias, written back)
@@ -388,6 +396,11 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
           if (BIAS) {
 #pragma unroll
             for (int i = 0; i < 32; ++i) cur[i] = __float_as_uint(fmaf(__uint_as_float(cur[i]), p.scale_log2, bp[-(c * 32 + i)]));
+          }
+          if (SLOPE) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              cur[i] = __float_as_uint(fmaf(__uint_as_float(cur[i]), p.scale_log2, fmaf(slope2, (float)(c * 32 + i), base)));
           }
           if (masked) {
 #pragma unroll
@@ -412,7 +425,7 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       else row_max(false);
       const bool low = CAP && !__any_sync(0xffffffffu, fmaxf(mx, -mn) * part > 1.f);      // every score of the tile is below the cap
       if (CAP) mx = capped_log2(mx, slope, top);             // (no key: -cap, below or equal to what any key would give)
-      else if (!BIAS) mx *= p.scale_log2;
+      else if (!BIAS && !SLOPE) mx *= p.scale_log2;
       // Lazy rescale: keep the old reference max unless it moved by more than 8 (a factor 256).
       float m_new = m_run;
       if (mx > m_run + 8.f) m_new = mx;
@@ -465,6 +478,12 @@ grouped_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
               x0 = gp_exp2(__uint_as_float(sc[i]) * slope);
               x1 = gp_exp2(__uint_as_float(sc[i + 1]) * slope);
               gp_fma2(x0, x1, gp_rcp(1.f + x0), gp_rcp(1.f + x1), -2.f * top, top - m_ref);
+            } else if (SLOPE) {
+              const float2 d = __ffma2_rn(make_float2(slope2, slope2), make_float2((float)(c * 32 + i), (float)(c * 32 + i + 1)),
+                                          make_float2(base - m_ref, base - m_ref));
+              const float2 y = __ffma2_rn(make_float2(__uint_as_float(sc[i]), __uint_as_float(sc[i + 1])), make_float2(scale2, scale2), d);
+              x0 = y.x;
+              x1 = y.y;
             } else {
               gp_fma2(x0, x1, __uint_as_float(sc[i]), __uint_as_float(sc[i + 1]), scale2, -m_ref);
             }
@@ -602,6 +621,7 @@ extern "C" int b200_grouped_prefill(const void* q, const void* cache, void* o, l
   if (!shape_ok(*s) || s->dim > 128 || s->vdim > 128 || s->qp % 64 || page_size < 8 || 128 % page_size || max_q <= 0) return -10;
   if (bias != nullptr ? (bias_len <= 0 || bias_len > B200_GROUPED_BIAS_MAX) : !(s->scale > 0.f)) return -11;
   if (s->softcap > 0.f && (bias != nullptr || s->maps != 1)) return -12;
+  if (s->slopes != nullptr && bias != nullptr) return -12;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15) return -10;
   const uint64_t qw = (uint64_t)s->heads * s->maps * s->qp, width = (uint64_t)s->kv_heads * (s->maps * s->kp + s->vp);
   CUtensorMap tm_q, tm_kv;
@@ -620,6 +640,7 @@ extern "C" int b200_grouped_prefill(const void* q, const void* cache, void* o, l
               : launch_grouped_prefill<1, MAPS, SCORES>(tm_q, tm_kv, p, st)
   if (s->maps == 1) {
     if (bias != nullptr) GROUPED_PREFILL(1, SCORES_BIAS);
+    if (s->slopes != nullptr) GROUPED_PREFILL(1, SCORES_SLOPE);
     if (s->softcap > 0.f) GROUPED_PREFILL(1, SCORES_CAP);
     GROUPED_PREFILL(1, SCORES_PLAIN);
   }

@@ -2,7 +2,8 @@
 //
 // The router's logits come out of a GEMM in fp32, or, for the few rows of a decode step, out of moe_route_rows itself (one block per row).
 // moe_route takes the softmax over all outputs of a row, chooses the `top` outputs
-// with the largest score + correction and weighs them with their share of the scores; outputs from `experts` on are identities (the
+// with the largest score + correction (without a correction: the largest logits) and weighs them with their share of the scores, which is the
+// softmax over the chosen logits; a bias may be added to the logits first; outputs from `experts` on are identities (the
 // experts' input itself) and need no expert row.  A chosen expert's place among the rows that chose it comes from a counter per
 // expert (counted per block in shared memory first).  moe_dispatch turns the counters into tiles (every block does the short prefix
 // sum itself), writes where each choice's row went and copies the rows there.  `always` further experts behind the others receive every
@@ -19,7 +20,8 @@ constexpr int ROUTE_ROWS = 4;              // rows of a warp
 struct RouteParams {
   const float* z;              // (rows, ld_z): logits of experts + identities
   long long ld_z;
-  const float* correction;     // (outputs)
+  const float* bias;           // (outputs) added to the logits, or null
+  const float* correction;     // (outputs), or null: the choice is by logit
   const long long* slots;      // negative = padding row
   int* choice;                 // (rows, top): chosen output, -1 for a padding row
   int* rank;                   // (rows, top): place among the rows of the chosen expert
@@ -28,22 +30,28 @@ struct RouteParams {
   int rows, experts, outputs, top, always;       // always > 0: z has one more column
 };
 
-// Choice of one row by one warp: the softmax of s[0 .. outputs) in place, then outputs with the largest score + correction, which go to
+// Choice of one row by one warp: the softmax of s[0 .. outputs) (plus bias) in place, then outputs with the largest score + correction, which go to
 // picked[0], picked[stride], ...  Returns the sum of the chosen scores.  key: scratch.  Ties go to the lower index.
-__device__ __forceinline__ float route_choose(float* s, float* key, const float* __restrict__ correction, int outputs, int top, int* picked,
-                                              int stride) {
+__device__ __forceinline__ float route_choose(float* s, float* key, const float* __restrict__ bias, const float* __restrict__ correction, int outputs,
+                                              int top, int* picked, int stride) {
   const int lane = threadIdx.x & 31;
   float mx = -INFINITY;
-  for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, s[e]);
+  for (int e = lane; e < outputs; e += 32) {
+    if (bias != nullptr) s[e] += bias[e];
+    mx = fmaxf(mx, s[e]);
+  }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
   float sum = 0.f;
-  for (int e = lane; e < outputs; e += 32) sum += s[e] = expf(s[e] - mx);
+  for (int e = lane; e < outputs; e += 32) {
+    key[e] = s[e];
+    sum += s[e] = expf(s[e] - mx);
+  }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
   for (int e = lane; e < outputs; e += 32) {
     s[e] /= sum;
-    key[e] = s[e] + correction[e];
+    if (correction != nullptr) key[e] = s[e] + correction[e];
   }
   __syncwarp();
   float total = 0.f;
@@ -100,7 +108,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(const Route
     }
     const float* z = p.z + (long long)row * p.ld_z;
     for (int e = lane; e < p.outputs; e += 32) s[e] = z[e];
-    const float total = route_choose(s, key, p.correction, p.outputs, p.top, mine, 2);
+    const float total = route_choose(s, key, p.bias, p.correction, p.outputs, p.top, mine, 2);
     for (int k = lane; k < p.top; k += 32)
       if (mine[2 * k] < p.experts) mine[2 * k + 1] = atomicAdd(&local[mine[2 * k]], 1);
     for (int k = lane; k < p.top; k += 32) {
@@ -184,7 +192,7 @@ __global__ void __launch_bounds__(512) moe_route_rows_kernel(const RouteRowsPara
   if (warp > 0) return;
   const bool live = r.slots[row] >= 0;
   const float share = r.always > 0 && live ? 1.f / (1.f + expf(-s[r.outputs])) : 0.f;
-  const float total = route_choose(s, key, r.correction, r.outputs, r.top, picked, 1);
+  const float total = route_choose(s, key, r.bias, r.correction, r.outputs, r.top, picked, 1);
   const int wide = r.top + r.always;
   for (int k = lane; k < wide; k += 32) {
     if (k >= r.top) {
@@ -280,20 +288,20 @@ __global__ void __launch_bounds__(256) moe_dispatch_kernel(const DispatchParams 
 
 using namespace b200;
 
-static int route_params(RouteParams& p, const float* z, long long ld_z, const float* correction, const long long* slots, int* choice, int* rank,
-                        float* weight, int* count, int rows, int experts, int outputs, int top, int always) {
+static int route_params(RouteParams& p, const float* z, long long ld_z, const float* bias, const float* correction, const long long* slots, int* choice,
+                        int* rank, float* weight, int* count, int rows, int experts, int outputs, int top, int always) {
   if (experts <= 0 || outputs < experts || top <= 0 || top > outputs || always < 0) return -10;
-  p.z = z; p.ld_z = ld_z; p.correction = correction; p.slots = slots; p.choice = choice; p.rank = rank; p.weight = weight; p.count = count;
+  p.z = z; p.ld_z = ld_z; p.bias = bias; p.correction = correction; p.slots = slots; p.choice = choice; p.rank = rank; p.weight = weight; p.count = count;
   p.rows = rows; p.experts = experts; p.outputs = outputs; p.top = top; p.always = always;
   return 0;
 }
 
 // `count` (experts ints) must be zero; identities are the outputs from `experts` on; with `always`, z has a column behind the outputs.
-extern "C" int b200_moe_route(const float* z, long long ld_z, const float* correction, const long long* slots, int* choice, int* rank,
-                              float* weight, int* count, int rows, int experts, int outputs, int top, int always, cudaStream_t st) {
+extern "C" int b200_moe_route(const float* z, long long ld_z, const float* bias, const float* correction, const long long* slots, int* choice,
+                              int* rank, float* weight, int* count, int rows, int experts, int outputs, int top, int always, cudaStream_t st) {
   if (rows <= 0) return 0;
   RouteParams p;
-  if (route_params(p, z, ld_z, correction, slots, choice, rank, weight, count, rows, experts, outputs, top, always)) return -10;
+  if (route_params(p, z, ld_z, bias, correction, slots, choice, rank, weight, count, rows, experts, outputs, top, always)) return -10;
   const size_t smem = (size_t)ROUTE_WARPS * 2 * outputs * 4 + 2ull * experts * 4 + (size_t)ROUTE_WARPS * ROUTE_ROWS * top * 8;
   if (smem > 200 * 1024) return -12;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
@@ -304,11 +312,11 @@ extern "C" int b200_moe_route(const float* z, long long ld_z, const float* corre
 
 // The same for few rows, with the product: h (rows, d), w (columns, d), columns = outputs or one more; z (rows, ld_z) is written.
 extern "C" int b200_moe_route_rows(const void* h, long long ld_h, const void* w, long long ld_w, int d, int columns, float* z, long long ld_z,
-                                   const float* correction, const long long* slots, int* choice, int* rank, float* weight, int* count,
-                                   int rows, int experts, int outputs, int top, int always, int f32, cudaStream_t st) {
+                                   const float* bias, const float* correction, const long long* slots, int* choice, int* rank, float* weight,
+                                   int* count, int rows, int experts, int outputs, int top, int always, int f32, cudaStream_t st) {
   if (rows <= 0) return 0;
   RouteRowsParams p;
-  if (route_params(p.r, z, ld_z, correction, slots, choice, rank, weight, count, rows, experts, outputs, top, always)) return -10;
+  if (route_params(p.r, z, ld_z, bias, correction, slots, choice, rank, weight, count, rows, experts, outputs, top, always)) return -10;
   if (d <= 0 || columns < outputs + (always > 0) || ld_z < columns) return -10;
   p.z = z; p.h = h; p.w = w; p.ld_h = ld_h; p.ld_w = ld_w; p.d = d; p.columns = columns;
   const size_t smem = (size_t)((columns + outputs + top + 3) / 4 * 4 + d) * 4;

@@ -45,6 +45,33 @@ struct alignas(sizeof(T) * VEC) Raw {       // VEC elements as they are stored
   T v[VEC];
 };
 
+template <typename T>
+struct Piece {                    // 8 elements as they are stored
+  uint4 v[sizeof(T) / 2];
+};
+__device__ __forceinline__ void unpack(const Piece<__nv_bfloat16>& r, float (&f)[8]) {
+  const float2 a = unpack_bf16x2(r.v[0].x), b = unpack_bf16x2(r.v[0].y), c = unpack_bf16x2(r.v[0].z), d = unpack_bf16x2(r.v[0].w);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
+}
+__device__ __forceinline__ void unpack(const Piece<float>& r, float (&f)[8]) {
+  f[0] = __uint_as_float(r.v[0].x); f[1] = __uint_as_float(r.v[0].y); f[2] = __uint_as_float(r.v[0].z); f[3] = __uint_as_float(r.v[0].w);
+  f[4] = __uint_as_float(r.v[1].x); f[5] = __uint_as_float(r.v[1].y); f[6] = __uint_as_float(r.v[1].z); f[7] = __uint_as_float(r.v[1].w);
+}
+template <typename T>
+__device__ __forceinline__ Piece<T> load_piece(const T* p) {
+  Piece<T> r;
+#pragma unroll
+  for (int j = 0; j < (int)sizeof(T) / 2; ++j) r.v[j] = reinterpret_cast<const uint4*>(p)[j];
+  return r;
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+}
+__device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+}
+
 // Sum over the block (blockDim.x a multiple of 32, at most 1024); every thread receives it.  `red`: 32 floats.
 __device__ __forceinline__ float block_total(float v, float* red) {
 #pragma unroll
