@@ -29,7 +29,7 @@ SERVING_LIB_PATH = PKG_DIR / "_b200_serving.so"
 NOT_FOR_SERVING = {"flash_attn_bwd.cu"}     # training only (comm_kernels.cu holds host code of the GEMMs)
 # kernels that belong to single mixers or feed-forwards; a model class names those it uses (KERNELS)
 MIXERS = {"flash_attn_fwd.cu", "latent_attention.cu", "latent_decode_tc.cu", "retention.cu", "grouped_attention.cu",
-          "grouped_prefill.cu", "mlstm.cu", "moe_route.cu"}
+          "grouped_prefill.cu", "mlstm.cu", "moe_route.cu", "short_conv.cu", "delta.cu", "group_norm.cu"}
 HOST_SRC = CSRC / "host" / "host_runtime.cpp"
 HOST_LIB_PATH = PKG_DIR / "_b200_host.so"
 

@@ -563,9 +563,6 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
     tmem_alloc(tmem_holder, 512);
     tmem_relinquish();
   }
-  // v of an unloaded half panel is never read; K and Q past dim stay finite
-  for (int i = tid; i < (2 * L::STAGE >> 4); i += DK_THREADS) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
-  fence_proxy_async_smem();
   pdl_sync();
   const int seq = blockIdx.x / p.heads, h = blockIdx.x - seq * p.heads, hk = h / (p.heads / p.kv_heads), D = p.dim, E = p.vdim;
   const int row0 = p.cu[seq], rows = p.cu[seq + 1] - row0, slot = p.state_slots[seq];
@@ -776,14 +773,11 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
     for (int ch = 0; ch < chunks; ++ch) {
       const int st = ch & 1, n = min(DC, rows - ch * DC);
       const float* f = reinterpret_cast<const float*>(smem + st * L::STAGE + L::X + L::V + DI_F) + 3 * DC;
-      ok = mbar_wait(&full[st], (ch >> 1) & 1, abort_word) && mbar_wait(o_full, ch & 1, abort_word);
-      if (!__all_sync(0xffffffffu, ok)) {
-        ok = false;
-        *abort_word = ERR_WAIT_TMEM_FULL;
-      }
+      // after a wait that gave up the loop goes on, without waiting, so that the four warps meet at every barrier
+      if (!mbar_wait(&full[st], (ch >> 1) & 1, abort_word) || !mbar_wait(o_full, ch & 1, abort_word)) *abort_word = ERR_WAIT_TMEM_FULL;
+      __syncwarp();
       tc_fence_after();
       asm volatile("bar.sync 2, 128;" ::: "memory");      // the rows of the chunk before have been read
-      if (*abort_word != 0) break;
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         uint32_t a[32], b[32];

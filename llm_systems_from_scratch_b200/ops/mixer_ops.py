@@ -33,8 +33,8 @@ def _lib():
             "b200_gate_sigmoid": [P, P, L, I, I, L, L, I, P],
             "b200_gemm_f32": [P, P, P, I, I, I, L, L, L, I, P, I, I, I, I, P, P],
             "b200_gemm_bf16_grouped": [P, P, P, P, I, I, I, L, L, L, L, P, I, I, I, I, I, I, I, I, P, P, P],
-            "b200_moe_route": [P, L, P, P, P, P, P, P, I, I, I, I, I, P],
-            "b200_moe_route_rows": [P, L, P, L, I, I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, P],
+            "b200_moe_route": [P, L, P, P, P, P, P, P, P, I, I, I, I, I, P],
+            "b200_moe_route_rows": [P, L, P, L, I, I, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
             "b200_moe_dispatch": [P, L, P, L, P, P, P, P, P, I, I, I, I, I, I, I, P],
             "b200_latent_norm_append": [P, L, P, P, P, L, P, P, I, I, I, I, L, F, I, P, P],
             "b200_latent_gather": [P, P, P, P, P, I, I, I, I, I, I, P, P],
@@ -50,6 +50,12 @@ def _lib():
             "b200_grouped_decode": [P, P, P, L, P, L, P, I, P, P, P, P, P, I, I, I, I, I, P, P, P],
             "b200_grouped_prefill": [P, P, P, L, P, L, P, I, P, P, P, I, I, I, I, I, I, P, P, P],
             "b200_mlstm": [P, L, P, L, P, L, P, L, I, P, P, P, L, P, P, P, P, I, I, I, I, I, I, I, F, F, I, I, P, P],
+            "b200_short_conv": [P, P, L, I, I, P, P],
+            "b200_short_conv_attend": [P, P, P, P, L, P, P, L, L, I, F, P, I, P, P],
+            "b200_group_step": [P, P, P, P, P, P, L, F, I, I, I, I, I, P, P],
+            "b200_delta": [P, I, I, P],
+            "b200_delta_image_bytes": [],
+            "b200_delta_chunk_tokens": [],
             "b200_retention_recurrent": [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
         }.items():
             fn = getattr(lib, name, None)
@@ -332,28 +338,30 @@ def moe_plan(tokens, slots, tables, experts):
     return ([pos[i, :rows * t.shape[1]].view(rows, t.shape[1]) for i, t in enumerate(tables)], [group[i] for i in range(len(tables))])
 
 
-def moe_route(z, correction, slots, experts: int, top: int, count, always: int = 0):
-    """Choose experts by score: z (R, outputs) fp32 logits of the experts and, behind them, of identities; scores are their softmax.  The
-    ``top`` outputs with the largest score + correction are chosen and weighted by their share of the chosen scores.  ``count``
+def moe_route(z, correction, slots, experts: int, top: int, count, always: int = 0, bias=None):
+    """Choose experts by score: z (R, outputs) fp32 logits of the experts and, behind them, of identities, plus ``bias``; scores are their
+    softmax.  The ``top`` outputs with the largest score + correction (``correction`` None: the largest logits) are chosen and weighted by
+    their share of the chosen scores.  ``count``
     (experts,) int32, zero on entry, receives the rows per expert.  ``always``: that many weights sigmoid(z[:, outputs]) more per row
     (z has one more column).  Returns choice (-1 in padding rows) and rank among the expert's rows, (R, top), and weight
     (R, top + always)."""
-    rows, outputs = z.shape[0], correction.numel()
-    _req(z.shape[1] == outputs + (always > 0) and 0 < top <= outputs and experts <= outputs, "bad router sizes")
+    rows, outputs = z.shape[0], z.shape[1] - (always > 0)
+    _req(0 < top <= outputs and experts <= outputs, "bad router sizes")
     if not z.is_cuda:
-        return mixer_torch.moe_route(z, correction, slots, experts, top, count, always)
+        return mixer_torch.moe_route(z, correction, slots, experts, top, count, always, bias)
     _req(z.dtype == torch.float32 and z.stride(1) == 1, "bad logits")
-    choice, rank, weight = _route_buffers(rows, top, always, correction, slots, experts, count)
-    _check(_lib().b200_moe_route(_ptr(z), z.stride(0), _ptr(correction), _ptr(slots), _ptr(choice), _ptr(rank), _ptr(weight),
+    choice, rank, weight = _route_buffers(rows, outputs, top, always, bias, correction, slots, experts, count)
+    _check(_lib().b200_moe_route(_ptr(z), z.stride(0), _ptr(bias), _ptr(correction), _ptr(slots), _ptr(choice), _ptr(rank), _ptr(weight),
                                  _ptr(count), rows, experts, outputs, top, always, _stream()), "moe_route")
     return choice, rank, weight
 
 
-def _route_buffers(rows, top, always, correction, slots, experts, count):
-    _req(correction.dtype == torch.float32 and correction.is_contiguous() and count.dtype == torch.int32 and count.is_contiguous()
+def _route_buffers(rows, outputs, top, always, bias, correction, slots, experts, count):
+    fits = lambda t: t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == outputs)
+    _req(fits(bias) and fits(correction) and count.dtype == torch.int32 and count.is_contiguous()
          and count.numel() == experts and slots.dtype == torch.int64 and slots.numel() == rows, "bad router inputs")
-    choice, rank = (torch.empty((rows, top), dtype=torch.int32, device=correction.device) for _ in range(2))
-    return choice, rank, torch.empty((rows, top + always), dtype=torch.float32, device=correction.device)
+    choice, rank = (torch.empty((rows, top), dtype=torch.int32, device=slots.device) for _ in range(2))
+    return choice, rank, torch.empty((rows, top + always), dtype=torch.float32, device=slots.device)
 
 
 ROUTE_ROWS, ROUTE_BYTES = 256, 32 << 20          # rows, and bytes of the router read once per row, up to which one kernel does it all
@@ -364,14 +372,15 @@ def routes_rows(rows: int, w) -> bool:
     return w.is_cuda and rows <= ROUTE_ROWS and rows * w.numel() * w.element_size() <= ROUTE_BYTES and 3 * w.shape[0] + w.shape[1] <= 12000
 
 
-def moe_route_rows(h, w, correction, slots, experts: int, top: int, count, always: int = 0):
+def moe_route_rows(h, w, correction, slots, experts: int, top: int, count, always: int = 0, bias=None):
     """``moe_route`` of the few rows of a decode step with the router's product, z = h w^T in fp32.  Returns z too."""
     (rows, d), columns = h.shape, w.shape[0]
-    _req(h.is_cuda and h.dtype == w.dtype and h.stride(1) == 1 and w.shape[1] == d and columns >= correction.numel() + (always > 0), "bad router")
+    outputs = columns if correction is None else correction.numel()
+    _req(h.is_cuda and h.dtype == w.dtype and h.stride(1) == 1 and w.shape[1] == d and columns >= outputs + (always > 0), "bad router")
     z = torch.empty((rows, columns), dtype=torch.float32, device=h.device)
-    choice, rank, weight = _route_buffers(rows, top, always, correction, slots, experts, count)
-    _check(_lib().b200_moe_route_rows(_ptr(h), h.stride(0), _ptr(w), w.stride(0), d, columns, _ptr(z), columns, _ptr(correction), _ptr(slots),
-                                      _ptr(choice), _ptr(rank), _ptr(weight), _ptr(count), rows, experts, correction.numel(), top, always,
+    choice, rank, weight = _route_buffers(rows, outputs, top, always, bias, correction, slots, experts, count)
+    _check(_lib().b200_moe_route_rows(_ptr(h), h.stride(0), _ptr(w), w.stride(0), d, columns, _ptr(z), columns, _ptr(bias), _ptr(correction),
+                                      _ptr(slots), _ptr(choice), _ptr(rank), _ptr(weight), _ptr(count), rows, experts, outputs, top, always,
                                       _f32(h), _stream()), "moe_route_rows")
     return z, choice, rank, weight
 
@@ -666,7 +675,8 @@ def mlstm(proj, gates, gate_bias, weight, state, state_slots, cu, spans, positio
 @dataclass
 class AttentionShape:
     """Sizes and constants of one grouped attention (``models.mixers.GroupedAttention``); ``bias`` (heads, n) fp32 holds the bias
-    per distance, distances from n - 1 on read its last column.  ``softcap`` 0: scores are not capped; ``sink`` (heads,) fp32 or None;
+    per distance, distances from n - 1 on read its last column; ``slopes`` (heads,) fp32 takes slope * distance off instead.  ``chunked``:
+    position i sees j <= i in the same chunk of ``window`` positions.  ``head_gate``: the output gate has a column per head.  ``softcap`` 0: scores are not capped; ``sink`` (heads,) fp32 or None;
     ``whole_norm``: one norm over all queries (and keys) of a token instead of one per head."""
     heads: int
     kv_heads: int
@@ -684,6 +694,9 @@ class AttentionShape:
     softcap: float = 0.0
     sink: torch.Tensor | None = None
     whole_norm: bool = False
+    slopes: torch.Tensor | None = None
+    chunked: bool = False
+    head_gate: bool = False
 
     @property
     def q_pitch(self) -> int:
@@ -706,7 +719,8 @@ class AttentionShape:
 class _NativeShape(ctypes.Structure):
     """csrc/grouped_attention.cuh: GroupedShape"""
     _fields_ = [(n, ctypes.c_int) for n in ("heads", "kv_heads", "maps", "dim", "vdim", "qp", "kp", "vp", "window", "keep")] + \
-               [(n, ctypes.c_float) for n in ("scale", "eps", "difference", "out_scale", "softcap")] + [("sink", ctypes.c_void_p)]
+               [(n, ctypes.c_float) for n in ("scale", "eps", "difference", "out_scale", "softcap")] + \
+               [("sink", ctypes.c_void_p), ("slopes", ctypes.c_void_p), ("chunked", ctypes.c_int), ("head_gate", ctypes.c_int)]
 
 
 def _native_shape(s: AttentionShape):
@@ -714,7 +728,7 @@ def _native_shape(s: AttentionShape):
     if got is None:
         got = s.__dict__["_native"] = _NativeShape(s.heads, s.kv_heads, s.maps, s.dim, s.vdim, s.q_pitch, s.k_pitch, s.v_pitch,
                                                    s.window, s.keep, s.scale, s.eps, s.difference, s.out_scale, s.softcap,
-                                                   _ptr(s.sink))
+                                                   _ptr(s.sink), _ptr(s.slopes), int(s.chunked), int(s.head_gate))
     return ctypes.byref(got)
 
 
@@ -759,7 +773,7 @@ def _attention_args(q, s, cache, positions, tables, out, gate):
          and cache.shape[-1] == s.cache_width, "bad queries or cache")
     _req(tables.dtype == torch.int32 and tables.is_contiguous() and positions.dtype == torch.int32, "bad tables")
     _req(out.shape == (q.shape[0], s.heads * s.vdim) and out.dtype == q.dtype and out.stride(1) == 1, "bad output")
-    _req(gate is None or (gate.shape == out.shape and gate.dtype == q.dtype and gate.stride(1) == 1), "bad gate")
+    _req(gate is None or (gate.shape == (out.shape[0], s.heads if s.head_gate else out.shape[1]) and gate.dtype == q.dtype and gate.stride(1) == 1), "bad gate")
     return (_ptr(q), _ptr(cache), _ptr(out), out.stride(0), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(s.bias),
             0 if s.bias is None else s.bias.shape[1])
 
@@ -815,3 +829,213 @@ def attention_portions(q, s: AttentionShape, cache, positions, cu, max_q: int, t
                                        tables.shape[1], cache.shape[1], cache.shape[0], _native_shape(s),
                                        _ptr(native.status_word(q.device)), _stream()), "grouped_prefill")
     return out
+
+
+# --------------------------------------------------------------------------------------- short convolution
+class _ConvInput(ctypes.Structure):
+    """csrc/short_conv.cu: ConvInput"""
+    _fields_ = [(n, ctypes.c_void_p) for n in ("u", "w", "ring", "state_slots", "row_seq", "cu", "positions")] + \
+               [("ld_u", ctypes.c_longlong)] + [(n, ctypes.c_int) for n in ("seq0", "seqs", "rows", "channels", "taps", "num_slots")]
+
+
+class StepRows(NamedTuple):
+    """A part of a step's rows: single rows (``cu`` None) or portions."""
+    positions: torch.Tensor                  # (R,) int32
+    slots: torch.Tensor                      # (R,) int64 cache slots
+    state_slots: torch.Tensor                # (sequences,) int32
+    row_seq: torch.Tensor                    # (R,) int32, the first sequence is ``seq0``
+    seq0: int
+    cu: torch.Tensor | None                  # (sequences + 1,) int32
+    spans: list                              # the same on the host: (first row, one past the last)
+
+
+def step_parts(batch):
+    """(rows, StepRows) of a step's single rows and of its portions, those that it has."""
+    n, rows = batch.n_single, batch.n_rows
+    out = []
+    if n:
+        one = slice(0, n)
+        out.append((one, StepRows(batch.positions[one], batch.slots[one], batch.state_slots[one], batch.row_seq[one], 0, None,
+                                  [(i, i + 1) for i in range(n)])))
+    if rows > n:
+        rest = slice(n, rows)
+        out.append((rest, StepRows(batch.positions[rest], batch.slots[rest], batch.state_slots[n:], batch.row_seq[rest], n, batch.cu,
+                                   batch.spans)))
+    return out
+
+
+def _conv_input(u, w, ring, at: StepRows):
+    taps, channels = w.shape
+    _req(u.shape[1] == channels and u.stride(1) == 1 and w.is_contiguous() and w.dtype == u.dtype, "bad convolution")
+    _req(ring.dtype == u.dtype and ring.is_contiguous() and ring.shape[1:] == (taps, channels), "bad ring")
+    _req(at.positions.dtype == torch.int32 and at.positions.numel() == u.shape[0] and at.state_slots.dtype == torch.int32
+         and at.row_seq.dtype == torch.int32 and at.row_seq.numel() == u.shape[0], "bad rows")
+    _req(at.cu is None or (at.cu.dtype == torch.int32 and at.cu.numel() == at.state_slots.numel() + 1), "bad row offsets")
+    single = at.cu is None
+    return _ConvInput(_ptr(u), _ptr(w), _ptr(ring), _ptr(at.state_slots), None if single else _ptr(at.row_seq), _ptr(at.cu),
+                      _ptr(at.positions), u.stride(0), at.seq0, at.state_slots.numel(), u.shape[0], channels, taps, ring.shape[0])
+
+
+def short_conv(u, w, ring, at: StepRows, y, silu: bool = False):
+    """Causal convolution over time: y_t = sum_j w[j] u_(t - taps + 1 + j) per channel, zeros in front of a sequence; w (taps, channels).
+    ``ring`` (slots, taps, channels) holds what earlier steps brought and receives what later ones need."""
+    if not u.is_cuda:
+        return y.copy_(mixer_torch.short_conv(u, w, ring, at, silu))
+    _req(y.shape == u.shape and y.dtype == u.dtype and y.stride(1) == 1, "bad output")
+    arg = _conv_input(u, w, ring, at)
+    _check(_lib().b200_short_conv(ctypes.byref(arg), _ptr(y), y.stride(0), int(silu), _f32(u), _ptr(native.status_word(u.device)), _stream()),
+           "short_conv")
+    return y
+
+
+def conv_attend(u, w, ring, at: StepRows, s: AttentionShape, temp, cache, first=None, mix: float = 0.0):
+    """The short convolution of q | k | v: returns the queries, times ``temp`` (heads,) fp32, (R, heads * q_pitch) with zeros behind every head;
+    keys and values go to their cache slots (negative slot: not written).  ``first``: another layer's cache; its values of the same
+    token join with weight ``mix``, v <- (1 - mix) v + mix v_first."""
+    q = torch.empty((u.shape[0], s.heads * s.q_pitch), dtype=u.dtype, device=u.device)
+    if not u.is_cuda:
+        return mixer_torch.conv_attend(u, w, ring, at, s, temp, cache, first, mix, q)
+    arg = _conv_input(u, w, ring, at)
+    _req(cache.is_contiguous() and cache.dtype == u.dtype and cache.shape[-1] == s.cache_width and at.slots.dtype == torch.int64
+         and at.slots.numel() == u.shape[0] and temp.dtype == torch.float32 and temp.numel() == s.heads, "bad cache or rows")
+    width = 0 if first is None else first.shape[-1]
+    _req(first is None or (first.is_contiguous() and first.dtype == u.dtype and first.shape[:2] == cache.shape[:2]
+                           and width >= s.kv_heads * s.v_pitch), "bad cache of the first values")
+    _check(_lib().b200_short_conv_attend(
+        ctypes.byref(arg), _ptr(q), _ptr(cache), _ptr(at.slots), cache.shape[0] * cache.shape[1], _ptr(temp), _ptr(first), width,
+        width - s.kv_heads * s.v_pitch, s.v_pitch, float(mix), _native_shape(s), _f32(u), _ptr(native.status_word(u.device)), _stream()),
+        "short_conv_attend")
+    return q
+
+
+# ------------------------------------------------------------------------------------------ gated delta rule
+class _DeltaArgs(ctypes.Structure):
+    """csrc/delta.cu: DeltaArgs"""
+    _fields_ = [(n, ctypes.c_void_p) for n in ("c", "gate", "ab", "h", "w_ab", "decay", "dt", "weight", "filter", "ring", "y", "state", "image",
+                                               "state_slots", "cu", "positions", "chunk_cu", "status")] + \
+               [(n, ctypes.c_longlong) for n in ("ld_c", "ld_gate", "ld_ab", "ld_h", "ld_w", "ld_y")] + \
+               [(n, ctypes.c_int) for n in ("width", "taps", "seqs", "rows", "heads", "kv_heads", "dim", "vdim", "num_slots", "chunks")] + \
+               [("eps", ctypes.c_float)]
+
+
+def delta_chunkable(dtype, dim: int, vdim: int) -> bool:
+    return dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and vdim <= 128
+
+
+def delta_steps(dim: int, vdim: int) -> bool:
+    """Whether a decode step of these sizes runs on the one-pass kernel, which also takes the gates' products and the convolution."""
+    groups = vdim // 4
+    return vdim % 4 == 0 and 0 < groups <= 256 and -(-dim // max(1, 256 // groups)) <= 16
+
+
+def delta_rule(c, gate, ab, decay, dt, weight, state, at: StepRows, kv_heads: int, eps: float, y, conv=None, chunks=None):
+    """Gated delta rule over rows q | k | v of ``c``: S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q with unit q (times dim^-1/2) and
+    k, g = exp(decay softplus(a + dt)), beta = sigmoid(b); y (R, heads * vdim) receives o / rms(o) * weight * silu(gate).  ``ab`` (R, 2 * heads)
+    fp32: a | b; or, in a step of ``delta_steps`` sizes, the pair (input rows h, weights of a | b).  The states (slots, heads, dim, vdim) are
+    read and left in their slots.  ``conv`` = (w (taps, channels), ring): single rows of ``delta_steps`` sizes pass the short convolution and
+    silu here.  ``chunks`` = (offsets, number) of 64-token chunks (``StepBatch.chunk_ranges``): the tensor-core kernels for portions."""
+    h = w_ab = None
+    if isinstance(ab, tuple):
+        h, w_ab = ab
+        ab = None if c.is_cuda else h.float() @ w_ab.float().t()
+    if not c.is_cuda:
+        if conv is not None:
+            c = mixer_torch.short_conv(c, conv[0], conv[1], at, True)
+        return mixer_torch.delta_rule(c, gate, ab, decay, dt, weight, state, at, kv_heads, eps, y)
+    slots, heads, dim, vdim = state.shape
+    _req(state.dtype == torch.float32 and state.is_contiguous() and c.shape[1] == 2 * kv_heads * dim + heads * vdim and c.stride(1) == 1, "bad state")
+    _req(at.state_slots.dtype == torch.int32 and at.positions.dtype == torch.int32 and decay.dtype == torch.float32 and dt.dtype == torch.float32
+         and decay.numel() == heads and dt.numel() == heads, "bad inputs")
+    _req(gate.shape == (c.shape[0], heads * vdim) and y.shape == gate.shape and gate.dtype == c.dtype and y.dtype == c.dtype
+         and gate.stride(1) == 1 and y.stride(1) == 1 and weight.dtype == c.dtype and weight.numel() == vdim, "bad shapes")
+    if ab is None:
+        _req(h.dtype == c.dtype and w_ab.dtype == c.dtype and h.stride(1) == 1 and w_ab.shape == (2 * heads, h.shape[1])
+             and at.cu is None and delta_steps(dim, vdim), "bad inputs of the gates")
+    else:
+        _req(ab.dtype == torch.float32 and ab.shape == (c.shape[0], 2 * heads) and ab.stride(1) == 1, "bad gates")
+    w = ring = image = None
+    if conv is not None:
+        w, ring = conv
+        _req(at.cu is None and delta_steps(dim, vdim) and w.is_contiguous() and w.dtype == c.dtype and ring.is_contiguous() and ring.dtype == c.dtype
+             and ring.shape == (slots, *w.shape) and w.shape[1] == c.shape[1], "bad convolution")
+    lib = _lib()
+    if chunks is not None:
+        _req(delta_chunkable(c.dtype, dim, vdim) and at.cu is not None, "sizes the chunked kernel does not take")
+        _req(chunks[0].dtype == torch.int32 and chunks[0].numel() == at.state_slots.numel() + 1, "bad chunks")
+        image = torch.empty(chunks[1] * heads * lib.b200_delta_image_bytes(), dtype=torch.uint8, device=c.device)
+    ld = lambda t: 0 if t is None else t.stride(0)
+    args = _DeltaArgs(_ptr(c), _ptr(gate), _ptr(ab), _ptr(h), _ptr(w_ab), _ptr(decay), _ptr(dt), _ptr(weight), _ptr(w), _ptr(ring), _ptr(y),
+                      _ptr(state), _ptr(image), _ptr(at.state_slots), _ptr(at.cu), _ptr(at.positions), None if chunks is None else _ptr(chunks[0]),
+                      _ptr(native.status_word(c.device)), ld(c), ld(gate), ld(ab), ld(h), ld(w_ab), ld(y), 0 if h is None else h.shape[1],
+                      0 if w is None else w.shape[0], at.state_slots.numel(), c.shape[0], heads, kv_heads, dim, vdim, slots,
+                      0 if chunks is None else chunks[1], float(eps))
+    _check(lib.b200_delta(ctypes.byref(args), int(chunks is not None), _f32(c), _stream()), "delta_chunk" if chunks is not None else "delta")
+    return y
+
+
+DELTA_CHUNK = 64                 # tokens per chunk of the tensor-core kernels (csrc/delta.cu: DC)
+
+
+# ------------------------------------------------------------------------- gated sublayers between group norms
+class _GroupStart(ctypes.Structure):
+    """csrc/group_norm.cu: GroupStart"""
+    _fields_ = [(n, ctypes.c_void_p) for n in ("tokens", "embed", "bigram", "prev", "state_slots", "row_seq", "positions", "cu")] + \
+               [(n, ctypes.c_longlong) for n in ("mul_prev", "mul_cur")] + \
+               [(n, ctypes.c_int) for n in ("vocab", "buckets", "num_slots", "n_single", "portions")] + [("scale", ctypes.c_float)]
+
+
+class _GroupSublayer(ctypes.Structure):
+    """csrc/group_norm.cu: GroupSublayer"""
+    _fields_ = [(n, ctypes.c_void_p) for n in ("y", "gate", "w_post", "ypos", "yweight")] + \
+               [(n, ctypes.c_longlong) for n in ("ld_y", "ld_gate")] + [(n, ctypes.c_int) for n in ("ytop", "y_rows")]
+
+
+class EmbeddingStart(NamedTuple):
+    """x = embed[token] * scale, plus bigram[(previous token * mul_prev + token * mul_cur) mod buckets] (its last row for a sequence's first
+    token); ``prev`` (slots, 1) int32 holds the sequences' last tokens."""
+    embed: torch.Tensor
+    scale: float
+    bigram: torch.Tensor | None = None       # (buckets + 1, d)
+    mul_prev: int = 0
+    mul_cur: int = 0
+    prev: torch.Tensor | None = None
+
+
+class GatedOutput(NamedTuple):
+    """What a gated sublayer adds to the residual stream: group_norm(y * sigmoid(gate)) * w_post."""
+    y: torch.Tensor | ExpertOutputs
+    gate: torch.Tensor                       # (R, d)
+    w_post: torch.Tensor
+
+
+def group_step(x, groups: int, eps: float, w=None, start: EmbeddingStart | None = None, batch=None, sub: GatedOutput | None = None, row_index=None):
+    """One pass over the fp32 residual stream x (R, d): starts the rows of ``batch``, or adds a sublayer's output; returns
+    h = group_norm(x) * w (no ``w``: None).  ``row_index``: h for these rows of x only, x itself stays as it is."""
+    if not x.is_cuda:
+        return mixer_torch.group_step(x, groups, eps, w, start, batch, sub, row_index)
+    d = x.shape[1]
+    rows = x.shape[0] if row_index is None else row_index.numel()
+    act = w if w is not None else (start.embed if start is not None else sub.w_post)
+    fits = lambda t: t is None or (t.dtype == act.dtype and t.is_contiguous() and t.shape[-1] == d)
+    _req(x.dtype == torch.float32 and x.is_contiguous() and d % groups == 0 and fits(w), "bad residual stream")
+    _req(row_index is None or (row_index.dtype == torch.int64 and row_index.is_contiguous() and start is None), "row_index must be int64")
+    a = b = None
+    if start is not None:
+        _req(fits(start.embed) and fits(start.bigram) and batch.tokens.dtype == torch.int64 and batch.tokens.numel() == rows, "bad embedding")
+        _req(start.bigram is None or (start.prev.dtype == torch.int32 and start.prev.is_contiguous()), "bad token state")
+        a = _GroupStart(_ptr(batch.tokens), _ptr(start.embed), _ptr(start.bigram), _ptr(start.prev), _ptr(batch.state_slots), _ptr(batch.row_seq),
+                        _ptr(batch.positions), _ptr(batch.cu), start.mul_prev, start.mul_cur, start.embed.shape[0],
+                        0 if start.bigram is None else start.bigram.shape[0] - 1, 0 if start.prev is None else start.prev.shape[0], batch.n_single,
+                        len(batch.portions), float(start.scale))
+    if sub is not None:
+        y, ex = (sub.y.y, sub.y) if isinstance(sub.y, ExpertOutputs) else (sub.y, None)
+        _req(y.dtype == act.dtype and y.shape[1] == d and y.stride(1) == 1 and fits(sub.w_post) and sub.gate.dtype == act.dtype
+             and sub.gate.shape == x.shape and sub.gate.stride(1) == 1, "bad sublayer output")
+        _req(y.shape[0] == x.shape[0] if ex is None else (ex.z is None and ex.s is None and ex.pos.shape == ex.weight.shape and ex.pos.is_contiguous()
+             and ex.weight.is_contiguous() and ex.scale == 1.0 and ex.pos.shape[0] == x.shape[0]), "bad expert outputs")
+        b = _GroupSublayer(_ptr(y), _ptr(sub.gate), _ptr(sub.w_post), None if ex is None else _ptr(ex.pos), None if ex is None else _ptr(ex.weight),
+                           y.stride(0), sub.gate.stride(0), 0 if ex is None else ex.pos.shape[1], y.shape[0])
+    h = None if w is None else rows_buffer(rows, d, w.dtype, x.device)
+    _check(_lib().b200_group_step(_ptr(x), _ref(a), _ref(b), _ptr(row_index), _ptr(w), _ptr(h), 0 if h is None else h.stride(0), float(eps), rows,
+                                  x.shape[0], d, groups, _f32(act), _ptr(native.status_word(x.device)), _stream()), "group_step")
+    return h

@@ -80,10 +80,11 @@ def moe_plan(tokens, slots, tables, experts, tiles):
     return pos, groups
 
 
-def moe_route(z, correction, slots, experts, top, count, always):
-    outputs = correction.numel()
-    s = torch.softmax(z[:, :outputs], -1)
-    choice = torch.topk(s + correction, top, dim=-1).indices
+def moe_route(z, correction, slots, experts, top, count, always, bias):
+    outputs = z.shape[1] - (always > 0)
+    logits = z[:, :outputs] if bias is None else z[:, :outputs] + bias
+    s = torch.softmax(logits, -1)
+    choice = torch.topk(logits if correction is None else s + correction, top, dim=-1).indices
     weight = s.gather(1, choice)
     weight = weight / (weight.sum(-1, keepdim=True) + 1e-20)
     if always:
@@ -284,7 +285,7 @@ def attention_rows(q, s, cache, row_seq, positions, slots, tables, out, gate):
             out[r] = 0
             continue
         p = int(positions[r])
-        lo = max(0, p - s.window + 1)
+        lo = p - p % s.window if s.chunked else max(0, p - s.window + 1)
         j = torch.cat((torch.arange(min(s.keep, lo)), torch.arange(lo, p + 1)))
         line = tables[int(row_seq[r]) if row_seq is not None else r].long()
         c = flat[line[j // page] * page + j % page].float()
@@ -295,6 +296,8 @@ def attention_rows(q, s, cache, row_seq, positions, slots, tables, out, gate):
             score = s.softcap * torch.tanh(score / s.softcap)
         if s.bias is not None:
             score = score + s.bias[:, (p - j).clamp(max=s.bias.shape[1] - 1)][:, None]
+        if s.slopes is not None:
+            score = score - (s.slopes[:, None] * (p - j))[:, None]
         if s.sink is not None:
             score = torch.cat((score, s.sink.view(-1, 1, 1).expand(-1, s.maps, 1)), -1)
         o = torch.einsum("hmj,jhe->hme", torch.softmax(score, -1)[..., :len(j)], v)
@@ -303,6 +306,96 @@ def attention_rows(q, s, cache, row_seq, positions, slots, tables, out, gate):
             o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + s.eps) * s.out_scale
         o = o.reshape(-1)
         if gate is not None:
-            o = o * torch.sigmoid(gate[r].float())
+            o = o * torch.sigmoid(gate[r].float()).repeat_interleave(len(o) // gate.shape[1])
         out[r] = o.to(out.dtype)
     return out
+
+
+def short_conv(u, w, ring, at, silu):
+    taps, f, y = w.shape[0], u.float(), torch.zeros_like(u, dtype=torch.float32)
+    kept = ring.clone()
+    for seq, (a, b) in enumerate(at.spans):
+        slot = int(at.state_slots[seq])
+        for r in range(a, b):
+            pos = int(at.positions[r])
+            for d in range(taps):
+                if r - d >= a:
+                    y[r] += w[taps - 1 - d].float() * f[r - d]
+                elif pos >= d and slot >= 0:
+                    y[r] += w[taps - 1 - d].float() * kept[slot, (pos - d) % taps].float()
+            if slot >= 0:
+                ring[slot, pos % taps] = u[r]
+    return torch.nn.functional.silu(y).to(u.dtype) if silu else y.to(u.dtype)
+
+
+def conv_attend(u, w, ring, at, s, temp, cache, first, mix, q):
+    c = short_conv(u.float(), w.float(), ring, at, False)
+    nq, nk = s.heads * s.dim, s.kv_heads * s.dim
+    q.zero_().view(-1, s.heads, s.q_pitch)[..., :s.dim] = c[:, :nq].view(-1, s.heads, s.dim) * temp[:, None]
+    live = at.slots >= 0
+    v = c[:, nq + nk:].view(-1, s.kv_heads, s.vdim)
+    if first is not None:
+        vf = first.view(-1, first.shape[-1])[at.slots.clamp(min=0)][:, first.shape[-1] - s.kv_heads * s.v_pitch:]
+        v = (1.0 - mix) * v + mix * vf.reshape(-1, s.kv_heads, s.v_pitch)[..., :s.vdim].float()
+    row = torch.zeros((len(u), s.cache_width), dtype=cache.dtype)
+    row[:, :s.kv_heads * s.k_pitch].view(-1, s.kv_heads, s.k_pitch)[..., :s.dim] = c[:, nq:nq + nk].view(-1, s.kv_heads, s.dim).to(cache.dtype)
+    row[:, s.kv_heads * s.k_pitch:].view(-1, s.kv_heads, s.v_pitch)[..., :s.vdim] = v.to(cache.dtype)
+    cache.view(-1, s.cache_width)[at.slots[live]] = row[live]
+    return q
+
+
+def delta_rule(c, gate, ab, decay, dt, weight, state, at, kv_heads, eps, y):
+    _, heads, dim, vdim = state.shape
+    rep = lambda t: t.view(kv_heads, dim).repeat_interleave(heads // kv_heads, 0)
+    unit = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)
+    g, beta = torch.exp(decay * torch.nn.functional.softplus(ab[:, :heads] + dt)), torch.sigmoid(ab[:, heads:])
+    for seq, (a, b) in enumerate(at.spans):
+        slot = int(at.state_slots[seq])
+        if slot < 0:
+            y[a:b] = 0
+            continue
+        S = state[slot]
+        for r in range(a, b):
+            if int(at.positions[r]) == 0:
+                S.zero_()
+            row = c[r].float()
+            q, k = unit(rep(row[:kv_heads * dim])) * dim ** -0.5, unit(rep(row[kv_heads * dim:2 * kv_heads * dim]))
+            S.mul_(g[r][:, None, None])
+            u = beta[r][:, None] * (row[2 * kv_heads * dim:].view(heads, vdim) - torch.einsum("hde,hd->he", S, k))
+            S.add_(k[:, :, None] * u[:, None])
+            o = torch.einsum("hde,hd->he", S, q)
+            o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+            y[r] = (o.reshape(-1) * torch.nn.functional.silu(gate[r].float())).to(y.dtype)
+    return y
+
+
+def group_step(x, groups, eps, w, start, batch, sub, row_index):
+    def norm(t, weight):
+        parts = t.view(len(t), groups, -1)
+        return (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).view(t.shape) * weight.float()
+    pick = (lambda t: t) if row_index is None else (lambda t: t[row_index.long()])
+    src = pick(x)
+    if start is not None:
+        src = start.embed[batch.tokens].float() * start.scale
+        if start.bigram is not None:
+            buckets, seen = len(start.bigram) - 1, {}
+            for r in range(len(x)):
+                seq, tok = int(batch.row_seq[r]), int(batch.tokens[r])
+                slot = int(batch.state_slots[seq])
+                before = seen.get(seq, int(start.prev[slot]) if slot >= 0 else 0)
+                pair = buckets if int(batch.positions[r]) == 0 else (before * start.mul_prev + tok * start.mul_cur) % buckets
+                src[r] += start.bigram[pair].float()
+                seen[seq] = tok
+                if slot >= 0:
+                    start.prev[slot] = tok
+    if sub is not None:
+        if isinstance(sub.y, torch.Tensor):
+            u = pick(sub.y).float()
+        else:
+            pos = pick(sub.y.pos)
+            part = sub.y.y.float()[pos.clamp(min=0).long()].masked_fill((pos < 0).unsqueeze(-1), 0.0)
+            u = (part * pick(sub.y.weight).unsqueeze(-1)).sum(1)
+        src = src + norm(u * torch.sigmoid(pick(sub.gate).float()), sub.w_post)
+    if row_index is None:
+        x.copy_(src)
+    return None if w is None else norm(src, w).to(w.dtype)

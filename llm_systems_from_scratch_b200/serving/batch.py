@@ -57,6 +57,15 @@ class StepBatch:
             got = self._ranges[window] = (_to(cu, dev), _to(np.asarray(first, dtype=np.int32), dev), int(cu[-1]), max(lens))
         return got
 
+    def chunk_ranges(self, tokens: int):
+        """Chunks of ``tokens`` that the portions consist of: device offsets (portions + 1,) and their number.  Computed once per step."""
+        got = self._ranges.get(("chunks", tokens))
+        if got is None:
+            cu = np.zeros(len(self.portions) + 1, dtype=np.int32)
+            cu[1:] = np.cumsum([-(-n // tokens) for _, n in self.portions])
+            got = self._ranges["chunks", tokens] = (_to(cu, self.tokens.device), int(cu[-1]))
+        return got
+
     @classmethod
     def build(cls, entries, page_size: int, max_pages: int, device) -> "StepBatch":
         """``entries``: (request, start position, token ids); the requests' pages cover the tokens."""

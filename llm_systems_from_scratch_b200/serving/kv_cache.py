@@ -7,8 +7,9 @@ Memory: one K and one V tensor of shape (layers, num_pages, page_size, d_model) 
 of thousands of pages next to the 2.8 GB of weights.
 
 ``LayerCache`` is the same for models whose layers differ: every layer run says what it keeps per token
-(``PagedSpec``: one vector in a paged pool) or per request (``StateSpec``: a recurrent state in a slot), or that it
-reads what an earlier run keeps (``SharedSpec``).  All paged layers share the page ids of a request, all recurrent
+(``PagedSpec``: one vector in a paged pool) or per request (``StateSpec``: a recurrent state in a slot), that it
+reads what an earlier run keeps (``SharedSpec``), or several of these (``Parts``).  What a model keeps besides its layers follows
+behind them.  All paged layers share the page ids of a request, all recurrent
 layers its slot.
 """
 from __future__ import annotations
@@ -26,14 +27,28 @@ class PagedSpec:
 
 @dataclass(frozen=True)
 class StateSpec:
-    """A layer run that carries one fp32 state of this shape per request."""
+    """A state of this shape per request: "float32", in the type of the activations ("activations") or a number of tokens ("tokens")."""
     shape: tuple
+    kind: str = "float32"
 
 
 @dataclass(frozen=True)
 class SharedSpec:
     """A layer run that keeps nothing of its own and reads the entry of an earlier run."""
     run: int
+
+
+@dataclass(frozen=True)
+class Parts:
+    """A layer run that keeps several things; its entry is a tuple."""
+    specs: tuple
+
+
+def flatten(specs) -> list:
+    out = []
+    for s in specs:
+        out += flatten(s.specs) if isinstance(s, Parts) else [s]
+    return out
 
 
 class PageAllocator:
@@ -111,28 +126,31 @@ class LayerCache:
     def __init__(self, specs: list, num_pages: int, page_size: int, num_slots: int, device, dtype):
         self.specs, self.page_size, self.num_pages, self.num_slots = specs, page_size, num_pages, num_slots
         self.entries = []
-        for s in specs:
+        types = {"float32": torch.float32, "activations": dtype, "tokens": torch.int32}
+
+        def entry(s):
+            if isinstance(s, Parts):
+                return tuple(entry(p) for p in s.specs)
             if isinstance(s, PagedSpec):
-                self.entries.append(torch.zeros((num_pages, page_size, s.width), dtype=dtype, device=device))
-            elif isinstance(s, StateSpec):
-                self.entries.append(torch.zeros((num_slots, *s.shape), dtype=torch.float32, device=device))
-            elif isinstance(s, SharedSpec):
-                self.entries.append(self.entries[s.run])
-            else:
-                self.entries.append(None)
+                return torch.zeros((num_pages, page_size, s.width), dtype=dtype, device=device)
+            if isinstance(s, StateSpec):
+                return torch.zeros((num_slots, *s.shape), dtype=types[s.kind], device=device)
+            return self.entries[s.run] if isinstance(s, SharedSpec) else None
+        for s in specs:
+            self.entries.append(entry(s))
         self.allocator = PageAllocator(num_pages)
         self.slot_allocator = PageAllocator(num_slots)
 
     @staticmethod
     def bytes_per_page(specs: list, page_size: int, itemsize: int) -> int:
-        return sum(s.width for s in specs if isinstance(s, PagedSpec)) * page_size * itemsize
+        return sum(s.width for s in flatten(specs) if isinstance(s, PagedSpec)) * page_size * itemsize
 
     @staticmethod
-    def bytes_per_slot(specs: list) -> int:
+    def bytes_per_slot(specs: list, itemsize: int = 4) -> int:
         total = 0
-        for s in specs:
+        for s in flatten(specs):
             if isinstance(s, StateSpec):
-                n = 4
+                n = itemsize if s.kind == "activations" else 4
                 for k in s.shape:
                     n *= k
                 total += n
