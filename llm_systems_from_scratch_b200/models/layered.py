@@ -1,5 +1,5 @@
-"""What models made of listed layers have in common (``tedirax.py``, ``beledra.py``, ``genedra.py``): configuration checks, loading from a
-folder, random weights, generation through the serving engine.
+"""What models made of listed layers have in common (``tedirax.py``, ``beledra.py``, ``genedra.py``, ``vilosun.py``): configuration checks,
+loading from a folder, random weights, generation through the serving engine.
 
 A subclass reads its configuration, packs its weights into ``layers`` / ``runs`` (objects with a ``mixer`` from ``mixers.py``
 among others) and names the serving backend that knows its order of sublayers; caches, batches, scheduling and sampling
@@ -106,7 +106,7 @@ class RandomTensors:
         t = self.special(name, shape, kw) if self.special is not None else None
         if t is not None:
             return t
-        if len(shape) == 1:
+        if len(shape) <= 1:
             return (1.0 + 0.1 * torch.randn(shape, **kw)).to(torch.bfloat16)
         std = 1.0 if name == "embed" else shape[1] ** -0.5
         return (std * torch.randn(shape, **kw)).to(torch.bfloat16)

@@ -9,7 +9,8 @@ input become one product; heads are padded to what the kernels tile by) and runs
 * a feed-forward does the same, or returns outputs that the next pass over the residual stream adds (``ops.mixer_ops``:
   ``residual_norm``, ``add_normed``)
 
-What a sublayer adds to ``x`` it multiplies with its ``gain``.
+What a sublayer adds to ``x`` it multiplies with its ``gain``.  Designs that gate a sublayer's output before they norm it give the gate's
+weights to the sublayer (``out_gate``), where their product joins those of the same input; it then returns (output, gate).
 
 ``get(name)`` gives a weight in its stored layout ([out, in])."""
 from __future__ import annotations
@@ -19,7 +20,7 @@ import math
 import torch
 
 from ..ops import mixer_ops as mo
-from ..serving.kv_cache import PagedSpec, SharedSpec, StateSpec
+from ..serving.kv_cache import PagedSpec, Parts, SharedSpec, StateSpec
 
 
 def _head_pad(w, heads: int, rows: int, to: int):
@@ -49,6 +50,33 @@ def _align(n: int, to: int) -> int:
 def _row_pad(w, to: int):
     """Zero rows up to ``to``."""
     return w if w.shape[0] == to else torch.cat((w, torch.zeros((to - w.shape[0], w.shape[1]), dtype=w.dtype, device=w.device)))
+
+
+class InputProducts:
+    """Weights that read a sublayer's input, as one matrix: each part starts at a multiple of 8 columns (``at``), biases where there are any."""
+
+    def __init__(self, parts: dict, biases: dict, dtype, device):
+        rows, self.at, n = [], {}, 0
+        bias = torch.zeros(sum(_align(len(w), 8) for w in parts.values()), dtype=torch.float32)
+        for name, w in parts.items():
+            self.at[name] = slice(n, n + len(w))
+            if biases.get(name) is not None:
+                bias[n:n + len(w)] = biases[name].float()
+            rows.append(_row_pad(w, _align(len(w), 8)))
+            n += len(rows[-1])
+        self.w = mo.padded_weight(torch.cat(rows), dtype, device)
+        self.bias = bias.to(device) if any(b is not None for b in biases.values()) else None
+
+    def __call__(self, h):
+        return mo.linear(h, self.w, bias=self.bias)
+
+
+def conv_filter(get, names, sizes, taps: int, dtype, device):
+    """The filters of some projections, (channels, taps) each, as one matrix (taps, channels)."""
+    if taps < 1:
+        raise ValueError("a convolution has one tap at least")
+    both = torch.cat([_expect(n + ".conv", get(n + ".conv"), size, taps) for n, size in zip(names, sizes)])
+    return both.t().to(device=device, dtype=dtype).contiguous()
 
 
 class LatentAttention:
@@ -267,7 +295,12 @@ class GroupedAttention:
       logarithmic up to ``bias_max``
     * ``difference`` (with ``out_scale``): two maps per head over the same values (queries and keys have twice the rows, laid
       out head by head); the output is first map - difference * second map, RMS-normed per head, times ``out_scale``
-    * ``gated``: heads are multiplied by sigmoid(W_g h)
+    * ``gated``: heads are multiplied by sigmoid(W_g h), element by element, or with one number per head (``gated`` "heads")
+    * ``chunked``: a query sees the keys of its own chunk of ``window`` positions instead
+    * ``slopes``: slope_h * distance comes off the scaled scores
+    * ``conv`` (with ``norm`` None, no rotation): projections pass a short convolution of that many taps; then
+      * ``temp``: scores are multiplied by a number per head
+      * ``mix_from`` (an earlier layer run, or None): values are mixed with that run's of the same token by the weight ``vmix``
     * ``kv_from``: keys and values of that earlier layer run instead of its own
 
     The cache holds the normed, rotated keys and the values of a token as one vector, every head padded to 8 elements."""
@@ -275,33 +308,51 @@ class GroupedAttention:
     def __init__(self, get, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, eps: float,
                  dtype, device, bias_max: float | None = None, rope=None, rot_dims: int = 0, difference: float | None = None,
                  out_scale: float = 1.0, gated: bool = False, kv_from: int | None = None, keep: int = 0, softcap: float | None = None,
-                 sink: bool = False, biased: bool = False, norm: str = "head", gain: float = 1.0):
-        self.gated, self.kv_from, self.rope, self.gain = gated, kv_from, rope, float(gain)
+                 sink: bool = False, biased: bool | str = False, norm: str | None = "head", gain: float = 1.0, chunked: bool = False,
+                 slopes=None, conv: int = 0, temp: bool = False, mix_from: int | None = None, out_gate=None):
+        self.gated, self.kv_from, self.rope, self.gain = bool(gated), kv_from, rope, float(gain)
+        self.taps, self.mix_from, self.mix, self.gates_output = int(conv), mix_from, 0.0, out_gate is not None
         if heads % kv_heads:
             raise ValueError("the query heads must share the key heads evenly")
         if rot_dims % 2 or rot_dims > dim:
             raise ValueError("the rotated dimensions must be even in number and fit the head")
-        if norm not in ("head", "projection"):
+        if norm not in ("head", "projection", None):
             raise ValueError(f"unknown norm {norm!r}")
         maps = 1 if difference is None else 2
-        if maps == 2 and (sink or norm == "projection"):
-            raise ValueError("sinks and norms over a projection are those of a single map")
+        if maps == 2 and (sink or norm == "projection" or slopes is not None):
+            raise ValueError("sinks, slopes and norms over a projection are those of a single map")
+        if bool(conv) != (norm is None) or (conv and (maps == 2 or rot_dims or kv_from is not None)):
+            raise ValueError("projections are normed, or pass a convolution and are neither rotated nor shared")
+        if (temp or mix_from is not None) and not conv:
+            raise ValueError("factors of the scores and mixed values come with the convolution")
+        if (chunked and keep) or (slopes is not None and (softcap or bias_max is not None)):
+            raise ValueError("chunks keep no first tokens, and slopes go with neither caps nor tables")
         w = lambda name, *shape: _expect(name, get(name), *shape)
         rows = {"q": heads * maps * dim}
         if kv_from is None:
             rows.update({"k": kv_heads * maps * dim, "v": kv_heads * vdim})
+        qkv = torch.cat([w(name, n, width) for name, n in rows.items()])
+        parts, biases = {"qkv": qkv}, {}
         if gated:
-            rows["g"] = heads * vdim
-        self.w_in = mo.padded_weight(torch.cat([w(name, n, width) for name, n in rows.items()]), dtype, device)
-        self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
+            parts["g"] = w("g", heads if gated == "heads" else heads * vdim, width)
+        if out_gate is not None:
+            parts["out"], biases["out"] = out_gate
         f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
-        self.b_in = self.b_o = None
-        if biased:
-            none = lambda n: torch.zeros(n, dtype=get("q.b").dtype, device=get("q.b").device)
-            self.b_in = f32(torch.cat([none(n) if name == "g" else w(name + ".b", n) for name, n in rows.items()]))
-            self.b_o = f32(w("o.b", width))
-        vec = lambda name, n: w(name, dim if norm == "head" else n * dim).to(device=device, dtype=dtype).contiguous()
-        self.n_q, self.n_k = vec("q.norm", heads), vec("k.norm", kv_heads) if kv_from is None else None
+        self.b_o = None
+        if biased:                                       # "inputs": q, k and v alone
+            biases["qkv"] = torch.cat([w(name + ".b", n) for name, n in rows.items()])
+            self.b_o = f32(w("o.b", width)) if biased != "inputs" else None
+        self.inputs = InputProducts(parts, biases, dtype, device)
+        self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
+        if norm is not None:
+            vec = lambda name, n: w(name, dim if norm == "head" else n * dim).to(device=device, dtype=dtype).contiguous()
+            self.n_q, self.n_k = vec("q.norm", heads), vec("k.norm", kv_heads) if kv_from is None else None
+        if conv:
+            self.channels = len(qkv)
+            self.filter = conv_filter(get, rows, rows.values(), self.taps, dtype, device)
+            self.temp = f32(w("temp", heads)) if temp else torch.ones(heads, dtype=torch.float32, device=device)
+            if mix_from is not None:
+                self.mix = float(w("vmix"))
         bias = None
         if bias_max is not None:
             rel = get("rel")
@@ -310,19 +361,37 @@ class GroupedAttention:
             bias = distance_table(rel, bias_max, window).to(device)
         self.shape = mo.AttentionShape(heads, kv_heads, maps, dim, vdim, rot_dims, float(scale), int(window), float(eps),
                                        float(difference or 0.0), float(out_scale), bias, int(keep), float(softcap or 0.0),
-                                       f32(w("sink", heads)) if sink else None, norm == "projection")
+                                       f32(w("sink", heads)) if sink else None, norm == "projection",
+                                       None if slopes is None else torch.tensor(slopes, dtype=torch.float32, device=device), bool(chunked),
+                                       gated == "heads")
         self.tensor_cores = torch.device(device).type == "cuda" and mo.attention_tiles(self.shape, dtype)
 
     def cache_spec(self):
-        return PagedSpec(self.shape.cache_width) if self.kv_from is None else SharedSpec(self.kv_from)
+        own = PagedSpec(self.shape.cache_width)
+        if self.taps:
+            ring = StateSpec((self.taps, self.channels), "activations")
+            return Parts((own, ring) if self.mix_from is None else (own, ring, SharedSpec(self.mix_from)))
+        return own if self.kv_from is None else SharedSpec(self.kv_from)
+
+    def _convolved(self, u, batch, cache):
+        """Queries behind the convolution; keys and values are in the cache then.  -> queries, the paged pool"""
+        pool, ring, *first = cache
+        parts = mo.step_parts(batch)
+        q = [mo.conv_attend(u[rows], self.filter, ring, at, self.shape, self.temp, pool, first[0][0] if first else None, self.mix)
+             for rows, at in parts]
+        return q[0] if len(q) == 1 else torch.cat(q), pool
 
     def __call__(self, h, x, batch, cache):
         s, n = self.shape, batch.n_single
-        proj = mo.linear(h, self.w_in, bias=self.b_in)
-        q = mo.attention_prepare(proj, s, self.n_q, self.n_k, self.rope.table if self.rope is not None else None,
-                                 batch.positions, batch.slots, cache)
+        proj = self.inputs(h)
+        at = self.inputs.at
+        if self.taps:
+            q, cache = self._convolved(proj[:, at["qkv"]], batch, cache)
+        else:
+            q = mo.attention_prepare(proj, s, self.n_q, self.n_k, self.rope.table if self.rope is not None else None,
+                                     batch.positions, batch.slots, cache)
         o = mo.rows_buffer(h.shape[0], s.heads * s.vdim, h.dtype, h.device)
-        gate = proj[:, proj.shape[1] - s.heads * s.vdim:] if self.gated else None
+        gate = proj[:, at["g"]] if self.gated else None
         part = lambda rows: None if gate is None else gate[rows]
         if n:
             one = slice(0, n)
@@ -335,7 +404,59 @@ class GroupedAttention:
             else:
                 mo.attention_rows(q[rest], s, cache, batch.row_seq[rest], batch.positions[rest], batch.slots[rest],
                                   batch.tables, o[rest], part(rest))
-        return _project(o, self.w_o, x, self.gain, self.b_o)
+        y = _project(o, self.w_o, x, self.gain, self.b_o)
+        return (y, proj[:, at["out"]]) if self.gates_output else y
+
+
+class DeltaRule:
+    """Gated delta rule: per head S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with unit q (times dim^(-1/2)) and k shared by
+    heads / kv_heads heads, a decay g = exp(-exp(A_log) softplus(W_a h + dt_bias)) and beta = sigmoid(W_b h) per head.
+
+    Projections of q, k and v pass a short convolution of ``taps`` taps and silu; heads are divided by their root mean square, multiplied
+    by the weight ``norm`` and by silu(W_g h), then W_o.  S is fp32; a request's state slot holds it and the convolution's last inputs."""
+
+    MIN_CHUNKED = 8            # the longest portion of a step from which the chunked kernels are used
+
+    def __init__(self, get, width: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float, dtype, device, out_gate=None):
+        if heads % kv_heads:
+            raise ValueError("the heads must share the keys evenly")
+        self.heads, self.kv_heads, self.dim, self.vdim, self.eps = heads, kv_heads, dim, vdim, float(eps)
+        w = lambda name, *shape: _expect(name, get(name), *shape)
+        rows = {"q": kv_heads * dim, "k": kv_heads * dim, "v": heads * vdim}
+        parts = {"qkv": torch.cat([w(name, n, width) for name, n in rows.items()]), "g": w("g", heads * vdim, width)}
+        self.channels, self.gates_output, biases = len(parts["qkv"]), out_gate is not None, {}
+        if out_gate is not None:
+            parts["out"], biases["out"] = out_gate
+        self.inputs = InputProducts(parts, biases, dtype, device)
+        self.w_ab = mo.padded_weight(torch.cat((w("a", heads, width), w("b", heads, width))), dtype, device)
+        f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+        self.decay, self.dt = f32(-torch.exp(w("A_log", heads).double())), f32(w("dt_bias", heads))
+        self.norm = w("norm", vdim).to(device=device, dtype=dtype).contiguous()
+        self.filter = conv_filter(get, rows, rows.values(), taps, dtype, device)
+        self.w_o = mo.padded_weight(w("o", width, heads * vdim), dtype, device)
+        self.one_pass = mo.delta_steps(dim, vdim)          # a decode step takes the gates' products and the convolution itself
+        self.chunked = torch.device(device).type == "cuda" and mo.delta_chunkable(dtype, dim, vdim)
+
+    def cache_spec(self):
+        return Parts((StateSpec((self.heads, self.dim, self.vdim)), StateSpec((len(self.filter), self.channels), "activations")))
+
+    def __call__(self, h, x, batch, cache):
+        state, ring = cache
+        proj = self.inputs(h)
+        at = self.inputs.at
+        u, gate = proj[:, at["qkv"]], proj[:, at["g"]]
+        y = mo.rows_buffer(h.shape[0], self.heads * self.vdim, h.dtype, h.device)
+        for rows, part in mo.step_parts(batch):
+            run = lambda c, ab, **kw: mo.delta_rule(c, gate[rows], ab, self.decay, self.dt, self.norm, state, part, self.kv_heads, self.eps, y[rows], **kw)
+            if part.cu is None and self.one_pass:
+                run(u[rows], (h[rows], self.w_ab), conv=(self.filter, ring))
+                continue
+            ab = mo.linear(h[rows], self.w_ab, out_dtype=torch.float32)        # the recurrence takes the gates in 32-bit
+            c = mo.short_conv(u[rows], self.filter, ring, part, mo.rows_buffer(len(part.positions), self.channels, h.dtype, h.device), silu=True)
+            chunks = part.cu is not None and self.chunked and batch.max_portion >= self.MIN_CHUNKED
+            run(c, ab, chunks=batch.chunk_ranges(mo.DELTA_CHUNK) if chunks else None)
+        out = _project(y, self.w_o, x)
+        return (out, proj[:, at["out"]]) if self.gates_output else out
 
 
 def distance_bucket(n: int, rows: int, far: float) -> int:
@@ -429,9 +550,10 @@ class TableExperts:
 
 
 class RoutedExperts:
-    """Experts W_down gelu(W_up h) chosen by a learned router.
+    """Experts chosen by a learned router: W_down gelu(W_up h), or, ``gated``, W_down (silu(W_gate h) * (W_up h)).
 
-    The router's softmax runs over ``experts`` + ``identity`` outputs; the last ``identity`` of them stand for h itself.  The ``top``
+    ``choice`` "logits": the ``top`` outputs with the largest logits (plus ``router.b``) are chosen, their weights are the softmax over the
+    chosen logits.  "corrected": the router's softmax runs over ``experts`` + ``identity`` outputs; the last ``identity`` of them stand for h itself.  The ``top``
     outputs with the largest score + ``correction`` are chosen and weighted by their share of the chosen scores.  ``shared``: rows of
     an expert that every token uses, times sigmoid of one number per token (``shared.sg``, a row of the router's product).
 
@@ -442,15 +564,21 @@ class RoutedExperts:
     FOLD_ROWS = 256            # the largest step in which the shared expert joins the others
 
     def __init__(self, get, width: int, ff: int, experts: int, top: int, identity: int, shared: int | None, dtype, device,
-                 gain: float = 1.0):
+                 gain: float = 1.0, gated: bool = False, choice: str = "corrected", out_gate=None):
         if not 0 < top <= experts + identity:
             raise ValueError(f"{top} of {experts + identity} outputs cannot be chosen")
+        if choice not in ("corrected", "logits"):
+            raise ValueError(f"unknown choice {choice!r}")
+        if gated and shared is not None:
+            raise ValueError("a shared expert is not gated")
+        self.gated, self.gate = gated, None if out_gate is None else InputProducts({"out": out_gate[0]}, {"out": out_gate[1]}, dtype, device)
         self.width, self.ff, self.experts, self.top, self.identity, self.gain = width, ff, experts, top, identity, float(gain)
         w = lambda name, *shape: _expect(name, get(name), *shape)
         pack = lambda *ts: mo.padded_weight(torch.cat(ts), dtype, device)
         self.shared = shared is not None
         self.folds = shared // ff if self.shared and shared % ff == 0 else 0          # pieces of the shared expert among the others
-        router, up = [w("router", experts + identity, width)], [w(f"e{e}.up", ff, width) for e in range(experts)]
+        router = [w("router", experts + identity, width)]
+        up = [w(f"e{e}.{k}", ff, width) for e in range(experts) for k in (("gate", "up") if gated else ("up",))]
         down = [w(f"e{e}.down", width, ff) for e in range(experts)]
         if self.shared:
             router.append(w("shared.sg", 1, width))
@@ -461,7 +589,8 @@ class RoutedExperts:
         if self.shared:
             self.w_shared_up = self.w_up[experts * ff:] if self.folds else pack(s_up)
             self.w_shared_down = self.w_down[experts * width:] if self.folds == 1 else pack(s_down)
-        self.correction = w("correction", experts + identity).to(device=device, dtype=torch.float32).contiguous()
+        f32 = lambda name: w(name, experts + identity).to(device=device, dtype=torch.float32).contiguous()
+        self.correction, self.bias = (f32("correction"), None) if choice == "corrected" else (None, f32("router.b"))
 
     def __call__(self, h, slots, count):
         """``count``: (experts,) int32 of zeros."""
@@ -469,12 +598,16 @@ class RoutedExperts:
         fold = self.folds if rows <= self.FOLD_ROWS else 0
         cols = outputs + (fold > 0)
         if mo.routes_rows(rows, self.w_router):
-            z, choice, rank, weight = mo.moe_route_rows(h, self.w_router, self.correction, slots, self.experts, self.top, count, fold)
+            z, choice, rank, weight = mo.moe_route_rows(h, self.w_router, self.correction, slots, self.experts, self.top, count, fold,
+                                                        self.bias)
         else:
             z = mo.linear(h, self.w_router, out_dtype=torch.float32)               # what is routed by is 32-bit
-            choice, rank, weight = mo.moe_route(z[:, :cols], self.correction, slots, self.experts, self.top, count, fold)
+            choice, rank, weight = mo.moe_route(z[:, :cols], self.correction, slots, self.experts, self.top, count, fold, self.bias)
         xg, pos, groups = mo.moe_dispatch(h, choice, rank, count, fold)
-        y = mo.gemm_rows(mo.gemm_rows(xg, self.w_up, groups, self.ff, False, "gelu"), self.w_down, groups, self.width, False)
+        y = mo.gemm_rows(mo.gemm_rows(xg, self.w_up, groups, self.ff, self.gated, None if self.gated else "gelu"), self.w_down, groups, self.width,
+                         False)
+        if self.gate is not None:
+            return mo.ExpertOutputs(y, pos, self.gain, weight, h if self.identity else None), self.gate(h)[:, self.gate.at["out"]]
         if fold or not self.shared:
             return mo.ExpertOutputs(y, pos, self.gain, weight, h)
         s = mo.linear(mo.linear(h, self.w_shared_up, act="gelu"), self.w_shared_down)

@@ -13,8 +13,9 @@ from .beledra import Beledra
 from .genedra import Genedra
 from .tedirax import Tedirax
 from .transformer import TransformerLM
+from .vilosun import Vilosun
 
-MODELS = {"TransformerLM": TransformerLM, "Tedirax": Tedirax, "Beledra": Beledra, "Genedra": Genedra}
+MODELS = {"TransformerLM": TransformerLM, "Tedirax": Tedirax, "Beledra": Beledra, "Genedra": Genedra, "Vilosun": Vilosun}
 
 
 def model_class(config: dict):

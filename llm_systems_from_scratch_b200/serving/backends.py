@@ -12,7 +12,7 @@ import torch
 from .. import ops
 from ..ops import mixer_ops as mo
 from ..ops import serving_ops
-from .kv_cache import LayerCache, PagedKVCache
+from .kv_cache import LayerCache, PagedKVCache, StateSpec
 
 
 class TransformerBackend:
@@ -130,10 +130,10 @@ class LayeredBackend:
         batch.gathered.clear()
         return torch.empty((batch.n_rows, self.model.config.width), dtype=torch.float32, device=self.device)
 
-    def head(self, h, cap: float | None = None):
-        """(rows, vocabulary) fp32 of normed rows; ``cap``: capped softly."""
+    def head(self, h, cap: float | None = None, scale: float = 1.0):
+        """(rows, vocabulary) fp32 of normed rows, times ``scale``; ``cap``: capped softly."""
         out = torch.empty((h.shape[0], mo.pitch(self.vocab)), dtype=torch.float32, device=self.device)
-        mo.linear(h, self.model.head, out=out[:, :self.vocab], act="cap" if cap else None, cap=cap or 0.0)
+        mo.linear(h, self.model.head, out=out[:, :self.vocab], alpha=scale, act="cap" if cap else None, cap=cap or 0.0)
         return out
 
 
@@ -255,6 +255,47 @@ class PreNormLayers(LayeredBackend):
         m = self.model
         h, _ = mo.residual_norm(x, m.final_norm, m.config.eps, row_index=rows, pending=pending, w_offset=1.0)
         return self.head(h, m.config.logit_softcap)
+
+
+class SandwichLayers(LayeredBackend):
+    """Sublayers one after the other, each reading a group norm of the residual stream; its output is multiplied by a gate of the same input
+    and normed before it is added (``models/vilosun.py``).  The pass that adds a sublayer's output also writes the next one's input; the last
+    one belongs to the logits.  The embedding of token pairs keeps every request's last token in its state slot."""
+
+    def __init__(self, model):
+        super().__init__(model)
+        self.counters = [layer.mlp.experts for layer in model.layers if layer.mlp is not None]
+        self.specs = [*self.specs, StateSpec((1,), "tokens")]
+
+    def forward(self, batch, trace=None):
+        """``trace``: a list that receives the residual stream after every layer run (a copy; for tests)."""
+        m, cfg = self.model, self.model.config
+        x = self.stream(batch)
+        counts = None
+        if self.counters:
+            counts = iter(torch.zeros(sum(self.counters), dtype=torch.int32, device=self.device).split(self.counters))
+        step = lambda w, **kw: mo.group_step(x, cfg.groups, cfg.eps, w, **kw)
+        start = mo.EmbeddingStart(m.embed, cfg.embed_scale, m.bigram, cfg.mul_prev, cfg.mul_cur, self.cache.entries[-1])
+        h, pending = step(m.runs[0].norm1 if m.runs else None, start=start, batch=batch), None
+        for run, layer in enumerate(m.runs):
+            if pending is not None:
+                h = step(layer.norm1, sub=pending)
+            pending = mo.GatedOutput(*layer.mixer(h, None, batch, self.cache.entries[run]), layer.norm1b)
+            if layer.mlp is not None:
+                h = step(layer.norm2, sub=pending)
+                pending = mo.GatedOutput(*layer.mlp(h, batch.slots, next(counts)), layer.norm2b)
+            if trace is not None:
+                after = m.runs[run + 1].norm1 if run + 1 < len(m.runs) else None
+                h, pending = step(after, sub=pending), None
+                trace.append(x.clone())
+        return x, pending
+
+    def logits(self, hidden, rows=None):
+        """(rows, vocabulary) fp32."""
+        x, pending = hidden
+        cfg = self.model.config
+        h = mo.group_step(x, cfg.groups, cfg.eps, self.model.final_norm, sub=pending, row_index=rows)
+        return self.head(h, scale=cfg.logit_scale)
 
 
 def wanted_index(rows: np.ndarray, device) -> torch.Tensor:
