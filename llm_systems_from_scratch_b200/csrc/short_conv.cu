@@ -71,13 +71,13 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const ConvParams p) {
   for (int row = r0; row < r1; ++row) {
     const int seq = p.row_seq != nullptr ? p.row_seq[row] - p.seq0 : row;
     if ((unsigned)seq >= (unsigned)p.seqs) {
-      if (threadIdx.x == 0) report_bad_arg(p.status, 30);
+      report_bad_arg(p.status, 30);
       continue;
     }
     const int first = p.cu != nullptr ? p.cu[seq] : row, pos = p.positions[row];
     int slot = p.state_slots[seq];
     if (slot >= p.num_slots) {
-      if (threadIdx.x == 0) report_bad_arg(p.status, 31);
+      report_bad_arg(p.status, 31);
       slot = -1;
     }
     T* ring = reinterpret_cast<T*>(p.ring) + (long long)max(slot, 0) * taps * p.channels + c;
@@ -140,7 +140,7 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const ConvParams p) {
       const long long to = p.slots[row];
       if (to < 0) continue;                              // padding row of the batch
       if (to >= p.cache_slots) {
-        if (threadIdx.x == 0) report_bad_arg(p.status, 32);
+        report_bad_arg(p.status, 32);
         continue;
       }
       T* line = reinterpret_cast<T*>(p.cache) + to * (long long)(s.kv_heads * (s.kp + s.vp));
