@@ -30,7 +30,7 @@ version of the same measurement (``--serving-requests`` requests, 0 switches it 
 engine; its arm replays the head of the same trace through its ``TransformerLM`` with a per-request greedy
 loop that re-runs the whole context for every token (what its ``generate`` does) for a bounded time.
 
-    python bench.py --workload layers [--layers-model Tedirax|Beledra|Genedra] [--layers-sizes 0.35b,1.3b,7b-8layers]
+    python bench.py --workload layers [--layers-model Tedirax|Beledra|Genedra|Vilosun] [--layers-sizes 0.35b,1.3b,7b-8layers]
 
 times a layered decoder beside the TransformerLM (and the layered ones before it) at equal size on one GPU: whole prompt and
 decode steps and every kernel against its roofline, one line per size (``ops/bench_layers.py``, ``ops/bench_beledra.py``,
@@ -146,7 +146,7 @@ def parse_args():
                     help="train (default) and serve: the headline metric; layers: a layered decoder beside the "
                          "TransformerLM at equal size, prompt and decode steps and every kernel, 1 GPU")
     ap.add_argument("--layers-sizes", default="0.35b,1.3b,7b-8layers", help="layers: sizes to run, with commas between them")
-    ap.add_argument("--layers-model", choices=["Tedirax", "Beledra", "Genedra"], default="Tedirax",
+    ap.add_argument("--layers-model", choices=["Tedirax", "Beledra", "Genedra", "Vilosun"], default="Tedirax",
                     help="layers: which layered decoder (Beledra: beside Tedirax and the TransformerLM; Genedra: beside all three)")
     ap.add_argument("--no-kernels", action="store_true", help="layers: whole steps only")
     ap.add_argument("--serving-requests", type=int, default=None,

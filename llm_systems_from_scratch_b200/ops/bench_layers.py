@@ -64,6 +64,9 @@ def build(kind: str, s: dict):
     if kind == "Genedra":
         from .bench_genedra import genedra_config
         return build_model(genedra_config(s))
+    if kind == "Vilosun":
+        from .bench_vilosun import vilosun_config
+        return build_model(vilosun_config(s))
     return build_model(dict(vocab_size=s["vocab"], context_length=4096, d_model=s["width"], num_layers=s["runs"],
                             num_heads=s["heads"], d_ff=s["ff"], rope_theta=10000.0))
 
@@ -377,7 +380,7 @@ def _decode_kernels(s, t, b):
 
 
 def run(sizes, steps: int = 10, warmup: int = 3, per_kernel: bool = True, model: str = "Tedirax"):
-    """One record per size: Tedirax beside the TransformerLM, Beledra beside both, or Genedra beside all three."""
+    """One record per size: Tedirax beside the TransformerLM, Beledra beside both, Genedra or Vilosun beside the models before it."""
     for size in sizes:
         if model == "Beledra":
             from . import bench_beledra
@@ -387,6 +390,10 @@ def run(sizes, steps: int = 10, warmup: int = 3, per_kernel: bool = True, model:
             from . import bench_genedra
             rec = models(size, steps, warmup, ("Genedra", "Tedirax", "Beledra", "TransformerLM"))
             more = bench_genedra.kernels
+        elif model == "Vilosun":
+            from . import bench_vilosun
+            rec = models(size, steps, warmup, ("Vilosun", "Tedirax", "Beledra", "Genedra", "TransformerLM"))
+            more = bench_vilosun.kernels
         else:
             rec, more = models(size, steps, warmup), kernels
         if per_kernel:
