@@ -308,8 +308,8 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) delta_step_kernel(const D
 //     u_t + sum_(s < t) A_ts u_s = beta_t (v_t - exp(b_t) S^T k_t),      A_ts = beta_t exp(b_t - b_s) k_t . k_s
 // and o_t = exp(b_t) S^T q_t + sum_(s <= t) P_ts u_s with P_ts = exp(b_t - b_s) q_t . k_s,  S <- exp(b_n) S + sum_s exp(b_n - b_s) k_s u_s^T.
 // Every exponent is at most zero.  T = (I + A)^-1 does not depend on S:
-//   delta_prepare   all chunks at once, one CTA each: scores of [K; Q] and K on tcgen05, T by forward substitution in fp32 (a thread per
-//                   column), T and P split into two bf16 parts (hi + lo, 16 significant bits), the per-token factors: an image of 33 KB
+//   delta_prepare   all chunks at once, one CTA each: scores of [K; Q] and K on tcgen05, T in fp32 by forward substitution of its diagonal
+//                   blocks and products, T and P split into two bf16 parts (hi + lo, 16 significant bits), the per-token factors: an image of 33 KB
 //                   that the second kernel copies as it is
 //   delta_chunk     one CTA per (portion, head), chunks in order, everything transposed so that a lane of tensor memory is a column of v:
 //                     [S^T K^T | S^T Q^T]  ->  R = beta (V - ...)^T  ->  U^T = R T^T  ->  S^T = exp(b_n) S^T + W K,  P U  (W: U with its factors)
@@ -325,6 +325,11 @@ __device__ __forceinline__ float dl_exp2(float x) {       // x <= 0
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float dl_sigmoid(float g) {    // (1 + tanh(g / 2)) / 2
+  float t;
+  asm("tanh.approx.f32 %0, %1;" : "=f"(t) : "f"(0.5f * g));
+  return fmaf(0.5f, t, 0.5f);
+}
 // Two values as hi + lo, both bf16: hi is cut off (the remainder is exact), lo rounded.
 __device__ __forceinline__ void dl_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
   const uint32_t a = __float_as_uint(x), b = __float_as_uint(y);
@@ -333,10 +338,10 @@ __device__ __forceinline__ void dl_split2(float x, float y, uint32_t& hi, uint32
 }
 __device__ __forceinline__ uint32_t dl_swz(int r, int c8) { return (uint32_t)r * 128u + (uint32_t)((c8 ^ (r & 7)) << 4); }
 
-struct DeltaPrepareSmem {                           // X: panels of [64 rows of K; 64 rows of Q] x 64 columns
-  static constexpr int OFF_X = 0, OFF_I = 32768;
+struct DeltaPrepareSmem {                           // X: panels of [64 rows of K; 64 rows of Q] x 64 columns, later the image
+  static constexpr int OFF_X = 0, OFF_I = 0;
   static constexpr int PITCH = 68;                  // floats between the rows of A
-  static constexpr int OFF_A = OFF_I + (DI_BYTES + 1023) / 1024 * 1024;
+  static constexpr int OFF_A = (DI_BYTES + 1023) / 1024 * 1024;
   static constexpr int OFF_F = OFF_A + DC * PITCH * 4;       // b [64], beta [64], inverse lengths [128]
   static constexpr int OFF_BAR = OFF_F + 4 * DC * 4;
   static constexpr int TOTAL = OFF_BAR + 2 * 8 + 16 + 1024;
@@ -468,29 +473,27 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
   }
   tc_fence_before();
   __syncthreads();
+  // ---- T by halves of 32: the diagonal blocks by forward substitution, a thread per column, then T21 = -T22 (A21 T11)
+  constexpr int HB = DC / 2;
   if (r < DC) {
-    // ---- column r of T: x_t = (t == r) - sum_(s < t) A_ts x_s
-    float x[DC];
+    const int c = r & (HB - 1), o = (r / HB) * HB;
+    float x[HB];
 #pragma unroll
-    for (int i = 0; i < DC; ++i) {
+    for (int i = 0; i < HB; ++i) {
       float a[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int s = 0; s < i; s += 4) {
-        const float4 v = *reinterpret_cast<const float4*>(A + i * L::PITCH + s);
+        const float4 v = *reinterpret_cast<const float4*>(A + (o + i) * L::PITCH + o + s);
         a[0] = fmaf(v.x, x[s], a[0]);
         if (s + 1 < i) a[1] = fmaf(v.y, x[s + 1], a[1]);
         if (s + 2 < i) a[2] = fmaf(v.z, x[s + 2], a[2]);
         if (s + 3 < i) a[3] = fmaf(v.w, x[s + 3], a[3]);
       }
-      x[i] = (i == r ? 1.f : 0.f) - ((a[0] + a[1]) + (a[2] + a[3]));
+      x[i] = (i == c ? 1.f : 0.f) - ((a[0] + a[1]) + (a[2] + a[3]));
     }
+    __syncwarp();                                   // the block has been read
 #pragma unroll
-    for (int i = 0; i < DC; ++i) {
-      const uint32_t u = __float_as_uint(x[i]);
-      const uint32_t at = dl_swz(i, r >> 3) + (r & 7) * 2;
-      *reinterpret_cast<uint16_t*>(image + DI_T + at) = (uint16_t)(u >> 16);
-      *reinterpret_cast<__nv_bfloat16*>(image + DI_T + DC_TILE + at) = __float2bfloat16(x[i] - __uint_as_float(u & 0xffff0000u));
-    }
+    for (int i = 0; i < HB; ++i) A[(o + i) * L::PITCH + o + c] = x[i];
   } else {
     float* f = reinterpret_cast<float*>(image + DI_F);
     const float end = sb[DC - 1], grown = dl_exp2(bt);
@@ -499,6 +502,47 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
     f[2 * DC + t] = dl_exp2(end - bt) * slen[t];    // of u_t where it joins the state
     f[3 * DC + t] = grown * slen[r];                // of S^T q_t
     if (t == 0) f[4 * DC] = dl_exp2(end);
+  }
+  __syncthreads();
+  // rows warp * 8 .. + 7 and column `lane` of L R, where L's rows start at l and R's at rt
+  auto product = [&](const float* l, const float* rt, float (&acc)[8]) __attribute__((always_inline)) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+#pragma unroll
+    for (int s = 0; s < HB; s += 4) {
+      float v[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] = rt[(s + j) * L::PITCH + lane];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float4 w = *reinterpret_cast<const float4*>(l + (warp * 8 + i) * L::PITCH + s);
+        acc[i] = fmaf(w.x, v[0], fmaf(w.y, v[1], fmaf(w.z, v[2], fmaf(w.w, v[3], acc[i]))));
+      }
+    }
+  };
+  float acc[8];
+  product(A + HB * L::PITCH, A, acc);               // A21 T11, kept above the diagonal
+#pragma unroll
+  for (int i = 0; i < 8; ++i) A[(warp * 8 + i) * L::PITCH + HB + lane] = acc[i];
+  __syncthreads();
+  product(A + HB * L::PITCH + HB, A + HB, acc);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) A[(HB + warp * 8 + i) * L::PITCH + lane] = -acc[i];
+  __syncthreads();
+  {
+    const int row = r >> 1, half = r & 1;
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const float4 u = *reinterpret_cast<const float4*>(A + row * L::PITCH + half * 32 + q * 8), v = *reinterpret_cast<const float4*>(A + row * L::PITCH + half * 32 + q * 8 + 4);
+      const bool zero = row < HB && half == 1;      // above the diagonal
+      uint4 hi4, lo4;
+      dl_split2(zero ? 0.f : u.x, zero ? 0.f : u.y, hi4.x, lo4.x);
+      dl_split2(zero ? 0.f : u.z, zero ? 0.f : u.w, hi4.y, lo4.y);
+      dl_split2(zero ? 0.f : v.x, zero ? 0.f : v.y, hi4.z, lo4.z);
+      dl_split2(zero ? 0.f : v.z, zero ? 0.f : v.w, hi4.w, lo4.w);
+      *reinterpret_cast<uint4*>(image + DI_T + dl_swz(row, half * 4 + q)) = hi4;
+      *reinterpret_cast<uint4*>(image + DI_T + DC_TILE + dl_swz(row, half * 4 + q)) = lo4;
+    }
   }
   fence_proxy_async_smem();
   __syncthreads();
@@ -517,20 +561,22 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
   }
 }
 
-// Warps 0 - 7: the chain R, U, S (a lane of tensor memory and half of the columns per thread); 8 - 11: outputs; 12: copies; 13: products.
-constexpr int DK_THREADS = 448;
+// Warps 0 - 7: the chain R, U, S (a lane of tensor memory and half of the columns per thread); 8 - 15: outputs; 16: copies; 17: products.
+constexpr int DK_CHAIN = 8, DK_OUT = 8, DK_THREADS = (DK_CHAIN + DK_OUT + 2) * 32;
 
 template <int PD, int PE>                            // panels of 64 columns of q and k, and of v
 struct DeltaChunkSmem {
   static constexpr int X = PD * 16384, V = PE * DC_TILE, I = (DI_BYTES + 1023) / 1024 * 1024, STAGE = X + V + I;
   static constexpr int OFF_O = 2 * STAGE;            // [64][PE * 64] floats
-  static constexpr int OFF_BAR = OFF_O + DC * PE * 64 * 4;
-  static constexpr int NUM_BARS = 12;
+  static constexpr int OFF_G = OFF_O + DC * PE * 64 * 4;       // output gates
+  static constexpr int OFF_BAR = OFF_G + PE * DC_TILE;
+  static constexpr int NUM_BARS = 14;
   static constexpr int TOTAL = OFF_BAR + NUM_BARS * 8 + 16 + 1024;
 };
 
 template <int PD, int PE>
-__global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid_constant__ CUtensorMap tm, const DeltaArgs p) {
+__global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid_constant__ CUtensorMap tm,
+                                                                     const __grid_constant__ CUtensorMap tm_gate, const DeltaArgs p) {
   using L = DeltaChunkSmem<PD, PE>;
   extern __shared__ uint8_t dl_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dl_raw) + 1023) & ~uintptr_t(1023));
@@ -538,28 +584,30 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
   uint64_t *full = bars, *empty = bars + 2;          // [2] per stage
   uint64_t *s_ready = bars + 4, *d1_full = bars + 5, *r_ready = bars + 6, *d2_full = bars + 7, *u_ready = bars + 8, *s_full = bars + 9,
            *o_full = bars + 10;
-  uint64_t* o_read = bars + 11;
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 12);
+  uint64_t *o_read = bars + 11, *g_full = bars + 12, *g_empty = bars + 13;
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + L::NUM_BARS);
   volatile uint32_t* abort_word = tmem_holder + 1;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0) {
     for (int i = 0; i < 2; ++i) {
       mbar_init(&full[i], 1);
-      mbar_init(&empty[i], 1 + 8 + 4);
+      mbar_init(&empty[i], 1 + DK_CHAIN + DK_OUT);
     }
-    mbar_init(s_ready, 256);
+    mbar_init(s_ready, DK_CHAIN * 32);
     mbar_init(d1_full, 1);
-    mbar_init(r_ready, 256);
+    mbar_init(r_ready, DK_CHAIN * 32);
     mbar_init(d2_full, 1);
-    mbar_init(u_ready, 256);
+    mbar_init(u_ready, DK_CHAIN * 32);
     mbar_init(s_full, 1);
     mbar_init(o_full, 1);
-    mbar_init(o_read, 128);
+    mbar_init(o_read, DK_OUT * 32);
+    mbar_init(g_full, 1);
+    mbar_init(g_empty, DK_OUT);
     *abort_word = 0;
     fence_barrier_init();
     prefetch_tensormap(&tm);
   }
-  if (warp == 13) {
+  if (warp == DK_CHAIN + DK_OUT + 1) {
     tmem_alloc(tmem_holder, 512);
     tmem_relinquish();
   }
@@ -576,13 +624,13 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_holder;
-  // columns: [S^T K^T, later U, later P U | S^T Q^T] 0 - 127, S^T 128 - 255, its parts 256, 320, R's then U's parts 384, 416, W's 448, 480
-  const uint32_t T_D = tmem, T_S = tmem + 128, T_SH = tmem + 256, T_SL = tmem + 320, T_RH = tmem + 384, T_RL = tmem + 416, T_WH = tmem + 448,
-                 T_WL = tmem + 480;
+  // columns: [S^T K^T, later U, later P U | S^T Q^T] 0 - 127, S^T 128 - 255, its parts 256 - 383, R's then U's parts 384 - 447, W's 448 - 511.
+  // Parts lie as a warp stores them: the hi, then the lo halves of 16 columns (tokens or dims), one k-step of a product.
+  const uint32_t T_D = tmem, T_S = tmem + 128, T_SP = tmem + 256, T_R = tmem + 384, T_W = tmem + 448;
   const int ksteps = (D + 15) / 16;
   bool ok = true;
 
-  if (warp == 12) {
+  if (warp == DK_CHAIN + DK_OUT) {
     if (chunks > 0 && elect_one()) {
       const int pd = (D + 63) / 64, pe = (E + 63) / 64;
       for (int ch = 0; ch < chunks; ++ch) {
@@ -602,7 +650,7 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
                   &full[st]);
       }
     }
-  } else if (warp == 13) {
+  } else if (warp == DK_CHAIN + DK_OUT + 1) {
     if (chunks > 0 && elect_one()) {
       constexpr uint32_t id_x = make_idesc_bf16(128, 128, false, false), id_t = make_idesc_bf16(128, DC, false, false);
       const uint32_t id_k = make_idesc_bf16(128, ksteps * 16, false, true);
@@ -620,7 +668,7 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
 #pragma unroll
         for (int part = 0; part < 2; ++part)
           for (int k = 0; k < ksteps; ++k)
-            umma_f16_ts(T_D, (part ? T_SL : T_SH) + k * 8, x + (uint32_t)(((k / 4) * 16384 + (k % 4) * 32) >> 4), id_x, (part | k) ? 1u : 0u);
+            umma_f16_ts(T_D, T_SP + k * 16 + part * 8, x + (uint32_t)(((k / 4) * 16384 + (k % 4) * 32) >> 4), id_x, (part | k) ? 1u : 0u);
         umma_commit(d1_full);
         ok = mbar_wait(r_ready, ph, abort_word);
         if (!ok) break;
@@ -629,7 +677,7 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
         for (int part = 0; part < 3; ++part)         // hi hi, hi lo, lo hi
 #pragma unroll
           for (int k = 0; k < 4; ++k)
-            umma_f16_ts(T_D, (part == 2 ? T_RL : T_RH) + k * 8, (part == 1 ? tl : th) + (uint32_t)(k * 2), id_t, (part | k) ? 1u : 0u);
+            umma_f16_ts(T_D, T_R + k * 16 + (part == 2 ? 8 : 0), (part == 1 ? tl : th) + (uint32_t)(k * 2), id_t, (part | k) ? 1u : 0u);
         umma_commit(d2_full);
         ok = mbar_wait(u_ready, ph, abort_word);
         if (!ok) break;
@@ -637,187 +685,211 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
 #pragma unroll
         for (int part = 0; part < 2; ++part)
 #pragma unroll
-          for (int k = 0; k < 4; ++k) umma_f16_ts(T_S, (part ? T_WL : T_WH) + k * 8, kt + (uint32_t)(k * 128), id_k, 1u);
+          for (int k = 0; k < 4; ++k) umma_f16_ts(T_S, T_W + k * 16 + part * 8, kt + (uint32_t)(k * 128), id_k, 1u);
         umma_commit(s_full);
 #pragma unroll
         for (int part = 0; part < 3; ++part)
 #pragma unroll
           for (int k = 0; k < 4; ++k)
-            umma_f16_ts(T_D, (part == 2 ? T_RL : T_RH) + k * 8, (part == 1 ? pl : ph_) + (uint32_t)(k * 2), id_t, (part | k) ? 1u : 0u);
+            umma_f16_ts(T_D, T_R + k * 16 + (part == 2 ? 8 : 0), (part == 1 ? pl : ph_) + (uint32_t)(k * 2), id_t, (part | k) ? 1u : 0u);
         umma_commit(o_full);
         umma_commit(&empty[st]);
       }
       if (!ok) *abort_word = ERR_WAIT_TMEM_FULL;
     }
-  } else if (warp < 8) {
-    const int quarter = warp & 3, half = warp >> 2, e = quarter * 32 + lane;      // this thread's column of v; half of the tokens or dims
+  } else if (warp < DK_CHAIN) {
+    const int quarter = warp & 3, cg = warp >> 2, e = quarter * 32 + lane;        // this thread's column of v; half of the tokens or dims
     const uint32_t la = uint32_t(quarter * 32) << 16;
-    constexpr int HD = PD * 32;                      // dims of S a thread looks after
-    // 32 dims of S: the parts into operand places, times the chunk's decay into the accumulator
-    auto publish = [&](const uint32_t (&raw)[32], int d0, float g) __attribute__((always_inline)) {
-      uint32_t hi[16], lo[16], scaled[32];
+    constexpr int HD = PD * 64 / (DK_CHAIN / 4), HT = DC / (DK_CHAIN / 4);        // dims of S and tokens a thread looks after
+    // 16 dims of S: the parts into operand places, times the chunk's decay into the accumulator
+    auto publish = [&](uint32_t (&raw)[16], int d0, float g) __attribute__((always_inline)) {
+      uint32_t parts[16];
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const int d = d0 + 2 * i;                    // dim is even
-        const float a = d < D ? __uint_as_float(raw[2 * i]) : 0.f, b = d < D ? __uint_as_float(raw[2 * i + 1]) : 0.f;
-        dl_split2(a, b, hi[i], lo[i]);
-        scaled[2 * i] = __float_as_uint(a * g);
-        scaled[2 * i + 1] = __float_as_uint(b * g);
+      for (int i = 0; i < 8; ++i) {
+        if (d0 + 2 * i >= D) raw[2 * i] = raw[2 * i + 1] = 0u;       // dim is even
+        dl_split2(__uint_as_float(raw[2 * i]), __uint_as_float(raw[2 * i + 1]), parts[i], parts[8 + i]);
       }
-      tmem_st_32x16(T_SH + la + d0 / 2, hi);
-      tmem_st_32x16(T_SL + la + d0 / 2, lo);
-      tmem_st_32x32(T_S + la + d0, scaled);
+      tmem_st_32x16(T_SP + la + d0, parts);
+#pragma unroll
+      for (int i = 0; i < 16; ++i) raw[i] = __float_as_uint(__uint_as_float(raw[i]) * g);
+      tmem_st_32x16(T_S + la + d0, raw);
     };
     auto signal = [&](uint64_t* bar) {
       tmem_st_wait();
       tc_fence_before();
       mbar_arrive(bar);
     };
+    // One warp polls, the others sleep at the barrier behind it and leave the issue slots to the output warps.
+    // After a wait that gave up the loop goes on, without waiting, so that the warps meet at every barrier.
+    auto wait = [&](uint64_t* bar, uint32_t parity) {
+      if (warp == 0 && !mbar_wait(bar, parity, abort_word)) *abort_word = ERR_WAIT_MISC;
+      __syncwarp();
+      asm volatile("bar.sync 3, %0;" ::"n"(DK_CHAIN * 32) : "memory");
+      tc_fence_after();
+    };
+    uint32_t v[HT / 2];                              // values of the chunk to come, pairs of tokens
+    auto load_values = [&](const uint8_t* stage) __attribute__((always_inline)) {
+      int c8 = (e >> 3) & 7;
+      asm volatile("" : "+r"(c8));                   // addresses are made anew in every chunk: kept, they would be spilled
+      const uint8_t* vp = stage + L::X + (e >> 6) * DC_TILE + (e & 7) * 2 + cg * HT * 128;
+#pragma unroll
+      for (int i = 0; i < HT / 2; ++i)
+        v[i] = e < E ? (uint32_t)*reinterpret_cast<const uint16_t*>(vp + dl_swz(2 * i, c8)) |
+                           (uint32_t)*reinterpret_cast<const uint16_t*>(vp + dl_swz(2 * i + 1, c8)) << 16
+                     : 0u;
+    };
     if (chunks > 0) {
-      ok = mbar_wait(&full[0], 0, abort_word);
+      wait(&full[0], 0);
+      load_values(smem);
       const float g = reinterpret_cast<const float*>(smem + L::X + L::V + DI_F)[4 * DC];
+#pragma unroll 1
+      for (int d0 = cg * HD; d0 < (cg + 1) * HD; d0 += 16) {
+        uint32_t raw[16];
 #pragma unroll
-      for (int part = 0; part < PD; ++part) {
-        uint32_t raw[32];
-        const int d0 = half * HD + part * 32;
-#pragma unroll
-        for (int i = 0; i < 32; ++i) raw[i] = carried && e < E && d0 + i < D ? __float_as_uint(state[(long long)(d0 + i) * E + e]) : 0u;
+        for (int i = 0; i < 16; ++i) raw[i] = carried && e < E && d0 + i < D ? __float_as_uint(state[(long long)(d0 + i) * E + e]) : 0u;
         publish(raw, d0, g);
       }
       signal(s_ready);
     }
-    for (int ch = 0; ch < chunks && ok; ++ch) {
+    for (int ch = 0; ch < chunks; ++ch) {
       const int st = ch & 1;
       const uint32_t ph = ch & 1;
       const uint8_t* stage = smem + st * L::STAGE;
-      const float* f = reinterpret_cast<const float*>(stage + L::X + L::V + DI_F) + half * 32;
-      ok = mbar_wait(&full[st], (ch >> 1) & 1, abort_word);
-      if (!ok) break;
-      uint32_t hi[16], lo[16], d[32];
-      float v[32];
-      {
-        const uint8_t* vp = stage + L::X + (e >> 6) * DC_TILE + (e & 7) * 2;
+      const float* f = reinterpret_cast<const float*>(stage + L::X + L::V + DI_F) + cg * HT;
+      uint32_t parts[16], d[16];                     // (the stage has landed: its decay was read a chunk ago)
+      wait(d1_full, ph);
 #pragma unroll
-        for (int i = 0; i < 32; ++i)
-          v[i] = e < E ? __uint_as_float((uint32_t)*reinterpret_cast<const uint16_t*>(vp + dl_swz(half * 32 + i, (e >> 3) & 7)) << 16) : 0.f;
-      }
-      ok = mbar_wait(d1_full, ph, abort_word);
-      if (!ok) break;
-      tc_fence_after();
-      tmem_ld_32x32(T_D + la + half * 32, d);
-      tmem_ld_wait();
+      for (int q = 0; q < HT / 16; ++q) {
+        tmem_ld_32x16(T_D + la + cg * HT + q * 16, d);
+        tmem_ld_wait();
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const float2 beta = *reinterpret_cast<const float2*>(f + 2 * i), c = *reinterpret_cast<const float2*>(f + DC + 2 * i);
-        dl_split2(beta.x * fmaf(-c.x, __uint_as_float(d[2 * i]), v[2 * i]), beta.y * fmaf(-c.y, __uint_as_float(d[2 * i + 1]), v[2 * i + 1]),
-                  hi[i], lo[i]);
+        for (int i = 0; i < 8; ++i) {
+          const float2 beta = *reinterpret_cast<const float2*>(f + q * 16 + 2 * i), c = *reinterpret_cast<const float2*>(f + DC + q * 16 + 2 * i);
+          const float2 x = unpack_bf16x2(v[q * 8 + i]);
+          dl_split2(beta.x * fmaf(-c.x, __uint_as_float(d[2 * i]), x.x), beta.y * fmaf(-c.y, __uint_as_float(d[2 * i + 1]), x.y), parts[i], parts[8 + i]);
+        }
+        tmem_st_32x16(T_R + la + cg * HT + q * 16, parts);
       }
-      tmem_st_32x16(T_RH + la + half * 16, hi);
-      tmem_st_32x16(T_RL + la + half * 16, lo);
       signal(r_ready);
-      ok = mbar_wait(d2_full, ph, abort_word);
-      if (!ok) break;
-      tc_fence_after();
-      tmem_ld_32x32(T_D + la + half * 32, d);
-      tmem_ld_wait();
+      wait(d2_full, ph);
 #pragma unroll
-      for (int i = 0; i < 16; ++i) dl_split2(__uint_as_float(d[2 * i]), __uint_as_float(d[2 * i + 1]), hi[i], lo[i]);
-      tmem_st_32x16(T_RH + la + half * 16, hi);
-      tmem_st_32x16(T_RL + la + half * 16, lo);
+      for (int q = 0; q < HT / 16; ++q) {
+        tmem_ld_32x16(T_D + la + cg * HT + q * 16, d);
+        tmem_ld_wait();
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const float2 w = *reinterpret_cast<const float2*>(f + 2 * DC + 2 * i);
-        dl_split2(__uint_as_float(d[2 * i]) * w.x, __uint_as_float(d[2 * i + 1]) * w.y, hi[i], lo[i]);
+        for (int i = 0; i < 8; ++i) {
+          const float2 w = *reinterpret_cast<const float2*>(f + 2 * DC + q * 16 + 2 * i);
+          dl_split2(__uint_as_float(d[2 * i]) * w.x, __uint_as_float(d[2 * i + 1]) * w.y, parts[i], parts[8 + i]);
+        }
+        tmem_st_32x16(T_W + la + cg * HT + q * 16, parts);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) dl_split2(__uint_as_float(d[2 * i]), __uint_as_float(d[2 * i + 1]), parts[i], parts[8 + i]);
+        tmem_st_32x16(T_R + la + cg * HT + q * 16, parts);
       }
-      tmem_st_32x16(T_WH + la + half * 16, hi);
-      tmem_st_32x16(T_WL + la + half * 16, lo);
       signal(u_ready);
       __syncwarp();
       if (lane == 0) mbar_arrive(&empty[st]);        // nothing of the stage is read here any more
-      const bool last = ch + 1 == chunks;
-      float g = 0.f;
-      if (!last) {
-        ok = mbar_wait(&full[st ^ 1], ((ch + 1) >> 1) & 1, abort_word);
-        if (!ok) break;
-        g = reinterpret_cast<const float*>(smem + (st ^ 1) * L::STAGE + L::X + L::V + DI_F)[4 * DC];
-      }
-      ok = mbar_wait(s_full, ph, abort_word);
-      if (!ok) break;
-      tc_fence_after();
+      if (ch + 1 == chunks) break;
+      wait(&full[st ^ 1], ((ch + 1) >> 1) & 1);
+      load_values(smem + (st ^ 1) * L::STAGE);
+      const float g = reinterpret_cast<const float*>(smem + (st ^ 1) * L::STAGE + L::X + L::V + DI_F)[4 * DC];
+      wait(s_full, ph);
 #pragma unroll
-      for (int part = 0; part < PD; ++part) {
-        uint32_t raw[32];
-        const int d0 = half * HD + part * 32;
-        tmem_ld_32x32(T_S + la + d0, raw);
+      for (int piece = 0; piece < HD / 16; ++piece) {
+        const int d0 = cg * HD + piece * 16;
+        tmem_ld_32x16(T_S + la + d0, d);
         tmem_ld_wait();
-        if (!last) {
-          publish(raw, d0, g);
-        } else if (e < E) {
+        publish(d, d0, g);
+      }
+      signal(s_ready);
+    }
+    if (chunks > 0) {
+      wait(s_full, (chunks - 1) & 1);
+#pragma unroll 1
+      for (int d0 = cg * HD; d0 < (cg + 1) * HD; d0 += 16) {
+        uint32_t raw[16];
+        tmem_ld_32x16(T_S + la + d0, raw);
+        tmem_ld_wait();
+        if (e < E && *abort_word == 0) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i)
+          for (int i = 0; i < 16; ++i)
             if (d0 + i < D) state[(long long)(d0 + i) * E + e] = __uint_as_float(raw[i]);
         }
       }
-      if (!last) signal(s_ready);
     }
-    if (!ok) *abort_word = ERR_WAIT_MISC;
   } else {
-    const int quarter = warp & 3, e = quarter * 32 + lane;
+    const int quarter = warp & 3, e = quarter * 32 + lane, ow = warp - DK_CHAIN, og = ow >> 2;       // half of the tokens
     const uint32_t la = uint32_t(quarter * 32) << 16;
     float* o = reinterpret_cast<float*>(smem + L::OFF_O);
-    constexpr int OP = PE * 64;
-    const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.gate) + (long long)row0 * p.ld_gate + h * E;
+    constexpr int OP = PE * 64, HT = DC / (DK_OUT / 4), RT = DC / DK_OUT;       // tokens read from tensor memory, and finished, per warp
     const int c = lane * 4;                          // columns of an output row that this lane finishes
     float w[4] = {0.f, 0.f, 0.f, 0.f};
     if (c < E) load_vec<4>(reinterpret_cast<const __nv_bfloat16*>(p.weight) + c, w);
+    const float share = 1.f / (float)E;
+    const uint8_t* gate = smem + L::OFF_G + (c < E ? (c >> 6) * DC_TILE + (c & 7) * 2 : 0);
+    auto load_gates = [&](int ch) {                  // by one thread, once the gates of the chunk before have been used
+      mbar_expect_tx(g_full, (uint32_t)((E + 63) / 64) * DC_TILE);
+      for (int i = 0; i < (E + 63) / 64; ++i) tma_load_2d(smem + L::OFF_G + i * DC_TILE, &tm_gate, g_full, h * E + i * 64, row0 + ch * DC);
+    };
+    if (chunks > 0 && warp == DK_CHAIN && lane == 0) load_gates(0);
+    __syncwarp();
     for (int ch = 0; ch < chunks; ++ch) {
       const int st = ch & 1, n = min(DC, rows - ch * DC);
-      const float* f = reinterpret_cast<const float*>(smem + st * L::STAGE + L::X + L::V + DI_F) + 3 * DC;
-      // after a wait that gave up the loop goes on, without waiting, so that the four warps meet at every barrier
-      if (!mbar_wait(&full[st], (ch >> 1) & 1, abort_word) || !mbar_wait(o_full, ch & 1, abort_word)) *abort_word = ERR_WAIT_TMEM_FULL;
+      const float* f = reinterpret_cast<const float*>(smem + st * L::STAGE + L::X + L::V + DI_F) + 3 * DC + og * HT;
+      if (warp == DK_CHAIN && (!mbar_wait(&full[st], (ch >> 1) & 1, abort_word) || !mbar_wait(g_full, ch & 1, abort_word) ||
+                               !mbar_wait(o_full, ch & 1, abort_word)))
+        *abort_word = ERR_WAIT_TMEM_FULL;
       __syncwarp();
+      asm volatile("bar.sync 2, %0;" ::"n"(DK_OUT * 32) : "memory");      // the rows of the chunk before have been read, too
       tc_fence_after();
-      asm volatile("bar.sync 2, 128;" ::: "memory");      // the rows of the chunk before have been read
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        uint32_t a[32], b[32];
-        tmem_ld_32x32(T_D + la + 64 + half * 32, a);
-        tmem_ld_32x32(T_D + la + half * 32, b);
+      for (int q = 0; q < HT / 16; ++q) {
+        uint32_t a[16], b[16];
+        tmem_ld_32x16(T_D + la + 64 + og * HT + q * 16, a);
+        tmem_ld_32x16(T_D + la + og * HT + q * 16, b);
         tmem_ld_wait();
         if (e < OP) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) o[(half * 32 + i) * OP + e] = fmaf(f[half * 32 + i], __uint_as_float(a[i]), __uint_as_float(b[i]));
+          for (int i = 0; i < 16; ++i)
+            o[(og * HT + q * 16 + i) * OP + e] = fmaf(f[q * 16 + i], __uint_as_float(a[i]), __uint_as_float(b[i]));
         }
       }
       tc_fence_before();
       mbar_arrive(o_read);
       __syncwarp();
       if (lane == 0) mbar_arrive(&empty[st]);
-      asm volatile("bar.sync 2, 128;" ::: "memory");
-      for (int t0 = warp - 8; t0 < n; t0 += 16) {
-        Raw<__nv_bfloat16, 4> z[4];
+      asm volatile("bar.sync 2, %0;" ::"n"(DK_OUT * 32) : "memory");
+      // rows ow, ow + DK_OUT, ... of the chunk, all of them at a time
+      float x[RT][4], ss[RT], g[4];
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (t0 + j * 4 < n && c < E)
-            z[j] = *reinterpret_cast<const Raw<__nv_bfloat16, 4>*>(gate + (long long)(ch * DC + t0 + j * 4) * p.ld_gate + c);
+      for (int j = 0; j < RT; ++j) {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const int t = t0 + j * 4;
-          if (t >= n) break;
-          float x[4] = {0.f, 0.f, 0.f, 0.f}, g[4];
-          if (c < E) load_vec<4>(o + t * OP + c, x);
-          float ss = fmaf(x[0], x[0], fmaf(x[1], x[1], fmaf(x[2], x[2], x[3] * x[3])));
-#pragma unroll
-          for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
-          const float inv = rsqrtf(ss / (float)E + p.eps);
-          if (c < E) {
-            load_vec<4>(z[j].v, g);
-#pragma unroll
-            for (int i = 0; i < 4; ++i) x[i] *= inv * w[i] * g[i] * sigmoid_f(g[i]);
-            store_vec<4>(gy + (long long)(ch * DC + t) * p.ld_y + c, x);
-          }
-        }
+        for (int i = 0; i < 4; ++i) x[j][i] = 0.f;
+        if (c < E) load_vec<4>(o + (ow + j * DK_OUT) * OP + c, x[j]);
+        ss[j] = fmaf(x[j][0], x[j][0], fmaf(x[j][1], x[j][1], fmaf(x[j][2], x[j][2], x[j][3] * x[j][3])));
       }
+#pragma unroll
+      for (int k = 16; k > 0; k >>= 1)
+#pragma unroll
+        for (int j = 0; j < RT; ++j) ss[j] += __shfl_xor_sync(0xffffffffu, ss[j], k);
+      __nv_bfloat16* yr = gy + (long long)(ch * DC + ow) * p.ld_y + c;
+#pragma unroll
+      for (int j = 0; j < RT; ++j) {
+        const int t = ow + j * DK_OUT;
+        const float inv = rsqrtf(fmaf(ss[j], share, p.eps));
+        load_vec<4>(reinterpret_cast<const __nv_bfloat16*>(gate + dl_swz(t, (c >> 3) & 7)), g);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) x[j][i] *= inv * w[i] * g[i] * dl_sigmoid(g[i]);
+        if (t < n && c < E) store_vec<4>(yr, x[j]);
+        yr += DK_OUT * p.ld_y;
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(g_empty);
+      if (warp == DK_CHAIN && lane == 0 && ch + 1 < chunks) {
+        if (mbar_wait(g_empty, ch & 1, abort_word)) load_gates(ch + 1);
+        else *abort_word = ERR_WAIT_EMPTY;
+      }
+      __syncwarp();
     }
   }
   if (!live) {
@@ -833,14 +905,14 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
     while (globaltimer_ns() - w0 < 200000ull) __nanosleep(1000);
     __syncthreads();
   }
-  if (warp == 13) {
+  if (warp == DK_CHAIN + DK_OUT + 1) {
     tc_fence_after();
     tmem_dealloc(tmem, 512);
   }
 }
 
 template <int PD, int PE>
-static int launch_delta_chunk(const CUtensorMap& tm, const DeltaArgs& p, cudaStream_t st) {
+static int launch_delta_chunk(const CUtensorMap& tm, const CUtensorMap& tm_gate, const DeltaArgs& p, cudaStream_t st) {
   auto kern = delta_chunk_kernel<PD, PE>;
   static bool configured = false;
   if (!configured) {
@@ -850,7 +922,7 @@ static int launch_delta_chunk(const CUtensorMap& tm, const DeltaArgs& p, cudaStr
     configured = true;
   }
   launch_dep(delta_prepare_kernel, (unsigned)(p.chunks * p.heads), 128, DeltaPrepareSmem::TOTAL, st, tm, p);
-  launch_dep(kern, (unsigned)(p.seqs * p.heads), DK_THREADS, DeltaChunkSmem<PD, PE>::TOTAL, st, tm, p);
+  launch_dep(kern, (unsigned)(p.seqs * p.heads), DK_THREADS, DeltaChunkSmem<PD, PE>::TOTAL, st, tm, tm_gate, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
@@ -885,14 +957,15 @@ extern "C" int b200_delta(const DeltaArgs* args, int mode, int f32, cudaStream_t
     if (f32 || p.cu == nullptr || p.chunk_cu == nullptr || p.ab == nullptr || p.image == nullptr || p.taps > 0 || p.dim > 128 || p.vdim > 128 ||
         p.dim % 8 || p.vdim % 8 || p.chunks <= 0)
       return -11;
-    if (p.ld_c % 8 || p.ld_y % 8 || p.ld_gate % 4 ||
+    if (p.ld_c % 8 || p.ld_y % 8 || p.ld_gate % 8 ||
         ((ptrs | reinterpret_cast<uintptr_t>(p.y) | reinterpret_cast<uintptr_t>(p.image) | reinterpret_cast<uintptr_t>(p.weight)) & 15) ||
-        (reinterpret_cast<uintptr_t>(p.gate) & 7))
+        (reinterpret_cast<uintptr_t>(p.gate) & 15))
       return -11;
-    CUtensorMap tm;
+    CUtensorMap tm, tm_gate;
+    if (make_tmap_bf16_2d(&tm_gate, p.gate, (uint64_t)p.rows, (uint64_t)p.heads * p.vdim, (uint64_t)p.ld_gate, 64, DC)) return -20;
     if (make_tmap_bf16_2d(&tm, p.c, (uint64_t)p.rows, (uint64_t)(2 * p.kv_heads * p.dim + p.heads * p.vdim), (uint64_t)p.ld_c, 64, DC)) return -20;
-    if (p.dim <= 64) return p.vdim <= 64 ? launch_delta_chunk<1, 1>(tm, p, st) : launch_delta_chunk<1, 2>(tm, p, st);
-    return p.vdim <= 64 ? launch_delta_chunk<2, 1>(tm, p, st) : launch_delta_chunk<2, 2>(tm, p, st);
+    if (p.dim <= 64) return p.vdim <= 64 ? launch_delta_chunk<1, 1>(tm, tm_gate, p, st) : launch_delta_chunk<1, 2>(tm, tm_gate, p, st);
+    return p.vdim <= 64 ? launch_delta_chunk<2, 1>(tm, tm_gate, p, st) : launch_delta_chunk<2, 2>(tm, tm_gate, p, st);
   }
   const bool vec = p.vdim % 4 == 0 && p.ld_c % 4 == 0 && (ptrs & 15) == 0;
   const int groups = vec ? p.vdim / 4 : p.vdim, rg = groups < 256 ? 256 / groups : 1, per = (p.dim + rg - 1) / rg;
