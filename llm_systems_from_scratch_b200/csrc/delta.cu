@@ -312,11 +312,11 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) delta_step_kernel(const D
 //                   blocks and products, T and P split into two bf16 parts (hi + lo, 16 significant bits), the per-token factors: an image of 33 KB
 //                   that the second kernel copies as it is
 //   delta_chunk     one CTA per (portion, head), chunks in order, everything transposed so that a lane of tensor memory is a column of v:
-//                     [S^T K^T | S^T Q^T]  ->  R = beta (V - ...)^T  ->  U^T = R T^T  ->  S^T = exp(b_n) S^T + W K,  P U  (W: U with its factors)
+//                     V^T (a product with the unit matrix)  [S^T K^T | S^T Q^T]  ->  R = beta (V - ...)^T  ->  U^T = R T^T  ->  S^T = exp(b_n) S^T + W K,  P U  (W: U with its factors)
 //                   S, R, U and W are A operands in tensor memory, split like T and P; products accumulate in fp32 (lo x lo is dropped)
 constexpr int DC = 64;                              // tokens of a chunk
 constexpr int DC_TILE = DC * 128;                   // bytes of 64 rows of 64 bf16 columns, 128-byte swizzle
-constexpr int DI_T = 0, DI_P = 2 * DC_TILE, DI_F = 4 * DC_TILE;      // image: T hi, lo | P hi, lo | beta, c, w, a per token | exp(b_n)
+constexpr int DI_T = 0, DI_P = 2 * DC_TILE, DI_F = 4 * DC_TILE;      // image: T hi, lo | P hi, lo | (beta, -beta c), w, a per token | exp(b_n)
 constexpr int DI_BYTES = DI_F + 4 * DC * 4 + 128;
 constexpr float DELTA_LOG2E = 1.4426950408889634f;
 
@@ -334,15 +334,14 @@ __device__ __forceinline__ float dl_sigmoid(float g) {    // (1 + tanh(g / 2)) /
 __device__ __forceinline__ void dl_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
   const uint32_t a = __float_as_uint(x), b = __float_as_uint(y);
   hi = __byte_perm(a, b, 0x7632);
-  lo = pack_bf16x2_alu(x - __uint_as_float(a & 0xffff0000u), y - __uint_as_float(b & 0xffff0000u));
+  lo = pack_bf16x2(x - __uint_as_float(a & 0xffff0000u), y - __uint_as_float(b & 0xffff0000u));
 }
 __device__ __forceinline__ uint32_t dl_swz(int r, int c8) { return (uint32_t)r * 128u + (uint32_t)((c8 ^ (r & 7)) << 4); }
 
 struct DeltaPrepareSmem {                           // X: panels of [64 rows of K; 64 rows of Q] x 64 columns, later the image
-  static constexpr int OFF_X = 0, OFF_I = 0;
+  static constexpr int OFF_X = 0, OFF_I = 0, OFF_A = (DI_BYTES + 1023) / 1024 * 1024;
   static constexpr int PITCH = 68;                  // floats between the rows of A
-  static constexpr int OFF_A = (DI_BYTES + 1023) / 1024 * 1024;
-  static constexpr int OFF_F = OFF_A + DC * PITCH * 4;       // b [64], beta [64], inverse lengths [128]
+  static constexpr int OFF_F = OFF_A + DC * PITCH * 4;        // b [64], beta [64], inverse lengths [128]
   static constexpr int OFF_BAR = OFF_F + 4 * DC * 4;
   static constexpr int TOTAL = OFF_BAR + 2 * 8 + 16 + 1024;
 };
@@ -350,8 +349,9 @@ struct DeltaPrepareSmem {                           // X: panels of [64 rows of 
 __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constant__ CUtensorMap tm, const DeltaArgs p) {
   using L = DeltaPrepareSmem;
   extern __shared__ uint8_t dl_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dl_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* smem = dl_raw + (-smem_u32(dl_raw) & 1023u);        // (an offset, so that accesses stay known as shared)
   float* A = reinterpret_cast<float*>(smem + L::OFF_A);
+  auto at = [&](int row, int col) { return A + row * L::PITCH + col; };
   float *sb = reinterpret_cast<float*>(smem + L::OFF_F), *sbeta = sb + DC, *slen = sbeta + DC;
   uint64_t *bar_l = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR), *bar_m = bar_l + 1;
   uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bar_l + 2);
@@ -442,24 +442,36 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
   const int t = r & (DC - 1);
   const float bt = sb[t], mine = slen[r] * (r < DC ? sbeta[t] : 1.f);
   uint8_t* image = smem + L::OFF_I;
+  const int last = r < DC ? t - 1 : t;              // A lies strictly below the diagonal
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
+    const bool any = half == 0 || (warp & 1) == 1;  // the first 32 tokens see none of the others
     uint32_t raw[32];
-    tmem_ld_32x32(tmem + (uint32_t(warp * 32) << 16) + half * 32, raw);
-    tmem_ld_wait();
-    const int last = r < DC ? t - 1 : t;            // A lies strictly below the diagonal
+    if (any) {
+      tmem_ld_32x32(tmem + (uint32_t(warp * 32) << 16) + half * 32, raw);
+      tmem_ld_wait();
+    } else if (r < DC) {
+      continue;                                     // (that part of A is not read)
+    }
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
       float f[8];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int s = half * 32 + q * 8 + i;
-        f[i] = s <= last ? __uint_as_float(raw[q * 8 + i]) * (mine * slen[s]) * dl_exp2(fminf(bt - sb[s], 0.f)) : 0.f;
+      for (int j = 0; j < 2; ++j) {
+        const int s = half * 32 + q * 8 + j * 4;
+        float4 lens = make_float4(0.f, 0.f, 0.f, 0.f), bs = lens;
+        if (any) {
+          lens = *reinterpret_cast<const float4*>(slen + s);
+          bs = *reinterpret_cast<const float4*>(sb + s);
+        }
+        const float l4[4] = {lens.x, lens.y, lens.z, lens.w}, b4[4] = {bs.x, bs.y, bs.z, bs.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          f[j * 4 + i] = any && s + i <= last ? __uint_as_float(raw[q * 8 + j * 4 + i]) * (mine * l4[i]) * dl_exp2(fminf(bt - b4[i], 0.f)) : 0.f;
       }
       if (r < DC) {
-        float* to = A + t * L::PITCH + half * 32 + q * 8;
-        *reinterpret_cast<float4*>(to) = make_float4(f[0], f[1], f[2], f[3]);
-        *reinterpret_cast<float4*>(to + 4) = make_float4(f[4], f[5], f[6], f[7]);
+        *reinterpret_cast<float4*>(at(t, half * 32 + q * 8)) = make_float4(f[0], f[1], f[2], f[3]);
+        *reinterpret_cast<float4*>(at(t, half * 32 + q * 8 + 4)) = make_float4(f[4], f[5], f[6], f[7]);
       } else {
         uint4 hi4, lo4;
         dl_split2(f[0], f[1], hi4.x, lo4.x);
@@ -473,17 +485,18 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
   }
   tc_fence_before();
   __syncthreads();
-  // ---- T by halves of 32: the diagonal blocks by forward substitution, a thread per column, then T21 = -T22 (A21 T11)
-  constexpr int HB = DC / 2;
-  if (r < DC) {
-    const int c = r & (HB - 1), o = (r / HB) * HB;
-    float x[HB];
+  // ---- T from its diagonal blocks of 16 (forward substitution, a warp per block, a lane per column), then twice
+  // T21 = -T22 (A21 T11), for blocks of 16 and of 32.  Products are kept above the diagonal, where A has nothing.
+  constexpr int HB = DC / 2, QB = DC / 4;
+  {
+    const int o = warp * QB, c = lane & (QB - 1);
+    float x[QB];
 #pragma unroll
-    for (int i = 0; i < HB; ++i) {
+    for (int i = 0; i < QB; ++i) {
       float a[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int s = 0; s < i; s += 4) {
-        const float4 v = *reinterpret_cast<const float4*>(A + (o + i) * L::PITCH + o + s);
+        const float4 v = *reinterpret_cast<const float4*>(at(o + i, o + s));
         a[0] = fmaf(v.x, x[s], a[0]);
         if (s + 1 < i) a[1] = fmaf(v.y, x[s + 1], a[1]);
         if (s + 2 < i) a[2] = fmaf(v.z, x[s + 2], a[2]);
@@ -492,54 +505,89 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
       x[i] = (i == c ? 1.f : 0.f) - ((a[0] + a[1]) + (a[2] + a[3]));
     }
     __syncwarp();                                   // the block has been read
+    if (lane < QB) {
 #pragma unroll
-    for (int i = 0; i < HB; ++i) A[(o + i) * L::PITCH + o + c] = x[i];
-  } else {
+      for (int i = 0; i < QB; ++i) *at(o + i, o + c) = x[i];
+    }
+  }
+  if (r >= DC) {
     float* f = reinterpret_cast<float*>(image + DI_F);
     const float end = sb[DC - 1], grown = dl_exp2(bt);
-    f[t] = sbeta[t];
-    f[DC + t] = grown * slen[t];                    // of S^T k_t
+    *reinterpret_cast<float2*>(f + 2 * t) = make_float2(sbeta[t], -sbeta[t] * grown * slen[t]);      // of v_t, of S^T k_t
     f[2 * DC + t] = dl_exp2(end - bt) * slen[t];    // of u_t where it joins the state
     f[3 * DC + t] = grown * slen[r];                // of S^T q_t
     if (t == 0) f[4 * DC] = dl_exp2(end);
   }
   __syncthreads();
-  // rows warp * 8 .. + 7 and column `lane` of L R, where L's rows start at l and R's at rt
-  auto product = [&](const float* l, const float* rt, float (&acc)[8]) __attribute__((always_inline)) {
+  {
+    // two pairs of blocks, two warps each: 8 rows of a 16 x 16 product per warp, four of them per half warp
+    const int o = (warp >> 1) * HB, c = lane & (QB - 1), i0 = (warp & 1) * 8 + (lane >> 4) * 4;
+    auto small = [&](int lr, int lc, int rr, int rc, float (&acc)[4]) __attribute__((always_inline)) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i] = 0.f;
+#pragma unroll
+      for (int s = 0; s < QB; s += 4) {
+        float v[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] = *at(rr + s + j, rc + c);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float4 w = *reinterpret_cast<const float4*>(at(lr + i0 + i, lc + s));
+          acc[i] = fmaf(w.x, v[0], fmaf(w.y, v[1], fmaf(w.z, v[2], fmaf(w.w, v[3], acc[i]))));
+        }
+      }
+    };
+    float acc[4];
+    small(o + QB, o, o, o, acc);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) *at(o + i0 + i, o + QB + c) = acc[i];
+    __syncthreads();
+    small(o + QB, o + QB, o, o + QB, acc);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) *at(o + QB + i0 + i, o + c) = -acc[i];
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 4; ++i) *at(o + i0 + i, o + QB + c) = 0.f;
+  }
+  __syncthreads();
+  // rows warp * 8 .. + 7 and column `lane` of the product of the blocks at (lr, lc) and (rr, rc)
+  auto product = [&](int lr, int lc, int rr, int rc, float (&acc)[8]) __attribute__((always_inline)) {
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[i] = 0.f;
 #pragma unroll
     for (int s = 0; s < HB; s += 4) {
       float v[4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) v[j] = rt[(s + j) * L::PITCH + lane];
+      for (int j = 0; j < 4; ++j) v[j] = *at(rr + s + j, rc + lane);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        const float4 w = *reinterpret_cast<const float4*>(l + (warp * 8 + i) * L::PITCH + s);
+        const float4 w = *reinterpret_cast<const float4*>(at(lr + warp * 8 + i, lc + s));
         acc[i] = fmaf(w.x, v[0], fmaf(w.y, v[1], fmaf(w.z, v[2], fmaf(w.w, v[3], acc[i]))));
       }
     }
   };
   float acc[8];
-  product(A + HB * L::PITCH, A, acc);               // A21 T11, kept above the diagonal
+  product(HB, 0, 0, 0, acc);               // A21 T11, kept above the diagonal
 #pragma unroll
-  for (int i = 0; i < 8; ++i) A[(warp * 8 + i) * L::PITCH + HB + lane] = acc[i];
+  for (int i = 0; i < 8; ++i) *at(warp * 8 + i, HB + lane) = acc[i];
   __syncthreads();
-  product(A + HB * L::PITCH + HB, A + HB, acc);
+  product(HB, HB, 0, HB, acc);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) A[(HB + warp * 8 + i) * L::PITCH + lane] = -acc[i];
+  for (int i = 0; i < 8; ++i) *at(HB + warp * 8 + i, lane) = -acc[i];
   __syncthreads();
   {
     const int row = r >> 1, half = r & 1;
+    const bool zero = row < HB && half == 1;        // above the diagonal
+    float4 u[8];
+#pragma unroll
+    for (int q = 0; q < 8; ++q) u[q] = zero ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(at(row, half * 32 + q * 4));
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
-      const float4 u = *reinterpret_cast<const float4*>(A + row * L::PITCH + half * 32 + q * 8), v = *reinterpret_cast<const float4*>(A + row * L::PITCH + half * 32 + q * 8 + 4);
-      const bool zero = row < HB && half == 1;      // above the diagonal
       uint4 hi4, lo4;
-      dl_split2(zero ? 0.f : u.x, zero ? 0.f : u.y, hi4.x, lo4.x);
-      dl_split2(zero ? 0.f : u.z, zero ? 0.f : u.w, hi4.y, lo4.y);
-      dl_split2(zero ? 0.f : v.x, zero ? 0.f : v.y, hi4.z, lo4.z);
-      dl_split2(zero ? 0.f : v.z, zero ? 0.f : v.w, hi4.w, lo4.w);
+      dl_split2(u[2 * q].x, u[2 * q].y, hi4.x, lo4.x);
+      dl_split2(u[2 * q].z, u[2 * q].w, hi4.y, lo4.y);
+      dl_split2(u[2 * q + 1].x, u[2 * q + 1].y, hi4.z, lo4.z);
+      dl_split2(u[2 * q + 1].z, u[2 * q + 1].w, hi4.w, lo4.w);
       *reinterpret_cast<uint4*>(image + DI_T + dl_swz(row, half * 4 + q)) = hi4;
       *reinterpret_cast<uint4*>(image + DI_T + DC_TILE + dl_swz(row, half * 4 + q)) = lo4;
     }
@@ -569,7 +617,8 @@ struct DeltaChunkSmem {
   static constexpr int X = PD * 16384, V = PE * DC_TILE, I = (DI_BYTES + 1023) / 1024 * 1024, STAGE = X + V + I;
   static constexpr int OFF_O = 2 * STAGE;            // [64][PE * 64] floats
   static constexpr int OFF_G = OFF_O + DC * PE * 64 * 4;       // output gates
-  static constexpr int OFF_BAR = OFF_G + PE * DC_TILE;
+  static constexpr int OFF_ONE = OFF_G + PE * DC_TILE;         // the unit matrix, bf16
+  static constexpr int OFF_BAR = OFF_ONE + DC_TILE;
   static constexpr int NUM_BARS = 14;
   static constexpr int TOTAL = OFF_BAR + NUM_BARS * 8 + 16 + 1024;
 };
@@ -579,7 +628,7 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
                                                                      const __grid_constant__ CUtensorMap tm_gate, const DeltaArgs p) {
   using L = DeltaChunkSmem<PD, PE>;
   extern __shared__ uint8_t dl_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dl_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* smem = dl_raw + (-smem_u32(dl_raw) & 1023u);        // (an offset, so that accesses stay known as shared)
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR);
   uint64_t *full = bars, *empty = bars + 2;          // [2] per stage
   uint64_t *s_ready = bars + 4, *d1_full = bars + 5, *r_ready = bars + 6, *d2_full = bars + 7, *u_ready = bars + 8, *s_full = bars + 9,
@@ -611,6 +660,14 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
     tmem_alloc(tmem_holder, 512);
     tmem_relinquish();
   }
+  for (int i = tid; i < DC * 8; i += DK_THREADS) {
+    const int r = i >> 3, c8 = i & 7;
+    uint32_t w[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) w[j] = c8 * 8 + 2 * j == r ? 0x3f80u : (c8 * 8 + 2 * j + 1 == r ? 0x3f800000u : 0u);
+    *reinterpret_cast<uint4*>(smem + L::OFF_ONE + dl_swz(r, c8)) = make_uint4(w[0], w[1], w[2], w[3]);
+  }
+  fence_proxy_async_smem();
   pdl_sync();
   const int seq = blockIdx.x / p.heads, h = blockIdx.x - seq * p.heads, hk = h / (p.heads / p.kv_heads), D = p.dim, E = p.vdim;
   const int row0 = p.cu[seq], rows = p.cu[seq + 1] - row0, slot = p.state_slots[seq];
@@ -624,7 +681,7 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_holder;
-  // columns: [S^T K^T, later U, later P U | S^T Q^T] 0 - 127, S^T 128 - 255, its parts 256 - 383, R's then U's parts 384 - 447, W's 448 - 511.
+  // columns: [S^T K^T, later U, later P U | S^T Q^T] 0 - 127, S^T 128 - 255, its parts 256 - 383, V^T, then R's, then U's parts 384 - 447, W's 448 - 511.
   // Parts lie as a warp stores them: the hi, then the lo halves of 16 columns (tokens or dims), one k-step of a product.
   const uint32_t T_D = tmem, T_S = tmem + 128, T_SP = tmem + 256, T_R = tmem + 384, T_W = tmem + 448;
   const int ksteps = (D + 15) / 16;
@@ -653,6 +710,8 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
   } else if (warp == DK_CHAIN + DK_OUT + 1) {
     if (chunks > 0 && elect_one()) {
       constexpr uint32_t id_x = make_idesc_bf16(128, 128, false, false), id_t = make_idesc_bf16(128, DC, false, false);
+      constexpr uint32_t id_v = make_idesc_bf16(128, DC, true, false);
+      const uint64_t one = make_smem_desc(smem_u32(smem + L::OFF_ONE), 16, 1024);
       const uint32_t id_k = make_idesc_bf16(128, ksteps * 16, false, true);
       for (int ch = 0; ch < chunks; ++ch) {
         const int st = ch & 1;
@@ -661,8 +720,12 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
         const uint64_t x = make_smem_desc(at, 16, 1024), kt = make_smem_desc(at, 16384, 1024);
         const uint64_t th = make_smem_desc(im + DI_T, 16, 1024), tl = make_smem_desc(im + DI_T + DC_TILE, 16, 1024);
         const uint64_t ph_ = make_smem_desc(im + DI_P, 16, 1024), pl = make_smem_desc(im + DI_P + DC_TILE, 16, 1024);
-        ok = mbar_wait(&full[st], (ch >> 1) & 1, abort_word) && mbar_wait(s_ready, ph, abort_word) &&
-             (ch == 0 || mbar_wait(o_read, ph ^ 1, abort_word));
+        const uint64_t vt = make_smem_desc(at + L::X, DC_TILE, 1024);
+        ok = mbar_wait(&full[st], (ch >> 1) & 1, abort_word);
+        if (!ok) break;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) umma_f16_ss(T_R, vt + (uint32_t)(k * 128), one + (uint32_t)(k * 2), id_v, k ? 1u : 0u);
+        ok = mbar_wait(s_ready, ph, abort_word) && (ch == 0 || mbar_wait(o_read, ph ^ 1, abort_word));
         if (!ok) break;
         tc_fence_after();
 #pragma unroll
@@ -727,20 +790,8 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
       asm volatile("bar.sync 3, %0;" ::"n"(DK_CHAIN * 32) : "memory");
       tc_fence_after();
     };
-    uint32_t v[HT / 2];                              // values of the chunk to come, pairs of tokens
-    auto load_values = [&](const uint8_t* stage) __attribute__((always_inline)) {
-      int c8 = (e >> 3) & 7;
-      asm volatile("" : "+r"(c8));                   // addresses are made anew in every chunk: kept, they would be spilled
-      const uint8_t* vp = stage + L::X + (e >> 6) * DC_TILE + (e & 7) * 2 + cg * HT * 128;
-#pragma unroll
-      for (int i = 0; i < HT / 2; ++i)
-        v[i] = e < E ? (uint32_t)*reinterpret_cast<const uint16_t*>(vp + dl_swz(2 * i, c8)) |
-                           (uint32_t)*reinterpret_cast<const uint16_t*>(vp + dl_swz(2 * i + 1, c8)) << 16
-                     : 0u;
-    };
     if (chunks > 0) {
       wait(&full[0], 0);
-      load_values(smem);
       const float g = reinterpret_cast<const float*>(smem + L::X + L::V + DI_F)[4 * DC];
 #pragma unroll 1
       for (int d0 = cg * HD; d0 < (cg + 1) * HD; d0 += 16) {
@@ -760,13 +811,15 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
       wait(d1_full, ph);
 #pragma unroll
       for (int q = 0; q < HT / 16; ++q) {
+        uint32_t v[16];
         tmem_ld_32x16(T_D + la + cg * HT + q * 16, d);
+        tmem_ld_32x16(T_R + la + cg * HT + q * 16, v);
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-          const float2 beta = *reinterpret_cast<const float2*>(f + q * 16 + 2 * i), c = *reinterpret_cast<const float2*>(f + DC + q * 16 + 2 * i);
-          const float2 x = unpack_bf16x2(v[q * 8 + i]);
-          dl_split2(beta.x * fmaf(-c.x, __uint_as_float(d[2 * i]), x.x), beta.y * fmaf(-c.y, __uint_as_float(d[2 * i + 1]), x.y), parts[i], parts[8 + i]);
+          const float4 w = *reinterpret_cast<const float4*>(f + cg * HT + q * 32 + 4 * i);
+          const float x = e < E ? __uint_as_float(v[2 * i]) : 0.f, y = e < E ? __uint_as_float(v[2 * i + 1]) : 0.f;
+          dl_split2(fmaf(w.y, __uint_as_float(d[2 * i]), w.x * x), fmaf(w.w, __uint_as_float(d[2 * i + 1]), w.z * y), parts[i], parts[8 + i]);
         }
         tmem_st_32x16(T_R + la + cg * HT + q * 16, parts);
       }
@@ -791,7 +844,6 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
       if (lane == 0) mbar_arrive(&empty[st]);        // nothing of the stage is read here any more
       if (ch + 1 == chunks) break;
       wait(&full[st ^ 1], ((ch + 1) >> 1) & 1);
-      load_values(smem + (st ^ 1) * L::STAGE);
       const float g = reinterpret_cast<const float*>(smem + (st ^ 1) * L::STAGE + L::X + L::V + DI_F)[4 * DC];
       wait(s_full, ph);
 #pragma unroll
@@ -842,22 +894,24 @@ __global__ void __launch_bounds__(DK_THREADS, 1) delta_chunk_kernel(const __grid
       __syncwarp();
       asm volatile("bar.sync 2, %0;" ::"n"(DK_OUT * 32) : "memory");      // the rows of the chunk before have been read, too
       tc_fence_after();
+      float r[HT];
 #pragma unroll
       for (int q = 0; q < HT / 16; ++q) {
         uint32_t a[16], b[16];
         tmem_ld_32x16(T_D + la + 64 + og * HT + q * 16, a);
         tmem_ld_32x16(T_D + la + og * HT + q * 16, b);
         tmem_ld_wait();
-        if (e < OP) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i)
-            o[(og * HT + q * 16 + i) * OP + e] = fmaf(f[q * 16 + i], __uint_as_float(a[i]), __uint_as_float(b[i]));
-        }
+        for (int i = 0; i < 16; ++i) r[q * 16 + i] = fmaf(f[q * 16 + i], __uint_as_float(a[i]), __uint_as_float(b[i]));
       }
       tc_fence_before();
       mbar_arrive(o_read);
       __syncwarp();
       if (lane == 0) mbar_arrive(&empty[st]);
+      if (e < OP) {
+#pragma unroll
+        for (int i = 0; i < HT; ++i) o[(og * HT + i) * OP + e] = r[i];
+      }
       asm volatile("bar.sync 2, %0;" ::"n"(DK_OUT * 32) : "memory");
       // rows ow, ow + DK_OUT, ... of the chunk, all of them at a time
       float x[RT][4], ss[RT], g[4];
