@@ -308,7 +308,7 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) delta_step_kernel(const D
 //     u_t + sum_(s < t) A_ts u_s = beta_t (v_t - exp(b_t) S^T k_t),      A_ts = beta_t exp(b_t - b_s) k_t . k_s
 // and o_t = exp(b_t) S^T q_t + sum_(s <= t) P_ts u_s with P_ts = exp(b_t - b_s) q_t . k_s,  S <- exp(b_n) S + sum_s exp(b_n - b_s) k_s u_s^T.
 // Every exponent is at most zero.  T = (I + A)^-1 does not depend on S:
-//   delta_prepare   all chunks at once, one CTA each: scores of [K; Q] and K on tcgen05, T in fp32 by forward substitution of its diagonal
+//   delta_prepare   all chunks at once, one CTA each: scores and squared lengths of [K; Q] on tcgen05, T in fp32 by forward substitution of its diagonal
 //                   blocks and products, T and P split into two bf16 parts (hi + lo, 16 significant bits), the per-token factors: an image of 33 KB
 //                   that the second kernel copies as it is
 //   delta_chunk     one CTA per (portion, head), chunks in order, everything transposed so that a lane of tensor memory is a column of v:
@@ -366,7 +366,7 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
     prefetch_tensormap(&tm);
   }
   if (warp == 0) {
-    tmem_alloc(tmem_holder, 64);
+    tmem_alloc(tmem_holder, 128);
     tmem_relinquish();
   }
   pdl_sync();
@@ -411,21 +411,10 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
   if (!ok) *abort_word = ERR_WAIT_FULL;
   const int r = tid;                                // row of X
   if (D & 15) *reinterpret_cast<uint4*>(smem + L::OFF_X + (D >> 6) * 16384 + dl_swz(r, (D >> 3) & 7)) = make_uint4(0, 0, 0, 0);
-  float ss = 0.f;
-  for (int c8 = 0; c8 < D / 8; ++c8) {
-    const uint4 v = *reinterpret_cast<const uint4*>(smem + L::OFF_X + (c8 >> 3) * 16384 + dl_swz(r, c8 & 7));
-    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float2 f = unpack_bf16x2(w[i]);
-      ss = fmaf(f.x, f.x, fmaf(f.y, f.y, ss));
-    }
-  }
-  slen[r] = rsqrtf(ss + 1e-6f) * (r < DC ? 1.f : rsqrtf((float)D));
   fence_proxy_async_smem();
   __syncthreads();
   if (warp == 0 && elect_one()) {
-    constexpr uint32_t id = make_idesc_bf16(128, DC, false, false);
+    constexpr uint32_t id = make_idesc_bf16(128, 128, false, false);
     const uint64_t x = make_smem_desc(smem_u32(smem + L::OFF_X), 16, 1024);
     for (int k = 0; k < ksteps; ++k) {
       const uint32_t off = ((k / 4) * 16384 + (k % 4) * 32) >> 4;
@@ -435,10 +424,19 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
   }
   if (tid >= 32 && tid < DC) b += half_sum;
   if (tid < DC) sb[tid] = b;
-  __syncthreads();
   ok = mbar_wait(bar_m, 0, abort_word) && ok;
   if (!ok) *abort_word = ERR_WAIT_MISC;
   tc_fence_after();
+  {                                                 // the diagonal: squared lengths
+    uint32_t raw[32];
+    tmem_ld_32x32(tmem + (uint32_t(warp * 32) << 16) + warp * 32, raw);
+    tmem_ld_wait();
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 32; ++i) ss = i == lane ? __uint_as_float(raw[i]) : ss;
+    slen[r] = rsqrtf(ss + 1e-6f) * (r < DC ? 1.f : rsqrtf((float)D));
+  }
+  __syncthreads();
   const int t = r & (DC - 1);
   const float bt = sb[t], mine = slen[r] * (r < DC ? sbeta[t] : 1.f);
   uint8_t* image = smem + L::OFF_I;
@@ -605,7 +603,7 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
   }
   if (warp == 0) {
     tc_fence_after();
-    tmem_dealloc(tmem, 64);
+    tmem_dealloc(tmem, 128);
   }
 }
 

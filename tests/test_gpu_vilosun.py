@@ -458,14 +458,18 @@ def test_bad_indices_are_reported_not_followed():
 
 
 # ------------------------------------------------------------------------------------------- whole models
-# Worst row, 95% of the rows and median row of a sequence.  In 16 bits a row of small heads is now and then ill-conditioned: the norm behind the
+# Worst row, nine in ten rows and median row of a sequence.  In 16 bits a row of small heads is now and then ill-conditioned: the norm behind the
 # delta rule scales an output up whose query hardly meets what is stored, its rounding with it.
 TOL = {F32: (1e-4, 5e-5, 2e-5), BF: (0.3, 0.12, 0.04)}
 
 
+def rows(got, want):
+    return torch.tensor([H.error(g[None], w[None]) for g, w in zip(got, want)])
+
+
 def agrees(got, want, dtype):
-    e = torch.tensor([H.error(g[None], w[None]) for g, w in zip(got, want)])
-    return all(float(e.quantile(q)) < t for q, t in zip((1.0, 0.95, 0.5), TOL[dtype]))
+    e = rows(got, want)
+    return all(float(e.quantile(q)) < t for q, t in zip((1.0, 0.9, 0.5), TOL[dtype]))
 
 
 def engine(cfg, ts, dtype, **kw):
@@ -501,7 +505,7 @@ def test_models_in_every_cut_and_company(name, dtype):
                          [[(0, 100), (1, 33), (3, 64), (4, 90)], [(5, 130), (0, 70), (2, 1)]]):
             got = H.feed(eng, seqs, schedule)
             for i in range(6):
-                assert agrees(got[i], want[i], dtype), (i, dtype, schedule[:3], H.error(got[i], want[i]))
+                assert agrees(got[i], want[i], dtype), (i, dtype, schedule[:3], rows(got[i], want[i]).sort().values[-12:])
             assert eng.cache.allocator.free == 1024 // page and eng.cache.slot_allocator.free == 4
 
 
