@@ -39,12 +39,31 @@ struct GroupStepParams {
   uint32_t* status;
 };
 
-// A thread holds KEEP pieces of VEC columns: columns c0 + j * step.  SEG lanes next to each other (a power of two) are inside one group.
+template <int VEC, typename T>
+__device__ __forceinline__ void gs_load(const T* p, float (&f)[VEC]) {
+  if constexpr (VEC == 8) unpack(load_piece(p), f);
+  else load_vec<VEC>(p, f);
+}
+template <int VEC, typename T>
+__device__ __forceinline__ void gs_store(T* p, const float (&f)[VEC]) {
+  if constexpr (VEC == 8) store8(p, f);
+  else store_vec<VEC>(p, f);
+}
+template <typename T>
+__device__ __forceinline__ float gs_gated(float u, float g) {
+  if constexpr (sizeof(T) == 4) return u / (1.f + expf(-g));
+  else return __fdividef(u, 1.f + __expf(-g));
+}
+
+// A thread holds KEEP pieces of VEC columns: columns c0 + j * step.  1 << seg lanes next to each other are inside one group.
 template <typename T, int VEC, int KEEP>
 __global__ void __launch_bounds__(512) group_step_kernel(const GroupStepParams p, const int seg) {
   pdl_sync();
-  extern __shared__ float gsum[];                        // [2][d / (seg * VEC)] sums of squares
+  extern __shared__ float gsum[];                        // [2][d / (VEC << seg)] sums of squares
   const int row = blockIdx.x, step = blockDim.x * VEC, c0 = threadIdx.x * VEC;
+  constexpr int SHIFT = VEC == 8 ? 3 : (VEC == 4 ? 2 : 0);
+  const int lanes = 1 << seg, size = p.d / p.groups, per_group = size >> (seg + SHIFT), segs = p.d >> (seg + SHIFT);
+  const float share = 1.f / (float)size;
   long long src = row;
   if (p.row_index != nullptr) {
     src = p.row_index[row];
@@ -54,43 +73,53 @@ __global__ void __launch_bounds__(512) group_step_kernel(const GroupStepParams p
     }
   }
   float* xr = p.x + src * p.d;
-  const int size = p.d / p.groups, per_group = size / (seg * VEC), segs = p.d / (seg * VEC);
-  // norm of the thread's pieces f in place: f / rms of the group * w
-  auto norm = [&](float (&f)[KEEP][VEC], const Raw<T, VEC> (&w)[KEEP], float* sums) __attribute__((always_inline)) {
+  // everything that is read in any case is requested first
+  float x[KEEP][VEC];
+  Raw<T, VEC> gate[KEEP], post[KEEP], w[KEEP], raw[KEEP];
+  auto request = [&](const T* from, Raw<T, VEC> (&to)[KEEP]) __attribute__((always_inline)) {
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j)
+      if (c0 + j * step < p.d) to[j] = *reinterpret_cast<const Raw<T, VEC>*>(from + c0 + j * step);
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) x[j][i] = 0.f;
+    if (p.tokens == nullptr && c0 + j * step < p.d) gs_load<VEC>(xr + c0 + j * step, x[j]);
+  }
+  if (p.y != nullptr) {
+    request(reinterpret_cast<const T*>(p.gate) + src * p.ld_gate, gate);
+    if (p.ypos == nullptr) request(reinterpret_cast<const T*>(p.y) + src * p.ld_y, raw);
+    request(reinterpret_cast<const T*>(p.w_post), post);
+  }
+  if (p.h != nullptr) request(reinterpret_cast<const T*>(p.w), w);
+  int first[KEEP];                                       // first sum of a piece's group
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) first[j] = (c0 + j * step) / size * per_group;
+  // norm of the thread's pieces f in place: f / rms of the group * weight
+  auto norm = [&](float (&f)[KEEP][VEC], const Raw<T, VEC> (&weight)[KEEP], float* sums) __attribute__((always_inline)) {
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
       float ss = 0.f;
 #pragma unroll
       for (int i = 0; i < VEC; ++i) ss = fmaf(f[j][i], f[j][i], ss);
-      for (int o = seg >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
       const int c = c0 + j * step;
-      if (c < p.d && (threadIdx.x & (seg - 1)) == 0) sums[c / (seg * VEC)] = ss;
+      if (c < p.d && (threadIdx.x & (lanes - 1)) == 0) sums[c >> (seg + SHIFT)] = ss;
     }
     __syncthreads();
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
-      const int c = c0 + j * step;
-      if (c >= p.d) break;
-      const float* mine = sums + c / size * per_group;
+      if (c0 + j * step >= p.d) break;
       float ss = 0.f;
-      for (int k = 0; k < per_group; ++k) ss += mine[k];
-      const float r = rsqrtf(ss / (float)size + p.eps);
+      for (int k = 0; k < per_group; ++k) ss += sums[first[j] + k];
+      const float r = rsqrtf(fmaf(ss, share, p.eps));
       float g[VEC];
-      load_vec<VEC>(w[j].v, g);
+      gs_load<VEC>(weight[j].v, g);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) f[j][i] *= r * g[i];
     }
   };
-  auto weights = [&](const void* from, Raw<T, VEC> (&w)[KEEP]) __attribute__((always_inline)) {
-#pragma unroll
-    for (int j = 0; j < KEEP; ++j)
-      if (c0 + j * step < p.d) w[j] = *reinterpret_cast<const Raw<T, VEC>*>(reinterpret_cast<const T*>(from) + c0 + j * step);
-  };
-  float x[KEEP][VEC];
-#pragma unroll
-  for (int j = 0; j < KEEP; ++j)
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) x[j][i] = 0.f;
   if (p.tokens != nullptr) {
     long long tok = p.tokens[row];
     if (tok < 0 || tok >= p.vocab) {
@@ -119,51 +148,37 @@ __global__ void __launch_bounds__(512) group_step_kernel(const GroupStepParams p
       float b[VEC];
 #pragma unroll
       for (int i = 0; i < VEC; ++i) b[i] = 0.f;
-      load_vec<VEC>(er + c, x[j]);
-      if (br != nullptr) load_vec<VEC>(br + c, b);
+      gs_load<VEC>(er + c, x[j]);
+      if (br != nullptr) gs_load<VEC>(br + c, b);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) x[j][i] = fmaf(x[j][i], p.scale, b[i]);
-      store_vec<VEC>(xr + c, x[j]);
+      gs_store<VEC>(xr + c, x[j]);
     }
-  } else {
-#pragma unroll
-    for (int j = 0; j < KEEP; ++j)
-      if (c0 + j * step < p.d) load_vec<VEC>(xr + c0 + j * step, x[j]);
   }
-  Raw<T, VEC> w[KEEP];
   if (p.y != nullptr) {
     float u[KEEP][VEC];
 #pragma unroll
     for (int j = 0; j < KEEP; ++j)
 #pragma unroll
       for (int i = 0; i < VEC; ++i) u[j][i] = 0.f;
-    Raw<T, VEC> gate[KEEP];
-    const T* gr = reinterpret_cast<const T*>(p.gate) + src * p.ld_gate;
-#pragma unroll
-    for (int j = 0; j < KEEP; ++j)
-      if (c0 + j * step < p.d) gate[j] = *reinterpret_cast<const Raw<T, VEC>*>(gr + c0 + j * step);
-    weights(p.w_post, w);
     if (p.ypos == nullptr) {
-      const T* yr = reinterpret_cast<const T*>(p.y) + src * p.ld_y;
 #pragma unroll
       for (int j = 0; j < KEEP; ++j)
-        if (c0 + j * step < p.d) load_vec<VEC>(yr + c0 + j * step, u[j]);
+        if (c0 + j * step < p.d) gs_load<VEC>(raw[j].v, u[j]);
     } else {
-#pragma unroll 1
+#pragma unroll 2
       for (int k = 0; k < p.ytop; ++k) {
         const int pos = p.ypos[src * p.ytop + k];
         if (pos < 0 || pos >= p.y_rows) continue;        // a padding row of the batch
         const float a = p.yweight[src * p.ytop + k];
-        const T* yr = reinterpret_cast<const T*>(p.y) + (long long)pos * p.ld_y;
-        float f[KEEP][VEC];
-#pragma unroll
-        for (int j = 0; j < KEEP; ++j)
-          if (c0 + j * step < p.d) load_vec<VEC>(yr + c0 + j * step, f[j]);
+        request(reinterpret_cast<const T*>(p.y) + (long long)pos * p.ld_y, raw);
 #pragma unroll
         for (int j = 0; j < KEEP; ++j)
           if (c0 + j * step < p.d) {
+            float f[VEC];
+            gs_load<VEC>(raw[j].v, f);
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) u[j][i] = fmaf(a, f[j][i], u[j][i]);
+            for (int i = 0; i < VEC; ++i) u[j][i] = fmaf(a, f[i], u[j][i]);
           }
       }
     }
@@ -171,26 +186,25 @@ __global__ void __launch_bounds__(512) group_step_kernel(const GroupStepParams p
     for (int j = 0; j < KEEP; ++j)
       if (c0 + j * step < p.d) {
         float g[VEC];
-        load_vec<VEC>(gate[j].v, g);
+        gs_load<VEC>(gate[j].v, g);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) u[j][i] = u[j][i] / (1.f + (sizeof(T) == 4 ? expf(-g[i]) : __expf(-g[i])));
+        for (int i = 0; i < VEC; ++i) u[j][i] = gs_gated<T>(u[j][i], g[i]);
       }
-    norm(u, w, gsum);
+    norm(u, post, gsum);
 #pragma unroll
     for (int j = 0; j < KEEP; ++j)
       if (c0 + j * step < p.d) {
 #pragma unroll
         for (int i = 0; i < VEC; ++i) x[j][i] += u[j][i];
-        if (p.row_index == nullptr) store_vec<VEC>(xr + c0 + j * step, x[j]);
+        if (p.row_index == nullptr) gs_store<VEC>(xr + c0 + j * step, x[j]);
       }
   }
   if (p.h == nullptr) return;
-  weights(p.w, w);
   norm(x, w, gsum + segs);
   T* hr = reinterpret_cast<T*>(p.h) + (long long)row * p.ld_h;
 #pragma unroll
   for (int j = 0; j < KEEP; ++j)
-    if (c0 + j * step < p.d) store_vec<VEC>(hr + c0 + j * step, x[j]);
+    if (c0 + j * step < p.d) gs_store<VEC>(hr + c0 + j * step, x[j]);
 }
 
 // The last token of every portion into its sequence's state.
@@ -205,18 +219,18 @@ __global__ void carry_tokens_kernel(const long long* tokens, const int* cu, cons
 template <typename T, int VEC>
 static int launch_group_step(const GroupStepParams& p, cudaStream_t st) {
   const int pieces = p.d / VEC, size = p.d / p.groups;
-  int seg = 1;
-  while (seg < 32 && size % (2 * seg * VEC) == 0) seg *= 2;
-  const int want = p.rows >= 148 * 8 ? (pieces + 1) / 2 : pieces;      // many rows share an SM, few have all of its threads
+  int seg = 0;
+  while (seg < 5 && size % ((2 << seg) * VEC) == 0) ++seg;
+  const int want = p.rows >= 148 * 8 && VEC < 8 ? (pieces + 1) / 2 : pieces;      // many rows share an SM, few have all of its threads
   int threads = (want + 31) / 32 * 32;
   if (threads > 512) threads = 512;
   const int keep = (pieces + threads - 1) / threads;
-  const size_t smem = 2ull * (p.d / (seg * VEC)) * sizeof(float);
+  const size_t smem = 2ull * (p.d / (VEC << seg)) * sizeof(float);
   if (smem > 48 * 1024) return -12;
   if (keep <= 1) launch_dep(group_step_kernel<T, VEC, 1>, p.rows, threads, smem, st, p, seg);
   else if (keep <= 2) launch_dep(group_step_kernel<T, VEC, 2>, p.rows, threads, smem, st, p, seg);
   else if (keep <= 4) launch_dep(group_step_kernel<T, VEC, 4>, p.rows, threads, smem, st, p, seg);
-  else if (keep <= 16) launch_dep(group_step_kernel<T, VEC, 16>, p.rows, threads, smem, st, p, seg);
+  else if (VEC < 8 && keep <= 16) launch_dep(group_step_kernel<T, VEC < 8 ? VEC : 4, 16>, p.rows, threads, smem, st, p, seg);
   else return -12;
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
@@ -267,8 +281,10 @@ extern "C" int b200_group_step(float* x, const GroupStart* start, const GroupSub
                          reinterpret_cast<uintptr_t>(p.y) | reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.w_post) |
                          reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(h);
   const bool vec = (d / groups) % 4 == 0 && (p.ld_y | p.ld_gate | ld_h) % 4 == 0 && (ptrs & 15) == 0;
+  const bool wide = vec && (d / groups) % 8 == 0 && (p.ld_y | p.ld_gate | ld_h) % 8 == 0 && d <= 8192 && rows >= 148 * 4;
   int r;
   if (f32) r = vec ? launch_group_step<float, 4>(p, st) : launch_group_step<float, 1>(p, st);
+  else if (wide) r = launch_group_step<__nv_bfloat16, 8>(p, st);
   else r = vec ? launch_group_step<__nv_bfloat16, 4>(p, st) : launch_group_step<__nv_bfloat16, 1>(p, st);
   if (r == 0 && start != nullptr && start->bigram != nullptr && start->portions > 0) {
     launch_dep(carry_tokens_kernel, (start->portions + 127) / 128, 128, 0, st, start->tokens + start->n_single, start->cu,

@@ -18,7 +18,7 @@ struct ConvParams {
   const int* row_seq;          // sequence of a row, less seq0; null: row i is sequence i
   const int* cu;               // (seqs + 1) rows of each sequence; null: one row each
   const int* positions;        // per row
-  int seq0, seqs, rows, channels, taps, num_slots, run;      // run: consecutive rows of a thread
+  int seq0, seqs, rows, channels, taps, num_slots;
   void* y;                     // plain: (rows, ld_y)
   long long ld_y;
   int silu;
@@ -45,113 +45,46 @@ __device__ __forceinline__ void conv_store(T* p, const float (&f)[VEC]) {
   else from_f(*p, f[0]);
 }
 
-// A thread owns VEC channels and walks `run` rows.  TAPS > 0: the filter and the rows in front stay in registers.
-template <typename T, int VEC, int TAPS, bool ATTEND>
-__global__ void __launch_bounds__(256) short_conv_kernel(const ConvParams p) {
-  pdl_sync();
-  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
-  if (c >= p.channels) return;
-  const int r0 = blockIdx.x * p.run, r1 = min(p.rows, r0 + p.run);
-  const int taps = TAPS > 0 ? TAPS : p.taps;
-  constexpr int HELD = TAPS > 0 ? TAPS : 1;
-  const T* u = reinterpret_cast<const T*>(p.u) + c;
-  const T* w = reinterpret_cast<const T*>(p.w) + c;
-  float filter[HELD][VEC], before[HELD][VEC];        // before[d]: the row d in front
-  if (TAPS > 0) {
-#pragma unroll
-    for (int j = 0; j < HELD; ++j) conv_load<VEC>(w + (long long)j * p.channels, filter[j]);
+__device__ __forceinline__ float conv_silu(float y, float) { return y / (1.f + expf(-y)); }                           // fp32 activations
+__device__ __forceinline__ float conv_silu(float y, __nv_bfloat16) { return __fdividef(y, 1.f + __expf(-y)); }
+
+// Where VEC channels from c on go (attention), and what becomes of them.
+template <typename T, int VEC>
+struct ConvTarget {
+  bool query, key;
+  int head, e, len, pitch;
+  float temp;
+  __device__ __forceinline__ ConvTarget(const ConvParams& p, int c, bool attend) {
+    if (!attend) return;
+    const GroupedShape& s = p.s;
+    const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim;
+    query = c < nq;
+    key = !query && c < nq + nk;
+    const int at = query ? c : (key ? c - nq : c - nq - nk);
+    len = query || key ? s.dim : s.vdim;
+    head = at / len;
+    e = at - head * len;
+    pitch = query ? s.qp : (key ? s.kp : s.vp);
+    temp = query ? p.temp[head] : 1.f;
   }
-  // where these channels go (attention)
-  const GroupedShape& s = p.s;
-  const int nq = s.heads * s.dim, nk = s.kv_heads * s.dim;
-  const bool query = c < nq, key = !query && c < nq + nk;
-  const int at = query ? c : (key ? c - nq : c - nq - nk), len = query || key ? s.dim : s.vdim;
-  const int head = ATTEND ? at / len : 0, e = at - head * len;
-  const float temp = ATTEND && query ? p.temp[head] : 1.f;
-  for (int row = r0; row < r1; ++row) {
-    const int seq = p.row_seq != nullptr ? p.row_seq[row] - p.seq0 : row;
-    if ((unsigned)seq >= (unsigned)p.seqs) {
-      report_bad_arg(p.status, 30);
-      continue;
-    }
-    const int first = p.cu != nullptr ? p.cu[seq] : row, pos = p.positions[row];
-    int slot = p.state_slots[seq];
-    if (slot >= p.num_slots) {
-      report_bad_arg(p.status, 31);
-      slot = -1;
-    }
-    T* ring = reinterpret_cast<T*>(p.ring) + (long long)max(slot, 0) * taps * p.channels + c;
-    auto earlier = [&](int d, float (&f)[VEC]) __attribute__((always_inline)) {
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) f[i] = 0.f;
-      if (row - d >= first) conv_load<VEC>(u + (long long)(row - d) * p.ld_u, f);
-      else if (pos >= d && slot >= 0) conv_load<VEC>(ring + (long long)((pos - d) % taps) * p.channels, f);
-    };
-    float now[VEC], y[VEC];
-    conv_load<VEC>(u + (long long)row * p.ld_u, now);
-    if (TAPS > 0) {
-      if (row == r0 || row == first) {
-#pragma unroll
-        for (int d = 1; d < HELD; ++d) earlier(d, before[d]);
-      }
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) y[i] = filter[HELD - 1][i] * now[i];
-#pragma unroll
-      for (int d = 1; d < HELD; ++d)
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) y[i] = fmaf(filter[HELD - 1 - d][i], before[d][i], y[i]);
-#pragma unroll
-      for (int d = HELD - 1; d > 1; --d)
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) before[d][i] = before[d - 1][i];
-      if (HELD > 1) {
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) before[HELD > 1 ? 1 : 0][i] = now[i];
-      }
-    } else {
-      float g[VEC], f[VEC];
-      conv_load<VEC>(w + (long long)(taps - 1) * p.channels, g);
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) y[i] = g[i] * now[i];
-      for (int d = 1; d < taps; ++d) {
-        conv_load<VEC>(w + (long long)(taps - 1 - d) * p.channels, g);
-        earlier(d, f);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) y[i] = fmaf(g[i], f[i], y[i]);
-      }
-    }
-    if (p.cu == nullptr && slot >= 0) conv_store<VEC>(ring + (long long)(pos % taps) * p.channels, now);
-    if (!ATTEND) {
-      if (p.silu) {
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) y[i] = y[i] / (1.f + expf(-y[i]));
-      }
-      conv_store<VEC>(reinterpret_cast<T*>(p.y) + (long long)row * p.ld_y + c, y);
-      continue;
-    }
+  // v_first of the same token, where values are mixed
+  __device__ __forceinline__ const T* first(const ConvParams& p, long long to) const {
+    return reinterpret_cast<const T*>(p.first) + to * p.first_width + p.first_off + head * p.first_pitch + e;
+  }
+  __device__ __forceinline__ bool mixes(const ConvParams& p) const { return !query && !key && p.first != nullptr; }
+  __device__ __forceinline__ void put(const ConvParams& p, int row, long long to, const float (&v1)[VEC], float (&y)[VEC]) const {
+    const GroupedShape& s = p.s;
     T* dst;
-    int pitch;
     if (query) {
 #pragma unroll
       for (int i = 0; i < VEC; ++i) y[i] *= temp;
       dst = reinterpret_cast<T*>(p.q) + ((long long)row * s.heads + head) * s.qp;
-      pitch = s.qp;
     } else {
-      const long long to = p.slots[row];
-      if (to < 0) continue;                              // padding row of the batch
-      if (to >= p.cache_slots) {
-        report_bad_arg(p.status, 32);
-        continue;
-      }
-      T* line = reinterpret_cast<T*>(p.cache) + to * (long long)(s.kv_heads * (s.kp + s.vp));
-      if (!key && p.first != nullptr) {
-        float f[VEC];
-        conv_load<VEC>(reinterpret_cast<const T*>(p.first) + to * p.first_width + p.first_off + head * p.first_pitch + e, f);
+      if (mixes(p)) {
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) y[i] = (1.f - p.mix) * y[i] + p.mix * f[i];
+        for (int i = 0; i < VEC; ++i) y[i] = (1.f - p.mix) * y[i] + p.mix * v1[i];
       }
-      dst = line + (key ? head * s.kp : s.kv_heads * s.kp + head * s.vp);
-      pitch = key ? s.kp : s.vp;
+      dst = reinterpret_cast<T*>(p.cache) + to * (long long)(s.kv_heads * (s.kp + s.vp)) + (key ? head * s.kp : s.kv_heads * s.kp + head * s.vp);
     }
     conv_store<VEC>(dst + e, y);
     if (e + VEC == len) {                                // the pad behind the vector
@@ -160,6 +93,154 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const ConvParams p) {
       for (int i = 0; i < VEC; ++i) z[i] = 0.f;
       for (int k = len; k + VEC <= pitch; k += VEC) conv_store<VEC>(dst + k, z);
     }
+  }
+};
+
+// y = the convolution of VEC channels of one row; false where an index is bad.
+template <typename T, int VEC>
+__device__ __forceinline__ bool conv_row(const ConvParams& p, int c, int row, float (&y)[VEC]) {
+  const int taps = p.taps;
+  const T* u = reinterpret_cast<const T*>(p.u) + (long long)row * p.ld_u + c;
+  const T* w = reinterpret_cast<const T*>(p.w) + c;
+  float now[VEC], g[VEC];
+  conv_load<VEC>(u, now);
+  conv_load<VEC>(w + (long long)(taps - 1) * p.channels, g);
+  const int seq = p.row_seq != nullptr ? p.row_seq[row] - p.seq0 : row, pos = p.positions[row];
+  if ((unsigned)seq >= (unsigned)p.seqs) {
+    report_bad_arg(p.status, 30);
+    return false;
+  }
+  const int first = p.cu != nullptr ? p.cu[seq] : row;
+  int slot = p.state_slots[seq];
+  if (slot >= p.num_slots) {
+    report_bad_arg(p.status, 31);
+    slot = -1;
+  }
+  T* ring = reinterpret_cast<T*>(p.ring) + (long long)max(slot, 0) * taps * p.channels + c;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) y[i] = g[i] * now[i];
+#pragma unroll 3
+  for (int d = 1; d < taps; ++d) {
+    float f[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) f[i] = 0.f;
+    if (row - d >= first) conv_load<VEC>(u - d * p.ld_u, f);
+    else if (pos >= d && slot >= 0) conv_load<VEC>(ring + (long long)((pos - d) % taps) * p.channels, f);
+    conv_load<VEC>(w + (long long)(taps - 1 - d) * p.channels, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) y[i] = fmaf(g[i], f[i], y[i]);
+  }
+  if (p.cu == nullptr && slot >= 0) conv_store<VEC>(ring + (long long)(pos % taps) * p.channels, now);
+  return true;
+}
+
+// What becomes of a row's y: stored, or sent where attention wants it (v1: the values to mix in).
+template <typename T, int VEC, bool ATTEND>
+__device__ __forceinline__ void conv_finish(const ConvParams& p, const ConvTarget<T, VEC>& at, int c, int row, long long to, const float (&v1)[VEC],
+                                            float (&y)[VEC]) {
+  if constexpr (ATTEND) {
+    if (!at.query && to < 0) return;                     // padding row of the batch
+    if (!at.query && to >= p.cache_slots) {
+      report_bad_arg(p.status, 32);
+      return;
+    }
+    at.put(p, row, to, v1, y);
+  } else {
+    if (p.silu) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) y[i] = conv_silu(y[i], T());
+    }
+    conv_store<VEC>(reinterpret_cast<T*>(p.y) + (long long)row * p.ld_y + c, y);
+  }
+}
+
+// One row per thread and piece of VEC channels: any number of taps, single rows (which leave their input in the ring) and portions.
+template <typename T, int VEC, bool ATTEND>
+__global__ void __launch_bounds__(256) short_conv_kernel(const ConvParams p) {
+  pdl_sync();
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC, row = blockIdx.x;
+  if (c >= p.channels) return;
+  const long long to = ATTEND ? p.slots[row] : 0;
+  const ConvTarget<T, VEC> at(p, c, ATTEND);
+  float y[VEC], v1[VEC];
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) v1[i] = 0.f;
+  if (ATTEND && at.mixes(p) && to >= 0 && to < p.cache_slots) conv_load<VEC>(at.first(p, to), v1);
+  if (conv_row<T, VEC>(p, c, row, y)) conv_finish<T, VEC, ATTEND>(p, at, c, row, to, v1, y);
+}
+
+template <bool ATTEND>
+constexpr int CONV_RUN = ATTEND ? 4 : 8;
+
+// CONV_RUN rows of portions per thread and piece of 8 channels: every row is requested once, before the first is worked on, and stays in
+// registers for the rows behind it.  Where a sequence ends among them, they are taken one by one.
+template <typename T, int TAPS, bool ATTEND>
+__global__ void __launch_bounds__(256) short_conv_run_kernel(const ConvParams p) {
+  pdl_sync();
+  constexpr int RUN = CONV_RUN<ATTEND>, H = TAPS - 1;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8, r0 = blockIdx.x * RUN, n = min(RUN, p.rows - r0);
+  if (c >= p.channels) return;
+  const T* u = reinterpret_cast<const T*>(p.u) + c;
+  Piece<T> in[H + RUN], filter[TAPS], mixed[ATTEND ? RUN : 1];
+  long long to[RUN];
+  const ConvTarget<T, 8> at(p, c, ATTEND);
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    if (i < n) in[H + i] = load_piece(u + (long long)(r0 + i) * p.ld_u);
+    to[i] = ATTEND && i < n ? p.slots[r0 + i] : -1;
+  }
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) filter[j] = load_piece(reinterpret_cast<const T*>(p.w) + (long long)j * p.channels + c);
+  const int seq = p.row_seq[r0] - p.seq0;
+  if (seq == p.row_seq[r0 + n - 1] - p.seq0 && (unsigned)seq < (unsigned)p.seqs) {
+    const int first = p.cu[seq], pos = p.positions[r0];
+    int slot = p.state_slots[seq];
+    if (slot >= p.num_slots) {
+      report_bad_arg(p.status, 31);
+      slot = -1;
+    }
+    const T* ring = reinterpret_cast<const T*>(p.ring) + (long long)max(slot, 0) * TAPS * p.channels + c;
+#pragma unroll
+    for (int d = 1; d <= H; ++d) {
+#pragma unroll
+      for (int k = 0; k < (int)sizeof(T) / 2; ++k) in[H - d].v[k] = make_uint4(0, 0, 0, 0);
+      if (r0 - d >= first) in[H - d] = load_piece(u + (long long)(r0 - d) * p.ld_u);
+      else if (pos >= d && slot >= 0) in[H - d] = load_piece(ring + (long long)((pos - d) % TAPS) * p.channels);
+    }
+    if constexpr (ATTEND) {
+      if (at.mixes(p)) {
+#pragma unroll
+        for (int i = 0; i < RUN; ++i)
+          if (to[i] >= 0 && to[i] < p.cache_slots) mixed[i] = load_piece(at.first(p, to[i]));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) {
+      if (i >= n) break;
+      float y[8], g[8], f[8], v1[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) y[k] = v1[k] = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        unpack(filter[j], g);
+        unpack(in[i + j], f);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) y[k] = fmaf(g[k], f[k], y[k]);
+      }
+      if constexpr (ATTEND) {
+        if (at.mixes(p) && to[i] >= 0 && to[i] < p.cache_slots) unpack(mixed[i], v1);
+      }
+      conv_finish<T, 8, ATTEND>(p, at, c, r0 + i, to[i], v1, y);
+    }
+    return;
+  }
+  for (int i = 0; i < n; ++i) {
+    float y[8], v1[8];
+    const long long line = ATTEND ? p.slots[r0 + i] : 0;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v1[k] = 0.f;
+    if (ATTEND && at.mixes(p) && line >= 0 && line < p.cache_slots) conv_load<8>(at.first(p, line), v1);
+    if (conv_row<T, 8>(p, c, r0 + i, y)) conv_finish<T, 8, ATTEND>(p, at, c, r0 + i, line, v1, y);
   }
 }
 
@@ -180,16 +261,17 @@ __global__ void __launch_bounds__(256) short_conv_carry_kernel(const ConvParams 
 }
 
 template <typename T, bool ATTEND>
-static void launch_conv(ConvParams& p, bool vec, cudaStream_t st) {
+static void launch_conv(const ConvParams& p, bool vec, cudaStream_t st) {
   const int pieces = p.channels / (vec ? 8 : 1);
-  p.run = p.cu == nullptr || (long long)p.rows * pieces < 148ll * 2048 * 4 ? 1 : 8;
   const int threads = pieces >= 256 ? 256 : (pieces + 31) / 32 * 32;
-  const dim3 grid((p.rows + p.run - 1) / p.run, (pieces + threads - 1) / threads);
-  if (!vec) launch_dep(short_conv_kernel<T, 1, 0, ATTEND>, grid, threads, 0, st, p);
-  else if (p.taps == 2) launch_dep(short_conv_kernel<T, 8, 2, ATTEND>, grid, threads, 0, st, p);
-  else if (p.taps == 3) launch_dep(short_conv_kernel<T, 8, 3, ATTEND>, grid, threads, 0, st, p);
-  else if (p.taps == 4) launch_dep(short_conv_kernel<T, 8, 4, ATTEND>, grid, threads, 0, st, p);
-  else launch_dep(short_conv_kernel<T, 8, 0, ATTEND>, grid, threads, 0, st, p);
+  const unsigned gy = (pieces + threads - 1) / threads;
+  const bool run = vec && p.cu != nullptr && p.taps >= 2 && p.taps <= 4 && (long long)p.rows * pieces >= 148ll * 2048 * 2;
+  const dim3 grid(run ? (p.rows + CONV_RUN<ATTEND> - 1) / CONV_RUN<ATTEND> : p.rows, gy);
+  if (!vec) launch_dep(short_conv_kernel<T, 1, ATTEND>, grid, threads, 0, st, p);
+  else if (!run) launch_dep(short_conv_kernel<T, 8, ATTEND>, grid, threads, 0, st, p);
+  else if (p.taps == 2) launch_dep(short_conv_run_kernel<T, 2, ATTEND>, grid, threads, 0, st, p);
+  else if (p.taps == 3) launch_dep(short_conv_run_kernel<T, 3, ATTEND>, grid, threads, 0, st, p);
+  else launch_dep(short_conv_run_kernel<T, 4, ATTEND>, grid, threads, 0, st, p);
   if (p.cu != nullptr && p.taps > 1)
     launch_dep(short_conv_carry_kernel<T>, dim3(p.seqs, p.channels >= 1024 ? 4 : 1), 256, 0, st, p);
 }

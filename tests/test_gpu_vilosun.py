@@ -137,11 +137,13 @@ def ring_before(u, start, taps, slots, slot, seed=0):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("channels,taps", [(13, 3), (40, 1), (40, 2), (96, 3), (2056, 4), (64, 7), (3000, 5)])
-def test_short_convolution_in_portions_and_single_rows(dtype, channels, taps):
+@pytest.mark.parametrize("channels,taps,many", [(13, 3, 0), (40, 1, 0), (40, 2, 0), (96, 3, 0), (2056, 4, 0), (64, 7, 0), (3000, 5, 0), (8192, 4, 400), (8200, 3, 500),
+                                                  (16384, 2, 300)])
+def test_short_convolution_in_portions_and_single_rows(dtype, channels, taps, many):
+    """``many``: enough rows for the kernel that walks eight of them."""
     mo, tol = mops(), 1e-2 if dtype == BF else 1e-5
     w = randn(taps, channels, seed=1, dtype=dtype)
-    spans = [(0, 1), (0, 2), (5, 2), (3, 130), (64, 1), (1, 9), (0, 40), (2, 3)]
+    spans = [(0, 1), (0, 2), (5, 2), (3, 130 + many), (64, 1), (1, 9), (0, 40), (2, 3)]
     us = [randn(a + n, channels, seed=10 + i, dtype=dtype) for i, (a, n) in enumerate(spans)]
     slots, at = [6, 0, 2, 9, 1, 4, 3, 8], None
     ring = torch.full((10, taps, channels), float("nan"), dtype=dtype, device="cuda")
