@@ -181,6 +181,31 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) delta_step_kernel(const D
     load_vec<4>(wa + threadIdx.x * 4, ha);
     load_vec<4>(wb + threadIdx.x * 4, hb);
   }
+  // q, k, v of this head, 2 D + E channels: those of a thread's first two, with up to four taps, are requested before the state as well
+  const T* cr = reinterpret_cast<const T*>(p.c) + (long long)seq * p.ld_c;
+  const int channels = 2 * p.kv_heads * D + p.heads * E, mine_n = 2 * D + E;
+  const T* filter = reinterpret_cast<const T*>(p.filter);
+  T* ring = reinterpret_cast<T*>(p.ring) + (long long)slot * p.taps * channels;
+  auto channel = [&](int i) {
+    return i < D ? hk * D + i : (i < 2 * D ? (p.kv_heads + hk) * D + i - D : 2 * p.kv_heads * D + h * E + i - 2 * D);
+  };
+  constexpr int AHEAD = 2, TAPS = 4;
+  T raw[AHEAD], past[AHEAD][TAPS], weight[AHEAD][TAPS];
+#pragma unroll
+  for (int k = 0; k < AHEAD; ++k) {
+    const int i = threadIdx.x + k * 256;
+    if (i >= mine_n) break;
+    const int ch = channel(i);
+    raw[k] = cr[ch];
+#pragma unroll
+    for (int d = 0; d < TAPS; ++d) {
+      from_f(past[k][d], 0.f);
+      if (d < p.taps) weight[k][d] = filter[(long long)(p.taps - 1 - d) * channels + ch];
+      if (d > 0 && d < p.taps && pos >= d) past[k][d] = ring[(long long)((pos - d) % p.taps) * channels + ch];
+    }
+  }
+  const T* gr = reinterpret_cast<const T*>(p.gate) + (long long)seq * p.ld_gate + h * E;
+  const float z0 = threadIdx.x < E ? to_f(gr[threadIdx.x]) : 0.f, w0 = threadIdx.x < E ? to_f(reinterpret_cast<const T*>(p.weight)[threadIdx.x]) : 0.f;
   float4 s[NR];
 #pragma unroll
   for (int j = 0; j < NR; ++j) {
@@ -188,24 +213,33 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) delta_step_kernel(const D
     s[j] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (on && d < D && !fresh) s[j] = __ldcs(S + (long long)d * groups);
   }
-  // ---- q, k, v of this head: 2 D + E channels
-  const T* cr = reinterpret_cast<const T*>(p.c) + (long long)seq * p.ld_c;
-  const int channels = 2 * p.kv_heads * D + p.heads * E;
-  const T* filter = reinterpret_cast<const T*>(p.filter);
-  T* ring = reinterpret_cast<T*>(p.ring) + (long long)slot * p.taps * channels;
   float qq = 0.f, kk = 0.f;
-  for (int i = threadIdx.x; i < 2 * D + E; i += 256) {
-    const int ch = i < D ? hk * D + i : (i < 2 * D ? (p.kv_heads + hk) * D + i - D : 2 * p.kv_heads * D + h * E + i - 2 * D);
-    const T raw = cr[ch];
-    float f = to_f(raw);
+  auto place = [&](int i, T now, float f) {                // f: the convolution, or the channel itself
     if (p.taps > 0) {
-      f *= to_f(filter[(long long)(p.taps - 1) * channels + ch]);
-      for (int d = 1; d < p.taps; ++d)
-        if (pos >= d) f = fmaf(to_f(filter[(long long)(p.taps - 1 - d) * channels + ch]), to_f(ring[(long long)((pos - d) % p.taps) * channels + ch]), f);
-      if (i >= 2 * D || h == hk * rep) ring[(long long)(pos % p.taps) * channels + ch] = raw;      // nobody reads this row in this step
+      if (i >= 2 * D || h == hk * rep) ring[(long long)(pos % p.taps) * channels + channel(i)] = now;      // nobody reads this row in this step
       f = f / (1.f + expf(-f));
     }
     qs[i] = f;                                       // qs | ks | vs
+  };
+#pragma unroll
+  for (int k = 0; k < AHEAD; ++k) {
+    const int i = threadIdx.x + k * 256;
+    if (i >= mine_n || p.taps > TAPS) break;
+    float f = to_f(raw[k]);
+    if (p.taps > 0) f *= to_f(weight[k][0]);
+#pragma unroll
+    for (int d = 1; d < TAPS; ++d)
+      if (d < p.taps) f = fmaf(to_f(weight[k][d]), to_f(past[k][d]), f);
+    place(i, raw[k], f);
+  }
+  for (int i = threadIdx.x + (p.taps > TAPS ? 0 : AHEAD * 256); i < mine_n; i += 256) {
+    const int ch = channel(i);
+    const T now = cr[ch];
+    float f = to_f(now);
+    if (p.taps > 0) f *= to_f(filter[(long long)(p.taps - 1) * channels + ch]);
+    for (int d = 1; d < p.taps; ++d)
+      if (pos >= d) f = fmaf(to_f(filter[(long long)(p.taps - 1 - d) * channels + ch]), to_f(ring[(long long)((pos - d) % p.taps) * channels + ch]), f);
+    place(i, now, f);
   }
   float za = 0.f, zb = 0.f;
   if (p.ab != nullptr) {
@@ -294,12 +328,10 @@ __global__ void __launch_bounds__(256, NR > 8 ? 2 : 3) delta_step_kernel(const D
       __stcs(S + (long long)d * groups, s[j]);
     }
   }
-  const T* gr = reinterpret_cast<const T*>(p.gate) + (long long)seq * p.ld_gate + h * E;
-  const T* w = reinterpret_cast<const T*>(p.weight);
   n = 0;
   for (int c = threadIdx.x; c < E && n < 4; c += 256, ++n) {
-    const float z = to_f(gr[c]);
-    from_f(y[c], mine[n] * inv * to_f(w[c]) * z * sigmoid_f(z));
+    const float z = n == 0 ? z0 : to_f(gr[c]), w = n == 0 ? w0 : to_f(reinterpret_cast<const T*>(p.weight)[c]);
+    from_f(y[c], mine[n] * inv * w * z * sigmoid_f(z));
   }
 }
 

@@ -177,7 +177,7 @@ def _decode_kernels(s, t, b):
         h, wab, filt, ring, params = _bf(b, w), _bf(2 * heads, w), _bf(TAPS, channels), _bf(b, TAPS, channels), _rule(heads)
         at = mo.StepRows(pos, slots, sl, lines, 0, None, [])
         return lambda: mo.delta_rule(proj[:, :channels], proj[:, channels:], (h, wab), *params, state, at, heads // SHARED, 1e-6, y, conv=(filt, ring))
-    add("delta step with convolution and gates", "mlstm step", b * heads * 128 * 128 * 8, 0, rule)
+    add("delta step with convolution and gates", "mlstm step", b * heads * 128 * 128 * 8 + b * channels * 2 * (TAPS + 1), 0, rule)
     at = torch.arange(b, device="cuda") * 16
     for name, like, a in zip(("grouped_prep (Beledra)", "short_conv_attend, mixed values"), ("-", "grouped_prep"), _grouped(s)):
         m = (heads + 2 * kv) * 128
@@ -190,7 +190,8 @@ def _decode_kernels(s, t, b):
                 return lambda: mo.conv_attend(pr, filt, ring, rows, a, temp, cache, first, 0.5)
             wq, wk = (torch.ones(128, device="cuda").bfloat16() for _ in range(2))
             return lambda: mo.attention_prepare(pr, a, wq, wk, None, pos, at, cache)
-        add(name, like, b * m * 4, 0, prep)
+        # (the convolution reads its input, the rows before it and the first values, and writes the result and its row of the ring)
+        add(name, like, b * m * 4 + (b * (m * 2 * ATTENTION_TAPS + kv * 256) if a.chunked else 0), 0, prep)
     # products
 
     def plain(n, k, **kw):
