@@ -370,6 +370,7 @@ __device__ __forceinline__ void dl_split2(float x, float y, uint32_t& hi, uint32
 }
 __device__ __forceinline__ uint32_t dl_swz(int r, int c8) { return (uint32_t)r * 128u + (uint32_t)((c8 ^ (r & 7)) << 4); }
 
+constexpr int DP_HEADS = 2;                         // heads with the same keys that a CTA takes, one after the other
 struct DeltaPrepareSmem {                           // X: panels of [64 rows of K; 64 rows of Q] x 64 columns, later the image
   static constexpr int OFF_X = 0, OFF_I = 0, OFF_A = (DI_BYTES + 1023) / 1024 * 1024;
   static constexpr int PITCH = 68;                  // floats between the rows of A
@@ -402,7 +403,9 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
     tmem_relinquish();
   }
   pdl_sync();
-  const int h = blockIdx.x % p.heads, chunk = blockIdx.x / p.heads, hk = h / (p.heads / p.kv_heads), D = p.dim;
+  const int rep = p.heads / p.kv_heads, sets = (rep + DP_HEADS - 1) / DP_HEADS, set = blockIdx.x % sets;
+  const int hk = blockIdx.x / sets % p.kv_heads, chunk = blockIdx.x / (sets * p.kv_heads), D = p.dim;
+  const int h0 = hk * rep + set * DP_HEADS, heads = min(DP_HEADS, rep - set * DP_HEADS);      // heads h0 .. share these keys
   int lo = 0, hi = p.seqs;                          // the portion the chunk belongs to
   while (hi - lo > 1) {
     const int mid = (lo + hi) / 2;
@@ -422,10 +425,9 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
       tma_load_2d(smem + L::OFF_X + i * 16384 + DC_TILE, &tm, bar_l, hk * D + i * 64, row0);
     }
   }
-  // ---- decays and write strengths; tokens that are not there neither decay nor write
-  float b = 0.f;
-  if (tid < DC) {
-    float beta = 0.f;
+  // ---- decays, added up over each half of the tokens, and write strengths; tokens that are not there neither decay nor write
+  auto gates = [&](int h) {
+    float b = 0.f, beta = 0.f;
     if (tid < n) {
       const float* ab = p.ab + (long long)(row0 + tid) * p.ld_ab;
       b = delta_log_decay(ab[h] + p.dt[h], p.decay[h]) * DELTA_LOG2E;
@@ -438,7 +440,9 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
     }
     if (tid == 31) half_sum = b;
     sbeta[tid] = beta;
-  }
+    return b;
+  };
+  float b = tid < DC ? gates(h0) : 0.f;
   bool ok = mbar_wait(bar_l, 0, abort_word);
   if (!ok) *abort_word = ERR_WAIT_FULL;
   const int r = tid;                                // row of X
@@ -454,8 +458,6 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
     }
     umma_commit(bar_m);
   }
-  if (tid >= 32 && tid < DC) b += half_sum;
-  if (tid < DC) sb[tid] = b;
   ok = mbar_wait(bar_m, 0, abort_word) && ok;
   if (!ok) *abort_word = ERR_WAIT_MISC;
   tc_fence_after();
@@ -468,168 +470,180 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
     for (int i = 0; i < 32; ++i) ss = i == lane ? __uint_as_float(raw[i]) : ss;
     slen[r] = rsqrtf(ss + 1e-6f) * (r < DC ? 1.f : rsqrtf((float)D));
   }
-  __syncthreads();
   const int t = r & (DC - 1);
-  const float bt = sb[t], mine = slen[r] * (r < DC ? sbeta[t] : 1.f);
   uint8_t* image = smem + L::OFF_I;
-  const int last = r < DC ? t - 1 : t;              // A lies strictly below the diagonal
-#pragma unroll
-  for (int half = 0; half < 2; ++half) {
-    const bool any = half == 0 || (warp & 1) == 1;  // the first 32 tokens see none of the others
-    uint32_t raw[32];
-    if (any) {
-      tmem_ld_32x32(tmem + (uint32_t(warp * 32) << 16) + half * 32, raw);
-      tmem_ld_wait();
-    } else if (r < DC) {
-      continue;                                     // (that part of A is not read)
+#pragma unroll 1
+  for (int head = 0; head < heads; ++head) {
+    if (head > 0) {
+      if (tid == 0) tma_store_wait_read<0>();
+      __syncthreads();                                // the image of the head before has left
+      if (tid < DC) b = gates(h0 + head);
+      __syncthreads();
     }
+    if (tid < DC) sb[tid] = tid >= 32 ? b + half_sum : b;
+    __syncthreads();
+    const float bt = sb[t], mine = slen[r] * (r < DC ? sbeta[t] : 1.f);
+    const int last = r < DC ? t - 1 : t;              // A lies strictly below the diagonal
 #pragma unroll
-    for (int q = 0; q < 4; ++q) {
-      float f[8];
+    for (int half = 0; half < 2; ++half) {
+      const bool any = half == 0 || (warp & 1) == 1;  // the first 32 tokens see none of the others
+      uint32_t raw[32];
+      if (any) {
+        tmem_ld_32x32(tmem + (uint32_t(warp * 32) << 16) + half * 32, raw);
+        tmem_ld_wait();
+      } else if (r < DC) {
+        continue;                                     // (that part of A is not read)
+      }
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int s = half * 32 + q * 8 + j * 4;
-        float4 lens = make_float4(0.f, 0.f, 0.f, 0.f), bs = lens;
-        if (any) {
-          lens = *reinterpret_cast<const float4*>(slen + s);
-          bs = *reinterpret_cast<const float4*>(sb + s);
+      for (int q = 0; q < 4; ++q) {
+        float f[8];
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const int s = half * 32 + q * 8 + j * 4;
+          float4 lens = make_float4(0.f, 0.f, 0.f, 0.f), bs = lens;
+          if (any) {
+            lens = *reinterpret_cast<const float4*>(slen + s);
+            bs = *reinterpret_cast<const float4*>(sb + s);
+          }
+          const float l4[4] = {lens.x, lens.y, lens.z, lens.w}, b4[4] = {bs.x, bs.y, bs.z, bs.w};
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            f[j * 4 + i] = any && s + i <= last ? __uint_as_float(raw[q * 8 + j * 4 + i]) * (mine * l4[i]) * dl_exp2(fminf(bt - b4[i], 0.f)) : 0.f;
         }
-        const float l4[4] = {lens.x, lens.y, lens.z, lens.w}, b4[4] = {bs.x, bs.y, bs.z, bs.w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-          f[j * 4 + i] = any && s + i <= last ? __uint_as_float(raw[q * 8 + j * 4 + i]) * (mine * l4[i]) * dl_exp2(fminf(bt - b4[i], 0.f)) : 0.f;
-      }
-      if (r < DC) {
-        *reinterpret_cast<float4*>(at(t, half * 32 + q * 8)) = make_float4(f[0], f[1], f[2], f[3]);
-        *reinterpret_cast<float4*>(at(t, half * 32 + q * 8 + 4)) = make_float4(f[4], f[5], f[6], f[7]);
-      } else {
-        uint4 hi4, lo4;
-        dl_split2(f[0], f[1], hi4.x, lo4.x);
-        dl_split2(f[2], f[3], hi4.y, lo4.y);
-        dl_split2(f[4], f[5], hi4.z, lo4.z);
-        dl_split2(f[6], f[7], hi4.w, lo4.w);
-        *reinterpret_cast<uint4*>(image + DI_P + dl_swz(t, half * 4 + q)) = hi4;
-        *reinterpret_cast<uint4*>(image + DI_P + DC_TILE + dl_swz(t, half * 4 + q)) = lo4;
+        if (r < DC) {
+          *reinterpret_cast<float4*>(at(t, half * 32 + q * 8)) = make_float4(f[0], f[1], f[2], f[3]);
+          *reinterpret_cast<float4*>(at(t, half * 32 + q * 8 + 4)) = make_float4(f[4], f[5], f[6], f[7]);
+        } else {
+          uint4 hi4, lo4;
+          dl_split2(f[0], f[1], hi4.x, lo4.x);
+          dl_split2(f[2], f[3], hi4.y, lo4.y);
+          dl_split2(f[4], f[5], hi4.z, lo4.z);
+          dl_split2(f[6], f[7], hi4.w, lo4.w);
+          *reinterpret_cast<uint4*>(image + DI_P + dl_swz(t, half * 4 + q)) = hi4;
+          *reinterpret_cast<uint4*>(image + DI_P + DC_TILE + dl_swz(t, half * 4 + q)) = lo4;
+        }
       }
     }
-  }
-  tc_fence_before();
-  __syncthreads();
-  // ---- T from its diagonal blocks of 16 (forward substitution, a warp per block, a lane per column), then twice
-  // T21 = -T22 (A21 T11), for blocks of 16 and of 32.  Products are kept above the diagonal, where A has nothing.
-  constexpr int HB = DC / 2, QB = DC / 4;
-  {
-    const int o = warp * QB, c = lane & (QB - 1);
-    float x[QB];
+    tc_fence_before();
+    __syncthreads();
+    // ---- T from its diagonal blocks of 16 (forward substitution, a warp per block, a lane per column), then twice
+    // T21 = -T22 (A21 T11), for blocks of 16 and of 32.  Products are kept above the diagonal, where A has nothing.
+    constexpr int HB = DC / 2, QB = DC / 4;
+    {
+      const int o = warp * QB, c = lane & (QB - 1);
+      float x[QB];
 #pragma unroll
-    for (int i = 0; i < QB; ++i) {
-      float a[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int i = 0; i < QB; ++i) {
+        float a[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int s = 0; s < i; s += 4) {
-        const float4 v = *reinterpret_cast<const float4*>(at(o + i, o + s));
-        a[0] = fmaf(v.x, x[s], a[0]);
-        if (s + 1 < i) a[1] = fmaf(v.y, x[s + 1], a[1]);
-        if (s + 2 < i) a[2] = fmaf(v.z, x[s + 2], a[2]);
-        if (s + 3 < i) a[3] = fmaf(v.w, x[s + 3], a[3]);
+        for (int s = 0; s < i; s += 4) {
+          const float4 v = *reinterpret_cast<const float4*>(at(o + i, o + s));
+          a[0] = fmaf(v.x, x[s], a[0]);
+          if (s + 1 < i) a[1] = fmaf(v.y, x[s + 1], a[1]);
+          if (s + 2 < i) a[2] = fmaf(v.z, x[s + 2], a[2]);
+          if (s + 3 < i) a[3] = fmaf(v.w, x[s + 3], a[3]);
+        }
+        x[i] = (i == c ? 1.f : 0.f) - ((a[0] + a[1]) + (a[2] + a[3]));
       }
-      x[i] = (i == c ? 1.f : 0.f) - ((a[0] + a[1]) + (a[2] + a[3]));
+      __syncwarp();                                   // the block has been read
+      if (lane < QB) {
+#pragma unroll
+        for (int i = 0; i < QB; ++i) *at(o + i, o + c) = x[i];
+      }
     }
-    __syncwarp();                                   // the block has been read
-    if (lane < QB) {
-#pragma unroll
-      for (int i = 0; i < QB; ++i) *at(o + i, o + c) = x[i];
+    if (r >= DC) {
+      float* f = reinterpret_cast<float*>(image + DI_F);
+      const float end = sb[DC - 1], grown = dl_exp2(bt);
+      *reinterpret_cast<float2*>(f + 2 * t) = make_float2(sbeta[t], -sbeta[t] * grown * slen[t]);      // of v_t, of S^T k_t
+      f[2 * DC + t] = dl_exp2(end - bt) * slen[t];    // of u_t where it joins the state
+      f[3 * DC + t] = grown * slen[r];                // of S^T q_t
+      if (t == 0) f[4 * DC] = dl_exp2(end);
     }
-  }
-  if (r >= DC) {
-    float* f = reinterpret_cast<float*>(image + DI_F);
-    const float end = sb[DC - 1], grown = dl_exp2(bt);
-    *reinterpret_cast<float2*>(f + 2 * t) = make_float2(sbeta[t], -sbeta[t] * grown * slen[t]);      // of v_t, of S^T k_t
-    f[2 * DC + t] = dl_exp2(end - bt) * slen[t];    // of u_t where it joins the state
-    f[3 * DC + t] = grown * slen[r];                // of S^T q_t
-    if (t == 0) f[4 * DC] = dl_exp2(end);
-  }
-  __syncthreads();
-  {
-    // two pairs of blocks, two warps each: 8 rows of a 16 x 16 product per warp, four of them per half warp
-    const int o = (warp >> 1) * HB, c = lane & (QB - 1), i0 = (warp & 1) * 8 + (lane >> 4) * 4;
-    auto small = [&](int lr, int lc, int rr, int rc, float (&acc)[4]) __attribute__((always_inline)) {
+    __syncthreads();
+    {
+      // two pairs of blocks, two warps each: 8 rows of a 16 x 16 product per warp, four of them per half warp
+      const int o = (warp >> 1) * HB, c = lane & (QB - 1), i0 = (warp & 1) * 8 + (lane >> 4) * 4;
+      auto small = [&](int lr, int lc, int rr, int rc, float (&acc)[4]) __attribute__((always_inline)) {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) acc[i] = 0.f;
+        for (int i = 0; i < 4; ++i) acc[i] = 0.f;
 #pragma unroll
-      for (int s = 0; s < QB; s += 4) {
+        for (int s = 0; s < QB; s += 4) {
+          float v[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[j] = *at(rr + s + j, rc + c);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float4 w = *reinterpret_cast<const float4*>(at(lr + i0 + i, lc + s));
+            acc[i] = fmaf(w.x, v[0], fmaf(w.y, v[1], fmaf(w.z, v[2], fmaf(w.w, v[3], acc[i]))));
+          }
+        }
+      };
+      float acc[4];
+      small(o + QB, o, o, o, acc);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) *at(o + i0 + i, o + QB + c) = acc[i];
+      __syncthreads();
+      small(o + QB, o + QB, o, o + QB, acc);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) *at(o + QB + i0 + i, o + c) = -acc[i];
+      __syncthreads();
+#pragma unroll
+      for (int i = 0; i < 4; ++i) *at(o + i0 + i, o + QB + c) = 0.f;
+    }
+    __syncthreads();
+    // rows warp * 8 .. + 7 and column `lane` of the product of the blocks at (lr, lc) and (rr, rc)
+    auto product = [&](int lr, int lc, int rr, int rc, float (&acc)[8]) __attribute__((always_inline)) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+#pragma unroll
+      for (int s = 0; s < HB; s += 4) {
         float v[4];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) v[j] = *at(rr + s + j, rc + c);
+        for (int j = 0; j < 4; ++j) v[j] = *at(rr + s + j, rc + lane);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float4 w = *reinterpret_cast<const float4*>(at(lr + i0 + i, lc + s));
+        for (int i = 0; i < 8; ++i) {
+          const float4 w = *reinterpret_cast<const float4*>(at(lr + warp * 8 + i, lc + s));
           acc[i] = fmaf(w.x, v[0], fmaf(w.y, v[1], fmaf(w.z, v[2], fmaf(w.w, v[3], acc[i]))));
         }
       }
     };
-    float acc[4];
-    small(o + QB, o, o, o, acc);
+    float acc[8];
+    product(HB, 0, 0, 0, acc);               // A21 T11, kept above the diagonal
 #pragma unroll
-    for (int i = 0; i < 4; ++i) *at(o + i0 + i, o + QB + c) = acc[i];
+    for (int i = 0; i < 8; ++i) *at(warp * 8 + i, HB + lane) = acc[i];
     __syncthreads();
-    small(o + QB, o + QB, o, o + QB, acc);
+    product(HB, HB, 0, HB, acc);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) *at(o + QB + i0 + i, o + c) = -acc[i];
+    for (int i = 0; i < 8; ++i) *at(HB + warp * 8 + i, lane) = -acc[i];
     __syncthreads();
+    {
+      const int row = r >> 1, half = r & 1;
+      const bool zero = row < HB && half == 1;        // above the diagonal
+      float4 u[8];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) *at(o + i0 + i, o + QB + c) = 0.f;
-  }
-  __syncthreads();
-  // rows warp * 8 .. + 7 and column `lane` of the product of the blocks at (lr, lc) and (rr, rc)
-  auto product = [&](int lr, int lc, int rr, int rc, float (&acc)[8]) __attribute__((always_inline)) {
+      for (int q = 0; q < 8; ++q) u[q] = zero ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(at(row, half * 32 + q * 4));
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i] = 0.f;
-#pragma unroll
-    for (int s = 0; s < HB; s += 4) {
-      float v[4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) v[j] = *at(rr + s + j, rc + lane);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const float4 w = *reinterpret_cast<const float4*>(at(lr + warp * 8 + i, lc + s));
-        acc[i] = fmaf(w.x, v[0], fmaf(w.y, v[1], fmaf(w.z, v[2], fmaf(w.w, v[3], acc[i]))));
+      for (int q = 0; q < 4; ++q) {
+        uint4 hi4, lo4;
+        dl_split2(u[2 * q].x, u[2 * q].y, hi4.x, lo4.x);
+        dl_split2(u[2 * q].z, u[2 * q].w, hi4.y, lo4.y);
+        dl_split2(u[2 * q + 1].x, u[2 * q + 1].y, hi4.z, lo4.z);
+        dl_split2(u[2 * q + 1].z, u[2 * q + 1].w, hi4.w, lo4.w);
+        *reinterpret_cast<uint4*>(image + DI_T + dl_swz(row, half * 4 + q)) = hi4;
+        *reinterpret_cast<uint4*>(image + DI_T + DC_TILE + dl_swz(row, half * 4 + q)) = lo4;
       }
     }
-  };
-  float acc[8];
-  product(HB, 0, 0, 0, acc);               // A21 T11, kept above the diagonal
-#pragma unroll
-  for (int i = 0; i < 8; ++i) *at(warp * 8 + i, HB + lane) = acc[i];
-  __syncthreads();
-  product(HB, HB, 0, HB, acc);
-#pragma unroll
-  for (int i = 0; i < 8; ++i) *at(HB + warp * 8 + i, lane) = -acc[i];
-  __syncthreads();
-  {
-    const int row = r >> 1, half = r & 1;
-    const bool zero = row < HB && half == 1;        // above the diagonal
-    float4 u[8];
-#pragma unroll
-    for (int q = 0; q < 8; ++q) u[q] = zero ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(at(row, half * 32 + q * 4));
-#pragma unroll
-    for (int q = 0; q < 4; ++q) {
-      uint4 hi4, lo4;
-      dl_split2(u[2 * q].x, u[2 * q].y, hi4.x, lo4.x);
-      dl_split2(u[2 * q].z, u[2 * q].w, hi4.y, lo4.y);
-      dl_split2(u[2 * q + 1].x, u[2 * q + 1].y, hi4.z, lo4.z);
-      dl_split2(u[2 * q + 1].z, u[2 * q + 1].w, hi4.w, lo4.w);
-      *reinterpret_cast<uint4*>(image + DI_T + dl_swz(row, half * 4 + q)) = hi4;
-      *reinterpret_cast<uint4*>(image + DI_T + DC_TILE + dl_swz(row, half * 4 + q)) = lo4;
+    fence_proxy_async_smem();
+    __syncthreads();
+    if (tid == 0) {
+      uint8_t* to = reinterpret_cast<uint8_t*>(p.image) + ((long long)chunk * p.heads + h0 + head) * DI_BYTES;
+      asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(reinterpret_cast<uint64_t>(to)), "r"(smem_u32(image)),
+                   "r"((uint32_t)DI_BYTES)
+                   : "memory");
+      tma_store_commit();
     }
   }
-  fence_proxy_async_smem();
-  __syncthreads();
   if (tid == 0) {
-    uint8_t* to = reinterpret_cast<uint8_t*>(p.image) + ((long long)chunk * p.heads + h) * DI_BYTES;
-    asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(reinterpret_cast<uint64_t>(to)), "r"(smem_u32(image)),
-                 "r"((uint32_t)DI_BYTES)
-                 : "memory");
-    tma_store_commit();
     tma_store_wait<0>();
     if (*abort_word != 0 && p.status != nullptr) atomicCAS(p.status, 0u, (*abort_word) | (blockIdx.x << 8));
   }
@@ -1005,7 +1019,8 @@ static int launch_delta_chunk(const CUtensorMap& tm, const CUtensorMap& tm_gate,
       return -3;
     configured = true;
   }
-  launch_dep(delta_prepare_kernel, (unsigned)(p.chunks * p.heads), 128, DeltaPrepareSmem::TOTAL, st, tm, p);
+  const int sets = (p.heads / p.kv_heads + DP_HEADS - 1) / DP_HEADS;
+  launch_dep(delta_prepare_kernel, (unsigned)(p.chunks * p.kv_heads * sets), 128, DeltaPrepareSmem::TOTAL, st, tm, p);
   launch_dep(kern, (unsigned)(p.seqs * p.heads), DK_THREADS, DeltaChunkSmem<PD, PE>::TOTAL, st, tm, tm_gate, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
