@@ -335,7 +335,7 @@ def state_of(before, spans, slots, n):
     return state
 
 
-SIZES = [(4, 2, 64, 64), (3, 1, 40, 72), (2, 2, 128, 128), (2, 1, 104, 24), (4, 4, 8, 128), (6, 3, 24, 8), (2, 1, 72, 40)]
+SIZES = [(6, 2, 64, 64), (3, 1, 40, 72), (2, 2, 128, 128), (2, 1, 104, 24), (4, 4, 8, 128), (6, 3, 24, 8), (2, 1, 72, 40)]
 
 
 @pytest.mark.parametrize("heads,kv,dim,vdim", SIZES)
@@ -356,7 +356,7 @@ def test_chunked_delta_rule(heads, kv, dim, vdim, keys, decay):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("heads,kv,dim,vdim", [(4, 2, 64, 64), (3, 3, 10, 7), (2, 1, 13, 12), (1, 1, 200, 144), (2, 1, 256, 130)])
+@pytest.mark.parametrize("heads,kv,dim,vdim", [(6, 2, 64, 64), (3, 3, 10, 7), (2, 1, 13, 12), (1, 1, 200, 144), (2, 1, 256, 130)])
 def test_general_delta_rule(dtype, heads, kv, dim, vdim):
     mo = mops()
     spans, slots = [(0, 1), (0, 20), (5, 2), (30, 9)], [3, 0, 4, 1]
@@ -372,7 +372,7 @@ def test_general_delta_rule(dtype, heads, kv, dim, vdim):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("heads,kv,dim,vdim,taps", [(4, 2, 64, 64, 4), (2, 2, 128, 128, 3), (6, 2, 24, 8, 1), (3, 1, 13, 12, 5), (2, 1, 64, 256, 2), (3, 3, 64, 16, 4)])
+@pytest.mark.parametrize("heads,kv,dim,vdim,taps", [(6, 2, 64, 64, 4), (2, 2, 128, 128, 3), (6, 2, 24, 8, 1), (3, 1, 13, 12, 5), (2, 1, 64, 256, 2), (3, 3, 64, 16, 4)])
 @pytest.mark.parametrize("fused", [False, True])
 def test_delta_decode_step(dtype, heads, kv, dim, vdim, taps, fused):
     """One token of some requests, at their first, second and later positions; with the gates' products and the convolution in the kernel, or
