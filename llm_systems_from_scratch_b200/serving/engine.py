@@ -15,6 +15,7 @@ whether that is a prompt, a decode step or - ``extend``, for callers that bring 
 """
 from __future__ import annotations
 
+import gc
 import time
 
 import numpy as np
@@ -167,8 +168,16 @@ class ServingEngine:
         torch.cuda.current_stream().wait_stream(side)
         torch.cuda.synchronize()
         graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(graph):
-            run()
+        # an engine that is no longer used would take its graphs with it when the collector finds it, which a capture does not survive
+        gc.collect()
+        collects = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.graph(graph):
+                run()
+        finally:
+            if collects:
+                gc.enable()
         for k, v in keep.items():
             d[k][:n].copy_(v)
         return graph
