@@ -647,6 +647,13 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const __grid_constan
     tma_store_wait<0>();
     if (*abort_word != 0 && p.status != nullptr) atomicCAS(p.status, 0u, (*abort_word) | (blockIdx.x << 8));
   }
+  tc_fence_before();
+  __syncthreads();
+  if (*abort_word != 0) {                           // give copies that may still be in flight time to land
+    const uint64_t w0 = globaltimer_ns();
+    while (globaltimer_ns() - w0 < 200000ull) __nanosleep(1000);
+    __syncthreads();
+  }
   if (warp == 0) {
     tc_fence_after();
     tmem_dealloc(tmem, 128);
